@@ -29,7 +29,8 @@ NVCC_FLAGS = [
 ]
 #: translation units whose arithmetic feeds the optimiser state or the loss: compiled without
 #: --use_fast_math (IEEE division and square root in the AdamW update, exact exp/log in the CE)
-EXACT_MATH = {"adamw.cu", "rs_adamw.cu", "ce.cu"}
+#: (the hybrid decoder's norms, recurrence and fp32 path: what is computed in 32-bit keeps its 32 bits)
+EXACT_MATH = {"adamw.cu", "rs_adamw.cu", "ce.cu", "hybrid_rows.cu", "mamba2.cu", "attn_rows.cu", "sgemm.cu"}
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread", "-march=x86-64-v3"]
 
 
@@ -62,7 +63,10 @@ def _run(cmd: list[str], log: Path | None = None) -> None:
 
 
 def build_cuda(force: bool = False, verbose: bool = False) -> Path:
-    srcs = sorted(CSRC.rglob("*.cu"))
+    return _build_cuda(sorted(CSRC.rglob("*.cu")), CUDA_LIB, force, verbose)
+
+
+def _build_cuda(srcs, lib: Path, force: bool = False, verbose: bool = False) -> Path:
     OBJDIR.mkdir(parents=True, exist_ok=True)
     LIBDIR.mkdir(parents=True, exist_ok=True)
     hdr = _newest_header()
@@ -89,15 +93,19 @@ def build_cuda(force: bool = False, verbose: bool = False) -> Path:
     if jobs:
         with ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 4)) as ex:
             list(ex.map(compile_one, jobs))
-    if jobs or not CUDA_LIB.exists():
-        _run([nvcc, "-shared", "-o", str(CUDA_LIB), *map(str, objs), "-lcudart"])
-    return CUDA_LIB
+    if jobs or not lib.exists() or any(o.stat().st_mtime > lib.stat().st_mtime for o in objs):
+        # linked beside its place and moved there, so a library that another process has open stays whole
+        tmp = lib.with_suffix(f".{os.getpid()}.tmp")
+        _run([nvcc, "-shared", "-o", str(tmp), *map(str, objs), "-lcudart"])
+        os.replace(tmp, lib)
+    return lib
 
 
 def build_host(force: bool = False, verbose: bool = False) -> Path:
-    srcs = sorted(CSRC.rglob("*.cpp"))
-    if not srcs:
-        return HOST_LIB
+    return _build_host(sorted(CSRC.rglob("*.cpp")), HOST_LIB, force, verbose)
+
+
+def _build_host(srcs, lib: Path, force: bool = False, verbose: bool = False) -> Path:
     OBJDIR.mkdir(parents=True, exist_ok=True)
     LIBDIR.mkdir(parents=True, exist_ok=True)
     hdr = _newest_header()
@@ -118,9 +126,11 @@ def build_host(force: bool = False, verbose: bool = False) -> Path:
     if jobs:
         with ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 4)) as ex:
             list(ex.map(compile_one, jobs))
-    if jobs or not HOST_LIB.exists():
-        _run([cxx, "-shared", "-o", str(HOST_LIB), *map(str, objs), "-pthread"])
-    return HOST_LIB
+    if jobs or not lib.exists() or any(o.stat().st_mtime > lib.stat().st_mtime for o in objs):
+        tmp = lib.with_suffix(f".{os.getpid()}.tmp")
+        _run([cxx, "-shared", "-o", str(tmp), *map(str, objs), "-pthread"])
+        os.replace(tmp, lib)
+    return lib
 
 
 #: translation units of the bounds-checking library (kernels whose addresses depend on data) and
@@ -153,6 +163,33 @@ def build_bounds(force: bool = False, verbose: bool = False) -> Path:
     if jobs or not BOUNDS_LIB.exists():
         _run([nvcc, "-shared", "-o", str(BOUNDS_LIB), *map(str, objs), "-lcudart"])
     return BOUNDS_LIB
+
+
+#: what serving a hybrid decoder needs of the kernel library, for programs that compile on first use
+HYBRID_TUS = ["common/host.cu", "kernels/attn_rows.cu", "kernels/flash_fwd.cu", "kernels/gemm_2cta.cu",
+              "kernels/gemm_tcgen05.cu", "kernels/hybrid_rows.cu", "kernels/mamba2.cu", "kernels/paged_kv.cu",
+              "kernels/router_quant_sample.cu", "kernels/sgemm.cu", "serve/hybrid_forward.cu"]
+HYBRID_LIB = LIBDIR / "libbrain_b200_hybrid.so"
+#: ... and of the host runtime (checkpoint reader, pages, slots, scheduler)
+HYBRID_HOST_SRCS = ["runtime/data.cpp", "runtime/safetensors.cpp", "runtime/serving.cpp"]
+HYBRID_HOST_LIB = LIBDIR / "libbrain_host_hybrid.so"
+
+
+def build_hybrid(verbose: bool = False) -> Path:
+    """The kernel library reduced to :data:`HYBRID_TUS` (objects are shared with the full build)."""
+    return _build_cuda([CSRC / t for t in HYBRID_TUS], HYBRID_LIB, verbose=verbose)
+
+
+def build_hybrid_host(verbose: bool = False) -> Path:
+    return _build_host([CSRC / t for t in HYBRID_HOST_SRCS], HYBRID_HOST_LIB, verbose=verbose)
+
+
+def library_current(lib: Path, suffix: str) -> bool:
+    """The library exists and is newer than every source file with that suffix and every header."""
+    if not lib.exists():
+        return False
+    m = lib.stat().st_mtime
+    return _newest_header() <= m and all(s.stat().st_mtime <= m for s in CSRC.rglob("*" + suffix))
 
 
 def build_all(force: bool = False, verbose: bool = False) -> None:

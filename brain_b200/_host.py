@@ -42,6 +42,17 @@ def _apply(lib, sigs):
         fn.argtypes = args
 
 
+def use_hybrid_library() -> None:
+    """For a program that only serves hybrid decoders and compiles on first use: take the full host
+    runtime when it is built and current, else build and take the part such a program needs."""
+    global _LIB
+    from . import _build
+    if _LIB is None and not _build.library_current(_PATH, ".cpp"):
+        lib_ = ctypes.CDLL(str(_build.build_hybrid_host()))
+        _apply(lib_, _SIGS)
+        _LIB = lib_
+
+
 def lib() -> ctypes.CDLL:
     global _LIB
     if _LIB is None:

@@ -220,9 +220,17 @@ def save_model(path: str, model, card: Optional[ModelCard] = None, dtype: str = 
 
 
 def load_model(path: str, device="cpu", dtype=None):
-    """Rebuild the model a checkpoint describes (its config wins) and load the weights."""
+    """Rebuild the model a checkpoint describes (its config wins) and load the weights.  ``path``: a
+    safetensors file that carries its configuration, or a directory with ``config.json`` and
+    ``model.safetensors``."""
+    import os
     from ..models import build_from_config
-    tensors, config, card = load(path)
+    if os.path.isdir(path):
+        with open(os.path.join(path, "config.json")) as f:
+            config = json.load(f)
+        tensors, _, card = load(os.path.join(path, "model.safetensors"))
+    else:
+        tensors, config, card = load(path)
     if config is None:
         raise ValueError(f"{path}: no brain.config metadata")
     model = build_from_config(config)

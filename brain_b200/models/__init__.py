@@ -1,5 +1,5 @@
-"""Model families: GPT-2, dense Qwen3/Qwen2, sparse MoE (toy and Qwen3-MoE)."""
-from .config import GptConfig, LoraCfg, MoeConfig, QwenConfig, config_from_json
+"""Model families: GPT-2, dense Qwen3/Qwen2, sparse MoE (toy and Qwen3-MoE), hybrid decoders (Pakalix)."""
+from .config import GptConfig, HybridConfig, LoraCfg, MoeConfig, QwenConfig, config_from_json
 
 
 def build_from_config(cfg):
@@ -12,6 +12,9 @@ def build_from_config(cfg):
     if isinstance(cfg, MoeConfig):
         from .moe import MoeModel
         return MoeModel(cfg)
+    if isinstance(cfg, HybridConfig):
+        from .hybrid import HybridDecoder
+        return HybridDecoder(cfg)
     from .qwen3 import Qwen3
     m = Qwen3(cfg)
     if cfg.lora is not None:

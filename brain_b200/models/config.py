@@ -301,10 +301,207 @@ class MoeConfig:
         return sum(n for _, n in self.param_list())
 
 
+# ------------------------------------------------------------------------------------ hybrid decoders
+# A decoder described layer by layer: every layer names its mixer (attention or a state-space
+# recurrence) with sizes of its own, and its feed-forward.  The records below are mechanisms with their
+# constants as fields; a design is a reader of its config file (``HYBRID_DESIGNS``) that fills them in.
+
+@dataclass
+class RotarySpec:
+    dims: int                    # leading dimensions of a head that are rotated, half-split pairs
+    base: float
+
+
+@dataclass
+class AttentionSpec:
+    heads: int
+    kv_heads: int
+    dim: int                     # query / key head size
+    vdim: int                    # value head size
+    scale: float
+    softcap: Optional[float] = None
+    rot: Optional[RotarySpec] = None
+    v_mix: bool = False          # values mixed with those of the first layer that has this set
+    kind = "attention"
+
+    def check(self):
+        if self.heads % self.kv_heads:
+            raise ValueError(f"attention: {self.heads} heads over {self.kv_heads} key/value heads")
+        if self.rot is not None and (self.rot.dims % 2 or self.rot.dims > self.dim):
+            raise ValueError(f"attention: cannot rotate {self.rot.dims} of {self.dim} dimensions")
+
+    def tensors(self, width: int):
+        out = [("q", (self.heads * self.dim, width)), ("k", (self.kv_heads * self.dim, width)),
+               ("v", (self.kv_heads * self.vdim, width)), ("q.norm", (self.heads * self.dim,)),
+               ("k.norm", (self.kv_heads * self.dim,))]
+        if self.v_mix:
+            out.append(("vmix", ()))
+        return out + [("g", (self.heads, width)), ("o", (width, self.heads * self.vdim))]
+
+
+@dataclass
+class Mamba2Spec:
+    heads: int
+    vdim: int                    # channels of a head
+    state: int
+    groups: int                  # heads of a group share B and C
+    conv: int                    # taps of the short convolution
+    norm_groups: int
+    kind = "mamba2"
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def channels(self) -> int:
+        return self.inner + 2 * self.groups * self.state
+
+    def check(self):
+        if self.heads % self.groups:
+            raise ValueError(f"mamba2: {self.heads} heads over {self.groups} groups")
+        if self.inner % self.norm_groups:
+            raise ValueError(f"mamba2: {self.inner} channels in {self.norm_groups} norm groups")
+        if self.conv < 1:
+            raise ValueError("mamba2: the convolution needs at least one tap")
+
+    def tensors(self, width: int):
+        return [("in", (self.inner + self.channels + self.heads, width)), ("conv", (self.channels, self.conv)),
+                ("conv.b", (self.channels,)), ("dt_bias", (self.heads,)), ("A_log", (self.heads,)),
+                ("D", (self.heads,)), ("norm", (self.inner,)), ("o", (width, self.inner))]
+
+
+@dataclass
+class ClampedGluSpec:
+    """min(g, limit) sigmoid(alpha g) (clamp(u) + shift) between the gate / up and down projections."""
+    ff: int
+    limit: float
+    alpha: float = 1.702
+    shift: float = 1.0
+
+    def tensors(self, width: int):
+        return [("gate", (self.ff, width)), ("up", (self.ff, width)), ("down", (width, self.ff))]
+
+
+@dataclass
+class HybridLayer:
+    mixer: object                # AttentionSpec | Mamba2Spec
+    mlp: Optional[ClampedGluSpec] = None
+
+
+@dataclass
+class HybridConfig:
+    vocab: int
+    width: int
+    layers: List[HybridLayer]
+    eps: float
+    residual_mult: float = 1.0
+    design: str = "Pakalix"
+    #: positions are not limited by the design; this is what a server may reserve pages for
+    max_position_embeddings: int = 131072
+
+    def __post_init__(self):
+        if not self.layers:
+            raise ValueError("a hybrid decoder needs at least one layer")
+        vals = set()
+        for l in self.layers:
+            l.mixer.check()
+            if l.mixer.kind == "attention" and l.mixer.v_mix:
+                vals.add((l.mixer.kv_heads, l.mixer.vdim))
+        if len(vals) > 1:
+            raise ValueError(f"layers that mix values differ in their value sizes: {sorted(vals)}")
+
+    @property
+    def n_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def d_model(self) -> int:
+        return self.width
+
+    @property
+    def block_size(self) -> int:
+        return self.max_position_embeddings
+
+    @property
+    def recurrent(self) -> bool:
+        return any(l.mixer.kind != "attention" for l in self.layers)
+
+    # ---- JSON: the design's own config file
+    def to_json(self) -> dict:
+        layers = []
+        for l in self.layers:
+            m = asdict(l.mixer)
+            if l.mixer.kind == "attention":
+                for k in ("softcap", "rot"):
+                    if m[k] is None:
+                        del m[k]
+            layers.append({"type": l.mixer.kind, "mixer": m,
+                           "mlp": None if l.mlp is None else {"kind": "dense", "ff": l.mlp.ff, "limit": l.mlp.limit}})
+        return {"architecture": self.design, "vocab": self.vocab, "width": self.width, "layers": layers,
+                "norm": {"eps": self.eps}, "residual_mult": self.residual_mult}
+
+    @staticmethod
+    def from_json(c: dict) -> "HybridConfig":
+        layers = []
+        for i, e in enumerate(c["layers"]):
+            m = dict(e["mixer"])
+            if e["type"] == "attention":
+                rot = m.get("rot")
+                mixer = AttentionSpec(
+                    heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                    scale=float(m["scale"]), softcap=float(m["softcap"]) if m.get("softcap") else None,
+                    rot=RotarySpec(int(rot["dims"]), float(rot["base"])) if rot else None,
+                    v_mix=bool(m.get("v_mix", False)))
+            elif e["type"] == "mamba2":
+                mixer = Mamba2Spec(heads=int(m["heads"]), vdim=int(m["vdim"]), state=int(m["state"]),
+                                   groups=int(m["groups"]), conv=int(m["conv"]), norm_groups=int(m["norm_groups"]))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
+            f = e.get("mlp")
+            if f is not None and f.get("kind", "dense") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward {f['kind']!r}")
+            layers.append(HybridLayer(mixer, None if f is None else ClampedGluSpec(int(f["ff"]), float(f["limit"]))))
+        return HybridConfig(vocab=int(c["vocab"]), width=int(c["width"]), layers=layers, eps=float(c["norm"]["eps"]),
+                            residual_mult=float(c.get("residual_mult", 1.0)), design=c["architecture"])
+
+    def tensors(self):
+        """(name, shape) of every tensor of a checkpoint, in order."""
+        d = self.width
+        out = [("embed", (self.vocab, d)), ("embed.norm", (d,))]
+        for i, l in enumerate(self.layers):
+            out.append((f"l{i}.norm1", (d,)))
+            out += [(f"l{i}.mix.{n}", s) for n, s in l.mixer.tensors(d)]
+            if l.mlp is not None:
+                out += [(f"l{i}.mlp.{n}", s) for n, s in l.mlp.tensors(d)]
+        return out + [("final.norm", (d,)), ("head", (self.vocab, d))]
+
+    def param_list(self):
+        out = []
+        for n, s in self.tensors():
+            k = 1
+            for x in s:
+                k *= x
+            out.append((n, k))
+        return out
+
+    def param_count(self) -> int:
+        return sum(n for _, n in self.param_list())
+
+
+#: architecture name of a config file -> reader of its configuration
+HYBRID_DESIGNS = {"Pakalix": HybridConfig.from_json}
+
+
 def config_from_json(c) -> object:
     """Rebuild the right config record from a checkpoint's ``brain.config`` JSON."""
     if isinstance(c, str):
         c = json.loads(c)
+    design = c.get("architecture")
+    if design is not None:
+        if design not in HYBRID_DESIGNS:
+            raise ValueError(f"unknown architecture {design!r}; have {sorted(HYBRID_DESIGNS)}")
+        return HYBRID_DESIGNS[design](c)
     kind = c.get("model", "qwen")
     if kind == "gpt":
         return GptConfig.from_json(c)

@@ -1,0 +1,103 @@
+"""Hybrid decoders (Pakalix): a parallel mixer + feed-forward per layer, the mixer being soft-capped
+attention with rotary positions, whole-projection query / key norms, value mixing and per-head output
+gates, or a Mamba-2 state-space recurrence.
+
+This is the weight container of the family (names, shapes, initial values, loading); its forward lives in
+the serving engine (``serve.hybrid.HybridEngine`` over ``csrc/serve/hybrid_forward.cu``)."""
+from __future__ import annotations
+
+import math
+from typing import Dict
+
+import torch
+import torch.nn as nn
+
+from .config import HybridConfig
+
+
+class HybridDecoder(nn.Module):
+    family = "hybrid"
+
+    def __init__(self, cfg: HybridConfig):
+        super().__init__()
+        self.cfg = cfg
+        self._names = {}
+        for name, shape in cfg.tensors():
+            attr = name.replace(".", "__")
+            self.register_parameter(attr, nn.Parameter(torch.zeros(shape), requires_grad=False))
+            self._names[name] = attr
+
+    def tensor(self, name: str) -> torch.Tensor:
+        return getattr(self, self._names[name])
+
+    @torch.no_grad()
+    def init_weights(self, seed: int = 1234) -> "HybridDecoder":
+        """Random values at which every mechanism works in its usual range: projections that keep the
+        scale of their input, norm gains near their neutral value, step sizes between 1e-3 and 1e-1, decay
+        rates between 1 and 16."""
+        g = torch.Generator().manual_seed(seed)
+
+        def uniform(shape, lo, hi):
+            return torch.rand(shape, generator=g) * (hi - lo) + lo
+
+        for name, shape in self.cfg.tensors():
+            p = self.tensor(name)
+            leaf = name.split(".", 2)[-1] if name[0] == "l" and name[1].isdigit() else name
+            if leaf in ("embed.norm", "final.norm", "norm1") or name.endswith(".norm1"):
+                v = 0.1 * torch.randn(shape, generator=g)
+            elif leaf in ("q.norm", "k.norm", "norm"):
+                v = 1.0 + 0.1 * torch.randn(shape, generator=g)
+            elif leaf == "vmix":
+                v = uniform(shape, 0.2, 0.6)
+            elif leaf == "dt_bias":
+                dt = torch.exp(uniform(shape, math.log(1e-3), math.log(1e-1)))
+                v = dt + torch.log(-torch.expm1(-dt))          # inverse of softplus
+            elif leaf == "A_log":
+                v = torch.log(uniform(shape, 1.0, 16.0))
+            elif leaf == "D":
+                v = uniform(shape, 0.5, 1.5)
+            elif leaf == "conv":
+                v = uniform(shape, -1.0, 1.0) / math.sqrt(shape[1])
+            elif leaf == "conv.b":
+                v = uniform(shape, -0.1, 0.1)
+            elif name == "embed":
+                v = torch.randn(shape, generator=g)
+            else:
+                v = torch.randn(shape, generator=g) / math.sqrt(shape[1])
+            p.copy_(v.to(p.dtype))
+        return self
+
+    # ---- checkpoint surface shared by the model families
+    def reference_state(self) -> Dict[str, torch.Tensor]:
+        return {n: self.tensor(n) for n, _ in self.cfg.tensors()}
+
+    @torch.no_grad()
+    def load_reference_state(self, state: Dict[str, torch.Tensor], strict: bool = True):
+        mine = self.reference_state()
+        missing = [n for n in mine if n not in state]
+        for n, dst in mine.items():
+            if n in missing:
+                continue
+            if state[n].numel() != dst.numel():
+                raise ValueError(f"{n}: checkpoint has {tuple(state[n].shape)}, the configuration asks for {tuple(dst.shape)}")
+            dst.copy_(state[n].reshape(dst.shape).to(dst.dtype))
+        if strict and missing:
+            raise KeyError(f"checkpoint is missing {len(missing)} tensors, e.g. {missing[:4]}")
+        return missing
+
+    def config_json(self) -> dict:
+        return self.cfg.to_json()
+
+    def flops_per_token(self, T: int, train: bool = False) -> float:
+        """Matrix-product FLOPs of one token with T tokens of context, attention and recurrence included."""
+        total = 0.0
+        for n, s in self.cfg.tensors():
+            if len(s) == 2 and n != "embed" and not n.endswith(".conv"):
+                total += 2.0 * s[0] * s[1]
+        for l in self.cfg.layers:
+            m = l.mixer
+            if m.kind == "attention":
+                total += 2.0 * m.heads * (m.dim + m.vdim) * T
+            else:
+                total += 6.0 * m.heads * m.state * m.vdim
+        return total

@@ -45,6 +45,15 @@ def lib() -> ctypes.CDLL:
     return _LIB
 
 
+def use_hybrid_library() -> None:
+    """For a program that only serves hybrid decoders and compiles on first use: take the full kernel
+    library when it is built and current, else build and take the part such a model needs."""
+    global _LIB
+    from .. import _build
+    if _LIB is None and not _build.library_current(_build.CUDA_LIB, ".cu"):
+        _LIB = ctypes.CDLL(str(_build.build_hybrid()))
+
+
 def available() -> bool:
     """True when the kernels can run: library present (or buildable) and a CUDA device visible."""
     return torch.cuda.is_available()

@@ -533,12 +533,12 @@ def quant_rows(x):
 
 
 def argmax_rows(logits):
-    """Greedy head: int32 argmax per row of bf16 logits (lowest index on ties)."""
+    """Greedy head: int32 argmax per row of bf16 or fp32 logits (lowest index on ties)."""
     if not logits.is_cuda:
         return logits.float().argmax(dim=-1).to(torch.int32)
     lg = logits.reshape(-1, logits.shape[-1])
     out = torch.empty(lg.shape[0], device=lg.device, dtype=torch.int32)
-    call("argmax_rows", lg, L(lg.stride(0)), lg.shape[0], lg.shape[1], out, stream_ptr())
+    call("argmax_rows_f32" if lg.dtype == torch.float32 else "argmax_rows", lg, L(lg.stride(0)), lg.shape[0], lg.shape[1], out, stream_ptr())
     return out
 
 
@@ -546,12 +546,12 @@ def topk_rows(logits, k: int):
     """The k largest logits of every row, descending (lowest index first among equals):
     (int32 indices [rows, k], fp32 values [rows, k])."""
     lg = logits.reshape(-1, logits.shape[-1])
-    if not lg.is_cuda or lg.dtype != torch.bfloat16:
+    if not lg.is_cuda or lg.dtype not in (torch.bfloat16, torch.float32):
         vals, idx = torch.topk(lg.float(), k, dim=-1)
         return idx.to(torch.int32), vals
     idx = torch.empty(lg.shape[0], k, device=lg.device, dtype=torch.int32)
     vals = torch.empty(lg.shape[0], k, device=lg.device, dtype=torch.float32)
-    call("topk_rows", lg, L(lg.stride(0)), lg.shape[0], lg.shape[1], int(k), idx, vals, stream_ptr())
+    call("topk_rows_f32" if lg.dtype == torch.float32 else "topk_rows", lg, L(lg.stride(0)), lg.shape[0], lg.shape[1], int(k), idx, vals, stream_ptr())
     return idx, vals
 
 

@@ -37,6 +37,7 @@ from ..ops import reference as ref
 from ..ops import _cuda
 from ..ops._cuda import L, call, stream_ptr
 from ..ops.attention import flash_attention, flash_attention_into
+from .base import PagedEngineBase
 
 
 class _Lin:
@@ -101,7 +102,7 @@ class _Lin:
         return self.w.numel() * self.w.element_size()
 
 
-class QwenEngine:
+class QwenEngine(PagedEngineBase):
     def __init__(self, model, block_size: int = 16, num_blocks: int = 1024, max_seq_len: int = 4096,
                  max_prefill: int = 512, weights: str = "bf16", topk: int = 64, tp=None,
                  decode_splits: int = 0, cuda_graphs: bool = True, kv_dtype: str = "bf16",
@@ -181,13 +182,7 @@ class QwenEngine:
                 self.kv_clip = [torch.stack([kc_[li, lo:hi], vc_[li, lo:hi]]).float().contiguous().to(dev)
                                 for li in range(len(model.blocks))]
         self.decode_splits = decode_splits
-        self.steps = 0
-        self.cuda_graphs = bool(cuda_graphs) and self.cuda
-        #: host-side fault-injection point: called with "prefill" / "decode" before the device work
-        #: of that call is issued; raising from it models a failed launch without touching the GPU
-        self.fault_hook = None
-        self._graphs = {}
-        self.graph_replays = 0
+        self._init_common(cuda_graphs)
         #: the layer sequence issued by one native call per layer half / per decode step instead of
         #: one Python wrapper per kernel (CUDA only; same kernels, same results)
         self.native = None
@@ -199,10 +194,6 @@ class QwenEngine:
                 (getattr(self.tp, "impl", "") == "fused" and cfg.d_model % (8 * self.tp_world) == 0)
             if tp_ok and NativeForward.supported(self):
                 self.native = NativeForward(self)
-        #: host wall time spent inside prefill / decode calls (each ends with a device-to-host read,
-        #: so it covers the device work) and what they processed; a serving run reports the split
-        self.acct = {"prefill_s": 0.0, "prefill_calls": 0, "prefill_tokens": 0, "prefill_seqs": 0,
-                     "decode_s": 0.0, "decode_calls": 0, "decode_rows": 0, "mixed_s": 0.0, "mixed_calls": 0}
 
     # ------------------------------------------------------------------ accounting
     def kv_pool_bytes(self) -> int:
@@ -210,9 +201,6 @@ class QwenEngine:
         if self.kv_int8:
             n += sum(t.numel() * 4 for t in self.ks) * 2
         return n
-
-    def kv_pool_capacity_tokens(self) -> int:
-        return self.num_blocks * self.block_size
 
     def weight_bytes(self) -> int:
         n = self.tok.numel() * self.tok.element_size()
@@ -469,12 +457,6 @@ class QwenEngine:
 
     # ------------------------------------------------------------------ PagedDecoder interface
     @torch.no_grad()
-    def check_device(self) -> None:
-        """Raise if a kernel of the step just read back reported a bounded-wait timeout (the
-        scheduler calls this once per step, after the token read-back, before it commits)."""
-        if self.device.type == "cuda":
-            _cuda.check_error()
-
     def prefill_chunk(self, tokens: np.ndarray, start: int, block_table: np.ndarray, last: bool,
                       greedy: bool = True):
         """Process prompt positions [start, start+n) of one sequence.  Returns (first token, top-k
@@ -657,41 +639,7 @@ class QwenEngine:
         a["decode_rows"] += B
         return results, [[int(p)] for p in picked[nf:]], (cands[nf:] if cands is not None else None)
 
-    @torch.no_grad()
-    def decode(self, tokens: np.ndarray, positions: np.ndarray, block_tables: np.ndarray,
-               window: int = 1, greedy: bool = True):
-        """One batched decode call: ``window`` on-device greedy steps (window > 1 requires greedy).
-        Returns (tokens [B][window], per-row top-k candidate lists or None)."""
-        if self.fault_hook is not None:
-            self.fault_hook("decode")
-        dev = self.device
-        B = int(tokens.shape[0])
-        t0 = time.perf_counter()
-        try:
-            return self._decode(tokens, positions, block_tables, window, greedy)
-        finally:
-            a = self.acct
-            a["decode_s"] += time.perf_counter() - t0
-            a["decode_calls"] += 1
-            a["decode_rows"] += B * window
-
-    def _decode(self, tokens, positions, block_tables, window, greedy):
-        dev = self.device
-        if self.cuda_graphs and (greedy or window > 1):
-            out = self._decode_graphed(tokens, positions, block_tables, window)
-            return [row.tolist() for row in out], None
-        tok = torch.from_numpy(np.ascontiguousarray(tokens)).to(dev)
-        pos = torch.from_numpy(np.ascontiguousarray(positions)).to(dev)
-        bts = torch.from_numpy(np.ascontiguousarray(block_tables)).to(dev)
-        out_t, topks = self._decode_steps(tok, pos, bts, window, greedy or window > 1)
-        out = out_t.cpu().numpy()
-        cand = None
-        if topks is not None:
-            idx, vals = topks[0].cpu().tolist(), topks[1].cpu().tolist()
-            cand = [list(zip(i, v)) for i, v in zip(idx, vals)]
-        return [row.tolist() for row in out], cand
-
-    def _decode_steps(self, tok, pos, bts, window: int, greedy: bool):
+    def _decode_steps(self, tok, pos, bts, window: int, greedy: bool, slots=None):
         """``window`` decode steps on device tensors -> (tokens [B, window], last top-k or None)."""
         B = tok.shape[0]
         outs = []
@@ -701,9 +649,9 @@ class QwenEngine:
             sc = nat.scratch(B, self._splits(B), key=("decode", B))
             tok = tok.to(torch.int32)
             for w in range(window):
-                slots = self._slots(bts, pos)
+                kv_slots = self._slots(bts, pos)
                 seqlens = (pos + 1).to(torch.int32)
-                hn = nat.decode(sc, tok, pos, slots, bts, seqlens, B)
+                hn = nat.decode(sc, tok, pos, kv_slots, bts, seqlens, B)
                 t, tk = self._head_normed(hn, greedy)
                 outs.append(t)
                 if tk is not None:
@@ -713,11 +661,11 @@ class QwenEngine:
                 self.steps += 1
             return torch.stack(outs, dim=1), topks
         for w in range(window):
-            slots = self._slots(bts, pos)
+            kv_slots = self._slots(bts, pos)
             seqlens = (pos + 1).to(torch.int32)
 
             def attn(li, q, k, v):
-                self._append_kv(li, k, v, slots)
+                self._append_kv(li, k, v, kv_slots)
                 return self._paged_attention(li, q, bts, seqlens)
 
             x = F.embedding(tok, self.tok).reshape(B, -1)
@@ -732,71 +680,6 @@ class QwenEngine:
             pos = pos + 1
             self.steps += 1
         return torch.stack(outs, dim=1), topks
-
-    # ---- CUDA-graph decode: one captured graph per (padded batch, window)
-    @staticmethod
-    def _bucket(b: int) -> int:
-        for cap in (1, 2, 4, 8, 16, 24, 32, 48, 64, 96, 128, 160, 192, 224, 256):
-            if b <= cap:
-                return cap
-        return -(-b // 64) * 64
-
-    def _decode_graphed(self, tokens, positions, block_tables, window: int):
-        """Greedy decode through a replayed CUDA graph.  The batch is padded to a bucket size with
-        rows that sit at position 0 of the dummy block; inputs travel through pinned staging."""
-        B = int(tokens.shape[0])
-        Bp = self._bucket(B)
-        key = (Bp, window)
-        g = self._graphs.get(key)
-        if g is None:
-            g = self._capture(Bp, window)
-            self._graphs[key] = g
-        h_tok, h_pos, h_bts = g["h_tok"], g["h_pos"], g["h_bts"]
-        h_tok[:B] = torch.from_numpy(np.ascontiguousarray(tokens, dtype=np.int32))
-        h_pos[:B] = torch.from_numpy(np.ascontiguousarray(positions, dtype=np.int32))
-        h_bts[:B] = torch.from_numpy(np.ascontiguousarray(block_tables, dtype=np.int32))
-        if Bp > B:
-            h_tok[B:] = 0
-            h_pos[B:] = 0
-            h_bts[B:] = self.dummy_block
-        g["tok"].copy_(h_tok, non_blocking=True)
-        g["pos"].copy_(h_pos, non_blocking=True)
-        g["bts"].copy_(h_bts, non_blocking=True)
-        g["graph"].replay()
-        self.graph_replays += 1
-        self.steps += window
-        g["h_out"].copy_(g["out"], non_blocking=True)
-        torch.cuda.current_stream().synchronize()
-        return g["h_out"][:B].numpy().copy()
-
-    def _capture(self, Bp: int, window: int):
-        dev = self.device
-        mb = self.max_blocks
-        g = {"tok": torch.zeros(Bp, device=dev, dtype=torch.int32),
-             "pos": torch.zeros(Bp, device=dev, dtype=torch.int32),
-             "bts": torch.full((Bp, mb), self.dummy_block, device=dev, dtype=torch.int32),
-             "h_tok": torch.zeros(Bp, dtype=torch.int32).pin_memory(),
-             "h_pos": torch.zeros(Bp, dtype=torch.int32).pin_memory(),
-             "h_bts": torch.zeros(Bp, mb, dtype=torch.int32).pin_memory(),
-             "h_out": torch.zeros(Bp, window, dtype=torch.int32).pin_memory()}
-        steps0 = self.steps
-        # warm-up on a side stream (lazy one-time setup such as kernel attributes and symmetric
-        # buffers must not happen during capture), then capture the same work
-        side = torch.cuda.Stream(device=dev)
-        side.wait_stream(torch.cuda.current_stream())
-        with torch.cuda.stream(side):
-            for _ in range(2):
-                self._decode_steps(g["tok"], g["pos"], g["bts"], window, True)
-        torch.cuda.current_stream().wait_stream(side)
-        torch.cuda.synchronize()
-        graph = torch.cuda.CUDAGraph()
-        # thread-local capture mode: other threads of the process (e.g. a process group's watchdog)
-        # keep making CUDA calls of their own while this thread captures
-        with torch.cuda.graph(graph, capture_error_mode="thread_local"):
-            out, _ = self._decode_steps(g["tok"], g["pos"], g["bts"], window, True)
-        g["graph"], g["out"] = graph, out
-        self.steps = steps0
-        return g
 
     # ------------------------------------------------------------------ convenience
     @torch.no_grad()
@@ -818,3 +701,12 @@ class QwenEngine:
             x, delta = self._layer(li, x, delta, pos, attn)
         h, _ = F.rmsnorm(delta, self.norm, self.cfg.rms_eps, residual=x)
         return self.head(h).float()
+
+
+def make_engine(model, **kw):
+    """The serving engine of a model: hybrid decoders (recurrent state slots, per-layer mixers) or the
+    dense Qwen family.  Options an engine does not know raise its own error."""
+    if getattr(model, "family", "") == "hybrid":
+        from .hybrid import HybridEngine
+        return HybridEngine(model, **kw)
+    return QwenEngine(model, **kw)

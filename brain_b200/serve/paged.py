@@ -32,6 +32,11 @@ _host.register({
     "bbh_table_fork": (c.c_void_p, [c.c_void_p, c.c_void_p]),
     "bbh_table_unshare_tail": (c.c_int, [c.c_void_p, c.c_void_p, c.POINTER(c.c_uint32), c.POINTER(c.c_uint32)]),
     "bbh_table_adopt_prefix": (None, [c.c_void_p, c.c_void_p, c.c_void_p, c.c_uint32]),
+    "bbh_slots_new": (c.c_void_p, [c.c_uint32]),
+    "bbh_slots_free": (None, [c.c_void_p]),
+    "bbh_slots_available": (c.c_uint32, [c.c_void_p]),
+    "bbh_slots_alloc": (c.c_int64, [c.c_void_p]),
+    "bbh_slots_release": (c.c_int, [c.c_void_p, c.c_uint32]),
     "bbh_prefix_new": (c.c_void_p, []),
     "bbh_prefix_free": (None, [c.c_void_p]),
     "bbh_prefix_len": (c.c_uint64, [c.c_void_p]),
@@ -130,6 +135,62 @@ class BlockTable:
             raise ValueError("adopt_prefix expects a fresh sequence")
         arr = np.asarray(blocks, dtype=np.uint32)
         _host.lib().bbh_table_adopt_prefix(self._h, alloc._h, arr.ctypes.data, arr.size)
+
+
+class StateSlots:
+    """Slots of recurrent state, one per live sequence."""
+
+    def __init__(self, n: int):
+        self.n = n
+        self._h = _host.lib().bbh_slots_new(n)
+
+    def __del__(self):
+        if getattr(self, "_h", None):
+            _host.lib().bbh_slots_free(self._h)
+            self._h = None
+
+    def available(self) -> int:
+        return int(_host.lib().bbh_slots_available(self._h))
+
+    def alloc(self) -> int:
+        s = int(_host.lib().bbh_slots_alloc(self._h))
+        if s < 0:
+            raise MemoryError("no free recurrent-state slot")
+        return s
+
+    def release(self, slot: int) -> None:
+        if _host.lib().bbh_slots_release(self._h, slot) != 0:
+            raise RuntimeError(f"state slot {slot} is not in use")
+
+
+class CachedSequence:
+    """The cache side of one sequence that is fed by its caller instead of the scheduler: pages for its
+    tokens as they come, and a recurrent-state slot when the engine has such state."""
+
+    def __init__(self, alloc: BlockAllocator, slots: Optional[StateSlots], max_blocks: int):
+        self.alloc, self.slots = alloc, slots
+        self.table = BlockTable()
+        self.slot = slots.alloc() if slots is not None else 0
+        self._bt = np.zeros(max_blocks, dtype=np.int32)
+        self._n = 0
+
+    def __len__(self) -> int:
+        return len(self.table)
+
+    def extend(self, n: int) -> Tuple[int, np.ndarray]:
+        """Back the next ``n`` positions; returns (first of them, block table)."""
+        start = self.table.reserve(n, self.alloc)
+        blocks = self.table.blocks()
+        if len(blocks) > len(self._bt):
+            raise MemoryError(f"a sequence of {len(self.table)} tokens exceeds the engine's context")
+        self._bt[:len(blocks)] = blocks
+        return start, self._bt
+
+    def release(self) -> None:
+        self.table.release(self.alloc)
+        if self.slots is not None and self.slot >= 0:
+            self.slots.release(self.slot)
+            self.slot = -1
 
 
 class PrefixCache:

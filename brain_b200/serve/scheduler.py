@@ -43,6 +43,10 @@ _host.register({
     "bbh_sched_seq_output": (None, [c.c_void_p, c.c_int64, c.c_void_p]),
     "bbh_sched_seq_prompt": (None, [c.c_void_p, c.c_int64, c.c_void_p]),
     "bbh_sched_seq_table": (c.c_uint32, [c.c_void_p, c.c_int64, c.c_void_p, c.c_uint32]),
+    "bbh_sched_set_state_slots": (None, [c.c_void_p, c.c_uint32]),
+    "bbh_sched_free_slots": (c.c_uint32, [c.c_void_p]),
+    "bbh_sched_seq_slot": (c.c_int64, [c.c_void_p, c.c_int64]),
+    "bbh_sched_decode_slots": (None, [c.c_void_p, c.c_void_p]),
     "bbh_sched_forget": (None, [c.c_void_p, c.c_int64]),
     "bbh_sched_decode_all_greedy": (c.c_int, [c.c_void_p]),
     "bbh_sched_set_admit": (None, [c.c_void_p, c.c_uint32, c.c_uint32]),
@@ -141,6 +145,11 @@ class Scheduler:
             float(policy_arg), int(prefix_cache))
         if not self._h:
             raise ValueError("invalid scheduler configuration")
+        # a decoder with recurrent state: one slot per running sequence, passed along with its block
+        # table; the prefix cache is off (the state at a shared prefix's end is not kept)
+        self.state_slots = int(getattr(decoder, "state_slots", 0))
+        if self.state_slots:
+            _host.lib().bbh_sched_set_state_slots(self._h, self.state_slots)
         if admit_batch > 1:
             _host.lib().bbh_sched_set_admit(self._h, int(admit_batch), int(admit_max_wait))
         if prefill_budget > 0:      # prompt tokens per step (default 2 x max_prefill)
@@ -271,12 +280,13 @@ class Scheduler:
             bt = np.full(self.max_blocks, -1, dtype=np.int32)
             lib.bbh_sched_seq_table(self._h, rid_v, bt.ctypes.data, self.max_blocks)
             plan.append((rid_v, s.value, e.value, bool(last.value), info.params.is_greedy(),
-                         prompt[s.value:e.value].astype(np.int32), bt))
+                         prompt[s.value:e.value].astype(np.int32), bt,
+                         int(lib.bbh_sched_seq_slot(self._h, rid_v)) if self.state_slots else -1))
             if s.value == info.prefix_hit:
                 rep.admitted += 1
             rep.prefill_tokens += e.value - s.value
         n = nd.value
-        ids = toks = pos = bts = None
+        ids = toks = pos = bts = slots = None
         if n:
             ids = np.empty(n, dtype=np.int64)
             toks = np.empty(n, dtype=np.int32)
@@ -284,23 +294,29 @@ class Scheduler:
             bts = np.empty((n, self.max_blocks), dtype=np.int32)
             lib.bbh_sched_decode_batch(self._h, ids.ctypes.data, toks.ctypes.data, pos.ctypes.data,
                                        bts.ctypes.data, self.max_blocks)
+            if self.state_slots:
+                slots = np.empty(n, dtype=np.int32)
+                lib.bbh_sched_decode_slots(self._h, slots.ctypes.data)
+        has = bool(self.state_slots)
+        item = (lambda p: (p[5], p[1], p[6], p[3], p[4], p[7])) if has else (lambda p: (p[5], p[1], p[6], p[3], p[4]))
+        dec_kw = {"slots": slots} if has else {}
         all_greedy = bool(lib.bbh_sched_decode_all_greedy(self._h)) if n else True
         outs = decoded = None
         mixed = getattr(self.dec, "mixed_step", None) if self.mixed else None
         if plan and n and mixed is not None and win.value == 1:
             # the decode set was fixed by the plan, so both kinds of rows can share one forward
             g = all_greedy and all(p[4] for p in plan if p[3])
-            outs, g_toks, topks = mixed([(p[5], p[1], p[6], p[3], p[4]) for p in plan], toks, pos, bts, g)
+            outs, g_toks, topks = mixed([item(p) for p in plan], toks, pos, bts, g, **dec_kw)
             decoded = (g_toks, topks)
             rep.mixed = True
         elif plan:
             batch = getattr(self.dec, "prefill_batch", None)
             if batch is not None and len(plan) > 1:
-                outs = batch([(p[5], p[1], p[6], p[3], p[4]) for p in plan])
+                outs = batch([item(p) for p in plan])
             else:
-                outs = [self.dec.prefill_chunk(p[5], p[1], p[6], p[3], p[4]) for p in plan]
+                outs = [self.dec.prefill_chunk(*item(p)) for p in plan]
         if n and decoded is None:
-            decoded = self.dec.decode(toks, pos, bts, win.value, all_greedy)
+            decoded = self.dec.decode(toks, pos, bts, win.value, all_greedy, **dec_kw)
         # the tokens were read back, so the device is idle: one look at the error word before the
         # commits.  A kernel whose bounded wait ran out raises here and the caller fails the step's
         # requests instead of committing garbage tokens.

@@ -23,6 +23,8 @@ def spec_decode(engine, prompt: Sequence[int], max_new: int, k: int, draft: Draf
     offline use of an engine no scheduler is driving)."""
     if not prompt or k < 1:
         raise ValueError("spec_decode needs a non-empty prompt and k >= 1")
+    if getattr(engine, "state_slots", 0):
+        raise ValueError("speculative decoding rolls rejected tokens back; a recurrent state cannot be rolled back")
     if len(prompt) + max_new > engine.max_seq_len:
         raise ValueError("prompt + max_new exceeds the engine's context")
     alloc = alloc or BlockAllocator(engine.num_blocks, engine.block_size)

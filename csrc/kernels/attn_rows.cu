@@ -1,0 +1,83 @@
+// Attention of single query rows against the paged K/V pool, one warp per (row, query head): any head
+// sizes up to 256, bf16 or fp32 pages, soft-capped scores, per-head output gate.  It is the fp32 path and
+// the path of head sizes the tensor-core prefill and the split-KV decode kernels do not cover.
+#include "../common/host.hpp"
+#include "../common/ptx.cuh"
+#include "../common/rows.cuh"
+
+namespace bb {
+
+constexpr int AR_VEC = 8;   // elements of a lane: head sizes up to 256
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+attn_rows_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ kc, const T* __restrict__ vc,
+                 const int* __restrict__ pos, const int* __restrict__ row_seq, const int* __restrict__ tables,
+                 int max_blocks, int bs, T* __restrict__ out, int ldo, const T* __restrict__ gate, int ldg, int rows,
+                 int hq, int hk, int dk, int dv, int dkp, int dvp, float scale, float softcap) {
+  const int w = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
+  if (w >= rows * hq) return;
+  const int r = w / hq, h = w % hq, g = h / (hq / hk);
+  float qf[AR_VEC], o[AR_VEC];
+#pragma unroll
+  for (int i = 0; i < AR_VEC; ++i) {
+    const int d = lane + 32 * i;
+    qf[i] = d < dk ? to_f(q[(size_t)r * ldq + h * dkp + d]) * scale : 0.f;
+    o[i] = 0.f;
+  }
+  const int last = pos[r];
+  const int* bt = tables + (size_t)row_seq[r] * max_blocks;
+  float m = -INFINITY, l = 0.f;
+  for (int j = 0; j <= last; ++j) {
+    const size_t row = ((size_t)bt[j / bs] * hk + g) * bs + j % bs;
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < AR_VEC; ++i) {
+      const int d = lane + 32 * i;
+      if (d < dk) s = fmaf(qf[i], to_f(kc[row * dkp + d]), s);
+    }
+    s = warp_sum(s);
+    if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+    const float mn = fmaxf(m, s);
+    const float al = expf(m - mn), p = expf(s - mn);
+    l = l * al + p;
+    m = mn;
+#pragma unroll
+    for (int i = 0; i < AR_VEC; ++i) {
+      const int d = lane + 32 * i;
+      if (d < dv) o[i] = fmaf(p, to_f(vc[row * dvp + d]), o[i] * al);
+    }
+  }
+  float f = 1.f / l;
+  if (gate) f *= sigmoid_f(to_f(gate[(size_t)r * ldg + h]));
+#pragma unroll
+  for (int i = 0; i < AR_VEC; ++i) {
+    const int d = lane + 32 * i;
+    if (d < dvp) out[(size_t)r * ldo + h * dvp + d] = from_f<T>(d < dv ? o[i] * f : 0.f);
+  }
+}
+
+}  // namespace bb
+
+// dtype 0 bf16, 1 fp32.  Row r attends keys [0, pos[r]] of sequence row_seq[r]; head h of q at column
+// h dkp, of out at column h dvp; gate (may be null): raw gate values, head h at column h.
+BB_API int bb_attn_rows(int dtype, const void* q, int ldq, const void* kc, const void* vc, const int* pos,
+                        const int* row_seq, const int* tables, int max_blocks, int bs, void* out, int ldo,
+                        const void* gate, int ldg, int rows, int hq, int hk, int dk, int dv, int dkp, int dvp,
+                        float scale, float softcap, void* stream) {
+  using namespace bb;
+  if (rows <= 0) return BB_OK;
+  if (dk > 32 * AR_VEC || dvp > 32 * AR_VEC || hq % hk) return BB_ESIZE;
+  const int grid = (int)(((long)rows * hq * 32 + 127) / 128);
+  cudaStream_t s = (cudaStream_t)stream;
+  if (dtype)
+    attn_rows_kernel<float><<<grid, 128, 0, s>>>((const float*)q, ldq, (const float*)kc, (const float*)vc, pos, row_seq,
+                                                 tables, max_blocks, bs, (float*)out, ldo, (const float*)gate, ldg, rows,
+                                                 hq, hk, dk, dv, dkp, dvp, scale, softcap);
+  else
+    attn_rows_kernel<__nv_bfloat16><<<grid, 128, 0, s>>>(
+        (const __nv_bfloat16*)q, ldq, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, pos, row_seq, tables,
+        max_blocks, bs, (__nv_bfloat16*)out, ldo, (const __nv_bfloat16*)gate, ldg, rows, hq, hk, dk, dv, dkp, dvp, scale,
+        softcap);
+  return (int)cudaGetLastError();
+}

@@ -19,6 +19,7 @@
 
 #include "../common/host.hpp"
 #include "../common/ptx.cuh"
+#include "../common/tanh.cuh"
 
 namespace bb {
 
@@ -40,17 +41,24 @@ struct FaFwdArgs {
   const int* tile_seq;       // [gridDim.x] sequence of every query tile
   const int* tile_qt;        // [gridDim.x] tile index inside its sequence
   int max_blocks, block_rows;  // pool block = block_rows token rows per KV head
+  // Extended form (EXT): K and V heads of their own sizes, soft-capped scores, per-head output gate.
+  int dq, dv;                // columns of a query / value head in memory (a tile's other columns are not its own)
+  float cap_in, cap_log2;    // scores become cap_log2 tanh(cap_in q.k) (log2 domain); cap_log2 = 0: no cap
+  const __nv_bfloat16* gate; // raw gate of row r, head h at gate[r ldg + h]; the output is multiplied by its
+  int ldg;                   // sigmoid; may be null
 };
 
-template <int HD>
+template <int HD, int HDV = HD>
 struct FaFwdCfg {
-  static constexpr int NSUB = HD / 64;             // 64-column swizzled sub-tiles per row
+  static constexpr int NSUB = HD / 64;             // 64-column swizzled sub-tiles per row of Q and K
+  static constexpr int NSUBV = HDV / 64;           // ... of V
   static constexpr int SUB_BYTES = 128 * 128;      // [128 rows][64 bf16]
   static constexpr int TILE_BYTES = NSUB * SUB_BYTES;
+  static constexpr int VTILE_BYTES = NSUBV * SUB_BYTES;
   static constexpr int OFF_Q = 0;
   static constexpr int OFF_K = OFF_Q + TILE_BYTES;
   static constexpr int OFF_V = OFF_K + TILE_BYTES;
-  static constexpr int OFF_BAR = OFF_V + TILE_BYTES;
+  static constexpr int OFF_BAR = OFF_V + VTILE_BYTES;
   static constexpr int SMEM_MIN = OFF_BAR + 256 + 1024;
   // at least 80 KB so at most two CTAs are resident per SM (each allocates 256 TMEM columns)
   static constexpr int SMEM = SMEM_MIN < 80 * 1024 ? 80 * 1024 : SMEM_MIN;
@@ -356,12 +364,14 @@ static constexpr float kFwdTruncLog2 = 0.0041778f;   // log2(1.0029), see the pa
 // buffer, O [128, 128+HD).  Same shared-memory footprint, still two CTAs per SM.
 // PAGED: one CTA per (query tile of a packed sequence, query head); K/V tiles are assembled from
 // the pool's blocks (one TMA copy per block and 64-column half) instead of one copy per tile.
-template <int HD, bool PAGED>
+// EXT: see FaFwdArgs; head sizes below the tile's are zero-filled by the copies (K, V) or multiplied by
+// zeros (Q), P is rounded to nearest when it is packed.
+template <int HD, bool PAGED, int HDV = HD, bool EXT = false>
 __global__ void __launch_bounds__(192, 2)
 fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                const __grid_constant__ CUtensorMap tmV, const FaFwdArgs args) {
-  using Cfg = FaFwdCfg<HD>;
-  constexpr int NSUB = Cfg::NSUB;
+  using Cfg = FaFwdCfg<HD, HDV>;
+  constexpr int NSUB = Cfg::NSUB, NSUBV = Cfg::NSUBV;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~uintptr_t(1023));
@@ -427,7 +437,7 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
       mbar_expect_tx(q_full, Cfg::TILE_BYTES);
 #pragma unroll
       for (int c = 0; c < NSUB; ++c)
-        tma_load_2d(sQ + c * Cfg::SUB_BYTES, &tmQ, q_full, h * HD + c * 64, row_base + q0);
+        tma_load_2d(sQ + c * Cfg::SUB_BYTES, &tmQ, q_full, h * (EXT ? args.dq : HD) + c * 64, row_base + q0);
       for (int j = 0; j < n_blocks; ++j) {
         const uint32_t ph = j & 1;
         if (!mbar_wait(k_empty, ph ^ 1)) {
@@ -455,20 +465,20 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
           set_error(args.err, ERR_WAIT_PRODUCER);
           break;
         }
-        mbar_expect_tx(v_full, Cfg::TILE_BYTES);
+        mbar_expect_tx(v_full, Cfg::VTILE_BYTES);
         if (PAGED) {
           const int br = args.block_rows, per_tile = 128 / br;
           const int* tab = args.block_tables + (size_t)seq * args.max_blocks + j * per_tile;
           for (int i = 0; i < per_tile; ++i) {
             const bool live = (j * 128 + i * br) < S && (j * per_tile + i) < args.max_blocks;
             const int blk = live ? max(tab[i], 0) : 0;
-            for (int c = 0; c < NSUB; ++c)
+            for (int c = 0; c < NSUBV; ++c)
               tma_load_2d(sV + c * Cfg::SUB_BYTES + i * br * 128, &tmV, v_full, c * 64,
                           (blk * args.hk + kvh) * br);
           }
         } else {
 #pragma unroll
-          for (int c = 0; c < NSUB; ++c)
+          for (int c = 0; c < NSUBV; ++c)
             tma_load_2d(sV + c * Cfg::SUB_BYTES, &tmV, v_full, kvh * HD + c * 64, b * S + j * 128);
         }
       }
@@ -476,7 +486,7 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
   } else if (warp == 1) {
     if (lane == 0) {
       constexpr uint32_t idesc_qk = umma_idesc(1, 1, 1, 0, 0, 128, 64);
-      constexpr uint32_t idesc_pv = umma_idesc(1, 1, 1, 0, 1, 128, HD);
+      constexpr uint32_t idesc_pv = umma_idesc(1, 1, 1, 0, 1, 128, HDV);
       const uint32_t aq = smem_u32(sQ), bk = smem_u32(sK), bv = smem_u32(sV);
       bool ok = mbar_wait(q_full, 0);
       if (!ok) set_error(args.err, ERR_WAIT_MMA_FULL);
@@ -543,6 +553,31 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
       tmem_ld32(tS, r0);
       tmem_ld32(tS + 32, r1);
       tmem_wait_ld();
+      const bool capped = EXT && args.cap_log2 > 0.f;
+      if (capped) {
+        // scores -> log2-domain capped scores, in place; one polynomial when the whole warp is below its bound
+        float am = 0.f, am2 = 0.f;
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          am = fmaxf(am, fabsf(__uint_as_float(r0[i])));
+          am2 = fmaxf(am2, fabsf(__uint_as_float(r1[i])));
+        }
+        const float ci = args.cap_in, co = args.cap_log2;
+        if (!__any_sync(0xffffffffu, fmaxf(am, am2) * ci >= 0.4f)) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            r0[i] = __float_as_uint(co * tanh_small(__uint_as_float(r0[i]) * ci));
+            r1[i] = __float_as_uint(co * tanh_small(__uint_as_float(r1[i]) * ci));
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            r0[i] = __float_as_uint(co * tanh_fp32(__uint_as_float(r0[i]) * ci));
+            r1[i] = __float_as_uint(co * tanh_fp32(__uint_as_float(r1[i]) * ci));
+          }
+        }
+      }
+      const float sc = capped ? 1.f : args.scale_log2;
       const int kv0 = u * 64;
       const bool need_mask = (kv0 + 63 > kv_limit_row);
       const int lim = kv_limit_row - kv0;  // columns <= lim are visible
@@ -565,7 +600,7 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
           if (i + 32 <= lim) mx = fmaxf(mx, __uint_as_float(r1[i]));
         }
       }
-      mx *= args.scale_log2;
+      mx *= sc;
       float m_new = m_ref;
       if (mx > m_ref + 8.f) m_new = mx;  // lazy: keep the old reference while p stays <= 2^8
       const float alpha =
@@ -577,7 +612,7 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
         if (!ok) break;
         tc_fence_after();
 #pragma unroll 1
-        for (int c = 0; c < HD / 32; ++c) {
+        for (int c = 0; c < HDV / 32; ++c) {
           uint32_t r[32];
           tmem_ld32(tO + c * 32, r);
           tmem_wait_ld();
@@ -591,8 +626,7 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
       // P is packed by truncation (one PRMT per pair) after a 1.0029 pre-scale that folds into the
       // exponent offset: truncation of the scaled value is unbiased on average, the row sum runs over
       // the same scaled values (so O / l is unchanged) and the stored log-sum-exp takes the factor out
-      const float m_use = ((m_ref == -INFINITY) ? 0.f : m_ref) - kFwdTruncLog2;
-      const float sc = args.scale_log2;
+      const float m_use = ((m_ref == -INFINITY) ? 0.f : m_ref) - (EXT ? 0.f : kFwdTruncLog2);
       uint32_t pk[32];  // 64 probabilities as 32 packed bf16x2 words
       float ls = 0.f, ls_b = 0.f;    // two running sums (alternating iterations) halve the add chain
 #pragma unroll
@@ -610,8 +644,13 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
         if (i & 2) ls_b += (a0 + a1) + (b0 + b1);
         else ls += (a0 + a1) + (b0 + b1);
         // integer-pipe packing: cvt.rn.bf16x2 would share the quarter-rate unit with ex2
-        pk[i >> 1] = __byte_perm(__float_as_uint(a0), __float_as_uint(a1), 0x7632);         // keys  0..31 -> words  0..15
-        pk[16 + (i >> 1)] = __byte_perm(__float_as_uint(b0), __float_as_uint(b1), 0x7632);  // keys 32..63 -> words 16..31
+        if constexpr (EXT) {
+          pk[i >> 1] = pack_bf16x2_alu(a0, a1);
+          pk[16 + (i >> 1)] = pack_bf16x2_alu(b0, b1);
+        } else {
+          pk[i >> 1] = __byte_perm(__float_as_uint(a0), __float_as_uint(a1), 0x7632);         // keys  0..31 -> words  0..15
+          pk[16 + (i >> 1)] = __byte_perm(__float_as_uint(b0), __float_as_uint(b1), 0x7632);  // keys 32..63 -> words 16..31
+        }
       }
       l += ls + ls_b;
       tmem_st32(tS, pk);
@@ -627,10 +666,17 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
       if (lane == 0) set_error(args.err, ERR_WAIT_SOFTMAX);
     } else {
       tc_fence_after();
-      const float inv = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* orow = args.O + (size_t)(row_base + q_idx) * args.ldo + h * HD;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if constexpr (EXT) {
+        if (args.gate && q_idx < T) {
+          const float gv = __bfloat162float(args.gate[(size_t)(row_base + q_idx) * args.ldg + h]);
+          inv *= 1.f / (1.f + exp2f(-1.4426950408889634f * gv));
+        }
+      }
+      const int dv = EXT ? args.dv : HD;   // columns of this head in the output
+      __nv_bfloat16* orow = args.O + (size_t)(row_base + q_idx) * args.ldo + h * dv;
 #pragma unroll 1
-      for (int c = 0; c < HD / 32; ++c) {
+      for (int c = 0; c < HDV / 32; ++c) {
         uint32_t r[32];
         __syncwarp();
         tmem_ld32(tO + c * 32, r);
@@ -638,6 +684,7 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
         if (q_idx < T) {
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
+            if (EXT && c * 32 + q * 8 >= dv) break;
             uint4 o;
             o.x = pack_bf16x2(__uint_as_float(r[q * 8 + 0]) * inv, __uint_as_float(r[q * 8 + 1]) * inv);
             o.y = pack_bf16x2(__uint_as_float(r[q * 8 + 2]) * inv, __uint_as_float(r[q * 8 + 3]) * inv);
@@ -763,6 +810,71 @@ BB_API int bb_flash_fwd_paged(const void* q, int ldq, const void* k_pool, const 
     fa_fwd2_kernel<64, true><<<grid, 192, FaFwdCfg<64>::SMEM, s>>>(tmQ, tmK, tmV, a);
   }
   return (int)cudaGetLastError();
+}
+
+namespace bb {
+template <int HD, int HDV>
+static int launch_paged_x(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const FaFwdArgs& a,
+                          int n_tiles, cudaStream_t s) {
+  static PerDeviceOnce once;
+  const cudaError_t e = ensure_dyn_smem(once, fa_fwd2_kernel<HD, true, HDV, true>, FaFwdCfg<HD, HDV>::SMEM);
+  if (e != cudaSuccess) return (int)e;
+  fa_fwd2_kernel<HD, true, HDV, true><<<dim3(n_tiles, a.hq, 1), 192, FaFwdCfg<HD, HDV>::SMEM, s>>>(tmQ, tmK, tmV, a);
+  return (int)cudaGetLastError();
+}
+}  // namespace bb
+
+// The same for heads of their own sizes: query / key heads dq columns wide and value heads dv (multiples
+// of 8, up to 128; zero padding counts as columns), scores softcap tanh(scale q.k / softcap) when softcap
+// > 0, and an optional per-head output gate (sigmoid of gate[row, head]).  Pools: bf16
+// [pool_blocks][hk][block_rows][dq | dv].
+BB_API int bb_flash_fwd_paged_x(const void* q, int ldq, const void* k_pool, const void* v_pool, void* out, int ldo,
+                                const int* block_tables, int max_blocks, int block_rows, int pool_blocks,
+                                const int* seq_row0, const int* seq_ctx, const int* tile_seq, const int* tile_qt,
+                                int n_tiles, int total_rows, int hq, int hk, int dq, int dv, float scale, float softcap,
+                                const void* gate, int ldg, void* stream) {
+  using namespace bb;
+  if (n_tiles <= 0) return BB_OK;
+  if (hq % hk || total_rows <= 0 || max_blocks <= 0 || pool_blocks <= 0) return BB_EARG;
+  if (block_rows != 16 && block_rows != 32 && block_rows != 64 && block_rows != 128) return BB_ESIZE;
+  if (dq % 8 || dv % 8 || dq > 128 || dv > 128 || ldq % 8 || ldo % 8) return BB_ESIZE;
+  FaFwdArgs a{};
+  a.O = static_cast<__nv_bfloat16*>(out);
+  a.ldo = ldo;
+  a.hq = hq;
+  a.hk = hk;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  a.causal = 1;
+  a.err = device_error_word();
+  a.block_tables = block_tables;
+  a.seq_row0 = seq_row0;
+  a.seq_ctx = seq_ctx;
+  a.tile_seq = tile_seq;
+  a.tile_qt = tile_qt;
+  a.max_blocks = max_blocks;
+  a.block_rows = block_rows;
+  a.dq = dq;
+  a.dv = dv;
+  if (softcap > 0.f) {
+    a.cap_in = scale / softcap;
+    a.cap_log2 = softcap * 1.4426950408889634f;
+  }
+  a.gate = static_cast<const __nv_bfloat16*>(gate);
+  a.ldg = ldg;
+  CUtensorMap tmQ, tmK, tmV;
+  const CUtensorMapDataType bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+  int rc = make_tmap_2d(&tmQ, bf, 2, q, (uint64_t)hq * dq, (uint64_t)total_rows, (uint64_t)ldq * 2, 64, 128);
+  if (rc) return rc;
+  const uint64_t pool_rows = (uint64_t)pool_blocks * hk * block_rows;
+  rc = make_tmap_2d(&tmK, bf, 2, k_pool, (uint64_t)dq, pool_rows, (uint64_t)dq * 2, 64, block_rows);
+  if (rc) return rc;
+  rc = make_tmap_2d(&tmV, bf, 2, v_pool, (uint64_t)dv, pool_rows, (uint64_t)dv * 2, 64, block_rows);
+  if (rc) return rc;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dq <= 64) return dv <= 64 ? launch_paged_x<64, 64>(tmQ, tmK, tmV, a, n_tiles, s)
+                                : launch_paged_x<64, 128>(tmQ, tmK, tmV, a, n_tiles, s);
+  return dv <= 64 ? launch_paged_x<128, 64>(tmQ, tmK, tmV, a, n_tiles, s)
+                  : launch_paged_x<128, 128>(tmQ, tmK, tmV, a, n_tiles, s);
 }
 
 BB_API int bb_flash_fwd(const void* q, int ldq, const void* k, int ldk, const void* v, int ldv,

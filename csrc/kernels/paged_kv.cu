@@ -15,6 +15,7 @@
 // decode_softmax_batched,paged_decode_apply_batched}.wgsl, crates/qwen3/src/serve.rs:1262-1288.
 #include "../common/host.hpp"
 #include "../common/ptx.cuh"
+#include "../common/tanh.cuh"
 #include "../common/vec.cuh"
 #include <type_traits>
 
@@ -174,7 +175,15 @@ __device__ __forceinline__ void cp_async_wait() {
 // I8: kc/vc point at int8 pools and ks/vs at their per-row scales; a lane's slice of a row is DPL
 // bytes, the dot product runs on the integer values and the key's scale multiplies the score, the
 // value's scale multiplies the probability.
-template <int HD, int G, bool I8>
+
+//
+// EXT: key and value heads of their own sizes (dk / dv columns in memory, multiples of 8, at most HD /
+// HDV) and soft-capped scores (x.cap_log2 tanh(x.cap_in q.k) in the log2 domain).
+struct PdExt {
+  int dk, dv;
+  float cap_in, cap_log2;   // cap_log2 = 0: no cap
+};
+template <int HD, int G, bool I8, int HDV = HD, bool EXT = false>
 __global__ void __launch_bounds__(128, 3)
 paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
                     const void* __restrict__ kc_, const void* __restrict__ vc_,
@@ -182,17 +191,21 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
                     const int* __restrict__ block_tables, int max_blocks,
                     const int* __restrict__ seqlens, float* __restrict__ part_o,
                     float* __restrict__ part_ml, int hq, int hk, int bs, int splits,
-                    float scale_log2, int gsplit) {
+                    float scale_log2, int gsplit, PdExt x) {
   // gsplit > 1: a kv head's query heads are divided over gsplit CTAs of G heads each (8 heads per
   // kv head would need 256 registers for q and o alone); the siblings re-read K/V through L2.
+  static_assert(!(EXT && I8), "the extended form reads bf16 pages");
   constexpr int DPL = HD / 8;            // dims per lane: 16 (hd 128) or 8 (hd 64)
+  constexpr int DPV = HDV / 8;           // value dims per lane
   constexpr int ES = I8 ? 1 : 2;         // bytes per stored element
   constexpr int ROWB = HD * ES;          // bytes per K or V row
-  constexpr int CPR = ROWB / 16;         // 16-byte requests per row
+  constexpr int ROWBV = HDV * ES;
+  constexpr int CPM = (ROWB > ROWBV ? ROWB : ROWBV) / 16;   // 16-byte requests per row
   constexpr int NST = 4;                 // pipeline depth (steps of 16 keys)
-  constexpr int STAGE = 16 * ROWB;       // bytes per stage per tensor
-  constexpr int PIPE_BYTES = 2 * NST * STAGE;
-  constexpr int MERGE_BYTES = 4 * G * HD * 4;
+  constexpr int STAGE = 16 * ROWB;       // bytes per stage of K
+  constexpr int STAGEV = 16 * ROWBV;     // ... of V
+  constexpr int PIPE_BYTES = NST * (STAGE + STAGEV);
+  constexpr int MERGE_BYTES = 4 * G * HDV * 4;
   constexpr int SMEM_BYTES = PIPE_BYTES > MERGE_BYTES ? PIPE_BYTES : MERGE_BYTES;
   __shared__ __align__(16) unsigned char s_raw[SMEM_BYTES];   // pipeline stages, then the merge buffer
   __shared__ float s_sc[NST][2][16];                          // I8: row scales (K, V) per stage
@@ -206,6 +219,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
   const int head0 = (kvh * gsplit + blockIdx.y % gsplit) * G;   // first query head of this CTA
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int grp = lane >> 3, sub = lane & 7;
+  const int rowk = EXT ? x.dk * ES : ROWB, rowv = EXT ? x.dv * ES : ROWBV;   // bytes of a stored row
   const int S = seqlens[b];
   const int per_split = ((S + splits - 1) / splits + 31) / 32 * 32;
   const int k_begin = sp * per_split;
@@ -218,14 +232,14 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
     const int st = i % NST;
     const int k0 = k_begin + i * 16;
 #pragma unroll
-    for (int c = threadIdx.x; c < 16 * CPR; c += 128) {
-      const int kl = c / CPR, part = c % CPR;
+    for (int c = threadIdx.x; c < 16 * CPM; c += 128) {
+      const int kl = c / CPM, part = c % CPM;
       const int key = k0 + kl;
       if (key < k_end) {
         const int blk = bt[key / bs], off = key % bs;
         const size_t r = ((size_t)blk * hk + kvh) * bs + off;
-        cp_async16(s_k + st * STAGE + kl * ROWB + part * 16, kc + r * ROWB + part * 16);
-        cp_async16(s_v + st * STAGE + kl * ROWB + part * 16, vc + r * ROWB + part * 16);
+        if (!EXT || part * 16 < rowk) cp_async16(s_k + st * STAGE + kl * ROWB + part * 16, kc + r * rowk + part * 16);
+        if (!EXT || part * 16 < rowv) cp_async16(s_v + st * STAGEV + kl * ROWBV + part * 16, vc + r * rowv + part * 16);
       }
     }
     if constexpr (I8) {
@@ -255,12 +269,17 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
   float qs[I8 ? G : 1];
 #pragma unroll
   for (int g = 0; g < G; ++g) {
-    const bf16x8* qp = reinterpret_cast<const bf16x8*>(q + (size_t)b * ldq + (head0 + g) * HD + sub * DPL);
+    const bf16x8* qp = reinterpret_cast<const bf16x8*>(q + (size_t)b * ldq + (head0 + g) * (EXT ? x.dk : HD) + sub * DPL);
     float qf[DPL];
 #pragma unroll
     for (int v = 0; v < DPL / 8; ++v) {
       float f[8];
-      unpack8(qp[v], f);
+      if (!EXT || sub * DPL + v * 8 < x.dk) {
+        unpack8(qp[v], f);
+      } else {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) f[j] = 0.f;
+      }
 #pragma unroll
       for (int j = 0; j < 8; ++j) qf[v * 8 + j] = f[j];
     }
@@ -292,13 +311,13 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
       for (int j = 0; j < DPL; ++j) qr[g][j] = qf[j] * scale_log2;
     }
   }
-  float m[G], l[G], o[G][DPL];
+  float m[G], l[G], o[G][DPV];
 #pragma unroll
   for (int g = 0; g < G; ++g) {
     m[g] = -INFINITY;
     l[g] = 0.f;
 #pragma unroll
-    for (int j = 0; j < DPL; ++j) o[g][j] = 0.f;
+    for (int j = 0; j < DPV; ++j) o[g][j] = 0.f;
   }
 
   const int kl = warp * 4 + grp;   // this group's key within a step
@@ -309,7 +328,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
     cp_async_commit();
     const int st = i % NST;
     if (k_begin + i * 16 + kl < k_end) {
-      float xf[DPL];
+      float xf[DPL > DPV ? DPL : DPV];
       float sc[G];
       const unsigned char* krow = s_k + st * STAGE + kl * ROWB + sub * DPL * ES;
       // the 8 lanes of a group are all valid or all invalid, so they shuffle among themselves
@@ -336,7 +355,12 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
 #pragma unroll
         for (int v = 0; v < DPL / 8; ++v) {
           float t[8];
-          unpack8(reinterpret_cast<const bf16x8*>(krow)[v], t);
+          if (!EXT || sub * DPL + v * 8 < x.dk) {
+            unpack8(reinterpret_cast<const bf16x8*>(krow)[v], t);
+          } else {   // shared memory past the stored row was never written
+#pragma unroll
+            for (int j = 0; j < 8; ++j) t[j] = 0.f;
+          }
 #pragma unroll
           for (int j = 0; j < 8; ++j) xf[v * 8 + j] = t[j];
         }
@@ -348,21 +372,29 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
           a += __shfl_xor_sync(gm, a, 1);
           a += __shfl_xor_sync(gm, a, 2);
           a += __shfl_xor_sync(gm, a, 4);
+          if constexpr (EXT) {
+            if (x.cap_log2 > 0.f) a = x.cap_log2 * tanh_fp32(a);
+          }
           sc[g] = a;
         }
       }
-      const unsigned char* vrow = s_v + st * STAGE + kl * ROWB + sub * DPL * ES;
+      const unsigned char* vrow = s_v + st * STAGEV + kl * ROWBV + sub * DPV * ES;
       if constexpr (I8) {
-        const i8vec<DPL> raw = *reinterpret_cast<const i8vec<DPL>*>(vrow);
+        const i8vec<DPV> raw = *reinterpret_cast<const i8vec<DPV>*>(vrow);
 #pragma unroll
-        for (int v = 0; v < DPL / 4; ++v)
+        for (int v = 0; v < DPV / 4; ++v)
 #pragma unroll
           for (int j = 0; j < 4; ++j) xf[v * 4 + j] = (float)(int8_t)(raw.w[v] >> (8 * j));
       } else {
 #pragma unroll
-        for (int v = 0; v < DPL / 8; ++v) {
+        for (int v = 0; v < DPV / 8; ++v) {
           float t[8];
-          unpack8(reinterpret_cast<const bf16x8*>(vrow)[v], t);
+          if (!EXT || sub * DPV + v * 8 < x.dv) {
+            unpack8(reinterpret_cast<const bf16x8*>(vrow)[v], t);
+          } else {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) t[j] = 0.f;
+          }
 #pragma unroll
           for (int j = 0; j < 8; ++j) xf[v * 8 + j] = t[j];
         }
@@ -374,14 +406,14 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
           const float alpha = exp2f(m[g] - sc[g]);   // exp2(-inf) = 0 on the first key
           l[g] *= alpha;
 #pragma unroll
-          for (int j = 0; j < DPL; ++j) o[g][j] *= alpha;
+          for (int j = 0; j < DPV; ++j) o[g][j] *= alpha;
           m[g] = sc[g];
         }
         const float pg = exp2f(sc[g] - m[g]);
         l[g] += pg;
         const float pv = I8 ? pg * vscale : pg;
 #pragma unroll
-        for (int j = 0; j < DPL; ++j) o[g][j] += pv * xf[j];
+        for (int j = 0; j < DPV; ++j) o[g][j] += pv * xf[j];
       }
     }
   }
@@ -397,7 +429,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
       const float a1 = (m[g] == -INFINITY) ? 0.f : exp2f(m[g] - mm);
       const float a2 = (m2 == -INFINITY) ? 0.f : exp2f(m2 - mm);
 #pragma unroll
-      for (int j = 0; j < DPL; ++j) {
+      for (int j = 0; j < DPV; ++j) {
         const float o2 = __shfl_xor_sync(0xffffffffu, o[g][j], step);
         o[g][j] = o[g][j] * a1 + o2 * a2;
       }
@@ -407,7 +439,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
   }
   // merge the 4 warps of the CTA through shared memory (the pipeline stages are free now)
   __syncthreads();
-  float* s_o = reinterpret_cast<float*>(s_raw);   // [4][G][HD]
+  float* s_o = reinterpret_cast<float*>(s_raw);   // [4][G][HDV]
   if (grp == 0) {
 #pragma unroll
     for (int g = 0; g < G; ++g) {
@@ -416,22 +448,22 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
         s_l[warp][g] = l[g];
       }
 #pragma unroll
-      for (int j = 0; j < DPL; ++j) s_o[(warp * G + g) * HD + sub * DPL + j] = o[g][j];
+      for (int j = 0; j < DPV; ++j) s_o[(warp * G + g) * HDV + sub * DPV + j] = o[g][j];
     }
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < G * HD; i += blockDim.x) {
-    const int g = i / HD, c = i % HD;
+  for (int i = threadIdx.x; i < G * HDV; i += blockDim.x) {
+    const int g = i / HDV, c = i % HDV;
     float mm = -INFINITY;
     for (int w = 0; w < 4; ++w) mm = fmaxf(mm, s_m[w][g]);
     float ll = 0.f, oo = 0.f;
     for (int w = 0; w < 4; ++w) {
       const float a = (s_m[w][g] == -INFINITY) ? 0.f : exp2f(s_m[w][g] - mm);
       ll += s_l[w][g] * a;
-      oo += s_o[(w * G + g) * HD + c] * a;
+      oo += s_o[(w * G + g) * HDV + c] * a;
     }
     const size_t idx = ((size_t)b * hq + head0 + g) * splits + sp;
-    part_o[idx * HD + c] = oo;
+    part_o[idx * HDV + c] = oo;
     if (c == 0) {
       part_ml[idx * 2] = mm;
       part_ml[idx * 2 + 1] = ll;
@@ -443,7 +475,10 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
 __global__ void paged_decode_merge_kernel(const float* __restrict__ part_o,
                                           const float* __restrict__ part_ml,
                                           __nv_bfloat16* __restrict__ out, int ldo, int hq, int hd,
-                                          int splits) {
+                                          int splits, int hd_out, const __nv_bfloat16* __restrict__ gate,
+                                          int ldg) {
+  // hd: columns of a partial row; hd_out: columns of a head in the output; gate (may be null): raw
+  // per-head output gate, the head is multiplied by its sigmoid
   const int b = blockIdx.x, h = blockIdx.y;
   const size_t base = ((size_t)b * hq + h) * splits;
   float mm = -INFINITY;
@@ -453,14 +488,15 @@ __global__ void paged_decode_merge_kernel(const float* __restrict__ part_o,
     const float ms = part_ml[(base + s) * 2];
     ll += (ms == -INFINITY) ? 0.f : part_ml[(base + s) * 2 + 1] * exp2f(ms - mm);
   }
-  const float inv = ll > 0.f ? 1.f / ll : 0.f;
-  for (int c = threadIdx.x; c < hd; c += blockDim.x) {
+  float inv = ll > 0.f ? 1.f / ll : 0.f;
+  if (gate) inv *= 1.f / (1.f + exp2f(-1.4426950408889634f * __bfloat162float(gate[(size_t)b * ldg + h])));
+  for (int c = threadIdx.x; c < hd_out; c += blockDim.x) {
     float acc = 0.f;
     for (int s = 0; s < splits; ++s) {
       const float ms = part_ml[(base + s) * 2];
       if (ms != -INFINITY) acc += part_o[(base + s) * hd + c] * exp2f(ms - mm);
     }
-    out[(size_t)b * ldo + h * hd + c] = __float2bfloat16(acc * inv);
+    out[(size_t)b * ldo + h * hd_out + c] = __float2bfloat16(acc * inv);
   }
 }
 
@@ -513,11 +549,11 @@ static int launch_paged_decode(bool i8, const void* q, int ldq, const void* kc, 
     if (i8)                                                                                       \
       paged_decode_kernel<HD_, G_, true><<<grid, 128, 0, s>>>(                                    \
           (const __nv_bfloat16*)q, ldq, kc, vc, ks, vs, block_tables, max_blocks, seqlens,        \
-          part_o, part_ml, hq, hk, bs, splits, sl2, gsplit);                                      \
+          part_o, part_ml, hq, hk, bs, splits, sl2, gsplit, PdExt{});                                      \
     else                                                                                          \
       paged_decode_kernel<HD_, G_, false><<<grid, 128, 0, s>>>(                                   \
           (const __nv_bfloat16*)q, ldq, kc, vc, nullptr, nullptr, block_tables, max_blocks,       \
-          seqlens, part_o, part_ml, hq, hk, bs, splits, sl2, gsplit);                             \
+          seqlens, part_o, part_ml, hq, hk, bs, splits, sl2, gsplit, PdExt{});                             \
   } while (0)
   if (hd == 128) {
     switch (G) {
@@ -542,7 +578,7 @@ static int launch_paged_decode(bool i8, const void* q, int ldq, const void* kc, 
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
   paged_decode_merge_kernel<<<dim3(B, hq), 128, 0, s>>>(part_o, part_ml, (__nv_bfloat16*)out, ldo,
-                                                        hq, hd, splits);
+                                                        hq, hd, splits, hd, nullptr, 0);
   return (int)cudaGetLastError();
 }
 
@@ -554,6 +590,53 @@ BB_API int bb_paged_decode(const void* q, int ldq, const void* kc, const void* v
   return launch_paged_decode(false, q, ldq, kc, vc, nullptr, nullptr, block_tables, max_blocks,
                              seqlens, out, ldo, part_o, part_ml, B, hq, hk, hd, bs, splits, scale,
                              stream);
+}
+
+// The same for key / value heads of their own sizes (dk / dv stored columns, multiples of 8, up to 128),
+// any number of query heads per kv head, scores softcap tanh(scale q.k / softcap) when softcap > 0, and
+// an optional output gate.  part_o: fp32 [B*hq*splits*(dv <= 64 ? 64 : 128)].
+BB_API int bb_paged_decode_x(const void* q, int ldq, const void* kc, const void* vc, const int* block_tables,
+                             int max_blocks, const int* seqlens, void* out, int ldo, float* part_o, float* part_ml,
+                             int B, int hq, int hk, int dk, int dv, int bs, int splits, float scale, float softcap,
+                             const void* gate, int ldg, void* stream) {
+  if (B <= 0) return BB_OK;
+  if (hq % hk || splits < 1) return BB_EARG;
+  if (dk % 8 || dv % 8 || dk > 128 || dv > 128 || ldq % 8) return BB_ESIZE;
+  const int ratio = hq / hk;
+  const int G = ratio % 4 == 0 ? 4 : (ratio % 3 == 0 ? 3 : (ratio % 2 == 0 ? 2 : 1));
+  const int gsplit = ratio / G;
+  dim3 grid(B, hk * gsplit, splits);
+  PdExt x{dk, dv, 0.f, 0.f};
+  float sl2 = scale * 1.4426950408889634f;
+  if (softcap > 0.f) {
+    sl2 = scale / softcap;     // the query is pre-scaled so that q.k is the argument of tanh
+    x.cap_in = sl2;
+    x.cap_log2 = softcap * 1.4426950408889634f;
+  }
+  cudaStream_t s = (cudaStream_t)stream;
+#define BB_LAUNCH_PX(HD_, HDV_, G_)                                                                        \
+  paged_decode_kernel<HD_, G_, false, HDV_, true><<<grid, 128, 0, s>>>(                                    \
+      (const __nv_bfloat16*)q, ldq, kc, vc, nullptr, nullptr, block_tables, max_blocks, seqlens, part_o, part_ml, \
+      hq, hk, bs, splits, sl2, gsplit, x)
+#define BB_LAUNCH_PXG(HD_, HDV_)                \
+  switch (G) {                                  \
+    case 4: BB_LAUNCH_PX(HD_, HDV_, 4); break;  \
+    case 3: BB_LAUNCH_PX(HD_, HDV_, 3); break;  \
+    case 2: BB_LAUNCH_PX(HD_, HDV_, 2); break;  \
+    default: BB_LAUNCH_PX(HD_, HDV_, 1); break; \
+  }
+  if (dk <= 64) {
+    if (dv <= 64) { BB_LAUNCH_PXG(64, 64) } else { BB_LAUNCH_PXG(64, 128) }
+  } else {
+    if (dv <= 64) { BB_LAUNCH_PXG(128, 64) } else { BB_LAUNCH_PXG(128, 128) }
+  }
+#undef BB_LAUNCH_PXG
+#undef BB_LAUNCH_PX
+  cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) return (int)e;
+  paged_decode_merge_kernel<<<dim3(B, hq), 128, 0, s>>>(part_o, part_ml, (__nv_bfloat16*)out, ldo, hq,
+                                                        dv <= 64 ? 64 : 128, splits, dv, (const __nv_bfloat16*)gate, ldg);
+  return (int)cudaGetLastError();
 }
 
 // int8 pools kc/vc with per-row scales ks/vs: fp32 [num_blocks, hk, bs].

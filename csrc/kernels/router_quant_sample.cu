@@ -140,16 +140,20 @@ __global__ void quant_rows_bf16_vec_kernel(const __nv_bfloat16* __restrict__ x, 
   }
 }
 
+__device__ __forceinline__ float logit_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float logit_f(float v) { return v; }
+
 // Greedy head: out[r] = argmax_c logits[r, c] (lowest index on ties).  One block per row.
-__global__ void argmax_rows_kernel(const __nv_bfloat16* __restrict__ logits, long ld, int V,
+template <typename T>
+__global__ void argmax_rows_kernel(const T* __restrict__ logits, long ld, int V,
                                    int* __restrict__ out) {
   __shared__ float sv[32];
   __shared__ int si[32];
-  const __nv_bfloat16* row = logits + (size_t)blockIdx.x * ld;
+  const T* row = logits + (size_t)blockIdx.x * ld;
   float best = -INFINITY;
   int bi = 0x7fffffff;
   for (int i = threadIdx.x; i < V; i += blockDim.x) {
-    const float f = __bfloat162float(row[i]);
+    const float f = logit_f(row[i]);
     if (f > best) {
       best = f;
       bi = i;
@@ -189,13 +193,14 @@ __global__ void argmax_rows_kernel(const __nv_bfloat16* __restrict__ logits, lon
 // Top-K per row by K rounds of "largest remaining" (value descending, lowest index first on ties —
 // the order of crates/kernels/wgsl/topk_extract_step.wgsl).  One block per row; every round is one
 // pass over the row (it stays in L2), "remaining" = lexicographically after the previous pick.
-__global__ void topk_rows_kernel(const __nv_bfloat16* __restrict__ logits, long ld, int V, int K,
+template <typename T>
+__global__ void topk_rows_kernel(const T* __restrict__ logits, long ld, int V, int K,
                                  int* __restrict__ out_idx, float* __restrict__ out_val) {
   __shared__ float sv[32];
   __shared__ int si[32];
   __shared__ float s_last_v;
   __shared__ int s_last_i;
-  const __nv_bfloat16* row = logits + (size_t)blockIdx.x * ld;
+  const T* row = logits + (size_t)blockIdx.x * ld;
   if (threadIdx.x == 0) {
     s_last_v = INFINITY;
     s_last_i = -1;
@@ -207,7 +212,7 @@ __global__ void topk_rows_kernel(const __nv_bfloat16* __restrict__ logits, long 
     float best = -INFINITY;
     int bi = 0x7fffffff;
     for (int i = threadIdx.x; i < V; i += blockDim.x) {
-      const float f = __bfloat162float(row[i]);
+      const float f = logit_f(row[i]);
       const bool remaining = f < lv || (f == lv && i > li);
       if (remaining && (f > best || (f == best && i < bi))) {
         best = f;
@@ -290,14 +295,28 @@ BB_API int bb_topk_rows(const void* logits, long ld, int rows, int V, int K, int
                         void* stream) {
   if (rows <= 0) return BB_OK;
   if (K < 1 || K > V) return BB_EARG;
-  topk_rows_kernel<<<rows, 512, 0, (cudaStream_t)stream>>>((const __nv_bfloat16*)logits, ld, V, K,
+  topk_rows_kernel<__nv_bfloat16><<<rows, 512, 0, (cudaStream_t)stream>>>((const __nv_bfloat16*)logits, ld, V, K,
                                                           idx, val);
   return (int)cudaGetLastError();
 }
 
 BB_API int bb_argmax_rows(const void* logits, long ld, int rows, int V, int* out, void* stream) {
   if (rows <= 0) return BB_OK;
-  argmax_rows_kernel<<<rows, 512, 0, (cudaStream_t)stream>>>((const __nv_bfloat16*)logits, ld, V,
+  argmax_rows_kernel<__nv_bfloat16><<<rows, 512, 0, (cudaStream_t)stream>>>((const __nv_bfloat16*)logits, ld, V,
                                                             out);
+  return (int)cudaGetLastError();
+}
+
+// The same two over fp32 logits.
+BB_API int bb_topk_rows_f32(const float* logits, long ld, int rows, int V, int K, int* idx, float* val, void* stream) {
+  if (rows <= 0) return BB_OK;
+  if (K < 1 || K > V) return BB_EARG;
+  topk_rows_kernel<float><<<rows, 512, 0, (cudaStream_t)stream>>>(logits, ld, V, K, idx, val);
+  return (int)cudaGetLastError();
+}
+
+BB_API int bb_argmax_rows_f32(const float* logits, long ld, int rows, int V, int* out, void* stream) {
+  if (rows <= 0) return BB_OK;
+  argmax_rows_kernel<float><<<rows, 512, 0, (cudaStream_t)stream>>>(logits, ld, V, out);
   return (int)cudaGetLastError();
 }

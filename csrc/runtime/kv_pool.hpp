@@ -76,6 +76,34 @@ class KvPool {
   PrefixIndex* index_ = nullptr;
 };
 
+// Slots of per-sequence recurrent state (one per running sequence): a LIFO of free indices.  Slots are
+// handed out as they are; the kernels start a sequence at position 0 from zeros.
+class StateSlots {
+ public:
+  explicit StateSlots(uint32_t n = 0) : used_(n, 0) {
+    for (uint32_t i = n; i-- > 0;) free_.push_back(i);
+  }
+  uint32_t size() const { return static_cast<uint32_t>(used_.size()); }
+  uint32_t free_slots() const { return static_cast<uint32_t>(free_.size()); }
+  int64_t alloc() {
+    if (free_.empty()) return -1;
+    const uint32_t s = free_.back();
+    free_.pop_back();
+    used_[s] = 1;
+    return s;
+  }
+  bool release(uint32_t s) {   // false: the slot was not in use
+    if (s >= used_.size() || !used_[s]) return false;
+    used_[s] = 0;
+    free_.push_back(s);
+    return true;
+  }
+
+ private:
+  std::vector<uint8_t> used_;
+  std::vector<uint32_t> free_;
+};
+
 inline uint64_t mix64(uint64_t x) {
   x ^= x >> 32;
   x *= 0xD6E8FEB86659FD93ull;

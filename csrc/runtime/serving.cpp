@@ -54,6 +54,7 @@ struct Seq {
   uint32_t prefilled = 0;      // prompt tokens whose K/V are stored
   uint32_t prefix_hit = 0;
   uint32_t last_token = 0;     // next decode input
+  int64_t slot = -1;           // recurrent-state slot while running (models that have such state)
   bool greedy() const { return temp <= 0.f; }
 };
 
@@ -120,6 +121,7 @@ class Scheduler {
     } else if (s.state == RUNNING) {
       running_.erase(std::remove(running_.begin(), running_.end(), id), running_.end());
       s.table.release(alloc_);
+      release_slot(s);
     } else {
       return 0;
     }
@@ -221,6 +223,7 @@ class Scheduler {
       const uint32_t remaining = static_cast<uint32_t>(s.prompt.size()) - static_cast<uint32_t>(hit.size()) * cfg_.block_size;
       const uint32_t n = std::min(cfg_.max_prefill, remaining);
       if (any && n > budget) break;
+      if (slots_.size() && (s.slot = slots_.alloc()) < 0) break;
       waiting_.pop_front();
       s.table.adopt_prefix(hit, alloc_);
       s.prefix_hit = s.table.len;
@@ -321,6 +324,13 @@ class Scheduler {
 
   const Config& cfg() const { return cfg_; }
   BlockAllocator& alloc() { return alloc_; }
+  // Sequences of a model with recurrent state hold one slot each from admission to the end; the state
+  // at a prompt prefix is not kept, so such models run without the prefix cache.
+  void set_state_slots(uint32_t n) {
+    slots_ = kv::StateSlots(n);
+    if (n) cfg_.prefix_cache = 0;
+  }
+  uint32_t free_slots() const { return slots_.free_slots(); }
   PrefixCache& prefix() { return prefix_; }
   size_t n_waiting() const { return waiting_.size(); }
   size_t n_running() const { return running_.size(); }
@@ -350,8 +360,13 @@ class Scheduler {
     s.state = FINISHED;
     s.finish = why;
     s.table.release(alloc_);  // prompt blocks indexed by the prefix cache keep the cache's ref
+    release_slot(s);
     running_.erase(std::remove(running_.begin(), running_.end(), s.id), running_.end());
     ++finished_;
+  }
+  void release_slot(Seq& s) {
+    if (s.slot >= 0) slots_.release(static_cast<uint32_t>(s.slot));
+    s.slot = -1;
   }
   void push_token(Seq& s, uint32_t tok) {
     if (s.state != RUNNING) return;
@@ -368,6 +383,7 @@ class Scheduler {
   Config cfg_;
   BlockAllocator alloc_;
   PrefixCache prefix_;
+  kv::StateSlots slots_;
   std::unordered_map<int64_t, std::unique_ptr<Seq>> seqs_;
   std::deque<int64_t> waiting_;
   std::vector<int64_t> running_;
@@ -418,6 +434,12 @@ BBH_API int bbh_table_unshare_tail(void* t, void* a, uint32_t* old_b, uint32_t* 
 BBH_API void bbh_table_adopt_prefix(void* t, void* a, const uint32_t* blocks, uint32_t n) {
   static_cast<BlockTable*>(t)->adopt_prefix(std::vector<uint32_t>(blocks, blocks + n), *static_cast<BlockAllocator*>(a));
 }
+
+BBH_API void* bbh_slots_new(uint32_t n) { return new kv::StateSlots(n); }
+BBH_API void bbh_slots_free(void* s) { delete static_cast<kv::StateSlots*>(s); }
+BBH_API uint32_t bbh_slots_available(void* s) { return static_cast<kv::StateSlots*>(s)->free_slots(); }
+BBH_API int64_t bbh_slots_alloc(void* s) { return static_cast<kv::StateSlots*>(s)->alloc(); }
+BBH_API int bbh_slots_release(void* s, uint32_t i) { return static_cast<kv::StateSlots*>(s)->release(i) ? 0 : -1; }
 
 BBH_API void* bbh_prefix_new() { return new PrefixCache(); }
 BBH_API void bbh_prefix_free(void* p) { delete static_cast<PrefixCache*>(p); }
@@ -483,6 +505,18 @@ BBH_API void bbh_sched_decode_batch(void* s, int64_t* ids, int32_t* tokens, int3
     for (uint32_t b = 0; b < max_blocks; ++b)
       block_tables[i * max_blocks + b] = b < q.table.blocks.size() ? static_cast<int32_t>(q.table.blocks[b]) : -1;
   }
+}
+BBH_API void bbh_sched_set_state_slots(void* s, uint32_t n) { static_cast<Scheduler*>(s)->set_state_slots(n); }
+BBH_API uint32_t bbh_sched_free_slots(void* s) { return static_cast<Scheduler*>(s)->free_slots(); }
+BBH_API int64_t bbh_sched_seq_slot(void* s, int64_t id) {
+  Seq* q = static_cast<Scheduler*>(s)->get(id);
+  return q ? q->slot : -1;
+}
+// state slots of the decode batch, in its order
+BBH_API void bbh_sched_decode_slots(void* s, int32_t* slots) {
+  auto* sc = static_cast<Scheduler*>(s);
+  for (size_t i = 0; i < sc->decode_plan.size(); ++i)
+    slots[i] = static_cast<int32_t>(sc->get(sc->decode_plan[i])->slot);
 }
 BBH_API void bbh_sched_commit_prefill(void* s, int64_t id, uint32_t end, int has_token, uint32_t token) {
   static_cast<Scheduler*>(s)->commit_prefill(id, end, has_token, token);

@@ -1,0 +1,82 @@
+// Structures of the hybrid decoder's native forward (recurrent and attention layers with a parallel
+// feed-forward), shared by the layer sequence and its kernels and mirrored field for field by the
+// ctypes classes in brain_b200/serve/hybrid_native.py.
+//
+// Every matrix is stored with both extents padded to multiples of 8 (zero rows / columns), so the
+// sections of a fused projection start on 16-byte boundaries and padded columns are zero throughout.
+// dtype 0: bf16 activations, weights and K/V pages; dtype 1: fp32 throughout.
+#pragma once
+#include <cstdint>
+
+struct BbHyLin {
+  const void* w;   // [n, k]
+  int n, k;
+};
+
+struct BbHyLayer {
+  int kind;            // 0 attention, 1 mamba2
+  const float* norm;   // [dp] gain of the layer's norm (one already added where it is stored around 0)
+  BbHyLin in;          // every projection that reads the normed input, stacked along the rows
+  BbHyLin out;         // mixer output projection | feed-forward down projection, side by side
+  // feed-forward (ff = 0: none): columns of its halves in the projection and of its product in `cat`
+  int ff, off_gate, off_up, off_act;
+  float glu_limit, glu_alpha, glu_shift;
+  // attention
+  int hq, hk, dk, dv, dkp, dvp;            // true and padded head sizes
+  int off_q, off_k, off_v, off_g;          // columns of the projection
+  const float *q_norm, *k_norm;            // [hq dkp] / [hk dkp] gains of the whole-projection norm
+  const float *cos_t, *sin_t;              // [max_pos][rot / 2]
+  int rot;                                 // rotated leading dimensions of a head (0: none)
+  float scale, softcap;                    // softcap <= 0: none
+  float vmix;
+  int v_role;                              // 0 plain, 1 stores its values for later layers, 2 mixes them in
+  void *kc, *vc;                           // pages [blocks][hk][block_size][dkp | dvp]
+  // mamba2
+  int heads, p, n, groups, taps, norm_groups;
+  int inner, innerp, ch, chp;              // heads * p, padded; convolved channels, padded
+  int off_z, off_xbc, off_dt;
+  const float *conv_w, *conv_b;            // [taps][chp], [chp]
+  const float *dt_bias, *a, *d_skip;       // [heads]; a = -exp(A_log)
+  const float* gnorm;                      // [innerp]
+  void* conv_state;                        // [slots][max(taps - 1, 1)][chp]: raw inputs, position p at p % (taps - 1)
+  float* ssm_state;                        // [slots][heads][n][p]
+};
+
+struct BbHyCfg {
+  int dtype, width, dp, vocab, vocabp, n_layers, block_size;
+  float eps, residual_mult;
+  const void* embed;                       // [vocab, dp]
+  const float *embed_norm, *final_norm;    // [dp]
+  const void* head;                        // [vocabp, dp]
+  const BbHyLayer* layers;
+};
+
+// One packed batch: rows of prompt portions first (n_pre rows of ns_pre sequences), then one row for
+// every decoding sequence.
+struct BbHyBatch {
+  const int *tok, *pos, *row_seq;          // [n]
+  const int *seq_row0;                     // [ns + 1]
+  const int *seq_pos0, *seq_ctx, *seq_slot;  // [ns] first position, context after the step, state slot
+  const int* tables;                       // [ns, max_blocks]
+  const int *tile_seq, *tile_qt;           // 128-row query tiles of the prompt portions
+  const int *want;                         // [n_want] rows whose logits are asked for (null: every row)
+  int max_blocks, n, n_pre, ns, ns_pre, n_tiles, n_want, max_len;   // max_len: longest portion
+};
+
+struct BbHyWork {
+  float* x;          // [rows, dp] residual stream
+  void* h;           // [rows, dp]
+  void* proj;        // [rows, ld_proj]
+  void* cat;         // [rows, ld_cat]
+  void* xbc;         // [rows, ld_xbc]
+  float* dt;         // [rows, ld_dt]
+  void* y;           // [rows, ld_y]
+  void* v_first;     // [rows, ld_v]
+  float *part_o, *part_ml;   // decode attention partials
+  float* seg;        // chunked state-space scratch
+  long seg_floats;
+  void* hn;          // [want, dp]
+  float* logits;     // [want, vocabp]
+  int rows, want_rows, ld_proj, ld_cat, ld_xbc, ld_dt, ld_y, ld_v, splits;
+  int pool_blocks;
+};
