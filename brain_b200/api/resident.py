@@ -245,12 +245,12 @@ class _Job:
 
 
 class LlmResident(ResidentModel):
-    """A Qwen-family checkpoint behind a paged-KV engine and one continuous-batching scheduler."""
+    """A Qwen-family or hybrid checkpoint behind its paged-KV engine and one continuous-batching scheduler."""
 
     def __init__(self, model, tokenizer, model_id: str = "brain/qwen3", ctx: Optional[int] = None,
                  max_batch: Optional[int] = None, weights: str = "bf16", block_size: int = 16, tp=None,
                  kv_dtype: str = "bf16", kv_clip=None):
-        from ..serve.engine import QwenEngine
+        from ..serve.engine import make_engine
         from ..serve.scheduler import Scheduler
         self.id = model_id
         self.tok = tokenizer
@@ -259,9 +259,9 @@ class LlmResident(ResidentModel):
         self.max_batch = max_batch or int(os.environ.get("BRAIN_SCHED_MAX_BATCH", "16"))
         blocks_per_ctx = -(-self.ctx // block_size)
         pool = int(os.environ.get("BRAIN_SCHED_NUM_BLOCKS", "0")) or 2 * blocks_per_ctx + self.max_batch
-        self.engine = QwenEngine(model, block_size=block_size, num_blocks=pool, max_seq_len=self.ctx,
-                                 max_prefill=min(self.ctx, 512), weights=weights, tp=tp,
-                                 kv_dtype=kv_dtype, kv_clip=kv_clip)
+        self.engine = make_engine(model, max_batch=self.max_batch, block_size=block_size, num_blocks=pool,
+                                  max_seq_len=self.ctx, max_prefill=min(self.ctx, 512), weights=weights, tp=tp,
+                                  kv_dtype=kv_dtype, kv_clip=kv_clip)
         ids = tokenizer.encode("<|im_end|>") if hasattr(tokenizer, "special") else []
         self.eos = ids[0] if len(ids) == 1 else getattr(tokenizer, "eos_id", None)
         # One forward per step for prompt chunks + decode rows is the default on the GPU.  On the CPU
@@ -283,7 +283,8 @@ class LlmResident(ResidentModel):
 
     # ---- contract
     def manifest(self) -> Manifest:
-        return Manifest(self.id, "Qwen-family decoder served with paged KV and continuous batching",
+        kind = "Hybrid" if self.engine.state_slots else "Qwen-family"
+        return Manifest(self.id, f"{kind} decoder served with paged KV and continuous batching",
                         [generate_spec("chat / text generation")], self.ctx)
 
     def context_length(self):

@@ -703,10 +703,11 @@ class QwenEngine(PagedEngineBase):
         return self.head(h).float()
 
 
-def make_engine(model, **kw):
-    """The serving engine of a model: hybrid decoders (recurrent state slots, per-layer mixers) or the
-    dense Qwen family.  Options an engine does not know raise its own error."""
+def make_engine(model, max_batch: int = 16, **kw):
+    """The serving engine of a model: hybrid decoders (per-layer mixers, one recurrent-state slot for each
+    of ``max_batch`` running sequences) or the dense Qwen family."""
     if getattr(model, "family", "") == "hybrid":
         from .hybrid import HybridEngine
+        kw.setdefault("state_slots", max_batch)
         return HybridEngine(model, **kw)
     return QwenEngine(model, **kw)
