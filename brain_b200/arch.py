@@ -27,6 +27,8 @@ _ARCHS: List[Arch] = [
           "calib"), aliases=("qwen",)),
     Arch("toymoe", "moe", "Top-k routed mixture-of-experts decoder (toy and Qwen3-MoE shapes)",
          ("train", "infer", "eval"), aliases=("qwen3moe", "moe")),
+    Arch("pakalix", "hybrid", "Hybrid decoder: Mamba-2 and soft-capped attention layers, parallel feed-forward",
+         ("import", "infer", "serve", "trace"), aliases=("hybrid",)),
     Arch("splat", "splat", "3D Gaussian splat rasteriser (headless)", ("render", "train"), built=True),
 ]
 

@@ -213,7 +213,7 @@ def save_model(path: str, model, card: Optional[ModelCard] = None, dtype: str = 
     state = model.reference_state()
     if card is None:
         fam = getattr(model, "family", "qwen")
-        card = ModelCard(id={"gpt": "brain/gpt", "qwen": "brain/qwen3"}.get(fam, f"brain/{fam}"),
+        card = ModelCard(id={"gpt": "brain/gpt", "qwen": "brain/qwen3", "hybrid": "brain/pakalix"}.get(fam, f"brain/{fam}"),
                          family=fam, param_count=sum(t.numel() for t in state.values()),
                          capabilities=["generate"])
     save(path, state, model.config_json(), card, dtype)

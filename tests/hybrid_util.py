@@ -10,7 +10,7 @@ from brain_b200.models.hybrid import HybridDecoder
 import hybrid_oracle as oracle
 
 
-def attn(heads=6, kv_heads=2, dim=40, vdim=24, scale=0.2, softcap=30.0, rot=16, base=7000.0, v_mix=True):
+def attn(heads=6, kv_heads=2, dim=40, vdim=24, scale=0.2, softcap=5.0, rot=16, base=7000.0, v_mix=True):
     return AttentionSpec(heads, kv_heads, dim, vdim, scale, softcap, RotarySpec(rot, base) if rot else None, v_mix)
 
 
@@ -30,6 +30,10 @@ def make(layers, vocab=211, width=104, eps=1e-5, mult=0.6, seed=3, sharp=1.0):
     for n, t in m.reference_state().items():
         if n.endswith("q.norm"):
             t.mul_(sharp)
+        if n.endswith("A_log"):
+            t.sub_(3.0)          # slow decay and a small skip: what the state carries shows
+        if n.endswith("mix.D"):
+            t.mul_(0.2)
         t.copy_(t.to(torch.bfloat16).float())
     W = {n: t.numpy().astype(np.float64) for n, t in m.reference_state().items()}
     return m, W, cfg.to_json()
