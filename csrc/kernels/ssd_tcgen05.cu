@@ -1,0 +1,366 @@
+// State-space recurrence of prompt portions in chunks of 128 tokens on the tensor cores (bf16 inputs,
+// fp32 accumulation and state).  One CTA per (sequence, head) walks its portion chunk by chunk:
+//
+//   G = C B^T                                  128 x 128, K = state size
+//   Y = exp(cum_i) (C S)  +  W X               W_ij = G_ij exp(cum_i - cum_j) dt_j for j <= i, else 0
+//   S = exp(cum_last) S + B^T X'               X'_j = exp(cum_last - cum_j) dt_j x_j
+//   y_i = Y_i + D x_i
+//
+// with cum the running sum of a dt inside the chunk.  The state S lives in TMEM as an fp32 accumulator
+// from the first chunk to the last.  The operands that are not bf16 by nature - the weights W, the
+// scaled inputs X' and the state S as an operand - go through the tensor core as two bf16 terms each
+// (value and remainder, 16 bits of mantissa), so the recurrence keeps its 32-bit character.
+//
+// 256 threads: TMEM lane = token (or state row), two warpgroups share a row's columns.  Thread 0 issues
+// TMA and MMA.  The phases of a chunk are separated by block barriers; with head sizes up to 64 two CTAs
+// share an SM (113 KB of shared memory, 256 TMEM columns each) and fill each other's gaps.
+// TMEM: G, then W as packed bf16 (value in columns 0-63, remainder in 64-127) | Y | S.
+#include "../common/host.hpp"
+#include "../common/ptx.cuh"
+#include "../common/rows.cuh"
+#include "../serve/hybrid.hpp"
+
+namespace bb {
+
+constexpr int SSD_THREADS = 256;
+constexpr int SSD_SUB = 128 * 128;   // one swizzled sub-tile: 128 rows of 64 bf16
+
+template <int PP>
+struct SsdCfg {
+  static constexpr int PSUB = PP / 64;
+  static constexpr int OFF_C = 0;                               // 2 sub-tiles
+  static constexpr int OFF_B = OFF_C + 2 * SSD_SUB;             // 2
+  static constexpr int OFF_X = OFF_B + 2 * SSD_SUB;             // PSUB
+  static constexpr int OFF_S = OFF_X + PSUB * SSD_SUB;          // 2 PSUB: S as two terms, then X' as two terms
+  static constexpr int OFF_E = OFF_S + 2 * PSUB * SSD_SUB;      // 128 floats, 8 partial sums, barriers
+  static constexpr int SMEM = OFF_E + 1024;
+  static constexpr int COL_Y = 128, COL_S = 128 + PP;
+  static constexpr int TMEM_COLS = PP == 64 ? 256 : 512;
+};
+
+__device__ __forceinline__ float2 split_pair(float a, float b) {
+  // packed bf16 pair of the values, packed pair of what rounding left over
+  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  const float2 f = __bfloat1622float2(h);
+  const __nv_bfloat162 l = __floats2bfloat162_rn(a - f.x, b - f.y);
+  return make_float2(__uint_as_float(*reinterpret_cast<const uint32_t*>(&h)),
+                     __uint_as_float(*reinterpret_cast<const uint32_t*>(&l)));
+}
+
+// 32 fp32 values of row `row`, columns col0.. (a multiple of 8), as two bf16 terms into two swizzled tiles.
+__device__ __forceinline__ void store_split(uint8_t* hi, uint8_t* lo, int row, int col0, const float (&v)[32]) {
+#pragma unroll
+  for (int q = 0; q < 4; ++q) {
+    uint32_t h[4], l[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const float2 t = split_pair(v[q * 8 + 2 * k], v[q * 8 + 2 * k + 1]);
+      h[k] = __float_as_uint(t.x);
+      l[k] = __float_as_uint(t.y);
+    }
+    const int col = col0 + q * 8;
+    const int o = (col >> 6) * SSD_SUB + row * 128 + ((((col & 63) >> 3) ^ (row & 7)) << 4);
+    *reinterpret_cast<uint4*>(hi + o) = make_uint4(h[0], h[1], h[2], h[3]);
+    *reinterpret_cast<uint4*>(lo + o) = make_uint4(l[0], l[1], l[2], l[3]);
+  }
+}
+
+template <int PP>
+__global__ void __launch_bounds__(SSD_THREADS, PP == 64 ? 2 : 1)
+ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant__ CUtensorMap tmX,
+                 const __grid_constant__ BbHyLayer L, const float* __restrict__ dt, int lddt,
+                 __nv_bfloat16* __restrict__ y, int ldy, const __grid_constant__ BbHyBatch b, int* err) {
+  using Cfg = SsdCfg<PP>;
+  constexpr int PSUB = Cfg::PSUB, HC = PP / 2;   // HC: Y / S / X columns of a thread
+  extern __shared__ __align__(1024) uint8_t smem[];
+  uint8_t* sC = smem + Cfg::OFF_C;
+  uint8_t* sB = smem + Cfg::OFF_B;
+  uint8_t* sX = smem + Cfg::OFF_X;
+  uint8_t* sS = smem + Cfg::OFF_S;
+  uint8_t* sSl = sS + PSUB * SSD_SUB;
+  float* s_e = reinterpret_cast<float*>(smem + Cfg::OFF_E);   // [128]
+  float* s_part = s_e + 128;                                  // [8]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(s_part + 8);
+  uint64_t *b_tma = bars, *b_gy = bars + 1, *b_y = bars + 2, *b_s = bars + 3;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 4);
+
+  const int seq = blockIdx.x, h = blockIdx.y, grp = h / (L.heads / L.groups);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int row = (warp & 3) * 32 + lane, half = warp >> 2;
+  const uint32_t lane_sel = (uint32_t)((warp & 3) * 32) << 16;
+  const int r0 = b.seq_row0[seq], len = b.seq_row0[seq + 1] - r0, slot = b.seq_slot[seq];
+  const int n_chunks = (len + 127) / 128;
+  const int nsub = (L.n + 63) / 64, nk = (L.n + 15) / 16;
+  const float a2 = L.a[h] * 1.4426950408889634f, D = L.d_skip[h];
+  float* state = L.ssm_state + ((size_t)slot * L.heads + h) * L.n * L.p;
+
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < 4; ++i) mbar_init(bars + i, 1);
+    mbar_fence_init();
+  }
+  if (warp == 0) {
+    tmem_alloc(tmem_slot, Cfg::TMEM_COLS);
+    tmem_relinquish();
+  }
+  if (nsub == 1) {   // the state rows above 64 that the 128-row accumulator has anyway stay zero
+    for (int i = threadIdx.x; i < SSD_SUB / 16; i += SSD_THREADS)
+      reinterpret_cast<uint4*>(sB + SSD_SUB)[i] = make_uint4(0, 0, 0, 0);
+    fence_proxy_async_smem();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tm = *tmem_slot;
+  const uint32_t tG = tm + lane_sel, tY = tm + Cfg::COL_Y + lane_sel + half * HC, tS = tm + Cfg::COL_S + lane_sel + half * HC;
+  // the state so far, one row of it per lane
+  {
+    const bool fresh = b.seq_pos0[seq] == 0 || row >= L.n;
+#pragma unroll
+    for (int c = 0; c < HC; c += 32) {
+      uint32_t r[32];
+#pragma unroll
+      for (int j = 0; j < 32; ++j) {
+        const int p = half * HC + c + j;
+        r[j] = fresh || p >= L.p ? 0u : __float_as_uint(state[(size_t)row * L.p + p]);
+      }
+      tmem_st32(tS + c, r);
+    }
+    tmem_wait_st();
+  }
+
+  bool ok = (smem_u32(smem) & 1023u) == 0;
+  if (!ok && threadIdx.x == 0) set_error(err, ERR_BAD_ARG);
+  for (int ch = 0; ch < n_chunks && ok; ++ch) {
+    const uint32_t ph = ch & 1;
+    const int c0 = r0 + ch * 128, valid = min(128, len - ch * 128);
+    if (threadIdx.x == 0) {
+      mbar_expect_tx(b_tma, (2 * nsub + PSUB) * SSD_SUB);
+      for (int s = 0; s < nsub; ++s) {
+        tma_load_3d(sC + s * SSD_SUB, &tmBC, b_tma, s * 64, c0, L.groups + grp);
+        tma_load_3d(sB + s * SSD_SUB, &tmBC, b_tma, s * 64, c0, grp);
+      }
+      for (int s = 0; s < PSUB; ++s) tma_load_3d(sX + s * SSD_SUB, &tmX, b_tma, s * 64, c0, h);
+    }
+    __syncwarp();
+    // step sizes and their running sum (log2 units); both warpgroups scan the same 128 tokens
+    const float d = row < valid ? dt[(size_t)(c0 + row) * lddt + h] : 0.f;
+    float cum = a2 * d;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float v = __shfl_up_sync(0xffffffffu, cum, o);
+      if (lane >= o) cum += v;
+    }
+    if (lane == 31) s_part[warp] = cum;
+    __syncthreads();
+    for (int w = 0; w < (warp & 3); ++w) cum += s_part[half * 4 + w];
+    const float total = (s_part[0] + s_part[1]) + (s_part[2] + s_part[3]);
+    if (half == 0) s_e[row] = d > 0.f ? cum - log2f(d) : INFINITY;   // W_ij = G_ij 2^(cum_i - e_j)
+    // the state as an operand (two terms), and scaled for the accumulation that follows
+    {
+      const float dec = exp2f(total);
+#pragma unroll
+      for (int c = 0; c < HC; c += 32) {
+        uint32_t r[32];
+        float v[32];
+        tmem_ld32(tS + c, r);
+        tmem_wait_ld();
+#pragma unroll
+        for (int j = 0; j < 32; ++j) {
+          v[j] = __uint_as_float(r[j]);
+          r[j] = __float_as_uint(v[j] * dec);
+        }
+        tmem_st32(tS + c, r);
+        store_split(sS, sSl, row, half * HC + c, v);
+      }
+      tmem_wait_st();
+    }
+    fence_proxy_async_smem();
+    tc_fence_before();
+    ok = mbar_wait(b_tma, ph);
+    ok = __syncthreads_and(ok);
+    if (!ok) {
+      if (threadIdx.x == 0) set_error(err, ERR_WAIT_MMA_FULL);
+      break;
+    }
+    if (threadIdx.x == 0) {
+      tc_fence_after();
+      constexpr uint32_t id_g = umma_idesc(1, 1, 1, 0, 0, 128, 128), id_y = umma_idesc(1, 1, 1, 0, 1, 128, PP);
+      const uint32_t aC = smem_u32(sC), aB = smem_u32(sB), aS = smem_u32(sS), aSl = smem_u32(sSl);
+      for (int t = 0; t < nk; ++t) {
+        const uint32_t o = (t / 4) * SSD_SUB + (t % 4) * 32;
+        umma_f16_ss(tm, umma_smem_desc(aC + o, 16, 1024), umma_smem_desc(aB + o, 16, 1024), id_g, t != 0);
+      }
+      for (int t = 0; t < nk; ++t) {
+        const uint32_t o = (t / 4) * SSD_SUB + (t % 4) * 32;
+        umma_f16_ss(tm + Cfg::COL_Y, umma_smem_desc(aC + o, 16, 1024), umma_smem_desc(aS + t * 2048, SSD_SUB, 1024), id_y,
+                    t != 0);
+        umma_f16_ss(tm + Cfg::COL_Y, umma_smem_desc(aC + o, 16, 1024), umma_smem_desc(aSl + t * 2048, SSD_SUB, 1024), id_y, 1);
+      }
+      umma_commit(b_gy);
+    }
+    __syncwarp();
+    ok = mbar_wait(b_gy, ph);
+    tc_fence_after();
+    __syncwarp();
+    // scores of this thread's 64 columns into registers before any thread writes weights over them
+    uint32_t g0[32], g1[32];
+    tmem_ld32(tG + half * 64, g0);
+    tmem_ld32(tG + half * 64 + 32, g1);
+    tmem_wait_ld();
+    tc_fence_before();
+    ok = __syncthreads_and(ok);
+    if (!ok) {
+      if (threadIdx.x == 0) set_error(err, ERR_WAIT_EPILOGUE);
+      break;
+    }
+    tc_fence_after();
+    {
+      const float* e = s_e + half * 64;
+      const int lim = row - half * 64;   // columns j <= lim are in the past
+      uint32_t hi[32], lo[32];
+#pragma unroll
+      for (int j = 0; j < 32; j += 2) {
+        const float a0 = j <= lim ? __uint_as_float(g0[j]) * exp2f(cum - e[j]) : 0.f;
+        const float a1 = j + 1 <= lim ? __uint_as_float(g0[j + 1]) * exp2f(cum - e[j + 1]) : 0.f;
+        const float2 s = split_pair(a0, a1);
+        hi[j >> 1] = __float_as_uint(s.x);
+        lo[j >> 1] = __float_as_uint(s.y);
+      }
+#pragma unroll
+      for (int j = 0; j < 32; j += 2) {
+        const float a0 = j + 32 <= lim ? __uint_as_float(g1[j]) * exp2f(cum - e[j + 32]) : 0.f;
+        const float a1 = j + 33 <= lim ? __uint_as_float(g1[j + 1]) * exp2f(cum - e[j + 33]) : 0.f;
+        const float2 s = split_pair(a0, a1);
+        hi[16 + (j >> 1)] = __float_as_uint(s.x);
+        lo[16 + (j >> 1)] = __float_as_uint(s.y);
+      }
+      tmem_st32(tG + half * 32, hi);
+      tmem_st32(tG + 64 + half * 32, lo);
+    }
+    {
+      const float sc = exp2f(cum), w = d * exp2f(total - cum);
+#pragma unroll
+      for (int c = 0; c < HC; c += 32) {
+        uint32_t r[32];
+        tmem_ld32(tY + c, r);
+        tmem_wait_ld();
+#pragma unroll
+        for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * sc);
+        tmem_st32(tY + c, r);
+        float v[32];
+        const int col0 = half * HC + c;
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          const int col = col0 + q * 8;
+          float f[8];
+          unpack8(*reinterpret_cast<const bf16x8*>(sX + (col >> 6) * SSD_SUB + row * 128 +
+                                                   ((((col & 63) >> 3) ^ (row & 7)) << 4)), f);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) v[q * 8 + j] = f[j] * w;
+        }
+        store_split(sS, sSl, row, col0, v);   // the state operand is behind its products
+      }
+    }
+    tmem_wait_st();
+    fence_proxy_async_smem();
+    tc_fence_before();
+    __syncthreads();
+    if (threadIdx.x == 0) {
+      tc_fence_after();
+      constexpr uint32_t id_y = umma_idesc(1, 1, 1, 0, 1, 128, PP), id_s = umma_idesc(1, 1, 1, 1, 1, 128, PP);
+      const uint32_t aB = smem_u32(sB), aX = smem_u32(sX), aW = smem_u32(sS), aWl = smem_u32(sSl);
+#pragma unroll
+      for (int t = 0; t < 8; ++t) {
+        umma_f16_ts(tm + Cfg::COL_Y, tm + t * 8, umma_smem_desc(aX + t * 2048, SSD_SUB, 1024), id_y, 1);
+        umma_f16_ts(tm + Cfg::COL_Y, tm + 64 + t * 8, umma_smem_desc(aX + t * 2048, SSD_SUB, 1024), id_y, 1);
+      }
+      umma_commit(b_y);
+#pragma unroll
+      for (int t = 0; t < 8; ++t) {
+        const uint64_t da = umma_smem_desc(aB + t * 2048, SSD_SUB, 1024);
+        umma_f16_ss(tm + Cfg::COL_S, da, umma_smem_desc(aW + t * 2048, SSD_SUB, 1024), id_s, 1);
+        umma_f16_ss(tm + Cfg::COL_S, da, umma_smem_desc(aWl + t * 2048, SSD_SUB, 1024), id_s, 1);
+      }
+      umma_commit(b_s);
+    }
+    __syncwarp();
+    ok = mbar_wait(b_y, ph);
+    tc_fence_after();
+    __syncwarp();
+    __nv_bfloat16* yr = y + (size_t)(c0 + row) * ldy + h * L.p;
+#pragma unroll
+    for (int c = 0; c < HC; c += 32) {
+      uint32_t r[32];
+      tmem_ld32(tY + c, r);
+      tmem_wait_ld();
+      const int col0 = half * HC + c;
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const int col = col0 + q * 8;
+        float f[8];
+        unpack8(*reinterpret_cast<const bf16x8*>(sX + (col >> 6) * SSD_SUB + row * 128 +
+                                                 ((((col & 63) >> 3) ^ (row & 7)) << 4)), f);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) f[j] = fmaf(D, f[j], __uint_as_float(r[q * 8 + j]));
+        if (ok && row < valid && col < L.p) store8(yr + col, f);
+      }
+    }
+    ok = mbar_wait(b_s, ph) && ok;
+    tc_fence_after();
+    ok = __syncthreads_and(ok);   // every tile and the accumulators are free for the next chunk
+    if (!ok && threadIdx.x == 0) set_error(err, ERR_WAIT_EPILOGUE);
+  }
+  __syncwarp();
+  if (ok) {
+#pragma unroll
+    for (int c = 0; c < HC; c += 32) {
+      uint32_t r[32];
+      tmem_ld32(tS + c, r);
+      tmem_wait_ld();
+      if (row < L.n) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) {
+          const int p = half * HC + c + j;
+          if (p < L.p) state[(size_t)row * L.p + p] = __uint_as_float(r[j]);
+        }
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 0) {
+    tc_fence_after();
+    tmem_dealloc(tm, Cfg::TMEM_COLS);
+  }
+}
+
+template <int PP>
+static int launch_ssd(const CUtensorMap& tmBC, const CUtensorMap& tmX, const BbHyLayer& L, const BbHyWork& w,
+                      const BbHyBatch& b, cudaStream_t s) {
+  static PerDeviceOnce once;
+  const cudaError_t e = ensure_dyn_smem(once, ssd_chunk_kernel<PP>, SsdCfg<PP>::SMEM);
+  if (e != cudaSuccess) return (int)e;
+  ssd_chunk_kernel<PP><<<dim3(b.ns_pre, L.heads), SSD_THREADS, SsdCfg<PP>::SMEM, s>>>(
+      tmBC, tmX, L, w.dt, w.ld_dt, static_cast<__nv_bfloat16*>(w.y), w.ld_y, b, device_error_word());
+  return (int)cudaGetLastError();
+}
+
+}  // namespace bb
+
+// Prompt portions of one layer, bf16; BB_ESIZE for sizes it does not cover (the caller then runs the
+// token-by-token scan): head and state sizes are multiples of 8 up to 128.
+BB_API int bb_ssd_chunk(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream) {
+  using namespace bb;
+  if (b->ns_pre <= 0) return BB_OK;
+  if (c->dtype || L->n % 8 || L->p % 8 || L->n > 128 || L->p > 128) return BB_ESIZE;
+  const __nv_bfloat16* xbc = static_cast<const __nv_bfloat16*>(w->xbc);
+  const uint64_t ld = (uint64_t)w->ld_xbc * 2;
+  CUtensorMap tmBC, tmX;
+  const CUtensorMapDataType bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+  int rc = make_tmap_3d(&tmBC, bf, 2, xbc + L->inner, L->n, b->n_pre, 2 * L->groups, ld, (uint64_t)L->n * 2, 64, 128);
+  if (rc) return rc;
+  rc = make_tmap_3d(&tmX, bf, 2, xbc, L->p, b->n_pre, L->heads, ld, (uint64_t)L->p * 2, 64, 128);
+  if (rc) return rc;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return L->p <= 64 ? launch_ssd<64>(tmBC, tmX, *L, *w, *b, s) : launch_ssd<128>(tmBC, tmX, *L, *w, *b, s);
+}

@@ -26,6 +26,7 @@ int bb_hy_attn_post(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, con
 int bb_hy_mamba_post(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
 int bb_hy_conv(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
 int bb_hy_ssm_scan(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_ssd_chunk(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
 int bb_hy_ssm_decode(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
 int bb_attn_rows(int dtype, const void* q, int ldq, const void* kc, const void* vc, const int* pos, const int* row_seq,
                  const int* tables, int max_blocks, int bs, void* out, int ldo, const void* gate, int ldg, int rows, int hq,
@@ -111,7 +112,9 @@ int attention(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbH
 int mamba2(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
   if (b.n_pre > 0) {
     BB_TRY(bb_hy_conv(&c, &L, &w, &b, s));
-    BB_TRY(bb_hy_ssm_scan(&c, &L, &w, &b, s));
+    const int rc = bb_ssd_chunk(&c, &L, &w, &b, s);
+    if (rc == BB_ESIZE) BB_TRY(bb_hy_ssm_scan(&c, &L, &w, &b, s));   // fp32, or sizes the tiles do not cover
+    else if (rc) return rc;
   }
   BB_TRY(bb_hy_ssm_decode(&c, &L, &w, &b, s));
   return bb_hy_mamba_post(&c, &L, &w, &b, s);
