@@ -171,3 +171,46 @@ def test_fp32_argmax_and_topk():
     idx, val = F.topk_rows(view, 20)
     tv = torch.topk(lg[:, :1000], 20).values
     assert torch.equal(val.cpu(), tv) and idx[0, :2].cpu().tolist() == [77, 900]
+
+
+@pytest.mark.parametrize("H,P,N,G", [(4, 64, 128, 1), (2, 128, 128, 2), (6, 16, 24, 3), (3, 40, 64, 1), (2, 72, 72, 1),
+                                     (8, 32, 8, 4), (5, 8, 120, 5)])
+def test_chunked_recurrence_keeps_fp32_state(H, P, N, G):
+    """The tensor-core chunks against the token-by-token fp32 scan on the same bf16 inputs: portions of
+    many lengths, from zero and from carried states, in slots that hold something else."""
+    import ctypes as C
+    from brain_b200.ops._cuda import check_error, lib, stream_ptr
+    from brain_b200.serve import hybrid_native as hn
+    g = torch.Generator().manual_seed(H * P + N)
+    lens, starts = [2, 300, 128, 129, 15, 256, 7], [0, 0, 5, 640, 64, 128, 0]
+    ns, n = len(lens), sum(lens)
+    inner, ch = H * P, H * P + 2 * G * N
+    ldx = (ch + 7) // 8 * 8 + 8
+    xbc = torch.randn(n, ldx, generator=g).to("cuda", torch.bfloat16)
+    dt = torch.nn.functional.softplus(torch.randn(n, H, generator=g) - 1.0).cuda()
+    a = -torch.exp(torch.rand(H, generator=g) * 5 - 4).cuda()
+    d = torch.randn(H, generator=g).cuda()
+    init = torch.randn(ns + 2, H, N, P, generator=g).cuda()
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device="cuda")
+    row0, pos0 = i32(np.concatenate([[0], np.cumsum(lens)]).tolist()), i32(starts)
+    slots = i32([3, 1, 0, 5, 8, 2, 4])
+    cfg, L, b, w = hn.Cfg(), hn.Layer(), hn.Batch(), hn.Work()
+    L.heads, L.p, L.n, L.groups, L.inner, L.ch = H, P, N, G, inner, ch
+    L.a, L.d_skip = a.data_ptr(), d.data_ptr()
+    b.seq_row0, b.seq_pos0, b.seq_slot, b.n_pre, b.ns_pre, b.ns, b.n = \
+        row0.data_ptr(), pos0.data_ptr(), slots.data_ptr(), n, ns, ns, n
+    w.xbc, w.ld_xbc, w.dt, w.ld_dt, w.ld_y = xbc.data_ptr(), ldx, dt.data_ptr(), H, inner
+    out = {}
+    for name in ("bb_ssd_chunk", "bb_hy_ssm_scan"):
+        y, st = torch.zeros(n, inner, device="cuda", dtype=torch.bfloat16), init.clone()
+        L.ssm_state, w.y = st.data_ptr(), y.data_ptr()
+        assert getattr(lib(), name)(C.byref(cfg), C.byref(L), C.byref(w), C.byref(b), stream_ptr()) == 0
+        check_error()
+        out[name] = (y.float().cpu(), st.cpu())
+    (y1, s1), (y2, s2) = out["bb_ssd_chunk"], out["bb_hy_ssm_scan"]
+    assert (s1 - s2).abs().max() < 3e-5 * s2.abs().max()
+    untouched = [i for i in range(ns + 2) if i not in slots.tolist()]
+    assert torch.equal(s1[untouched], init.cpu()[untouched])
+    assert (y1 - y2).abs().max() < 2 ** -7 * y2.abs().max()
+    # two roundings of the same value to bf16: almost every output is bit-equal
+    assert (y1 != y2).float().mean() < 0.02
