@@ -248,6 +248,13 @@ class HybridEngine(PagedEngineBase):
     def _step(self, entries: Sequence[Entry], trace: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Run one packed step; fp32 logits [wanted, vocab] on the device in entry order (a view of step
         buffers: valid until the next step)."""
+        sc, b, blob = self._prepare(entries)
+        out = self._run(sc, b, trace)
+        self._last_blob = blob        # stays alive until the step's kernels are behind the next one
+        return out
+
+    def _prepare(self, entries: Sequence[Entry]):
+        """Check and pack a step: (step buffers, batch structure, the device memory it points into)."""
         # portions first, single tokens after them: the latter take the decode kernels
         order = [i for i, e in enumerate(entries) if len(e.tokens) > 1]
         ns_pre = len(order)
@@ -299,9 +306,7 @@ class HybridEngine(PagedEngineBase):
         b.n_tiles, b.n_want, b.max_len = len(tiles), len(want), max(lens[:ns_pre], default=0)
         up = lambda v, q: -(-v // q) * q
         sc = self._scratch_for("step", up(n, 256), up(len(want), 16), up(ns - ns_pre, 16) if ns > ns_pre else 0)
-        out = self._run(sc, b, trace)
-        self._last_blob = d_blob      # stays alive until the step's kernels are behind the next one
-        return out
+        return sc, b, d_blob
 
     @torch.no_grad()
     def step_logits(self, entries: Sequence[Entry]) -> torch.Tensor:
