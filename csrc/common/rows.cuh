@@ -50,11 +50,26 @@ __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
+// Activations whose result is stored as T: with bf16 the exponential and the division are the hardware's
+// approximations (2^-22, far below the rounding that follows), with fp32 they are exact.
+template <typename T>
+__device__ __forceinline__ float sigmoid_as(float x) {
+  if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-x));
+  else return sigmoid_f(x);
+}
+template <typename T>
+__device__ __forceinline__ float silu_as(float x) {
+  // (an argument of the fast division above 2^126 gives 0, which is silu's limit there)
+  if constexpr (sizeof(T) == 2) return __fdividef(x, 1.f + __expf(-x));
+  else return silu_f(x);
+}
+
 // Clamped gated unit: g' = min(g, limit), u' = clamp(u, +-limit); g' sigmoid(alpha g') (u' + shift).
-__device__ __forceinline__ float clamped_glu_f(float g, float u, float limit, float alpha, float shift) {
+template <typename T>
+__device__ __forceinline__ float clamped_glu_as(float g, float u, float limit, float alpha, float shift) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
-  return g * sigmoid_f(alpha * g) * (u + shift);
+  return g * sigmoid_as<T>(alpha * g) * (u + shift);
 }
 
 }  // namespace bb

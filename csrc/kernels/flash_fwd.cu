@@ -44,9 +44,28 @@ struct FaFwdArgs {
   // Extended form (EXT): K and V heads of their own sizes, soft-capped scores, per-head output gate.
   int dq, dv;                // columns of a query / value head in memory (a tile's other columns are not its own)
   float cap_in, cap_log2;    // scores become cap_log2 tanh(cap_in q.k) (log2 domain); cap_log2 = 0: no cap
+  float cap_poly[6];         // ... as an odd polynomial in q.k itself, for |cap_in q.k| < 0.4
   const __nv_bfloat16* gate; // raw gate of row r, head h at gate[r ldg + h]; the output is multiplied by its
   int ldg;                   // sigmoid; may be null
 };
+
+// s <- s (c0 + s^2 (c1 + s^2 (...))) for two scores with packed fp32 arithmetic.
+__device__ __forceinline__ void cap_pair(uint32_t& x, uint32_t& y, const float (&c)[6]) {
+  asm("{\n\t.reg .b64 s, q, p, k;\n\t"
+      "mov.b64 s, {%0, %1};\n\t"
+      "mul.rn.f32x2 q, s, s;\n\t"
+      "mov.b64 p, {%7, %7};\n\t"
+      "mov.b64 k, {%6, %6};\n\tfma.rn.f32x2 p, p, q, k;\n\t"
+      "mov.b64 k, {%5, %5};\n\tfma.rn.f32x2 p, p, q, k;\n\t"
+      "mov.b64 k, {%4, %4};\n\tfma.rn.f32x2 p, p, q, k;\n\t"
+      "mov.b64 k, {%3, %3};\n\tfma.rn.f32x2 p, p, q, k;\n\t"
+      "mov.b64 k, {%2, %2};\n\tfma.rn.f32x2 p, p, q, k;\n\t"
+      "mul.rn.f32x2 s, s, p;\n\t"
+      "mov.b64 {%0, %1}, s;\n\t}"
+      : "+r"(x), "+r"(y)
+      : "r"(__float_as_uint(c[0])), "r"(__float_as_uint(c[1])), "r"(__float_as_uint(c[2])), "r"(__float_as_uint(c[3])),
+        "r"(__float_as_uint(c[4])), "r"(__float_as_uint(c[5])));
+}
 
 template <int HD, int HDV = HD>
 struct FaFwdCfg {
@@ -565,9 +584,9 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
         const float ci = args.cap_in, co = args.cap_log2;
         if (!__any_sync(0xffffffffu, fmaxf(am, am2) * ci >= 0.4f)) {
 #pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            r0[i] = __float_as_uint(co * tanh_small(__uint_as_float(r0[i]) * ci));
-            r1[i] = __float_as_uint(co * tanh_small(__uint_as_float(r1[i]) * ci));
+          for (int i = 0; i < 32; i += 2) {
+            cap_pair(r0[i], r0[i + 1], args.cap_poly);
+            cap_pair(r1[i], r1[i + 1], args.cap_poly);
           }
         } else {
 #pragma unroll
@@ -858,6 +877,10 @@ BB_API int bb_flash_fwd_paged_x(const void* q, int ldq, const void* k_pool, cons
   if (softcap > 0.f) {
     a.cap_in = scale / softcap;
     a.cap_log2 = softcap * 1.4426950408889634f;
+    // Taylor coefficients of tanh up to u^11 (truncation 6e-8 relative at u = 0.4)
+    static const double taylor[6] = {1.0, -1.0 / 3, 2.0 / 15, -17.0 / 315, 62.0 / 2835, -1382.0 / 155925};
+    double u = (double)scale / softcap, f = (double)softcap * 1.4426950408889634 * u;
+    for (int k = 0; k < 6; ++k, f *= u * u) a.cap_poly[k] = (float)(f * taylor[k]);
   }
   a.gate = static_cast<const __nv_bfloat16*>(gate);
   a.ldg = ldg;

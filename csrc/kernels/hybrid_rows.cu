@@ -92,17 +92,20 @@ hy_norm_kernel(const float* __restrict__ x, const int* __restrict__ rows, const 
   }
 }
 
+// Blocks of a "post" launch: blockIdx.y = 0 is the row's mixer part, every further one GLU_COLS columns of
+// its feed-forward product.
+constexpr int GLU_COLS = ROW_THREADS * 8;
+
 template <typename T>
-__device__ __forceinline__ void glu_row(const BbHyLayer& L, const T* row, T* crow) {
-  const int n = (L.ff + 7) & ~7;
-  for (int i = threadIdx.x * 8; i < n; i += blockDim.x * 8) {
-    float g[8], u[8];
-    load8(row + L.off_gate + i, g);
-    load8(row + L.off_up + i, u);
+__device__ __forceinline__ void glu_part(const BbHyLayer& L, const T* row, T* crow) {
+  const int i = (blockIdx.y - 1) * GLU_COLS + threadIdx.x * 8;
+  if (i >= ((L.ff + 7) & ~7)) return;
+  float g[8], u[8];
+  load8(row + L.off_gate + i, g);
+  load8(row + L.off_up + i, u);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) g[j] = clamped_glu_f(g[j], u[j], L.glu_limit, L.glu_alpha, L.glu_shift);
-    store8(crow + L.off_act + i, g);
-  }
+  for (int j = 0; j < 8; ++j) g[j] = clamped_glu_as<T>(g[j], u[j], L.glu_limit, L.glu_alpha, L.glu_shift);
+  store8(crow + L.off_act + i, g);
 }
 
 template <typename T>
@@ -110,57 +113,71 @@ __global__ void __launch_bounds__(ROW_THREADS)
 hy_attn_post_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, int ld, T* __restrict__ cat, int ldc,
                     T* __restrict__ v_first, int ldv, const int* __restrict__ pos_, const int* __restrict__ row_seq,
                     const int* __restrict__ tables, int max_blocks, int bs, float eps) {
-  extern __shared__ float s_row[];   // q | k of the row
+  extern __shared__ __align__(16) float s_row[];   // q | k of the row, times their gains
   __shared__ float buf[2][32];
   const int r = blockIdx.x;
   T* row = proj + (size_t)r * ld;
+  if (blockIdx.y > 0) {
+    glu_part(L, row, cat + (size_t)r * ldc);
+    return;
+  }
   const int nq = L.hq * L.dkp, nk = L.hk * L.dkp, nv = L.hk * L.dvp;
   float ssq = 0.f, ssk = 0.f;
-  for (int i = threadIdx.x * 8; i < nq + nk; i += blockDim.x * 8) {
-    float f[8];
+  for (int i = threadIdx.x * 8; i < nq + nk; i += ROW_THREADS * 8) {
+    float f[8], g[8];
     const bool is_q = i < nq;
     load8(is_q ? row + L.off_q + i : row + L.off_k + (i - nq), f);
+    load8(is_q ? L.q_norm + i : L.k_norm + (i - nq), g);
     float s = 0.f;
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       s += f[j] * f[j];
-      s_row[i + j] = f[j];
+      g[j] *= f[j];
     }
+    store8(s_row + i, g);
     if (is_q) ssq += s; else ssk += s;
   }
+  const int pos = pos_[r], seq = row_seq[r];
+  const int blk = tables[(size_t)seq * max_blocks + pos / bs], off = pos % bs;
   ssq = block_sum(ssq, buf[0]);
   ssk = block_sum(ssk, buf[1]);    // (its barrier also orders the row in shared memory)
   const float rq = 1.f / sqrtf(ssq / (float)(L.hq * L.dk) + eps);
   const float rk = 1.f / sqrtf(ssk / (float)(L.hk * L.dk) + eps);
-  for (int i = threadIdx.x; i < nq + nk; i += blockDim.x)
-    s_row[i] *= i < nq ? rq * L.q_norm[i] : rk * L.k_norm[i - nq];
-  __syncthreads();
-  const int pos = pos_[r], seq = row_seq[r];
-  const int blk = tables[(size_t)seq * max_blocks + pos / bs], off = pos % bs;
   const int half = L.rot >> 1;
   const float* ct = L.cos_t + (size_t)pos * half;
   const float* st = L.sin_t + (size_t)pos * half;
   T* kc = static_cast<T*>(L.kc);
   T* vc = static_cast<T*>(L.vc);
-  for (int i = threadIdx.x * 8; i < nq + nk; i += blockDim.x * 8) {
-    const int d0 = i % L.dkp;
+  for (int i = threadIdx.x * 8; i < nq + nk; i += ROW_THREADS * 8) {
+    const bool is_q = i < nq;
+    const int h = (is_q ? i : i - nq) / L.dkp, d0 = (is_q ? i : i - nq) - h * L.dkp;
+    const float rs = is_q ? rq : rk;
     float f[8];
+    load8(s_row + i, f);
+    if ((half & 7) == 0) {           // a vector lies in one half of the rotated part, or past it
+      if (d0 < L.rot) {
+        const bool lo = d0 < half;
+        float g[8], c[8], sn[8];
+        load8(s_row + (lo ? i + half : i - half), g);
+        load8(ct + (lo ? d0 : d0 - half), c);
+        load8(st + (lo ? d0 : d0 - half), sn);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      const int d = d0 + j, e = i + j;
-      float v = s_row[e];
-      if (d < half) v = v * ct[d] - s_row[e + half] * st[d];
-      else if (d < L.rot) v = v * ct[d - half] + s_row[e - half] * st[d - half];
-      f[j] = v;
-    }
-    if (i < nq) {
-      store8(row + L.off_q + i, f);
+        for (int j = 0; j < 8; ++j) f[j] = lo ? f[j] * c[j] - g[j] * sn[j] : f[j] * c[j] + g[j] * sn[j];
+      }
     } else {
-      const int h = (i - nq) / L.dkp;
-      store8(kc + (((size_t)blk * L.hk + h) * bs + off) * L.dkp + d0, f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const int d = d0 + j, e = i + j;
+        if (d < half) f[j] = f[j] * ct[d] - s_row[e + half] * st[d];
+        else if (d < L.rot) f[j] = f[j] * ct[d - half] + s_row[e - half] * st[d - half];
+      }
     }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) f[j] *= rs;
+    if (is_q) store8(row + L.off_q + i, f);
+    else store8(kc + (((size_t)blk * L.hk + h) * bs + off) * L.dkp + d0, f);
   }
-  for (int i = threadIdx.x * 8; i < nv; i += blockDim.x * 8) {
+  for (int i = threadIdx.x * 8; i < nv; i += ROW_THREADS * 8) {
     float f[8];
     load8(row + L.off_v + i, f);
     T* vf = v_first + (size_t)r * ldv + i;
@@ -171,10 +188,9 @@ hy_attn_post_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, i
 #pragma unroll
       for (int j = 0; j < 8; ++j) f[j] = (1.f - L.vmix) * f[j] + L.vmix * g[j];
     }
-    const int h = i / L.dvp, d0 = i % L.dvp;
+    const int h = i / L.dvp, d0 = i - h * L.dvp;
     store8(vc + (((size_t)blk * L.hk + h) * bs + off) * L.dvp + d0, f);
   }
-  if (L.ff) glu_row(L, row, cat + (size_t)r * ldc);
 }
 
 template <typename T>
@@ -183,17 +199,22 @@ hy_mamba_post_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
                      int ldy, T* __restrict__ cat, int ldc, const int* __restrict__ pos_,
                      const int* __restrict__ row_seq, const int* __restrict__ seq_ctx,
                      const int* __restrict__ seq_slot, float eps) {
-  extern __shared__ float s_row[];   // gated row, then one 1/rms per part
+  extern __shared__ __align__(16) float s_row[];   // gated row, then one 1/rms per part
   float* s_rstd = s_row + L.innerp;
   __shared__ float part[ROW_THREADS / 32];
   const int r = blockIdx.x;
   const T* row = proj + (size_t)r * ld;
+  if (blockIdx.y > 0) {
+    glu_part(L, row, cat + (size_t)r * ldc);
+    return;
+  }
   for (int i = threadIdx.x * 8; i < L.innerp; i += blockDim.x * 8) {
     float f[8], z[8];
     load8(y + (size_t)r * ldy + i, f);
     load8(row + L.off_z + i, z);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) s_row[i + j] = i + j < L.inner ? f[j] * silu_f(z[j]) : 0.f;
+    for (int j = 0; j < 8; ++j) f[j] = i + j < L.inner ? f[j] * silu_as<T>(z[j]) : 0.f;
+    store8(s_row + i, f);
   }
   __syncthreads();
   // one root mean square per part: with few parts several warps share one, with many a warp takes several
@@ -204,7 +225,13 @@ hy_mamba_post_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
     const int g = g0 + warp / per, sub = warp % per;
     float s = 0.f;
     if (g < ng && warp < (nw / per) * per)
-      for (int i = sub * 32 + lane; i < len; i += per * 32) s += s_row[g * len + i] * s_row[g * len + i];
+      if ((len & 3) == 0)
+        for (int i = (sub * 32 + lane) * 4; i < len; i += per * 128) {
+          const float4 v = *reinterpret_cast<const float4*>(s_row + g * len + i);
+          s += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+        }
+      else
+        for (int i = sub * 32 + lane; i < len; i += per * 32) s += s_row[g * len + i] * s_row[g * len + i];
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
     if (lane == 0) part[warp] = s;
@@ -219,11 +246,15 @@ hy_mamba_post_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
   T* crow = cat + (size_t)r * ldc;
   for (int i = threadIdx.x * 8; i < L.innerp; i += blockDim.x * 8) {
     float f[8], w[8];
-    load8(L.gnorm + i, w);
+    load8(L.gnorm + i, w);           // zero past the last channel
+    load8(s_row + i, f);
+    if ((len & 7) == 0) {
+      const float rs = s_rstd[min(i / len, ng - 1)];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      const int e = i + j;
-      f[j] = e < L.inner ? s_row[e] * s_rstd[e / len] * w[j] : 0.f;
+      for (int j = 0; j < 8; ++j) f[j] *= rs * w[j];
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[j] *= s_rstd[min((i + j) / len, ng - 1)] * w[j];
     }
     store8(crow + i, f);
   }
@@ -238,7 +269,6 @@ hy_mamba_post_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
       store8(ring + i, f);
     }
   }
-  if (L.ff) glu_row(L, row, crow);
 }
 
 template <typename T>
@@ -262,7 +292,7 @@ static int launch_attn_post(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork
   const size_t smem = (size_t)(L.hq + L.hk) * L.dkp * 4;
   const int rc = row_smem(once, hy_attn_post_kernel<T>, smem);
   if (rc) return rc;
-  hy_attn_post_kernel<T><<<b.n, ROW_THREADS, smem, s>>>(
+  hy_attn_post_kernel<T><<<dim3(b.n, 1 + (L.ff + GLU_COLS - 1) / GLU_COLS), ROW_THREADS, smem, s>>>(
       L, static_cast<T*>(w.proj), w.ld_proj, static_cast<T*>(w.cat), w.ld_cat, static_cast<T*>(w.v_first), w.ld_v,
       b.pos, b.row_seq, b.tables, b.max_blocks, c.block_size, c.eps);
   return (int)cudaGetLastError();
@@ -274,7 +304,7 @@ static int launch_mamba_post(const BbHyCfg& c, const BbHyLayer& L, const BbHyWor
   const size_t smem = (size_t)(L.innerp + L.norm_groups) * 4;
   const int rc = row_smem(once, hy_mamba_post_kernel<T>, smem);
   if (rc) return rc;
-  hy_mamba_post_kernel<T><<<b.n, ROW_THREADS, smem, s>>>(
+  hy_mamba_post_kernel<T><<<dim3(b.n, 1 + (L.ff + GLU_COLS - 1) / GLU_COLS), ROW_THREADS, smem, s>>>(
       L, static_cast<const T*>(w.proj), w.ld_proj, static_cast<const T*>(w.y), w.ld_y, static_cast<T*>(w.cat), w.ld_cat,
       b.pos, b.row_seq, b.seq_ctx, b.seq_slot, c.eps);
   return (int)cudaGetLastError();

@@ -30,7 +30,18 @@ __device__ __forceinline__ void conv_tap(const BbHyLayer& L, const T* proj, int 
   }
 }
 
-constexpr int CONV_ROWS = 8;   // consecutive rows of a thread: its window of inputs slides in registers
+constexpr int CONV_ROWS = 16;   // consecutive rows of a thread: its window of inputs slides in registers
+constexpr int CONV_BATCH = 8;   // rows whose inputs are asked for together
+
+template <typename T>
+struct alignas(sizeof(T) * 8) Raw8 {
+  T v[8];
+};
+template <typename T>
+__device__ __forceinline__ void unpack_raw(const Raw8<T>& p, float (&f)[8]) {
+#pragma unroll
+  for (int j = 0; j < 8; ++j) f[j] = to_f(p.v[j]);
+}
 
 // TAPS = 4 keeps the window in registers; TAPS = 0 reads every tap again (any length).
 template <typename T, int TAPS>
@@ -43,12 +54,15 @@ hy_conv_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, 
   if (cv >= nch + ndt) return;
   if (cv >= nch) {
     const int h0 = (cv - nch) * 8;
+    float bias[8];
+    load8(L.dt_bias + h0, bias);
+#pragma unroll 4
     for (int r = r0; r < r1; ++r) {
       float f[8];
       load8(proj + (size_t)r * ld + L.off_dt + h0, f);
 #pragma unroll
-      for (int j = 0; j < 8; ++j)
-        if (h0 + j < L.heads) dt[(size_t)r * lddt + h0 + j] = softplus_f(f[j] + L.dt_bias[h0 + j]);
+      for (int j = 0; j < 8; ++j) f[j] = softplus_f(f[j] + bias[j]);
+      store8(dt + (size_t)r * lddt + h0, f);
     }
     return;
   }
@@ -60,28 +74,38 @@ hy_conv_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, 
 #pragma unroll
     for (int k = 0; k < TAPS; ++k) load8(L.conv_w + (size_t)(TAPS - 1 - k) * L.chp + c, w[k]);
     int last_seq = -1;
-    for (int r = r0; r < r1; ++r) {
-      const int seq = b.row_seq[r];
-      if (seq != last_seq) {
-        const int pos = b.pos[r], pos0 = b.seq_pos0[seq], slot = b.seq_slot[seq];
+    const bool one = b.row_seq[r0] == b.row_seq[r1 - 1];   // all rows of this thread belong to one sequence
+    for (int rb = r0; rb < r1; rb += CONV_BATCH) {
+      Raw8<T> raw[CONV_BATCH];
 #pragma unroll
-        for (int k = 1; k < TAPS; ++k) conv_tap(L, proj, ld, b, r, k, c, pos, pos0, slot, win[k]);
-        last_seq = seq;
+      for (int i = 0; i < CONV_BATCH; ++i)
+        if (rb + i < r1) raw[i] = *reinterpret_cast<const Raw8<T>*>(proj + (size_t)(rb + i) * ld + L.off_xbc + c);
+#pragma unroll
+      for (int i = 0; i < CONV_BATCH; ++i) {
+        const int r = rb + i;
+        if (r >= r1) break;
+        const int seq = one && last_seq >= 0 ? last_seq : b.row_seq[r];
+        if (seq != last_seq) {
+          const int pos = b.pos[r], pos0 = b.seq_pos0[seq], slot = b.seq_slot[seq];
+#pragma unroll
+          for (int k = 1; k < TAPS; ++k) conv_tap(L, proj, ld, b, r, k, c, pos, pos0, slot, win[k]);
+          last_seq = seq;
+        }
+        unpack_raw(raw[i], win[0]);
+        float o[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          float s = bias[j];
+#pragma unroll
+          for (int k = TAPS - 1; k >= 0; --k) s = fmaf(w[k][j], win[k][j], s);
+          o[j] = silu_as<T>(s);
+        }
+        store8(xbc + (size_t)r * ldx + c, o);
+#pragma unroll
+        for (int k = TAPS - 1; k > 0; --k)
+#pragma unroll
+          for (int j = 0; j < 8; ++j) win[k][j] = win[k - 1][j];
       }
-      load8(proj + (size_t)r * ld + L.off_xbc + c, win[0]);
-      float o[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        float s = bias[j];
-#pragma unroll
-        for (int k = TAPS - 1; k >= 0; --k) s = fmaf(w[k][j], win[k][j], s);
-        o[j] = silu_f(s);
-      }
-      store8(xbc + (size_t)r * ldx + c, o);
-#pragma unroll
-      for (int k = TAPS - 1; k > 0; --k)
-#pragma unroll
-        for (int j = 0; j < 8; ++j) win[k][j] = win[k - 1][j];
     }
   } else {
     for (int r = r0; r < r1; ++r) {
@@ -98,7 +122,7 @@ hy_conv_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, 
         for (int j = 0; j < 8; ++j) s[j] = fmaf(w[j], u[j], s[j]);
       }
 #pragma unroll
-      for (int j = 0; j < 8; ++j) s[j] = silu_f(s[j]);
+      for (int j = 0; j < 8; ++j) s[j] = silu_as<T>(s[j]);
       store8(xbc + (size_t)r * ldx + c, s);
     }
   }
@@ -221,7 +245,7 @@ hy_ssm_decode_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
       acc = fmaf(L.conv_w[(size_t)(keep - k) * L.chp + c], to_f(ring[(size_t)((pos - k) % keep) * L.chp + c]), acc);
     acc = fmaf(L.conv_w[(size_t)keep * L.chp + c], to_f(row[L.off_xbc + c]), acc);
     // the same rounding of the convolution's output as in a prompt portion
-    sm[i] = to_f(from_f<T>(silu_f(acc)));
+    sm[i] = to_f(from_f<T>(silu_as<T>(acc)));
   }
   __syncthreads();
   for (int p = lane; p < pv; p += lanes) {

@@ -364,6 +364,34 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
 #pragma unroll
           for (int j = 0; j < 8; ++j) xf[v * 8 + j] = t[j];
         }
+        if constexpr (EXT && (G == 4 || G == 2)) {
+          // the lanes of a group share the heads out while they add up (each ends with one head's score),
+          // so the cap is computed once per score; then every lane collects all of them
+          float a[G];
+#pragma unroll
+          for (int g = 0; g < G; ++g) {
+            a[g] = 0.f;
+#pragma unroll
+            for (int j = 0; j < DPL; ++j) a[g] += xf[j] * qr[g][j];
+          }
+          float s1;
+          if constexpr (G == 4) {
+            const bool hi4 = sub & 4, hi2 = sub & 2;
+            float b0 = hi4 ? a[2] : a[0], b1 = hi4 ? a[3] : a[1];
+            b0 += __shfl_xor_sync(gm, hi4 ? a[0] : a[2], 4);
+            b1 += __shfl_xor_sync(gm, hi4 ? a[1] : a[3], 4);
+            s1 = (hi2 ? b1 : b0) + __shfl_xor_sync(gm, hi2 ? b0 : b1, 2);
+            s1 += __shfl_xor_sync(gm, s1, 1);
+          } else {
+            const bool hi4 = sub & 4;
+            s1 = (hi4 ? a[1] : a[0]) + __shfl_xor_sync(gm, hi4 ? a[0] : a[1], 4);
+            s1 += __shfl_xor_sync(gm, s1, 2);
+            s1 += __shfl_xor_sync(gm, s1, 1);
+          }
+          if (x.cap_log2 > 0.f) s1 = x.cap_log2 * tanh_fp32(s1);
+#pragma unroll
+          for (int g = 0; g < G; ++g) sc[g] = __shfl_sync(gm, s1, grp * 8 + g * (8 / G));
+        } else
 #pragma unroll
         for (int g = 0; g < G; ++g) {
           float a = 0.f;

@@ -79,7 +79,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
   uint8_t* sS = smem + Cfg::OFF_S;
   uint8_t* sSl = sS + PSUB * SSD_SUB;
   float* s_e = reinterpret_cast<float*>(smem + Cfg::OFF_E);   // [128]
-  float* s_part = s_e + 128;                                  // [8]
+  float* s_part = s_e + 128;                                  // [8] warp sums of the coming chunk
   uint64_t* bars = reinterpret_cast<uint64_t*>(s_part + 8);
   uint64_t *b_tma = bars, *b_gy = bars + 1, *b_y = bars + 2, *b_s = bars + 3;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 4);
@@ -128,6 +128,26 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
     tmem_wait_st();
   }
 
+  // step sizes of a chunk and their running sum inside a warp (log2 units), a chunk ahead of their use;
+  // both warpgroups scan the same 128 tokens
+  float d_next = 0.f, cum_next = 0.f;
+  auto load_dt = [&](int ch) {
+    const int i = ch * 128 + row;
+    d_next = i < len ? dt[(size_t)(r0 + i) * lddt + h] : 0.f;
+  };
+  auto scan_dt = [&]() {
+    cum_next = a2 * d_next;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float v = __shfl_up_sync(0xffffffffu, cum_next, o);
+      if (lane >= o) cum_next += v;
+    }
+    if (lane == 31) s_part[warp] = cum_next;
+  };
+  load_dt(0);
+  scan_dt();
+  __syncthreads();
+
   bool ok = (smem_u32(smem) & 1023u) == 0;
   if (!ok && threadIdx.x == 0) set_error(err, ERR_BAD_ARG);
   for (int ch = 0; ch < n_chunks && ok; ++ch) {
@@ -142,18 +162,11 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
       for (int s = 0; s < PSUB; ++s) tma_load_3d(sX + s * SSD_SUB, &tmX, b_tma, s * 64, c0, h);
     }
     __syncwarp();
-    // step sizes and their running sum (log2 units); both warpgroups scan the same 128 tokens
-    const float d = row < valid ? dt[(size_t)(c0 + row) * lddt + h] : 0.f;
-    float cum = a2 * d;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const float v = __shfl_up_sync(0xffffffffu, cum, o);
-      if (lane >= o) cum += v;
-    }
-    if (lane == 31) s_part[warp] = cum;
-    __syncthreads();
+    const float d = d_next;
+    float cum = cum_next;
     for (int w = 0; w < (warp & 3); ++w) cum += s_part[half * 4 + w];
     const float total = (s_part[0] + s_part[1]) + (s_part[2] + s_part[3]);
+    load_dt(ch + 1);
     if (half == 0) s_e[row] = d > 0.f ? cum - log2f(d) : INFINITY;   // W_ij = G_ij 2^(cum_i - e_j)
     // the state as an operand (two terms), and scaled for the accumulation that follows
     {
@@ -287,7 +300,8 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
     ok = mbar_wait(b_y, ph);
     tc_fence_after();
     __syncwarp();
-    __nv_bfloat16* yr = y + (size_t)(c0 + row) * ldy + h * L.p;
+    // outputs go through the C tile's place (its products are behind us), so that a row's columns leave
+    // as one contiguous piece
 #pragma unroll
     for (int c = 0; c < HC; c += 32) {
       uint32_t r[32];
@@ -302,9 +316,22 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
                                                  ((((col & 63) >> 3) ^ (row & 7)) << 4)), f);
 #pragma unroll
         for (int j = 0; j < 8; ++j) f[j] = fmaf(D, f[j], __uint_as_float(r[q * 8 + j]));
-        if (ok && row < valid && col < L.p) store8(yr + col, f);
+        store8(reinterpret_cast<__nv_bfloat16*>(sC + (col >> 6) * SSD_SUB + row * 128 +
+                                                ((((col & 63) >> 3) ^ (row & 7)) << 4)), f);
       }
     }
+    ok = __syncthreads_and(ok);
+    if (ok) {
+      constexpr int VR = PP / 8;   // 16-byte pieces of a row
+      for (int i = threadIdx.x; i < valid * VR; i += SSD_THREADS) {
+        const int rr = i / VR, q = i % VR;
+        if (q * 8 < L.p)
+          *reinterpret_cast<uint4*>(y + (size_t)(c0 + rr) * ldy + h * L.p + q * 8) =
+              *reinterpret_cast<const uint4*>(sC + (q >> 3) * SSD_SUB + rr * 128 + (((q & 7) ^ (rr & 7)) << 4));
+      }
+    }
+    scan_dt();
+    fence_proxy_async_smem();     // the C tile's place was read and written by threads; TMA writes it next
     ok = mbar_wait(b_s, ph) && ok;
     tc_fence_after();
     ok = __syncthreads_and(ok);   // every tile and the accumulators are free for the next chunk
