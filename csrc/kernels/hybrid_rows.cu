@@ -93,19 +93,36 @@ hy_norm_kernel(const float* __restrict__ x, const int* __restrict__ rows, const 
 }
 
 // Blocks of a "post" launch: blockIdx.y = 0 is the row's mixer part, every further one GLU_COLS columns of
-// its feed-forward product.
-constexpr int GLU_COLS = ROW_THREADS * 8;
+// its feed-forward product (GLU_VECS vectors of a thread, all asked for before the first is used).
+constexpr int GLU_VECS = 3;
+constexpr int GLU_COLS = ROW_THREADS * 8 * GLU_VECS;
 
 template <typename T>
 __device__ __forceinline__ void glu_part(const BbHyLayer& L, const T* row, T* crow) {
-  const int i = (blockIdx.y - 1) * GLU_COLS + threadIdx.x * 8;
-  if (i >= ((L.ff + 7) & ~7)) return;
-  float g[8], u[8];
-  load8(row + L.off_gate + i, g);
-  load8(row + L.off_up + i, u);
+  struct alignas(sizeof(T) * 8) Raw {
+    T v[8];
+  };
+  const int n = (L.ff + 7) & ~7, i0 = (blockIdx.y - 1) * GLU_COLS + threadIdx.x * 8;
+  Raw g[GLU_VECS], u[GLU_VECS];
 #pragma unroll
-  for (int j = 0; j < 8; ++j) g[j] = clamped_glu_as<T>(g[j], u[j], L.glu_limit, L.glu_alpha, L.glu_shift);
-  store8(crow + L.off_act + i, g);
+  for (int t = 0; t < GLU_VECS; ++t) {
+    const int i = i0 + t * ROW_THREADS * 8;
+    if (i < n) {
+      g[t] = *reinterpret_cast<const Raw*>(row + L.off_gate + i);
+      u[t] = *reinterpret_cast<const Raw*>(row + L.off_up + i);
+    }
+  }
+#pragma unroll
+  for (int t = 0; t < GLU_VECS; ++t) {
+    const int i = i0 + t * ROW_THREADS * 8;
+    if (i < n) {
+      float f[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+        f[j] = clamped_glu_as<T>(to_f(g[t].v[j]), to_f(u[t].v[j]), L.glu_limit, L.glu_alpha, L.glu_shift);
+      store8(crow + L.off_act + i, f);
+    }
+  }
 }
 
 template <typename T>

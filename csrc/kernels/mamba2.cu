@@ -15,115 +15,117 @@
 
 namespace bb {
 
-// Raw convolution input of row r, k tokens back, 8 channels from c.
-template <typename T>
-__device__ __forceinline__ void conv_tap(const BbHyLayer& L, const T* proj, int ld, const BbHyBatch& b, int r, int k,
-                                         int c, int pos, int pos0, int slot, float (&f)[8]) {
-  if (k <= pos - pos0) {
-    load8(proj + (size_t)(r - k) * ld + L.off_xbc + c, f);
-  } else if (k <= pos) {
-    const int keep = L.taps - 1;
-    load8(static_cast<const T*>(L.conv_state) + ((size_t)slot * keep + (pos - k) % keep) * L.chp + c, f);
-  } else {
-#pragma unroll
-    for (int j = 0; j < 8; ++j) f[j] = 0.f;
-  }
-}
-
-constexpr int CONV_ROWS = 16;   // consecutive rows of a thread: its window of inputs slides in registers
-constexpr int CONV_BATCH = 8;   // rows whose inputs are asked for together
+constexpr int CONV_ROWS = 8;   // consecutive rows of a thread, their inputs asked for together
 
 template <typename T>
-struct alignas(sizeof(T) * 8) Raw8 {
-  T v[8];
+struct alignas(sizeof(T) * 4) Raw4 {
+  T v[4];
 };
+
+// Raw convolution input of row r, k tokens back, 4 channels from c: from the portion itself, from the
+// sequence's slot, or zeros before its start.
 template <typename T>
-__device__ __forceinline__ void unpack_raw(const Raw8<T>& p, float (&f)[8]) {
+__device__ __forceinline__ Raw4<T> conv_tap(const BbHyLayer& L, const T* proj, int ld, int r, int k, int c, int pos,
+                                            int pos0, int slot) {
+  if (k <= pos - pos0) return *reinterpret_cast<const Raw4<T>*>(proj + (size_t)(r - k) * ld + L.off_xbc + c);
+  if (k <= pos) {
+    const int keep = L.taps - 1;
+    return *reinterpret_cast<const Raw4<T>*>(static_cast<const T*>(L.conv_state) +
+                                             ((size_t)slot * keep + (pos - k) % keep) * L.chp + c);
+  }
+  Raw4<T> z;
 #pragma unroll
-  for (int j = 0; j < 8; ++j) f[j] = to_f(p.v[j]);
+  for (int j = 0; j < 4; ++j) z.v[j] = from_f<T>(0.f);
+  return z;
 }
 
-// TAPS = 4 keeps the window in registers; TAPS = 0 reads every tap again (any length).
+// TAPS = 4 keeps a thread's inputs in registers as they are stored; TAPS = 0 reads every tap again (any
+// length).
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128)
 hy_conv_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, int ld, T* __restrict__ xbc, int ldx,
                float* __restrict__ dt, int lddt, const __grid_constant__ BbHyBatch b) {
-  const int cv = blockIdx.y * 128 + threadIdx.x;   // vector of 8 channels, then the vectors of step sizes
-  const int nch = L.chp / 8, ndt = (L.heads + 7) / 8;
-  const int r0 = blockIdx.x * CONV_ROWS, r1 = min(r0 + CONV_ROWS, b.n_pre);
+  const int cv = blockIdx.x * 128 + threadIdx.x;   // vector of 4 channels, then vectors of 4 step sizes
+  const int nch = L.chp / 4, ndt = (L.heads + 7) / 8 * 2;
+  const int r0 = blockIdx.y * CONV_ROWS, r1 = min(r0 + CONV_ROWS, b.n_pre);
   if (cv >= nch + ndt) return;
   if (cv >= nch) {
-    const int h0 = (cv - nch) * 8;
-    float bias[8];
-    load8(L.dt_bias + h0, bias);
+    const int h0 = (cv - nch) * 4;
+    const float4 bias = *reinterpret_cast<const float4*>(L.dt_bias + h0);
 #pragma unroll 4
     for (int r = r0; r < r1; ++r) {
-      float f[8];
-      load8(proj + (size_t)r * ld + L.off_dt + h0, f);
-#pragma unroll
-      for (int j = 0; j < 8; ++j) f[j] = softplus_f(f[j] + bias[j]);
-      store8(dt + (size_t)r * lddt + h0, f);
+      const Raw4<T> f = *reinterpret_cast<const Raw4<T>*>(proj + (size_t)r * ld + L.off_dt + h0);
+      *reinterpret_cast<float4*>(dt + (size_t)r * lddt + h0) =
+          make_float4(softplus_f(to_f(f.v[0]) + bias.x), softplus_f(to_f(f.v[1]) + bias.y),
+                      softplus_f(to_f(f.v[2]) + bias.z), softplus_f(to_f(f.v[3]) + bias.w));
     }
     return;
   }
-  const int c = cv * 8;
-  float bias[8];
-  load8(L.conv_b + c, bias);
+  const int c = cv * 4;
+  const float4 bias4 = *reinterpret_cast<const float4*>(L.conv_b + c);
+  const float bias[4] = {bias4.x, bias4.y, bias4.z, bias4.w};
   if constexpr (TAPS > 0) {
-    float w[TAPS][8], win[TAPS][8];   // win[k]: the input k tokens back
+    constexpr int K = TAPS - 1;
+    Raw4<T> raw[CONV_ROWS + K];   // raw[K + i]: row r0 + i; before it the inputs ahead of r0
 #pragma unroll
-    for (int k = 0; k < TAPS; ++k) load8(L.conv_w + (size_t)(TAPS - 1 - k) * L.chp + c, w[k]);
-    int last_seq = -1;
-    const bool one = b.row_seq[r0] == b.row_seq[r1 - 1];   // all rows of this thread belong to one sequence
-    for (int rb = r0; rb < r1; rb += CONV_BATCH) {
-      Raw8<T> raw[CONV_BATCH];
+    for (int i = 0; i < CONV_ROWS; ++i)
+      if (r0 + i < r1) raw[K + i] = *reinterpret_cast<const Raw4<T>*>(proj + (size_t)(r0 + i) * ld + L.off_xbc + c);
+    // the rows before r0 are asked for before it is known whether they are this sequence's
 #pragma unroll
-      for (int i = 0; i < CONV_BATCH; ++i)
-        if (rb + i < r1) raw[i] = *reinterpret_cast<const Raw8<T>*>(proj + (size_t)(rb + i) * ld + L.off_xbc + c);
+    for (int k = 1; k <= K; ++k)
+      if (r0 >= k) raw[K - k] = *reinterpret_cast<const Raw4<T>*>(proj + (size_t)(r0 - k) * ld + L.off_xbc + c);
+    int last_seq = b.row_seq[r0];
+    const bool one = last_seq == b.row_seq[r1 - 1];   // all rows of this thread belong to one sequence
+    {
+      const int pos = b.pos[r0], pos0 = b.seq_pos0[last_seq], slot = b.seq_slot[last_seq];
 #pragma unroll
-      for (int i = 0; i < CONV_BATCH; ++i) {
-        const int r = rb + i;
-        if (r >= r1) break;
-        const int seq = one && last_seq >= 0 ? last_seq : b.row_seq[r];
-        if (seq != last_seq) {
+      for (int k = 1; k <= K; ++k)
+        if (k > pos - pos0) raw[K - k] = conv_tap(L, proj, ld, r0, k, c, pos, pos0, slot);
+    }
+    float w[TAPS][4];
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k) {
+      const float4 t = *reinterpret_cast<const float4*>(L.conv_w + (size_t)k * L.chp + c);
+      w[k][0] = t.x; w[k][1] = t.y; w[k][2] = t.z; w[k][3] = t.w;
+    }
+#pragma unroll
+    for (int i = 0; i < CONV_ROWS; ++i) {
+      const int r = r0 + i;
+      if (r >= r1) break;
+      if (!one) {
+        const int seq = b.row_seq[r];
+        if (seq != last_seq) {    // a sequence starts inside: what lies ahead of it is its own
           const int pos = b.pos[r], pos0 = b.seq_pos0[seq], slot = b.seq_slot[seq];
 #pragma unroll
-          for (int k = 1; k < TAPS; ++k) conv_tap(L, proj, ld, b, r, k, c, pos, pos0, slot, win[k]);
+          for (int k = 1; k <= K; ++k) raw[K + i - k] = conv_tap(L, proj, ld, r, k, c, pos, pos0, slot);
           last_seq = seq;
         }
-        unpack_raw(raw[i], win[0]);
-        float o[8];
-#pragma unroll
-        for (int j = 0; j < 8; ++j) {
-          float s = bias[j];
-#pragma unroll
-          for (int k = TAPS - 1; k >= 0; --k) s = fmaf(w[k][j], win[k][j], s);
-          o[j] = silu_as<T>(s);
-        }
-        store8(xbc + (size_t)r * ldx + c, o);
-#pragma unroll
-        for (int k = TAPS - 1; k > 0; --k)
-#pragma unroll
-          for (int j = 0; j < 8; ++j) win[k][j] = win[k - 1][j];
       }
+      Raw4<T> o;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        float s = bias[j];
+#pragma unroll
+        for (int k = 0; k < TAPS; ++k) s = fmaf(w[k][j], to_f(raw[i + k].v[j]), s);
+        o.v[j] = from_f<T>(silu_as<T>(s));
+      }
+      *reinterpret_cast<Raw4<T>*>(xbc + (size_t)r * ldx + c) = o;
     }
   } else {
     for (int r = r0; r < r1; ++r) {
       const int seq = b.row_seq[r];
       const int pos = b.pos[r], pos0 = b.seq_pos0[seq], slot = b.seq_slot[seq];
-      float s[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) s[j] = bias[j];
+      float s[4] = {bias[0], bias[1], bias[2], bias[3]};
       for (int k = L.taps - 1; k >= 0; --k) {
-        float u[8], w[8];
-        conv_tap(L, proj, ld, b, r, k, c, pos, pos0, slot, u);
-        load8(L.conv_w + (size_t)(L.taps - 1 - k) * L.chp + c, w);
+        const Raw4<T> u = conv_tap(L, proj, ld, r, k, c, pos, pos0, slot);
+        const float* w = L.conv_w + (size_t)(L.taps - 1 - k) * L.chp + c;
 #pragma unroll
-        for (int j = 0; j < 8; ++j) s[j] = fmaf(w[j], u[j], s[j]);
+        for (int j = 0; j < 4; ++j) s[j] = fmaf(w[j], to_f(u.v[j]), s[j]);
       }
+      Raw4<T> o;
 #pragma unroll
-      for (int j = 0; j < 8; ++j) s[j] = silu_as<T>(s[j]);
-      store8(xbc + (size_t)r * ldx + c, s);
+      for (int j = 0; j < 4; ++j) o.v[j] = from_f<T>(silu_as<T>(s[j]));
+      *reinterpret_cast<Raw4<T>*>(xbc + (size_t)r * ldx + c) = o;
     }
   }
 }
@@ -288,8 +290,9 @@ hy_ssm_decode_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
 
 template <typename T>
 static int launch_conv(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, cudaStream_t s) {
-  const int vecs = L.chp / 8 + (L.heads + 7) / 8;
-  dim3 grid((b.n_pre + CONV_ROWS - 1) / CONV_ROWS, (vecs + 127) / 128);
+  const int vecs = L.chp / 4 + (L.heads + 7) / 8 * 2;
+  dim3 grid((vecs + 127) / 128, (b.n_pre + CONV_ROWS - 1) / CONV_ROWS);
+  if (grid.y > 65535) return BB_ESIZE;
   const T* proj = static_cast<const T*>(w.proj);
   T* xbc = static_cast<T*>(w.xbc);
   if (L.taps == 4) hy_conv_kernel<T, 4><<<grid, 128, 0, s>>>(L, proj, w.ld_proj, xbc, w.ld_xbc, w.dt, w.ld_dt, b);

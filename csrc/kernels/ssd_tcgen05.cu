@@ -14,7 +14,7 @@
 // 256 threads: TMEM lane = token (or state row), two warpgroups share a row's columns.  Thread 0 issues
 // TMA and MMA.  The phases of a chunk are separated by block barriers; with head sizes up to 64 two CTAs
 // share an SM (113 KB of shared memory, 256 TMEM columns each) and fill each other's gaps.
-// TMEM: G, then W as packed bf16 (value in columns 0-63, remainder in 64-127) | Y | S.
+// TMEM: G, then W as packed bf16 (value in its first 64 columns, remainder in the others); Y; S.
 #include "../common/host.hpp"
 #include "../common/ptx.cuh"
 #include "../common/rows.cuh"
@@ -34,7 +34,11 @@ struct SsdCfg {
   static constexpr int OFF_S = OFF_X + PSUB * SSD_SUB;          // 2 PSUB: S as two terms, then X' as two terms
   static constexpr int OFF_E = OFF_S + 2 * PSUB * SSD_SUB;      // 128 floats, 8 partial sums, barriers
   static constexpr int SMEM = OFF_E + 1024;
-  static constexpr int COL_Y = 128, COL_S = 128 + PP;
+  // TMEM columns.  The state product of a chunk leaves its two terms side by side: the first added to S,
+  // the second in T right behind it (one 2 PP wide MMA per step instead of two, which cost the same each).
+  // With PP = 64 T lies over the first half of W, whose products are issued before.
+  static constexpr int COL_G = PP == 64 ? 128 : 0, COL_Y = PP == 64 ? 0 : 128, COL_S = PP == 64 ? 64 : 256;
+  static constexpr int COL_T = COL_S + PP;
   static constexpr int TMEM_COLS = PP == 64 ? 256 : 512;
 };
 
@@ -111,7 +115,8 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
   __syncthreads();
   tc_fence_after();
   const uint32_t tm = *tmem_slot;
-  const uint32_t tG = tm + lane_sel, tY = tm + Cfg::COL_Y + lane_sel + half * HC, tS = tm + Cfg::COL_S + lane_sel + half * HC;
+  const uint32_t tG = tm + Cfg::COL_G + lane_sel, tY = tm + Cfg::COL_Y + lane_sel + half * HC, tS = tm + Cfg::COL_S + lane_sel + half * HC,
+                 tT = tm + Cfg::COL_T + lane_sel + half * HC;
   // the state so far, one row of it per lane
   {
     const bool fresh = b.seq_pos0[seq] == 0 || row >= L.n;
@@ -160,6 +165,13 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
         tma_load_3d(sB + s * SSD_SUB, &tmBC, b_tma, s * 64, c0, grp);
       }
       for (int s = 0; s < PSUB; ++s) tma_load_3d(sX + s * SSD_SUB, &tmX, b_tma, s * 64, c0, h);
+      if (ch + 1 < n_chunks) {   // the coming chunk's tiles start on their way to L2
+        for (int s = 0; s < nsub; ++s) {
+          tma_prefetch_3d(&tmBC, s * 64, c0 + 128, L.groups + grp);
+          tma_prefetch_3d(&tmBC, s * 64, c0 + 128, grp);
+        }
+        for (int s = 0; s < PSUB; ++s) tma_prefetch_3d(&tmX, s * 64, c0 + 128, h);
+      }
     }
     __syncwarp();
     const float d = d_next;
@@ -176,10 +188,19 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
         uint32_t r[32];
         float v[32];
         tmem_ld32(tS + c, r);
-        tmem_wait_ld();
+        if (ch > 0) {
+          uint32_t t[32];
+          tmem_ld32(tT + c, t);
+          tmem_wait_ld();
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]) + __uint_as_float(t[j]);
+        } else {
+          tmem_wait_ld();
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]);
+        }
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
-          v[j] = __uint_as_float(r[j]);
           r[j] = __float_as_uint(v[j] * dec);
         }
         tmem_st32(tS + c, r);
@@ -201,7 +222,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
       const uint32_t aC = smem_u32(sC), aB = smem_u32(sB), aS = smem_u32(sS), aSl = smem_u32(sSl);
       for (int t = 0; t < nk; ++t) {
         const uint32_t o = (t / 4) * SSD_SUB + (t % 4) * 32;
-        umma_f16_ss(tm, umma_smem_desc(aC + o, 16, 1024), umma_smem_desc(aB + o, 16, 1024), id_g, t != 0);
+        umma_f16_ss(tm + Cfg::COL_G, umma_smem_desc(aC + o, 16, 1024), umma_smem_desc(aB + o, 16, 1024), id_g, t != 0);
       }
       for (int t = 0; t < nk; ++t) {
         const uint32_t o = (t / 4) * SSD_SUB + (t % 4) * 32;
@@ -230,25 +251,26 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
     {
       const float* e = s_e + half * 64;
       const int lim = row - half * 64;   // columns j <= lim are in the past
-      uint32_t hi[32], lo[32];
+      auto weights = [&](const uint32_t (&g)[32], int j0) {
+        uint32_t hi[16], lo[16];
 #pragma unroll
-      for (int j = 0; j < 32; j += 2) {
-        const float a0 = j <= lim ? __uint_as_float(g0[j]) * exp2f(cum - e[j]) : 0.f;
-        const float a1 = j + 1 <= lim ? __uint_as_float(g0[j + 1]) * exp2f(cum - e[j + 1]) : 0.f;
-        const float2 s = split_pair(a0, a1);
-        hi[j >> 1] = __float_as_uint(s.x);
-        lo[j >> 1] = __float_as_uint(s.y);
-      }
-#pragma unroll
-      for (int j = 0; j < 32; j += 2) {
-        const float a0 = j + 32 <= lim ? __uint_as_float(g1[j]) * exp2f(cum - e[j + 32]) : 0.f;
-        const float a1 = j + 33 <= lim ? __uint_as_float(g1[j + 1]) * exp2f(cum - e[j + 33]) : 0.f;
-        const float2 s = split_pair(a0, a1);
-        hi[16 + (j >> 1)] = __float_as_uint(s.x);
-        lo[16 + (j >> 1)] = __float_as_uint(s.y);
-      }
-      tmem_st32(tG + half * 32, hi);
-      tmem_st32(tG + 64 + half * 32, lo);
+        for (int j = 0; j < 32; j += 4) {
+          const float4 ev = *reinterpret_cast<const float4*>(e + j0 + j);
+          const float w0 = j0 + j <= lim ? __uint_as_float(g[j]) * exp2f(cum - ev.x) : 0.f;
+          const float w1 = j0 + j + 1 <= lim ? __uint_as_float(g[j + 1]) * exp2f(cum - ev.y) : 0.f;
+          const float w2 = j0 + j + 2 <= lim ? __uint_as_float(g[j + 2]) * exp2f(cum - ev.z) : 0.f;
+          const float w3 = j0 + j + 3 <= lim ? __uint_as_float(g[j + 3]) * exp2f(cum - ev.w) : 0.f;
+          const float2 s01 = split_pair(w0, w1), s23 = split_pair(w2, w3);
+          hi[j >> 1] = __float_as_uint(s01.x);
+          lo[j >> 1] = __float_as_uint(s01.y);
+          hi[(j >> 1) + 1] = __float_as_uint(s23.x);
+          lo[(j >> 1) + 1] = __float_as_uint(s23.y);
+        }
+        tmem_st16(tG + half * 32 + (j0 >> 1), hi);
+        tmem_st16(tG + 64 + half * 32 + (j0 >> 1), lo);
+      };
+      weights(g0, 0);
+      weights(g1, 32);
     }
     {
       const float sc = exp2f(cum), w = d * exp2f(total - cum);
@@ -280,19 +302,24 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
     __syncthreads();
     if (threadIdx.x == 0) {
       tc_fence_after();
-      constexpr uint32_t id_y = umma_idesc(1, 1, 1, 0, 1, 128, PP), id_s = umma_idesc(1, 1, 1, 1, 1, 128, PP);
+      constexpr uint32_t id_y = umma_idesc(1, 1, 1, 0, 1, 128, PP), id_s = umma_idesc(1, 1, 1, 1, 1, 128, PP),
+                         id_s2 = umma_idesc(1, 1, 1, 1, 1, 128, 2 * PP);
       const uint32_t aB = smem_u32(sB), aX = smem_u32(sX), aW = smem_u32(sS), aWl = smem_u32(sSl);
 #pragma unroll
       for (int t = 0; t < 8; ++t) {
-        umma_f16_ts(tm + Cfg::COL_Y, tm + t * 8, umma_smem_desc(aX + t * 2048, SSD_SUB, 1024), id_y, 1);
-        umma_f16_ts(tm + Cfg::COL_Y, tm + 64 + t * 8, umma_smem_desc(aX + t * 2048, SSD_SUB, 1024), id_y, 1);
+        umma_f16_ts(tm + Cfg::COL_Y, tm + Cfg::COL_G + t * 8, umma_smem_desc(aX + t * 2048, SSD_SUB, 1024), id_y, 1);
+        umma_f16_ts(tm + Cfg::COL_Y, tm + Cfg::COL_G + 64 + t * 8, umma_smem_desc(aX + t * 2048, SSD_SUB, 1024), id_y, 1);
       }
       umma_commit(b_y);
 #pragma unroll
       for (int t = 0; t < 8; ++t) {
         const uint64_t da = umma_smem_desc(aB + t * 2048, SSD_SUB, 1024);
-        umma_f16_ss(tm + Cfg::COL_S, da, umma_smem_desc(aW + t * 2048, SSD_SUB, 1024), id_s, 1);
-        umma_f16_ss(tm + Cfg::COL_S, da, umma_smem_desc(aWl + t * 2048, SSD_SUB, 1024), id_s, 1);
+        if (t == 0) {   // S goes on, T starts anew
+          umma_f16_ss(tm + Cfg::COL_S, da, umma_smem_desc(aW, SSD_SUB, 1024), id_s, 1);
+          umma_f16_ss(tm + Cfg::COL_T, da, umma_smem_desc(aWl, SSD_SUB, 1024), id_s, 0);
+        } else {
+          umma_f16_ss(tm + Cfg::COL_S, da, umma_smem_desc(aW + t * 2048, SSD_SUB, 1024), id_s2, 1);
+        }
       }
       umma_commit(b_s);
     }
@@ -338,17 +365,18 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
     if (!ok && threadIdx.x == 0) set_error(err, ERR_WAIT_EPILOGUE);
   }
   __syncwarp();
-  if (ok) {
+  if (ok && n_chunks > 0) {
 #pragma unroll
     for (int c = 0; c < HC; c += 32) {
-      uint32_t r[32];
+      uint32_t r[32], t[32];
       tmem_ld32(tS + c, r);
+      tmem_ld32(tT + c, t);
       tmem_wait_ld();
       if (row < L.n) {
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
           const int p = half * HC + c + j;
-          if (p < L.p) state[(size_t)row * L.p + p] = __uint_as_float(r[j]);
+          if (p < L.p) state[(size_t)row * L.p + p] = __uint_as_float(r[j]) + __uint_as_float(t[j]);
         }
       }
     }
