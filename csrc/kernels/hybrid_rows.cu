@@ -126,7 +126,7 @@ __device__ __forceinline__ void glu_part(const BbHyLayer& L, const T* row, T* cr
 }
 
 template <typename T>
-__global__ void __launch_bounds__(ROW_THREADS)
+__global__ void __launch_bounds__(ROW_THREADS, sizeof(T) == 2 ? 5 : 4)
 hy_attn_post_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, int ld, T* __restrict__ cat, int ldc,
                     T* __restrict__ v_first, int ldv, const int* __restrict__ pos_, const int* __restrict__ row_seq,
                     const int* __restrict__ tables, int max_blocks, int bs, float eps) {
@@ -211,7 +211,7 @@ hy_attn_post_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, i
 }
 
 template <typename T>
-__global__ void __launch_bounds__(ROW_THREADS)
+__global__ void __launch_bounds__(ROW_THREADS, sizeof(T) == 2 ? 5 : 4)
 hy_mamba_post_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, int ld, const T* __restrict__ y,
                      int ldy, T* __restrict__ cat, int ldc, const int* __restrict__ pos_,
                      const int* __restrict__ row_seq, const int* __restrict__ seq_ctx,

@@ -42,7 +42,7 @@ __device__ __forceinline__ Raw4<T> conv_tap(const BbHyLayer& L, const T* proj, i
 // TAPS = 4 keeps a thread's inputs in registers as they are stored; TAPS = 0 reads every tap again (any
 // length).
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, sizeof(T) == 2 ? 7 : 5)
 hy_conv_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, int ld, T* __restrict__ xbc, int ldx,
                float* __restrict__ dt, int lddt, const __grid_constant__ BbHyBatch b) {
   const int cv = blockIdx.x * 128 + threadIdx.x;   // vector of 4 channels, then vectors of 4 step sizes
