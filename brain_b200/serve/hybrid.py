@@ -48,7 +48,7 @@ def _ptr(t: Optional[torch.Tensor]):
 class _Scratch:
     """Device buffers of a step of up to ``rows`` rows, ``want`` logit rows and ``dec`` decode rows."""
 
-    def __init__(self, eng: "HybridEngine", rows: int, want: int, dec: int):
+    def __init__(self, eng: "HybridEngine", rows: int, want: int, dec: int, portions: bool = True):
         dev, dt = eng.device, eng.dtype
         m = eng.ld
         self.rows, self.want, self.dec = rows, want, dec
@@ -64,7 +64,9 @@ class _Scratch:
                 n = dec * l.hq * self._max_splits(l.hk, dec)
                 po, pm = max(po, n * (64 if l.dvp <= 64 else 128)), max(pm, n * 2)
         self.part_o, self.part_ml = z(po, dtype=f32), z(pm, dtype=f32)
-        self.seg = z(1, dtype=f32)
+        # segment states of the chunked recurrence (prompt portions): two machine-fulls of states
+        npmax = max([l.n * l.p for l in eng.layer_list if l.kind == 1], default=0)
+        self.seg = z(2 * 2 * eng.sm_count * (npmax + 1) if portions and not eng.fp32 and npmax <= 128 * 128 else 1, dtype=f32)
         self.hn, self.logits = z(max(want, 1), eng.dp), z(max(want, 1), eng.vocabp, dtype=f32)
         w = self.work = hn.Work()
         for n in ("x", "h", "proj", "cat", "xbc", "dt", "y", "v_first", "part_o", "part_ml", "seg", "hn", "logits"):
@@ -105,6 +107,7 @@ class HybridEngine(PagedEngineBase):
         self.max_blocks = (max_seq_len + block_size - 1) // block_size
         self.state_slots, self.dummy_slot = state_slots, state_slots
         self.dummy_block = num_blocks      # padded rows of a bucketed decode batch live there
+        self.sm_count = torch.cuda.get_device_properties(dev).multi_processor_count
         self._init_common(cuda_graphs)
         self._keep: List[torch.Tensor] = []
         self._scratch: Dict[tuple, _Scratch] = {}
@@ -234,7 +237,7 @@ class HybridEngine(PagedEngineBase):
                 raise RuntimeError("step buffers must exist before graph capture")
             if s is not None:
                 rows, want, dec = max(rows, s.rows), max(want, s.want), max(dec, s.dec)
-            s = self._scratch[key] = _Scratch(self, rows, want, dec)
+            s = self._scratch[key] = _Scratch(self, rows, want, dec, portions=key == "step")
         return s
 
     def _run(self, sc: _Scratch, b: hn.Batch, trace: Optional[torch.Tensor] = None) -> torch.Tensor:

@@ -11,6 +11,11 @@
 // scaled inputs X' and the state S as an operand - go through the tensor core as two bf16 terms each
 // (value and remainder, 16 bits of mantissa), so the recurrence keeps its 32-bit character.
 //
+// With few (sequence, head) pairs a portion is cut into segments of whole chunks that run side by side:
+// a first launch (LOCAL) computes what each segment adds to the state on its own, and its decay; the
+// segments of the main launch then start from the state carried in, decayed and summed over the segments
+// before them.
+//
 // 256 threads: TMEM lane = token (or state row), two warpgroups share a row's columns.  Thread 0 issues
 // TMA and MMA.  The phases of a chunk are separated by block barriers; with head sizes up to 64 two CTAs
 // share an SM (113 KB of shared memory, 256 TMEM columns each) and fill each other's gaps.
@@ -69,11 +74,12 @@ __device__ __forceinline__ void store_split(uint8_t* hi, uint8_t* lo, int row, i
   }
 }
 
-template <int PP>
+template <int PP, bool LOCAL>
 __global__ void __launch_bounds__(SSD_THREADS, PP == 64 ? 2 : 1)
 ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant__ CUtensorMap tmX,
                  const __grid_constant__ BbHyLayer L, const float* __restrict__ dt, int lddt,
-                 __nv_bfloat16* __restrict__ y, int ldy, const __grid_constant__ BbHyBatch b, int* err) {
+                 __nv_bfloat16* __restrict__ y, int ldy, const __grid_constant__ BbHyBatch b, int segs,
+                 float* __restrict__ seg, int* err) {
   using Cfg = SsdCfg<PP>;
   constexpr int PSUB = Cfg::PSUB, HC = PP / 2;   // HC: Y / S / X columns of a thread
   extern __shared__ __align__(1024) uint8_t smem[];
@@ -98,6 +104,15 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
   const float a2 = L.a[h] * 1.4426950408889634f, D = L.d_skip[h];
   float* state = L.ssm_state + ((size_t)slot * L.heads + h) * L.n * L.p;
 
+  // this CTA's chunks, and the scratch of its (sequence, head): segment states, the state carried in, decays
+  const int z = blockIdx.z, per = (n_chunks + segs - 1) / segs, z_last = (n_chunks - 1) / per;
+  if (z > z_last || (LOCAL && z > 0 && z == z_last)) return;
+  const int ch0 = z * per, ch1 = LOCAL && z == z_last ? ch0 : min(n_chunks, ch0 + per);
+  const size_t np = (size_t)L.n * L.p;
+  float* sg = seg + ((size_t)seq * L.heads + h) * ((segs + 1) * np + segs);
+  float* s_carry = sg + segs * np;
+  float* s_dec = s_carry + np;
+
   if (threadIdx.x == 0) {
     for (int i = 0; i < 4; ++i) mbar_init(bars + i, 1);
     mbar_fence_init();
@@ -117,17 +132,42 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
   const uint32_t tm = *tmem_slot;
   const uint32_t tG = tm + Cfg::COL_G + lane_sel, tY = tm + Cfg::COL_Y + lane_sel + half * HC, tS = tm + Cfg::COL_S + lane_sel + half * HC,
                  tT = tm + Cfg::COL_T + lane_sel + half * HC;
-  // the state so far, one row of it per lane
+  // The state between memory and TMEM goes through the operand tiles' place as fp32 [128][PP], columns
+  // exclusive-or'ed with the row: a warp moves whole rows of memory, a thread reads or writes its own row.
+  float* s_st = reinterpret_cast<float*>(sS);
   {
-    const bool fresh = b.seq_pos0[seq] == 0 || row >= L.n;
+    const bool fresh = b.seq_pos0[seq] == 0;
+#pragma unroll 4
+    for (int n = warp; n < 128; n += SSD_THREADS / 32) {
+#pragma unroll
+      for (int p0 = 0; p0 < PP; p0 += 32) {
+        const int p = p0 + lane;
+        const size_t i = (size_t)n * L.p + p;
+        float v = 0.f;
+        if (n < L.n && p < L.p) {
+          if (LOCAL) {
+            if (z == 0) {
+              v = fresh ? 0.f : state[i];
+              s_carry[i] = v;      // the main launch may write the slot before its first segment reads it
+            }
+          } else if (segs == 1) {
+            v = fresh ? 0.f : state[i];
+          } else if (z == 0) {
+            v = s_carry[i];
+          } else {
+            v = sg[i];             // (it includes the state carried in)
+            for (int k = 1; k < z; ++k) v = fmaf(v, s_dec[k], sg[k * np + i]);
+          }
+        }
+        s_st[n * PP + (p ^ (n & 31))] = v;
+      }
+    }
+    __syncthreads();
 #pragma unroll
     for (int c = 0; c < HC; c += 32) {
       uint32_t r[32];
 #pragma unroll
-      for (int j = 0; j < 32; ++j) {
-        const int p = half * HC + c + j;
-        r[j] = fresh || p >= L.p ? 0u : __float_as_uint(state[(size_t)row * L.p + p]);
-      }
+      for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(s_st[row * PP + ((half * HC + c + j) ^ (row & 31))]);
       tmem_st32(tS + c, r);
     }
     tmem_wait_st();
@@ -149,25 +189,26 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
     }
     if (lane == 31) s_part[warp] = cum_next;
   };
-  load_dt(0);
+  load_dt(ch0);
   scan_dt();
   __syncthreads();
 
   bool ok = (smem_u32(smem) & 1023u) == 0;
   if (!ok && threadIdx.x == 0) set_error(err, ERR_BAD_ARG);
-  for (int ch = 0; ch < n_chunks && ok; ++ch) {
-    const uint32_t ph = ch & 1;
+  float decay_log = 0.f;
+  for (int ch = ch0; ch < ch1 && ok; ++ch) {
+    const uint32_t ph = (ch - ch0) & 1;
     const int c0 = r0 + ch * 128, valid = min(128, len - ch * 128);
     if (threadIdx.x == 0) {
-      mbar_expect_tx(b_tma, (2 * nsub + PSUB) * SSD_SUB);
+      mbar_expect_tx(b_tma, ((LOCAL ? 1 : 2) * nsub + PSUB) * SSD_SUB);
       for (int s = 0; s < nsub; ++s) {
-        tma_load_3d(sC + s * SSD_SUB, &tmBC, b_tma, s * 64, c0, L.groups + grp);
+        if (!LOCAL) tma_load_3d(sC + s * SSD_SUB, &tmBC, b_tma, s * 64, c0, L.groups + grp);
         tma_load_3d(sB + s * SSD_SUB, &tmBC, b_tma, s * 64, c0, grp);
       }
       for (int s = 0; s < PSUB; ++s) tma_load_3d(sX + s * SSD_SUB, &tmX, b_tma, s * 64, c0, h);
-      if (ch + 1 < n_chunks) {   // the coming chunk's tiles start on their way to L2
+      if (ch + 1 < ch1) {   // the coming chunk's tiles start on their way to L2
         for (int s = 0; s < nsub; ++s) {
-          tma_prefetch_3d(&tmBC, s * 64, c0 + 128, L.groups + grp);
+          if (!LOCAL) tma_prefetch_3d(&tmBC, s * 64, c0 + 128, L.groups + grp);
           tma_prefetch_3d(&tmBC, s * 64, c0 + 128, grp);
         }
         for (int s = 0; s < PSUB; ++s) tma_prefetch_3d(&tmX, s * 64, c0 + 128, h);
@@ -179,6 +220,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
     for (int w = 0; w < (warp & 3); ++w) cum += s_part[half * 4 + w];
     const float total = (s_part[0] + s_part[1]) + (s_part[2] + s_part[3]);
     load_dt(ch + 1);
+    decay_log += total;
     if (half == 0) s_e[row] = d > 0.f ? cum - log2f(d) : INFINITY;   // W_ij = G_ij 2^(cum_i - e_j)
     // the state as an operand (two terms), and scaled for the accumulation that follows
     {
@@ -188,7 +230,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
         uint32_t r[32];
         float v[32];
         tmem_ld32(tS + c, r);
-        if (ch > 0) {
+        if (ch > ch0) {
           uint32_t t[32];
           tmem_ld32(tT + c, t);
           tmem_wait_ld();
@@ -204,7 +246,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
           r[j] = __float_as_uint(v[j] * dec);
         }
         tmem_st32(tS + c, r);
-        store_split(sS, sSl, row, half * HC + c, v);
+        if (!LOCAL) store_split(sS, sSl, row, half * HC + c, v);
       }
       tmem_wait_st();
     }
@@ -216,6 +258,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
       if (threadIdx.x == 0) set_error(err, ERR_WAIT_MMA_FULL);
       break;
     }
+    if constexpr (!LOCAL) {
     if (threadIdx.x == 0) {
       tc_fence_after();
       constexpr uint32_t id_g = umma_idesc(1, 1, 1, 0, 0, 128, 128), id_y = umma_idesc(1, 1, 1, 0, 1, 128, PP);
@@ -272,16 +315,19 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
       weights(g0, 0);
       weights(g1, 32);
     }
+    }
     {
       const float sc = exp2f(cum), w = d * exp2f(total - cum);
 #pragma unroll
       for (int c = 0; c < HC; c += 32) {
-        uint32_t r[32];
-        tmem_ld32(tY + c, r);
-        tmem_wait_ld();
+        if constexpr (!LOCAL) {
+          uint32_t r[32];
+          tmem_ld32(tY + c, r);
+          tmem_wait_ld();
 #pragma unroll
-        for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * sc);
-        tmem_st32(tY + c, r);
+          for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * sc);
+          tmem_st32(tY + c, r);
+        }
         float v[32];
         const int col0 = half * HC + c;
 #pragma unroll
@@ -306,11 +352,11 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
                          id_s2 = umma_idesc(1, 1, 1, 1, 1, 128, 2 * PP);
       const uint32_t aB = smem_u32(sB), aX = smem_u32(sX), aW = smem_u32(sS), aWl = smem_u32(sSl);
 #pragma unroll
-      for (int t = 0; t < 8; ++t) {
+      for (int t = 0; t < (LOCAL ? 0 : 8); ++t) {
         umma_f16_ts(tm + Cfg::COL_Y, tm + Cfg::COL_G + t * 8, umma_smem_desc(aX + t * 2048, SSD_SUB, 1024), id_y, 1);
         umma_f16_ts(tm + Cfg::COL_Y, tm + Cfg::COL_G + 64 + t * 8, umma_smem_desc(aX + t * 2048, SSD_SUB, 1024), id_y, 1);
       }
-      umma_commit(b_y);
+      if (!LOCAL) umma_commit(b_y);
 #pragma unroll
       for (int t = 0; t < 8; ++t) {
         const uint64_t da = umma_smem_desc(aB + t * 2048, SSD_SUB, 1024);
@@ -324,6 +370,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
       umma_commit(b_s);
     }
     __syncwarp();
+    if constexpr (!LOCAL) {
     ok = mbar_wait(b_y, ph);
     tc_fence_after();
     __syncwarp();
@@ -357,6 +404,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
               *reinterpret_cast<const uint4*>(sC + (q >> 3) * SSD_SUB + rr * 128 + (((q & 7) ^ (rr & 7)) << 4));
       }
     }
+    }
     scan_dt();
     fence_proxy_async_smem();     // the C tile's place was read and written by threads; TMA writes it next
     ok = mbar_wait(b_s, ph) && ok;
@@ -365,19 +413,26 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
     if (!ok && threadIdx.x == 0) set_error(err, ERR_WAIT_EPILOGUE);
   }
   __syncwarp();
-  if (ok && n_chunks > 0) {
+  if (LOCAL && threadIdx.x == 0) s_dec[z] = exp2f(decay_log);
+  if (ok && ch1 > ch0 && (LOCAL || z == z_last)) {
+    float* dst = LOCAL ? sg + z * np : state;
 #pragma unroll
     for (int c = 0; c < HC; c += 32) {
       uint32_t r[32], t[32];
       tmem_ld32(tS + c, r);
       tmem_ld32(tT + c, t);
       tmem_wait_ld();
-      if (row < L.n) {
 #pragma unroll
-        for (int j = 0; j < 32; ++j) {
-          const int p = half * HC + c + j;
-          if (p < L.p) state[(size_t)row * L.p + p] = __uint_as_float(r[j]) + __uint_as_float(t[j]);
-        }
+      for (int j = 0; j < 32; ++j)
+        s_st[row * PP + ((half * HC + c + j) ^ (row & 31))] = __uint_as_float(r[j]) + __uint_as_float(t[j]);
+    }
+    __syncthreads();
+#pragma unroll 4
+    for (int n = warp; n < L.n; n += SSD_THREADS / 32) {
+#pragma unroll
+      for (int p0 = 0; p0 < PP; p0 += 32) {
+        const int p = p0 + lane;
+        if (p < L.p) dst[(size_t)n * L.p + p] = s_st[n * PP + (p ^ (n & 31))];
       }
     }
   }
@@ -392,11 +447,32 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
 template <int PP>
 static int launch_ssd(const CUtensorMap& tmBC, const CUtensorMap& tmX, const BbHyLayer& L, const BbHyWork& w,
                       const BbHyBatch& b, cudaStream_t s) {
-  static PerDeviceOnce once;
-  const cudaError_t e = ensure_dyn_smem(once, ssd_chunk_kernel<PP>, SsdCfg<PP>::SMEM);
+  static PerDeviceOnce once, once_local;
+  constexpr int SMEM = SsdCfg<PP>::SMEM;
+  cudaError_t e = ensure_dyn_smem(once, ssd_chunk_kernel<PP, false>, SMEM);
   if (e != cudaSuccess) return (int)e;
-  ssd_chunk_kernel<PP><<<dim3(b.ns_pre, L.heads), SSD_THREADS, SsdCfg<PP>::SMEM, s>>>(
-      tmBC, tmX, L, w.dt, w.ld_dt, static_cast<__nv_bfloat16*>(w.y), w.ld_y, b, device_error_word());
+  e = ensure_dyn_smem(once_local, ssd_chunk_kernel<PP, true>, SMEM);
+  if (e != cudaSuccess) return (int)e;
+  // segments: as many as fill the machine once, of four chunks or more (a 2048-token prompt of 64 heads
+  // alone: 75 us against 112 us in one piece; at two chunks the extra launch costs more than it saves),
+  // and as the scratch allows
+  const long pairs = (long)b.ns_pre * L.heads, np = (long)L.n * L.p;
+  int segs = (int)((PP == 64 ? 2 : 1) * sm_count() / pairs);
+  const int most = (b.max_len + 127) / 128 / 4;
+  if (segs > most) segs = most;
+  if (segs > 16) segs = 16;
+  while (segs > 1 && pairs * ((segs + 1) * np + segs) > w.seg_floats) --segs;
+  if (segs < 2) segs = 1;
+  __nv_bfloat16* y = static_cast<__nv_bfloat16*>(w.y);
+  const dim3 grid(b.ns_pre, L.heads, segs);
+  if (segs > 1) {
+    ssd_chunk_kernel<PP, true><<<grid, SSD_THREADS, SMEM, s>>>(tmBC, tmX, L, w.dt, w.ld_dt, y, w.ld_y, b, segs, w.seg,
+                                                               device_error_word());
+    e = cudaGetLastError();
+    if (e != cudaSuccess) return (int)e;
+  }
+  ssd_chunk_kernel<PP, false><<<grid, SSD_THREADS, SMEM, s>>>(tmBC, tmX, L, w.dt, w.ld_dt, y, w.ld_y, b, segs, w.seg,
+                                                              device_error_word());
   return (int)cudaGetLastError();
 }
 

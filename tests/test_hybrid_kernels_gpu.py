@@ -173,16 +173,18 @@ def test_fp32_argmax_and_topk():
     assert torch.equal(val.cpu(), tv) and idx[0, :2].cpu().tolist() == [77, 900]
 
 
+@pytest.mark.parametrize("segments", [False, True])
 @pytest.mark.parametrize("H,P,N,G", [(4, 64, 128, 1), (2, 128, 128, 2), (6, 16, 24, 3), (3, 40, 64, 1), (2, 72, 72, 1),
                                      (8, 32, 8, 4), (5, 8, 120, 5)])
-def test_chunked_recurrence_keeps_fp32_state(H, P, N, G):
+def test_chunked_recurrence_keeps_fp32_state(H, P, N, G, segments):
     """The tensor-core chunks against the token-by-token fp32 scan on the same bf16 inputs: portions of
-    many lengths, from zero and from carried states, in slots that hold something else."""
+    many lengths, from zero and from carried states, in slots that hold something else; with and without
+    scratch to run a portion's segments side by side."""
     import ctypes as C
     from brain_b200.ops._cuda import check_error, lib, stream_ptr
     from brain_b200.serve import hybrid_native as hn
     g = torch.Generator().manual_seed(H * P + N)
-    lens, starts = [2, 300, 128, 129, 15, 256, 7], [0, 0, 5, 640, 64, 128, 0]
+    lens, starts = [2, 300, 128, 129, 15, 1500, 7], [0, 0, 5, 640, 64, 128, 0]
     ns, n = len(lens), sum(lens)
     inner, ch = H * P, H * P + 2 * G * N
     ldx = (ch + 7) // 8 * 8 + 8
@@ -200,6 +202,10 @@ def test_chunked_recurrence_keeps_fp32_state(H, P, N, G):
     b.seq_row0, b.seq_pos0, b.seq_slot, b.n_pre, b.ns_pre, b.ns, b.n = \
         row0.data_ptr(), pos0.data_ptr(), slots.data_ptr(), n, ns, ns, n
     w.xbc, w.ld_xbc, w.dt, w.ld_dt, w.ld_y = xbc.data_ptr(), ldx, dt.data_ptr(), H, inner
+    seg = torch.full((4 << 20,), float("nan"), device="cuda")
+    b.max_len = max(lens)
+    if segments:
+        w.seg, w.seg_floats = seg.data_ptr(), seg.numel()
     out = {}
     for name in ("bb_ssd_chunk", "bb_hy_ssm_scan"):
         y, st = torch.zeros(n, inner, device="cuda", dtype=torch.bfloat16), init.clone()
