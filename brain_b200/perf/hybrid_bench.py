@@ -297,3 +297,34 @@ def run(size: str = "m", steps: int = 10, kernels: bool = True, n_seq: int = 4, 
         torch.cuda.empty_cache()
     res["gpu_launches"] = _cuda.launch_count - launches0
     return res
+
+
+def steps(portion: int, seqs: int, ctx: int, n: int = 3, size: str = "m") -> None:
+    """``n`` equal steps of a two-layer model (one layer of each kind): prompts of ``portion`` tokens, or one
+    token each (``portion`` 1), at position ``ctx``.  A small program to put under a profiler."""
+    from ..models.hybrid import HybridDecoder
+    from ..ops import _cuda
+    from ..serve.engine import make_engine
+    from ..serve.hybrid import Entry
+    s = dict(SIZES[size], pairs=1, vocab=1024)
+    model = HybridDecoder(hybrid_config(s)).init_weights(0).to("cuda", torch.bfloat16)
+    per = (portion + ctx) // 16 + 1
+    eng = make_engine(model, max_batch=seqs, block_size=16, num_blocks=seqs * per, max_seq_len=portion + ctx + 16,
+                      max_prefill=portion)
+    rng = np.random.default_rng(0)
+    for _ in range(n):
+        eng.step_logits([Entry(rng.integers(0, 1024, portion), ctx, np.arange(i * per, (i + 1) * per), i, [portion - 1])
+                         for i in range(seqs)])
+    torch.cuda.synchronize()
+    _cuda.check_error()
+    print("ok")
+
+
+if __name__ == "__main__":
+    import argparse
+    ap = argparse.ArgumentParser(description="equal steps of a two-layer hybrid decoder (for a profiler)")
+    ap.add_argument("--portion", type=int, default=1024)
+    ap.add_argument("--seqs", type=int, default=2)
+    ap.add_argument("--ctx", type=int, default=0)
+    a = ap.parse_args()
+    steps(a.portion, a.seqs, a.ctx)
