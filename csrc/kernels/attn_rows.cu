@@ -1,5 +1,5 @@
 // Attention of single query rows against the paged K/V pool, one warp per (row, query head): any head
-// sizes up to 256, bf16 or fp32 pages, soft-capped scores, per-head output gate.  It is the fp32 path and
+// sizes up to 512, bf16 or fp32 pages, soft-capped scores, per-head output gate.  It is the fp32 path and
 // the path of head sizes the tensor-core prefill and the split-KV decode kernels do not cover.
 #include "../common/host.hpp"
 #include "../common/ptx.cuh"
@@ -7,9 +7,8 @@
 
 namespace bb {
 
-constexpr int AR_VEC = 8;   // elements of a lane: head sizes up to 256
-
-template <typename T>
+// AR_VEC: elements of a lane (head sizes up to 32 times that)
+template <typename T, int AR_VEC>
 __global__ void __launch_bounds__(128)
 attn_rows_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ kc, const T* __restrict__ vc,
                  const int* __restrict__ pos, const int* __restrict__ row_seq, const int* __restrict__ tables,
@@ -67,17 +66,24 @@ BB_API int bb_attn_rows(int dtype, const void* q, int ldq, const void* kc, const
                         float scale, float softcap, void* stream) {
   using namespace bb;
   if (rows <= 0) return BB_OK;
-  if (dk > 32 * AR_VEC || dvp > 32 * AR_VEC || hq % hk) return BB_ESIZE;
+  const int d = dk > dvp ? dk : dvp;
+  if (d > 512 || hq % hk) return BB_ESIZE;
   const int grid = (int)(((long)rows * hq * 32 + 127) / 128);
   cudaStream_t s = (cudaStream_t)stream;
-  if (dtype)
-    attn_rows_kernel<float><<<grid, 128, 0, s>>>((const float*)q, ldq, (const float*)kc, (const float*)vc, pos, row_seq,
-                                                 tables, max_blocks, bs, (float*)out, ldo, (const float*)gate, ldg, rows,
-                                                 hq, hk, dk, dv, dkp, dvp, scale, softcap);
-  else
-    attn_rows_kernel<__nv_bfloat16><<<grid, 128, 0, s>>>(
-        (const __nv_bfloat16*)q, ldq, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, pos, row_seq, tables,
-        max_blocks, bs, (__nv_bfloat16*)out, ldo, (const __nv_bfloat16*)gate, ldg, rows, hq, hk, dk, dv, dkp, dvp, scale,
-        softcap);
+#define BB_LAUNCH_AR(T, V)                                                                                          \
+  attn_rows_kernel<T, V><<<grid, 128, 0, s>>>((const T*)q, ldq, (const T*)kc, (const T*)vc, pos, row_seq, tables,   \
+                                              max_blocks, bs, (T*)out, ldo, (const T*)gate, ldg, rows, hq, hk, dk,  \
+                                              dv, dkp, dvp, scale, softcap)
+#define BB_LAUNCH_AR_T(T)                  \
+  do {                                     \
+    if (d <= 64) BB_LAUNCH_AR(T, 2);       \
+    else if (d <= 128) BB_LAUNCH_AR(T, 4); \
+    else if (d <= 256) BB_LAUNCH_AR(T, 8); \
+    else BB_LAUNCH_AR(T, 16);              \
+  } while (0)
+  if (dtype) BB_LAUNCH_AR_T(float);
+  else BB_LAUNCH_AR_T(__nv_bfloat16);
+#undef BB_LAUNCH_AR_T
+#undef BB_LAUNCH_AR
   return (int)cudaGetLastError();
 }

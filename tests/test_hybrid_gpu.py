@@ -23,6 +23,7 @@ MECHANISMS = {
     "attention_wide": [(attn(heads=4, kv_heads=2, dim=104, vdim=120, rot=64), None)],
     "attention_wide_keys": [(attn(heads=4, kv_heads=4, dim=96, vdim=16, rot=96), None)],
     "attention_very_wide": [(attn(heads=2, kv_heads=1, dim=160, vdim=136, rot=32), None)],
+    "attention_huge": [(attn(heads=2, kv_heads=2, dim=320, vdim=264, rot=64), None)],
     "attention_low_cap": [(attn(softcap=2.0, scale=1.0), None)],
     "attention_many_shared": [(attn(heads=14, kv_heads=2, dim=8, vdim=8, rot=2), None)],
     "v_mix_skips_a_layer": [(attn(v_mix=False, vdim=16), None), (attn(), None), (attn(dim=16), glu()), (attn(), None)],
