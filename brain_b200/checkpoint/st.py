@@ -213,7 +213,7 @@ def save_model(path: str, model, card: Optional[ModelCard] = None, dtype: str = 
     state = model.reference_state()
     if card is None:
         fam = getattr(model, "family", "qwen")
-        card = ModelCard(id={"gpt": "brain/gpt", "qwen": "brain/qwen3", "hybrid": "brain/pakalix"}.get(fam, f"brain/{fam}"),
+        card = ModelCard(id={"gpt": "brain/gpt", "qwen": "brain/qwen3", "hybrid": f"brain/{getattr(model.cfg, 'design', '').lower()}"}.get(fam, f"brain/{fam}"),
                          family=fam, param_count=sum(t.numel() for t in state.values()),
                          capabilities=["generate"])
     save(path, state, model.config_json(), card, dtype)
@@ -224,7 +224,7 @@ def load_model(path: str, device="cpu", dtype=None):
     safetensors file that carries its configuration, or a directory with ``config.json`` and
     ``model.safetensors``."""
     import os
-    from ..models import build_from_config
+    from ..models import build_from_config, config_from_json
     if os.path.isdir(path):
         with open(os.path.join(path, "config.json")) as f:
             config = json.load(f)
@@ -233,7 +233,10 @@ def load_model(path: str, device="cpu", dtype=None):
         tensors, config, card = load(path)
     if config is None:
         raise ValueError(f"{path}: no brain.config metadata")
-    model = build_from_config(config)
+    cfg = config_from_json(config)
+    if hasattr(cfg, "fill_sizes"):
+        cfg.fill_sizes({n: tuple(t.shape) for n, t in tensors.items()})
+    model = build_from_config(cfg)
     model.load_reference_state(tensors, strict=True)
     if dtype is not None or device != "cpu":
         model = model.to(device=device, dtype=dtype)

@@ -7,6 +7,7 @@ added here (the reference has none)."""
 from __future__ import annotations
 
 import json
+import math
 from dataclasses import dataclass, field, asdict
 from typing import List, Optional
 
@@ -307,9 +308,40 @@ class MoeConfig:
 # constants as fields; a design is a reader of its config file (``HYBRID_DESIGNS``) that fills them in.
 
 @dataclass
+class YarnSpec:
+    """Per-pair frequency interpolation: pairs that turn more than ``fast`` times over the original context
+    keep their frequency, those that turn less than ``slow`` times have it divided by ``factor``, with a
+    ramp in between; cos and sin grow by 0.1 ln(factor) + 1."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+
+@dataclass
 class RotarySpec:
-    dims: int                    # leading dimensions of a head that are rotated, half-split pairs
+    dims: int                    # leading dimensions of a head that are rotated
     base: float
+    scaling: Optional[YarnSpec] = None
+    interleaved: bool = False    # neighbouring pairs (2i, 2i + 1) instead of half-split ones
+
+    def frequencies(self):
+        """(angle per position of every pair, factor on cos and sin), in double precision."""
+        f = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        y = self.scaling
+        if y is None:
+            return f, 1.0
+        turns = lambda t: self.dims * math.log(y.original / (2 * math.pi * t)) / (2 * math.log(self.base))
+        lo, hi = max(math.floor(turns(y.fast)), 0), min(math.ceil(turns(y.slow)), self.dims - 1)
+        ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(len(f))]
+        return [v / y.factor * r + v * (1.0 - r) for v, r in zip(f, ramp)], 0.1 * math.log(y.factor) + 1.0
+
+    @staticmethod
+    def from_json(c: dict, interleaved: bool = False) -> "RotarySpec":
+        y = c.get("scaling")
+        return RotarySpec(int(c["dims"]), float(c["base"]),
+                          None if not y else YarnSpec(*(float(y[k]) for k in ("factor", "original", "fast", "slow"))),
+                          interleaved)
 
 
 @dataclass
@@ -323,6 +355,19 @@ class AttentionSpec:
     rot: Optional[RotarySpec] = None
     v_mix: bool = False          # values mixed with those of the first layer that has this set
     kind = "attention"
+
+    @staticmethod
+    def from_json(m: dict) -> "AttentionSpec":
+        rot = m.get("rot")
+        return AttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                             scale=float(m["scale"]), softcap=float(m["softcap"]) if m.get("softcap") else None,
+                             rot=RotarySpec.from_json(rot) if rot else None, v_mix=bool(m.get("v_mix", False)))
+
+    def to_json(self) -> dict:
+        m = {k: v for k, v in asdict(self).items() if v is not None}
+        if self.rot is not None:
+            m["rot"] = {"dims": self.rot.dims, "base": self.rot.base}
+        return m
 
     def check(self):
         if self.heads % self.kv_heads:
@@ -349,6 +394,14 @@ class Mamba2Spec:
     norm_groups: int
     kind = "mamba2"
 
+    @staticmethod
+    def from_json(m: dict) -> "Mamba2Spec":
+        return Mamba2Spec(heads=int(m["heads"]), vdim=int(m["vdim"]), state=int(m["state"]), groups=int(m["groups"]),
+                          conv=int(m["conv"]), norm_groups=int(m["norm_groups"]))
+
+    def to_json(self) -> dict:
+        return asdict(self)
+
     @property
     def inner(self) -> int:
         return self.heads * self.vdim
@@ -372,21 +425,186 @@ class Mamba2Spec:
 
 
 @dataclass
+class LatentAttentionSpec:
+    """Attention whose keys and values are projections of one cached latent per token, plus one rotated key
+    part that all heads share; queries go through a latent of their own."""
+    heads: int
+    dim: int                     # unrotated query / key dimensions of a head
+    rot_dim: int                 # rotated ones
+    vdim: int
+    kv_rank: int
+    q_rank: int
+    scale: float
+    rot: RotarySpec = None
+    window: Optional[int] = None     # keys a query sees, itself included (None: every earlier one)
+    kv_from: Optional[int] = None    # the layer whose latents and rotated key parts are used
+    kind = "latent_attention"
+
+    @staticmethod
+    def from_json(m: dict) -> "LatentAttentionSpec":
+        mask, j = m.get("mask") or {}, m.get("kv_from")
+        rot = dict(m["rot"])
+        rot.setdefault("dims", m["rot_dim"])
+        return LatentAttentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]),
+                                   kv_rank=int(m["kv_rank"]), q_rank=int(m.get("q_rank") or 0), scale=float(m["scale"]),
+                                   rot=RotarySpec.from_json(rot, interleaved=True),
+                                   window=int(mask["size"]) if mask.get("size") else None,
+                                   kv_from=None if j is None else int(j))
+
+    def to_json(self) -> dict:
+        m = {k: v for k, v in asdict(self).items() if k not in ("rot", "window", "kv_from")}
+        m["rot"] = {"dims": self.rot.dims, "base": self.rot.base}
+        if self.rot.scaling is not None:
+            m["rot"]["scaling"] = asdict(self.rot.scaling)
+        if self.window is not None:
+            m["mask"] = {"size": self.window}
+        if self.kv_from is not None:
+            m["kv_from"] = self.kv_from
+        return m
+
+    def fill(self, shape):
+        self.q_rank = self.q_rank or shape("dq")[0]
+
+    def check(self):
+        if self.rot.dims != self.rot_dim or self.rot_dim % 2:
+            raise ValueError(f"latent attention: cannot rotate {self.rot.dims} of {self.rot_dim} dimensions")
+        if self.window is not None and self.window < 1:
+            raise ValueError("latent attention: the window holds at least the token itself")
+
+    def tensors(self, width: int):
+        out = [("dq", (self.q_rank, width)), ("dq.norm", (self.q_rank,)),
+               ("uq", (self.heads * (self.dim + self.rot_dim), self.q_rank))]
+        if self.kv_from is None:
+            out += [("dkv", (self.kv_rank + self.rot_dim, width)), ("dkv.norm", (self.kv_rank,))]
+        return out + [("uk", (self.heads * self.dim, self.kv_rank)), ("uv", (self.heads * self.vdim, self.kv_rank)),
+                      ("o", (width, self.heads * self.vdim))]
+
+
+@dataclass
+class GeneralDeltaSpec:
+    """Delta rule with a decay and a removal rate of its own for every key channel; the decay comes from a
+    low-rank projection of ``decay_rank`` (0: as the checkpoint has it)."""
+    heads: int
+    dim: int
+    decay_rank: int = 0
+    kind = "general_delta"
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.dim
+
+    @staticmethod
+    def from_json(m: dict) -> "GeneralDeltaSpec":
+        return GeneralDeltaSpec(heads=int(m["heads"]), dim=int(m["dim"]), decay_rank=int(m.get("decay_rank") or 0))
+
+    def to_json(self) -> dict:
+        return asdict(self)
+
+    def fill(self, shape):
+        self.decay_rank = self.decay_rank or shape("w1")[0]
+
+    def check(self):
+        pass
+
+    def tensors(self, width: int):
+        n = self.inner
+        return [("r", (n, width)), ("k", (n, width)), ("v", (n, width)), ("g", (n, width)), ("a", (n, width)),
+                ("a.b", (n,)), ("w1", (self.decay_rank, width)), ("w2", (n, self.decay_rank)), ("w0", (n,)),
+                ("norm", (n,)), ("o", (width, n))]
+
+
+@dataclass
+class RgLruSpec:
+    """Gated linear recurrence per channel behind a short convolution, its gates from block-diagonal maps,
+    beside a gelu branch that multiplies its output."""
+    width: int                   # channels
+    blocks: int                  # equal parts of the gates' maps
+    conv: int
+    decay: float = 8.0           # log a = -decay r softplus(lam)
+    kind = "rglru"
+
+    @staticmethod
+    def from_json(m: dict) -> "RgLruSpec":
+        return RgLruSpec(width=int(m["width"]), blocks=int(m["blocks"]), conv=int(m["conv"]))
+
+    def to_json(self) -> dict:
+        return {"width": self.width, "blocks": self.blocks, "conv": self.conv}
+
+    def check(self):
+        if self.blocks < 1 or self.width % self.blocks:
+            raise ValueError(f"rglru: {self.width} channels in {self.blocks} blocks")
+        if self.conv < 1:
+            raise ValueError("rglru: the convolution needs at least one tap")
+
+    def tensors(self, width: int):
+        n, b = self.width, self.width // self.blocks
+        return [("y", (n, width)), ("y.b", (n,)), ("x", (n, width)), ("x.b", (n,)), ("conv", (n, self.conv)), ("conv.b", (n,)),
+                ("ra", (self.blocks, b, b)), ("ra.b", (self.blocks, b)), ("ri", (self.blocks, b, b)),
+                ("ri.b", (self.blocks, b)), ("lam", (n,)), ("o", (width, n))]
+
+
+@dataclass
 class ClampedGluSpec:
     """min(g, limit) sigmoid(alpha g) (clamp(u) + shift) between the gate / up and down projections."""
     ff: int
     limit: float
     alpha: float = 1.702
     shift: float = 1.0
+    kind = "clamped_glu"
+
+    @staticmethod
+    def from_json(f: dict) -> "ClampedGluSpec":
+        return ClampedGluSpec(int(f["ff"]), float(f["limit"]))
+
+    def to_json(self) -> dict:
+        return {"kind": "dense", "ff": self.ff, "limit": self.limit}
 
     def tensors(self, width: int):
         return [("gate", (self.ff, width)), ("up", (self.ff, width)), ("down", (width, self.ff))]
 
 
 @dataclass
+class PolyNormSpec:
+    """a N(z) + b N(z^2) + c N(z^3) + e between the up and down projections, N dividing by the root mean
+    square; projections with biases."""
+    ff: int
+    kind = "polynorm"
+
+    @staticmethod
+    def from_json(f: dict) -> "PolyNormSpec":
+        return PolyNormSpec(int(f["ff"]))
+
+    def to_json(self) -> dict:
+        return {"kind": "dense", "ff": self.ff}
+
+    def tensors(self, width: int):
+        return [("up", (self.ff, width)), ("up.b", (self.ff,)), ("down", (width, self.ff)), ("down.b", (width,)), ("act", (4,))]
+
+
+@dataclass
 class HybridLayer:
-    mixer: object                # AttentionSpec | Mamba2Spec
-    mlp: Optional[ClampedGluSpec] = None
+    mixer: object                # one of the mixer records above
+    mlp: Optional[object] = None
+
+
+@dataclass(frozen=True)
+class HybridDesign:
+    """What the layers of a design have in common."""
+    mixers: tuple                # mixer records its layers may name
+    mlp: type                    # its dense feed-forward
+    norm_offset: float = 0.0     # norms multiply by this plus the stored gain
+    embed_norm: bool = False     # a norm behind the embedding
+    two_norms: bool = False      # the feed-forward reads a norm of its own
+    depth_average: bool = False  # what a layer passes on is a weighted sum of all results so far
+    tied: bool = False           # the embedding table is the output projection
+    residual_mult: bool = False  # a factor on what a layer adds
+
+
+HYBRID_FAMILY = {
+    "Pakalix": HybridDesign((AttentionSpec, Mamba2Spec), ClampedGluSpec, norm_offset=1.0, embed_norm=True, residual_mult=True),
+    "Nezalorn": HybridDesign((LatentAttentionSpec, GeneralDeltaSpec, RgLruSpec), PolyNormSpec, two_norms=True,
+                             depth_average=True, tied=True),
+}
 
 
 @dataclass
@@ -404,12 +622,23 @@ class HybridConfig:
         if not self.layers:
             raise ValueError("a hybrid decoder needs at least one layer")
         vals = set()
-        for l in self.layers:
-            l.mixer.check()
-            if l.mixer.kind == "attention" and l.mixer.v_mix:
-                vals.add((l.mixer.kv_heads, l.mixer.vdim))
+        for i, l in enumerate(self.layers):
+            m = l.mixer
+            m.check()
+            if m.kind == "attention" and m.v_mix:
+                vals.add((m.kv_heads, m.vdim))
+            if m.kind == "latent_attention" and m.kv_from is not None:
+                src = self.layers[m.kv_from].mixer if 0 <= m.kv_from < i else None
+                if src is None or src.kind != m.kind or src.kv_from is not None:
+                    raise ValueError(f"layer {i}: layer {m.kv_from} has no latents of its own to share")
+                if (src.kv_rank, src.rot_dim, src.rot) != (m.kv_rank, m.rot_dim, m.rot):
+                    raise ValueError(f"layer {i}: its latents differ in size or rotation from those of layer {m.kv_from}")
         if len(vals) > 1:
             raise ValueError(f"layers that mix values differ in their value sizes: {sorted(vals)}")
+
+    @property
+    def traits(self) -> HybridDesign:
+        return HYBRID_FAMILY[self.design]
 
     @property
     def n_layers(self) -> int:
@@ -425,56 +654,56 @@ class HybridConfig:
 
     @property
     def recurrent(self) -> bool:
-        return any(l.mixer.kind != "attention" for l in self.layers)
+        return any(l.mixer.kind not in ("attention", "latent_attention") for l in self.layers)
 
     # ---- JSON: the design's own config file
     def to_json(self) -> dict:
-        layers = []
-        for l in self.layers:
-            m = asdict(l.mixer)
-            if l.mixer.kind == "attention":
-                for k in ("softcap", "rot"):
-                    if m[k] is None:
-                        del m[k]
-            layers.append({"type": l.mixer.kind, "mixer": m,
-                           "mlp": None if l.mlp is None else {"kind": "dense", "ff": l.mlp.ff, "limit": l.mlp.limit}})
-        return {"architecture": self.design, "vocab": self.vocab, "width": self.width, "layers": layers,
-                "norm": {"eps": self.eps}, "residual_mult": self.residual_mult}
+        out = {"architecture": self.design, "vocab": self.vocab, "width": self.width,
+               "layers": [{"type": l.mixer.kind, "mixer": l.mixer.to_json(), "mlp": None if l.mlp is None else l.mlp.to_json()}
+                          for l in self.layers],
+               "norm": {"eps": self.eps}}
+        if self.traits.residual_mult:
+            out["residual_mult"] = self.residual_mult
+        return out
 
     @staticmethod
     def from_json(c: dict) -> "HybridConfig":
+        design = HYBRID_FAMILY[c["architecture"]]
+        mixers = {m.kind: m for m in design.mixers}
         layers = []
         for i, e in enumerate(c["layers"]):
-            m = dict(e["mixer"])
-            if e["type"] == "attention":
-                rot = m.get("rot")
-                mixer = AttentionSpec(
-                    heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
-                    scale=float(m["scale"]), softcap=float(m["softcap"]) if m.get("softcap") else None,
-                    rot=RotarySpec(int(rot["dims"]), float(rot["base"])) if rot else None,
-                    v_mix=bool(m.get("v_mix", False)))
-            elif e["type"] == "mamba2":
-                mixer = Mamba2Spec(heads=int(m["heads"]), vdim=int(m["vdim"]), state=int(m["state"]),
-                                   groups=int(m["groups"]), conv=int(m["conv"]), norm_groups=int(m["norm_groups"]))
-            else:
+            if e["type"] not in mixers:
                 raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
             f = e.get("mlp")
             if f is not None and f.get("kind", "dense") != "dense":
                 raise ValueError(f"layer {i}: unknown feed-forward {f['kind']!r}")
-            layers.append(HybridLayer(mixer, None if f is None else ClampedGluSpec(int(f["ff"]), float(f["limit"]))))
+            layers.append(HybridLayer(mixers[e["type"]].from_json(e["mixer"]), None if f is None else design.mlp.from_json(f)))
         return HybridConfig(vocab=int(c["vocab"]), width=int(c["width"]), layers=layers, eps=float(c["norm"]["eps"]),
                             residual_mult=float(c.get("residual_mult", 1.0)), design=c["architecture"])
 
+    def fill_sizes(self, shapes) -> None:
+        """Sizes that the config file leaves to the tensors; ``shapes``: tensor name -> shape."""
+        for i, l in enumerate(self.layers):
+            if hasattr(l.mixer, "fill"):
+                l.mixer.fill(lambda n, p=f"l{i}.mix.": shapes[p + n])
+
     def tensors(self):
         """(name, shape) of every tensor of a checkpoint, in order."""
-        d = self.width
-        out = [("embed", (self.vocab, d)), ("embed.norm", (d,))]
+        d, t = self.width, self.traits
+        out = [("embed", (self.vocab, d))]
+        if t.embed_norm:
+            out.append(("embed.norm", (d,)))
         for i, l in enumerate(self.layers):
             out.append((f"l{i}.norm1", (d,)))
+            if t.two_norms and l.mlp is not None:
+                out.append((f"l{i}.norm2", (d,)))
             out += [(f"l{i}.mix.{n}", s) for n, s in l.mixer.tensors(d)]
             if l.mlp is not None:
                 out += [(f"l{i}.mlp.{n}", s) for n, s in l.mlp.tensors(d)]
-        return out + [("final.norm", (d,)), ("head", (self.vocab, d))]
+            if t.depth_average:
+                out.append((f"l{i}.dwa", (i + 2,)))
+        out.append(("final.norm", (d,)))
+        return out if t.tied else out + [("head", (self.vocab, d))]
 
     def param_list(self):
         out = []
@@ -490,7 +719,7 @@ class HybridConfig:
 
 
 #: architecture name of a config file -> reader of its configuration
-HYBRID_DESIGNS = {"Pakalix": HybridConfig.from_json}
+HYBRID_DESIGNS = {name: HybridConfig.from_json for name in HYBRID_FAMILY}
 
 
 def config_from_json(c) -> object:

@@ -1,6 +1,8 @@
-"""Hybrid decoders (Pakalix): a parallel mixer + feed-forward per layer, the mixer being soft-capped
-attention with rotary positions, whole-projection query / key norms, value mixing and per-head output
-gates, or a Mamba-2 state-space recurrence.
+"""Hybrid decoders: a parallel mixer + feed-forward per layer.
+Pakalix mixers: soft-capped attention with rotary positions, whole-projection query / key norms, value
+mixing and per-head output gates, or a Mamba-2 state-space recurrence.
+Nezalorn mixers: windowed latent attention, a generalised delta rule, or a real-gated linear recurrence;
+what a layer passes on is a weighted sum of all results so far.
 
 This is the weight container of the family (names, shapes, initial values, loading); its forward lives in
 the serving engine (``serve.hybrid.HybridEngine`` over ``csrc/serve/hybrid_forward.cu``)."""
@@ -43,10 +45,23 @@ class HybridDecoder(nn.Module):
         for name, shape in self.cfg.tensors():
             p = self.tensor(name)
             leaf = name.split(".", 2)[-1] if name[0] == "l" and name[1].isdigit() else name
-            if leaf in ("embed.norm", "final.norm", "norm1") or name.endswith(".norm1"):
-                v = 0.1 * torch.randn(shape, generator=g)
-            elif leaf in ("q.norm", "k.norm", "norm"):
+            if leaf in ("embed.norm", "final.norm") or name.endswith((".norm1", ".norm2")):
+                v = 1.0 - self.cfg.traits.norm_offset + 0.1 * torch.randn(shape, generator=g)
+            elif leaf in ("q.norm", "k.norm", "norm", "dq.norm", "dkv.norm"):
                 v = 1.0 + 0.1 * torch.randn(shape, generator=g)
+            elif name.endswith(".dwa"):
+                v = 0.2 * torch.randn(shape, generator=g) / shape[0]     # mostly the layer's own result
+                v[-1] += 1.0
+            elif leaf == "act":
+                v = uniform(shape, 0.2, 0.8)
+            elif leaf == "lam":
+                v = uniform(shape, -5.0, -0.5)                           # decays between slow and fast
+            elif leaf == "w0":
+                v = uniform(shape, -8.0, 0.0)
+            elif leaf == "a.b":
+                v = uniform(shape, -2.0, 1.0)
+            elif leaf.endswith(".b") and leaf != "conv.b":
+                v = uniform(shape, -0.3, 0.3)
             elif leaf == "vmix":
                 v = uniform(shape, 0.2, 0.6)
             elif leaf == "dt_bias":
@@ -63,7 +78,7 @@ class HybridDecoder(nn.Module):
             elif name == "embed":
                 v = torch.randn(shape, generator=g)
             else:
-                v = torch.randn(shape, generator=g) / math.sqrt(shape[1])
+                v = torch.randn(shape, generator=g) / math.sqrt(shape[-1])
             p.copy_(v.to(p.dtype))
         return self
 
@@ -92,12 +107,18 @@ class HybridDecoder(nn.Module):
         """Matrix-product FLOPs of one token with T tokens of context, attention and recurrence included."""
         total = 0.0
         for n, s in self.cfg.tensors():
-            if len(s) == 2 and n != "embed" and not n.endswith(".conv"):
-                total += 2.0 * s[0] * s[1]
+            if len(s) > 1 and (n != "embed" or self.cfg.traits.tied) and not n.endswith((".conv", "a.b", "i.b")):
+                total += 2.0 * math.prod(s)
         for l in self.cfg.layers:
             m = l.mixer
             if m.kind == "attention":
                 total += 2.0 * m.heads * (m.dim + m.vdim) * T
-            else:
+            elif m.kind == "latent_attention":
+                total += 2.0 * m.heads * (m.dim + m.rot_dim + m.vdim) * min(T, m.window or T)
+            elif m.kind == "mamba2":
                 total += 6.0 * m.heads * m.state * m.vdim
+            elif m.kind == "general_delta":
+                total += 10.0 * m.heads * m.dim * m.dim
+            else:
+                total += 12.0 * m.width
         return total

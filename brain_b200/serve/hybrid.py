@@ -1,13 +1,14 @@
-"""Serving engine of the hybrid decoders (Pakalix): paged K/V for the attention layers, recurrent-state
-slots for the state-space layers, one native call per step.
+"""Serving engine of the hybrid decoders (Pakalix, Nezalorn): pages for the attention layers, recurrent-state
+slots for the recurrent layers, one native call per step.
 
 * A step is ONE packed batch: prompt portions of any length and single decoded tokens of several
   sequences run together (``csrc/serve/hybrid_forward.cu``).  Every entry point - the scheduler's prefill,
   mixed and decode calls and :meth:`HybridEngine.step_logits` - goes through it.
-* K/V pages: per attention layer ``[num_blocks + 1, kv_heads, block_size, head size]``.  State slots: per
-  state-space layer a ring of the last taps - 1 raw convolution inputs and the fp32 state
-  ``[heads, state, head size]``.  A sequence at position 0 starts from zeros, so pages and slots are
-  reused as they are.
+* Pages: per attention layer keys and values ``[num_blocks + 1, kv_heads, block_size, head size]``, per latent
+  attention layer with latents of its own ``[num_blocks + 1, block_size, latent | rotated key part]``.  State
+  slots: per recurrent layer the fp32 state (``[heads, state, head size]``, ``[heads, key, value]`` or one value
+  per channel) and, where it has a convolution, a ring of the last taps - 1 raw inputs.  A sequence at position
+  0 starts from zeros, so pages and slots are reused as they are.
 * ``dtype='bf16'``: bf16 weights, activations, pages and convolution inputs; the residual stream, norms,
   rotation, scores, softmax, step sizes, decays and the recurrent state are fp32.  ``dtype='fp32'``:
   everything in fp32, no tensor-core rounding."""
@@ -23,7 +24,6 @@ import torch
 from ..models.config import HybridConfig
 from ..ops import _cuda
 from ..ops import functional as F
-from ..ops import reference as ref
 from ..ops._cuda import NativeError, stream_ptr
 from . import hybrid_native as hn
 from .base import PagedEngineBase
@@ -46,34 +46,46 @@ def _ptr(t: Optional[torch.Tensor]):
 
 
 class _Scratch:
-    """Device buffers of a step of up to ``rows`` rows, ``want`` logit rows and ``dec`` decode rows."""
+    """Device buffers of a step of up to ``rows`` rows, ``want`` logit rows, ``dec`` decode rows and ``exp``
+    page rows whose keys and values are multiplied out."""
 
-    def __init__(self, eng: "HybridEngine", rows: int, want: int, dec: int, portions: bool = True):
+    def __init__(self, eng: "HybridEngine", rows: int, want: int, dec: int, exp: int, portions: bool = True):
         dev, dt = eng.device, eng.dtype
         m = eng.ld
-        self.rows, self.want, self.dec = rows, want, dec
+        self.rows, self.want, self.dec, self.exp = rows, want, dec, exp
         z = lambda *s, dtype=dt: torch.zeros(*s, device=dev, dtype=dtype)
         f32 = torch.float32
-        self.x, self.h = z(rows, eng.dp, dtype=f32), z(rows, eng.dp)
+        traits = eng.cfg.traits
+        self.x = z(eng.cfg.n_layers + 1 if traits.depth_average else 1, rows, eng.dp, dtype=f32)
+        self.h, self.h2 = z(rows, eng.dp), z(rows if traits.two_norms else 1, eng.dp)
         self.proj, self.cat = z(rows, m["proj"]), z(rows, m["cat"])
         self.xbc, self.dt, self.y = z(rows, m["xbc"]), z(rows, m["dt"], dtype=f32), z(rows, m["y"])
         self.v_first = z(rows, m["v"])
+        # latent attention: absorbed queries are needed for decoded rows only where portions multiply keys out
+        ab = rows if eng.absorb_portions else max(dec, 1)
+        self.q, self.qa, self.ol, self.aux = z(rows, m["q"]), z(ab, m["qa"]), z(ab, m["ol"]), z(rows, m["aux"])
+        self.ckv, self.kvx = z(max(exp, 1), m["ckv"]), z(max(exp, 1), m["kvx"])
         po = pm = 1
         for l in eng.layer_list:
             if l.kind == 0 and dec and not eng.fp32:
                 n = dec * l.hq * self._max_splits(l.hk, dec)
                 po, pm = max(po, n * (64 if l.dvp <= 64 else 128)), max(pm, n * 2)
+            if l.kind == 2 and dec and not eng.fp32:
+                n = dec * l.hq * _MAX_SPLITS
+                po, pm = max(po, n * l.kvrp), max(pm, n * 2)
         self.part_o, self.part_ml = z(po, dtype=f32), z(pm, dtype=f32)
         # segment states of the chunked recurrence (prompt portions): two machine-fulls of states
         npmax = max([l.n * l.p for l in eng.layer_list if l.kind == 1], default=0)
-        self.seg = z(2 * 2 * eng.sm_count * (npmax + 1) if portions and not eng.fp32 and npmax <= 128 * 128 else 1, dtype=f32)
+        self.seg = z(2 * 2 * eng.sm_count * (npmax + 1) if portions and not eng.fp32 and 0 < npmax <= 128 * 128 else 1, dtype=f32)
         self.hn, self.logits = z(max(want, 1), eng.dp), z(max(want, 1), eng.vocabp, dtype=f32)
         w = self.work = hn.Work()
-        for n in ("x", "h", "proj", "cat", "xbc", "dt", "y", "v_first", "part_o", "part_ml", "seg", "hn", "logits"):
+        for n in ("x", "h", "proj", "cat", "xbc", "dt", "y", "v_first", "part_o", "part_ml", "seg", "hn", "logits", "h2", "q",
+                  "qa", "ol", "aux", "ckv", "kvx"):
             setattr(w, n, _ptr(getattr(self, n)))
         w.seg_floats = self.seg.numel()
-        w.rows, w.want_rows = rows, max(want, 1)
-        w.ld_proj, w.ld_cat, w.ld_xbc, w.ld_dt, w.ld_y, w.ld_v = (m[k] for k in ("proj", "cat", "xbc", "dt", "y", "v"))
+        w.rows, w.want_rows, w.exp_rows = rows, max(want, 1), exp
+        for k in m:
+            setattr(w, "ld_" + k, m[k])
         w.splits, w.pool_blocks = _MAX_SPLITS, eng.num_blocks + 1
 
     @staticmethod
@@ -123,121 +135,229 @@ class HybridEngine(PagedEngineBase):
         self._keep.append(t)
         return t.data_ptr()
 
-    def _mat(self, t: torch.Tensor) -> torch.Tensor:
-        return t.detach().to(self.device, self.dtype)
+    def _hold_matrix(self, t: torch.Tensor) -> int:
+        self._matrix_bytes += t.numel() * t.element_size()
+        return self._hold(t)
 
-    def _rope_tables(self, dims: int, base: float):
-        key = (dims, base)
+    def _lin(self, w: torch.Tensor) -> hn.Lin:
+        return hn.Lin(self._hold_matrix(w), w.shape[0], w.shape[1])
+
+    def _mat(self, name: str) -> torch.Tensor:
+        return self._tensor(name).detach().to(self.device, self.dtype)
+
+    def _vec(self, t: torch.Tensor, n: int) -> int:
+        return self._hold(hn.vec(t, n, self.device))
+
+    def _head_vec(self, name: str, heads: int, size: int) -> int:
+        return self._hold(hn.head_vec(self._tensor(name), heads, size, pad8(size), self.device))
+
+    def _rows(self, name: str, heads: int, size: int) -> torch.Tensor:
+        return hn.padded_rows(self._mat(name), heads, size, pad8(size))
+
+    def _cols(self, name: str, heads: int, size: int) -> torch.Tensor:
+        """An output projection with its input columns padded head by head."""
+        return hn.padded_rows(self._mat(name).t().contiguous(), heads, size, pad8(size)).t()
+
+    def _widest(self, **kw) -> None:
+        for k, n in kw.items():
+            self.ld[k] = max(self.ld[k], n)
+
+    def _pages(self, *shape) -> int:
+        t = torch.zeros(self.num_blocks + 1, *shape, device=self.device, dtype=self.dtype)
+        self.kv_bytes += t.numel() * t.element_size()
+        return self._hold(t)
+
+    def _slots(self, *shape, dtype=torch.float32) -> int:
+        t = torch.zeros(self.state_slots + 1, *shape, device=self.device, dtype=dtype)
+        self.state_bytes += t.numel() * t.element_size()
+        return self._hold(t)
+
+    def _rotary(self, L, rot) -> None:
+        key = (rot.dims, rot.base, str(rot.scaling))
         if key not in self._rope:
-            self._rope[key] = ref.rope_tables(self.max_seq_len, dims, base, device=self.device)
-        return self._rope[key]
+            f, mag = rot.frequencies()
+            ang = torch.arange(self.max_seq_len, dtype=torch.float64)[:, None] * torch.tensor(f, dtype=torch.float64)
+            self._rope[key] = tuple((mag * t).float().to(self.device) for t in (ang.cos(), ang.sin()))
+        L.cos_t, L.sin_t, L.rot = *map(_ptr, self._rope[key]), rot.dims
+
+    # Every packer adds what reads the normed input to ``stack`` and returns the mixer's output projection with
+    # its padded input width.
+    def _pack_attention(self, i: int, L, m, p: str, stack):
+        dkp, dvp = pad8(m.dim), pad8(m.vdim)
+        L.kind, L.hq, L.hk, L.dk, L.dv, L.dkp, L.dvp = 0, m.heads, m.kv_heads, m.dim, m.vdim, dkp, dvp
+        L.off_q = stack.add(self._rows(p + "q", m.heads, m.dim))
+        L.off_k = stack.add(self._rows(p + "k", m.kv_heads, m.dim))
+        L.off_v = stack.add(self._rows(p + "v", m.kv_heads, m.vdim))
+        L.off_g = stack.add(self._mat(p + "g"))
+        L.q_norm, L.k_norm = self._head_vec(p + "q.norm", m.heads, m.dim), self._head_vec(p + "k.norm", m.kv_heads, m.dim)
+        if m.rot is not None and m.rot.dims:
+            self._rotary(L, m.rot)
+        L.scale, L.softcap = m.scale, m.softcap or 0.0
+        first = next((j for j, l in enumerate(self.cfg.layers) if l.mixer.kind == "attention" and l.mixer.v_mix), None)
+        L.v_role = 0 if not m.v_mix else (1 if i == first else 2)
+        L.vmix = float(self._tensor(p + "vmix").float()) if m.v_mix else 0.0
+        L.kc, L.vc = (self._pages(m.kv_heads, self.block_size, d) for d in (dkp, dvp))
+        self._widest(v=m.kv_heads * dvp)
+        return self._cols(p + "o", m.heads, m.vdim), m.heads * dvp
+
+    def _pack_mamba2(self, i: int, L, m, p: str, stack):
+        inner, ch = m.inner, m.channels
+        L.kind, L.heads, L.p, L.n, L.groups = 1, m.heads, m.vdim, m.state, m.groups
+        L.taps, L.norm_groups = m.conv, m.norm_groups
+        L.inner, L.innerp, L.ch, L.chp = inner, pad8(inner), ch, pad8(ch)
+        w_in = self._mat(p + "in")
+        L.off_z = stack.add(w_in[:inner])
+        L.off_xbc = stack.add(w_in[inner:inner + ch])
+        L.off_dt = stack.add(w_in[inner + ch:])
+        T = self._tensor
+        self._pack_conv(L, T(p + "conv"), T(p + "conv.b"), 1, ch)
+        L.dt_bias = self._vec(T(p + "dt_bias"), pad8(m.heads))
+        L.a = self._vec(-torch.exp(T(p + "A_log").detach().double()).float(), pad8(m.heads))
+        L.d_skip = self._vec(T(p + "D"), pad8(m.heads))
+        L.gnorm = self._vec(T(p + "norm"), pad8(inner))
+        L.ssm_state = self._slots(m.heads, m.state, m.vdim)
+        self._widest(dt=pad8(m.heads), y=pad8(inner))
+        return self._mat(p + "o"), pad8(inner)
+
+    def _pack_conv(self, L, w: torch.Tensor, b: torch.Tensor, blocks: int, size: int) -> None:
+        """Short convolution over ``blocks`` x ``size`` channels, padded block by block."""
+        taps, chp = w.shape[1], blocks * pad8(size)
+        cw = hn.padded_rows(w.detach().float().cpu(), blocks, size, pad8(size)).t()
+        L.conv_w = self._hold(cw.contiguous().to(self.device))
+        L.conv_b = self._hold(hn.head_vec(b, blocks, size, pad8(size), self.device))
+        L.conv_state = self._slots(max(taps - 1, 1), chp, dtype=self.dtype)
+        self._widest(xbc=chp)
+
+    def _pack_latent_attention(self, i: int, L, m, p: str, stack):
+        H, dkp, rotp, dvp, kvrp, qrp = m.heads, *map(pad8, (m.dim, m.rot_dim, m.vdim, m.kv_rank, m.q_rank))
+        L.kind, L.hq, L.hk, L.dk, L.dkp, L.dv, L.dvp = 2, H, 1, m.dim, dkp, m.vdim, dvp
+        L.qr, L.qrp, L.kvr, L.kvrp, L.rotp, L.scale, L.window = m.q_rank, qrp, m.kv_rank, kvrp, rotp, m.scale, m.window or 0
+        self._rotary(L, m.rot)
+        L.off_dq = stack.add(self._mat(p + "dq"))
+        L.dq_norm = self._vec(self._tensor(p + "dq.norm"), qrp)
+        row = kvrp + rotp
+        if m.kv_from is None:
+            w = self._mat(p + "dkv")
+            L.own_kv, L.off_ckv = 1, stack.add(w[:m.kv_rank])
+            stack.add(w[m.kv_rank:])
+            L.dkv_norm = self._vec(self._tensor(p + "dkv.norm"), kvrp)
+            L.kc = self._pages(self.block_size, row)
+        else:
+            L.kc = self.layers[m.kv_from].kc
+        per_head = lambda name, n: self._mat(p + name).view(H, n, -1)
+        q = per_head("uq", m.dim + m.rot_dim)
+        uq = torch.cat([hn.padded_groups(q[:, :m.dim], dkp, qrp), hn.padded_groups(q[:, m.dim:], rotp, qrp)], dim=1)
+        L.uq = self._lin(uq.view(-1, qrp))
+        uk, uv = per_head("uk", m.dim), per_head("uv", m.vdim)
+        L.w_abs = self._hold_matrix(hn.padded_groups(uk.transpose(1, 2), kvrp, dkp))
+        L.w_uv = self._hold_matrix(hn.padded_groups(uv, dvp, kvrp))
+        fits = not self.fp32 and dkp + rotp <= 128 and dvp <= 128       # sizes of the tensor-core prefill
+        if fits:
+            # one matrix makes keys and values of page rows; the rotated part passes through its identity
+            k = uk.new_zeros(H, dkp + rotp, row)
+            k[:, :m.dim, :m.kv_rank] = uk
+            k[:, dkp:dkp + m.rot_dim, kvrp:kvrp + m.rot_dim] = torch.eye(m.rot_dim, device=k.device, dtype=k.dtype)
+            v = hn.padded_groups(uv, dvp, row)
+            L.expand = self._lin(torch.cat([k.view(-1, row), v.view(-1, row)]).contiguous())
+            self._widest(ckv=row, kvx=H * (dkp + rotp + dvp))
+        self._widest(q=H * (dkp + rotp), qa=H * row, ol=H * kvrp)
+        self.absorb_portions |= not fits
+        self.exp_window = None if m.window is None or self.exp_window is None else max(self.exp_window, m.window)
+        return self._cols(p + "o", H, m.vdim), H * dvp
+
+    def _pack_general_delta(self, i: int, L, m, p: str, stack):
+        pp = pad8(m.dim)
+        L.kind, L.heads, L.p, L.pp, L.inner, L.innerp = 3, m.heads, m.dim, pp, m.inner, m.heads * pp
+        L.off_r, L.off_kk, L.off_vv, L.off_gg, L.off_a = (stack.add(self._rows(p + n, m.heads, m.dim)) for n in "rkvga")
+        L.wr, L.wrp, L.off_w1 = m.decay_rank, pad8(m.decay_rank), stack.add(self._mat(p + "w1"))
+        L.w2 = self._lin(hn.columns([(self._rows(p + "w2", m.heads, m.dim), L.wrp)], L.innerp))
+        L.w0, L.a_b, L.gnorm = (self._head_vec(p + n, m.heads, m.dim) for n in ("w0", "a.b", "norm"))
+        L.ssm_state = self._slots(m.heads, m.dim, m.dim)
+        self._widest(aux=L.innerp, y=L.innerp)
+        return self._cols(p + "o", m.heads, m.dim), L.innerp
+
+    def _pack_rglru(self, i: int, L, m, p: str, stack):
+        B, n = m.blocks, m.width // m.blocks
+        np_ = pad8(n)
+        L.kind, L.blocks, L.bw, L.bwp, L.taps = 4, B, n, np_, m.conv
+        L.inner, L.innerp, L.ch, L.chp = m.width, B * np_, m.width, B * np_
+        L.off_y, L.off_xbc = stack.add(self._rows(p + "y", B, n)), stack.add(self._rows(p + "x", B, n))
+        L.y_b, L.x_b, L.r_b, L.i_b = (self._head_vec(p + k, B, n) for k in ("y.b", "x.b", "ra.b", "ri.b"))
+        self._pack_conv(L, self._tensor(p + "conv"), self._tensor(p + "conv.b"), B, n)
+        lam = m.decay * torch.nn.functional.softplus(self._tensor(p + "lam").detach().double())
+        L.lam = self._hold(hn.head_vec(lam, B, n, np_, self.device))
+        L.w_gate = self._hold_matrix(torch.cat([hn.padded_groups(self._mat(p + k), np_, np_) for k in ("ra", "ri")], dim=1))
+        L.ssm_state = self._slots(L.chp)
+        self._widest(aux=2 * L.chp)
+        return self._cols(p + "o", B, n), L.innerp
 
     def _pack(self, model) -> None:
-        cfg, dev = self.cfg, self.device
-        dp, fdt = self.dp, self.dtype
-        T = model.tensor
-        zeros = lambda *s, dtype=fdt: torch.zeros(*s, device=dev, dtype=dtype)
+        cfg, dev, dp = self.cfg, self.device, self.dp
+        traits = cfg.traits
+        T = self._tensor = model.tensor
         n = cfg.n_layers
         self.layers = (hn.Layer * n)()
         self.layer_list = [self.layers[i] for i in range(n)]
-        self.ld = dict(proj=8, cat=8, xbc=8, dt=8, y=8, v=8)
-        self.kv_bytes = self.state_bytes = 0
-        first_values = next((i for i, l in enumerate(cfg.layers) if l.mixer.kind == "attention" and l.mixer.v_mix), None)
+        self.ld = dict.fromkeys(("proj", "cat", "xbc", "dt", "y", "v", "q", "qa", "ol", "ckv", "kvx", "aux"), 8)
+        self.kv_bytes = self.state_bytes = self._matrix_bytes = 0
+        # prompt portions of latent attention: whether they also take the absorbed form, and how many keys the
+        # widest window of a layer holds (None: all)
+        self.absorb_portions, self.exp_window = False, 1
+        gain = lambda name: self._vec(traits.norm_offset + T(name).float(), dp)
         for i, spec in enumerate(cfg.layers):
-            L, m, p = self.layers[i], spec.mixer, f"l{i}."
-            L.norm = self._hold(hn.vec(1.0 + T(p + "norm1").float(), dp, dev))
+            L, p = self.layers[i], f"l{i}."
+            L.norm = gain(p + "norm1")
             stack = hn.RowStack()
-            if m.kind == "attention":
-                dkp, dvp = pad8(m.dim), pad8(m.vdim)
-                L.kind, L.hq, L.hk, L.dk, L.dv, L.dkp, L.dvp = 0, m.heads, m.kv_heads, m.dim, m.vdim, dkp, dvp
-                L.off_q = stack.add(hn.padded_rows(self._mat(T(p + "mix.q")), m.heads, m.dim, dkp))
-                L.off_k = stack.add(hn.padded_rows(self._mat(T(p + "mix.k")), m.kv_heads, m.dim, dkp))
-                L.off_v = stack.add(hn.padded_rows(self._mat(T(p + "mix.v")), m.kv_heads, m.vdim, dvp))
-                L.off_g = stack.add(self._mat(T(p + "mix.g")))
-                L.q_norm = self._hold(hn.head_vec(T(p + "mix.q.norm"), m.heads, m.dim, dkp, dev))
-                L.k_norm = self._hold(hn.head_vec(T(p + "mix.k.norm"), m.kv_heads, m.dim, dkp, dev))
-                if m.rot is not None and m.rot.dims:
-                    cos, sin = self._rope_tables(m.rot.dims, m.rot.base)
-                    L.cos_t, L.sin_t, L.rot = _ptr(cos), _ptr(sin), m.rot.dims
-                L.scale, L.softcap = m.scale, m.softcap or 0.0
-                L.v_role = 0 if not m.v_mix else (1 if i == first_values else 2)
-                L.vmix = float(T(p + "mix.vmix").float()) if m.v_mix else 0.0
-                kc = zeros(self.num_blocks + 1, m.kv_heads, self.block_size, dkp)
-                vc = zeros(self.num_blocks + 1, m.kv_heads, self.block_size, dvp)
-                L.kc, L.vc = self._hold(kc), self._hold(vc)
-                self.kv_bytes += (kc.numel() + vc.numel()) * kc.element_size()
-                o = hn.padded_rows(self._mat(T(p + "mix.o")).t().contiguous(), m.heads, m.vdim, dvp).t()
-                mixer_w = m.heads * dvp
-                self.ld["v"] = max(self.ld["v"], m.kv_heads * dvp)
-            else:
-                inner, ch = m.inner, m.channels
-                L.kind, L.heads, L.p, L.n, L.groups = 1, m.heads, m.vdim, m.state, m.groups
-                L.taps, L.norm_groups = m.conv, m.norm_groups
-                L.inner, L.innerp, L.ch, L.chp = inner, pad8(inner), ch, pad8(ch)
-                w_in = self._mat(T(p + "mix.in"))
-                L.off_z = stack.add(w_in[:inner])
-                L.off_xbc = stack.add(w_in[inner:inner + ch])
-                L.off_dt = stack.add(w_in[inner + ch:])
-                cw = torch.zeros(m.conv, pad8(ch))
-                cw[:, :ch] = T(p + "mix.conv").detach().float().cpu().t()
-                L.conv_w = self._hold(cw.contiguous().to(dev))
-                L.conv_b = self._hold(hn.vec(T(p + "mix.conv.b"), pad8(ch), dev))
-                L.dt_bias = self._hold(hn.vec(T(p + "mix.dt_bias"), pad8(m.heads), dev))
-                L.a = self._hold(hn.vec(-torch.exp(T(p + "mix.A_log").detach().double()).float(), pad8(m.heads), dev))
-                L.d_skip = self._hold(hn.vec(T(p + "mix.D"), pad8(m.heads), dev))
-                L.gnorm = self._hold(hn.vec(T(p + "mix.norm"), pad8(inner), dev))
-                ring = zeros(self.state_slots + 1, max(m.conv - 1, 1), pad8(ch))
-                ssm = zeros(self.state_slots + 1, m.heads, m.state, m.vdim, dtype=torch.float32)
-                L.conv_state, L.ssm_state = self._hold(ring), self._hold(ssm)
-                self.state_bytes += ring.numel() * ring.element_size() + ssm.numel() * 4
-                o = self._mat(T(p + "mix.o"))
-                mixer_w = pad8(inner)
-                self.ld["xbc"] = max(self.ld["xbc"], pad8(ch))
-                self.ld["dt"] = max(self.ld["dt"], pad8(m.heads))
-                self.ld["y"] = max(self.ld["y"], pad8(inner))
-            sections = [(o, mixer_w)]
+            sections = [getattr(self, "_pack_" + spec.mixer.kind)(i, L, spec.mixer, p + "mix.", stack)]
+            width = stack.n
             if spec.mlp is not None:
                 f = spec.mlp
-                L.ff, L.glu_limit, L.glu_alpha, L.glu_shift = f.ff, f.limit, f.alpha, f.shift
-                L.off_gate = stack.add(self._mat(T(p + "mlp.gate")))
-                L.off_up = stack.add(self._mat(T(p + "mlp.up")))
-                L.off_act = mixer_w
-                sections.append((self._mat(T(p + "mlp.down")), pad8(f.ff)))
-            w_in, w_out = stack.matrix(dp), hn.columns(sections, dp)
-            L.inp = hn.Lin(self._hold(w_in), w_in.shape[0], w_in.shape[1])
-            L.out = hn.Lin(self._hold(w_out), w_out.shape[0], w_out.shape[1])
-            self.ld["proj"] = max(self.ld["proj"], w_in.shape[0])
-            self.ld["cat"] = max(self.ld["cat"], w_out.shape[1])
+                ffp = pad8(f.ff)
+                L.ff, L.off_act = f.ff, sections[0][1]
+                if f.kind == "clamped_glu":
+                    L.glu_limit, L.glu_alpha, L.glu_shift = f.limit, f.alpha, f.shift
+                    L.off_gate = stack.add(self._mat(p + "mlp.gate"))
+                    L.off_up = stack.add(self._mat(p + "mlp.up"))
+                    width = stack.n
+                else:
+                    L.norm2 = gain(p + "norm2")
+                    L.up = self._lin(hn.columns([(self._mat(p + "mlp.up"), dp)], ffp))
+                    L.up_b, L.down_b = self._vec(T(p + "mlp.up.b"), ffp), self._vec(T(p + "mlp.down.b"), dp)
+                    L.poly, L.off_up = self._vec(T(p + "mlp.act"), 4), stack.n
+                    width = stack.n + ffp
+                sections.append((self._mat(p + "mlp.down"), ffp))
+            if traits.depth_average:
+                L.dwa = self._vec(T(p + "dwa"), i + 2)
+            L.inp, L.out = self._lin(stack.matrix(dp)), self._lin(hn.columns(sections, dp))
+            self._widest(proj=width, cat=L.out.k)
         c = self.ccfg = hn.Cfg()
         c.dtype, c.width, c.dp, c.vocab, c.vocabp = int(self.fp32), cfg.width, dp, cfg.vocab, self.vocabp
         c.n_layers, c.block_size, c.eps, c.residual_mult = n, self.block_size, cfg.eps, cfg.residual_mult
-        pad_cols = lambda w: hn.columns([(w, dp)], pad8(w.shape[0]))
-        c.embed = self._hold(pad_cols(self._mat(T("embed"))))
-        c.head = self._hold(pad_cols(self._mat(T("head"))))
-        c.embed_norm = self._hold(hn.vec(1.0 + T("embed.norm").float(), dp, dev))
-        c.final_norm = self._hold(hn.vec(1.0 + T("final.norm").float(), dp, dev))
+        c.depth_avg = int(traits.depth_average)
+        pad_cols = lambda name: self._hold_matrix(hn.columns([(self._mat(name), dp)], self.vocabp))
+        c.embed = pad_cols("embed")
+        c.head = c.embed if traits.tied else pad_cols("head")
+        c.embed_norm = gain("embed.norm") if traits.embed_norm else None
+        c.final_norm = gain("final.norm")
         c.layers = C.cast(self.layers, C.c_void_p)
+        del self._tensor
 
     # ------------------------------------------------------------------ accounting
     def kv_pool_bytes(self) -> int:
         return self.kv_bytes
 
     def weight_bytes(self) -> int:
-        es = 4 if self.fp32 else 2
-        n = self.vocabp * self.dp * 2
-        for l in self.layer_list:
-            n += l.inp.n * l.inp.k + l.out.n * l.out.k
-        return n * es
+        return self._matrix_bytes
 
     # ------------------------------------------------------------------ steps
-    def _scratch_for(self, key, rows: int, want: int, dec: int) -> _Scratch:
+    def _scratch_for(self, key, rows: int, want: int, dec: int, exp: int = 0) -> _Scratch:
         s = self._scratch.get(key)
-        if s is None or s.rows < rows or s.want < want or s.dec < dec:
+        if s is None or s.rows < rows or s.want < want or s.dec < dec or s.exp < exp:
             if torch.cuda.is_current_stream_capturing():
                 raise RuntimeError("step buffers must exist before graph capture")
             if s is not None:
-                rows, want, dec = max(rows, s.rows), max(want, s.want), max(dec, s.dec)
-            s = self._scratch[key] = _Scratch(self, rows, want, dec, portions=key == "step")
+                rows, want, dec, exp = max(rows, s.rows), max(want, s.want), max(dec, s.dec), max(exp, s.exp)
+            s = self._scratch[key] = _Scratch(self, rows, want, dec, exp, portions=key == "step")
         return s
 
     def _run(self, sc: _Scratch, b: hn.Batch, trace: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -292,9 +412,10 @@ class HybridEngine(PagedEngineBase):
         tiles.sort(key=lambda t: -(int(starts[t[0]]) + min(lens[t[0]], (t[1] + 1) * 128)))
         first_row = {i: int(row0[r]) for r, i in enumerate(order)}
         want = [first_row[i] + int(w) for i, e in enumerate(entries) for w in e.want]
+        exp_src, kv_row0, kv_pos0 = self._expansion(starts[:ns_pre], ctx[:ns_pre], tables)
         parts = [tok, pos, row_seq, row0, starts, ctx, slot, tables.reshape(-1),
                  np.array([t[0] for t in tiles], dtype=np.int32), np.array([t[1] for t in tiles], dtype=np.int32),
-                 np.array(want, dtype=np.int32)]
+                 np.array(want, dtype=np.int32), exp_src, kv_row0, kv_pos0]
         offs = np.concatenate([[0], np.cumsum([-(-p.size // 4) * 4 for p in parts])]).astype(np.int64)
         blob = np.zeros(int(offs[-1]), dtype=np.int32)
         for o, p in zip(offs[:-1].tolist(), parts):
@@ -303,13 +424,28 @@ class HybridEngine(PagedEngineBase):
         base = d_blob.data_ptr()
         b = hn.Batch()
         for name, o in zip(("tok", "pos", "row_seq", "seq_row0", "seq_pos0", "seq_ctx", "seq_slot", "tables", "tile_seq",
-                            "tile_qt", "want"), offs[:-1].tolist()):
+                            "tile_qt", "want", "exp_src", "kv_row0", "kv_pos0"), offs[:-1].tolist()):
             setattr(b, name, base + 4 * o)
         b.max_blocks, b.n, b.n_pre, b.ns, b.ns_pre = self.max_blocks, n, n_pre, ns, ns_pre
-        b.n_tiles, b.n_want, b.max_len = len(tiles), len(want), max(lens[:ns_pre], default=0)
+        b.n_tiles, b.n_want, b.max_len, b.n_exp = len(tiles), len(want), max(lens[:ns_pre], default=0), exp_src.size
         up = lambda v, q: -(-v // q) * q
-        sc = self._scratch_for("step", up(n, 256), up(len(want), 16), up(ns - ns_pre, 16) if ns > ns_pre else 0)
+        sc = self._scratch_for("step", up(n, 256), up(len(want), 16), up(ns - ns_pre, 16) if ns > ns_pre else 0,
+                               up(exp_src.size, 256))
         return sc, b, d_blob
+
+    def _expansion(self, starts, ctx, tables):
+        """Page rows whose keys and values the prompt portions of latent attention multiply out: for every
+        portion its own tokens and the keys that the widest window reaches back to.  Returns (page rows, first
+        of them per portion, position of that first)."""
+        if self.ld["kvx"] <= 8 or not len(starts):
+            return (np.zeros(0, dtype=np.int32),) * 3
+        lo = np.zeros_like(starts) if self.exp_window is None else np.maximum(starts - (self.exp_window - 1), 0)
+        src = []
+        for r, (a, e) in enumerate(zip(lo.tolist(), ctx.tolist())):
+            p = np.arange(a, e)
+            src.append(tables[r, p // self.block_size] * self.block_size + p % self.block_size)
+        row0 = np.concatenate([[0], np.cumsum(ctx - lo)]).astype(np.int32)
+        return np.concatenate(src).astype(np.int32), row0, lo.astype(np.int32)
 
     @torch.no_grad()
     def step_logits(self, entries: Sequence[Entry]) -> torch.Tensor:
@@ -326,7 +462,7 @@ class HybridEngine(PagedEngineBase):
         n = len(tokens)
         out = torch.zeros(self.cfg.n_layers, n, self.dp, device=self.device)
         bt = np.arange(self.max_blocks, dtype=np.int32)
-        self._step([Entry(np.asarray(tokens, dtype=np.int32), 0, bt, self.dummy_slot, [])], out)
+        self._step([Entry(np.asarray(tokens, dtype=np.int32), 0, bt, self.dummy_slot, list(range(n)))], out)
         torch.cuda.synchronize()
         return out[:, :, :self.cfg.width]
 

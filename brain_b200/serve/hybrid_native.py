@@ -31,26 +31,36 @@ class Layer(C.Structure):
                 ("inner", I), ("innerp", I), ("ch", I), ("chp", I),
                 ("off_z", I), ("off_xbc", I), ("off_dt", I),
                 ("conv_w", P), ("conv_b", P), ("dt_bias", P), ("a", P), ("d_skip", P), ("gnorm", P),
-                ("conv_state", P), ("ssm_state", P)]
+                ("conv_state", P), ("ssm_state", P),
+                ("norm2", P), ("up", Lin), ("up_b", P), ("down_b", P), ("poly", P), ("dwa", P),
+                ("qr", I), ("qrp", I), ("kvr", I), ("kvrp", I), ("rotp", I), ("own_kv", I), ("window", I),
+                ("off_dq", I), ("off_ckv", I), ("dq_norm", P), ("dkv_norm", P), ("uq", Lin), ("w_abs", P), ("w_uv", P),
+                ("expand", Lin), ("pp", I), ("wr", I), ("wrp", I),
+                ("off_r", I), ("off_kk", I), ("off_vv", I), ("off_gg", I), ("off_a", I), ("off_w1", I),
+                ("w2", Lin), ("w0", P), ("a_b", P),
+                ("blocks", I), ("bw", I), ("bwp", I), ("off_y", I), ("y_b", P), ("x_b", P), ("w_gate", P),
+                ("r_b", P), ("i_b", P), ("lam", P)]
 
 
 class Cfg(C.Structure):
     _fields_ = [("dtype", I), ("width", I), ("dp", I), ("vocab", I), ("vocabp", I), ("n_layers", I),
                 ("block_size", I), ("eps", F), ("residual_mult", F), ("embed", P), ("embed_norm", P),
-                ("final_norm", P), ("head", P), ("layers", P)]
+                ("final_norm", P), ("head", P), ("layers", P), ("depth_avg", I)]
 
 
 class Batch(C.Structure):
     _fields_ = [(n, P) for n in ("tok", "pos", "row_seq", "seq_row0", "seq_pos0", "seq_ctx", "seq_slot", "tables",
-                                 "tile_seq", "tile_qt", "want")] + \
-               [(n, I) for n in ("max_blocks", "n", "n_pre", "ns", "ns_pre", "n_tiles", "n_want", "max_len")]
+                                 "tile_seq", "tile_qt", "want", "exp_src", "kv_row0", "kv_pos0")] + \
+               [(n, I) for n in ("n_exp", "max_blocks", "n", "n_pre", "ns", "ns_pre", "n_tiles", "n_want", "max_len")]
 
 
 class Work(C.Structure):
     _fields_ = [(n, P) for n in ("x", "h", "proj", "cat", "xbc", "dt", "y", "v_first", "part_o", "part_ml", "seg")] + \
                [("seg_floats", C.c_long), ("hn", P), ("logits", P)] + \
                [(n, I) for n in ("rows", "want_rows", "ld_proj", "ld_cat", "ld_xbc", "ld_dt", "ld_y", "ld_v", "splits",
-                                 "pool_blocks")]
+                                 "pool_blocks")] + \
+               [(n, P) for n in ("h2", "q", "qa", "ol", "ckv", "kvx", "aux")] + \
+               [(n, I) for n in ("ld_q", "ld_qa", "ld_ol", "ld_ckv", "ld_kvx", "ld_aux", "exp_rows")]
 
 
 def padded_rows(w: torch.Tensor, heads: int, size: int, sizep: int) -> torch.Tensor:
@@ -60,6 +70,16 @@ def padded_rows(w: torch.Tensor, heads: int, size: int, sizep: int) -> torch.Ten
     out = w.new_zeros(heads, sizep, w.shape[1])
     out[:, :size] = w.view(heads, size, w.shape[1])
     return out.view(heads * sizep, w.shape[1])
+
+
+def padded_groups(w: torch.Tensor, rows_p: int, cols_p: int) -> torch.Tensor:
+    """[groups, rows, cols] -> [groups, rows_p, cols_p], zeros around every matrix."""
+    g, r, c = w.shape
+    if (r, c) == (rows_p, cols_p):
+        return w.contiguous()
+    out = w.new_zeros(g, rows_p, cols_p)
+    out[:, :r, :c] = w
+    return out
 
 
 class RowStack:

@@ -47,6 +47,10 @@ struct FaFwdArgs {
   float cap_poly[6];         // ... as an odd polynomial in q.k itself, for |cap_in q.k| < 0.4
   const __nv_bfloat16* gate; // raw gate of row r, head h at gate[r ldg + h]; the output is multiplied by its
   int ldg;                   // sigmoid; may be null
+  // Windowed form (WIN): keys and values of a packed sequence in rows of their own, from kv_row0[seq] on, the
+  // first of them at position kv_pos0[seq]; a query sees the `window` latest keys (0: all), itself included
+  const int *kv_row0, *kv_pos0;
+  int window;
 };
 
 // s <- s (c0 + s^2 (c1 + s^2 (...))) for two scores with packed fp32 arithmetic.
@@ -385,7 +389,9 @@ static constexpr float kFwdTruncLog2 = 0.0041778f;   // log2(1.0029), see the pa
 // the pool's blocks (one TMA copy per block and 64-column half) instead of one copy per tile.
 // EXT: see FaFwdArgs; head sizes below the tile's are zero-filled by the copies (K, V) or multiplied by
 // zeros (Q), P is rounded to nearest when it is packed.
-template <int HD, bool PAGED, int HDV = HD, bool EXT = false>
+// WIN (with PAGED and EXT): packed sequences whose keys and values are rows of one matrix; blocks that lie
+// before every query's window are not visited.
+template <int HD, bool PAGED, int HDV = HD, bool EXT = false, bool WIN = false>
 __global__ void __launch_bounds__(192, 2)
 fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                const __grid_constant__ CUtensorMap tmV, const FaFwdArgs args) {
@@ -414,7 +420,7 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
   const int h = blockIdx.y, b = blockIdx.z;
   const int row_base = PAGED ? args.seq_row0[seq] : b * args.T;   // first packed row of this sequence
   const int T = PAGED ? args.seq_row0[seq + 1] - row_base : args.T;
-  const int S = PAGED ? args.seq_ctx[seq] : args.S;
+  const int S = (PAGED ? args.seq_ctx[seq] : args.S) - (WIN ? args.kv_pos0[seq] : 0);
   const int q0 = qt * 128;
   const int kvh = h / (args.hq / args.hk);
   const int off = S - T;
@@ -423,7 +429,12 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
     const int last = (q0 + 127 + off) / 128 + 1;
     n_blocks = last < n_blocks ? last : n_blocks;
   }
+  // first block that a query of this tile sees a key of; blocks are counted from it
+  const int window = WIN && args.window > 0 ? args.window : 0x3fffffff;
+  const int j_first = WIN ? max(q0 + off - window + 1, 0) / 128 : 0;
+  if (WIN) n_blocks -= j_first;
   const int n_units = 2 * n_blocks;
+  const int kv_base = WIN ? args.kv_row0[seq] + j_first * 128 : 0;
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -464,7 +475,11 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
           break;
         }
         mbar_expect_tx(k_full, Cfg::TILE_BYTES);
-        if (PAGED) {
+        if (WIN) {
+#pragma unroll
+          for (int c = 0; c < NSUB; ++c)
+            tma_load_3d(sK + c * Cfg::SUB_BYTES, &tmK, k_full, c * 64, kv_base + j * 128, kvh);
+        } else if (PAGED) {
           // pool layout [blocks][kv heads][block_rows][HD]: block i of this tile lands at row i*block_rows
           const int br = args.block_rows, per_tile = 128 / br;
           const int* tab = args.block_tables + (size_t)seq * args.max_blocks + j * per_tile;
@@ -485,7 +500,11 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
           break;
         }
         mbar_expect_tx(v_full, Cfg::VTILE_BYTES);
-        if (PAGED) {
+        if (WIN) {
+#pragma unroll
+          for (int c = 0; c < NSUBV; ++c)
+            tma_load_3d(sV + c * Cfg::SUB_BYTES, &tmV, v_full, c * 64, kv_base + j * 128, kvh);
+        } else if (PAGED) {
           const int br = args.block_rows, per_tile = 128 / br;
           const int* tab = args.block_tables + (size_t)seq * args.max_blocks + j * per_tile;
           for (int i = 0; i < per_tile; ++i) {
@@ -597,9 +616,10 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
         }
       }
       const float sc = capped ? 1.f : args.scale_log2;
-      const int kv0 = u * 64;
-      const bool need_mask = (kv0 + 63 > kv_limit_row);
+      const int kv0 = (WIN ? j_first * 128 : 0) + u * 64;
       const int lim = kv_limit_row - kv0;  // columns <= lim are visible
+      const int low = WIN ? q_idx + off - window + 1 - kv0 : 0;   // ... and, with a window, columns >= low
+      const bool need_mask = (kv0 + 63 > kv_limit_row) || (WIN && low > 0);
       float mx = -INFINITY;
       if (!need_mask) {
         // four independent running maxima: one chain of 32 dependent FMNMX would leave the two warps
@@ -615,8 +635,8 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
       } else {
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          if (i <= lim) mx = fmaxf(mx, __uint_as_float(r0[i]));
-          if (i + 32 <= lim) mx = fmaxf(mx, __uint_as_float(r1[i]));
+          if (i <= lim && (!WIN || i >= low)) mx = fmaxf(mx, __uint_as_float(r0[i]));
+          if (i + 32 <= lim && (!WIN || i + 32 >= low)) mx = fmaxf(mx, __uint_as_float(r1[i]));
         }
       }
       mx *= sc;
@@ -655,10 +675,10 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
         float b0 = exp2f(__uint_as_float(r1[i]) * sc - m_use);
         float b1 = exp2f(__uint_as_float(r1[i + 1]) * sc - m_use);
         if (need_mask) {
-          if (i > lim) a0 = 0.f;
-          if (i + 1 > lim) a1 = 0.f;
-          if (i + 32 > lim) b0 = 0.f;
-          if (i + 33 > lim) b1 = 0.f;
+          if (i > lim || (WIN && i < low)) a0 = 0.f;
+          if (i + 1 > lim || (WIN && i + 1 < low)) a1 = 0.f;
+          if (i + 32 > lim || (WIN && i + 32 < low)) b0 = 0.f;
+          if (i + 33 > lim || (WIN && i + 33 < low)) b1 = 0.f;
         }
         if (i & 2) ls_b += (a0 + a1) + (b0 + b1);
         else ls += (a0 + a1) + (b0 + b1);
@@ -898,6 +918,61 @@ BB_API int bb_flash_fwd_paged_x(const void* q, int ldq, const void* k_pool, cons
                                 : launch_paged_x<64, 128>(tmQ, tmK, tmV, a, n_tiles, s);
   return dv <= 64 ? launch_paged_x<128, 64>(tmQ, tmK, tmV, a, n_tiles, s)
                   : launch_paged_x<128, 128>(tmQ, tmK, tmV, a, n_tiles, s);
+}
+
+namespace bb {
+template <int HD, int HDV>
+static int launch_window(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const FaFwdArgs& a,
+                         int n_tiles, cudaStream_t s) {
+  static PerDeviceOnce once;
+  const cudaError_t e = ensure_dyn_smem(once, fa_fwd2_kernel<HD, true, HDV, true, true>, FaFwdCfg<HD, HDV>::SMEM);
+  if (e != cudaSuccess) return (int)e;
+  fa_fwd2_kernel<HD, true, HDV, true, true><<<dim3(n_tiles, a.hq, 1), 192, FaFwdCfg<HD, HDV>::SMEM, s>>>(tmQ, tmK, tmV, a);
+  return (int)cudaGetLastError();
+}
+}  // namespace bb
+
+// The same over keys and values that are rows of matrices of pitch ldkv (head h at columns h dq | h dv; kv_rows
+// rows): sequence s owns rows [kv_row0[s], kv_row0[s + 1]), the first of them at position kv_pos0[s]; a query
+// sees its `window` latest keys, itself included (0: all that are there).  Head sizes as above.
+BB_API int bb_flash_fwd_window(const void* q, int ldq, const void* k, const void* v, int ldkv, int kv_rows, void* out,
+                               int ldo, const int* seq_row0, const int* kv_row0, const int* kv_pos0, const int* seq_ctx,
+                               const int* tile_seq, const int* tile_qt, int n_tiles, int total_rows, int hq, int hk, int dq,
+                               int dv, float scale, int window, void* stream) {
+  using namespace bb;
+  if (n_tiles <= 0) return BB_OK;
+  if (hq % hk || total_rows <= 0 || kv_rows <= 0 || window < 0) return BB_EARG;
+  if (dq % 8 || dv % 8 || dq > 128 || dv > 128 || ldq % 8 || ldo % 8 || ldkv % 8) return BB_ESIZE;
+  FaFwdArgs a{};
+  a.O = static_cast<__nv_bfloat16*>(out);
+  a.ldo = ldo;
+  a.hq = hq;
+  a.hk = hk;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  a.causal = 1;
+  a.err = device_error_word();
+  a.seq_row0 = seq_row0;
+  a.seq_ctx = seq_ctx;
+  a.tile_seq = tile_seq;
+  a.tile_qt = tile_qt;
+  a.dq = dq;
+  a.dv = dv;
+  a.kv_row0 = kv_row0;
+  a.kv_pos0 = kv_pos0;
+  a.window = window;
+  CUtensorMap tmQ, tmK, tmV;
+  const CUtensorMapDataType bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+  int rc = make_tmap_2d(&tmQ, bf, 2, q, (uint64_t)hq * dq, (uint64_t)total_rows, (uint64_t)ldq * 2, 64, 128);
+  if (rc) return rc;
+  rc = make_tmap_3d(&tmK, bf, 2, k, dq, kv_rows, hk, (uint64_t)ldkv * 2, (uint64_t)dq * 2, 64, 128);
+  if (rc) return rc;
+  rc = make_tmap_3d(&tmV, bf, 2, v, dv, kv_rows, hk, (uint64_t)ldkv * 2, (uint64_t)dv * 2, 64, 128);
+  if (rc) return rc;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dq <= 64) return dv <= 64 ? launch_window<64, 64>(tmQ, tmK, tmV, a, n_tiles, s)
+                                : launch_window<64, 128>(tmQ, tmK, tmV, a, n_tiles, s);
+  return dv <= 64 ? launch_window<128, 64>(tmQ, tmK, tmV, a, n_tiles, s)
+                  : launch_window<128, 128>(tmQ, tmK, tmV, a, n_tiles, s);
 }
 
 BB_API int bb_flash_fwd(const void* q, int ldq, const void* k, int ldk, const void* v, int ldv,

@@ -1,0 +1,224 @@
+// Latent attention, everything but its matrix products, for bf16 and fp32 storage:
+//   hy_latent_in     after the input projection: RMS norm of the query latent in place; the key/value latent
+//                    (normed) and the shared rotated key part into the token's page row; in blocks of their own
+//                    nothing else
+//   hy_latent_q      rotation of every head's rotated query part, in place for rows whose keys are multiplied
+//                    out, beside the absorbed query for the others
+//   hy_latent_gather page rows of prompt portions and the keys before them into one contiguous matrix
+//   hy_latent_attn   absorbed attention straight on page rows, one warp per (row, head), any sizes: the fp32
+//                    path, and the path of head sizes the tensor-core kernels do not cover
+// A page row is (latent | rotated key part): its score with the absorbed query (W_uk^T q | rotated q) is the
+// head's whole score, and the weighted sum of its first part is what W_uv turns into the head's output.
+#include "../common/host.hpp"
+#include "../common/ptx.cuh"
+#include "../common/rows.cuh"
+#include "../serve/hybrid.hpp"
+
+namespace bb {
+
+constexpr int LAT_THREADS = 128;
+
+// Rotates the pairs (2i, 2i + 1) of 8 consecutive entries starting at d.
+__device__ __forceinline__ void rotate_pairs8(float (&f)[8], const float* ct, const float* st, int d, int rot) {
+#pragma unroll
+  for (int j = 0; j < 8; j += 2) {
+    if (d + j < rot) {
+      const float c = ct[(d + j) >> 1], s = st[(d + j) >> 1], u = f[j], v = f[j + 1];
+      f[j] = u * c - v * s;
+      f[j + 1] = v * c + u * s;
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(LAT_THREADS)
+hy_latent_in_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, int ld, const int* __restrict__ pos_,
+                    const int* __restrict__ row_seq, const int* __restrict__ tables, int max_blocks, int bs, float eps) {
+  __shared__ float buf[2][32];
+  const int r = blockIdx.x;
+  T* q = proj + (size_t)r * ld + L.off_dq;
+  const T* c = proj + (size_t)r * ld + L.off_ckv;
+  float sq = 0.f, sc = 0.f;
+  for (int i = threadIdx.x * 8; i < L.qrp; i += LAT_THREADS * 8) {
+    float f[8];
+    load8(q + i, f);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) sq += f[j] * f[j];
+  }
+  if (L.own_kv)
+    for (int i = threadIdx.x * 8; i < L.kvrp; i += LAT_THREADS * 8) {
+      float f[8];
+      load8(c + i, f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) sc += f[j] * f[j];
+    }
+  sq = block_sum(sq, buf[0]);
+  sc = block_sum(sc, buf[1]);
+  const float rq = 1.f / sqrtf(sq / (float)L.qr + eps), rc = 1.f / sqrtf(sc / (float)L.kvr + eps);
+  for (int i = threadIdx.x * 8; i < L.qrp; i += LAT_THREADS * 8) {
+    float f[8], g[8];
+    load8(q + i, f);
+    load8(L.dq_norm + i, g);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) f[j] *= rq * g[j];
+    store8(q + i, f);
+  }
+  if (!L.own_kv) return;
+  const int pos = pos_[r], width = L.kvrp + L.rotp;
+  T* page = static_cast<T*>(L.kc) + ((size_t)tables[(size_t)row_seq[r] * max_blocks + pos / bs] * bs + pos % bs) * width;
+  const float* ct = L.cos_t + (size_t)pos * (L.rot >> 1);
+  const float* st = L.sin_t + (size_t)pos * (L.rot >> 1);
+  for (int i = threadIdx.x * 8; i < width; i += LAT_THREADS * 8) {
+    float f[8], g[8];
+    load8(c + i, f);
+    if (i < L.kvrp) {
+      load8(L.dkv_norm + i, g);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[j] *= rc * g[j];
+    } else {
+      rotate_pairs8(f, ct, st, i - L.kvrp, L.rot);
+    }
+    store8(page + i, f);
+  }
+}
+
+// Rows below n_in place rotate inside q; row r of the others writes to qa row r - n_in.
+template <typename T>
+__global__ void __launch_bounds__(LAT_THREADS)
+hy_latent_q_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ q, int ldq, T* __restrict__ qa, int ldqa,
+                   const int* __restrict__ pos_, int rows, int n_in) {
+  const int vecs = L.rotp / 8;
+  const long t = (long)blockIdx.x * LAT_THREADS + threadIdx.x;
+  const int r = (int)(t / (L.hq * vecs)), hv = (int)(t % (L.hq * vecs));
+  if (r >= rows) return;
+  const int h = hv / vecs, d = (hv % vecs) * 8, pos = pos_[r];
+  T* src = q + (size_t)r * ldq + h * (L.dkp + L.rotp) + L.dkp + d;
+  float f[8];
+  load8(src, f);
+  rotate_pairs8(f, L.cos_t + (size_t)pos * (L.rot >> 1), L.sin_t + (size_t)pos * (L.rot >> 1), d, L.rot);
+  T* dst = r < n_in ? src : qa + (size_t)(r - n_in) * ldqa + h * (L.kvrp + L.rotp) + L.kvrp + d;
+  store8(dst, f);
+}
+
+__global__ void __launch_bounds__(LAT_THREADS)
+hy_latent_gather_kernel(const uint4* __restrict__ pages, const int* __restrict__ src, uint4* __restrict__ out, int vecs,
+                        int ld_vecs, int rows, int pool_rows) {
+  const long t = (long)blockIdx.x * LAT_THREADS + threadIdx.x;
+  const int r = (int)(t / vecs), v = (int)(t % vecs);
+  if (r >= rows) return;
+  const int p = min(max(src[r], 0), pool_rows - 1);
+  out[(size_t)r * ld_vecs + v] = pages[(size_t)p * vecs + v];
+}
+
+// V: elements of a lane (page rows up to 32 V wide).  Row r of qa / out is batch row r.
+template <typename T, int V>
+__global__ void __launch_bounds__(LAT_THREADS)
+hy_latent_attn_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ qa, int ldq, T* __restrict__ out, int ldo,
+                      const int* __restrict__ pos_, const int* __restrict__ row_seq, const int* __restrict__ tables,
+                      int max_blocks, int bs, int rows) {
+  const int w = (blockIdx.x * LAT_THREADS + threadIdx.x) >> 5, lane = threadIdx.x & 31;
+  if (w >= rows * L.hq) return;
+  const int r = w / L.hq, h = w % L.hq, width = L.kvrp + L.rotp;
+  const T* q = qa + (size_t)r * ldq + h * width;
+  float qf[V], o[V];
+#pragma unroll
+  for (int i = 0; i < V; ++i) {
+    const int d = lane + 32 * i;
+    qf[i] = d < width ? to_f(q[d]) * L.scale : 0.f;
+    o[i] = 0.f;
+  }
+  const int last = pos_[r], first = L.window > 0 ? max(0, last - L.window + 1) : 0;
+  const int* bt = tables + (size_t)row_seq[r] * max_blocks;
+  const T* pages = static_cast<const T*>(L.kc);
+  float m = -INFINITY, l = 0.f;
+  for (int j = first; j <= last; ++j) {
+    const T* row = pages + ((size_t)bt[j / bs] * bs + j % bs) * width;
+    float k[V], s = 0.f;
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      const int d = lane + 32 * i;
+      k[i] = d < width ? to_f(row[d]) : 0.f;
+      s = fmaf(qf[i], k[i], s);
+    }
+    s = warp_sum(s);
+    const float mn = fmaxf(m, s);
+    const float al = expf(m - mn), p = expf(s - mn);
+    l = fmaf(l, al, p);
+    m = mn;
+#pragma unroll
+    for (int i = 0; i < V; ++i) o[i] = fmaf(p, k[i], o[i] * al);
+  }
+  const float f = 1.f / l;
+  T* dst = out + (size_t)r * ldo + h * L.kvrp;
+#pragma unroll
+  for (int i = 0; i < V; ++i) {
+    const int d = lane + 32 * i;
+    if (d < L.kvrp) dst[d] = from_f<T>(o[i] * f);
+  }
+}
+
+template <typename T>
+static int launch_attn(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, int bs, int r0, cudaStream_t s) {
+  const int rows = b.n - r0, width = L.kvrp + L.rotp;
+  const int grid = (int)(((long)rows * L.hq * 32 + LAT_THREADS - 1) / LAT_THREADS);
+#define BB_LAUNCH_LA(V)                                                                                            \
+  hy_latent_attn_kernel<T, V><<<grid, LAT_THREADS, 0, s>>>(L, static_cast<const T*>(w.qa), w.ld_qa,                \
+                                                           static_cast<T*>(w.ol), w.ld_ol, b.pos + r0,             \
+                                                           b.row_seq + r0, b.tables, b.max_blocks, bs, rows)
+  if (width <= 128) BB_LAUNCH_LA(4);
+  else if (width <= 256) BB_LAUNCH_LA(8);
+  else if (width <= 640) BB_LAUNCH_LA(20);
+  else if (width <= 1280) BB_LAUNCH_LA(40);
+  else return BB_ESIZE;
+#undef BB_LAUNCH_LA
+  return (int)cudaGetLastError();
+}
+
+}  // namespace bb
+
+using namespace bb;
+
+BB_API int bb_hy_latent_in(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream) {
+  cudaStream_t s = (cudaStream_t)stream;
+  if (c->dtype)
+    hy_latent_in_kernel<float><<<b->n, LAT_THREADS, 0, s>>>(*L, static_cast<float*>(w->proj), w->ld_proj, b->pos, b->row_seq,
+                                                            b->tables, b->max_blocks, c->block_size, c->eps);
+  else
+    hy_latent_in_kernel<__nv_bfloat16><<<b->n, LAT_THREADS, 0, s>>>(*L, static_cast<__nv_bfloat16*>(w->proj), w->ld_proj,
+                                                                    b->pos, b->row_seq, b->tables, b->max_blocks,
+                                                                    c->block_size, c->eps);
+  return (int)cudaGetLastError();
+}
+
+// n_in: leading rows whose rotated queries stay in place.
+BB_API int bb_hy_latent_q(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int n_in, void* stream) {
+  cudaStream_t s = (cudaStream_t)stream;
+  const long t = (long)b->n * L->hq * (L->rotp / 8);
+  const int grid = (int)((t + LAT_THREADS - 1) / LAT_THREADS);
+  if (c->dtype)
+    hy_latent_q_kernel<float><<<grid, LAT_THREADS, 0, s>>>(*L, static_cast<float*>(w->q), w->ld_q, static_cast<float*>(w->qa),
+                                                           w->ld_qa, b->pos, b->n, n_in);
+  else
+    hy_latent_q_kernel<__nv_bfloat16><<<grid, LAT_THREADS, 0, s>>>(*L, static_cast<__nv_bfloat16*>(w->q), w->ld_q,
+                                                                   static_cast<__nv_bfloat16*>(w->qa), w->ld_qa, b->pos, b->n,
+                                                                   n_in);
+  return (int)cudaGetLastError();
+}
+
+BB_API int bb_hy_latent_gather(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream) {
+  if (b->n_exp <= 0) return BB_OK;
+  if (c->dtype || b->n_exp > w->exp_rows) return BB_EARG;
+  const int vecs = (L->kvrp + L->rotp) / 8;
+  const long t = (long)b->n_exp * vecs;
+  hy_latent_gather_kernel<<<(int)((t + LAT_THREADS - 1) / LAT_THREADS), LAT_THREADS, 0, (cudaStream_t)stream>>>(
+      static_cast<const uint4*>(L->kc), b->exp_src, static_cast<uint4*>(w->ckv), vecs, w->ld_ckv / 8, b->n_exp,
+      w->pool_blocks * c->block_size);
+  return (int)cudaGetLastError();
+}
+
+// Absorbed attention of batch rows r0 .. n - 1 (rows 0 .. of w->qa and w->ol).
+BB_API int bb_hy_latent_attn(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int r0, void* stream) {
+  if (r0 >= b->n) return BB_OK;
+  return c->dtype ? launch_attn<float>(*L, *w, *b, c->block_size, r0, (cudaStream_t)stream)
+                  : launch_attn<__nv_bfloat16>(*L, *w, *b, c->block_size, r0, (cudaStream_t)stream);
+}

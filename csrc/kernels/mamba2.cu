@@ -1,7 +1,8 @@
 // Mamba-2 mixer kernels (fp32 state and recurrence; bf16 or fp32 projections and convolution).
-//   hy_conv         causal per-channel convolution + bias + silu over the packed rows of prompt portions;
-//                   taps that reach back before the portion come from the sequence's state slot.  The same
-//                   launch turns the raw step sizes into softplus(dt + bias).
+//   hy_conv         causal per-channel convolution + bias (+ silu) over packed rows; taps that reach back
+//                   before a portion come from the sequence's state slot.  The same launch turns raw step
+//                   sizes, where a layer has them, into softplus(dt + bias).  Inputs may carry a bias of their
+//                   own, which places before the start of the sequence do not have.
 //   hy_ssm_scan     recurrence of a prompt portion, one token after the other, one block per (sequence,
 //                   head): any sizes, fp32 throughout
 //   hy_ssm_decode   one token per sequence: convolution, step size, state update and output in one
@@ -41,13 +42,13 @@ __device__ __forceinline__ Raw4<T> conv_tap(const BbHyLayer& L, const T* proj, i
 
 // TAPS = 4 keeps a thread's inputs in registers as they are stored; TAPS = 0 reads every tap again (any
 // length).
-template <typename T, int TAPS>
+template <typename T, int TAPS, bool SILU>
 __global__ void __launch_bounds__(128, sizeof(T) == 2 ? 7 : 5)
 hy_conv_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, int ld, T* __restrict__ xbc, int ldx,
-               float* __restrict__ dt, int lddt, const __grid_constant__ BbHyBatch b) {
+               float* __restrict__ dt, int lddt, const __grid_constant__ BbHyBatch b, int rows) {
   const int cv = blockIdx.x * 128 + threadIdx.x;   // vector of 4 channels, then vectors of 4 step sizes
   const int nch = L.chp / 4, ndt = (L.heads + 7) / 8 * 2;
-  const int r0 = blockIdx.y * CONV_ROWS, r1 = min(r0 + CONV_ROWS, b.n_pre);
+  const int r0 = blockIdx.y * CONV_ROWS, r1 = min(r0 + CONV_ROWS, rows);
   if (cv >= nch + ndt) return;
   if (cv >= nch) {
     const int h0 = (cv - nch) * 4;
@@ -64,6 +65,11 @@ hy_conv_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, 
   const int c = cv * 4;
   const float4 bias4 = *reinterpret_cast<const float4*>(L.conv_b + c);
   const float bias[4] = {bias4.x, bias4.y, bias4.z, bias4.w};
+  float xb[4] = {0.f, 0.f, 0.f, 0.f};              // bias of the inputs
+  if (!SILU) {
+    const float4 t = *reinterpret_cast<const float4*>(L.x_b + c);
+    xb[0] = t.x; xb[1] = t.y; xb[2] = t.z; xb[3] = t.w;
+  }
   if constexpr (TAPS > 0) {
     constexpr int K = TAPS - 1;
     Raw4<T> raw[CONV_ROWS + K];   // raw[K + i]: row r0 + i; before it the inputs ahead of r0
@@ -102,12 +108,14 @@ hy_conv_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, 
         }
       }
       Raw4<T> o;
+      const int first = SILU ? 0 : K - b.pos[r];       // taps before it lie ahead of the sequence
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         float s = bias[j];
 #pragma unroll
-        for (int k = 0; k < TAPS; ++k) s = fmaf(w[k][j], to_f(raw[i + k].v[j]), s);
-        o.v[j] = from_f<T>(silu_as<T>(s));
+        for (int k = 0; k < TAPS; ++k)
+          s = fmaf(w[k][j], SILU ? to_f(raw[i + k].v[j]) : (k >= first ? to_f(raw[i + k].v[j]) + xb[j] : 0.f), s);
+        o.v[j] = from_f<T>(SILU ? silu_as<T>(s) : s);
       }
       *reinterpret_cast<Raw4<T>*>(xbc + (size_t)r * ldx + c) = o;
     }
@@ -120,11 +128,11 @@ hy_conv_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, 
         const Raw4<T> u = conv_tap(L, proj, ld, r, k, c, pos, pos0, slot);
         const float* w = L.conv_w + (size_t)(L.taps - 1 - k) * L.chp + c;
 #pragma unroll
-        for (int j = 0; j < 4; ++j) s[j] = fmaf(w[j], to_f(u.v[j]), s[j]);
+        for (int j = 0; j < 4; ++j) s[j] = fmaf(w[j], k <= pos ? to_f(u.v[j]) + xb[j] : 0.f, s[j]);
       }
       Raw4<T> o;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) o.v[j] = from_f<T>(silu_as<T>(s[j]));
+      for (int j = 0; j < 4; ++j) o.v[j] = from_f<T>(SILU ? silu_as<T>(s[j]) : s[j]);
       *reinterpret_cast<Raw4<T>*>(xbc + (size_t)r * ldx + c) = o;
     }
   }
@@ -288,15 +296,15 @@ hy_ssm_decode_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
   }
 }
 
-template <typename T>
-static int launch_conv(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, cudaStream_t s) {
+template <typename T, bool SILU>
+static int launch_conv(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, int rows, cudaStream_t s) {
   const int vecs = L.chp / 4 + (L.heads + 7) / 8 * 2;
-  dim3 grid((vecs + 127) / 128, (b.n_pre + CONV_ROWS - 1) / CONV_ROWS);
+  dim3 grid((vecs + 127) / 128, (rows + CONV_ROWS - 1) / CONV_ROWS);
   if (grid.y > 65535) return BB_ESIZE;
   const T* proj = static_cast<const T*>(w.proj);
   T* xbc = static_cast<T*>(w.xbc);
-  if (L.taps == 4) hy_conv_kernel<T, 4><<<grid, 128, 0, s>>>(L, proj, w.ld_proj, xbc, w.ld_xbc, w.dt, w.ld_dt, b);
-  else hy_conv_kernel<T, 0><<<grid, 128, 0, s>>>(L, proj, w.ld_proj, xbc, w.ld_xbc, w.dt, w.ld_dt, b);
+  if (L.taps == 4) hy_conv_kernel<T, 4, SILU><<<grid, 128, 0, s>>>(L, proj, w.ld_proj, xbc, w.ld_xbc, w.dt, w.ld_dt, b, rows);
+  else hy_conv_kernel<T, 0, SILU><<<grid, 128, 0, s>>>(L, proj, w.ld_proj, xbc, w.ld_xbc, w.dt, w.ld_dt, b, rows);
   return (int)cudaGetLastError();
 }
 
@@ -342,8 +350,14 @@ using namespace bb;
 
 BB_API int bb_hy_conv(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream) {
   if (b->n_pre <= 0) return BB_OK;
-  return c->dtype ? launch_conv<float>(*L, *w, *b, (cudaStream_t)stream)
-                  : launch_conv<__nv_bfloat16>(*L, *w, *b, (cudaStream_t)stream);
+  return c->dtype ? launch_conv<float, true>(*L, *w, *b, b->n_pre, (cudaStream_t)stream)
+                  : launch_conv<__nv_bfloat16, true>(*L, *w, *b, b->n_pre, (cudaStream_t)stream);
+}
+
+// The same without activation, with the inputs' bias x_b, for every row of the step.
+BB_API int bb_hy_conv_linear(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream) {
+  return c->dtype ? launch_conv<float, false>(*L, *w, *b, b->n, (cudaStream_t)stream)
+                  : launch_conv<__nv_bfloat16, false>(*L, *w, *b, b->n, (cudaStream_t)stream);
 }
 
 BB_API int bb_hy_ssm_scan(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream) {

@@ -1,0 +1,194 @@
+// Gated linear recurrence per channel (fp32 state; bf16 or fp32 projections, convolution and gates' maps):
+//   r = sigmoid(gate + bias), i = sigmoid(gate + bias), log a = -lam r,
+//   S <- a S + sqrt(1 - a^2) i u,   output S gelu(y + bias).
+//   hy_rglru_scan    prompt portions: a block owns 64 channels of a sequence and takes 128 tokens at a time,
+//                    eight to a warp; the warps' (product of a, local S) pairs are chained through shared memory
+//   hy_rglru_step    one token per sequence, one thread per two channels
+// Both write the sequence's last taps - 1 raw convolution inputs into its slot (the convolution ran before).
+// State: [slot][channel] fp32; a sequence at position 0 starts from zeros whatever its slot holds.
+#include "../common/host.hpp"
+#include "../common/rows.cuh"
+#include "../serve/hybrid.hpp"
+
+namespace bb {
+
+template <typename T>
+struct Pair {
+  T v[2];
+};
+template <typename T>
+__device__ __forceinline__ float2 load_pair(const T* p) {
+  struct alignas(sizeof(T) * 2) P {
+    T v[2];
+  };
+  const P q = *reinterpret_cast<const P*>(p);
+  return make_float2(to_f(q.v[0]), to_f(q.v[1]));
+}
+template <typename T>
+__device__ __forceinline__ void store_pair(T* p, float a, float b) {
+  struct alignas(sizeof(T) * 2) P {
+    T v[2];
+  };
+  P q;
+  q.v[0] = from_f<T>(a);
+  q.v[1] = from_f<T>(b);
+  *reinterpret_cast<P*>(p) = q;
+}
+
+// Everything below is 32-bit; with bf16 storage exponentials and divisions are the hardware's (2^-22).
+template <typename T>
+__device__ __forceinline__ float gelu_as(float z) {
+  const float t = 0.79788456080286536f * fmaf(0.044715f * z * z, z, z);   // sqrt(2 / pi) (z + 0.044715 z^3)
+  if constexpr (sizeof(T) == 2) return z * __fdividef(1.f, 1.f + __expf(-2.f * t));
+  else return 0.5f * z * (1.f + tanhf(t));
+}
+// log a = -x (x >= 0) -> a and sqrt(1 - a^2)
+template <typename T>
+__device__ __forceinline__ float2 decay_of(float x) {
+  if constexpr (sizeof(T) == 2) {
+    const float a = __expf(-x), y = 2.f * x;
+    // 1 - e^-y: its series where the difference would cancel
+    const float d = y < 0.05f ? y * fmaf(y, fmaf(y, fmaf(y, -1.f / 24.f, 1.f / 6.f), -0.5f), 1.f) : 1.f - a * a;
+    return make_float2(a, sqrtf(d));
+  } else {
+    return make_float2(expf(-x), sqrtf(-expm1f(-2.f * x)));
+  }
+}
+
+struct LruChannels {
+  float2 yb, rb, ib, lam;
+};
+__device__ __forceinline__ LruChannels lru_channels(const BbHyLayer& L, int c) {
+  auto two = [&](const float* p) { return *reinterpret_cast<const float2*>(p + c); };
+  return {two(L.y_b), two(L.r_b), two(L.i_b), two(L.lam)};
+}
+// Raw values of a token and two channels -> decay and input of the recurrence.
+template <typename T>
+__device__ __forceinline__ void lru_token(const LruChannels& p, float2 r, float2 i, float2 u, float2& a, float2& in) {
+  const float2 d0 = decay_of<T>(p.lam.x * sigmoid_as<T>(r.x + p.rb.x)), d1 = decay_of<T>(p.lam.y * sigmoid_as<T>(r.y + p.rb.y));
+  a = make_float2(d0.x, d1.x);
+  in = make_float2(d0.y * sigmoid_as<T>(i.x + p.ib.x) * u.x, d1.y * sigmoid_as<T>(i.y + p.ib.y) * u.y);
+}
+
+template <typename T>
+__device__ __forceinline__ void keep_input(const BbHyLayer& L, const T* row, int c, int pos, int ctx, int slot) {
+  const int keep = L.taps - 1;
+  if (keep <= 0 || pos < ctx - keep) return;
+  T* ring = static_cast<T*>(L.conv_state) + ((size_t)slot * keep + pos % keep) * L.chp + c;
+  const float2 x = load_pair(row + L.off_xbc + c);
+  store_pair(ring, x.x, x.y);
+}
+
+constexpr int LRU_WARPS = 16, LRU_T = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(LRU_WARPS * 32)
+hy_rglru_scan_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, int ld, const T* __restrict__ u, int ldu,
+                     const T* __restrict__ gates, int ldg, T* __restrict__ cat, int ldc, const __grid_constant__ BbHyBatch b) {
+  __shared__ float2 chain[2][LRU_WARPS][2][32];      // [buffer][warp][product of a | local S][lane]
+  const int seq = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int c = blockIdx.x * 64 + lane * 2;
+  const bool live = c < L.chp;
+  const int cc = live ? c : 0;
+  const int r0 = b.seq_row0[seq], n = b.seq_row0[seq + 1] - r0, slot = b.seq_slot[seq], pos0 = b.seq_pos0[seq];
+  const int ctx = pos0 + n;
+  const int g0 = (cc / L.bwp) * 2 * L.bwp + cc % L.bwp;
+  const LruChannels ch = lru_channels(L, cc);
+  float* state = L.ssm_state + (size_t)slot * L.chp + cc;
+  float2 carry = pos0 == 0 ? make_float2(0.f, 0.f) : *reinterpret_cast<const float2*>(state);
+  for (int t0 = 0, it = 0; t0 < n; t0 += LRU_WARPS * LRU_T, ++it) {
+    const int tw = t0 + warp * LRU_T;
+    float2 p[LRU_T], s[LRU_T];
+    {
+      float2 rr[LRU_T], ii[LRU_T], uu[LRU_T];
+#pragma unroll
+      for (int k = 0; k < LRU_T; ++k) {
+        const size_t row = r0 + min(tw + k, n - 1);
+        rr[k] = load_pair(gates + row * ldg + g0);
+        ii[k] = load_pair(gates + row * ldg + g0 + L.bwp);
+        uu[k] = load_pair(u + row * ldu + cc);
+      }
+      float2 pa = make_float2(1.f, 1.f), sa = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int k = 0; k < LRU_T; ++k) {
+        float2 a, in;
+        lru_token<T>(ch, rr[k], ii[k], uu[k], a, in);
+        if (tw + k >= n) {           // past the end: nothing changes
+          a = make_float2(1.f, 1.f);
+          in = make_float2(0.f, 0.f);
+        }
+        sa = make_float2(fmaf(a.x, sa.x, in.x), fmaf(a.y, sa.y, in.y));
+        pa = make_float2(pa.x * a.x, pa.y * a.y);
+        p[k] = pa;
+        s[k] = sa;
+      }
+    }
+    chain[it & 1][warp][0][lane] = p[LRU_T - 1];
+    chain[it & 1][warp][1][lane] = s[LRU_T - 1];
+    __syncthreads();
+    float2 mine = carry;
+#pragma unroll
+    for (int w = 0; w < LRU_WARPS; ++w) {
+      if (w == warp) mine = carry;
+      const float2 cp = chain[it & 1][w][0][lane], cs = chain[it & 1][w][1][lane];
+      carry = make_float2(fmaf(cp.x, carry.x, cs.x), fmaf(cp.y, carry.y, cs.y));
+    }
+#pragma unroll
+    for (int k = 0; k < LRU_T; ++k) {
+      if (tw + k < n && live) {
+        const size_t row = r0 + tw + k;
+        const float2 yv = load_pair(proj + row * ld + L.off_y + cc);
+        const float sx = fmaf(p[k].x, mine.x, s[k].x), sy = fmaf(p[k].y, mine.y, s[k].y);
+        store_pair(cat + row * ldc + cc, sx * gelu_as<T>(yv.x + ch.yb.x), sy * gelu_as<T>(yv.y + ch.yb.y));
+        keep_input<T>(L, proj + row * ld, cc, pos0 + tw + k, ctx, slot);
+      }
+    }
+  }
+  if (warp == 0 && live) *reinterpret_cast<float2*>(state) = carry;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+hy_rglru_step_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, int ld, const T* __restrict__ u, int ldu,
+                     const T* __restrict__ gates, int ldg, T* __restrict__ cat, int ldc, const __grid_constant__ BbHyBatch b) {
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 2;
+  if (c >= L.chp) return;
+  const int seq = b.ns_pre + blockIdx.y;
+  const size_t row = b.n_pre + blockIdx.y;
+  const int pos = b.pos[row], slot = b.seq_slot[seq];
+  const int g0 = (c / L.bwp) * 2 * L.bwp + c % L.bwp;
+  float* state = L.ssm_state + (size_t)slot * L.chp + c;
+  const float2 old = *reinterpret_cast<const float2*>(state);
+  const float2 yv = load_pair(proj + row * ld + L.off_y + c);
+  const LruChannels ch = lru_channels(L, c);
+  float2 a, in;
+  lru_token<T>(ch, load_pair(gates + row * ldg + g0), load_pair(gates + row * ldg + g0 + L.bwp), load_pair(u + row * ldu + c), a, in);
+  const bool fresh = pos == 0;
+  const float2 s = make_float2(fresh ? in.x : fmaf(a.x, old.x, in.x), fresh ? in.y : fmaf(a.y, old.y, in.y));
+  *reinterpret_cast<float2*>(state) = s;
+  store_pair(cat + row * ldc + c, s.x * gelu_as<T>(yv.x + ch.yb.x), s.y * gelu_as<T>(yv.y + ch.yb.y));
+  keep_input<T>(L, proj + row * ld, c, pos, pos + 1, slot);
+}
+
+template <typename T>
+static int launch_rglru(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, cudaStream_t s) {
+  const T *proj = static_cast<const T*>(w.proj), *u = static_cast<const T*>(w.xbc), *g = static_cast<const T*>(w.aux);
+  T* cat = static_cast<T*>(w.cat);
+  if (b.ns_pre > 0)
+    hy_rglru_scan_kernel<T><<<dim3((L.chp + 63) / 64, b.ns_pre), LRU_WARPS * 32, 0, s>>>(L, proj, w.ld_proj, u, w.ld_xbc, g,
+                                                                                         w.ld_aux, cat, w.ld_cat, b);
+  if (b.ns > b.ns_pre)
+    hy_rglru_step_kernel<T><<<dim3((L.chp + 255) / 256, b.ns - b.ns_pre), 128, 0, s>>>(L, proj, w.ld_proj, u, w.ld_xbc, g,
+                                                                                       w.ld_aux, cat, w.ld_cat, b);
+  return (int)cudaGetLastError();
+}
+
+}  // namespace bb
+
+using namespace bb;
+
+// Recurrence of every row of the step (w->xbc: convolution outputs, w->aux: gate maps) -> w->cat.
+BB_API int bb_hy_rglru(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream) {
+  return c->dtype ? launch_rglru<float>(*L, *w, *b, (cudaStream_t)stream)
+                  : launch_rglru<__nv_bfloat16>(*L, *w, *b, (cudaStream_t)stream);
+}

@@ -1,5 +1,6 @@
 // fp32 GEMM on the CUDA cores (no tensor-core rounding): C[M,N] = alpha A[M,K] B[N,K]^T, or C += that.
-// Serves the 32-bit mode of the engines; 64 x 64 tiles, 16-wide k-steps, 4 x 4 outputs per thread.
+// Serves the 32-bit mode of the engines; 64 x 64 tiles, 16-wide k-steps, 4 x 4 outputs per thread.  Several
+// products of equal shape (one per head, one per diagonal block) run side by side along the grid's z.
 #include "../common/host.hpp"
 
 namespace bb {
@@ -8,7 +9,10 @@ constexpr int SG_T = 64, SG_K = 16;
 
 __global__ void __launch_bounds__(256)
 sgemm_kernel(const float* __restrict__ A, const float* __restrict__ B, float* __restrict__ C, int M, int N, int K, int lda,
-             int ldb, int ldc, float alpha, int accumulate) {
+             int ldb, int ldc, float alpha, int accumulate, size_t a_step, size_t b_step, size_t c_step) {
+  A += blockIdx.z * a_step;
+  B += blockIdx.z * b_step;
+  C += blockIdx.z * c_step;
   __shared__ float sa[SG_K][SG_T + 4], sb[SG_K][SG_T + 4];
   const int m0 = blockIdx.y * SG_T, n0 = blockIdx.x * SG_T;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
@@ -55,6 +59,17 @@ BB_API int bb_sgemm(const float* A, const float* B, float* C, int M, int N, int 
   using namespace bb;
   if (M <= 0 || N <= 0 || K <= 0) return BB_EARG;
   sgemm_kernel<<<dim3((N + SG_T - 1) / SG_T, (M + SG_T - 1) / SG_T), 256, 0, (cudaStream_t)stream>>>(
-      A, B, C, M, N, K, lda, ldb, ldc, alpha, accumulate);
+      A, B, C, M, N, K, lda, ldb, ldc, alpha, accumulate, 0, 0, 0);
+  return (int)cudaGetLastError();
+}
+
+// C_g = A_g B_g^T for g < groups: A_g starts a_step elements after A_(g-1), C_g c_step after C_(g-1), B holds
+// [groups][N][K].
+BB_API int bb_sgemm_groups(const float* A, const float* B, float* C, int M, int N, int K, int groups, int lda, int a_step,
+                           int ldc, int c_step, void* stream) {
+  using namespace bb;
+  if (M <= 0 || N <= 0 || K <= 0 || groups <= 0) return BB_EARG;
+  sgemm_kernel<<<dim3((N + SG_T - 1) / SG_T, (M + SG_T - 1) / SG_T, groups), 256, 0, (cudaStream_t)stream>>>(
+      A, B, C, M, N, K, lda, K, ldc, 1.f, 0, a_step, (size_t)N * K, c_step);
   return (int)cudaGetLastError();
 }

@@ -14,7 +14,7 @@ struct BbHyLin {
 };
 
 struct BbHyLayer {
-  int kind;            // 0 attention, 1 mamba2
+  int kind;            // 0 attention, 1 mamba2, 2 latent attention, 3 generalised delta rule, 4 gated linear recurrence
   const float* norm;   // [dp] gain of the layer's norm (one already added where it is stored around 0)
   BbHyLin in;          // every projection that reads the normed input, stacked along the rows
   BbHyLin out;         // mixer output projection | feed-forward down projection, side by side
@@ -39,7 +39,33 @@ struct BbHyLayer {
   const float *dt_bias, *a, *d_skip;       // [heads]; a = -exp(A_log)
   const float* gnorm;                      // [innerp]
   void* conv_state;                        // [slots][max(taps - 1, 1)][chp]: raw inputs, position p at p % (taps - 1)
-  float* ssm_state;                        // [slots][heads][n][p]
+  float* ssm_state;                        // [slots][heads][n][p]; 3: [slots][heads][p][p]; 4: [slots][chp]
+  // a feed-forward with a norm and a GEMM of its own: polynomial of root-mean-square norms
+  const float* norm2;                      // [dp] (null: the feed-forward reads the mixer's norm)
+  BbHyLin up;                              // [ffp, dp]; its output takes columns off_up of the projection
+  const float *up_b, *down_b;              // [ffp], [dp]; down_b is added where the layer's residual starts
+  const float* poly;                       // [4]
+  // depth average: weights of the results so far, [layer index + 2]
+  const float* dwa;
+  // latent attention (hq heads; dk / dkp unrotated, rot / rotp rotated, dv / dvp value sizes; one page row
+  // per token in kc: latent | rotated key part, kvrp + rotp wide)
+  int qr, qrp, kvr, kvrp, rotp, own_kv, window;   // window 0: every earlier key
+  int off_dq, off_ckv;
+  const float *dq_norm, *dkv_norm;         // [qrp], [kvrp]
+  BbHyLin uq;                              // [hq (dkp + rotp), qrp]
+  const void *w_abs;                       // [hq][kvrp][dkp]: queries into the latents' space
+  const void *w_uv;                        // [hq][dvp][kvrp]: values out of it
+  BbHyLin expand;                          // [hq (dkp + rotp) | hq dvp, kvrp + rotp]: keys and values of page rows
+  // generalised delta rule (heads of p, padded pp)
+  int pp, wr, wrp;                         // ... and the rank of its decay
+  int off_r, off_kk, off_vv, off_gg, off_a, off_w1;
+  BbHyLin w2;                              // [heads pp, wrp]
+  const float *w0, *a_b;                   // [heads pp]
+  // gated linear recurrence (blocks of bw channels, padded bwp; chp = innerp = blocks bwp)
+  int blocks, bw, bwp, off_y;
+  const float *y_b, *x_b;                  // [chp]
+  const void* w_gate;                      // [blocks][2 bwp][bwp]: recurrence gate rows, then input gate rows
+  const float *r_b, *i_b, *lam;            // [chp]; lam = decay constant times softplus of the parameter
 };
 
 struct BbHyCfg {
@@ -49,6 +75,7 @@ struct BbHyCfg {
   const float *embed_norm, *final_norm;    // [dp]
   const void* head;                        // [vocabp, dp]
   const BbHyLayer* layers;
+  int depth_avg;                           // layers pass on weighted sums of all results (see BbHyWork::x)
 };
 
 // One packed batch: rows of prompt portions first (n_pre rows of ns_pre sequences), then one row for
@@ -60,11 +87,16 @@ struct BbHyBatch {
   const int* tables;                       // [ns, max_blocks]
   const int *tile_seq, *tile_qt;           // 128-row query tiles of the prompt portions
   const int *want;                         // [n_want] rows whose logits are asked for (null: every row)
+  // page rows whose keys and values prompt portions multiply out: n_exp rows of the page pool, of sequence
+  // s from kv_row0[s], the first of them at position kv_pos0[s]
+  const int *exp_src, *kv_row0, *kv_pos0;
+  int n_exp;
   int max_blocks, n, n_pre, ns, ns_pre, n_tiles, n_want, max_len;   // max_len: longest portion
 };
 
 struct BbHyWork {
-  float* x;          // [rows, dp] residual stream
+  float* x;          // [rows, dp] residual stream; with depth averages [n_layers + 1][rows, dp]: the
+                     // embedding, then every layer's result
   void* h;           // [rows, dp]
   void* proj;        // [rows, ld_proj]
   void* cat;         // [rows, ld_cat]
@@ -79,4 +111,8 @@ struct BbHyWork {
   float* logits;     // [want, vocabp]
   int rows, want_rows, ld_proj, ld_cat, ld_xbc, ld_dt, ld_y, ld_v, splits;
   int pool_blocks;
+  // second normed input, latent attention (queries, absorbed queries, latent outputs; gathered page rows and
+  // their keys and values), and gate / decay projections of the recurrences
+  void *h2, *q, *qa, *ol, *ckv, *kvx, *aux;
+  int ld_q, ld_qa, ld_ol, ld_ckv, ld_kvx, ld_aux, exp_rows;
 };

@@ -5,6 +5,9 @@
 //   -> mixer (attention over the pages, or the state-space recurrence over the slots)
 //   -> ONE output GEMM over (mixer output | feed-forward product), scaled and added into the fp32
 //      residual stream by its epilogue.
+// Designs with depth averages keep every layer's result: a layer starts from the weighted sum of all of them
+// (written where its own result will be, so the output GEMM adds in place), and its feed-forward has a norm
+// and a GEMM of its own.
 // bf16: the tensor-core GEMM, paged flash prefill, split-KV decode attention and chunked state-space
 // kernels; fp32: the CUDA-core forms of the same steps.
 #include <cstdint>
@@ -28,6 +31,25 @@ int bb_hy_conv(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const Bb
 int bb_hy_ssm_scan(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
 int bb_ssd_chunk(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
 int bb_hy_ssm_decode(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_conv_linear(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_mix_norm(const BbHyCfg* c, int li, const BbHyWork* w, const BbHyBatch* b, float* trace, void* stream);
+int bb_hy_polynorm(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream);
+int bb_hy_latent_in(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_latent_q(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int n_in, void* stream);
+int bb_hy_latent_gather(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_latent_attn(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int r0, void* stream);
+int bb_hy_delta_tanh(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_delta_scan(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_delta_post(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_rglru(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_gemm_bf16_groups(const void* A, const void* B, void* C, int M, int N, int K, int groups, int lda, int a_step, int ldc,
+                        int c_step, void* stream);
+int bb_sgemm_groups(const float* A, const float* B, float* C, int M, int N, int K, int groups, int lda, int a_step, int ldc,
+                    int c_step, void* stream);
+int bb_flash_fwd_window(const void* q, int ldq, const void* k, const void* v, int ldkv, int kv_rows, void* out, int ldo,
+                        const int* seq_row0, const int* kv_row0, const int* kv_pos0, const int* seq_ctx, const int* tile_seq,
+                        const int* tile_qt, int n_tiles, int total_rows, int hq, int hk, int dq, int dv, float scale,
+                        int window, void* stream);
 int bb_attn_rows(int dtype, const void* q, int ldq, const void* kc, const void* vc, const int* pos, const int* row_seq,
                  const int* tables, int max_blocks, int bs, void* out, int ldo, const void* gate, int ldg, int rows, int hq,
                  int hk, int dk, int dv, int dkp, int dvp, float scale, float softcap, void* stream);
@@ -54,6 +76,16 @@ int project(const BbHyCfg& c, const BbHyLin& L, const void* x, int ldx, void* y,
     return bb_sgemm(static_cast<const float*>(x), static_cast<const float*>(L.w), static_cast<float*>(y), rows, L.n, L.k,
                     ldx, L.k, ldy, 1.f, 0, s);
   return bb_gemm_bf16(x, L.w, y, nullptr, rows, L.n, L.k, ldx, L.k, ldy, 0, 0, 0, 1.f, 0, 0, s);
+}
+
+// y_g = x_g W_g^T for column ranges x_g of x and y_g of y, `xs` and `ys` elements apart; W [groups][n][k]
+int project_groups(const BbHyCfg& c, const void* w, int groups, int n, int k, const void* x, int ldx, int xs, void* y, int ldy,
+                   int ys, int rows, void* s) {
+  if (rows <= 0) return BB_OK;
+  if (c.dtype)
+    return bb_sgemm_groups(static_cast<const float*>(x), static_cast<const float*>(w), static_cast<float*>(y), rows, n, k,
+                           groups, ldx, xs, ldy, ys, s);
+  return bb_gemm_bf16_groups(x, w, y, rows, n, k, groups, ldx, xs, ldy, ys, s);
 }
 
 // fp32 y (+)= alpha x W^T
@@ -120,18 +152,94 @@ int mamba2(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBa
   return bb_hy_mamba_post(&c, &L, &w, &b, s);
 }
 
+// Prompt portions in bf16: keys and values of the window's page rows are multiplied out and the flash kernel
+// runs over them; decoded rows (and every row where that kernel does not reach): queries go into the latents'
+// space and attention runs on the page rows themselves.
+int latent_attention(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
+  const int dq = L.dkp + L.rotp, width = L.kvrp + L.rotp;
+  const int n_in = L.expand.w ? b.n_pre : 0;
+  BB_TRY(bb_hy_latent_in(&c, &L, &w, &b, s));
+  BB_TRY(project(c, L.uq, at(c, w.proj, L.off_dq), w.ld_proj, w.q, w.ld_q, b.n, s));
+  BB_TRY(bb_hy_latent_q(&c, &L, &w, &b, n_in, s));
+  if (n_in > 0) {
+    BB_TRY(bb_hy_latent_gather(&c, &L, &w, &b, s));
+    BB_TRY(project(c, L.expand, w.ckv, w.ld_ckv, w.kvx, w.ld_kvx, b.n_exp, s));
+    BB_TRY(bb_flash_fwd_window(w.q, w.ld_q, w.kvx, at(c, w.kvx, (size_t)L.hq * dq), w.ld_kvx, b.n_exp, w.cat, w.ld_cat,
+                               b.seq_row0, b.kv_row0, b.kv_pos0, b.seq_ctx, b.tile_seq, b.tile_qt, b.n_tiles, b.n_pre, L.hq,
+                               L.hq, dq, L.dvp, L.scale, L.window, s));
+  }
+  const int rows = b.n - n_in;
+  BB_TRY(project_groups(c, L.w_abs, L.hq, L.kvrp, L.dkp, at(c, w.q, (size_t)n_in * w.ld_q), w.ld_q, dq, w.qa, w.ld_qa, width,
+                        rows, s));
+  BB_TRY(bb_hy_latent_attn(&c, &L, &w, &b, n_in, s));
+  return project_groups(c, L.w_uv, L.hq, L.dvp, L.kvrp, w.ol, w.ld_ol, L.kvrp, at(c, w.cat, (size_t)n_in * w.ld_cat), w.ld_cat,
+                        L.dvp, rows, s);
+}
+
+int general_delta(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
+  BB_TRY(bb_hy_delta_tanh(&c, &L, &w, &b, s));
+  BB_TRY(project(c, L.w2, at(c, w.proj, L.off_w1), w.ld_proj, w.aux, w.ld_aux, b.n, s));
+  BB_TRY(bb_hy_delta_scan(&c, &L, &w, &b, s));
+  return bb_hy_delta_post(&c, &L, &w, &b, s);
+}
+
+int rglru(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
+  BB_TRY(bb_hy_conv_linear(&c, &L, &w, &b, s));
+  BB_TRY(project_groups(c, L.w_gate, L.blocks, 2 * L.bwp, L.bwp, w.xbc, w.ld_xbc, L.bwp, w.aux, w.ld_aux, 2 * L.bwp, b.n, s));
+  return bb_hy_rglru(&c, &L, &w, &b, s);
+}
+
+int mixer(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
+  switch (L.kind) {
+    case 0: return attention(c, L, w, b, s);
+    case 1: return mamba2(c, L, w, b, s);
+    case 2: return latent_attention(c, L, w, b, s);
+    case 3: return general_delta(c, L, w, b, s);
+    case 4: return rglru(c, L, w, b, s);
+    default: return BB_EARG;
+  }
+}
+
+int forward_depth(const BbHyCfg& c, const BbHyWork& w, const BbHyBatch& b, float* trace, void* s) {
+  const size_t level = (size_t)w.rows * c.dp;
+  for (int li = 0; li < c.n_layers; ++li) {
+    const BbHyLayer& L = c.layers[li];
+    BB_TRY(bb_hy_mix_norm(&c, li, &w, &b, trace && li ? trace + (size_t)(li - 1) * b.n * c.dp : nullptr, s));
+    BB_TRY(project(c, L.in, w.h, c.dp, w.proj, w.ld_proj, b.n, s));
+    if (L.ff > 0) {
+      BB_TRY(project(c, L.up, w.h2, c.dp, at(c, w.proj, L.off_up), w.ld_proj, b.n, s));
+      BB_TRY(bb_hy_polynorm(&c, &L, &w, b.n, s));
+    }
+    BB_TRY(mixer(c, L, w, b, s));
+    BB_TRY(project_f32(c, L.out, w.cat, w.ld_cat, w.x + (li + 1) * level, c.dp, b.n, 1.f, 1, s));
+  }
+  if (trace) {
+    BbHyBatch all = b;      // the last layer's sum for every row
+    all.want = nullptr;
+    all.n_want = b.n < w.want_rows ? b.n : w.want_rows;
+    BB_TRY(bb_hy_mix_norm(&c, c.n_layers, &w, &all, trace + (size_t)(c.n_layers - 1) * b.n * c.dp, s));
+  }
+  return bb_hy_mix_norm(&c, c.n_layers, &w, &b, nullptr, s);
+}
+
 }  // namespace
 
 // One step.  Logits land in w->logits [n_want, vocabp]; `trace` (may be null): fp32 [n_layers][n][dp]
 // copies of the residual stream after every layer.
 BB_API int bb_hybrid_forward(const BbHyCfg* c, const BbHyWork* w, const BbHyBatch* b, float* trace, void* stream) {
   if (!c || !w || !b || b->n <= 0 || b->n > w->rows || b->n_want > w->want_rows) return BB_EARG;
+  if (c->depth_avg) {
+    BB_TRY(forward_depth(*c, *w, *b, trace, stream));
+    if (b->n_want <= 0) return BB_OK;
+    const BbHyLin head{c->head, c->vocabp, c->dp};
+    return project_f32(*c, head, w->hn, c->dp, w->logits, c->vocabp, b->n_want, 1.f, 0, stream);
+  }
   BB_TRY(bb_hy_embed_norm(c, b->tok, w->x, b->n, stream));
   for (int li = 0; li < c->n_layers; ++li) {
     const BbHyLayer& L = c->layers[li];
     BB_TRY(bb_hy_norm(c->dtype, w->x, nullptr, L.norm, w->h, b->n, c->width, c->dp, c->eps, stream));
     BB_TRY(project(*c, L.in, w->h, c->dp, w->proj, w->ld_proj, b->n, stream));
-    BB_TRY(L.kind ? mamba2(*c, L, *w, *b, stream) : attention(*c, L, *w, *b, stream));
+    BB_TRY(mixer(*c, L, *w, *b, stream));
     BB_TRY(project_f32(*c, L.out, w->cat, w->ld_cat, w->x, c->dp, b->n, c->residual_mult, 1, stream));
     if (trace) {
       const size_t n = (size_t)b->n * c->dp;
