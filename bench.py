@@ -36,11 +36,11 @@ def parse():
     ap.add_argument("--micro-batch", type=int, default=4)
     ap.add_argument("--layers", type=int, default=0, help="debug only: override depth (invalidates the number)")
     ap.add_argument("--no-e2e", action="store_true")
-    ap.add_argument("--workload", default="train", choices=["train", "hybrid"],
+    ap.add_argument("--workload", default="train", choices=["train", "hybrid", "nezalorn"],
                     help="train: the headline benchmark; hybrid: prefill and decode of the hybrid decoder beside "
-                         "the dense one (one GPU)")
+                         "the dense one; nezalorn: of that design beside the hybrid decoder (one GPU)")
     ap.add_argument("--hybrid-size", default="m", choices=["s", "m", "l"])
-    ap.add_argument("--no-kernels", action="store_true", help="hybrid workload: throughput only")
+    ap.add_argument("--no-kernels", action="store_true", help="hybrid / nezalorn workload: throughput only")
     return ap.parse_args()
 
 
@@ -92,24 +92,28 @@ class ClockSampler:
 
 
 def hybrid_workload(args):
-    """Serving throughput of the hybrid decoder (value: decode tokens/s) with the dense decoder's beside it
-    and, unless --no-kernels, the per-kernel table of both on standard error."""
+    """Serving throughput of a hybrid decoder (value: decode tokens/s) with that of the decoder it is compared
+    with beside it and, unless --no-kernels, the per-kernel table of both on standard error."""
     import torch
-    from brain_b200.perf import hybrid_bench
     torch.cuda.set_device(0)
     sampler = ClockSampler(0)
     sampler.start()
-    r = hybrid_bench.run(args.hybrid_size, steps=max(args.steps, 3), kernels=not args.no_kernels)
+    if args.workload == "nezalorn":
+        from brain_b200.perf import nezalorn_bench
+        r = nezalorn_bench.run(args.hybrid_size, steps=max(args.steps, 3), with_kernels=not args.no_kernels)
+    else:
+        from brain_b200.perf import hybrid_bench
+        r = hybrid_bench.run(args.hybrid_size, steps=max(args.steps, 3), kernels=not args.no_kernels)
     clocks = sampler.stop()
     for who, rows in r["kernels"].items():
         for k in rows:
             print(f"{who:7s} {k['phase']:8s} {k['kernel']:44s} {k['us']:9.1f} us  {k['of_measured']:.3f} of measured {k['bound']}",
                   file=sys.stderr)
     print(json.dumps({
-        "metric": "decode tok/s (hybrid decoder, batch 64, context 2048)", "value": r["decode_tokens_per_s"]["hybrid"],
+        "metric": f"decode tok/s ({args.workload} decoder, batch 64, context 2048)", "value": r["decode_tokens_per_s"][args.workload],
         "unit": "tokens/s", "n_gpus": 1, "steps": max(args.steps, 3), "warmup": 3, "higher_is_better": True,
-        "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "workload": "hybrid", "clocks": clocks,
-        "config": {"model": f"hybrid-{r['size']}", "shape": r["shape"],
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "workload": args.workload, "clocks": clocks,
+        "config": {"model": f"{args.workload}-{r['size']}", "shape": r["shape"],
                    "l2": "kernels: a buffer larger than L2 is written before each launch; throughput: weights + pages exceed L2"},
         "gpu_launches": r["gpu_launches"], "prefill_tokens_per_s": r["prefill_tokens_per_s"],
         "decode_tokens_per_s": r["decode_tokens_per_s"], "kernels": r["kernels"]}))
@@ -125,7 +129,7 @@ def main():
                           "(unavailable on this box)"}))
         return 0
 
-    if args.workload == "hybrid":
+    if args.workload != "train":
         return hybrid_workload(args)
 
     import torch

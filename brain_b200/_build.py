@@ -169,7 +169,7 @@ def build_bounds(force: bool = False, verbose: bool = False) -> Path:
 #: what serving a hybrid decoder needs of the kernel library, for programs that compile on first use
 HYBRID_TUS = ["common/host.cu", "kernels/attn_rows.cu", "kernels/delta.cu", "kernels/depth_rows.cu", "kernels/flash_fwd.cu",
               "kernels/gemm_2cta.cu", "kernels/gemm_groups.cu", "kernels/gemm_tcgen05.cu", "kernels/hybrid_rows.cu",
-              "kernels/latent_rows.cu", "kernels/mamba2.cu", "kernels/paged_kv.cu", "kernels/rglru.cu",
+              "kernels/latent_decode.cu", "kernels/latent_rows.cu", "kernels/mamba2.cu", "kernels/paged_kv.cu", "kernels/rglru.cu",
               "kernels/router_quant_sample.cu", "kernels/sgemm.cu", "kernels/ssd_tcgen05.cu", "serve/hybrid_forward.cu"]
 HYBRID_LIB = LIBDIR / "libbrain_b200_hybrid.so"
 #: ... and of the host runtime (checkpoint reader, pages, slots, scheduler)

@@ -29,6 +29,8 @@ _ARCHS: List[Arch] = [
          ("train", "infer", "eval"), aliases=("qwen3moe", "moe")),
     Arch("pakalix", "hybrid", "Hybrid decoder: Mamba-2 and soft-capped attention layers, parallel feed-forward",
          ("import", "infer", "serve", "trace"), aliases=("hybrid",)),
+    Arch("nezalorn", "hybrid", "Hybrid decoder: windowed latent attention, generalised delta rule and gated linear "
+         "recurrence layers, depth averages", ("import", "infer", "serve", "trace")),
     Arch("splat", "splat", "3D Gaussian splat rasteriser (headless)", ("render", "train"), built=True),
 ]
 

@@ -1,4 +1,4 @@
-"""``brain pakalix <import|infer|serve|trace>``: hybrid decoders (attention and state-space layers) on the
+"""``brain pakalix|nezalorn <import|infer|serve|trace>``: hybrid decoders (attention and recurrent layers) on the
 serving engine.  ``--model`` takes a directory with ``config.json`` and ``model.safetensors`` or a brain
 checkpoint; prompts are text with ``--tokenizer`` or token ids with ``--tokens 1,2,3``."""
 from __future__ import annotations
@@ -10,20 +10,20 @@ from typing import List
 
 from .args import Args, canon_verb
 
-_USAGE = "usage: brain pakalix <import|infer|serve|trace> ..."
+_USAGE = "usage: brain %s <import|infer|serve|trace> ..."
 
 
-def run_hybrid(argv: List[str], device: str = "auto") -> int:
+def run_hybrid(argv: List[str], device: str = "auto", arch: str = "pakalix") -> int:
     verb = canon_verb(argv[0]) if argv else None
     table = {"import": _import, "infer": _generate, "serve": _generate, "trace": _trace}
     fn = table.get(verb)
     if fn is None:
-        print(f"{_USAGE}  (got {verb!r})", file=sys.stderr)
+        print(f"{_USAGE % arch}  (got {verb!r})", file=sys.stderr)
         return 2
-    return fn(argv[1:], device) or 0
+    return fn(argv[1:], device, arch) or 0
 
 
-def _import(args, device):
+def _import(args, device, arch):
     """Directory -> one brain checkpoint (configuration in its metadata), optionally into the model store."""
     from ..checkpoint import st
     from ..models.config import HybridConfig
@@ -35,7 +35,7 @@ def _import(args, device):
     mdir = a.take_str("--models-dir")
     a.finish()
     if not src:
-        print("usage: brain pakalix import <DIR> [--out F | --id VENDOR/REPO [--models-dir D]] [--dtype F32|BF16]",
+        print(f"usage: brain {arch} import <DIR> [--out F | --id VENDOR/REPO [--models-dir D]] [--dtype F32|BF16]",
               file=sys.stderr)
         return 2
     try:
@@ -70,12 +70,12 @@ def _import(args, device):
             os.remove(tmp)
         print(f"ok: installed {ref} -> {lm.weights}")
         return 0
-    out = out or "pakalix.safetensors"
+    out = out or f"{arch}.safetensors"
     st.save_model(out, model, dtype=dtype)
     print(f"ok: wrote {out} ({model.cfg.n_layers} layers, width {model.cfg.width}, vocab {model.cfg.vocab})")
 
 
-def _generate(args, device):
+def _generate(args, device, arch):
     from ..checkpoint import st
     from ..models.config import HybridConfig
     from ..serve.offline import serve_prompts
@@ -94,13 +94,13 @@ def _generate(args, device):
     dtype = a.str_or("--dtype", "bf16")
     a.finish()
     if not src or not (prompts and tokenizer or ids):
-        print("usage: brain pakalix infer|serve --model DIR|F (--tokenizer T --prompt \"...\" | --tokens 1,2,3)... "
+        print(f"usage: brain {arch} infer|serve --model DIR|F (--tokenizer T --prompt \"...\" | --tokens 1,2,3)... "
               "[--max-new N --max-batch B --block-size 16 --temp X --top-k K --top-p P --seed S --dtype bf16|fp32]",
               file=sys.stderr)
         return 2
     dev = pick_device(device)
     if dev.type != "cuda":
-        print("brain pakalix: the hybrid engine needs a CUDA device", file=sys.stderr)
+        print(f"brain {arch}: the hybrid engine needs a CUDA device", file=sys.stderr)
         return 1
     tok, eos = None, None
     batch = [[int(t) for t in s.split(",") if t.strip()] for s in ids]
@@ -123,6 +123,6 @@ def _generate(args, device):
           f"{time.time() - t0:.2f}s with set-up) [{dtype}]", file=sys.stderr)
 
 
-def _trace(args, device):
+def _trace(args, device, arch):
     from ..serve.trace_run import main
     return main(args)

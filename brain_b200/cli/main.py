@@ -37,7 +37,8 @@ model commands
   toymoe   train [--steps N --batch-size B --block-size T --lr X --out F]
            infer --weights F [--prompt 1,2,3,4 --max-new N --temperature X --top-k K]
            eval  --weights F [--samples N]
-  pakalix  import DIR [--out F | --id VENDOR/REPO]
+  pakalix, nezalorn
+           import DIR [--out F | --id VENDOR/REPO]
            infer|serve --model DIR|F (--tokenizer T --prompt "..." | --tokens 1,2,3)... [--max-new N
                  --max-batch B --temp X --top-k K --top-p P --seed S --dtype bf16|fp32]
            trace --model DIR --out DIR --max-tokens N [--dtype bfloat16|float32]     (same as bin/trace_run)
@@ -140,9 +141,9 @@ def _dispatch_arch(arch_id: str, rest: List[str], device: str) -> int:
     if a.id == "toymoe":
         from .toymoe_cli import run_toymoe
         return run_toymoe(rest, device)
-    if a.id == "pakalix":
+    if a.family == "hybrid":
         from .hybrid_cli import run_hybrid
-        return run_hybrid(rest, device)
+        return run_hybrid(rest, device, a.id)
     if a.id == "splat":
         try:
             from .splat_cli import run_splat

@@ -1,7 +1,6 @@
 // Latent attention, everything but its matrix products, for bf16 and fp32 storage:
 //   hy_latent_in     after the input projection: RMS norm of the query latent in place; the key/value latent
-//                    (normed) and the shared rotated key part into the token's page row; in blocks of their own
-//                    nothing else
+//                    (normed) and the shared rotated key part into the token's page row
 //   hy_latent_q      rotation of every head's rotated query part, in place for rows whose keys are multiplied
 //                    out, beside the absorbed query for the others
 //   hy_latent_gather page rows of prompt portions and the keys before them into one contiguous matrix
@@ -158,8 +157,9 @@ hy_latent_attn_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__
 }
 
 template <typename T>
-static int launch_attn(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, int bs, int r0, cudaStream_t s) {
-  const int rows = b.n - r0, width = L.kvrp + L.rotp;
+static int launch_attn(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, int bs, int r0, int r1,
+                       cudaStream_t s) {
+  const int rows = r1 - r0, width = L.kvrp + L.rotp;
   const int grid = (int)(((long)rows * L.hq * 32 + LAT_THREADS - 1) / LAT_THREADS);
 #define BB_LAUNCH_LA(V)                                                                                            \
   hy_latent_attn_kernel<T, V><<<grid, LAT_THREADS, 0, s>>>(L, static_cast<const T*>(w.qa), w.ld_qa,                \
@@ -216,9 +216,10 @@ BB_API int bb_hy_latent_gather(const BbHyCfg* c, const BbHyLayer* L, const BbHyW
   return (int)cudaGetLastError();
 }
 
-// Absorbed attention of batch rows r0 .. n - 1 (rows 0 .. of w->qa and w->ol).
-BB_API int bb_hy_latent_attn(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int r0, void* stream) {
-  if (r0 >= b->n) return BB_OK;
-  return c->dtype ? launch_attn<float>(*L, *w, *b, c->block_size, r0, (cudaStream_t)stream)
-                  : launch_attn<__nv_bfloat16>(*L, *w, *b, c->block_size, r0, (cudaStream_t)stream);
+// Absorbed attention of batch rows r0 .. r1 - 1 (rows 0 .. of w->qa and w->ol).
+BB_API int bb_hy_latent_attn(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int r0, int r1,
+                             void* stream) {
+  if (r0 >= r1) return BB_OK;
+  return c->dtype ? launch_attn<float>(*L, *w, *b, c->block_size, r0, r1, (cudaStream_t)stream)
+                  : launch_attn<__nv_bfloat16>(*L, *w, *b, c->block_size, r0, r1, (cudaStream_t)stream);
 }

@@ -1,6 +1,8 @@
 // Gated linear recurrence per channel (fp32 state; bf16 or fp32 projections, convolution and gates' maps):
 //   r = sigmoid(gate + bias), i = sigmoid(gate + bias), log a = -lam r,
 //   S <- a S + sqrt(1 - a^2) i u,   output S gelu(y + bias).
+// a is carried as e = a - 1: where a is close to one its rounding to 32 bits would change the rate of a slow
+// decay by 2^-25 / (1 - a), which long sequences show.  1 - a^2 = -e (2 + e).
 //   hy_rglru_scan    prompt portions: a block owns 64 channels of a sequence and takes 128 tokens at a time,
 //                    eight to a warp; the warps' (product of a, local S) pairs are chained through shared memory
 //   hy_rglru_step    one token per sequence, one thread per two channels
@@ -12,10 +14,6 @@
 
 namespace bb {
 
-template <typename T>
-struct Pair {
-  T v[2];
-};
 template <typename T>
 __device__ __forceinline__ float2 load_pair(const T* p) {
   struct alignas(sizeof(T) * 2) P {
@@ -42,17 +40,22 @@ __device__ __forceinline__ float gelu_as(float z) {
   if constexpr (sizeof(T) == 2) return z * __fdividef(1.f, 1.f + __expf(-2.f * t));
   else return 0.5f * z * (1.f + tanhf(t));
 }
-// log a = -x (x >= 0) -> a and sqrt(1 - a^2)
+// e^-x - 1 for x >= 0
 template <typename T>
-__device__ __forceinline__ float2 decay_of(float x) {
+__device__ __forceinline__ float decay_m1(float x) {
   if constexpr (sizeof(T) == 2) {
-    const float a = __expf(-x), y = 2.f * x;
-    // 1 - e^-y: its series where the difference would cancel
-    const float d = y < 0.05f ? y * fmaf(y, fmaf(y, fmaf(y, -1.f / 24.f, 1.f / 6.f), -0.5f), 1.f) : 1.f - a * a;
-    return make_float2(a, sqrtf(d));
+    // the series where the difference would cancel
+    return x < 0.05f ? -x * fmaf(x, fmaf(x, fmaf(x, -1.f / 24.f, 1.f / 6.f), -0.5f), 1.f) : __expf(-x) - 1.f;
   } else {
-    return make_float2(expf(-x), sqrtf(-expm1f(-2.f * x)));
+    return expm1f(-x);
   }
+}
+// S after a token of (e, in); product of two decays
+__device__ __forceinline__ float2 lru_apply(float2 e, float2 s, float2 in) {
+  return make_float2(s.x + fmaf(e.x, s.x, in.x), s.y + fmaf(e.y, s.y, in.y));
+}
+__device__ __forceinline__ float2 lru_product(float2 p, float2 e) {
+  return make_float2(p.x + fmaf(e.x, p.x, e.x), p.y + fmaf(e.y, p.y, e.y));
 }
 
 struct LruChannels {
@@ -62,12 +65,12 @@ __device__ __forceinline__ LruChannels lru_channels(const BbHyLayer& L, int c) {
   auto two = [&](const float* p) { return *reinterpret_cast<const float2*>(p + c); };
   return {two(L.y_b), two(L.r_b), two(L.i_b), two(L.lam)};
 }
-// Raw values of a token and two channels -> decay and input of the recurrence.
+// Raw values of a token and two channels -> decay (less one) and input of the recurrence.
 template <typename T>
-__device__ __forceinline__ void lru_token(const LruChannels& p, float2 r, float2 i, float2 u, float2& a, float2& in) {
-  const float2 d0 = decay_of<T>(p.lam.x * sigmoid_as<T>(r.x + p.rb.x)), d1 = decay_of<T>(p.lam.y * sigmoid_as<T>(r.y + p.rb.y));
-  a = make_float2(d0.x, d1.x);
-  in = make_float2(d0.y * sigmoid_as<T>(i.x + p.ib.x) * u.x, d1.y * sigmoid_as<T>(i.y + p.ib.y) * u.y);
+__device__ __forceinline__ void lru_token(const LruChannels& p, float2 r, float2 i, float2 u, float2& e, float2& in) {
+  e = make_float2(decay_m1<T>(p.lam.x * sigmoid_as<T>(r.x + p.rb.x)), decay_m1<T>(p.lam.y * sigmoid_as<T>(r.y + p.rb.y)));
+  in = make_float2(sqrtf(-e.x * (2.f + e.x)) * sigmoid_as<T>(i.x + p.ib.x) * u.x,
+                   sqrtf(-e.y * (2.f + e.y)) * sigmoid_as<T>(i.y + p.ib.y) * u.y);
 }
 
 template <typename T>
@@ -108,17 +111,14 @@ hy_rglru_scan_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
         ii[k] = load_pair(gates + row * ldg + g0 + L.bwp);
         uu[k] = load_pair(u + row * ldu + cc);
       }
-      float2 pa = make_float2(1.f, 1.f), sa = make_float2(0.f, 0.f);
+      float2 pa = make_float2(0.f, 0.f), sa = make_float2(0.f, 0.f);
 #pragma unroll
       for (int k = 0; k < LRU_T; ++k) {
-        float2 a, in;
-        lru_token<T>(ch, rr[k], ii[k], uu[k], a, in);
-        if (tw + k >= n) {           // past the end: nothing changes
-          a = make_float2(1.f, 1.f);
-          in = make_float2(0.f, 0.f);
-        }
-        sa = make_float2(fmaf(a.x, sa.x, in.x), fmaf(a.y, sa.y, in.y));
-        pa = make_float2(pa.x * a.x, pa.y * a.y);
+        float2 e, in;
+        lru_token<T>(ch, rr[k], ii[k], uu[k], e, in);
+        if (tw + k >= n) e = in = make_float2(0.f, 0.f);      // past the end: nothing changes
+        sa = lru_apply(e, sa, in);
+        pa = lru_product(pa, e);
         p[k] = pa;
         s[k] = sa;
       }
@@ -130,16 +130,15 @@ hy_rglru_scan_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
 #pragma unroll
     for (int w = 0; w < LRU_WARPS; ++w) {
       if (w == warp) mine = carry;
-      const float2 cp = chain[it & 1][w][0][lane], cs = chain[it & 1][w][1][lane];
-      carry = make_float2(fmaf(cp.x, carry.x, cs.x), fmaf(cp.y, carry.y, cs.y));
+      carry = lru_apply(chain[it & 1][w][0][lane], carry, chain[it & 1][w][1][lane]);
     }
 #pragma unroll
     for (int k = 0; k < LRU_T; ++k) {
       if (tw + k < n && live) {
         const size_t row = r0 + tw + k;
         const float2 yv = load_pair(proj + row * ld + L.off_y + cc);
-        const float sx = fmaf(p[k].x, mine.x, s[k].x), sy = fmaf(p[k].y, mine.y, s[k].y);
-        store_pair(cat + row * ldc + cc, sx * gelu_as<T>(yv.x + ch.yb.x), sy * gelu_as<T>(yv.y + ch.yb.y));
+        const float2 st = lru_apply(p[k], mine, s[k]);
+        store_pair(cat + row * ldc + cc, st.x * gelu_as<T>(yv.x + ch.yb.x), st.y * gelu_as<T>(yv.y + ch.yb.y));
         keep_input<T>(L, proj + row * ld, cc, pos0 + tw + k, ctx, slot);
       }
     }
@@ -161,10 +160,10 @@ hy_rglru_step_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
   const float2 old = *reinterpret_cast<const float2*>(state);
   const float2 yv = load_pair(proj + row * ld + L.off_y + c);
   const LruChannels ch = lru_channels(L, c);
-  float2 a, in;
-  lru_token<T>(ch, load_pair(gates + row * ldg + g0), load_pair(gates + row * ldg + g0 + L.bwp), load_pair(u + row * ldu + c), a, in);
+  float2 e, in;
+  lru_token<T>(ch, load_pair(gates + row * ldg + g0), load_pair(gates + row * ldg + g0 + L.bwp), load_pair(u + row * ldu + c), e, in);
   const bool fresh = pos == 0;
-  const float2 s = make_float2(fresh ? in.x : fmaf(a.x, old.x, in.x), fresh ? in.y : fmaf(a.y, old.y, in.y));
+  const float2 s = fresh ? in : lru_apply(e, old, in);
   *reinterpret_cast<float2*>(state) = s;
   store_pair(cat + row * ldc + c, s.x * gelu_as<T>(yv.x + ch.yb.x), s.y * gelu_as<T>(yv.y + ch.yb.y));
   keep_input<T>(L, proj + row * ld, c, pos, pos + 1, slot);

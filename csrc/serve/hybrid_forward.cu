@@ -37,10 +37,11 @@ int bb_hy_polynorm(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int 
 int bb_hy_latent_in(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
 int bb_hy_latent_q(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int n_in, void* stream);
 int bb_hy_latent_gather(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
-int bb_hy_latent_attn(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int r0, void* stream);
+int bb_hy_latent_attn(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int r0, int r1,
+                      void* stream);
+int bb_hy_latent_decode(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int qa_row0, void* stream);
 int bb_hy_delta_tanh(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
-int bb_hy_delta_scan(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
-int bb_hy_delta_post(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_delta(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
 int bb_hy_rglru(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
 int bb_gemm_bf16_groups(const void* A, const void* B, void* C, int M, int N, int K, int groups, int lda, int a_step, int ldc,
                         int c_step, void* stream);
@@ -171,7 +172,10 @@ int latent_attention(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, co
   const int rows = b.n - n_in;
   BB_TRY(project_groups(c, L.w_abs, L.hq, L.kvrp, L.dkp, at(c, w.q, (size_t)n_in * w.ld_q), w.ld_q, dq, w.qa, w.ld_qa, width,
                         rows, s));
-  BB_TRY(bb_hy_latent_attn(&c, &L, &w, &b, n_in, s));
+  const int rc = bb_hy_latent_decode(&c, &L, &w, &b, b.n_pre - n_in, s);
+  if (rc == BB_OK && n_in < b.n_pre) BB_TRY(bb_hy_latent_attn(&c, &L, &w, &b, n_in, b.n_pre, s));
+  else if (rc == BB_ESIZE) BB_TRY(bb_hy_latent_attn(&c, &L, &w, &b, n_in, b.n, s));
+  else if (rc) return rc;
   return project_groups(c, L.w_uv, L.hq, L.dvp, L.kvrp, w.ol, w.ld_ol, L.kvrp, at(c, w.cat, (size_t)n_in * w.ld_cat), w.ld_cat,
                         L.dvp, rows, s);
 }
@@ -179,8 +183,7 @@ int latent_attention(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, co
 int general_delta(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
   BB_TRY(bb_hy_delta_tanh(&c, &L, &w, &b, s));
   BB_TRY(project(c, L.w2, at(c, w.proj, L.off_w1), w.ld_proj, w.aux, w.ld_aux, b.n, s));
-  BB_TRY(bb_hy_delta_scan(&c, &L, &w, &b, s));
-  return bb_hy_delta_post(&c, &L, &w, &b, s);
+  return bb_hy_delta(&c, &L, &w, &b, s);
 }
 
 int rglru(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
