@@ -40,14 +40,15 @@ def dense_config(s):
 
 
 class KernelTimer:
-    """Device microseconds of a launch behind a buffer write larger than L2."""
+    """Device microseconds of a launch behind a buffer write larger than L2: replays of (write + kernel) and of the
+    write alone take turns, so both see the same clocks, and the difference counts."""
 
-    def __init__(self, reps: int = 8, rounds: int = 5):
+    def __init__(self, reps: int = 8, rounds: int = 7):
         self.buf = torch.empty(192 << 20, device="cuda", dtype=torch.uint8)
         self.reps, self.rounds = reps, rounds
-        self.base = self._time(lambda: None)
+        self.base = self._graph(lambda: None)
 
-    def _time(self, fn) -> float:
+    def _graph(self, fn):
         fn()
         torch.cuda.synchronize()
         g = torch.cuda.CUDAGraph()
@@ -55,20 +56,23 @@ class KernelTimer:
             for _ in range(self.reps):
                 self.buf.zero_()
                 fn()
-        ms = []
-        for i in range(self.rounds + 2):
-            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            torch.cuda.synchronize()
-            a.record()
-            g.replay()
-            b.record()
-            torch.cuda.synchronize()
-            if i >= 2:
-                ms.append(a.elapsed_time(b))
-        return statistics.median(ms) / self.reps * 1e3
+        return g
 
     def __call__(self, fn) -> float:
-        return max(self._time(fn) - self.base, 0.1)
+        g = self._graph(fn)
+        us = []
+        for i in range(self.rounds + 2):
+            ev = [torch.cuda.Event(enable_timing=True) for _ in range(3)]
+            torch.cuda.synchronize()
+            ev[0].record()
+            self.base.replay()
+            ev[1].record()
+            g.replay()
+            ev[2].record()
+            torch.cuda.synchronize()
+            if i >= 2:
+                us.append((ev[1].elapsed_time(ev[2]) - ev[0].elapsed_time(ev[1])) / self.reps * 1e3)
+        return max(statistics.median(us), 0.1)
 
 
 def _time_calls(fn, n: int) -> float:

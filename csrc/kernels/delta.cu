@@ -5,8 +5,8 @@
 //   o = (w r)^T S_old - (r . a u)(u^T S_old) + (r . k) v
 // so one sweep over S yields both dot products and a second one updates it.
 //   hy_delta_tanh    tanh of the low-rank decay projection, in place, ahead of its second matrix
-//   hy_delta_scan    prompt portions, token by token; the state in registers, its columns spread over warps and
-//                    blocks, while other warps prepare the next tokens' vectors (bf16, heads up to 128)
+//   hy_delta_scan    prompt portions, four tokens at a time; the state in registers, its columns spread over warps
+//                    and blocks, while other warps prepare the next tokens (bf16, heads up to 128)
 //   hy_delta_scan_any  the same with the state in shared memory: fp32, and other head sizes
 //   hy_delta_decode  one token per sequence: the state is read and written once, norm and gate included
 //   hy_delta_post    per head root-mean-square norm, gain, sigmoid gate -> the output projection's input
@@ -137,10 +137,24 @@ hy_delta_scan_any_kernel(const __grid_constant__ BbHyLayer L, const T* __restric
   for (int i = threadIdx.x; i < D * D; i += DS_THREADS) state[i] = S[i];
 }
 
-// ---- state in registers.  A thread holds CT columns of DP / KL keys (the float4 groups q, q + KL, ... of lane
-// q), so a token's vectors are read from shared memory without bank conflicts and two shuffles finish a dot
-// product.  CW warps walk through the tokens; four others prepare the next DT_T tokens meanwhile.
-constexpr int DT_T = 16, DT_PREP = 4;
+// ---- state in registers, four tokens at a time.  With W_i..j the product of the decays of tokens i .. j of a
+// group and S the state before it, the four dot products with the removed directions all run over the same S:
+//   x_i = (W_0..i-1 u_i)^T S - sum_{j<i} (u_i . W_j+1..i-1 a_j u_j) x_j + sum_{j<i} (u_i . W_j+1..i-1 k_j) v_j
+//   o_i = (W_0..i r_i)^T S   - sum_{j<=i} (r_i . W_j+1..i a_j u_j) x_j  + sum_{j<=i} (r_i . W_j+1..i k_j) v_j
+//   S   <- W_0..3 S + sum_j (W_j+1..3 k_j) v_j^T - (W_j+1..3 a_j u_j) x_j^T
+// (no decay is ever divided by).  The bracketed numbers do not depend on S: the warps that prepare a group have
+// them ready, and one round of shuffles serves four tokens.  A thread holds CT columns of DP / KL keys, the
+// float4 groups q, q + KL, ... of lane q, so vectors are read from shared memory without bank conflicts.
+constexpr int DG = 4, DT_GROUPS = 4, DT_PREP = 4;      // tokens of a group, groups of a buffer, preparing warps
+static_assert(DT_GROUPS == DT_PREP, "a preparing warp has one group of each buffer");
+
+template <int DP>
+struct DeltaGroup {
+  // per group: U_i, R_i (4 each), W, K_j, A_j (4 each), v_j (4), then the 4 x 4 numbers of x (removal, value)
+  // and of o
+  static constexpr int U = 0, R = DG * DP, W = 2 * DG * DP, K = W + DP, A = K + DG * DP, V = A + DG * DP, X = V + DG * DP;
+  static constexpr int SIZE = X + 64;
+};
 
 __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
   float2 d;
@@ -163,30 +177,175 @@ __device__ __forceinline__ float2 mul2(float2 a, float2 b) {
   return d;
 }
 
+// A group by one warp, DP / 32 neighbouring channels to a lane.
+template <typename T, int DP>
+struct DeltaPrep {
+  using G = DeltaGroup<DP>;
+  static constexpr int V = DP / 32;
+  struct alignas(sizeof(T) * V) Raw {
+    T v[V];
+  };
+  struct alignas(4 * V) Out {
+    float v[V];
+  };
+  const BbHyLayer& L;
+  const T *proj, *low;
+  int ld, ldl, h;
+  Raw r[DG], k[DG], v[DG], a[DG], x[DG];
+
+  __device__ __forceinline__ void fetch(int r0, int t0, int n) {
+    const int d = (threadIdx.x & 31) * V, o = h * L.pp + d;
+    const bool in = d < L.pp;                        // (pp is a multiple of V)
+#pragma unroll
+    for (int i = 0; i < DG; ++i) {
+      if (in && t0 + i < n) {
+        const T* row = proj + (size_t)(r0 + t0 + i) * ld + o;
+        k[i] = *reinterpret_cast<const Raw*>(row + L.off_kk);
+        r[i] = *reinterpret_cast<const Raw*>(row + L.off_r);
+        v[i] = *reinterpret_cast<const Raw*>(row + L.off_vv);
+        a[i] = *reinterpret_cast<const Raw*>(row + L.off_a);
+        x[i] = *reinterpret_cast<const Raw*>(low + (size_t)(r0 + t0 + i) * ldl + o);
+        if (L.p != L.pp)
+#pragma unroll
+          for (int j = 0; j < V; ++j)
+            if (d + j >= L.p) k[i].v[j] = r[i].v[j] = v[i].v[j] = from_f<T>(0.f);
+      } else {
+#pragma unroll
+        for (int j = 0; j < V; ++j) k[i].v[j] = r[i].v[j] = v[i].v[j] = a[i].v[j] = x[i].v[j] = from_f<T>(0.f);
+      }
+    }
+  }
+  // Tokens past n leave the state as it is: their keys and values are zero and their decay is one.
+  __device__ __forceinline__ void finish(float* p, int t0, int n) {
+    if (t0 >= n) return;
+    const int lane = threadIdx.x & 31, d = lane * V, o = h * L.pp + d;
+    float s[32];
+#pragma unroll
+    for (int i = 0; i < DG; ++i) {
+      s[i] = 0.f;
+#pragma unroll
+      for (int j = 0; j < V; ++j) s[i] = fmaf(to_f(k[i].v[j]), to_f(k[i].v[j]), s[i]);
+    }
+#pragma unroll
+    for (int q = 16; q > 0; q >>= 1)
+#pragma unroll
+      for (int i = 0; i < DG; ++i) s[i] += __shfl_xor_sync(0xffffffffu, s[i], q);
+    float unit[DG];
+#pragma unroll
+    for (int i = 0; i < DG; ++i) unit[i] = rsqrtf(s[i] + kDeltaUnit);
+#pragma unroll
+    for (int i = 0; i < 32; ++i) s[i] = 0.f;
+    Out O[3 * DG + 1 + 2 * DG];                      // U, R, W, K, A in the group's order, then v
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      const float w0 = d < L.pp ? L.w0[o + j] : 0.f, ab = d < L.pp ? L.a_b[o + j] : 0.f;
+      float w[DG], u[DG], rr[DG], kk[DG], au[DG];
+#pragma unroll
+      for (int i = 0; i < DG; ++i) {
+        w[i] = t0 + i < n ? __expf(-kDecayScale * sigmoid_as<T>(to_f(x[i].v[j]) + w0)) : 1.f;
+        kk[i] = to_f(k[i].v[j]);
+        rr[i] = to_f(r[i].v[j]);
+        u[i] = kk[i] * unit[i];
+        au[i] = sigmoid_as<T>(to_f(a[i].v[j]) + ab) * u[i];
+      }
+      // numbers: row i of x at 0 (removal) and 6 (value), of o at 12 and 22
+      int nx = 0, no = 0;
+      float before = 1.f;
+#pragma unroll
+      for (int i = 0; i < DG; ++i) {
+        O[i].v[j] = before * u[i];
+        before *= w[i];
+        O[DG + i].v[j] = before * rr[i];
+      }
+      O[2 * DG].v[j] = before;
+#pragma unroll
+      for (int i = 0; i < DG; ++i) {
+        float au_w[DG], k_w[DG];                     // vectors of earlier tokens as token i finds them
+#pragma unroll
+        for (int q = 0; q < DG; ++q) {
+          if (q >= i) continue;
+          float m = 1.f;
+#pragma unroll
+          for (int e = 0; e < DG; ++e)
+            if (e > q && e < i) m *= w[e];
+          au_w[q] = m * au[q];
+          k_w[q] = m * kk[q];
+          s[nx] = fmaf(u[i], au_w[q], s[nx]);
+          s[6 + nx] = fmaf(u[i], k_w[q], s[6 + nx]);
+          ++nx;
+        }
+#pragma unroll
+        for (int q = 0; q < DG; ++q) {
+          if (q > i) continue;
+          const float rw = q < i ? rr[i] * w[i] : rr[i];
+          s[12 + no] = fmaf(rw, q < i ? au_w[q] : au[q], s[12 + no]);
+          s[22 + no] = fmaf(rw, q < i ? k_w[q] : kk[q], s[22 + no]);
+          ++no;
+        }
+      }
+#pragma unroll
+      for (int q = 0; q < DG; ++q) {
+        float m = 1.f;
+#pragma unroll
+        for (int e = 0; e < DG; ++e)
+          if (e > q) m *= w[e];
+        O[2 * DG + 1 + q].v[j] = m * kk[q];
+        O[3 * DG + 1 + q].v[j] = m * au[q];
+        O[4 * DG + 1 + q].v[j] = to_f(v[q].v[j]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 5 * DG + 1; ++i) *reinterpret_cast<Out*>(p + i * DP + d) = O[i];
+    // 32 sums over the warp, sum i to lane i
+#pragma unroll
+    for (int c = 16; c > 0; c >>= 1) {
+      const bool up = lane & c;
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        if (i >= c) break;
+        const float keep = up ? s[i + c] : s[i], send = up ? s[i] : s[i + c];
+        s[i] = keep + __shfl_xor_sync(0xffffffffu, send, c);
+      }
+    }
+    // ... and into the 4 x 4 tables (their other places stay zero)
+    const int set = lane < 6 ? 0 : (lane < 12 ? 1 : (lane < 22 ? 2 : 3));
+    const int e = lane - (set == 0 ? 0 : (set == 1 ? 6 : (set == 2 ? 12 : 22)));
+    int i, q;
+    if (set < 2) {
+      i = e == 0 ? 1 : (e < 3 ? 2 : 3);
+      q = e - i * (i - 1) / 2;
+    } else {
+      i = e == 0 ? 0 : (e < 3 ? 1 : (e < 6 ? 2 : 3));
+      q = e - i * (i + 1) / 2;
+    }
+    p[G::X + set * 16 + i * 4 + q] = s[0];
+  }
+};
+
 template <typename T, int DP, int CW>
-__global__ void __launch_bounds__((CW + DT_PREP) * 32, 2)
+__global__ void __launch_bounds__((CW + DT_PREP) * 32)
 hy_delta_scan_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, int ld, const T* __restrict__ low,
                      int ldl, T* __restrict__ y, int ldy, const __grid_constant__ BbHyBatch b) {
-  constexpr int KT = 16, KL = DP / KT, CT = 2, PAIRS = KT / 2;
+  using G = DeltaGroup<DP>;
+  constexpr int KL = DP > 64 ? 8 : 4, KT = DP / KL, CT = 2, QUADS = KT / 4, STEP = DG * DT_GROUPS;
   constexpr int COLS = CW * (32 / KL) * CT;          // columns of a block
-  constexpr int STRIDE = 6 * DP + 4;                 // floats of a token: vectors, then the two scalars
-  extern __shared__ __align__(16) float sm[];        // [2][DT_T][STRIDE]
+  extern __shared__ __align__(16) float sm[];        // [2][DT_GROUPS][G::SIZE]
   const int seq = blockIdx.z, h = blockIdx.y, D = L.p;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int r0 = b.seq_row0[seq], n = b.seq_row0[seq + 1] - r0;
-  auto prepare = [&](int t0, int w, int nw) {
-    for (int t = w; t < DT_T && t0 + t < n; t += nw) {
-      float* p = sm + (((t0 / DT_T) & 1) * DT_T + t) * STRIDE;
-      const size_t r = r0 + t0 + t;
-      const float2 d = delta_token<T>(L, proj + r * ld, low + r * ldl, h, DeltaVecs::at(p, DP), DP);
-      if (lane == 0) *reinterpret_cast<float2*>(p + 6 * DP) = d;
-    }
-  };
-  prepare(0, warp, CW + DT_PREP);
+  for (int i = threadIdx.x; i < 2 * DT_GROUPS * 64; i += blockDim.x) sm[(i / 64) * G::SIZE + G::X + i % 64] = 0.f;
   __syncthreads();
   if (warp >= CW) {
-    for (int t0 = 0; t0 < n; t0 += DT_T) {
-      prepare(t0 + DT_T, warp - CW, DT_PREP);
+    DeltaPrep<T, DP> prep{L, proj, low, ld, ldl, h};
+    const int w = warp - CW;
+    prep.fetch(r0, w * DG, n);
+    prep.finish(sm + w * G::SIZE, w * DG, n);
+    prep.fetch(r0, STEP + w * DG, n);
+    __syncthreads();
+    for (int t0 = 0, it = 1; t0 < n; t0 += STEP, ++it) {
+      const int t = t0 + STEP + w * DG;
+      prep.finish(sm + ((it & 1) * DT_GROUPS + w) * G::SIZE, t, n);
+      prep.fetch(r0, t + STEP, n);
       __syncthreads();
     }
     return;
@@ -194,81 +353,122 @@ hy_delta_scan_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
   const int q = lane % KL, c0 = blockIdx.x * COLS + (warp * (32 / KL) + lane / KL) * CT;
   float* state = L.ssm_state + ((size_t)b.seq_slot[seq] * L.heads + h) * D * D;
   const bool fresh = b.seq_pos0[seq] == 0;
-  float2 S[CT][PAIRS];                               // two neighbouring keys of a column
+  float2 S[CT][2 * QUADS];                           // two neighbouring keys of a column
   auto key = [&](int i) { return 4 * (q + KL * (i / 2)) + 2 * (i & 1); };
 #pragma unroll
-  for (int i = 0; i < PAIRS; ++i)
+  for (int i = 0; i < 2 * QUADS; ++i)
 #pragma unroll
     for (int c = 0; c < CT; ++c) {
       const int k = key(i), col = c0 + c;
       S[c][i].x = !fresh && k < D && col < D ? state[(size_t)k * D + col] : 0.f;
       S[c][i].y = !fresh && k + 1 < D && col < D ? state[(size_t)(k + 1) * D + col] : 0.f;
     }
-  T* yc = y + (size_t)r0 * ldy + h * L.pp + c0;
-  const bool writes = q == 0 && c0 < L.pp;           // (pp is even: both columns or none)
-  for (int t0 = 0; t0 < n; t0 += DT_T) {
-    const int nt = min(DT_T, n - t0);
-    const float* p = sm + ((t0 / DT_T) & 1) * DT_T * STRIDE;
-    for (int t = 0; t < nt; ++t, p += STRIDE) {
-      const float4* u4 = reinterpret_cast<const float4*>(p) + q;
-      const float4* wr4 = u4 + DP / 4;
-      float2 pu[CT], pr[CT];
+  const int cv = min(c0, DP - CT), tok = q & (DG - 1);   // lane q finishes the output of token q of a group
+  T* yc = y + (size_t)(r0 + tok) * ldy + h * L.pp + c0;
+  const bool writes = q < DG && c0 < L.pp;           // (pp is even: both columns or none)
+  __syncthreads();
+  for (int t0 = 0, it = 0; t0 < n; t0 += STEP, ++it) {
+    const float* p = sm + (it & 1) * DT_GROUPS * G::SIZE;
+    for (int t = t0; t < min(t0 + STEP, n); t += DG, p += G::SIZE) {
+      float2 pu[DG][CT], pr[DG][CT];
 #pragma unroll
-      for (int c = 0; c < CT; ++c) pu[c] = pr[c] = make_float2(0.f, 0.f);
+      for (int i = 0; i < DG; ++i)
 #pragma unroll
-      for (int i = 0; i < PAIRS; i += 2) {
-        const float4 u = u4[KL * (i / 2)], wr = wr4[KL * (i / 2)];
+        for (int c = 0; c < CT; ++c) pu[i][c] = pr[i][c] = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int m = 0; m < QUADS; ++m)
+#pragma unroll
+        for (int i = 0; i < DG; ++i) {
+          const float4 u = reinterpret_cast<const float4*>(p + G::U + i * DP)[q + KL * m];
+          const float4 r = reinterpret_cast<const float4*>(p + G::R + i * DP)[q + KL * m];
+#pragma unroll
+          for (int c = 0; c < CT; ++c) {
+            pu[i][c] = fma2(make_float2(u.x, u.y), S[c][2 * m], pu[i][c]);
+            pr[i][c] = fma2(make_float2(r.x, r.y), S[c][2 * m], pr[i][c]);
+            pu[i][c] = fma2(make_float2(u.z, u.w), S[c][2 * m + 1], pu[i][c]);
+            pr[i][c] = fma2(make_float2(r.z, r.w), S[c][2 * m + 1], pr[i][c]);
+          }
+        }
+      float x[DG][CT], os[DG][CT];
+#pragma unroll
+      for (int i = 0; i < DG; ++i)
 #pragma unroll
         for (int c = 0; c < CT; ++c) {
-          pu[c] = fma2(make_float2(u.x, u.y), S[c][i], pu[c]);
-          pr[c] = fma2(make_float2(wr.x, wr.y), S[c][i], pr[c]);
-          pu[c] = fma2(make_float2(u.z, u.w), S[c][i + 1], pu[c]);
-          pr[c] = fma2(make_float2(wr.z, wr.w), S[c][i + 1], pr[c]);
+          x[i][c] = pu[i][c].x + pu[i][c].y;
+          os[i][c] = pr[i][c].x + pr[i][c].y;
         }
-      }
-      const float2 v = *reinterpret_cast<const float2*>(p + 5 * DP + min(c0, DP - CT));
-      const float2 dots = *reinterpret_cast<const float2*>(p + 6 * DP);
-      float us[CT], os[CT];
-#pragma unroll
-      for (int c = 0; c < CT; ++c) {
-        us[c] = pu[c].x + pu[c].y;
-        os[c] = pr[c].x + pr[c].y;
-      }
 #pragma unroll
       for (int o = 1; o < KL; o <<= 1)
 #pragma unroll
-        for (int c = 0; c < CT; ++c) {
-          us[c] += __shfl_xor_sync(0xffffffffu, us[c], o);
-          os[c] += __shfl_xor_sync(0xffffffffu, os[c], o);
-        }
-      const float4* w4 = u4 + 2 * (DP / 4);
-      const float4* k4 = u4 + 3 * (DP / 4);
-      const float4* au4 = u4 + 4 * (DP / 4);
-      const float vc[CT] = {v.x, v.y};
+        for (int i = 0; i < DG; ++i)
 #pragma unroll
-      for (int i = 0; i < PAIRS; i += 2) {
-        const float4 w = w4[KL * (i / 2)], k = k4[KL * (i / 2)], au = au4[KL * (i / 2)];
+          for (int c = 0; c < CT; ++c) x[i][c] += __shfl_xor_sync(0xffffffffu, x[i][c], o);
+      float2 v[DG];
 #pragma unroll
-        for (int c = 0; c < CT; ++c) {
-          const float2 vv = make_float2(vc[c], vc[c]), uu = make_float2(-us[c], -us[c]);
-          S[c][i] = fma2(make_float2(w.x, w.y), S[c][i], fma2(make_float2(au.x, au.y), uu, mul2(make_float2(k.x, k.y), vv)));
-          S[c][i + 1] =
-              fma2(make_float2(w.z, w.w), S[c][i + 1], fma2(make_float2(au.z, au.w), uu, mul2(make_float2(k.z, k.w), vv)));
+      for (int i = 0; i < DG; ++i) v[i] = *reinterpret_cast<const float2*>(p + G::V + i * DP + cv);
+#pragma unroll
+      for (int i = 1; i < DG; ++i) {
+        const float4 ra = *reinterpret_cast<const float4*>(p + G::X + i * 4), rv = *reinterpret_cast<const float4*>(p + G::X + 16 + i * 4);
+        const float ca[4] = {ra.x, ra.y, ra.z, ra.w}, cw[4] = {rv.x, rv.y, rv.z, rv.w};
+#pragma unroll
+        for (int j = 0; j < i; ++j) {
+          x[i][0] = fmaf(cw[j], v[j].x, fmaf(-ca[j], x[j][0], x[i][0]));
+          x[i][1] = fmaf(cw[j], v[j].y, fmaf(-ca[j], x[j][1], x[i][1]));
         }
       }
-      if (writes) {
+      // the state first: the next group waits for it
+#pragma unroll
+      for (int m = 0; m < QUADS; ++m) {
+        const float4 w = reinterpret_cast<const float4*>(p + G::W)[q + KL * m];
+#pragma unroll
+        for (int c = 0; c < CT; ++c) {
+          S[c][2 * m] = mul2(make_float2(w.x, w.y), S[c][2 * m]);
+          S[c][2 * m + 1] = mul2(make_float2(w.z, w.w), S[c][2 * m + 1]);
+        }
+#pragma unroll
+        for (int j = 0; j < DG; ++j) {
+          const float4 k = reinterpret_cast<const float4*>(p + G::K + j * DP)[q + KL * m];
+          const float4 a = reinterpret_cast<const float4*>(p + G::A + j * DP)[q + KL * m];
+#pragma unroll
+          for (int c = 0; c < CT; ++c) {
+            const float vc = c ? v[j].y : v[j].x, xc = -x[j][c];
+            S[c][2 * m] = fma2(make_float2(k.x, k.y), make_float2(vc, vc), S[c][2 * m]);
+            S[c][2 * m + 1] = fma2(make_float2(k.z, k.w), make_float2(vc, vc), S[c][2 * m + 1]);
+            S[c][2 * m] = fma2(make_float2(a.x, a.y), make_float2(xc, xc), S[c][2 * m]);
+            S[c][2 * m + 1] = fma2(make_float2(a.z, a.w), make_float2(xc, xc), S[c][2 * m + 1]);
+          }
+        }
+      }
+      // outputs: sums of the four tokens, one token to a lane
+      const bool b1 = q & 2, b0 = q & 1;
+#pragma unroll
+      for (int c = 0; c < CT; ++c) {
+        const float k0 = b1 ? os[2][c] : os[0][c], k1 = b1 ? os[3][c] : os[1][c];
+        const float s0 = b1 ? os[0][c] : os[2][c], s1 = b1 ? os[1][c] : os[3][c];
+        const float e0 = k0 + __shfl_xor_sync(0xffffffffu, s0, 2), e1 = k1 + __shfl_xor_sync(0xffffffffu, s1, 2);
+        os[0][c] = (b0 ? e1 : e0) + __shfl_xor_sync(0xffffffffu, b0 ? e0 : e1, 1);
+        if (KL == 8) os[0][c] += __shfl_xor_sync(0xffffffffu, os[0][c], 4);
+      }
+      const float4 ga = *reinterpret_cast<const float4*>(p + G::X + 32 + tok * 4), gv = *reinterpret_cast<const float4*>(p + G::X + 48 + tok * 4);
+      const float ca[4] = {ga.x, ga.y, ga.z, ga.w}, cw[4] = {gv.x, gv.y, gv.z, gv.w};
+#pragma unroll
+      for (int j = 0; j < DG; ++j) {
+        os[0][0] = fmaf(cw[j], v[j].x, fmaf(-ca[j], x[j][0], os[0][0]));
+        os[0][1] = fmaf(cw[j], v[j].y, fmaf(-ca[j], x[j][1], os[0][1]));
+      }
+      if (writes && t + tok < n) {
         struct alignas(sizeof(T) * 2) Two {
           T v[2];
         } o;
-#pragma unroll
-        for (int c = 0; c < CT; ++c) o.v[c] = from_f<T>(fmaf(dots.y, vc[c], fmaf(-dots.x, us[c], os[c])));
-        *reinterpret_cast<Two*>(yc + (size_t)(t0 + t) * ldy) = o;
+        o.v[0] = from_f<T>(os[0][0]);
+        o.v[1] = from_f<T>(os[0][1]);
+        *reinterpret_cast<Two*>(yc + (size_t)t * ldy) = o;
       }
     }
     __syncthreads();
   }
 #pragma unroll
-  for (int i = 0; i < PAIRS; ++i)
+  for (int i = 0; i < 2 * QUADS; ++i)
 #pragma unroll
     for (int c = 0; c < CT; ++c) {
       const int k = key(i), col = c0 + c;
@@ -364,24 +564,42 @@ hy_delta_decode_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict_
   }
 }
 
+// One block per row; a head's vectors of 8 lie in `lanes` neighbouring threads (a power of two up to 32).
+constexpr int DPOST_THREADS = 256;
+
 template <typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(DPOST_THREADS)
 hy_delta_post_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, int ld, const T* __restrict__ y, int ldy,
-                     T* __restrict__ cat, int ldc, int rows, float eps) {
-  const long w = ((long)blockIdx.x * 128 + threadIdx.x) >> 5;
-  const int lane = threadIdx.x & 31, r = (int)(w / L.heads), h = (int)(w % L.heads), o = h * L.pp;
-  if (r >= rows) return;
-  const T* src = y + (size_t)r * ldy + o;
-  float s = 0.f;
-  for (int d = lane; d < L.p; d += 32) {
-    const float f = to_f(src[d]);
-    s = fmaf(f, f, s);
+                     T* __restrict__ cat, int ldc, int lanes, float eps) {
+  const size_t r = blockIdx.x;
+  const int lane = threadIdx.x % lanes, vecs = L.pp / 8;
+  for (int h = threadIdx.x / lanes; h < ((L.heads + DPOST_THREADS / lanes - 1) & ~(DPOST_THREADS / lanes - 1));
+       h += DPOST_THREADS / lanes) {
+    const bool live = h < L.heads;
+    float ss = 0.f, f[8], g[8], w[8];
+    auto load = [&](int v) {
+      const int o = h * L.pp + v * 8;
+      load8(y + r * ldy + o, f);
+      load8(proj + r * ld + L.off_gg + o, g);
+      load8(L.gnorm + o, w);
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+        if (v * 8 + j >= L.p) f[j] = 0.f;
+    };
+    for (int v = lane; live && v < vecs; v += lanes) {
+      load(v);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss = fmaf(f[j], f[j], ss);
+    }
+    for (int o = 1; o < lanes; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float rstd = 1.f / sqrtf(ss / (float)L.p + eps);
+    for (int v = lane; live && v < vecs; v += lanes) {
+      if (vecs > lanes) load(v);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[j] *= rstd * w[j] * sigmoid_as<T>(g[j]);
+      store8(cat + r * ldc + h * L.pp + v * 8, f);
+    }
   }
-  const float rstd = 1.f / sqrtf(warp_sum(s) / (float)L.p + eps);
-  const T* g = proj + (size_t)r * ld + L.off_gg + o;
-  T* dst = cat + (size_t)r * ldc + o;
-  for (int d = lane; d < L.pp; d += 32)
-    dst[d] = from_f<T>(d < L.p ? to_f(src[d]) * rstd * L.gnorm[o + d] * sigmoid_as<T>(to_f(g[d])) : 0.f);
 }
 
 template <typename T>
@@ -402,7 +620,7 @@ template <int DP, int CW>
 static int launch_scan_regs(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, cudaStream_t s) {
   using T = __nv_bfloat16;
   static PerDeviceOnce once;
-  constexpr int smem = 2 * DT_T * (6 * DP + 4) * 4, cols = CW * (32 / (DP / 16)) * 2;
+  constexpr int smem = 2 * DT_GROUPS * DeltaGroup<DP>::SIZE * 4, cols = CW * (32 / (DP > 64 ? 8 : 4)) * 2;
   const cudaError_t e = ensure_dyn_smem(once, hy_delta_scan_kernel<T, DP, CW>, smem);
   if (e != cudaSuccess) return (int)e;
   hy_delta_scan_kernel<T, DP, CW><<<dim3((L.p + cols - 1) / cols, L.heads, b.ns_pre), (CW + DT_PREP) * 32, smem, s>>>(
@@ -414,11 +632,8 @@ static int launch_scan_regs(const BbHyLayer& L, const BbHyWork& w, const BbHyBat
 static int launch_scan_bf16(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, cudaStream_t s) {
   const long pairs = (long)b.ns_pre * L.heads;
   const int sms = sm_count();
-  if (L.p <= 32) return launch_scan_regs<32, 1>(L, w, b, s);
-  if (L.p <= 64) {
-    if (pairs * 4 <= sms) return launch_scan_regs<64, 1>(L, w, b, s);
-    return pairs <= sms ? launch_scan_regs<64, 2>(L, w, b, s) : launch_scan_regs<64, 4>(L, w, b, s);
-  }
+  if (L.p <= 32) return launch_scan_regs<32, 2>(L, w, b, s);
+  if (L.p <= 64) return pairs * 4 <= sms ? launch_scan_regs<64, 1>(L, w, b, s) : (pairs * 2 <= sms ? launch_scan_regs<64, 2>(L, w, b, s) : launch_scan_regs<64, 4>(L, w, b, s));
   if (L.p <= 128) return pairs * 8 <= sms ? launch_scan_regs<128, 2>(L, w, b, s) : launch_scan_regs<128, 4>(L, w, b, s);
   return BB_ESIZE;
 }
@@ -443,9 +658,11 @@ static int launch_decode(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch&
 
 template <typename T>
 static int launch_post(const BbHyLayer& L, const BbHyWork& w, int rows, float eps, cudaStream_t s) {
-  const int grid = (int)(((long)rows * L.heads * 32 + 127) / 128);
-  hy_delta_post_kernel<T><<<grid, 128, 0, s>>>(L, static_cast<const T*>(w.proj), w.ld_proj, static_cast<const T*>(w.y), w.ld_y,
-                                               static_cast<T*>(w.cat), w.ld_cat, rows, eps);
+  int lanes = 1;
+  while (lanes < L.pp / 8 && lanes < 32) lanes <<= 1;
+  hy_delta_post_kernel<T><<<rows, DPOST_THREADS, 0, s>>>(L, static_cast<const T*>(w.proj), w.ld_proj,
+                                                         static_cast<const T*>(w.y), w.ld_y, static_cast<T*>(w.cat), w.ld_cat,
+                                                         lanes, eps);
   return (int)cudaGetLastError();
 }
 

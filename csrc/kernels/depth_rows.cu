@@ -5,6 +5,7 @@
 //   hy_polynorm    a N(z) + b N(z^2) + c N(z^3) + e over a row of the up projection, N dividing by the root
 //                  mean square -> the feed-forward's part of the row the output projection multiplies
 #include "../common/host.hpp"
+#include "../common/ptx.cuh"
 #include "../common/rows.cuh"
 #include "../serve/hybrid.hpp"
 
@@ -162,9 +163,21 @@ hy_polynorm_kernel(const T* __restrict__ proj, int ld, int off_up, const float* 
     value(i, f);
     add(f);
   }
-  s2 = block_sum(s2, buf[0]);
-  s4 = block_sum(s4, buf[1]);
-  s6 = block_sum(s6, buf[2]);
+  s2 = warp_sum(s2);
+  s4 = warp_sum(s4);
+  s6 = warp_sum(s6);
+  if ((threadIdx.x & 31) == 0) {
+    buf[0][threadIdx.x >> 5] = s2;
+    buf[1][threadIdx.x >> 5] = s4;
+    buf[2][threadIdx.x >> 5] = s6;
+  }
+  __syncthreads();
+  s2 = s4 = s6 = 0.f;
+  for (int i = 0; i < (int)blockDim.x >> 5; ++i) {
+    s2 += buf[0][i];
+    s4 += buf[1][i];
+    s6 += buf[2][i];
+  }
   const float inv = 1.f / (float)ff;
   const float ca = poly[0] / sqrtf(s2 * inv + eps), cb = poly[1] / sqrtf(s4 * inv + eps);
   const float cc = poly[2] / sqrtf(s6 * inv + eps), ce = poly[3];

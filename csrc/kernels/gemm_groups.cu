@@ -1,7 +1,7 @@
 // Side-by-side bf16 products on tcgen05: C_g[M, N] = A_g[M, K] B_g[N, K]^T for g < groups, where A_g and C_g
 // are column ranges of shared row-major buffers (heads of a projection, blocks of a block-diagonal map).
 // One CTA per (128 rows, 128 columns, group): warp 0 feeds a ring of 64-wide K slices by TMA, warp 1 issues
-// the MMAs into TMEM, warps 2..5 store.  K and N are short (a head, a block), so there is one tile per CTA and
+// the MMAs into TMEM, warps 2..5 store through shared memory.  K and N are short (a head, a block), so there is one tile per CTA and
 // two or three CTAs share an SM.  Columns of a slice past K are zero-filled by the copy.
 #include "../common/host.hpp"
 #include "../common/ptx.cuh"
@@ -13,7 +13,7 @@ constexpr int GG_SMEM = GG_STAGES * 2 * GG_TILE + 1024 + 128;
 
 __global__ void __launch_bounds__(192, 3)
 gemm_groups_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
-                   __nv_bfloat16* __restrict__ C, int M, int N, int K, int ldc, int c_step, int* err) {
+                   const __grid_constant__ CUtensorMap tmC, int N, int K, int* err) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint64_t* full = reinterpret_cast<uint64_t*>(smem + GG_STAGES * 2 * GG_TILE);
@@ -73,33 +73,39 @@ gemm_groups_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constan
       umma_commit(done);
     }
   } else {
-    const int ew = warp & 3, row = m0 + ew * 32 + lane;
+    const int ew = warp & 3;
     bool ok = mbar_wait(done, 0);
     ok = __all_sync(0xffffffffu, ok);
     if (!ok) {
       if (lane == 0) set_error(err, ERR_WAIT_EPILOGUE);
     } else {
       tc_fence_after();
-      __nv_bfloat16* crow = C + (size_t)row * ldc + (size_t)g * c_step + n0;
-      const int cols = min(GG_BN, N - n0);
+      // every operand tile has been read: the ring holds the output, 64 columns to a swizzled slab
+      const int cols = min(GG_BN, N - n0), r = ew * 32 + lane;
 #pragma unroll 1
       for (int c = 0; c * 32 < cols; ++c) {
-        uint32_t r[32];
+        uint32_t v[32];
         __syncwarp();
-        tmem_ld32(tmem + ((uint32_t)(ew * 32) << 16) + c * 32, r);
+        tmem_ld32(tmem + ((uint32_t)(ew * 32) << 16) + c * 32, v);
         tmem_wait_ld();
-        if (row >= M) continue;
+        uint8_t* p = smem + (c >> 1) * GG_TILE + r * 128;
 #pragma unroll
         for (int q = 0; q < 4; ++q) {
-          if (c * 32 + q * 8 >= cols) break;
           uint4 o;
-          o.x = pack_bf16x2(__uint_as_float(r[q * 8 + 0]), __uint_as_float(r[q * 8 + 1]));
-          o.y = pack_bf16x2(__uint_as_float(r[q * 8 + 2]), __uint_as_float(r[q * 8 + 3]));
-          o.z = pack_bf16x2(__uint_as_float(r[q * 8 + 4]), __uint_as_float(r[q * 8 + 5]));
-          o.w = pack_bf16x2(__uint_as_float(r[q * 8 + 6]), __uint_as_float(r[q * 8 + 7]));
-          *reinterpret_cast<uint4*>(crow + c * 32 + q * 8) = o;
+          o.x = pack_bf16x2(__uint_as_float(v[q * 8 + 0]), __uint_as_float(v[q * 8 + 1]));
+          o.y = pack_bf16x2(__uint_as_float(v[q * 8 + 2]), __uint_as_float(v[q * 8 + 3]));
+          o.z = pack_bf16x2(__uint_as_float(v[q * 8 + 4]), __uint_as_float(v[q * 8 + 5]));
+          o.w = pack_bf16x2(__uint_as_float(v[q * 8 + 6]), __uint_as_float(v[q * 8 + 7]));
+          *reinterpret_cast<uint4*>(p + (((c & 1) * 4 + q) ^ (r & 7)) * 16) = o;
         }
       }
+      fence_proxy_async_smem();
+    }
+    asm volatile("bar.sync 1, 128;" ::: "memory");
+    if (ok && ew == 0 && lane == 0) {
+      for (int c = 0; c * 64 < N - n0 && c < GG_BN / 64; ++c) tma_store_3d(&tmC, smem + c * GG_TILE, n0 + c * 64, m0, g);
+      tma_store_commit();
+      tma_store_wait<0>();
     }
   }
   tc_fence_before();
@@ -119,16 +125,18 @@ BB_API int bb_gemm_bf16_groups(const void* A, const void* B, void* C, int M, int
   using namespace bb;
   if (M <= 0 || N <= 0 || K <= 0 || groups <= 0 || groups > 65535) return BB_EARG;
   if (N % 8 || K % 8 || lda % 8 || a_step % 8 || ldc % 8 || c_step % 8) return BB_EARG;
-  CUtensorMap ta, tb;
+  CUtensorMap ta, tb, tc;
   const CUtensorMapDataType bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   int rc = make_tmap_3d(&ta, bf, 2, A, K, M, groups, (uint64_t)lda * 2, (uint64_t)a_step * 2, 64, GG_BM);
   if (rc) return rc;
   rc = make_tmap_3d(&tb, bf, 2, B, K, N, groups, (uint64_t)K * 2, (uint64_t)N * K * 2, 64, GG_BN);
   if (rc) return rc;
+  rc = make_tmap_3d(&tc, bf, 2, C, N, M, groups, (uint64_t)ldc * 2, (uint64_t)c_step * 2, 64, GG_BM);
+  if (rc) return rc;
   static PerDeviceOnce once;
   const cudaError_t e = ensure_dyn_smem(once, gemm_groups_kernel, GG_SMEM);
   if (e != cudaSuccess) return (int)e;
   gemm_groups_kernel<<<dim3((N + GG_BN - 1) / GG_BN, (M + GG_BM - 1) / GG_BM, groups), 192, GG_SMEM, (cudaStream_t)stream>>>(
-      ta, tb, static_cast<__nv_bfloat16*>(C), M, N, K, ldc, c_step, device_error_word());
+      ta, tb, tc, N, K, device_error_word());
   return (int)cudaGetLastError();
 }

@@ -17,93 +17,148 @@ namespace bb {
 
 constexpr int LAT_THREADS = 128;
 
-// Rotates the pairs (2i, 2i + 1) of 8 consecutive entries starting at d.
-__device__ __forceinline__ void rotate_pairs8(float (&f)[8], const float* ct, const float* st, int d, int rot) {
+// Rotation of the pairs (2i, 2i + 1) of 8 consecutive entries: their angles, then the entries.
+struct Angles4 {
+  float c[4], s[4];
+};
+__device__ __forceinline__ Angles4 load_angles(const float* ct, const float* st, int d, int rot) {
+  Angles4 a;
+  if ((rot & 7) == 0) {
+    const float4 c = *reinterpret_cast<const float4*>(ct + (d >> 1)), s = *reinterpret_cast<const float4*>(st + (d >> 1));
+    return {{c.x, c.y, c.z, c.w}, {s.x, s.y, s.z, s.w}};
+  }
 #pragma unroll
-  for (int j = 0; j < 8; j += 2) {
-    if (d + j < rot) {
-      const float c = ct[(d + j) >> 1], s = st[(d + j) >> 1], u = f[j], v = f[j + 1];
-      f[j] = u * c - v * s;
-      f[j + 1] = v * c + u * s;
-    }
+  for (int j = 0; j < 4; ++j) {
+    const bool in = d + 2 * j < rot;         // padding is zero and stays so
+    a.c[j] = in ? ct[(d >> 1) + j] : 1.f;
+    a.s[j] = in ? st[(d >> 1) + j] : 0.f;
+  }
+  return a;
+}
+__device__ __forceinline__ void rotate_pairs8(float (&f)[8], const Angles4& a) {
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const float u = f[2 * j], v = f[2 * j + 1];
+    f[2 * j] = u * a.c[j] - v * a.s[j];
+    f[2 * j + 1] = v * a.c[j] + u * a.s[j];
   }
 }
 
+// A thread's vectors of the row (query latent, then page row) stay in registers up to KEEP of them.
 template <typename T>
 __global__ void __launch_bounds__(LAT_THREADS)
 hy_latent_in_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, int ld, const int* __restrict__ pos_,
                     const int* __restrict__ row_seq, const int* __restrict__ tables, int max_blocks, int bs, float eps) {
+  constexpr int KEEP = 3;
   __shared__ float buf[2][32];
-  const int r = blockIdx.x;
+  const int r = blockIdx.x, width = L.kvrp + L.rotp, n = L.qrp + (L.own_kv ? width : 0);
   T* q = proj + (size_t)r * ld + L.off_dq;
   const T* c = proj + (size_t)r * ld + L.off_ckv;
-  float sq = 0.f, sc = 0.f;
-  for (int i = threadIdx.x * 8; i < L.qrp; i += LAT_THREADS * 8) {
+  const int pos = pos_[r];
+  float v[KEEP][8], sq = 0.f, sc = 0.f;
+  auto sum = [&](int i, const float (&f)[8]) {
+    float t = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) t += f[j] * f[j];
+    if (i < L.qrp) sq += t;
+    else if (i < L.qrp + L.kvrp) sc += t;
+  };
+#pragma unroll
+  for (int t = 0; t < KEEP; ++t) {
+    const int i = (threadIdx.x + t * LAT_THREADS) * 8;
+    if (i < n) load8(i < L.qrp ? q + i : c + (i - L.qrp), v[t]);
+  }
+#pragma unroll
+  for (int t = 0; t < KEEP; ++t) {
+    const int i = (threadIdx.x + t * LAT_THREADS) * 8;
+    if (i < n) sum(i, v[t]);
+  }
+  for (int i = (threadIdx.x + KEEP * LAT_THREADS) * 8; i < n; i += LAT_THREADS * 8) {
     float f[8];
-    load8(q + i, f);
-#pragma unroll
-    for (int j = 0; j < 8; ++j) sq += f[j] * f[j];
+    load8(i < L.qrp ? q + i : c + (i - L.qrp), f);
+    sum(i, f);
   }
-  if (L.own_kv)
-    for (int i = threadIdx.x * 8; i < L.kvrp; i += LAT_THREADS * 8) {
-      float f[8];
-      load8(c + i, f);
+  const int blk = L.own_kv ? tables[(size_t)row_seq[r] * max_blocks + pos / bs] : 0;
+  sq = warp_sum(sq);
+  sc = warp_sum(sc);
+  if ((threadIdx.x & 31) == 0) {
+    buf[0][threadIdx.x >> 5] = sq;
+    buf[1][threadIdx.x >> 5] = sc;
+  }
+  __syncthreads();
+  sq = sc = 0.f;
 #pragma unroll
-      for (int j = 0; j < 8; ++j) sc += f[j] * f[j];
-    }
-  sq = block_sum(sq, buf[0]);
-  sc = block_sum(sc, buf[1]);
+  for (int i = 0; i < LAT_THREADS / 32; ++i) {
+    sq += buf[0][i];
+    sc += buf[1][i];
+  }
   const float rq = 1.f / sqrtf(sq / (float)L.qr + eps), rc = 1.f / sqrtf(sc / (float)L.kvr + eps);
-  for (int i = threadIdx.x * 8; i < L.qrp; i += LAT_THREADS * 8) {
-    float f[8], g[8];
-    load8(q + i, f);
-    load8(L.dq_norm + i, g);
+  T* page = static_cast<T*>(L.kc) + ((size_t)blk * bs + pos % bs) * width;
+  auto emit = [&](int i, float (&f)[8]) {
+    float g[8];
+    if (i < L.qrp) {
+      load8(L.dq_norm + i, g);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) f[j] *= rq * g[j];
-    store8(q + i, f);
-  }
-  if (!L.own_kv) return;
-  const int pos = pos_[r], width = L.kvrp + L.rotp;
-  T* page = static_cast<T*>(L.kc) + ((size_t)tables[(size_t)row_seq[r] * max_blocks + pos / bs] * bs + pos % bs) * width;
-  const float* ct = L.cos_t + (size_t)pos * (L.rot >> 1);
-  const float* st = L.sin_t + (size_t)pos * (L.rot >> 1);
-  for (int i = threadIdx.x * 8; i < width; i += LAT_THREADS * 8) {
-    float f[8], g[8];
-    load8(c + i, f);
+      for (int j = 0; j < 8; ++j) f[j] *= rq * g[j];
+      store8(q + i, f);
+      return;
+    }
+    i -= L.qrp;
     if (i < L.kvrp) {
       load8(L.dkv_norm + i, g);
 #pragma unroll
       for (int j = 0; j < 8; ++j) f[j] *= rc * g[j];
     } else {
-      rotate_pairs8(f, ct, st, i - L.kvrp, L.rot);
+      const size_t at = (size_t)pos * (L.rot >> 1);
+      rotate_pairs8(f, load_angles(L.cos_t + at, L.sin_t + at, i - L.kvrp, L.rot));
     }
     store8(page + i, f);
+  };
+#pragma unroll
+  for (int t = 0; t < KEEP; ++t) {
+    const int i = (threadIdx.x + t * LAT_THREADS) * 8;
+    if (i < n) emit(i, v[t]);
+  }
+  for (int i = (threadIdx.x + KEEP * LAT_THREADS) * 8; i < n; i += LAT_THREADS * 8) {
+    float f[8];
+    load8(i < L.qrp ? q + i : c + (i - L.qrp), f);
+    emit(i, f);
   }
 }
 
-// Rows below n_in place rotate inside q; row r of the others writes to qa row r - n_in.
+// Rows below n_in rotate in place inside q; row r of the others writes to qa row r - n_in.  Lanes run over the
+// vectors of a head's rotated part, then heads; a thread takes every step-th head.
+constexpr int LQ_HEADS = 4;
+
 template <typename T>
 __global__ void __launch_bounds__(LAT_THREADS)
 hy_latent_q_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ q, int ldq, T* __restrict__ qa, int ldqa,
-                   const int* __restrict__ pos_, int rows, int n_in) {
-  const int vecs = L.rotp / 8;
-  const long t = (long)blockIdx.x * LAT_THREADS + threadIdx.x;
-  const int r = (int)(t / (L.hq * vecs)), hv = (int)(t % (L.hq * vecs));
-  if (r >= rows) return;
-  const int h = hv / vecs, d = (hv % vecs) * 8, pos = pos_[r];
-  T* src = q + (size_t)r * ldq + h * (L.dkp + L.rotp) + L.dkp + d;
-  float f[8];
-  load8(src, f);
-  rotate_pairs8(f, L.cos_t + (size_t)pos * (L.rot >> 1), L.sin_t + (size_t)pos * (L.rot >> 1), d, L.rot);
-  T* dst = r < n_in ? src : qa + (size_t)(r - n_in) * ldqa + h * (L.kvrp + L.rotp) + L.kvrp + d;
-  store8(dst, f);
+                   const int* __restrict__ pos_, int n_in, int step) {
+  const unsigned vecs = L.rotp / 8, t = blockIdx.y * LAT_THREADS + threadIdx.x;
+  const int h0 = t / vecs, d = (t - h0 * vecs) * 8, r = blockIdx.x;
+  if (h0 >= step) return;
+  const int pos = pos_[r];
+  T* row = q + (size_t)r * ldq + L.dkp + d;
+  float f[LQ_HEADS][8];
+#pragma unroll
+  for (int i = 0; i < LQ_HEADS; ++i)
+    if (h0 + i * step < L.hq) load8(row + (h0 + i * step) * (L.dkp + L.rotp), f[i]);
+  const size_t at = (size_t)pos * (L.rot >> 1);
+  const Angles4 a = load_angles(L.cos_t + at, L.sin_t + at, d, L.rot);
+#pragma unroll
+  for (int i = 0; i < LQ_HEADS; ++i) {
+    const int h = h0 + i * step;
+    if (h >= L.hq) break;
+    rotate_pairs8(f[i], a);
+    store8(r < n_in ? row + h * (L.dkp + L.rotp) : qa + (size_t)(r - n_in) * ldqa + h * (L.kvrp + L.rotp) + L.kvrp + d, f[i]);
+  }
 }
 
 __global__ void __launch_bounds__(LAT_THREADS)
 hy_latent_gather_kernel(const uint4* __restrict__ pages, const int* __restrict__ src, uint4* __restrict__ out, int vecs,
                         int ld_vecs, int rows, int pool_rows) {
-  const long t = (long)blockIdx.x * LAT_THREADS + threadIdx.x;
-  const int r = (int)(t / vecs), v = (int)(t % vecs);
+  const unsigned t = blockIdx.x * LAT_THREADS + threadIdx.x;
+  const int r = t / (unsigned)vecs, v = t - r * vecs;
   if (r >= rows) return;
   const int p = min(max(src[r], 0), pool_rows - 1);
   out[(size_t)r * ld_vecs + v] = pages[(size_t)p * vecs + v];
@@ -193,15 +248,15 @@ BB_API int bb_hy_latent_in(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork*
 // n_in: leading rows whose rotated queries stay in place.
 BB_API int bb_hy_latent_q(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int n_in, void* stream) {
   cudaStream_t s = (cudaStream_t)stream;
-  const long t = (long)b->n * L->hq * (L->rotp / 8);
-  const int grid = (int)((t + LAT_THREADS - 1) / LAT_THREADS);
+  const int step = (L->hq + LQ_HEADS - 1) / LQ_HEADS;
+  const dim3 grid(b->n, (step * (L->rotp / 8) + LAT_THREADS - 1) / LAT_THREADS);
   if (c->dtype)
     hy_latent_q_kernel<float><<<grid, LAT_THREADS, 0, s>>>(*L, static_cast<float*>(w->q), w->ld_q, static_cast<float*>(w->qa),
-                                                           w->ld_qa, b->pos, b->n, n_in);
+                                                           w->ld_qa, b->pos, n_in, step);
   else
     hy_latent_q_kernel<__nv_bfloat16><<<grid, LAT_THREADS, 0, s>>>(*L, static_cast<__nv_bfloat16*>(w->q), w->ld_q,
-                                                                   static_cast<__nv_bfloat16*>(w->qa), w->ld_qa, b->pos, b->n,
-                                                                   n_in);
+                                                                   static_cast<__nv_bfloat16*>(w->qa), w->ld_qa, b->pos, n_in,
+                                                                   step);
   return (int)cudaGetLastError();
 }
 

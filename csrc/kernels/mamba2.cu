@@ -16,7 +16,7 @@
 
 namespace bb {
 
-constexpr int CONV_ROWS = 8;   // consecutive rows of a thread, their inputs asked for together
+constexpr int CONV_ROWS = 8;   // consecutive rows of a thread in portions, their inputs asked for together
 
 template <typename T>
 struct alignas(sizeof(T) * 4) Raw4 {
@@ -42,13 +42,13 @@ __device__ __forceinline__ Raw4<T> conv_tap(const BbHyLayer& L, const T* proj, i
 
 // TAPS = 4 keeps a thread's inputs in registers as they are stored; TAPS = 0 reads every tap again (any
 // length).
-template <typename T, int TAPS, bool SILU>
+template <typename T, int TAPS, bool SILU, int ROWS>
 __global__ void __launch_bounds__(128, sizeof(T) == 2 ? 7 : 5)
 hy_conv_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, int ld, T* __restrict__ xbc, int ldx,
-               float* __restrict__ dt, int lddt, const __grid_constant__ BbHyBatch b, int rows) {
+               float* __restrict__ dt, int lddt, const __grid_constant__ BbHyBatch b, int row0, int rows) {
   const int cv = blockIdx.x * 128 + threadIdx.x;   // vector of 4 channels, then vectors of 4 step sizes
   const int nch = L.chp / 4, ndt = (L.heads + 7) / 8 * 2;
-  const int r0 = blockIdx.y * CONV_ROWS, r1 = min(r0 + CONV_ROWS, rows);
+  const int r0 = row0 + blockIdx.y * ROWS, r1 = min(r0 + ROWS, row0 + rows);
   if (cv >= nch + ndt) return;
   if (cv >= nch) {
     const int h0 = (cv - nch) * 4;
@@ -72,14 +72,14 @@ hy_conv_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, 
   }
   if constexpr (TAPS > 0) {
     constexpr int K = TAPS - 1;
-    Raw4<T> raw[CONV_ROWS + K];   // raw[K + i]: row r0 + i; before it the inputs ahead of r0
+    Raw4<T> raw[ROWS + K];   // raw[K + i]: row r0 + i; before it the inputs ahead of r0
 #pragma unroll
-    for (int i = 0; i < CONV_ROWS; ++i)
+    for (int i = 0; i < ROWS; ++i)
       if (r0 + i < r1) raw[K + i] = *reinterpret_cast<const Raw4<T>*>(proj + (size_t)(r0 + i) * ld + L.off_xbc + c);
     // the rows before r0 are asked for before it is known whether they are this sequence's
 #pragma unroll
     for (int k = 1; k <= K; ++k)
-      if (r0 >= k) raw[K - k] = *reinterpret_cast<const Raw4<T>*>(proj + (size_t)(r0 - k) * ld + L.off_xbc + c);
+      if (ROWS > 1 && r0 >= k) raw[K - k] = *reinterpret_cast<const Raw4<T>*>(proj + (size_t)(r0 - k) * ld + L.off_xbc + c);
     int last_seq = b.row_seq[r0];
     const bool one = last_seq == b.row_seq[r1 - 1];   // all rows of this thread belong to one sequence
     {
@@ -95,7 +95,7 @@ hy_conv_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, 
       w[k][0] = t.x; w[k][1] = t.y; w[k][2] = t.z; w[k][3] = t.w;
     }
 #pragma unroll
-    for (int i = 0; i < CONV_ROWS; ++i) {
+    for (int i = 0; i < ROWS; ++i) {
       const int r = r0 + i;
       if (r >= r1) break;
       if (!one) {
@@ -296,15 +296,15 @@ hy_ssm_decode_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
   }
 }
 
-template <typename T, bool SILU>
-static int launch_conv(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, int rows, cudaStream_t s) {
+template <typename T, bool SILU, int ROWS>
+static int launch_conv(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, int row0, int rows, cudaStream_t s) {
   const int vecs = L.chp / 4 + (L.heads + 7) / 8 * 2;
-  dim3 grid((vecs + 127) / 128, (rows + CONV_ROWS - 1) / CONV_ROWS);
+  dim3 grid((vecs + 127) / 128, (rows + ROWS - 1) / ROWS);
   if (grid.y > 65535) return BB_ESIZE;
   const T* proj = static_cast<const T*>(w.proj);
   T* xbc = static_cast<T*>(w.xbc);
-  if (L.taps == 4) hy_conv_kernel<T, 4, SILU><<<grid, 128, 0, s>>>(L, proj, w.ld_proj, xbc, w.ld_xbc, w.dt, w.ld_dt, b, rows);
-  else hy_conv_kernel<T, 0, SILU><<<grid, 128, 0, s>>>(L, proj, w.ld_proj, xbc, w.ld_xbc, w.dt, w.ld_dt, b, rows);
+  if (L.taps == 4) hy_conv_kernel<T, 4, SILU, ROWS><<<grid, 128, 0, s>>>(L, proj, w.ld_proj, xbc, w.ld_xbc, w.dt, w.ld_dt, b, row0, rows);
+  else hy_conv_kernel<T, 0, SILU, ROWS><<<grid, 128, 0, s>>>(L, proj, w.ld_proj, xbc, w.ld_xbc, w.dt, w.ld_dt, b, row0, rows);
   return (int)cudaGetLastError();
 }
 
@@ -350,14 +350,22 @@ using namespace bb;
 
 BB_API int bb_hy_conv(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream) {
   if (b->n_pre <= 0) return BB_OK;
-  return c->dtype ? launch_conv<float, true>(*L, *w, *b, b->n_pre, (cudaStream_t)stream)
-                  : launch_conv<__nv_bfloat16, true>(*L, *w, *b, b->n_pre, (cudaStream_t)stream);
+  return c->dtype ? launch_conv<float, true, CONV_ROWS>(*L, *w, *b, 0, b->n_pre, (cudaStream_t)stream)
+                  : launch_conv<__nv_bfloat16, true, CONV_ROWS>(*L, *w, *b, 0, b->n_pre, (cudaStream_t)stream);
 }
 
 // The same without activation, with the inputs' bias x_b, for every row of the step.
 BB_API int bb_hy_conv_linear(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream) {
-  return c->dtype ? launch_conv<float, false>(*L, *w, *b, b->n, (cudaStream_t)stream)
-                  : launch_conv<__nv_bfloat16, false>(*L, *w, *b, b->n, (cudaStream_t)stream);
+  cudaStream_t s = (cudaStream_t)stream;
+  const int dec = b->n - b->n_pre;       // rows of different sequences: one to a thread
+  int rc = BB_OK;
+  if (b->n_pre > 0)
+    rc = c->dtype ? launch_conv<float, false, CONV_ROWS>(*L, *w, *b, 0, b->n_pre, s)
+                  : launch_conv<__nv_bfloat16, false, CONV_ROWS>(*L, *w, *b, 0, b->n_pre, s);
+  if (rc == BB_OK && dec > 0)
+    rc = c->dtype ? launch_conv<float, false, 1>(*L, *w, *b, b->n_pre, dec, s)
+                  : launch_conv<__nv_bfloat16, false, 1>(*L, *w, *b, b->n_pre, dec, s);
+  return rc;
 }
 
 BB_API int bb_hy_ssm_scan(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream) {

@@ -14,23 +14,26 @@
 
 namespace bb {
 
+// Two channels as they are stored.
+template <typename T>
+struct alignas(sizeof(T) * 2) Pair {
+  T v[2];
+  __device__ __forceinline__ float2 f() const { return make_float2(to_f(v[0]), to_f(v[1])); }
+};
+template <typename T>
+__device__ __forceinline__ Pair<T> raw_pair(const T* p) {
+  return *reinterpret_cast<const Pair<T>*>(p);
+}
 template <typename T>
 __device__ __forceinline__ float2 load_pair(const T* p) {
-  struct alignas(sizeof(T) * 2) P {
-    T v[2];
-  };
-  const P q = *reinterpret_cast<const P*>(p);
-  return make_float2(to_f(q.v[0]), to_f(q.v[1]));
+  return raw_pair(p).f();
 }
 template <typename T>
 __device__ __forceinline__ void store_pair(T* p, float a, float b) {
-  struct alignas(sizeof(T) * 2) P {
-    T v[2];
-  };
-  P q;
+  Pair<T> q;
   q.v[0] = from_f<T>(a);
   q.v[1] = from_f<T>(b);
-  *reinterpret_cast<P*>(p) = q;
+  *reinterpret_cast<Pair<T>*>(p) = q;
 }
 
 // Everything below is 32-bit; with bf16 storage exponentials and divisions are the hardware's (2^-22).
@@ -49,6 +52,11 @@ __device__ __forceinline__ float decay_m1(float x) {
   } else {
     return expm1f(-x);
   }
+}
+template <typename T>
+__device__ __forceinline__ float root_of(float x) {
+  if constexpr (sizeof(T) == 2) return x * rsqrtf(fmaxf(x, 1e-37f));
+  else return sqrtf(x);
 }
 // S after a token of (e, in); product of two decays
 __device__ __forceinline__ float2 lru_apply(float2 e, float2 s, float2 in) {
@@ -69,8 +77,8 @@ __device__ __forceinline__ LruChannels lru_channels(const BbHyLayer& L, int c) {
 template <typename T>
 __device__ __forceinline__ void lru_token(const LruChannels& p, float2 r, float2 i, float2 u, float2& e, float2& in) {
   e = make_float2(decay_m1<T>(p.lam.x * sigmoid_as<T>(r.x + p.rb.x)), decay_m1<T>(p.lam.y * sigmoid_as<T>(r.y + p.rb.y)));
-  in = make_float2(sqrtf(-e.x * (2.f + e.x)) * sigmoid_as<T>(i.x + p.ib.x) * u.x,
-                   sqrtf(-e.y * (2.f + e.y)) * sigmoid_as<T>(i.y + p.ib.y) * u.y);
+  in = make_float2(root_of<T>(-e.x * (2.f + e.x)) * sigmoid_as<T>(i.x + p.ib.x) * u.x,
+                   root_of<T>(-e.y * (2.f + e.y)) * sigmoid_as<T>(i.y + p.ib.y) * u.y);
 }
 
 template <typename T>
@@ -99,23 +107,29 @@ hy_rglru_scan_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
   const LruChannels ch = lru_channels(L, cc);
   float* state = L.ssm_state + (size_t)slot * L.chp + cc;
   float2 carry = pos0 == 0 ? make_float2(0.f, 0.f) : *reinterpret_cast<const float2*>(state);
+  // a warp's tokens of the next step are on their way while it works on this one's
+  Pair<T> rr[LRU_T], ii[LRU_T], uu[LRU_T], yy[LRU_T];
+  auto fetch = [&](int tw) {
+#pragma unroll
+    for (int k = 0; k < LRU_T; ++k) {
+      const size_t row = r0 + min(tw + k, n - 1);
+      rr[k] = raw_pair(gates + row * ldg + g0);
+      ii[k] = raw_pair(gates + row * ldg + g0 + L.bwp);
+      uu[k] = raw_pair(u + row * ldu + cc);
+    }
+  };
+  fetch(warp * LRU_T);
   for (int t0 = 0, it = 0; t0 < n; t0 += LRU_WARPS * LRU_T, ++it) {
     const int tw = t0 + warp * LRU_T;
+#pragma unroll
+    for (int k = 0; k < LRU_T; ++k) yy[k] = raw_pair(proj + (size_t)(r0 + min(tw + k, n - 1)) * ld + L.off_y + cc);
     float2 p[LRU_T], s[LRU_T];
     {
-      float2 rr[LRU_T], ii[LRU_T], uu[LRU_T];
-#pragma unroll
-      for (int k = 0; k < LRU_T; ++k) {
-        const size_t row = r0 + min(tw + k, n - 1);
-        rr[k] = load_pair(gates + row * ldg + g0);
-        ii[k] = load_pair(gates + row * ldg + g0 + L.bwp);
-        uu[k] = load_pair(u + row * ldu + cc);
-      }
       float2 pa = make_float2(0.f, 0.f), sa = make_float2(0.f, 0.f);
 #pragma unroll
       for (int k = 0; k < LRU_T; ++k) {
         float2 e, in;
-        lru_token<T>(ch, rr[k], ii[k], uu[k], e, in);
+        lru_token<T>(ch, rr[k].f(), ii[k].f(), uu[k].f(), e, in);
         if (tw + k >= n) e = in = make_float2(0.f, 0.f);      // past the end: nothing changes
         sa = lru_apply(e, sa, in);
         pa = lru_product(pa, e);
@@ -123,6 +137,7 @@ hy_rglru_scan_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
         s[k] = sa;
       }
     }
+    fetch(tw + LRU_WARPS * LRU_T);
     chain[it & 1][warp][0][lane] = p[LRU_T - 1];
     chain[it & 1][warp][1][lane] = s[LRU_T - 1];
     __syncthreads();
@@ -136,7 +151,7 @@ hy_rglru_scan_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
     for (int k = 0; k < LRU_T; ++k) {
       if (tw + k < n && live) {
         const size_t row = r0 + tw + k;
-        const float2 yv = load_pair(proj + row * ld + L.off_y + cc);
+        const float2 yv = yy[k].f();
         const float2 st = lru_apply(p[k], mine, s[k]);
         store_pair(cat + row * ldc + cc, st.x * gelu_as<T>(yv.x + ch.yb.x), st.y * gelu_as<T>(yv.y + ch.yb.y));
         keep_input<T>(L, proj + row * ld, cc, pos0 + tw + k, ctx, slot);

@@ -11,6 +11,7 @@
 // bf16: the tensor-core GEMM, paged flash prefill, split-KV decode attention and chunked state-space
 // kernels; fp32: the CUDA-core forms of the same steps.
 #include <cstdint>
+#include <mutex>
 
 #include "../common/host.hpp"
 #include "hybrid.hpp"
@@ -203,17 +204,55 @@ int mixer(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBat
   }
 }
 
+// Small steps leave most of the machine idle, so a layer's feed-forward half runs beside its mixer: on a stream
+// of its own, forked behind the norms and joined before the output GEMM (a captured graph gets both branches).
+constexpr int BESIDE_ROWS = 256;
+
+struct SideStream {
+  cudaStream_t s = nullptr;
+  cudaEvent_t fork = nullptr, join = nullptr;
+};
+SideStream* side_stream() {
+  static SideStream per_device[64];
+  static std::mutex lock;
+  int dev = 0;
+  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return nullptr;
+  std::lock_guard<std::mutex> g(lock);
+  SideStream& d = per_device[dev];
+  if (!d.s && (cudaEventCreateWithFlags(&d.fork, cudaEventDisableTiming) != cudaSuccess ||
+               cudaEventCreateWithFlags(&d.join, cudaEventDisableTiming) != cudaSuccess ||
+               cudaStreamCreateWithFlags(&d.s, cudaStreamNonBlocking) != cudaSuccess))
+    return nullptr;
+  return &d;
+}
+#define BB_CUDA(expr)                           \
+  do {                                          \
+    const cudaError_t e_ = (expr);              \
+    if (e_ != cudaSuccess) return (int)e_;      \
+  } while (0)
+
+int feed_forward(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
+  BB_TRY(project(c, L.up, w.h2, c.dp, at(c, w.proj, L.off_up), w.ld_proj, b.n, s));
+  return bb_hy_polynorm(&c, &L, &w, b.n, s);
+}
+
 int forward_depth(const BbHyCfg& c, const BbHyWork& w, const BbHyBatch& b, float* trace, void* s) {
   const size_t level = (size_t)w.rows * c.dp;
+  SideStream* side = b.n <= BESIDE_ROWS ? side_stream() : nullptr;
   for (int li = 0; li < c.n_layers; ++li) {
     const BbHyLayer& L = c.layers[li];
     BB_TRY(bb_hy_mix_norm(&c, li, &w, &b, trace && li ? trace + (size_t)(li - 1) * b.n * c.dp : nullptr, s));
-    BB_TRY(project(c, L.in, w.h, c.dp, w.proj, w.ld_proj, b.n, s));
-    if (L.ff > 0) {
-      BB_TRY(project(c, L.up, w.h2, c.dp, at(c, w.proj, L.off_up), w.ld_proj, b.n, s));
-      BB_TRY(bb_hy_polynorm(&c, &L, &w, b.n, s));
+    const bool fork = side && L.ff > 0;
+    if (fork) {
+      BB_CUDA(cudaEventRecord(side->fork, (cudaStream_t)s));
+      BB_CUDA(cudaStreamWaitEvent(side->s, side->fork, 0));
+      BB_TRY(feed_forward(c, L, w, b, side->s));
+      BB_CUDA(cudaEventRecord(side->join, side->s));
     }
+    BB_TRY(project(c, L.in, w.h, c.dp, w.proj, w.ld_proj, b.n, s));
     BB_TRY(mixer(c, L, w, b, s));
+    if (fork) BB_CUDA(cudaStreamWaitEvent((cudaStream_t)s, side->join, 0));
+    else if (L.ff > 0) BB_TRY(feed_forward(c, L, w, b, s));
     BB_TRY(project_f32(c, L.out, w.cat, w.ld_cat, w.x + (li + 1) * level, c.dp, b.n, 1.f, 1, s));
   }
   if (trace) {
