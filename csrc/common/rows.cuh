@@ -50,17 +50,36 @@ __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
+// The hardware's approximations (2^-22) with tiny arguments flushed: no code around them for denormals.
+__device__ __forceinline__ float exp2_hw(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp_hw(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rsqrt_hw(float x) {
+  float y;
+  asm("rsqrt.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+constexpr float kLog2e = 1.4426950408889634f;
+__device__ __forceinline__ float exp_hw(float x) { return exp2_hw(x * kLog2e); }
+
 // Activations whose result is stored as T: with bf16 the exponential and the division are the hardware's
-// approximations (2^-22, far below the rounding that follows), with fp32 they are exact.
+// approximations (far below the rounding that follows), with fp32 they are exact.  An exponential that
+// overflows gives a reciprocal of 0, which is the limit of either function there.
 template <typename T>
 __device__ __forceinline__ float sigmoid_as(float x) {
-  if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-x));
+  if constexpr (sizeof(T) == 2) return rcp_hw(1.f + exp2_hw(-kLog2e * x));
   else return sigmoid_f(x);
 }
 template <typename T>
 __device__ __forceinline__ float silu_as(float x) {
-  // (an argument of the fast division above 2^126 gives 0, which is silu's limit there)
-  if constexpr (sizeof(T) == 2) return __fdividef(x, 1.f + __expf(-x));
+  if constexpr (sizeof(T) == 2) return x * rcp_hw(1.f + exp2_hw(-kLog2e * x));
   else return silu_f(x);
 }
 

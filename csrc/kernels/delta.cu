@@ -60,7 +60,7 @@ __device__ __forceinline__ float2 delta_token(const BbHyLayer& L, const T* row, 
     const float k = in ? to_f(row[L.off_kk + o + d]) : 0.f, r = in ? to_f(row[L.off_r + o + d]) : 0.f, u = k * unit;
     const float x = in ? -kDecayScale * sigmoid_as<T>(to_f(low[o + d]) + L.w0[o + d]) : 0.f;
     const float au = in ? sigmoid_as<T>(to_f(row[L.off_a + o + d]) + L.a_b[o + d]) * u : 0.f;
-    const float w = sizeof(T) == 2 ? __expf(x) : expf(x);
+    const float w = sizeof(T) == 2 ? exp_hw(x) : expf(x);
     s.u[d] = u;
     s.wr[d] = w * r;
     s.w[d] = sizeof(T) == 2 ? w : expm1f(x);
@@ -143,10 +143,10 @@ hy_delta_scan_any_kernel(const __grid_constant__ BbHyLayer L, const T* __restric
 //   o_i = (W_0..i r_i)^T S   - sum_{j<=i} (r_i . W_j+1..i a_j u_j) x_j  + sum_{j<=i} (r_i . W_j+1..i k_j) v_j
 //   S   <- W_0..3 S + sum_j (W_j+1..3 k_j) v_j^T - (W_j+1..3 a_j u_j) x_j^T
 // (no decay is ever divided by).  The bracketed numbers do not depend on S: the warps that prepare a group have
-// them ready, and one round of shuffles serves four tokens.  A thread holds CT columns of DP / KL keys, the
-// float4 groups q, q + KL, ... of lane q, so vectors are read from shared memory without bank conflicts.
-constexpr int DG = 4, DT_GROUPS = 4, DT_PREP = 4;      // tokens of a group, groups of a buffer, preparing warps
-static_assert(DT_GROUPS == DT_PREP, "a preparing warp has one group of each buffer");
+// them ready, and one round of shuffles serves four tokens.  A thread holds four columns of eight keys, KL = DP / 8
+// lanes a column: what bounds the kernel is the vectors' way from shared memory into registers, and every one of
+// them then serves four columns.  Sums over keys end with a column to a lane, which solves for x and writes o.
+constexpr int DG = 4;                                // tokens of a group
 
 template <int DP>
 struct DeltaGroup {
@@ -196,15 +196,15 @@ struct DeltaPrep {
   __device__ __forceinline__ void fetch(int r0, int t0, int n) {
     const int d = (threadIdx.x & 31) * V, o = h * L.pp + d;
     const bool in = d < L.pp;                        // (pp is a multiple of V)
+    const T *row = proj + (size_t)(r0 + t0) * ld + o, *lrow = low + (size_t)(r0 + t0) * ldl + o;
 #pragma unroll
-    for (int i = 0; i < DG; ++i) {
+    for (int i = 0; i < DG; ++i, row += ld, lrow += ldl) {
       if (in && t0 + i < n) {
-        const T* row = proj + (size_t)(r0 + t0 + i) * ld + o;
         k[i] = *reinterpret_cast<const Raw*>(row + L.off_kk);
         r[i] = *reinterpret_cast<const Raw*>(row + L.off_r);
         v[i] = *reinterpret_cast<const Raw*>(row + L.off_vv);
         a[i] = *reinterpret_cast<const Raw*>(row + L.off_a);
-        x[i] = *reinterpret_cast<const Raw*>(low + (size_t)(r0 + t0 + i) * ldl + o);
+        x[i] = *reinterpret_cast<const Raw*>(lrow);
         if (L.p != L.pp)
 #pragma unroll
           for (int j = 0; j < V; ++j)
@@ -232,7 +232,7 @@ struct DeltaPrep {
       for (int i = 0; i < DG; ++i) s[i] += __shfl_xor_sync(0xffffffffu, s[i], q);
     float unit[DG];
 #pragma unroll
-    for (int i = 0; i < DG; ++i) unit[i] = rsqrtf(s[i] + kDeltaUnit);
+    for (int i = 0; i < DG; ++i) unit[i] = rsqrt_hw(s[i] + kDeltaUnit);
 #pragma unroll
     for (int i = 0; i < 32; ++i) s[i] = 0.f;
     Out O[3 * DG + 1 + 2 * DG];                      // U, R, W, K, A in the group's order, then v
@@ -242,7 +242,7 @@ struct DeltaPrep {
       float w[DG], u[DG], rr[DG], kk[DG], au[DG];
 #pragma unroll
       for (int i = 0; i < DG; ++i) {
-        w[i] = t0 + i < n ? __expf(-kDecayScale * sigmoid_as<T>(to_f(x[i].v[j]) + w0)) : 1.f;
+        w[i] = t0 + i < n ? exp2_hw(-kDecayScale * kLog2e * sigmoid_as<T>(to_f(x[i].v[j]) + w0)) : 1.f;
         kk[i] = to_f(k[i].v[j]);
         rr[i] = to_f(r[i].v[j]);
         u[i] = kk[i] * unit[i];
@@ -322,18 +322,21 @@ struct DeltaPrep {
   }
 };
 
-template <typename T, int DP, int CW>
-__global__ void __launch_bounds__((CW + DT_PREP) * 32)
+// CW warps walk through the tokens, PREP others prepare one group each of the buffer that comes next; BLOCKS of
+// them are to share an SM.
+template <typename T, int DP, int CW, int PREP, int BLOCKS>
+__global__ void __launch_bounds__((CW + PREP) * 32, BLOCKS)
 hy_delta_scan_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, int ld, const T* __restrict__ low,
                      int ldl, T* __restrict__ y, int ldy, const __grid_constant__ BbHyBatch b) {
   using G = DeltaGroup<DP>;
-  constexpr int KL = DP > 64 ? 8 : 4, KT = DP / KL, CT = 2, QUADS = KT / 4, STEP = DG * DT_GROUPS;
+  constexpr int KL = DP / 8, CT = 4, STEP = DG * PREP, NT = DG * 4 / KL;   // NT: tokens whose outputs a lane finishes
+  static_assert(KL >= 4 && NT >= 1, "a lane for every column of a thread");
   constexpr int COLS = CW * (32 / KL) * CT;          // columns of a block
-  extern __shared__ __align__(16) float sm[];        // [2][DT_GROUPS][G::SIZE]
+  extern __shared__ __align__(16) float sm[];        // [2][PREP][G::SIZE]
   const int seq = blockIdx.z, h = blockIdx.y, D = L.p;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int r0 = b.seq_row0[seq], n = b.seq_row0[seq + 1] - r0;
-  for (int i = threadIdx.x; i < 2 * DT_GROUPS * 64; i += blockDim.x) sm[(i / 64) * G::SIZE + G::X + i % 64] = 0.f;
+  for (int i = threadIdx.x; i < 2 * PREP * 64; i += blockDim.x) sm[(i / 64) * G::SIZE + G::X + i % 64] = 0.f;
   __syncthreads();
   if (warp >= CW) {
     DeltaPrep<T, DP> prep{L, proj, low, ld, ldl, h};
@@ -344,136 +347,179 @@ hy_delta_scan_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ 
     __syncthreads();
     for (int t0 = 0, it = 1; t0 < n; t0 += STEP, ++it) {
       const int t = t0 + STEP + w * DG;
-      prep.finish(sm + ((it & 1) * DT_GROUPS + w) * G::SIZE, t, n);
+      prep.finish(sm + ((it & 1) * PREP + w) * G::SIZE, t, n);
       prep.fetch(r0, t + STEP, n);
       __syncthreads();
     }
     return;
   }
+  // keys 4 q .. 4 q + 3 and DP / 2 + 4 q .. of columns c0 .. c0 + 3
   const int q = lane % KL, c0 = blockIdx.x * COLS + (warp * (32 / KL) + lane / KL) * CT;
   float* state = L.ssm_state + ((size_t)b.seq_slot[seq] * L.heads + h) * D * D;
   const bool fresh = b.seq_pos0[seq] == 0;
-  float2 S[CT][2 * QUADS];                           // two neighbouring keys of a column
-  auto key = [&](int i) { return 4 * (q + KL * (i / 2)) + 2 * (i & 1); };
+  float2 S[CT][4];                                   // two neighbouring keys of a column
+  auto key = [&](int i) { return (i / 2) * (DP / 2) + 4 * q + 2 * (i & 1); };
 #pragma unroll
-  for (int i = 0; i < 2 * QUADS; ++i)
+  for (int i = 0; i < 4; ++i)
 #pragma unroll
     for (int c = 0; c < CT; ++c) {
       const int k = key(i), col = c0 + c;
       S[c][i].x = !fresh && k < D && col < D ? state[(size_t)k * D + col] : 0.f;
       S[c][i].y = !fresh && k + 1 < D && col < D ? state[(size_t)(k + 1) * D + col] : 0.f;
     }
-  const int cv = min(c0, DP - CT), tok = q & (DG - 1);   // lane q finishes the output of token q of a group
-  T* yc = y + (size_t)(r0 + tok) * ldy + h * L.pp + c0;
-  const bool writes = q < DG && c0 < L.pp;           // (pp is even: both columns or none)
+  const int cv = min(c0, DP - CT), col = q & 3, tok = (q >> 2) * NT;   // this lane's column and first output token
+  const bool b1 = q & 2, b0 = q & 1;
+  T* yt = y + (size_t)(r0 + tok) * ldy + h * L.pp + c0 + col;   // first output of this lane in the group at hand
+  const bool writes = c0 < L.pp;                     // (pp is a multiple of 4: all four columns or none)
   __syncthreads();
   for (int t0 = 0, it = 0; t0 < n; t0 += STEP, ++it) {
-    const float* p = sm + (it & 1) * DT_GROUPS * G::SIZE;
+    const float* p = sm + (it & 1) * PREP * G::SIZE;
     for (int t = t0; t < min(t0 + STEP, n); t += DG, p += G::SIZE) {
-      float2 pu[DG][CT], pr[DG][CT];
+      auto vec = [&](int off, int m) { return reinterpret_cast<const float4*>(p + off + m * (DP / 2))[q]; };
+      auto dots = [&](int off, float (&out)[CT]) {
+        float2 acc[CT];
 #pragma unroll
-      for (int i = 0; i < DG; ++i)
-#pragma unroll
-        for (int c = 0; c < CT; ++c) pu[i][c] = pr[i][c] = make_float2(0.f, 0.f);
-#pragma unroll
-      for (int m = 0; m < QUADS; ++m)
-#pragma unroll
-        for (int i = 0; i < DG; ++i) {
-          const float4 u = reinterpret_cast<const float4*>(p + G::U + i * DP)[q + KL * m];
-          const float4 r = reinterpret_cast<const float4*>(p + G::R + i * DP)[q + KL * m];
+        for (int m = 0; m < 2; ++m) {
+          const float4 u = vec(off, m);
 #pragma unroll
           for (int c = 0; c < CT; ++c) {
-            pu[i][c] = fma2(make_float2(u.x, u.y), S[c][2 * m], pu[i][c]);
-            pr[i][c] = fma2(make_float2(r.x, r.y), S[c][2 * m], pr[i][c]);
-            pu[i][c] = fma2(make_float2(u.z, u.w), S[c][2 * m + 1], pu[i][c]);
-            pr[i][c] = fma2(make_float2(r.z, r.w), S[c][2 * m + 1], pr[i][c]);
+            acc[c] = m ? fma2(make_float2(u.x, u.y), S[c][2], acc[c]) : mul2(make_float2(u.x, u.y), S[c][0]);
+            acc[c] = fma2(make_float2(u.z, u.w), S[c][2 * m + 1], acc[c]);
           }
         }
-      float x[DG][CT], os[DG][CT];
 #pragma unroll
-      for (int i = 0; i < DG; ++i)
+        for (int c = 0; c < CT; ++c) out[c] = acc[c].x + acc[c].y;
+      };
+      // in phases, so that the latency of one token's shuffles and loads covers the others'
+      float x[DG], o[DG], v[DG];                     // of this lane's column
+      float f[DG][CT], g[DG][CT];
 #pragma unroll
-        for (int c = 0; c < CT; ++c) {
-          x[i][c] = pu[i][c].x + pu[i][c].y;
-          os[i][c] = pr[i][c].x + pr[i][c].y;
-        }
+      for (int i = 0; i < DG; ++i) dots(G::U + i * DP, f[i]);
 #pragma unroll
-      for (int o = 1; o < KL; o <<= 1)
+      for (int i = 0; i < DG; ++i) {
+        f[i][0] = (b1 ? f[i][2] : f[i][0]) + __shfl_xor_sync(0xffffffffu, b1 ? f[i][0] : f[i][2], 2);
+        f[i][1] = (b1 ? f[i][3] : f[i][1]) + __shfl_xor_sync(0xffffffffu, b1 ? f[i][1] : f[i][3], 2);
+      }
 #pragma unroll
-        for (int i = 0; i < DG; ++i)
+      for (int i = 0; i < DG; ++i) dots(G::R + i * DP, g[i]);
 #pragma unroll
-          for (int c = 0; c < CT; ++c) x[i][c] += __shfl_xor_sync(0xffffffffu, x[i][c], o);
-      float2 v[DG];
+      for (int i = 0; i < DG; ++i) x[i] = (b0 ? f[i][1] : f[i][0]) + __shfl_xor_sync(0xffffffffu, b0 ? f[i][0] : f[i][1], 1);
 #pragma unroll
-      for (int i = 0; i < DG; ++i) v[i] = *reinterpret_cast<const float2*>(p + G::V + i * DP + cv);
+      for (int i = 0; i < DG; ++i) v[i] = p[G::V + i * DP + cv + col];
+      float ca[DG][DG], cw[DG][DG];
 #pragma unroll
       for (int i = 1; i < DG; ++i) {
         const float4 ra = *reinterpret_cast<const float4*>(p + G::X + i * 4), rv = *reinterpret_cast<const float4*>(p + G::X + 16 + i * 4);
-        const float ca[4] = {ra.x, ra.y, ra.z, ra.w}, cw[4] = {rv.x, rv.y, rv.z, rv.w};
-#pragma unroll
-        for (int j = 0; j < i; ++j) {
-          x[i][0] = fmaf(cw[j], v[j].x, fmaf(-ca[j], x[j][0], x[i][0]));
-          x[i][1] = fmaf(cw[j], v[j].y, fmaf(-ca[j], x[j][1], x[i][1]));
-        }
+        ca[i][0] = ra.x; ca[i][1] = ra.y; ca[i][2] = ra.z; ca[i][3] = ra.w;
+        cw[i][0] = rv.x; cw[i][1] = rv.y; cw[i][2] = rv.z; cw[i][3] = rv.w;
       }
-      // the state first: the next group waits for it
 #pragma unroll
-      for (int m = 0; m < QUADS; ++m) {
-        const float4 w = reinterpret_cast<const float4*>(p + G::W)[q + KL * m];
+      for (int d = 4; d < KL; d <<= 1)
+#pragma unroll
+        for (int i = 0; i < DG; ++i) x[i] += __shfl_xor_sync(0xffffffffu, x[i], d);
+#pragma unroll
+      for (int i = 0; i < DG; ++i) {
+        g[i][0] = (b1 ? g[i][2] : g[i][0]) + __shfl_xor_sync(0xffffffffu, b1 ? g[i][0] : g[i][2], 2);
+        g[i][1] = (b1 ? g[i][3] : g[i][1]) + __shfl_xor_sync(0xffffffffu, b1 ? g[i][1] : g[i][3], 2);
+      }
+#pragma unroll
+      for (int m = 0; m < 2; ++m) {
+        const float4 w = vec(G::W, m);
 #pragma unroll
         for (int c = 0; c < CT; ++c) {
           S[c][2 * m] = mul2(make_float2(w.x, w.y), S[c][2 * m]);
           S[c][2 * m + 1] = mul2(make_float2(w.z, w.w), S[c][2 * m + 1]);
         }
+      }
 #pragma unroll
-        for (int j = 0; j < DG; ++j) {
-          const float4 k = reinterpret_cast<const float4*>(p + G::K + j * DP)[q + KL * m];
-          const float4 a = reinterpret_cast<const float4*>(p + G::A + j * DP)[q + KL * m];
+      for (int i = 0; i < DG; ++i) o[i] = (b0 ? g[i][1] : g[i][0]) + __shfl_xor_sync(0xffffffffu, b0 ? g[i][0] : g[i][1], 1);
+      // ... NT tokens to a lane
+#pragma unroll
+      for (int d = KL / 2, c = DG / 2; d >= 4; d >>= 1, c >>= 1) {
+        const bool up = q & d;
+#pragma unroll
+        for (int i = 0; i < DG / 2; ++i)
+          if (i < c) {
+            const float keep = up ? o[i + c] : o[i], send = up ? o[i] : o[i + c];
+            o[i] = keep + __shfl_xor_sync(0xffffffffu, send, d);
+          }
+      }
+      float4 ga[NT];
+#pragma unroll
+      for (int i = 0; i < NT; ++i) {
+        ga[i] = *reinterpret_cast<const float4*>(p + G::X + 32 + (tok + i) * 4);
+        const float4 gv = *reinterpret_cast<const float4*>(p + G::X + 48 + (tok + i) * 4);
+        o[i] = (o[i] + fmaf(gv.y, v[1], gv.x * v[0])) + fmaf(gv.w, v[3], gv.z * v[2]);
+      }
+      // the part of the update and of x that the values alone make
+#pragma unroll
+      for (int j = 0; j < DG; ++j) {
+        const float4 v4 = *reinterpret_cast<const float4*>(p + G::V + j * DP + cv);
+        const float vc[CT] = {v4.x, v4.y, v4.z, v4.w};
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+          const float4 k = vec(G::K + j * DP, m);
 #pragma unroll
           for (int c = 0; c < CT; ++c) {
-            const float vc = c ? v[j].y : v[j].x, xc = -x[j][c];
-            S[c][2 * m] = fma2(make_float2(k.x, k.y), make_float2(vc, vc), S[c][2 * m]);
-            S[c][2 * m + 1] = fma2(make_float2(k.z, k.w), make_float2(vc, vc), S[c][2 * m + 1]);
-            S[c][2 * m] = fma2(make_float2(a.x, a.y), make_float2(xc, xc), S[c][2 * m]);
-            S[c][2 * m + 1] = fma2(make_float2(a.z, a.w), make_float2(xc, xc), S[c][2 * m + 1]);
+            const float2 vv = make_float2(vc[c], vc[c]);
+            S[c][2 * m] = fma2(make_float2(k.x, k.y), vv, S[c][2 * m]);
+            S[c][2 * m + 1] = fma2(make_float2(k.z, k.w), vv, S[c][2 * m + 1]);
           }
         }
       }
-      // outputs: sums of the four tokens, one token to a lane
-      const bool b1 = q & 2, b0 = q & 1;
 #pragma unroll
-      for (int c = 0; c < CT; ++c) {
-        const float k0 = b1 ? os[2][c] : os[0][c], k1 = b1 ? os[3][c] : os[1][c];
-        const float s0 = b1 ? os[0][c] : os[2][c], s1 = b1 ? os[1][c] : os[3][c];
-        const float e0 = k0 + __shfl_xor_sync(0xffffffffu, s0, 2), e1 = k1 + __shfl_xor_sync(0xffffffffu, s1, 2);
-        os[0][c] = (b0 ? e1 : e0) + __shfl_xor_sync(0xffffffffu, b0 ? e0 : e1, 1);
-        if (KL == 8) os[0][c] += __shfl_xor_sync(0xffffffffu, os[0][c], 4);
-      }
-      const float4 ga = *reinterpret_cast<const float4*>(p + G::X + 32 + tok * 4), gv = *reinterpret_cast<const float4*>(p + G::X + 48 + tok * 4);
-      const float ca[4] = {ga.x, ga.y, ga.z, ga.w}, cw[4] = {gv.x, gv.y, gv.z, gv.w};
+      for (int i = 1; i < DG; ++i)
+#pragma unroll
+        for (int j = 0; j < i; ++j) x[i] = fmaf(cw[i][j], v[j], x[i]);
+#pragma unroll
+      for (int i = 1; i < DG; ++i)
+#pragma unroll
+        for (int j = 0; j < i; ++j) x[i] = fmaf(-ca[i][j], x[j], x[i]);
+      // every lane gets the x of its four columns, and the state moves on
+      float lo[DG], hi[DG], xc[DG][CT];
 #pragma unroll
       for (int j = 0; j < DG; ++j) {
-        os[0][0] = fmaf(cw[j], v[j].x, fmaf(-ca[j], x[j][0], os[0][0]));
-        os[0][1] = fmaf(cw[j], v[j].y, fmaf(-ca[j], x[j][1], os[0][1]));
+        const float n1 = __shfl_xor_sync(0xffffffffu, x[j], 1);
+        lo[j] = b0 ? n1 : x[j];
+        hi[j] = b0 ? x[j] : n1;
       }
-      if (writes && t + tok < n) {
-        struct alignas(sizeof(T) * 2) Two {
-          T v[2];
-        } o;
-        o.v[0] = from_f<T>(os[0][0]);
-        o.v[1] = from_f<T>(os[0][1]);
-        *reinterpret_cast<Two*>(yc + (size_t)t * ldy) = o;
+#pragma unroll
+      for (int j = 0; j < DG; ++j) {
+        const float lo2 = __shfl_xor_sync(0xffffffffu, lo[j], 2), hi2 = __shfl_xor_sync(0xffffffffu, hi[j], 2);
+        xc[j][0] = b1 ? lo2 : lo[j];
+        xc[j][1] = b1 ? hi2 : hi[j];
+        xc[j][2] = b1 ? lo[j] : lo2;
+        xc[j][3] = b1 ? hi[j] : hi2;
       }
+      // outputs, while the shuffles are on their way
+#pragma unroll
+      for (int i = 0; i < NT; ++i) {
+        const float f = fmaf(-ga[i].y, x[1], fmaf(-ga[i].x, x[0], o[i])) - fmaf(ga[i].w, x[3], ga[i].z * x[2]);
+        if (writes && t + tok + i < n) yt[i * ldy] = from_f<T>(f);
+      }
+      yt += DG * (size_t)ldy;
+#pragma unroll
+      for (int j = 0; j < DG; ++j)
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+          const float4 a = vec(G::A + j * DP, m);
+#pragma unroll
+          for (int c = 0; c < CT; ++c) {
+            const float2 xx = make_float2(-xc[j][c], -xc[j][c]);
+            S[c][2 * m] = fma2(make_float2(a.x, a.y), xx, S[c][2 * m]);
+            S[c][2 * m + 1] = fma2(make_float2(a.z, a.w), xx, S[c][2 * m + 1]);
+          }
+        }
     }
     __syncthreads();
   }
 #pragma unroll
-  for (int i = 0; i < 2 * QUADS; ++i)
+  for (int i = 0; i < 4; ++i)
 #pragma unroll
     for (int c = 0; c < CT; ++c) {
-      const int k = key(i), col = c0 + c;
-      if (k < D && col < D) state[(size_t)k * D + col] = S[c][i].x;
-      if (k + 1 < D && col < D) state[(size_t)(k + 1) * D + col] = S[c][i].y;
+      const int k = key(i), cl = c0 + c;
+      if (k < D && cl < D) state[(size_t)k * D + cl] = S[c][i].x;
+      if (k + 1 < D && cl < D) state[(size_t)(k + 1) * D + cl] = S[c][i].y;
     }
 }
 
@@ -616,25 +662,29 @@ static int launch_scan_any(const BbHyLayer& L, const BbHyWork& w, const BbHyBatc
   return (int)cudaGetLastError();
 }
 
-template <int DP, int CW>
+template <int DP, int CW, int PREP, int BLOCKS>
 static int launch_scan_regs(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, cudaStream_t s) {
   using T = __nv_bfloat16;
   static PerDeviceOnce once;
-  constexpr int smem = 2 * DT_GROUPS * DeltaGroup<DP>::SIZE * 4, cols = CW * (32 / (DP > 64 ? 8 : 4)) * 2;
-  const cudaError_t e = ensure_dyn_smem(once, hy_delta_scan_kernel<T, DP, CW>, smem);
+  constexpr int smem = 2 * PREP * DeltaGroup<DP>::SIZE * 4, cols = CW * (32 / (DP / 8)) * 4;
+  const cudaError_t e = ensure_dyn_smem(once, hy_delta_scan_kernel<T, DP, CW, PREP, BLOCKS>, smem);
   if (e != cudaSuccess) return (int)e;
-  hy_delta_scan_kernel<T, DP, CW><<<dim3((L.p + cols - 1) / cols, L.heads, b.ns_pre), (CW + DT_PREP) * 32, smem, s>>>(
+  hy_delta_scan_kernel<T, DP, CW, PREP, BLOCKS><<<dim3((L.p + cols - 1) / cols, L.heads, b.ns_pre), (CW + PREP) * 32, smem, s>>>(
       L, static_cast<const T*>(w.proj), w.ld_proj, static_cast<const T*>(w.aux), w.ld_aux, static_cast<T*>(w.y), w.ld_y, b);
   return (int)cudaGetLastError();
 }
 
-// Few heads: the columns of a head are spread over more blocks.
+// Few heads: the columns of a head are spread over more blocks.  Many: two blocks share an SM.
 static int launch_scan_bf16(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, cudaStream_t s) {
   const long pairs = (long)b.ns_pre * L.heads;
   const int sms = sm_count();
-  if (L.p <= 32) return launch_scan_regs<32, 2>(L, w, b, s);
-  if (L.p <= 64) return pairs * 4 <= sms ? launch_scan_regs<64, 1>(L, w, b, s) : (pairs * 2 <= sms ? launch_scan_regs<64, 2>(L, w, b, s) : launch_scan_regs<64, 4>(L, w, b, s));
-  if (L.p <= 128) return pairs * 8 <= sms ? launch_scan_regs<128, 2>(L, w, b, s) : launch_scan_regs<128, 4>(L, w, b, s);
+  if (L.p <= 32) return launch_scan_regs<32, 1, 8, 2>(L, w, b, s);
+  if (L.p <= 64) {
+    if (pairs * 4 <= sms) return launch_scan_regs<64, 1, 8, 1>(L, w, b, s);
+    if (pairs * 2 <= sms) return launch_scan_regs<64, 2, 8, 1>(L, w, b, s);
+    return pairs <= sms ? launch_scan_regs<64, 4, 8, 1>(L, w, b, s) : launch_scan_regs<64, 4, 6, 2>(L, w, b, s);
+  }
+  if (L.p <= 128) return pairs * 8 <= sms ? launch_scan_regs<128, 2, 8, 1>(L, w, b, s) : launch_scan_regs<128, 4, 8, 1>(L, w, b, s);
   return BB_ESIZE;
 }
 

@@ -40,7 +40,7 @@ __device__ __forceinline__ void store_pair(T* p, float a, float b) {
 template <typename T>
 __device__ __forceinline__ float gelu_as(float z) {
   const float t = 0.79788456080286536f * fmaf(0.044715f * z * z, z, z);   // sqrt(2 / pi) (z + 0.044715 z^3)
-  if constexpr (sizeof(T) == 2) return z * __fdividef(1.f, 1.f + __expf(-2.f * t));
+  if constexpr (sizeof(T) == 2) return z * rcp_hw(1.f + exp2_hw(-2.f * kLog2e * t));
   else return 0.5f * z * (1.f + tanhf(t));
 }
 // e^-x - 1 for x >= 0
@@ -48,14 +48,14 @@ template <typename T>
 __device__ __forceinline__ float decay_m1(float x) {
   if constexpr (sizeof(T) == 2) {
     // the series where the difference would cancel
-    return x < 0.05f ? -x * fmaf(x, fmaf(x, fmaf(x, -1.f / 24.f, 1.f / 6.f), -0.5f), 1.f) : __expf(-x) - 1.f;
+    return x < 0.05f ? -x * fmaf(x, fmaf(x, fmaf(x, -1.f / 24.f, 1.f / 6.f), -0.5f), 1.f) : exp_hw(-x) - 1.f;
   } else {
     return expm1f(-x);
   }
 }
 template <typename T>
 __device__ __forceinline__ float root_of(float x) {
-  if constexpr (sizeof(T) == 2) return x * rsqrtf(fmaxf(x, 1e-37f));
+  if constexpr (sizeof(T) == 2) return x * rsqrt_hw(fmaxf(x, 1e-37f));
   else return sqrtf(x);
 }
 // S after a token of (e, in); product of two decays
