@@ -6,6 +6,8 @@
 // One CTA per (range of keys, sequence, 256 latent columns x 128 heads); warp 0 feeds a ring of 64-key tiles,
 // page by page through the block table, warp 1 issues the MMAs, warps 2..5 do the softmax of one head per
 // thread.  Two score buffers keep the tensor pipe a tile ahead.  Key ranges are merged by a second kernel.
+// The query tile holds the rows that are heads and no more: the MMA's further rows read whatever lies behind
+// them in shared memory, and their results are never looked at.
 #include "../common/host.hpp"
 #include "../common/ptx.cuh"
 #include "../common/rows.cuh"
@@ -13,13 +15,13 @@
 
 namespace bb {
 
-constexpr int LD_KEYS = 64, LD_SUB = LD_KEYS * 128, LD_QSUB = 128 * 128, LD_COLS = 256, LD_MAX_STAGES = 4;
+constexpr int LD_KEYS = 64, LD_SUB = LD_KEYS * 128, LD_ROWS = 128, LD_COLS = 256, LD_MAX_STAGES = 4;
 constexpr int LD_SMEM_MAX = 226 * 1024, LD_BARS = 256;
 
 struct LatDecArgs {
   const int *pos, *tables;     // [rows], [rows][max_blocks]
   int max_blocks, bs, window;
-  int hq, width, kvrp, nsub, stages, vchunks, splits, tmem_cols;
+  int hq, q_rows, width, kvrp, nsub, stages, vchunks, splits, tmem_cols;   // q_rows: rows of the query tile
   float scale_log2;
   __nv_bfloat16* out;          // [rows, ldo], head h at h kvrp (one key range)
   int ldo;
@@ -32,9 +34,9 @@ hy_latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
                         const __grid_constant__ LatDecArgs a) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  const int tile_bytes = a.nsub * LD_SUB;
+  const int tile_bytes = a.nsub * LD_SUB, q_sub = a.q_rows * 128;
   uint8_t* sQ = smem;
-  uint8_t* sP = smem + a.nsub * LD_QSUB;
+  uint8_t* sP = smem + a.nsub * q_sub;
   uint64_t* bars = reinterpret_cast<uint64_t*>(sP + a.stages * tile_bytes);
   uint64_t* q_full = bars;
   uint64_t* k_full = bars + 1;                       // [stages]
@@ -76,8 +78,8 @@ hy_latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
 
   if (warp == 0) {
     if (lane == 0 && n_units > 0) {
-      mbar_expect_tx(q_full, a.nsub * LD_QSUB);
-      for (int c = 0; c < a.nsub; ++c) tma_load_3d(sQ + c * LD_QSUB, &tmQ, q_full, c * 64, h0, row);
+      mbar_expect_tx(q_full, a.nsub * q_sub);
+      for (int c = 0; c < a.nsub; ++c) tma_load_3d(sQ + c * q_sub, &tmQ, q_full, c * 64, h0, row);
       const int* tab = a.tables + (size_t)row * a.max_blocks;
       for (int u = 0; u < n_units; ++u) {
         const int st = u % a.stages;
@@ -105,13 +107,14 @@ hy_latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         if (!mbar_wait(k_full + st, (u / a.stages) & 1)) return false;
         tc_fence_after();
         for (int t = 0; t < ksteps; ++t)
-          umma_f16_ss(tmem + (u & 1) * 64, umma_smem_desc(aq + (t / 4) * LD_QSUB + (t % 4) * 32, 16, 1024),
+          umma_f16_ss(tmem + (u & 1) * 64, umma_smem_desc(aq + (t / 4) * q_sub + (t % 4) * 32, 16, 1024),
                       umma_smem_desc(bp + st * tile_bytes + (t / 4) * LD_SUB + (t % 4) * 32, 16, 1024), idesc_s, t != 0);
         umma_commit(s_full + (u & 1));
         return true;
       };
-      // with one stage a tile is finished before the next one arrives
-      const int ahead = a.stages > 1 ? 2 : 1;
+      // scores run two tiles ahead where the ring holds a third tile; with two stages, one, so that finishing a
+      // tile never waits for the load into the stage it frees
+      const int ahead = a.stages > 2 ? 2 : 1;
       for (int u = 0; u < ahead && u < n_units && ok; ++u) ok = issue_s(u);
       if (!ok) set_error(a.err, ERR_WAIT_MMA_FULL);
       for (int u = 0; u < n_units && ok; ++u) {
@@ -153,9 +156,10 @@ hy_latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       const int kv0 = (t0 + u) * LD_KEYS, lim = last - kv0, low = first - kv0;
       const bool need_mask = lim < LD_KEYS - 1 || low > 0;     // the same for every head
       const float sc = a.scale_log2;
-      if (need_mask) {
+      if (need_mask || h >= a.hq) {
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
+          if (h >= a.hq) r0[i] = r1[i] = 0u;         // not a head
           if (i > lim || i < low) r0[i] = 0xff800000u;
           if (i + 32 > lim || i + 32 < low) r1[i] = 0xff800000u;
         }
@@ -292,7 +296,8 @@ BB_API int bb_hy_latent_decode(const BbHyCfg* c, const BbHyLayer* L, const BbHyW
   a.nsub = (a.width + 63) / 64;
   a.bs = c->block_size;
   if (c->dtype || a.nsub > 9 || (a.bs != 16 && a.bs != 32 && a.bs != 64)) return BB_ESIZE;
-  const int q_bytes = a.nsub * LD_QSUB, tile = a.nsub * LD_SUB;
+  a.q_rows = L->hq >= LD_ROWS ? LD_ROWS : (L->hq + 7) & ~7;
+  const int q_bytes = a.nsub * a.q_rows * 128, tile = a.nsub * LD_SUB;
   a.stages = (LD_SMEM_MAX - 1024 - LD_BARS - q_bytes) / tile;
   if (a.stages < 1) return BB_ESIZE;
   if (a.stages > LD_MAX_STAGES) a.stages = LD_MAX_STAGES;
@@ -319,7 +324,7 @@ BB_API int bb_hy_latent_decode(const BbHyCfg* c, const BbHyLayer* L, const BbHyW
   CUtensorMap tq, tp;
   const CUtensorMapDataType bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   const __nv_bfloat16* qa = static_cast<const __nv_bfloat16*>(w->qa) + (size_t)qa_row0 * w->ld_qa;
-  int rc = make_tmap_3d(&tq, bf, 2, qa, a.width, L->hq, rows, (uint64_t)a.width * 2, (uint64_t)w->ld_qa * 2, 64, 128);
+  int rc = make_tmap_3d(&tq, bf, 2, qa, a.width, L->hq, rows, (uint64_t)a.width * 2, (uint64_t)w->ld_qa * 2, 64, a.q_rows);
   if (rc) return rc;
   rc = make_tmap_2d(&tp, bf, 2, L->kc, a.width, (uint64_t)w->pool_blocks * a.bs, (uint64_t)a.width * 2, 64, a.bs);
   if (rc) return rc;
@@ -327,8 +332,11 @@ BB_API int bb_hy_latent_decode(const BbHyCfg* c, const BbHyLayer* L, const BbHyW
   const cudaError_t e = ensure_dyn_smem(once, hy_latent_decode_kernel, LD_SMEM_MAX);
   if (e != cudaSuccess) return (int)e;
   cudaStream_t s = (cudaStream_t)stream;
+  // the MMA reads 128 rows of every query sub-tile
+  const int q_read = (a.nsub - 1) * a.q_rows * 128 + LD_ROWS * 128, ring = q_bytes + a.stages * tile + LD_BARS;
+  const int smem = (ring > q_read ? ring : q_read) + 1024;
   hy_latent_decode_kernel<<<dim3(a.splits, rows, a.vchunks * ((L->hq + 127) / 128)), 192,
-                            q_bytes + a.stages * tile + 1024 + LD_BARS, s>>>(tq, tp, a);
+                            smem, s>>>(tq, tp, a);
   if (a.splits > 1) {
     const long t = (long)rows * L->hq * (L->kvrp / 8);
     hy_latent_merge_kernel<<<(int)((t + 127) / 128), 128, 0, s>>>(w->part_o, w->part_ml, a.out, w->ld_ol, rows, L->hq,

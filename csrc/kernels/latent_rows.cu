@@ -46,16 +46,16 @@ __device__ __forceinline__ void rotate_pairs8(float (&f)[8], const Angles4& a) {
 
 // A thread's vectors of the row (query latent, then page row) stay in registers up to KEEP of them.
 template <typename T>
-__global__ void __launch_bounds__(LAT_THREADS)
+__global__ void __launch_bounds__(LAT_THREADS, sizeof(T) == 2 ? 10 : 6)
 hy_latent_in_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, int ld, const int* __restrict__ pos_,
                     const int* __restrict__ row_seq, const int* __restrict__ tables, int max_blocks, int bs, float eps) {
-  constexpr int KEEP = 3;
+  constexpr int KEEP = 2;
   __shared__ float buf[2][32];
   const int r = blockIdx.x, width = L.kvrp + L.rotp, n = L.qrp + (L.own_kv ? width : 0);
   T* q = proj + (size_t)r * ld + L.off_dq;
   const T* c = proj + (size_t)r * ld + L.off_ckv;
   const int pos = pos_[r];
-  float v[KEEP][8], sq = 0.f, sc = 0.f;
+  float v[KEEP][8], gain[8], sq = 0.f, sc = 0.f;
   auto sum = [&](int i, const float (&f)[8]) {
     float t = 0.f;
 #pragma unroll
@@ -68,6 +68,9 @@ hy_latent_in_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, i
     const int i = (threadIdx.x + t * LAT_THREADS) * 8;
     if (i < n) load8(i < L.qrp ? q + i : c + (i - L.qrp), v[t]);
   }
+  // the first vector's gains are asked for before the sums are known
+  auto gains = [&](int i) { return i < L.qrp ? L.dq_norm + i : L.dkv_norm + (i - L.qrp); };
+  if (threadIdx.x * 8 < min(n, L.qrp + L.kvrp)) load8(gains(threadIdx.x * 8), gain);
 #pragma unroll
   for (int t = 0; t < KEEP; ++t) {
     const int i = (threadIdx.x + t * LAT_THREADS) * 8;
@@ -94,10 +97,17 @@ hy_latent_in_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, i
   }
   const float rq = 1.f / sqrtf(sq / (float)L.qr + eps), rc = 1.f / sqrtf(sc / (float)L.kvr + eps);
   T* page = static_cast<T*>(L.kc) + ((size_t)blk * bs + pos % bs) * width;
-  auto emit = [&](int i, float (&f)[8]) {
+  auto emit = [&](int i, float (&f)[8], bool first) {
     float g[8];
+    if (i < L.qrp + L.kvrp) {
+      if (first) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) g[j] = gain[j];
+      } else {
+        load8(gains(i), g);
+      }
+    }
     if (i < L.qrp) {
-      load8(L.dq_norm + i, g);
 #pragma unroll
       for (int j = 0; j < 8; ++j) f[j] *= rq * g[j];
       store8(q + i, f);
@@ -105,7 +115,6 @@ hy_latent_in_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, i
     }
     i -= L.qrp;
     if (i < L.kvrp) {
-      load8(L.dkv_norm + i, g);
 #pragma unroll
       for (int j = 0; j < 8; ++j) f[j] *= rc * g[j];
     } else {
@@ -117,12 +126,12 @@ hy_latent_in_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, i
 #pragma unroll
   for (int t = 0; t < KEEP; ++t) {
     const int i = (threadIdx.x + t * LAT_THREADS) * 8;
-    if (i < n) emit(i, v[t]);
+    if (i < n) emit(i, v[t], t == 0);
   }
   for (int i = (threadIdx.x + KEEP * LAT_THREADS) * 8; i < n; i += LAT_THREADS * 8) {
     float f[8];
     load8(i < L.qrp ? q + i : c + (i - L.qrp), f);
-    emit(i, f);
+    emit(i, f, false);
   }
 }
 
