@@ -143,7 +143,7 @@ template <typename T>
 __global__ void __launch_bounds__(LAT_THREADS)
 hy_latent_q_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ q, int ldq, T* __restrict__ qa, int ldqa,
                    const int* __restrict__ pos_, int n_in, int step) {
-  const unsigned vecs = L.rotp / 8, t = blockIdx.y * LAT_THREADS + threadIdx.x;
+  const unsigned vecs = L.rotp / 8, t = blockIdx.y * blockDim.x + threadIdx.x;
   const int h0 = t / vecs, d = (t - h0 * vecs) * 8, r = blockIdx.x;
   if (h0 >= step) return;
   const int pos = pos_[r];
@@ -258,14 +258,14 @@ BB_API int bb_hy_latent_in(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork*
 BB_API int bb_hy_latent_q(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int n_in, void* stream) {
   cudaStream_t s = (cudaStream_t)stream;
   const int step = (L->hq + LQ_HEADS - 1) / LQ_HEADS;
-  const dim3 grid(b->n, (step * (L->rotp / 8) + LAT_THREADS - 1) / LAT_THREADS);
+  const int lanes = step * (L->rotp / 8), t = lanes < LAT_THREADS ? (lanes + 31) & ~31 : LAT_THREADS;
+  const dim3 grid(b->n, (lanes + t - 1) / t);
   if (c->dtype)
-    hy_latent_q_kernel<float><<<grid, LAT_THREADS, 0, s>>>(*L, static_cast<float*>(w->q), w->ld_q, static_cast<float*>(w->qa),
-                                                           w->ld_qa, b->pos, n_in, step);
+    hy_latent_q_kernel<float><<<grid, t, 0, s>>>(*L, static_cast<float*>(w->q), w->ld_q, static_cast<float*>(w->qa), w->ld_qa,
+                                                 b->pos, n_in, step);
   else
-    hy_latent_q_kernel<__nv_bfloat16><<<grid, LAT_THREADS, 0, s>>>(*L, static_cast<__nv_bfloat16*>(w->q), w->ld_q,
-                                                                   static_cast<__nv_bfloat16*>(w->qa), w->ld_qa, b->pos, n_in,
-                                                                   step);
+    hy_latent_q_kernel<__nv_bfloat16><<<grid, t, 0, s>>>(*L, static_cast<__nv_bfloat16*>(w->q), w->ld_q,
+                                                         static_cast<__nv_bfloat16*>(w->qa), w->ld_qa, b->pos, n_in, step);
   return (int)cudaGetLastError();
 }
 

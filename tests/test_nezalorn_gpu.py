@@ -35,7 +35,7 @@ MECHANISMS = {
     "latent_huge_rank": [(latent(heads=2, dim=32, rot=32, vdim=32, kv_rank=700), None)],
     "delta": [(delta(), None)],
     "delta_small": [(delta(heads=5, dim=8, rank=1), None)],
-    "delta_32": [(delta(heads=2, dim=32, rank=16), poly())],
+    "delta_32": [(delta(heads=3, dim=32, rank=12), poly())],
     "delta_64": [(delta(heads=2, dim=64), None)],
     "delta_odd": [(delta(heads=2, dim=37, rank=3), poly(33))],
     "delta_128": [(delta(heads=1, dim=128, rank=32), None)],
