@@ -31,6 +31,8 @@ _ARCHS: List[Arch] = [
          ("import", "infer", "serve", "trace"), aliases=("hybrid",)),
     Arch("nezalorn", "hybrid", "Hybrid decoder: windowed latent attention, generalised delta rule and gated linear "
          "recurrence layers, depth averages", ("import", "infer", "serve", "trace")),
+    Arch("zepesun", "hybrid", "Hybrid decoder: latent attention, matrix memories and windowed attention beside them, "
+         "mixture of experts", ("import", "infer", "serve", "trace")),
     Arch("splat", "splat", "3D Gaussian splat rasteriser (headless)", ("render", "train"), built=True),
 ]
 

@@ -354,19 +354,29 @@ class AttentionSpec:
     softcap: Optional[float] = None
     rot: Optional[RotarySpec] = None
     v_mix: bool = False          # values mixed with those of the first layer that has this set
+    window: Optional[int] = None     # keys a query sees, itself included (None: every earlier one)
+    qk_norm: bool = True         # root-mean-square norm over the whole query and the whole key projection
+    bias: bool = False           # on the query, key, value and output projections
+    gate: str = "head"           # sigmoid gate on the output: one value per head, or one per element
     kind = "attention"
+    recurrent = False
 
     @staticmethod
-    def from_json(m: dict) -> "AttentionSpec":
-        rot = m.get("rot")
+    def from_json(m: dict, **constants) -> "AttentionSpec":
+        rot, mask = m.get("rot"), m.get("mask") or {}
         return AttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
                              scale=float(m["scale"]), softcap=float(m["softcap"]) if m.get("softcap") else None,
-                             rot=RotarySpec.from_json(rot) if rot else None, v_mix=bool(m.get("v_mix", False)))
+                             rot=RotarySpec.from_json(rot) if rot else None, v_mix=bool(m.get("v_mix", False)),
+                             window=int(mask["size"]) if mask.get("size") else None, **constants)
 
     def to_json(self) -> dict:
-        m = {k: v for k, v in asdict(self).items() if v is not None}
+        m = {k: v for k, v in asdict(self).items() if v is not None and k not in ("window", "qk_norm", "bias", "gate")}
         if self.rot is not None:
             m["rot"] = {"dims": self.rot.dims, "base": self.rot.base}
+        if self.window is not None:
+            m["mask"] = {"size": self.window}
+        if not self.qk_norm:
+            del m["v_mix"]
         return m
 
     def check(self):
@@ -374,14 +384,26 @@ class AttentionSpec:
             raise ValueError(f"attention: {self.heads} heads over {self.kv_heads} key/value heads")
         if self.rot is not None and (self.rot.dims % 2 or self.rot.dims > self.dim):
             raise ValueError(f"attention: cannot rotate {self.rot.dims} of {self.dim} dimensions")
+        if self.window is not None and self.window < 1:
+            raise ValueError("attention: the window holds at least the token itself")
+        if not self.qk_norm and (self.rot is not None or self.v_mix):
+            raise ValueError("attention: rotation and value mixing come with normed queries and keys")
 
     def tensors(self, width: int):
-        out = [("q", (self.heads * self.dim, width)), ("k", (self.kv_heads * self.dim, width)),
-               ("v", (self.kv_heads * self.vdim, width)), ("q.norm", (self.heads * self.dim,)),
-               ("k.norm", (self.kv_heads * self.dim,))]
+        out = []
+        for n, rows in (("q", self.heads * self.dim), ("k", self.kv_heads * self.dim), ("v", self.kv_heads * self.vdim)):
+            out.append((n, (rows, width)))
+            if self.bias:
+                out.append((n + ".b", (rows,)))
+        if self.qk_norm:
+            out += [("q.norm", (self.heads * self.dim,)), ("k.norm", (self.kv_heads * self.dim,))]
         if self.v_mix:
             out.append(("vmix", ()))
-        return out + [("g", (self.heads, width)), ("o", (width, self.heads * self.vdim))]
+        out += [("g", (self.heads * (self.vdim if self.gate == "element" else 1), width)), ("o", (width, self.heads * self.vdim))]
+        return out + [("o.b", (width,))] if self.bias else out
+
+    def flops(self, T: int) -> float:
+        return 2.0 * self.heads * (self.dim + self.vdim) * min(T, self.window or T)
 
 
 @dataclass
@@ -393,6 +415,7 @@ class Mamba2Spec:
     conv: int                    # taps of the short convolution
     norm_groups: int
     kind = "mamba2"
+    recurrent = True
 
     @staticmethod
     def from_json(m: dict) -> "Mamba2Spec":
@@ -423,36 +446,44 @@ class Mamba2Spec:
                 ("conv.b", (self.channels,)), ("dt_bias", (self.heads,)), ("A_log", (self.heads,)),
                 ("D", (self.heads,)), ("norm", (self.inner,)), ("o", (width, self.inner))]
 
+    def flops(self, T: int) -> float:
+        return 6.0 * self.heads * self.state * self.vdim
+
 
 @dataclass
 class LatentAttentionSpec:
     """Attention whose keys and values are projections of one cached latent per token, plus one rotated key
-    part that all heads share; queries go through a latent of their own."""
+    part that all heads share; queries go through a latent of their own, or straight from the input."""
     heads: int
     dim: int                     # unrotated query / key dimensions of a head
     rot_dim: int                 # rotated ones
     vdim: int
     kv_rank: int
-    q_rank: int
+    q_rank: int                  # 0 with q_latent: as the checkpoint has it
     scale: float
     rot: RotarySpec = None
     window: Optional[int] = None     # keys a query sees, itself included (None: every earlier one)
     kv_from: Optional[int] = None    # the layer whose latents and rotated key parts are used
+    q_latent: bool = True        # queries go through a latent of their own
+    head_gate: bool = False      # sigmoid gate on every head's output
     kind = "latent_attention"
+    recurrent = False
 
     @staticmethod
-    def from_json(m: dict) -> "LatentAttentionSpec":
+    def from_json(m: dict, interleaved: bool = True, **constants) -> "LatentAttentionSpec":
         mask, j = m.get("mask") or {}, m.get("kv_from")
         rot = dict(m["rot"])
         rot.setdefault("dims", m["rot_dim"])
         return LatentAttentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]),
                                    kv_rank=int(m["kv_rank"]), q_rank=int(m.get("q_rank") or 0), scale=float(m["scale"]),
-                                   rot=RotarySpec.from_json(rot, interleaved=True),
+                                   rot=RotarySpec.from_json(rot, interleaved=interleaved),
                                    window=int(mask["size"]) if mask.get("size") else None,
-                                   kv_from=None if j is None else int(j))
+                                   kv_from=None if j is None else int(j), **constants)
 
     def to_json(self) -> dict:
-        m = {k: v for k, v in asdict(self).items() if k not in ("rot", "window", "kv_from")}
+        m = {k: v for k, v in asdict(self).items() if k not in ("rot", "window", "kv_from", "q_latent", "head_gate")}
+        if not self.q_latent:
+            del m["q_rank"]
         m["rot"] = {"dims": self.rot.dims, "base": self.rot.base}
         if self.rot.scaling is not None:
             m["rot"]["scaling"] = asdict(self.rot.scaling)
@@ -463,7 +494,8 @@ class LatentAttentionSpec:
         return m
 
     def fill(self, shape):
-        self.q_rank = self.q_rank or shape("dq")[0]
+        if self.q_latent:
+            self.q_rank = self.q_rank or shape("dq")[0]
 
     def check(self):
         if self.rot.dims != self.rot_dim or self.rot_dim % 2:
@@ -472,12 +504,18 @@ class LatentAttentionSpec:
             raise ValueError("latent attention: the window holds at least the token itself")
 
     def tensors(self, width: int):
-        out = [("dq", (self.q_rank, width)), ("dq.norm", (self.q_rank,)),
-               ("uq", (self.heads * (self.dim + self.rot_dim), self.q_rank))]
+        rows = self.heads * (self.dim + self.rot_dim)
+        out = [("dq", (self.q_rank, width)), ("dq.norm", (self.q_rank,)), ("uq", (rows, self.q_rank))] if self.q_latent else \
+            [("q", (rows, width))]
         if self.kv_from is None:
             out += [("dkv", (self.kv_rank + self.rot_dim, width)), ("dkv.norm", (self.kv_rank,))]
-        return out + [("uk", (self.heads * self.dim, self.kv_rank)), ("uv", (self.heads * self.vdim, self.kv_rank)),
-                      ("o", (width, self.heads * self.vdim))]
+        out += [("uk", (self.heads * self.dim, self.kv_rank)), ("uv", (self.heads * self.vdim, self.kv_rank))]
+        if self.head_gate:
+            out.append(("g", (self.heads, width)))
+        return out + [("o", (width, self.heads * self.vdim))]
+
+    def flops(self, T: int) -> float:
+        return 2.0 * self.heads * (self.dim + self.rot_dim + self.vdim) * min(T, self.window or T)
 
 
 @dataclass
@@ -488,6 +526,7 @@ class GeneralDeltaSpec:
     dim: int
     decay_rank: int = 0
     kind = "general_delta"
+    recurrent = True
 
     @property
     def inner(self) -> int:
@@ -512,6 +551,9 @@ class GeneralDeltaSpec:
                 ("a.b", (n,)), ("w1", (self.decay_rank, width)), ("w2", (n, self.decay_rank)), ("w0", (n,)),
                 ("norm", (n,)), ("o", (width, n))]
 
+    def flops(self, T: int) -> float:
+        return 10.0 * self.heads * self.dim * self.dim
+
 
 @dataclass
 class RgLruSpec:
@@ -522,6 +564,7 @@ class RgLruSpec:
     conv: int
     decay: float = 8.0           # log a = -decay r softplus(lam)
     kind = "rglru"
+    recurrent = True
 
     @staticmethod
     def from_json(m: dict) -> "RgLruSpec":
@@ -541,6 +584,76 @@ class RgLruSpec:
         return [("y", (n, width)), ("y.b", (n,)), ("x", (n, width)), ("x.b", (n,)), ("conv", (n, self.conv)), ("conv.b", (n,)),
                 ("ra", (self.blocks, b, b)), ("ra.b", (self.blocks, b)), ("ri", (self.blocks, b, b)),
                 ("ri.b", (self.blocks, b)), ("lam", (n,)), ("o", (width, n))]
+
+    def flops(self, T: int) -> float:
+        return 12.0 * self.width
+
+
+@dataclass
+class MlstmSpec:
+    """Matrix memory with exponential gates: per head a state of key x value channels, a normaliser of key
+    channels and the running maximum of the gates' logarithms, which are bounded by ``gate_cap``."""
+    heads: int
+    dim: int                     # query / key head size
+    vdim: int
+    gate_cap: float
+    kind = "mlstm"
+    recurrent = True
+
+    @staticmethod
+    def from_json(m: dict) -> "MlstmSpec":
+        return MlstmSpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), gate_cap=float(m["gate_cap"]))
+
+    def to_json(self) -> dict:
+        return asdict(self)
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    def check(self):
+        if not self.gate_cap > 0:
+            raise ValueError("mlstm: the gates' bound is positive")
+
+    def tensors(self, width: int):
+        n, h = self.inner, self.heads
+        return [("q", (h * self.dim, width)), ("k", (h * self.dim, width)), ("v", (n, width)), ("g", (n, width)),
+                ("o", (width, n)), ("norm", (n,)), ("i", (h, width)), ("i.b", (h,)), ("f", (h, width)), ("f.b", (h,))]
+
+    def flops(self, T: int) -> float:
+        return 6.0 * self.heads * self.dim * self.vdim
+
+
+@dataclass
+class ParallelSpec:
+    """Two mixers reading the same input; their results are added with a factor each."""
+    left: object
+    right: object
+    left_scale: float
+    right_scale: float
+    kind = "parallel"
+
+    @staticmethod
+    def from_json(m: dict, left, right) -> "ParallelSpec":
+        return ParallelSpec(left(m["left"]), right(m["right"]), float(m["left_scale"]), float(m["right_scale"]))
+
+    def to_json(self) -> dict:
+        return {"left": self.left.to_json(), "left_scale": self.left_scale, "right": self.right.to_json(),
+                "right_scale": self.right_scale}
+
+    @property
+    def recurrent(self) -> bool:
+        return self.left.recurrent or self.right.recurrent
+
+    def check(self):
+        self.left.check()
+        self.right.check()
+
+    def tensors(self, width: int):
+        return [(side + "." + n, s) for side in ("left", "right") for n, s in getattr(self, side).tensors(width)]
+
+    def flops(self, T: int) -> float:
+        return self.left.flops(T) + self.right.flops(T)
 
 
 @dataclass
@@ -582,28 +695,116 @@ class PolyNormSpec:
 
 
 @dataclass
+class GeluGluSpec:
+    """gelu(gate) up between the gate / up and down projections (gelu in its tanh form); projections with biases."""
+    ff: int
+    kind = "gelu_glu"
+
+    @staticmethod
+    def from_json(f: dict) -> "GeluGluSpec":
+        return GeluGluSpec(int(f["ff"]))
+
+    def to_json(self) -> dict:
+        return {"kind": "dense", "ff": self.ff}
+
+    def tensors(self, width: int):
+        return [("gate", (self.ff, width)), ("gate.b", (self.ff,)), ("up", (self.ff, width)), ("up.b", (self.ff,)),
+                ("down", (width, self.ff)), ("down.b", (width,))]
+
+
+@dataclass
+class RoutedSpec:
+    """Mixture of clamped gated experts.  A router's softmax scores pick ``top`` experts of every token, within
+    the ``keep`` groups (of ``groups`` equal ones) whose best expert scores highest; their weights are their
+    scores over the scores' sum, times ``scale``.  An optional shared expert runs for every token."""
+    expert: ClampedGluSpec
+    experts: int
+    top: int
+    groups: int = 1
+    keep: int = 1
+    scale: float = 1.0
+    shared: Optional[ClampedGluSpec] = None
+    kind = "routed"
+    #: added to the sum that the chosen scores are divided by
+    tiny = 1e-20
+
+    @staticmethod
+    def from_json(f: dict) -> "RoutedSpec":
+        r, sh = f["router"], f.get("shared")
+        g = r.get("groups") or {}
+        return RoutedSpec(ClampedGluSpec.from_json(f["expert"]), int(r["experts"]), int(r["top"]), int(g.get("count", 1)),
+                          int(g.get("keep", 1)), float(r.get("scale", 1.0)), ClampedGluSpec.from_json(sh) if sh else None)
+
+    def to_json(self) -> dict:
+        size = lambda e: {"ff": e.ff, "limit": e.limit}
+        out = {"kind": "moe", "expert": size(self.expert),
+               "router": {"experts": self.experts, "groups": {"count": self.groups, "keep": self.keep}, "scale": self.scale,
+                          "top": self.top}}
+        return out if self.shared is None else dict(out, shared=size(self.shared))
+
+    def check(self):
+        if self.groups < 1 or self.experts % self.groups or not 1 <= self.keep <= self.groups:
+            raise ValueError(f"routed: {self.experts} experts in {self.groups} groups, {self.keep} of them kept")
+        if not 1 <= self.top <= self.experts // self.groups * self.keep:
+            raise ValueError(f"routed: {self.top} experts out of {self.experts // self.groups * self.keep}")
+        if self.experts > 1024 or self.top > 32:
+            raise ValueError("routed: up to 1024 experts, 32 of a token")
+
+    def tensors(self, width: int):
+        out = [(f"e{e}.{n}", s) for e in range(self.experts) for n, s in self.expert.tensors(width)]
+        out.append(("router", (self.experts, width)))
+        return out + ([] if self.shared is None else [("shared." + n, s) for n, s in self.shared.tensors(width)])
+
+
+@dataclass
 class HybridLayer:
     mixer: object                # one of the mixer records above
     mlp: Optional[object] = None
 
 
 @dataclass(frozen=True)
+class MixerForm:
+    """A mixer record as a design has it: with some of its constants fixed."""
+    spec: type
+    constants: tuple = ()
+
+    @property
+    def kind(self) -> str:
+        return self.spec.kind
+
+    def __call__(self, m: dict):
+        return self.spec.from_json(m, **dict(self.constants))
+
+
+def mixer_form(spec: type, **constants) -> MixerForm:
+    return MixerForm(spec, tuple(constants.items()))
+
+
+@dataclass(frozen=True)
 class HybridDesign:
     """What the layers of a design have in common."""
-    mixers: tuple                # mixer records its layers may name
+    mixers: tuple                # mixers its layers may name
     mlp: type                    # its dense feed-forward
+    routed: Optional[type] = None    # its mixture of experts
     norm_offset: float = 0.0     # norms multiply by this plus the stored gain
     embed_norm: bool = False     # a norm behind the embedding
+    positions: bool = False      # a factor on the embedding, and a learned vector per position added to it
     two_norms: bool = False      # the feed-forward reads a norm of its own
     depth_average: bool = False  # what a layer passes on is a weighted sum of all results so far
     tied: bool = False           # the embedding table is the output projection
     residual_mult: bool = False  # a factor on what a layer adds
 
 
+_MATRIX_MEMORY = mixer_form(MlstmSpec)
 HYBRID_FAMILY = {
-    "Pakalix": HybridDesign((AttentionSpec, Mamba2Spec), ClampedGluSpec, norm_offset=1.0, embed_norm=True, residual_mult=True),
-    "Nezalorn": HybridDesign((LatentAttentionSpec, GeneralDeltaSpec, RgLruSpec), PolyNormSpec, two_norms=True,
-                             depth_average=True, tied=True),
+    "Pakalix": HybridDesign((mixer_form(AttentionSpec), mixer_form(Mamba2Spec)), ClampedGluSpec, norm_offset=1.0, embed_norm=True,
+                            residual_mult=True),
+    "Nezalorn": HybridDesign((mixer_form(LatentAttentionSpec), mixer_form(GeneralDeltaSpec), mixer_form(RgLruSpec)), PolyNormSpec,
+                             two_norms=True, depth_average=True, tied=True),
+    "Zepesun": HybridDesign((mixer_form(LatentAttentionSpec, interleaved=False, q_latent=False, head_gate=True), _MATRIX_MEMORY,
+                             mixer_form(ParallelSpec, left=mixer_form(AttentionSpec, qk_norm=False, bias=True, gate="element"),
+                                        right=_MATRIX_MEMORY)),
+                            GeluGluSpec, RoutedSpec, positions=True),
 }
 
 
@@ -615,8 +816,10 @@ class HybridConfig:
     eps: float
     residual_mult: float = 1.0
     design: str = "Pakalix"
-    #: positions are not limited by the design; this is what a server may reserve pages for
+    #: rows of the table of positions; without one positions are not limited, and this is what a server may
+    #: reserve pages for
     max_position_embeddings: int = 131072
+    embed_scale: float = 1.0
 
     def __post_init__(self):
         if not self.layers:
@@ -625,6 +828,8 @@ class HybridConfig:
         for i, l in enumerate(self.layers):
             m = l.mixer
             m.check()
+            if hasattr(l.mlp, "check"):
+                l.mlp.check()
             if m.kind == "attention" and m.v_mix:
                 vals.add((m.kv_heads, m.vdim))
             if m.kind == "latent_attention" and m.kv_from is not None:
@@ -654,7 +859,7 @@ class HybridConfig:
 
     @property
     def recurrent(self) -> bool:
-        return any(l.mixer.kind not in ("attention", "latent_attention") for l in self.layers)
+        return any(l.mixer.recurrent for l in self.layers)
 
     # ---- JSON: the design's own config file
     def to_json(self) -> dict:
@@ -664,22 +869,30 @@ class HybridConfig:
                "norm": {"eps": self.eps}}
         if self.traits.residual_mult:
             out["residual_mult"] = self.residual_mult
+        if self.traits.positions:
+            out.update(embedding={"scale": self.embed_scale}, max_positions=self.max_position_embeddings)
         return out
 
     @staticmethod
     def from_json(c: dict) -> "HybridConfig":
         design = HYBRID_FAMILY[c["architecture"]]
         mixers = {m.kind: m for m in design.mixers}
+        mlps = {"dense": design.mlp, "moe": design.routed}
         layers = []
         for i, e in enumerate(c["layers"]):
             if e["type"] not in mixers:
                 raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
             f = e.get("mlp")
-            if f is not None and f.get("kind", "dense") != "dense":
+            if f is not None and mlps.get(f.get("kind", "dense")) is None:
                 raise ValueError(f"layer {i}: unknown feed-forward {f['kind']!r}")
-            layers.append(HybridLayer(mixers[e["type"]].from_json(e["mixer"]), None if f is None else design.mlp.from_json(f)))
+            layers.append(HybridLayer(mixers[e["type"]](e["mixer"]),
+                                      None if f is None else mlps[f.get("kind", "dense")].from_json(f)))
+        more = {}
+        if design.positions:
+            more = dict(max_position_embeddings=int(c["max_positions"]),
+                        embed_scale=float((c.get("embedding") or {}).get("scale", 1.0)))
         return HybridConfig(vocab=int(c["vocab"]), width=int(c["width"]), layers=layers, eps=float(c["norm"]["eps"]),
-                            residual_mult=float(c.get("residual_mult", 1.0)), design=c["architecture"])
+                            residual_mult=float(c.get("residual_mult", 1.0)), design=c["architecture"], **more)
 
     def fill_sizes(self, shapes) -> None:
         """Sizes that the config file leaves to the tensors; ``shapes``: tensor name -> shape."""
@@ -693,6 +906,8 @@ class HybridConfig:
         out = [("embed", (self.vocab, d))]
         if t.embed_norm:
             out.append(("embed.norm", (d,)))
+        if t.positions:
+            out.append(("pos", (self.max_position_embeddings, d)))
         for i, l in enumerate(self.layers):
             out.append((f"l{i}.norm1", (d,)))
             if t.two_norms and l.mlp is not None:

@@ -3,6 +3,8 @@ Pakalix mixers: soft-capped attention with rotary positions, whole-projection qu
 mixing and per-head output gates, or a Mamba-2 state-space recurrence.
 Nezalorn mixers: windowed latent attention, a generalised delta rule, or a real-gated linear recurrence;
 what a layer passes on is a weighted sum of all results so far.
+Zepesun mixers: latent attention, a matrix memory with exponential gates, or windowed attention and a matrix
+memory side by side; feed-forwards dense or a mixture of experts; learned positions.
 
 This is the weight container of the family (names, shapes, initial values, loading); its forward lives in
 the serving engine (``serve.hybrid.HybridEngine`` over ``csrc/serve/hybrid_forward.cu``)."""
@@ -45,6 +47,7 @@ class HybridDecoder(nn.Module):
         for name, shape in self.cfg.tensors():
             p = self.tensor(name)
             leaf = name.split(".", 2)[-1] if name[0] == "l" and name[1].isdigit() else name
+            leaf = leaf.removeprefix("left.").removeprefix("right.")
             if leaf in ("embed.norm", "final.norm") or name.endswith((".norm1", ".norm2")):
                 v = 1.0 - self.cfg.traits.norm_offset + 0.1 * torch.randn(shape, generator=g)
             elif leaf in ("q.norm", "k.norm", "norm", "dq.norm", "dkv.norm"):
@@ -60,6 +63,8 @@ class HybridDecoder(nn.Module):
                 v = uniform(shape, -8.0, 0.0)
             elif leaf == "a.b":
                 v = uniform(shape, -2.0, 1.0)
+            elif leaf == "f.b":
+                v = uniform(shape, 2.0, 5.0)                             # most of the memory is kept
             elif leaf.endswith(".b") and leaf != "conv.b":
                 v = uniform(shape, -0.3, 0.3)
             elif leaf == "vmix":
@@ -76,7 +81,9 @@ class HybridDecoder(nn.Module):
             elif leaf == "conv.b":
                 v = uniform(shape, -0.1, 0.1)
             elif name == "embed":
-                v = torch.randn(shape, generator=g)
+                v = torch.randn(shape, generator=g) / self.cfg.embed_scale
+            elif name == "pos":
+                v = 0.3 * torch.randn(shape, generator=g)
             else:
                 v = torch.randn(shape, generator=g) / math.sqrt(shape[-1])
             p.copy_(v.to(p.dtype))
@@ -107,18 +114,10 @@ class HybridDecoder(nn.Module):
         """Matrix-product FLOPs of one token with T tokens of context, attention and recurrence included."""
         total = 0.0
         for n, s in self.cfg.tensors():
-            if len(s) > 1 and (n != "embed" or self.cfg.traits.tied) and not n.endswith((".conv", "a.b", "i.b")):
-                total += 2.0 * math.prod(s)
-        for l in self.cfg.layers:
-            m = l.mixer
-            if m.kind == "attention":
-                total += 2.0 * m.heads * (m.dim + m.vdim) * T
-            elif m.kind == "latent_attention":
-                total += 2.0 * m.heads * (m.dim + m.rot_dim + m.vdim) * min(T, m.window or T)
-            elif m.kind == "mamba2":
-                total += 6.0 * m.heads * m.state * m.vdim
-            elif m.kind == "general_delta":
-                total += 10.0 * m.heads * m.dim * m.dim
-            else:
-                total += 12.0 * m.width
-        return total
+            if len(s) > 1 and n != "pos" and (n != "embed" or self.cfg.traits.tied) and not n.endswith((".conv", "a.b", "i.b")):
+                share = 1.0
+                if ".mlp.e" in n:            # of a token's own experts
+                    f = self.cfg.layers[int(n[1:n.index(".")])].mlp
+                    share = f.top / f.experts
+                total += 2.0 * share * math.prod(s)
+        return total + sum(l.mixer.flops(T) for l in self.cfg.layers)

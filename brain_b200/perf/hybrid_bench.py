@@ -169,7 +169,7 @@ def hybrid_kernels(eng, entries, phase, timer, peaks):
     if b.n_pre:
         us = t("bb_flash_fwd_paged_x", q, eng.ld["proj"], P(a.kc), P(a.vc), cat, eng.ld["cat"], P(b.tables), b.max_blocks,
                eng.block_size, eng.num_blocks + 1, P(b.seq_row0), P(b.seq_ctx), P(b.tile_seq), P(b.tile_qt), b.n_tiles, n,
-               a.hq, a.hk, a.dkp, a.dvp, C.c_float(a.scale), C.c_float(a.softcap), gate, eng.ld["proj"])
+               a.hq, a.hk, a.dkp, a.dvp, C.c_float(a.scale), C.c_float(a.softcap), gate, eng.ld["proj"], 0, C.c_float(1.0), 0)
         pairs = sum(l * (c - l) + l * (l + 1) / 2 for l, c in zip(lens, ctxs))
         _row(out, phase, "attention: scores and values", us, tflop=2e-12 * pairs * a.hq * (a.dk + a.dv), peaks=peaks,
              like="attention")
@@ -184,7 +184,7 @@ def hybrid_kernels(eng, entries, phase, timer, peaks):
         splits = C.c_int(max(1, min(16, -(-4 * 148 // (n * a.hk)))))
         us = t("bb_paged_decode_x", q, eng.ld["proj"], P(a.kc), P(a.vc), P(b.tables), b.max_blocks, P(b.seq_ctx), cat,
                eng.ld["cat"], P(sc.part_o.data_ptr()), P(sc.part_ml.data_ptr()), n, a.hq, a.hk, a.dkp, a.dvp, eng.block_size,
-               splits, C.c_float(a.scale), C.c_float(a.softcap), gate, eng.ld["proj"])
+               splits, C.c_float(a.scale), C.c_float(a.softcap), gate, eng.ld["proj"], 0, C.c_float(1.0), 0)
         _row(out, phase, "attention: scores and values", us, sum(ctxs) * a.hk * (a.dkp + a.dvp) * 2 / 1e9, peaks=peaks,
              like="attention")
         us = t("bb_hy_ssm_decode", cfg, lm, w, bb)

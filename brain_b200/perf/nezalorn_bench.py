@@ -106,7 +106,7 @@ def kernels(eng, entries, phase, timer, peaks):
         gemm("latent: keys and values", "input projections", at("ckv"), ld["ckv"], a.expand, at("kvx"), ld["kvx"], rows=b.n_exp)
         us = t("bb_flash_fwd_window", at("q"), ld["q"], at("kvx"), at("kvx", a.hq * dq), ld["kvx"], b.n_exp, at("cat"), ld["cat"],
                P(b.seq_row0), P(b.kv_row0), P(b.kv_pos0), P(b.seq_ctx), P(b.tile_seq), P(b.tile_qt), b.n_tiles, n, a.hq, a.hq,
-               dq, a.dvp, C.c_float(a.scale), win)
+               dq, a.dvp, C.c_float(a.scale), win, P(None), 0)
         pairs = sum(min(p + 1, win) for l, c in zip(lens, ctxs) for p in range(c - l, c))
         row("latent: scores and values", us, "attention", tflop=2e-12 * pairs * a.hq * (a.dk + a.rot + a.dv))
     else:

@@ -1,4 +1,4 @@
-"""Serving engine of the hybrid decoders (Pakalix, Nezalorn): pages for the attention layers, recurrent-state
+"""Serving engine of the hybrid decoders (Pakalix, Nezalorn, Zepesun): pages for the attention layers, recurrent-state
 slots for the recurrent layers, one native call per step.
 
 * A step is ONE packed batch: prompt portions of any length and single decoded tokens of several
@@ -6,11 +6,12 @@ slots for the recurrent layers, one native call per step.
   mixed and decode calls and :meth:`HybridEngine.step_logits` - goes through it.
 * Pages: per attention layer keys and values ``[num_blocks + 1, kv_heads, block_size, head size]``, per latent
   attention layer with latents of its own ``[num_blocks + 1, block_size, latent | rotated key part]``.  State
-  slots: per recurrent layer the fp32 state (``[heads, state, head size]``, ``[heads, key, value]`` or one value
-  per channel) and, where it has a convolution, a ring of the last taps - 1 raw inputs.  A sequence at position
+  slots: per recurrent layer the fp32 state (``[heads, state, head size]``, ``[heads, key, value]``, a matrix
+  memory with its normaliser and running maximum, or one value per channel) and, where it has a convolution, a ring of the last taps - 1 raw inputs.  A sequence at position
   0 starts from zeros, so pages and slots are reused as they are.
+* Mixtures of experts: rows of a step sorted by expert onto 128-row tiles, one grouped product per matrix.
 * ``dtype='bf16'``: bf16 weights, activations, pages and convolution inputs; the residual stream, norms,
-  rotation, scores, softmax, step sizes, decays and the recurrent state are fp32.  ``dtype='fp32'``:
+  rotation, scores, softmax, routers, step sizes, gates of a recurrence, decays and the recurrent state are fp32.  ``dtype='fp32'``:
   everything in fp32, no tensor-core rounding."""
 from __future__ import annotations
 
@@ -65,8 +66,20 @@ class _Scratch:
         ab = rows if eng.absorb_portions else max(dec, 1)
         self.q, self.qa, self.ol, self.aux = z(rows, m["q"]), z(ab, m["qa"]), z(ab, m["ol"]), z(rows, m["aux"])
         self.ckv, self.kvx = z(max(exp, 1), m["ckv"]), z(max(exp, 1), m["kvx"])
+        self.f32 = z(rows, m["f32"], dtype=f32)
+        # mixture of experts: every expert that has rows takes at most one 128-row tile that is not full
+        routed = [l for l in eng.layers if l.n_experts]
+        top = max((l.top for l in routed), default=0)
+        moe = 128 * max((rows * l.top // 128 + min(rows * l.top, l.n_experts) for l in routed), default=0)
+        i32 = torch.int32
+        self.ex_in, self.ex_out = (z(max(moe, 1), eng.dp if routed else 8) for _ in range(2))
+        self.ex_gu, self.ex_act = z(max(moe, 1), m["gu"]), z(max(moe, 1), m["act"])
+        self.pair_expert, self.pair_row = (z(max(rows * top, 1), dtype=i32) for _ in range(2))
+        self.pair_w = z(max(rows * top, 1), dtype=f32)
+        self.ex_count = z(max((l.n_experts for l in routed), default=1), dtype=i32)
+        self.ex_tile = z(max(moe // 128, 1), dtype=i32)
         po = pm = 1
-        for l in eng.layer_list:
+        for l in eng.mixers:
             if l.kind == 0 and dec and not eng.fp32:
                 n = dec * l.hq * self._max_splits(l.hk, dec)
                 po, pm = max(po, n * (64 if l.dvp <= 64 else 128)), max(pm, n * 2)
@@ -75,15 +88,16 @@ class _Scratch:
                 po, pm = max(po, n * l.kvrp), max(pm, n * 2)
         self.part_o, self.part_ml = z(po, dtype=f32), z(pm, dtype=f32)
         # segment states of the chunked recurrence (prompt portions): two machine-fulls of states
-        npmax = max([l.n * l.p for l in eng.layer_list if l.kind == 1], default=0)
+        npmax = max([l.n * l.p for l in eng.mixers if l.kind == 1], default=0)
         self.seg = z(2 * 2 * eng.sm_count * (npmax + 1) if portions and not eng.fp32 and 0 < npmax <= 128 * 128 else 1, dtype=f32)
         self.hn, self.logits = z(max(want, 1), eng.dp), z(max(want, 1), eng.vocabp, dtype=f32)
         w = self.work = hn.Work()
         for n in ("x", "h", "proj", "cat", "xbc", "dt", "y", "v_first", "part_o", "part_ml", "seg", "hn", "logits", "h2", "q",
-                  "qa", "ol", "aux", "ckv", "kvx"):
+                  "qa", "ol", "aux", "ckv", "kvx", "f32", "ex_in", "ex_gu", "ex_act", "ex_out", "pair_expert", "pair_row",
+                  "pair_w", "ex_count", "ex_tile"):
             setattr(w, n, _ptr(getattr(self, n)))
         w.seg_floats = self.seg.numel()
-        w.rows, w.want_rows, w.exp_rows = rows, max(want, 1), exp
+        w.rows, w.want_rows, w.exp_rows, w.moe_rows = rows, max(want, 1), exp, moe
         for k in m:
             setattr(w, "ld_" + k, m[k])
         w.splits, w.pool_blocks = _MAX_SPLITS, eng.num_blocks + 1
@@ -114,7 +128,8 @@ class HybridEngine(PagedEngineBase):
         self.vocab, self.vocabp = cfg.vocab, pad8(cfg.vocab)
         self.dp = pad8(cfg.width)
         self.block_size, self.num_blocks = block_size, num_blocks
-        self.max_seq_len, self.max_prefill_tokens = max_seq_len, max_prefill
+        self.max_seq_len, self.max_prefill_tokens = min(max_seq_len, cfg.max_position_embeddings), max_prefill
+        max_seq_len = self.max_seq_len
         self.topk_capacity = topk
         self.max_blocks = (max_seq_len + block_size - 1) // block_size
         self.state_slots, self.dummy_slot = state_slots, state_slots
@@ -176,20 +191,27 @@ class HybridEngine(PagedEngineBase):
         key = (rot.dims, rot.base, str(rot.scaling))
         if key not in self._rope:
             f, mag = rot.frequencies()
-            ang = torch.arange(self.max_seq_len, dtype=torch.float64)[:, None] * torch.tensor(f, dtype=torch.float64)
+            ang = torch.arange(self.max_blocks * self.block_size, dtype=torch.float64)[:, None] * torch.tensor(f, dtype=torch.float64)
             self._rope[key] = tuple((mag * t).float().to(self.device) for t in (ang.cos(), ang.sin()))
         L.cos_t, L.sin_t, L.rot = *map(_ptr, self._rope[key]), rot.dims
 
-    # Every packer adds what reads the normed input to ``stack`` and returns the mixer's output projection with
-    # its padded input width.
-    def _pack_attention(self, i: int, L, m, p: str, stack):
+    # Every packer adds what reads the normed input to ``stack`` (to ``stack32`` where the product stays fp32) and
+    # returns the mixer's output projection with its padded input width.  ``scale``: a factor on the mixer's result.
+    def _pack_attention(self, i: int, L, m, p: str, stack, scale: float = 1.0):
         dkp, dvp = pad8(m.dim), pad8(m.vdim)
         L.kind, L.hq, L.hk, L.dk, L.dv, L.dkp, L.dvp = 0, m.heads, m.kv_heads, m.dim, m.vdim, dkp, dvp
         L.off_q = stack.add(self._rows(p + "q", m.heads, m.dim))
         L.off_k = stack.add(self._rows(p + "k", m.kv_heads, m.dim))
         L.off_v = stack.add(self._rows(p + "v", m.kv_heads, m.vdim))
-        L.off_g = stack.add(self._mat(p + "g"))
-        L.q_norm, L.k_norm = self._head_vec(p + "q.norm", m.heads, m.dim), self._head_vec(p + "k.norm", m.kv_heads, m.dim)
+        elems = m.gate == "element"
+        L.off_g = stack.add(self._rows(p + "g", m.heads, m.vdim) if elems else self._mat(p + "g"))
+        L.gate_kind, L.out_scale, L.window = 2 if elems else 1, scale, m.window or 0
+        if m.qk_norm:
+            L.q_norm, L.k_norm = self._head_vec(p + "q.norm", m.heads, m.dim), self._head_vec(p + "k.norm", m.kv_heads, m.dim)
+        if m.bias:
+            L.q_b, L.k_b, L.v_b = (self._head_vec(p + n + ".b", h, d) for n, h, d in
+                                   (("q", m.heads, m.dim), ("k", m.kv_heads, m.dim), ("v", m.kv_heads, m.vdim)))
+            self.out_bias.append(scale * self._tensor(p + "o.b").float().cpu())
         if m.rot is not None and m.rot.dims:
             self._rotary(L, m.rot)
         L.scale, L.softcap = m.scale, m.softcap or 0.0
@@ -229,25 +251,37 @@ class HybridEngine(PagedEngineBase):
         self._widest(xbc=chp)
 
     def _pack_latent_attention(self, i: int, L, m, p: str, stack):
-        H, dkp, rotp, dvp, kvrp, qrp = m.heads, *map(pad8, (m.dim, m.rot_dim, m.vdim, m.kv_rank, m.q_rank))
+        H, dkp, rotp, dvp, kvrp, qrp = m.heads, *map(pad8, (m.dim, m.rot_dim, m.vdim, m.kv_rank, m.q_rank if m.q_latent else 0))
         L.kind, L.hq, L.hk, L.dk, L.dkp, L.dv, L.dvp = 2, H, 1, m.dim, dkp, m.vdim, dvp
+        L.out_scale = 1.0
         L.qr, L.qrp, L.kvr, L.kvrp, L.rotp, L.scale, L.window = m.q_rank, qrp, m.kv_rank, kvrp, rotp, m.scale, m.window or 0
         self._rotary(L, m.rot)
-        L.off_dq = stack.add(self._mat(p + "dq"))
-        L.dq_norm = self._vec(self._tensor(p + "dq.norm"), qrp)
+        # the kernels rotate neighbouring pairs: half-split ones are brought there by the order of the rows
+        R = m.rot_dim
+        order = list(range(R)) if m.rot.interleaved else [i // 2 + (i % 2) * (R // 2) for i in range(R)]
+        per_head = lambda name, n: self._mat(p + name).view(H, n, -1)
+        q = per_head("uq" if m.q_latent else "q", m.dim + R)
+        qin = qrp if m.q_latent else q.shape[2]
+        q = torch.cat([hn.padded_groups(q[:, :m.dim], dkp, qin), hn.padded_groups(q[:, m.dim:][:, order], rotp, qin)],
+                      dim=1).view(-1, qin)
+        if m.q_latent:
+            L.off_dq = stack.add(self._mat(p + "dq"))
+            L.dq_norm = self._vec(self._tensor(p + "dq.norm"), qrp)
+            L.uq = self._lin(q)
+            self._widest(q=H * (dkp + rotp))
+        else:
+            L.off_q = stack.add(q)
+        if m.head_gate:
+            L.gate_kind, L.off_g = 1, stack.add(self._mat(p + "g"))
         row = kvrp + rotp
         if m.kv_from is None:
             w = self._mat(p + "dkv")
             L.own_kv, L.off_ckv = 1, stack.add(w[:m.kv_rank])
-            stack.add(w[m.kv_rank:])
+            stack.add(w[m.kv_rank:][order])
             L.dkv_norm = self._vec(self._tensor(p + "dkv.norm"), kvrp)
             L.kc = self._pages(self.block_size, row)
         else:
             L.kc = self.layers[m.kv_from].kc
-        per_head = lambda name, n: self._mat(p + name).view(H, n, -1)
-        q = per_head("uq", m.dim + m.rot_dim)
-        uq = torch.cat([hn.padded_groups(q[:, :m.dim], dkp, qrp), hn.padded_groups(q[:, m.dim:], rotp, qrp)], dim=1)
-        L.uq = self._lin(uq.view(-1, qrp))
         uk, uv = per_head("uk", m.dim), per_head("uv", m.vdim)
         L.w_abs = self._hold_matrix(hn.padded_groups(uk.transpose(1, 2), kvrp, dkp))
         L.w_uv = self._hold_matrix(hn.padded_groups(uv, dvp, kvrp))
@@ -260,7 +294,7 @@ class HybridEngine(PagedEngineBase):
             v = hn.padded_groups(uv, dvp, row)
             L.expand = self._lin(torch.cat([k.view(-1, row), v.view(-1, row)]).contiguous())
             self._widest(ckv=row, kvx=H * (dkp + rotp + dvp))
-        self._widest(q=H * (dkp + rotp), qa=H * row, ol=H * kvrp)
+        self._widest(qa=H * row, ol=H * kvrp)
         self.absorb_portions |= not fits
         self.exp_window = None if m.window is None or self.exp_window is None else max(self.exp_window, m.window)
         return self._cols(p + "o", H, m.vdim), H * dvp
@@ -291,6 +325,43 @@ class HybridEngine(PagedEngineBase):
         self._widest(aux=2 * L.chp)
         return self._cols(p + "o", B, n), L.innerp
 
+    def _pack_mlstm(self, i: int, L, m, p: str, stack, scale: float = 1.0):
+        H, np_, pp = m.heads, pad8(m.dim), pad8(m.vdim)
+        L.kind, L.heads, L.n, L.np, L.p, L.pp, L.inner, L.innerp = 5, H, m.dim, np_, m.vdim, pp, m.inner, H * pp
+        L.groups, L.gate_cap, L.q_scale = H, m.gate_cap, m.dim ** -0.5
+        L.off_kk, L.off_q = (stack.add(self._rows(p + n, H, m.dim)) for n in "kq")
+        L.off_vv, L.off_gg = (stack.add(self._rows(p + n, H, m.vdim)) for n in "vg")
+        L.off32_i, L.off32_f = (self.stack32.add(self._mat(p + n)) for n in "if")
+        L.i_b, L.f_b = (self._vec(self._tensor(p + n + ".b"), pad8(H)) for n in "if")
+        L.gnorm = self._hold(hn.head_vec(scale * self._tensor(p + "norm").float(), H, m.vdim, pp, self.device))
+        L.mem = -(-(m.dim * m.vdim + m.dim + 1) // 4) * 4
+        L.ssm_state = self._slots(H, L.mem)
+        self._widest(y=L.innerp)
+        return self._cols(p + "o", H, m.vdim), L.innerp
+
+    def _pack_parallel(self, i: int, L, m, p: str, stack):
+        left = self._pack_attention(i, L, m.left, p + "left.", stack, m.left_scale)
+        R = hn.Layer()
+        right = self._pack_mlstm(i, R, m.right, p + "right.", stack, m.right_scale)
+        R.off_cat = left[1]
+        self.mixers.append(R)                  # (kept alive there)
+        L.beside = C.addressof(R)
+        return [left, right]
+
+    def _pack_routed(self, L, f, p: str) -> None:
+        effp, dp, E = pad8(f.expert.ff), self.dp, f.experts
+        L.n_experts, L.top, L.groups_all, L.groups_keep, L.eff, L.effp = E, f.top, f.groups, f.keep, f.expert.ff, effp
+        L.route_scale, L.route_tiny = f.scale, f.tiny
+        L.e_limit, L.e_alpha, L.e_shift = f.expert.limit, f.expert.alpha, f.expert.shift
+        gu = torch.zeros(E, 2, effp, dp, device=self.device, dtype=self.dtype)
+        down = torch.zeros(E, dp, effp, device=self.device, dtype=self.dtype)
+        for e in range(E):
+            gate, up, out = (self._mat(f"{p}e{e}.{n}") for n in ("gate", "up", "down"))
+            gu[e, 0, :f.expert.ff, :gate.shape[1]], gu[e, 1, :f.expert.ff, :up.shape[1]] = gate, up
+            down[e, :out.shape[0], :f.expert.ff] = out
+        L.w_egu, L.w_edown = self._hold_matrix(gu), self._hold_matrix(down)
+        self._widest(gu=2 * effp, act=effp)
+
     def _pack(self, model) -> None:
         cfg, dev, dp = self.cfg, self.device, self.dp
         traits = cfg.traits
@@ -298,7 +369,8 @@ class HybridEngine(PagedEngineBase):
         n = cfg.n_layers
         self.layers = (hn.Layer * n)()
         self.layer_list = [self.layers[i] for i in range(n)]
-        self.ld = dict.fromkeys(("proj", "cat", "xbc", "dt", "y", "v", "q", "qa", "ol", "ckv", "kvx", "aux"), 8)
+        self.mixers = list(self.layer_list)    # and the second mixers of layers that have two
+        self.ld = dict.fromkeys(("proj", "cat", "xbc", "dt", "y", "v", "q", "qa", "ol", "ckv", "kvx", "aux", "f32", "gu", "act"), 8)
         self.kv_bytes = self.state_bytes = self._matrix_bytes = 0
         # prompt portions of latent attention: whether they also take the absorbed form, and how many keys the
         # widest window of a layer holds (None: all)
@@ -307,40 +379,58 @@ class HybridEngine(PagedEngineBase):
         for i, spec in enumerate(cfg.layers):
             L, p = self.layers[i], f"l{i}."
             L.norm = gain(p + "norm1")
-            stack = hn.RowStack()
-            sections = [getattr(self, "_pack_" + spec.mixer.kind)(i, L, spec.mixer, p + "mix.", stack)]
+            stack, self.stack32, self.out_bias = hn.RowStack(), hn.RowStack(), []
+            f, fp = spec.mlp, p + "mlp."
+            if f is not None and f.kind == "routed":
+                self.stack32.add(self._mat(fp + "router"))
+                self._pack_routed(L, f, fp)
+                f, fp = f.shared, fp + "shared."
+            sections = getattr(self, "_pack_" + spec.mixer.kind)(i, L, spec.mixer, p + "mix.", stack)
+            sections = sections if isinstance(sections, list) else [sections]
             width = stack.n
-            if spec.mlp is not None:
-                f = spec.mlp
+            if f is not None:
                 ffp = pad8(f.ff)
-                L.ff, L.off_act = f.ff, sections[0][1]
-                if f.kind == "clamped_glu":
-                    L.glu_limit, L.glu_alpha, L.glu_shift = f.limit, f.alpha, f.shift
-                    L.off_gate = stack.add(self._mat(p + "mlp.gate"))
-                    L.off_up = stack.add(self._mat(p + "mlp.up"))
-                    width = stack.n
-                else:
+                L.ff, L.off_act = f.ff, sum(w for _, w in sections)
+                if f.kind == "polynorm":
                     L.norm2 = gain(p + "norm2")
-                    L.up = self._lin(hn.columns([(self._mat(p + "mlp.up"), dp)], ffp))
-                    L.up_b, L.down_b = self._vec(T(p + "mlp.up.b"), ffp), self._vec(T(p + "mlp.down.b"), dp)
-                    L.poly, L.off_up = self._vec(T(p + "mlp.act"), 4), stack.n
+                    L.up = self._lin(hn.columns([(self._mat(fp + "up"), dp)], ffp))
+                    L.up_b = self._vec(T(fp + "up.b"), ffp)
+                    L.poly, L.off_up = self._vec(T(fp + "act"), 4), stack.n
                     width = stack.n + ffp
-                sections.append((self._mat(p + "mlp.down"), ffp))
+                else:
+                    if f.kind == "clamped_glu":
+                        L.glu_limit, L.glu_alpha, L.glu_shift = f.limit, f.alpha, f.shift
+                    else:
+                        L.glu_kind, L.gate_b, L.up_b = 1, self._vec(T(fp + "gate.b"), ffp), self._vec(T(fp + "up.b"), ffp)
+                    L.off_gate, L.off_up = stack.add(self._mat(fp + "gate")), stack.add(self._mat(fp + "up"))
+                    width = stack.n
+                if f.kind != "clamped_glu":
+                    self.out_bias.append(T(fp + "down.b").float().cpu())
+                sections.append((self._mat(fp + "down"), ffp))
+            if self.out_bias:
+                L.down_b = self._vec(sum(self.out_bias), dp)
             if traits.depth_average:
                 L.dwa = self._vec(T(p + "dwa"), i + 2)
             L.inp, L.out = self._lin(stack.matrix(dp)), self._lin(hn.columns(sections, dp))
-            self._widest(proj=width, cat=L.out.k)
+            self._widest(proj=width, cat=L.out.k, f32=self.stack32.n)
+            if self.stack32.n:
+                L.in32 = self._lin(self.stack32.matrix(dp))
         c = self.ccfg = hn.Cfg()
         c.dtype, c.width, c.dp, c.vocab, c.vocabp = int(self.fp32), cfg.width, dp, cfg.vocab, self.vocabp
         c.n_layers, c.block_size, c.eps, c.residual_mult = n, self.block_size, cfg.eps, cfg.residual_mult
         c.depth_avg = int(traits.depth_average)
         pad_cols = lambda name: self._hold_matrix(hn.columns([(self._mat(name), dp)], self.vocabp))
         c.embed = pad_cols("embed")
+        if traits.positions:
+            pos = torch.zeros(cfg.max_position_embeddings, dp, device=dev, dtype=self.dtype)
+            pos[:, :cfg.width] = self._mat("pos")
+            c.pos, c.max_pos = self._hold_matrix(pos), cfg.max_position_embeddings
+        c.embed_scale = cfg.embed_scale
         c.head = c.embed if traits.tied else pad_cols("head")
         c.embed_norm = gain("embed.norm") if traits.embed_norm else None
         c.final_norm = gain("final.norm")
         c.layers = C.cast(self.layers, C.c_void_p)
-        del self._tensor
+        del self._tensor, self.stack32, self.out_bias
 
     # ------------------------------------------------------------------ accounting
     def kv_pool_bytes(self) -> int:

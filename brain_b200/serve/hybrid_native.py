@@ -39,13 +39,19 @@ class Layer(C.Structure):
                 ("off_r", I), ("off_kk", I), ("off_vv", I), ("off_gg", I), ("off_a", I), ("off_w1", I),
                 ("w2", Lin), ("w0", P), ("a_b", P),
                 ("blocks", I), ("bw", I), ("bwp", I), ("off_y", I), ("y_b", P), ("x_b", P), ("w_gate", P),
-                ("r_b", P), ("i_b", P), ("lam", P)]
+                ("r_b", P), ("i_b", P), ("lam", P),
+                ("beside", P), ("off_cat", I), ("gate_kind", I), ("out_scale", F), ("q_b", P), ("k_b", P), ("v_b", P),
+                ("glu_kind", I), ("gate_b", P), ("in32", Lin), ("off32_i", I), ("off32_f", I),
+                ("np", I), ("mem", I), ("gate_cap", F), ("q_scale", F), ("f_b", P),
+                ("n_experts", I), ("top", I), ("groups_all", I), ("groups_keep", I), ("eff", I), ("effp", I),
+                ("route_scale", F), ("route_tiny", F), ("e_limit", F), ("e_alpha", F), ("e_shift", F),
+                ("w_egu", P), ("w_edown", P)]
 
 
 class Cfg(C.Structure):
     _fields_ = [("dtype", I), ("width", I), ("dp", I), ("vocab", I), ("vocabp", I), ("n_layers", I),
                 ("block_size", I), ("eps", F), ("residual_mult", F), ("embed", P), ("embed_norm", P),
-                ("final_norm", P), ("head", P), ("layers", P), ("depth_avg", I)]
+                ("final_norm", P), ("head", P), ("layers", P), ("pos", P), ("max_pos", I), ("embed_scale", F), ("depth_avg", I)]
 
 
 class Batch(C.Structure):
@@ -60,7 +66,10 @@ class Work(C.Structure):
                [(n, I) for n in ("rows", "want_rows", "ld_proj", "ld_cat", "ld_xbc", "ld_dt", "ld_y", "ld_v", "splits",
                                  "pool_blocks")] + \
                [(n, P) for n in ("h2", "q", "qa", "ol", "ckv", "kvx", "aux")] + \
-               [(n, I) for n in ("ld_q", "ld_qa", "ld_ol", "ld_ckv", "ld_kvx", "ld_aux", "exp_rows")]
+               [(n, I) for n in ("ld_q", "ld_qa", "ld_ol", "ld_ckv", "ld_kvx", "ld_aux", "exp_rows")] + \
+               [(n, P) for n in ("f32", "ex_in", "ex_gu", "ex_act", "ex_out", "pair_expert", "pair_row", "pair_w", "ex_count",
+                                 "ex_tile")] + \
+               [(n, I) for n in ("ld_f32", "ld_gu", "ld_act", "moe_rows")]
 
 
 def padded_rows(w: torch.Tensor, heads: int, size: int, sizep: int) -> torch.Tensor:

@@ -83,6 +83,14 @@ __device__ __forceinline__ float silu_as(float x) {
   else return silu_f(x);
 }
 
+// gelu in its tanh form.
+template <typename T>
+__device__ __forceinline__ float gelu_as(float z) {
+  const float t = 0.79788456080286536f * fmaf(0.044715f * z * z, z, z);   // sqrt(2 / pi) (z + 0.044715 z^3)
+  if constexpr (sizeof(T) == 2) return z * rcp_hw(1.f + exp2_hw(-2.f * kLog2e * t));
+  else return 0.5f * z * (1.f + tanhf(t));
+}
+
 // Clamped gated unit: g' = min(g, limit), u' = clamp(u, +-limit); g' sigmoid(alpha g') (u' + shift).
 template <typename T>
 __device__ __forceinline__ float clamped_glu_as(float g, float u, float limit, float alpha, float shift) {

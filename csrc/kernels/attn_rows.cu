@@ -1,5 +1,5 @@
 // Attention of single query rows against the paged K/V pool, one warp per (row, query head): any head
-// sizes up to 512, bf16 or fp32 pages, soft-capped scores, per-head output gate.  It is the fp32 path and
+// sizes up to 512, bf16 or fp32 pages, soft-capped scores, windows, output gates (per head or per element).  It is the fp32 path and
 // the path of head sizes the tensor-core prefill and the split-KV decode kernels do not cover.
 #include "../common/host.hpp"
 #include "../common/ptx.cuh"
@@ -13,7 +13,8 @@ __global__ void __launch_bounds__(128)
 attn_rows_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ kc, const T* __restrict__ vc,
                  const int* __restrict__ pos, const int* __restrict__ row_seq, const int* __restrict__ tables,
                  int max_blocks, int bs, T* __restrict__ out, int ldo, const T* __restrict__ gate, int ldg, int rows,
-                 int hq, int hk, int dk, int dv, int dkp, int dvp, float scale, float softcap) {
+                 int hq, int hk, int dk, int dv, int dkp, int dvp, float scale, float softcap, int gate_elems, float out_scale,
+                 int window) {
   const int w = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (w >= rows * hq) return;
   const int r = w / hq, h = w % hq, g = h / (hq / hk);
@@ -27,7 +28,7 @@ attn_rows_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ kc, con
   const int last = pos[r];
   const int* bt = tables + (size_t)row_seq[r] * max_blocks;
   float m = -INFINITY, l = 0.f;
-  for (int j = 0; j <= last; ++j) {
+  for (int j = window > 0 ? max(last - window + 1, 0) : 0; j <= last; ++j) {
     const size_t row = ((size_t)bt[j / bs] * hk + g) * bs + j % bs;
     float s = 0.f;
 #pragma unroll
@@ -47,23 +48,27 @@ attn_rows_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ kc, con
       if (d < dv) o[i] = fmaf(p, to_f(vc[row * dvp + d]), o[i] * al);
     }
   }
-  float f = 1.f / l;
-  if (gate) f *= sigmoid_f(to_f(gate[(size_t)r * ldg + h]));
+  float f = out_scale / l;
+  if (gate && !gate_elems) f *= sigmoid_f(to_f(gate[(size_t)r * ldg + h]));
 #pragma unroll
   for (int i = 0; i < AR_VEC; ++i) {
     const int d = lane + 32 * i;
-    if (d < dvp) out[(size_t)r * ldo + h * dvp + d] = from_f<T>(d < dv ? o[i] * f : 0.f);
+    if (d >= dvp) continue;
+    float v = d < dv ? o[i] * f : 0.f;
+    if (gate && gate_elems) v *= sigmoid_f(to_f(gate[(size_t)r * ldg + h * dvp + d]));
+    out[(size_t)r * ldo + h * dvp + d] = from_f<T>(v);
   }
 }
 
 }  // namespace bb
 
 // dtype 0 bf16, 1 fp32.  Row r attends keys [0, pos[r]] of sequence row_seq[r]; head h of q at column
-// h dkp, of out at column h dvp; gate (may be null): raw gate values, head h at column h.
+// h dkp, of out at column h dvp; gate (may be null): raw gate values, head h at column h, or with gate_elems one for
+// every output column.  window: the latest keys of a row, itself included (0: all).
 BB_API int bb_attn_rows(int dtype, const void* q, int ldq, const void* kc, const void* vc, const int* pos,
                         const int* row_seq, const int* tables, int max_blocks, int bs, void* out, int ldo,
                         const void* gate, int ldg, int rows, int hq, int hk, int dk, int dv, int dkp, int dvp,
-                        float scale, float softcap, void* stream) {
+                        float scale, float softcap, int gate_elems, float out_scale, int window, void* stream) {
   using namespace bb;
   if (rows <= 0) return BB_OK;
   const int d = dk > dvp ? dk : dvp;
@@ -73,7 +78,7 @@ BB_API int bb_attn_rows(int dtype, const void* q, int ldq, const void* kc, const
 #define BB_LAUNCH_AR(T, V)                                                                                          \
   attn_rows_kernel<T, V><<<grid, 128, 0, s>>>((const T*)q, ldq, (const T*)kc, (const T*)vc, pos, row_seq, tables,   \
                                               max_blocks, bs, (T*)out, ldo, (const T*)gate, ldg, rows, hq, hk, dk,  \
-                                              dv, dkp, dvp, scale, softcap)
+                                              dv, dkp, dvp, scale, softcap, gate_elems, out_scale, window)
 #define BB_LAUNCH_AR_T(T)                  \
   do {                                     \
     if (d <= 64) BB_LAUNCH_AR(T, 2);       \

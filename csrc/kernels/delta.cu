@@ -755,6 +755,13 @@ BB_API int bb_hy_delta(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, 
                   : run_delta<__nv_bfloat16>(*L, *w, *b, c->eps, (cudaStream_t)stream);
 }
 
+// Norm and gate of the first `rows` rows of w->y -> w->cat: any recurrence whose heads end that way.
+BB_API int bb_hy_head_post(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int rows, void* stream) {
+  if (rows <= 0) return BB_OK;
+  return c->dtype ? launch_post<float>(*L, *w, rows, c->eps, (cudaStream_t)stream)
+                  : launch_post<__nv_bfloat16>(*L, *w, rows, c->eps, (cudaStream_t)stream);
+}
+
 // The recurrence of the prompt portions alone -> w->y; `any`: by the kernel that covers every size.
 BB_API int bb_hy_delta_scan(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int any, void* stream) {
   cudaStream_t s = (cudaStream_t)stream;

@@ -1,0 +1,270 @@
+// Mixture of experts of a serving step, everything but its matrix products, for bf16 and fp32 storage:
+//   hy_route         one warp per token: softmax over the router's fp32 logits, the best groups by their best
+//                    expert, the best experts of those, their weights; a place among the rows of each
+//   hy_expert_rows   rows of the normed input to their experts' places, every expert's rows on 128-row tiles of
+//                    their own; the tiles' experts
+//   hy_expert_glu    clamped gated product of the experts' two halves
+// A row's place inside its expert's tiles depends on the order in which blocks arrive; its values do not.  The
+// weighted sum over a token's experts is taken where the next layer starts (hy_start).
+#include "../common/host.hpp"
+#include "../common/ptx.cuh"
+#include "../common/rows.cuh"
+#include "../serve/hybrid.hpp"
+
+namespace bb {
+
+constexpr int EX_THREADS = 256, EX_TOKENS = 4;   // tokens of a warp
+
+// Largest value of the warp and the lowest index that has it, in every lane.
+__device__ __forceinline__ void warp_best(float& v, int& i) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float v2 = __shfl_xor_sync(0xffffffffu, v, o);
+    const int i2 = __shfl_xor_sync(0xffffffffu, i, o);
+    if (v2 > v || (v2 == v && i2 < i)) {
+      v = v2;
+      i = i2;
+    }
+  }
+}
+
+// V: experts of a lane (expert j * 32 + lane).
+template <int V>
+__global__ void __launch_bounds__(EX_THREADS)
+hy_route_kernel(const __grid_constant__ BbHyLayer L, const float* __restrict__ logits, int ld, int* __restrict__ pair_expert,
+                int* __restrict__ pair_row, float* __restrict__ pair_w, int* __restrict__ count, int n, int tokens) {
+  __shared__ int hist[V * 32];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, E = L.n_experts, size = E / L.groups_all;
+  for (int e = threadIdx.x; e < E; e += EX_THREADS) hist[e] = 0;
+  __syncthreads();
+  const int t0 = (blockIdx.x * (EX_THREADS / 32) + warp) * tokens;
+  for (int t = t0; t < min(t0 + tokens, n); ++t) {
+    float s[V], mx = -INFINITY, sum = 0.f;
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      s[j] = j * 32 + lane < E ? logits[(size_t)t * ld + j * 32 + lane] : -INFINITY;
+      mx = fmaxf(mx, s[j]);
+    }
+    mx = warp_max(mx);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      s[j] = j * 32 + lane < E ? expf(s[j] - mx) : 0.f;
+      sum += s[j];
+    }
+    const float inv = 1.f / warp_sum(sum);
+#pragma unroll
+    for (int j = 0; j < V; ++j) s[j] *= inv;
+    // groups: take the best expert left in any group not yet kept, keep its group
+    unsigned kept[V];        // bit: the expert's group is kept (an expert's own bit only)
+#pragma unroll
+    for (int j = 0; j < V; ++j) kept[j] = L.groups_keep >= L.groups_all;
+    if (L.groups_keep < L.groups_all) {
+      for (int g = 0; g < L.groups_keep; ++g) {
+        float best = -1.f;
+        int bi = 0x7fffffff;
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+          const int e = j * 32 + lane;
+          if (e < E && !kept[j] && s[j] > best) {
+            best = s[j];
+            bi = e;
+          }
+        }
+        warp_best(best, bi);
+        const int first = bi / size * size;
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+          const int e = j * 32 + lane;
+          if (e >= first && e < first + size) kept[j] = 1;
+        }
+      }
+    }
+    float total = 0.f, my_w = 0.f;
+    int my_e = 0;
+    for (int c = 0; c < L.top; ++c) {
+      float best = -1.f;
+      int bi = 0x7fffffff;
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        const int e = j * 32 + lane;
+        if (e < E && kept[j] && s[j] > best) {
+          best = s[j];
+          bi = e;
+        }
+      }
+      warp_best(best, bi);
+#pragma unroll
+      for (int j = 0; j < V; ++j)
+        if (j * 32 + lane == bi) kept[j] = 0;
+      total += best;
+      if (lane == c) {
+        my_w = best;
+        my_e = bi;
+      }
+    }
+    if (lane < L.top) {
+      const size_t p = (size_t)t * L.top + lane;
+      my_e = min(my_e, E - 1);                     // (logits that are not numbers pick no expert)
+      pair_expert[p] = my_e;
+      pair_row[p] = atomicAdd(&hist[my_e], 1);     // place among the block's rows of this expert
+      pair_w[p] = my_w / (total + L.route_tiny) * L.route_scale;
+    }
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += EX_THREADS)
+    if (hist[e] > 0) hist[e] = atomicAdd(&count[e], hist[e]);   // ... and the block's first place among all
+  __syncthreads();
+  const size_t p1 = (size_t)min(t0 + tokens, n) * L.top;
+  for (size_t p = (size_t)t0 * L.top + lane; p < p1; p += 32) pair_row[p] += hist[pair_expert[p]];
+}
+
+// Every expert's first row, from the counts: rows of expert e start on a 128-row tile.
+__device__ __forceinline__ void expert_offsets(const int* count, int E, int* off) {
+  if (threadIdx.x < 32) {
+    int base = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int e = e0 + threadIdx.x, c = e < E ? (count[e] + 127) & ~127 : 0;
+      int x = c;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int y = __shfl_up_sync(0xffffffffu, x, o);
+        if ((int)threadIdx.x >= o) x += y;
+      }
+      if (e < E) off[e] = base + x - c;
+      base += __shfl_sync(0xffffffffu, x, 31);
+    }
+    if (threadIdx.x == 0) off[E] = base;
+  }
+  __syncthreads();
+}
+
+// A warp per token; the last block writes the tiles' experts.
+template <typename T>
+__global__ void __launch_bounds__(EX_THREADS)
+hy_expert_rows_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ h, int dp, const int* __restrict__ pair_expert,
+                      int* __restrict__ pair_row, const int* __restrict__ count, T* __restrict__ out, int* __restrict__ tiles,
+                      int n_tiles, int n) {
+  extern __shared__ int off[];
+  const int E = L.n_experts;
+  expert_offsets(count, E, off);
+  if (blockIdx.x == gridDim.x - 1) {
+    for (int t = threadIdx.x; t < n_tiles; t += EX_THREADS) {
+      int e = -1;
+      if (t * 128 < off[E]) {
+        int lo = 0, hi = E - 1;                   // the last expert that starts at or before the tile
+        while (lo < hi) {
+          const int mid = (lo + hi + 1) >> 1;
+          if (off[mid] <= t * 128) lo = mid; else hi = mid - 1;
+        }
+        e = lo;
+      }
+      tiles[t] = e;
+    }
+    return;
+  }
+  const int lane = threadIdx.x & 31, t = blockIdx.x * (EX_THREADS / 32) + (threadIdx.x >> 5);
+  if (t >= n) return;
+  int row = 0;
+  if (lane < L.top) {
+    const size_t p = (size_t)t * L.top + lane;
+    row = min(off[pair_expert[p]] + pair_row[p], n_tiles * 128 - 1);
+    pair_row[p] = row;
+  }
+  struct alignas(16) Vec {
+    T v[16 / sizeof(T)];
+  };
+  constexpr int VN = 16 / sizeof(T);
+  const Vec* src = reinterpret_cast<const Vec*>(h + (size_t)t * dp);
+  constexpr int U = 4;
+  for (int i0 = 0; i0 < dp / VN; i0 += 32 * U) {
+    Vec x[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (i0 + u * 32 + lane < dp / VN) x[u] = src[i0 + u * 32 + lane];
+    for (int c = 0; c < L.top; ++c) {
+      Vec* dst = reinterpret_cast<Vec*>(out + (size_t)__shfl_sync(0xffffffffu, row, c) * dp);
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+        if (i0 + u * 32 + lane < dp / VN) dst[i0 + u * 32 + lane] = x[u];
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(EX_THREADS)
+hy_expert_glu_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ gu, int ldgu, T* __restrict__ act, int lda,
+                     const int* __restrict__ tiles, int tile_blocks) {
+  const int tile = blockIdx.x / tile_blocks;
+  if (tiles[tile] < 0) return;
+  const int vecs = L.effp / 8, total = 128 * vecs, stride = tile_blocks * EX_THREADS;
+  for (int i = (blockIdx.x % tile_blocks) * EX_THREADS + threadIdx.x; i < total; i += stride) {
+    const size_t r = (size_t)tile * 128 + i / vecs;
+    const int c = i % vecs * 8;
+    float g[8], u[8];
+    load8(gu + r * ldgu + c, g);
+    load8(gu + r * ldgu + L.effp + c, u);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) g[j] = clamped_glu_as<T>(g[j], u[j], L.e_limit, L.e_alpha, L.e_shift);
+    store8(act + r * lda + c, g);
+  }
+}
+
+}  // namespace bb
+
+using namespace bb;
+
+// Tiles that n tokens of the layer can take.
+static int moe_tiles(const BbHyLayer& L, int n) {
+  const long pairs = (long)n * L.top;
+  return (int)(pairs / 128 + (pairs < L.n_experts ? pairs : L.n_experts));
+}
+BB_API int bb_hy_moe_tiles(const BbHyLayer* L, int n) { return moe_tiles(*L, n); }
+
+// Router logits in columns [0, experts) of w->f32; the counts are clear (hy_start).
+BB_API int bb_hy_route(const BbHyCfg*, const BbHyLayer* L, const BbHyWork* w, int n, void* stream) {
+  if (n <= 0) return BB_OK;
+  const int E = L->n_experts;
+  if (E > 1024 || L->top > 32) return BB_ESIZE;
+  cudaStream_t s = (cudaStream_t)stream;
+  const int warps = EX_THREADS / 32, tokens = n >= 148 * warps * EX_TOKENS ? EX_TOKENS : 1;
+  const int grid = (n + warps * tokens - 1) / (warps * tokens);
+#define BB_ROUTE(V) \
+  hy_route_kernel<V><<<grid, EX_THREADS, 0, s>>>(*L, w->f32, w->ld_f32, w->pair_expert, w->pair_row, w->pair_w, w->ex_count, n, tokens)
+  if (E <= 32) BB_ROUTE(1);
+  else if (E <= 64) BB_ROUTE(2);
+  else if (E <= 128) BB_ROUTE(4);
+  else if (E <= 256) BB_ROUTE(8);
+  else BB_ROUTE(32);
+#undef BB_ROUTE
+  return (int)cudaGetLastError();
+}
+
+BB_API int bb_hy_expert_rows(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream) {
+  if (n <= 0) return BB_OK;
+  cudaStream_t s = (cudaStream_t)stream;
+  const int tiles = moe_tiles(*L, n), grid = (n + EX_THREADS / 32 - 1) / (EX_THREADS / 32) + 1;
+  if (tiles * 128 > w->moe_rows) return BB_EARG;
+  const size_t smem = 4 * (size_t)(L->n_experts + 1);
+  if (c->dtype)
+    hy_expert_rows_kernel<float><<<grid, EX_THREADS, smem, s>>>(*L, static_cast<const float*>(w->h), c->dp, w->pair_expert, w->pair_row,
+                                                                w->ex_count, static_cast<float*>(w->ex_in), w->ex_tile, tiles, n);
+  else
+    hy_expert_rows_kernel<__nv_bfloat16><<<grid, EX_THREADS, smem, s>>>(*L, static_cast<const __nv_bfloat16*>(w->h), c->dp,
+                                                                        w->pair_expert, w->pair_row, w->ex_count,
+                                                                        static_cast<__nv_bfloat16*>(w->ex_in), w->ex_tile, tiles, n);
+  return (int)cudaGetLastError();
+}
+
+BB_API int bb_hy_expert_glu(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream) {
+  if (n <= 0) return BB_OK;
+  cudaStream_t s = (cudaStream_t)stream;
+  const int tiles = moe_tiles(*L, n), per = (128 * (L->effp / 8) + 4 * EX_THREADS - 1) / (4 * EX_THREADS);
+  if (c->dtype)
+    hy_expert_glu_kernel<float><<<tiles * per, EX_THREADS, 0, s>>>(*L, static_cast<const float*>(w->ex_gu), w->ld_gu,
+                                                                   static_cast<float*>(w->ex_act), w->ld_act, w->ex_tile, per);
+  else
+    hy_expert_glu_kernel<__nv_bfloat16><<<tiles * per, EX_THREADS, 0, s>>>(*L, static_cast<const __nv_bfloat16*>(w->ex_gu), w->ld_gu,
+                                                                           static_cast<__nv_bfloat16*>(w->ex_act), w->ld_act,
+                                                                           w->ex_tile, per);
+  return (int)cudaGetLastError();
+}

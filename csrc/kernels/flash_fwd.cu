@@ -47,8 +47,11 @@ struct FaFwdArgs {
   float cap_poly[6];         // ... as an odd polynomial in q.k itself, for |cap_in q.k| < 0.4
   const __nv_bfloat16* gate; // raw gate of row r, head h at gate[r ldg + h]; the output is multiplied by its
   int ldg;                   // sigmoid; may be null
-  // Windowed form (WIN): keys and values of a packed sequence in rows of their own, from kv_row0[seq] on, the
-  // first of them at position kv_pos0[seq]; a query sees the `window` latest keys (0: all), itself included
+  int gate_elems;            // 1: a gate for every element, column c of head h at gate[r ldg + h dv + c]
+  float out_scale;           // factor on the output
+  // Windowed forms (WIN): a query sees the `window` latest keys (0: all), itself included.  WIN = 1: keys and
+  // values of a packed sequence in rows of their own, from kv_row0[seq] on, the first of them at position
+  // kv_pos0[seq]; WIN = 2: in pages
   const int *kv_row0, *kv_pos0;
   int window;
 };
@@ -389,9 +392,9 @@ static constexpr float kFwdTruncLog2 = 0.0041778f;   // log2(1.0029), see the pa
 // the pool's blocks (one TMA copy per block and 64-column half) instead of one copy per tile.
 // EXT: see FaFwdArgs; head sizes below the tile's are zero-filled by the copies (K, V) or multiplied by
 // zeros (Q), P is rounded to nearest when it is packed.
-// WIN (with PAGED and EXT): packed sequences whose keys and values are rows of one matrix; blocks that lie
-// before every query's window are not visited.
-template <int HD, bool PAGED, int HDV = HD, bool EXT = false, bool WIN = false>
+// WIN (with PAGED and EXT): windows, over rows of one matrix (1) or over pages (2); blocks that lie before every
+// query's window are not visited.
+template <int HD, bool PAGED, int HDV = HD, bool EXT = false, int WIN = 0>
 __global__ void __launch_bounds__(192, 2)
 fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                const __grid_constant__ CUtensorMap tmV, const FaFwdArgs args) {
@@ -420,7 +423,7 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
   const int h = blockIdx.y, b = blockIdx.z;
   const int row_base = PAGED ? args.seq_row0[seq] : b * args.T;   // first packed row of this sequence
   const int T = PAGED ? args.seq_row0[seq + 1] - row_base : args.T;
-  const int S = (PAGED ? args.seq_ctx[seq] : args.S) - (WIN ? args.kv_pos0[seq] : 0);
+  const int S = (PAGED ? args.seq_ctx[seq] : args.S) - (WIN == 1 ? args.kv_pos0[seq] : 0);
   const int q0 = qt * 128;
   const int kvh = h / (args.hq / args.hk);
   const int off = S - T;
@@ -434,7 +437,7 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
   const int j_first = WIN ? max(q0 + off - window + 1, 0) / 128 : 0;
   if (WIN) n_blocks -= j_first;
   const int n_units = 2 * n_blocks;
-  const int kv_base = WIN ? args.kv_row0[seq] + j_first * 128 : 0;
+  const int kv_base = WIN == 1 ? args.kv_row0[seq] + j_first * 128 : 0;
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -475,16 +478,17 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
           break;
         }
         mbar_expect_tx(k_full, Cfg::TILE_BYTES);
-        if (WIN) {
+        if (WIN == 1) {
 #pragma unroll
           for (int c = 0; c < NSUB; ++c)
             tma_load_3d(sK + c * Cfg::SUB_BYTES, &tmK, k_full, c * 64, kv_base + j * 128, kvh);
         } else if (PAGED) {
           // pool layout [blocks][kv heads][block_rows][HD]: block i of this tile lands at row i*block_rows
           const int br = args.block_rows, per_tile = 128 / br;
-          const int* tab = args.block_tables + (size_t)seq * args.max_blocks + j * per_tile;
+          const int jt = j_first + j;
+          const int* tab = args.block_tables + (size_t)seq * args.max_blocks + jt * per_tile;
           for (int i = 0; i < per_tile; ++i) {
-            const bool live = (j * 128 + i * br) < S && (j * per_tile + i) < args.max_blocks;
+            const bool live = (jt * 128 + i * br) < S && (jt * per_tile + i) < args.max_blocks;
             const int blk = live ? max(tab[i], 0) : 0;   // dead blocks are masked by the key limit
             for (int c = 0; c < NSUB; ++c)
               tma_load_2d(sK + c * Cfg::SUB_BYTES + i * br * 128, &tmK, k_full, c * 64,
@@ -500,15 +504,16 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
           break;
         }
         mbar_expect_tx(v_full, Cfg::VTILE_BYTES);
-        if (WIN) {
+        if (WIN == 1) {
 #pragma unroll
           for (int c = 0; c < NSUBV; ++c)
             tma_load_3d(sV + c * Cfg::SUB_BYTES, &tmV, v_full, c * 64, kv_base + j * 128, kvh);
         } else if (PAGED) {
           const int br = args.block_rows, per_tile = 128 / br;
-          const int* tab = args.block_tables + (size_t)seq * args.max_blocks + j * per_tile;
+          const int jt = j_first + j;
+          const int* tab = args.block_tables + (size_t)seq * args.max_blocks + jt * per_tile;
           for (int i = 0; i < per_tile; ++i) {
-            const bool live = (j * 128 + i * br) < S && (j * per_tile + i) < args.max_blocks;
+            const bool live = (jt * 128 + i * br) < S && (jt * per_tile + i) < args.max_blocks;
             const int blk = live ? max(tab[i], 0) : 0;
             for (int c = 0; c < NSUBV; ++c)
               tma_load_2d(sV + c * Cfg::SUB_BYTES + i * br * 128, &tmV, v_full, c * 64,
@@ -706,8 +711,12 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
     } else {
       tc_fence_after();
       float inv = l > 0.f ? 1.f / l : 0.f;
+      const __nv_bfloat16* grow = nullptr;     // this row's gates of every element
       if constexpr (EXT) {
-        if (args.gate && q_idx < T) {
+        inv *= args.out_scale;
+        if (args.gate && args.gate_elems) {
+          grow = args.gate + (size_t)(row_base + q_idx) * args.ldg + h * args.dv;
+        } else if (args.gate && q_idx < T) {
           const float gv = __bfloat162float(args.gate[(size_t)(row_base + q_idx) * args.ldg + h]);
           inv *= 1.f / (1.f + exp2f(-1.4426950408889634f * gv));
         }
@@ -724,6 +733,17 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
             if (EXT && c * 32 + q * 8 >= dv) break;
+            if constexpr (EXT) {
+              if (grow) {
+                const uint4 g4 = *reinterpret_cast<const uint4*>(grow + c * 32 + q * 8);
+                const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                  const float gv = __uint_as_float(j & 1 ? gw[j >> 1] & 0xffff0000u : gw[j >> 1] << 16);
+                  r[q * 8 + j] = __float_as_uint(__uint_as_float(r[q * 8 + j]) / (1.f + exp2f(-1.4426950408889634f * gv)));
+                }
+              }
+            }
             uint4 o;
             o.x = pack_bf16x2(__uint_as_float(r[q * 8 + 0]) * inv, __uint_as_float(r[q * 8 + 1]) * inv);
             o.y = pack_bf16x2(__uint_as_float(r[q * 8 + 2]) * inv, __uint_as_float(r[q * 8 + 3]) * inv);
@@ -852,26 +872,27 @@ BB_API int bb_flash_fwd_paged(const void* q, int ldq, const void* k_pool, const 
 }
 
 namespace bb {
-template <int HD, int HDV>
+template <int HD, int HDV, int WIN = 0>
 static int launch_paged_x(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const FaFwdArgs& a,
                           int n_tiles, cudaStream_t s) {
+  if (WIN == 0 && a.window > 0) return launch_paged_x<HD, HDV, 2>(tmQ, tmK, tmV, a, n_tiles, s);
   static PerDeviceOnce once;
-  const cudaError_t e = ensure_dyn_smem(once, fa_fwd2_kernel<HD, true, HDV, true>, FaFwdCfg<HD, HDV>::SMEM);
+  const cudaError_t e = ensure_dyn_smem(once, fa_fwd2_kernel<HD, true, HDV, true, WIN>, FaFwdCfg<HD, HDV>::SMEM);
   if (e != cudaSuccess) return (int)e;
-  fa_fwd2_kernel<HD, true, HDV, true><<<dim3(n_tiles, a.hq, 1), 192, FaFwdCfg<HD, HDV>::SMEM, s>>>(tmQ, tmK, tmV, a);
+  fa_fwd2_kernel<HD, true, HDV, true, WIN><<<dim3(n_tiles, a.hq, 1), 192, FaFwdCfg<HD, HDV>::SMEM, s>>>(tmQ, tmK, tmV, a);
   return (int)cudaGetLastError();
 }
 }  // namespace bb
 
 // The same for heads of their own sizes: query / key heads dq columns wide and value heads dv (multiples
 // of 8, up to 128; zero padding counts as columns), scores softcap tanh(scale q.k / softcap) when softcap
-// > 0, and an optional per-head output gate (sigmoid of gate[row, head]).  Pools: bf16
-// [pool_blocks][hk][block_rows][dq | dv].
+// > 0, an optional output gate (sigmoid of gate[row, head], or with gate_elems of gate[row, output column]), a
+// factor on the output, and a window of the latest keys (0: all).  Pools: bf16 [pool_blocks][hk][block_rows][dq | dv].
 BB_API int bb_flash_fwd_paged_x(const void* q, int ldq, const void* k_pool, const void* v_pool, void* out, int ldo,
                                 const int* block_tables, int max_blocks, int block_rows, int pool_blocks,
                                 const int* seq_row0, const int* seq_ctx, const int* tile_seq, const int* tile_qt,
                                 int n_tiles, int total_rows, int hq, int hk, int dq, int dv, float scale, float softcap,
-                                const void* gate, int ldg, void* stream) {
+                                const void* gate, int ldg, int gate_elems, float out_scale, int window, void* stream) {
   using namespace bb;
   if (n_tiles <= 0) return BB_OK;
   if (hq % hk || total_rows <= 0 || max_blocks <= 0 || pool_blocks <= 0) return BB_EARG;
@@ -904,6 +925,9 @@ BB_API int bb_flash_fwd_paged_x(const void* q, int ldq, const void* k_pool, cons
   }
   a.gate = static_cast<const __nv_bfloat16*>(gate);
   a.ldg = ldg;
+  a.gate_elems = gate_elems;
+  a.out_scale = out_scale;
+  a.window = window;
   CUtensorMap tmQ, tmK, tmV;
   const CUtensorMapDataType bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   int rc = make_tmap_2d(&tmQ, bf, 2, q, (uint64_t)hq * dq, (uint64_t)total_rows, (uint64_t)ldq * 2, 64, 128);
@@ -925,20 +949,20 @@ template <int HD, int HDV>
 static int launch_window(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const FaFwdArgs& a,
                          int n_tiles, cudaStream_t s) {
   static PerDeviceOnce once;
-  const cudaError_t e = ensure_dyn_smem(once, fa_fwd2_kernel<HD, true, HDV, true, true>, FaFwdCfg<HD, HDV>::SMEM);
+  const cudaError_t e = ensure_dyn_smem(once, fa_fwd2_kernel<HD, true, HDV, true, 1>, FaFwdCfg<HD, HDV>::SMEM);
   if (e != cudaSuccess) return (int)e;
-  fa_fwd2_kernel<HD, true, HDV, true, true><<<dim3(n_tiles, a.hq, 1), 192, FaFwdCfg<HD, HDV>::SMEM, s>>>(tmQ, tmK, tmV, a);
+  fa_fwd2_kernel<HD, true, HDV, true, 1><<<dim3(n_tiles, a.hq, 1), 192, FaFwdCfg<HD, HDV>::SMEM, s>>>(tmQ, tmK, tmV, a);
   return (int)cudaGetLastError();
 }
 }  // namespace bb
 
 // The same over keys and values that are rows of matrices of pitch ldkv (head h at columns h dq | h dv; kv_rows
 // rows): sequence s owns rows [kv_row0[s], kv_row0[s + 1]), the first of them at position kv_pos0[s]; a query
-// sees its `window` latest keys, itself included (0: all that are there).  Head sizes as above.
+// sees its `window` latest keys, itself included (0: all that are there).  Head sizes and per-head gate as above.
 BB_API int bb_flash_fwd_window(const void* q, int ldq, const void* k, const void* v, int ldkv, int kv_rows, void* out,
                                int ldo, const int* seq_row0, const int* kv_row0, const int* kv_pos0, const int* seq_ctx,
                                const int* tile_seq, const int* tile_qt, int n_tiles, int total_rows, int hq, int hk, int dq,
-                               int dv, float scale, int window, void* stream) {
+                               int dv, float scale, int window, const void* gate, int ldg, void* stream) {
   using namespace bb;
   if (n_tiles <= 0) return BB_OK;
   if (hq % hk || total_rows <= 0 || kv_rows <= 0 || window < 0) return BB_EARG;
@@ -960,6 +984,9 @@ BB_API int bb_flash_fwd_window(const void* q, int ldq, const void* k, const void
   a.kv_row0 = kv_row0;
   a.kv_pos0 = kv_pos0;
   a.window = window;
+  a.gate = static_cast<const __nv_bfloat16*>(gate);
+  a.ldg = ldg;
+  a.out_scale = 1.f;
   CUtensorMap tmQ, tmK, tmV;
   const CUtensorMapDataType bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   int rc = make_tmap_2d(&tmQ, bf, 2, q, (uint64_t)hq * dq, (uint64_t)total_rows, (uint64_t)ldq * 2, 64, 128);

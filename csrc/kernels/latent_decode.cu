@@ -26,6 +26,8 @@ struct LatDecArgs {
   __nv_bfloat16* out;          // [rows, ldo], head h at h kvrp (one key range)
   int ldo;
   float *part_o, *part_ml;     // [rows][heads][splits][kvrp | 2]
+  const __nv_bfloat16* gate;   // raw gate of row r, head h at gate[r ldg + h] (null: none)
+  int ldg;
   int* err;
 };
 
@@ -217,7 +219,8 @@ hy_latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
     } else {
       tc_fence_after();
       const bool one = a.splits == 1;
-      const float inv = one && l > 0.f ? 1.f / l : 1.f;
+      float inv = one && l > 0.f ? 1.f / l : 1.f;
+      if (one && a.gate && h < a.hq) inv *= sigmoid_as<__nv_bfloat16>(__bfloat162float(a.gate[(size_t)row * a.ldg + h]));
       const size_t part = ((size_t)row * a.hq + min(h, a.hq - 1)) * a.splits + split;
       if (!one && h < a.hq && vc == 0) {
         a.part_ml[part * 2] = m_ref;
@@ -257,7 +260,7 @@ hy_latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
 
 __global__ void __launch_bounds__(128)
 hy_latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, __nv_bfloat16* __restrict__ out,
-                       int ldo, int rows, int hq, int kvrp, int splits) {
+                       int ldo, int rows, int hq, int kvrp, int splits, const __nv_bfloat16* __restrict__ gate, int ldg) {
   const int vecs = kvrp / 8;
   const long t = (long)blockIdx.x * 128 + threadIdx.x;
   const long rh = t / vecs;
@@ -275,7 +278,8 @@ hy_latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict
 #pragma unroll
     for (int j = 0; j < 8; ++j) acc[j] = fmaf(w, f[j], acc[j]);
   }
-  const float inv = 1.f / l;
+  float inv = 1.f / l;
+  if (gate) inv *= sigmoid_as<__nv_bfloat16>(__bfloat162float(gate[(size_t)row * ldg + h]));
 #pragma unroll
   for (int j = 0; j < 8; ++j) acc[j] *= inv;
   store8(out + (size_t)row * ldo + h * kvrp + v, acc);
@@ -314,6 +318,8 @@ BB_API int bb_hy_latent_decode(const BbHyCfg* c, const BbHyLayer* L, const BbHyW
   a.ldo = w->ld_ol;
   a.part_o = w->part_o;
   a.part_ml = w->part_ml;
+  if (L->gate_kind == 1) a.gate = static_cast<const __nv_bfloat16*>(w->proj) + (size_t)b->n_pre * w->ld_proj + L->off_g;
+  a.ldg = w->ld_proj;
   a.err = device_error_word();
   // key ranges: enough CTAs to fill the machine, at most one per tile a query can see
   const int per_range = rows * a.vchunks * ((L->hq + 127) / 128);
@@ -340,7 +346,7 @@ BB_API int bb_hy_latent_decode(const BbHyCfg* c, const BbHyLayer* L, const BbHyW
   if (a.splits > 1) {
     const long t = (long)rows * L->hq * (L->kvrp / 8);
     hy_latent_merge_kernel<<<(int)((t + 127) / 128), 128, 0, s>>>(w->part_o, w->part_ml, a.out, w->ld_ol, rows, L->hq,
-                                                                  L->kvrp, a.splits);
+                                                                  L->kvrp, a.splits, a.gate, a.ldg);
   }
   return (int)cudaGetLastError();
 }

@@ -1,5 +1,5 @@
 // Latent attention, everything but its matrix products, for bf16 and fp32 storage:
-//   hy_latent_in     after the input projection: RMS norm of the query latent in place; the key/value latent
+//   hy_latent_in     after the input projection: RMS norm of the query latent (if any) in place; the key/value latent
 //                    (normed) and the shared rotated key part into the token's page row
 //   hy_latent_q      rotation of every head's rotated query part, in place for rows whose keys are multiplied
 //                    out, beside the absorbed query for the others
@@ -95,7 +95,7 @@ hy_latent_in_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, i
     sq += buf[0][i];
     sc += buf[1][i];
   }
-  const float rq = 1.f / sqrtf(sq / (float)L.qr + eps), rc = 1.f / sqrtf(sc / (float)L.kvr + eps);
+  const float rq = 1.f / sqrtf(sq / (float)max(L.qr, 1) + eps), rc = 1.f / sqrtf(sc / (float)L.kvr + eps);
   T* page = static_cast<T*>(L.kc) + ((size_t)blk * bs + pos % bs) * width;
   auto emit = [&](int i, float (&f)[8], bool first) {
     float g[8];
@@ -178,7 +178,7 @@ template <typename T, int V>
 __global__ void __launch_bounds__(LAT_THREADS)
 hy_latent_attn_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ qa, int ldq, T* __restrict__ out, int ldo,
                       const int* __restrict__ pos_, const int* __restrict__ row_seq, const int* __restrict__ tables,
-                      int max_blocks, int bs, int rows) {
+                      int max_blocks, int bs, int rows, const T* __restrict__ gate, int ldg) {
   const int w = (blockIdx.x * LAT_THREADS + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (w >= rows * L.hq) return;
   const int r = w / L.hq, h = w % L.hq, width = L.kvrp + L.rotp;
@@ -211,7 +211,8 @@ hy_latent_attn_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__
 #pragma unroll
     for (int i = 0; i < V; ++i) o[i] = fmaf(p, k[i], o[i] * al);
   }
-  const float f = 1.f / l;
+  float f = 1.f / l;
+  if (gate) f *= sigmoid_f(to_f(gate[(size_t)r * ldg + h]));
   T* dst = out + (size_t)r * ldo + h * L.kvrp;
 #pragma unroll
   for (int i = 0; i < V; ++i) {
@@ -224,11 +225,13 @@ template <typename T>
 static int launch_attn(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, int bs, int r0, int r1,
                        cudaStream_t s) {
   const int rows = r1 - r0, width = L.kvrp + L.rotp;
+  const T* gate = L.gate_kind == 1 ? static_cast<const T*>(w.proj) + (size_t)r0 * w.ld_proj + L.off_g : nullptr;
   const int grid = (int)(((long)rows * L.hq * 32 + LAT_THREADS - 1) / LAT_THREADS);
 #define BB_LAUNCH_LA(V)                                                                                            \
   hy_latent_attn_kernel<T, V><<<grid, LAT_THREADS, 0, s>>>(L, static_cast<const T*>(w.qa), w.ld_qa,                \
                                                            static_cast<T*>(w.ol), w.ld_ol, b.pos + r0,             \
-                                                           b.row_seq + r0, b.tables, b.max_blocks, bs, rows)
+                                                           b.row_seq + r0, b.tables, b.max_blocks, bs, rows, gate, \
+                                                           w.ld_proj)
   if (width <= 128) BB_LAUNCH_LA(4);
   else if (width <= 256) BB_LAUNCH_LA(8);
   else if (width <= 640) BB_LAUNCH_LA(20);
@@ -260,11 +263,13 @@ BB_API int bb_hy_latent_q(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* 
   const int step = (L->hq + LQ_HEADS - 1) / LQ_HEADS;
   const int lanes = step * (L->rotp / 8), t = lanes < LAT_THREADS ? (lanes + 31) & ~31 : LAT_THREADS;
   const dim3 grid(b->n, (lanes + t - 1) / t);
+  int ldq;
+  void* q = hy_latent_queries(*c, *L, *w, &ldq);
   if (c->dtype)
-    hy_latent_q_kernel<float><<<grid, t, 0, s>>>(*L, static_cast<float*>(w->q), w->ld_q, static_cast<float*>(w->qa), w->ld_qa,
-                                                 b->pos, n_in, step);
+    hy_latent_q_kernel<float><<<grid, t, 0, s>>>(*L, static_cast<float*>(q), ldq, static_cast<float*>(w->qa), w->ld_qa, b->pos,
+                                                 n_in, step);
   else
-    hy_latent_q_kernel<__nv_bfloat16><<<grid, t, 0, s>>>(*L, static_cast<__nv_bfloat16*>(w->q), w->ld_q,
+    hy_latent_q_kernel<__nv_bfloat16><<<grid, t, 0, s>>>(*L, static_cast<__nv_bfloat16*>(q), ldq,
                                                          static_cast<__nv_bfloat16*>(w->qa), w->ld_qa, b->pos, n_in, step);
   return (int)cudaGetLastError();
 }

@@ -178,10 +178,11 @@ __device__ __forceinline__ void cp_async_wait() {
 
 //
 // EXT: key and value heads of their own sizes (dk / dv columns in memory, multiples of 8, at most HD /
-// HDV) and soft-capped scores (x.cap_log2 tanh(x.cap_in q.k) in the log2 domain).
+// HDV), soft-capped scores (x.cap_log2 tanh(x.cap_in q.k) in the log2 domain), and a window of the latest keys.
 struct PdExt {
   int dk, dv;
   float cap_in, cap_log2;   // cap_log2 = 0: no cap
+  int window;               // 0: every key
 };
 template <int HD, int G, bool I8, int HDV = HD, bool EXT = false>
 __global__ void __launch_bounds__(128, 3)
@@ -221,8 +222,9 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
   const int grp = lane >> 3, sub = lane & 7;
   const int rowk = EXT ? x.dk * ES : ROWB, rowv = EXT ? x.dv * ES : ROWBV;   // bytes of a stored row
   const int S = seqlens[b];
-  const int per_split = ((S + splits - 1) / splits + 31) / 32 * 32;
-  const int k_begin = sp * per_split;
+  const int k_low = EXT && x.window > 0 ? max(S - x.window, 0) : 0;    // first key in the window
+  const int per_split = ((S - k_low + splits - 1) / splits + 31) / 32 * 32;
+  const int k_begin = k_low + sp * per_split;
   const int k_end = min(S, k_begin + per_split);
   const int nsteps = k_end > k_begin ? (k_end - k_begin + 15) >> 4 : 0;
   const int* bt = block_tables + (size_t)b * max_blocks;
@@ -504,9 +506,9 @@ __global__ void paged_decode_merge_kernel(const float* __restrict__ part_o,
                                           const float* __restrict__ part_ml,
                                           __nv_bfloat16* __restrict__ out, int ldo, int hq, int hd,
                                           int splits, int hd_out, const __nv_bfloat16* __restrict__ gate,
-                                          int ldg) {
+                                          int ldg, int gate_elems, float out_scale) {
   // hd: columns of a partial row; hd_out: columns of a head in the output; gate (may be null): raw
-  // per-head output gate, the head is multiplied by its sigmoid
+  // output gate (one per head, or with gate_elems one per output column), the output is multiplied by its sigmoid
   const int b = blockIdx.x, h = blockIdx.y;
   const size_t base = ((size_t)b * hq + h) * splits;
   float mm = -INFINITY;
@@ -516,14 +518,16 @@ __global__ void paged_decode_merge_kernel(const float* __restrict__ part_o,
     const float ms = part_ml[(base + s) * 2];
     ll += (ms == -INFINITY) ? 0.f : part_ml[(base + s) * 2 + 1] * exp2f(ms - mm);
   }
-  float inv = ll > 0.f ? 1.f / ll : 0.f;
-  if (gate) inv *= 1.f / (1.f + exp2f(-1.4426950408889634f * __bfloat162float(gate[(size_t)b * ldg + h])));
+  float inv = ll > 0.f ? out_scale / ll : 0.f;
+  if (gate && !gate_elems) inv *= 1.f / (1.f + exp2f(-1.4426950408889634f * __bfloat162float(gate[(size_t)b * ldg + h])));
   for (int c = threadIdx.x; c < hd_out; c += blockDim.x) {
     float acc = 0.f;
     for (int s = 0; s < splits; ++s) {
       const float ms = part_ml[(base + s) * 2];
       if (ms != -INFINITY) acc += part_o[(base + s) * hd + c] * exp2f(ms - mm);
     }
+    if (gate_elems)
+      acc *= 1.f / (1.f + exp2f(-1.4426950408889634f * __bfloat162float(gate[(size_t)b * ldg + h * hd_out + c])));
     out[(size_t)b * ldo + h * hd_out + c] = __float2bfloat16(acc * inv);
   }
 }
@@ -606,7 +610,7 @@ static int launch_paged_decode(bool i8, const void* q, int ldq, const void* kc, 
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
   paged_decode_merge_kernel<<<dim3(B, hq), 128, 0, s>>>(part_o, part_ml, (__nv_bfloat16*)out, ldo,
-                                                        hq, hd, splits, hd, nullptr, 0);
+                                                        hq, hd, splits, hd, nullptr, 0, 0, 1.f);
   return (int)cudaGetLastError();
 }
 
@@ -621,12 +625,12 @@ BB_API int bb_paged_decode(const void* q, int ldq, const void* kc, const void* v
 }
 
 // The same for key / value heads of their own sizes (dk / dv stored columns, multiples of 8, up to 128),
-// any number of query heads per kv head, scores softcap tanh(scale q.k / softcap) when softcap > 0, and
-// an optional output gate.  part_o: fp32 [B*hq*splits*(dv <= 64 ? 64 : 128)].
+// any number of query heads per kv head, scores softcap tanh(scale q.k / softcap) when softcap > 0, a window of the
+// latest keys (0: all), a factor on the output and an optional output gate (per head, or with gate_elems per element).  part_o: fp32 [B*hq*splits*(dv <= 64 ? 64 : 128)].
 BB_API int bb_paged_decode_x(const void* q, int ldq, const void* kc, const void* vc, const int* block_tables,
                              int max_blocks, const int* seqlens, void* out, int ldo, float* part_o, float* part_ml,
                              int B, int hq, int hk, int dk, int dv, int bs, int splits, float scale, float softcap,
-                             const void* gate, int ldg, void* stream) {
+                             const void* gate, int ldg, int gate_elems, float out_scale, int window, void* stream) {
   if (B <= 0) return BB_OK;
   if (hq % hk || splits < 1) return BB_EARG;
   if (dk % 8 || dv % 8 || dk > 128 || dv > 128 || ldq % 8) return BB_ESIZE;
@@ -634,7 +638,7 @@ BB_API int bb_paged_decode_x(const void* q, int ldq, const void* kc, const void*
   const int G = ratio % 4 == 0 ? 4 : (ratio % 3 == 0 ? 3 : (ratio % 2 == 0 ? 2 : 1));
   const int gsplit = ratio / G;
   dim3 grid(B, hk * gsplit, splits);
-  PdExt x{dk, dv, 0.f, 0.f};
+  PdExt x{dk, dv, 0.f, 0.f, window};
   float sl2 = scale * 1.4426950408889634f;
   if (softcap > 0.f) {
     sl2 = scale / softcap;     // the query is pre-scaled so that q.k is the argument of tanh
@@ -663,7 +667,8 @@ BB_API int bb_paged_decode_x(const void* q, int ldq, const void* kc, const void*
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
   paged_decode_merge_kernel<<<dim3(B, hq), 128, 0, s>>>(part_o, part_ml, (__nv_bfloat16*)out, ldo, hq,
-                                                        dv <= 64 ? 64 : 128, splits, dv, (const __nv_bfloat16*)gate, ldg);
+                                                        dv <= 64 ? 64 : 128, splits, dv, (const __nv_bfloat16*)gate, ldg,
+                                                        gate ? gate_elems : 0, out_scale);
   return (int)cudaGetLastError();
 }
 

@@ -37,12 +37,6 @@ __device__ __forceinline__ void store_pair(T* p, float a, float b) {
 }
 
 // Everything below is 32-bit; with bf16 storage exponentials and divisions are the hardware's (2^-22).
-template <typename T>
-__device__ __forceinline__ float gelu_as(float z) {
-  const float t = 0.79788456080286536f * fmaf(0.044715f * z * z, z, z);   // sqrt(2 / pi) (z + 0.044715 z^3)
-  if constexpr (sizeof(T) == 2) return z * rcp_hw(1.f + exp2_hw(-2.f * kLog2e * t));
-  else return 0.5f * z * (1.f + tanhf(t));
-}
 // e^-x - 1 for x >= 0
 template <typename T>
 __device__ __forceinline__ float decay_m1(float x) {

@@ -9,10 +9,16 @@ constexpr int SG_T = 64, SG_K = 16;
 
 __global__ void __launch_bounds__(256)
 sgemm_kernel(const float* __restrict__ A, const float* __restrict__ B, float* __restrict__ C, int M, int N, int K, int lda,
-             int ldb, int ldc, float alpha, int accumulate, size_t a_step, size_t b_step, size_t c_step) {
+             int ldb, int ldc, float alpha, int accumulate, size_t a_step, size_t b_step, size_t c_step,
+             const int* __restrict__ row_group) {
   A += blockIdx.z * a_step;
   B += blockIdx.z * b_step;
   C += blockIdx.z * c_step;
+  if (row_group) {                     // 128 rows share one of several B
+    const int g = row_group[blockIdx.y * SG_T / 128];
+    if (g < 0) return;
+    B += g * b_step;
+  }
   __shared__ float sa[SG_K][SG_T + 4], sb[SG_K][SG_T + 4];
   const int m0 = blockIdx.y * SG_T, n0 = blockIdx.x * SG_T;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
@@ -59,7 +65,7 @@ BB_API int bb_sgemm(const float* A, const float* B, float* C, int M, int N, int 
   using namespace bb;
   if (M <= 0 || N <= 0 || K <= 0) return BB_EARG;
   sgemm_kernel<<<dim3((N + SG_T - 1) / SG_T, (M + SG_T - 1) / SG_T), 256, 0, (cudaStream_t)stream>>>(
-      A, B, C, M, N, K, lda, ldb, ldc, alpha, accumulate, 0, 0, 0);
+      A, B, C, M, N, K, lda, ldb, ldc, alpha, accumulate, 0, 0, 0, nullptr);
   return (int)cudaGetLastError();
 }
 
@@ -70,6 +76,16 @@ BB_API int bb_sgemm_groups(const float* A, const float* B, float* C, int M, int 
   using namespace bb;
   if (M <= 0 || N <= 0 || K <= 0 || groups <= 0) return BB_EARG;
   sgemm_kernel<<<dim3((N + SG_T - 1) / SG_T, (M + SG_T - 1) / SG_T, groups), 256, 0, (cudaStream_t)stream>>>(
-      A, B, C, M, N, K, lda, K, ldc, 1.f, 0, a_step, (size_t)N * K, c_step);
+      A, B, C, M, N, K, lda, K, ldc, 1.f, 0, a_step, (size_t)N * K, c_step, nullptr);
+  return (int)cudaGetLastError();
+}
+
+// C = A B_g^T per 128 rows, g = tile_group[row / 128] (negative: skipped); B: [groups][N][K].
+BB_API int bb_sgemm_tiles(const float* A, const float* B, float* C, int M, int N, int K, int lda, int ldc, const int* tile_group,
+                          void* stream) {
+  using namespace bb;
+  if (M <= 0 || N <= 0 || K <= 0 || M % 128) return BB_EARG;
+  sgemm_kernel<<<dim3((N + SG_T - 1) / SG_T, M / SG_T), 256, 0, (cudaStream_t)stream>>>(A, B, C, M, N, K, lda, K, ldc, 1.f, 0, 0,
+                                                                                       (size_t)N * K, 0, tile_group);
   return (int)cudaGetLastError();
 }

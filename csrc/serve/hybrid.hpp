@@ -6,6 +6,7 @@
 // sections of a fused projection start on 16-byte boundaries and padded columns are zero throughout.
 // dtype 0: bf16 activations, weights and K/V pages; dtype 1: fp32 throughout.
 #pragma once
+#include <cstddef>
 #include <cstdint>
 
 struct BbHyLin {
@@ -14,7 +15,8 @@ struct BbHyLin {
 };
 
 struct BbHyLayer {
-  int kind;            // 0 attention, 1 mamba2, 2 latent attention, 3 generalised delta rule, 4 gated linear recurrence
+  int kind;            // 0 attention, 1 mamba2, 2 latent attention, 3 generalised delta rule, 4 gated linear recurrence,
+                       // 5 matrix memory (mLSTM)
   const float* norm;   // [dp] gain of the layer's norm (one already added where it is stored around 0)
   BbHyLin in;          // every projection that reads the normed input, stacked along the rows
   BbHyLin out;         // mixer output projection | feed-forward down projection, side by side
@@ -66,6 +68,30 @@ struct BbHyLayer {
   const float *y_b, *x_b;                  // [chp]
   const void* w_gate;                      // [blocks][2 bwp][bwp]: recurrence gate rows, then input gate rows
   const float *r_b, *i_b, *lam;            // [chp]; lam = decay constant times softplus of the parameter
+  // a second mixer that reads the same input; its output takes the columns of `cat` from its off_cat on
+  const BbHyLayer* beside;
+  int off_cat;
+  // attention: sigmoid gate at off_g (0 none, 1 one value per head, 2 one per element of the output), a factor
+  // on the output, biases [hq dkp] / [hk dkp] / [hk dvp] (null: none; q_norm and k_norm null: no norms)
+  int gate_kind;
+  float out_scale;
+  const float *q_b, *k_b, *v_b;
+  // feed-forward: 0 clamped gated unit, 1 gelu(gate) up; biases [ffp] (null: none; up_b as above)
+  int glu_kind;
+  const float* gate_b;
+  // products of the normed input that stay fp32: router logits, then the raw gates of a matrix memory
+  BbHyLin in32;
+  int off32_i, off32_f;
+  // matrix memory (heads of n query / key channels, padded np, and p value channels, padded pp): keys at
+  // off_kk, queries right behind them at off_q, values off_vv, output gate off_gg; i_b and f_b [heads].
+  // State [slots][heads][mem >= n p + n + 1, a multiple of 4]: matrix, normaliser, running maximum
+  int np, mem;
+  float gate_cap, q_scale;
+  const float* f_b;
+  // mixture of experts (n_experts = 0: none): [experts][gate effp | up effp][dp], [experts][dp][effp]
+  int n_experts, top, groups_all, groups_keep, eff, effp;
+  float route_scale, route_tiny, e_limit, e_alpha, e_shift;
+  const void *w_egu, *w_edown;
 };
 
 struct BbHyCfg {
@@ -75,6 +101,9 @@ struct BbHyCfg {
   const float *embed_norm, *final_norm;    // [dp]
   const void* head;                        // [vocabp, dp]
   const BbHyLayer* layers;
+  const void* pos;                         // [max positions, dp] added to the embedding (null: none)
+  int max_pos;
+  float embed_scale;
   int depth_avg;                           // layers pass on weighted sums of all results (see BbHyWork::x)
 };
 
@@ -115,4 +144,19 @@ struct BbHyWork {
   // their keys and values), and gate / decay projections of the recurrences
   void *h2, *q, *qa, *ol, *ckv, *kvx, *aux;
   int ld_q, ld_qa, ld_ol, ld_ckv, ld_kvx, ld_aux, exp_rows;
+  // fp32 products of the normed input; mixture of experts: rows sorted by expert, every expert's on 128-row
+  // tiles of their own (input, both halves, their product, output), and of every (token, choice) its expert, row
+  // and weight; rows of every expert; expert of every tile (-1: unused)
+  float* f32;                              // [rows, ld_f32]
+  void *ex_in, *ex_gu, *ex_act, *ex_out;   // [moe_rows, dp | ld_gu | ld_act | dp]
+  int *pair_expert, *pair_row;             // [rows top]
+  float* pair_w;
+  int *ex_count, *ex_tile;                 // [experts], [moe_rows / 128]
+  int ld_f32, ld_gu, ld_act, moe_rows;
 };
+
+// Rows and pitch of a latent attention layer's queries: through their own latent, or straight from the input.
+static inline void* hy_latent_queries(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, int* ld) {
+  *ld = L.uq.w ? w.ld_q : w.ld_proj;
+  return L.uq.w ? w.q : static_cast<char*>(w.proj) + (size_t)L.off_q * (c.dtype ? 4 : 2);
+}

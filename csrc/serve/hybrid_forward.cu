@@ -5,6 +5,9 @@
 //   -> mixer (attention over the pages, or the state-space recurrence over the slots)
 //   -> ONE output GEMM over (mixer output | feed-forward product), scaled and added into the fp32
 //      residual stream by its epilogue.
+// Designs with learned positions or routed experts start their layers in one kernel (hy_start): residual row, plus
+// the experts' outputs of the layer before, normed.  A layer may have two mixers side by side, and fp32 products of
+// its normed input (router logits, gates of a recurrence) beside the projection GEMM.
 // Designs with depth averages keep every layer's result: a layer starts from the weighted sum of all of them
 // (written where its own result will be, so the output GEMM adds in place), and its feed-forward has a norm
 // and a GEMM of its own.
@@ -51,17 +54,37 @@ int bb_sgemm_groups(const float* A, const float* B, float* C, int M, int N, int 
 int bb_flash_fwd_window(const void* q, int ldq, const void* k, const void* v, int ldkv, int kv_rows, void* out, int ldo,
                         const int* seq_row0, const int* kv_row0, const int* kv_pos0, const int* seq_ctx, const int* tile_seq,
                         const int* tile_qt, int n_tiles, int total_rows, int hq, int hk, int dq, int dv, float scale,
-                        int window, void* stream);
+                        int window, const void* gate, int ldg, void* stream);
 int bb_attn_rows(int dtype, const void* q, int ldq, const void* kc, const void* vc, const int* pos, const int* row_seq,
                  const int* tables, int max_blocks, int bs, void* out, int ldo, const void* gate, int ldg, int rows, int hq,
-                 int hk, int dk, int dv, int dkp, int dvp, float scale, float softcap, void* stream);
+                 int hk, int dk, int dv, int dkp, int dvp, float scale, float softcap, int gate_elems, float out_scale,
+                 int window, void* stream);
 int bb_flash_fwd_paged_x(const void* q, int ldq, const void* k_pool, const void* v_pool, void* out, int ldo,
                          const int* block_tables, int max_blocks, int block_rows, int pool_blocks, const int* seq_row0,
                          const int* seq_ctx, const int* tile_seq, const int* tile_qt, int n_tiles, int total_rows, int hq,
-                         int hk, int dq, int dv, float scale, float softcap, const void* gate, int ldg, void* stream);
+                         int hk, int dq, int dv, float scale, float softcap, const void* gate, int ldg, int gate_elems,
+                         float out_scale, int window, void* stream);
 int bb_paged_decode_x(const void* q, int ldq, const void* kc, const void* vc, const int* block_tables, int max_blocks,
                       const int* seqlens, void* out, int ldo, float* part_o, float* part_ml, int B, int hq, int hk, int dk,
-                      int dv, int bs, int splits, float scale, float softcap, const void* gate, int ldg, void* stream);
+                      int dv, int bs, int splits, float scale, float softcap, const void* gate, int ldg, int gate_elems,
+                      float out_scale, int window, void* stream);
+int bb_hy_start(const BbHyCfg* c, int li, const BbHyWork* w, const BbHyBatch* b, int all, float* trace, void* stream);
+int bb_hy_kv_post(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_glu(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream);
+int bb_hy_moe_tiles(const BbHyLayer* L, int n);
+int bb_hy_route(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream);
+int bb_hy_expert_rows(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream);
+int bb_hy_expert_glu(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream);
+int bb_hy_mlstm_gates(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream);
+int bb_hy_mlstm_scan(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int seq0, int n_seq,
+                     void* stream);
+int bb_hy_mlstm_decode(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_head_post(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int rows, void* stream);
+int bb_gemm_bf16_grouped(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc, int b_mn,
+                         int out_mode, int group_mode, const int* tile_group, int b_group_rows, int b_total_rows,
+                         const int* group_offsets, int num_groups, long c_group_stride, int bn, void* stream);
+int bb_sgemm_tiles(const float* A, const float* B, float* C, int M, int N, int K, int lda, int ldc, const int* tile_group,
+                   void* stream);
 }
 
 namespace {
@@ -105,39 +128,43 @@ const void* at(const BbHyCfg& c, const void* p, size_t elems) {
 void* at(const BbHyCfg& c, void* p, size_t elems) { return static_cast<char*>(p) + elems * (c.dtype ? 4 : 2); }
 
 int attention(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
-  BB_TRY(bb_hy_attn_post(&c, &L, &w, &b, s));
+  if (L.q_norm) BB_TRY(bb_hy_attn_post(&c, &L, &w, &b, s));
+  else BB_TRY(bb_hy_kv_post(&c, &L, &w, &b, s));
   const void* q = at(c, w.proj, L.off_q);
-  const void* gate = at(c, w.proj, L.off_g);
+  const void* gate = L.gate_kind ? at(c, w.proj, L.off_g) : nullptr;
+  const int elems = L.gate_kind == 2;
   const int n_dec = b.n - b.n_pre;
   if (b.n_pre > 0) {
     int rc = BB_ESIZE;
     if (!c.dtype)
       rc = bb_flash_fwd_paged_x(q, w.ld_proj, L.kc, L.vc, w.cat, w.ld_cat, b.tables, b.max_blocks, c.block_size,
                                 w.pool_blocks, b.seq_row0, b.seq_ctx, b.tile_seq, b.tile_qt, b.n_tiles, b.n_pre, L.hq, L.hk,
-                                L.dkp, L.dvp, L.scale, L.softcap, gate, w.ld_proj, s);
+                                L.dkp, L.dvp, L.scale, L.softcap, gate, w.ld_proj, elems, L.out_scale, L.window, s);
     if (rc == BB_ESIZE)
       rc = bb_attn_rows(c.dtype, q, w.ld_proj, L.kc, L.vc, b.pos, b.row_seq, b.tables, b.max_blocks, c.block_size, w.cat,
-                        w.ld_cat, gate, w.ld_proj, b.n_pre, L.hq, L.hk, L.dk, L.dv, L.dkp, L.dvp, L.scale, L.softcap, s);
+                        w.ld_cat, gate, w.ld_proj, b.n_pre, L.hq, L.hk, L.dk, L.dv, L.dkp, L.dvp, L.scale, L.softcap, elems,
+                        L.out_scale, L.window, s);
     if (rc) return rc;
   }
   if (n_dec > 0) {
     const void* qd = at(c, q, (size_t)b.n_pre * w.ld_proj);
-    const void* gd = at(c, gate, (size_t)b.n_pre * w.ld_proj);
+    const void* gd = gate ? at(c, gate, (size_t)b.n_pre * w.ld_proj) : nullptr;
     void* od = at(c, w.cat, (size_t)b.n_pre * w.ld_cat);
     int rc = BB_ESIZE;
     if (!c.dtype) {
       // K/V splits: enough blocks to fill the machine, at most what the partial buffers were sized for
       const int base = n_dec * L.hk;
       int splits = (4 * sm_count() + base - 1) / base;
+      if (L.window > 0 && splits > (L.window + 31) / 32) splits = (L.window + 31) / 32;
       splits = splits < 1 ? 1 : (splits > w.splits ? w.splits : splits);
       rc = bb_paged_decode_x(qd, w.ld_proj, L.kc, L.vc, b.tables + (size_t)b.ns_pre * b.max_blocks, b.max_blocks,
                              b.seq_ctx + b.ns_pre, od, w.ld_cat, w.part_o, w.part_ml, n_dec, L.hq, L.hk, L.dkp, L.dvp,
-                             c.block_size, splits, L.scale, L.softcap, gd, w.ld_proj, s);
+                             c.block_size, splits, L.scale, L.softcap, gd, w.ld_proj, elems, L.out_scale, L.window, s);
     }
     if (rc == BB_ESIZE)
       rc = bb_attn_rows(c.dtype, qd, w.ld_proj, L.kc, L.vc, b.pos + b.n_pre, b.row_seq + b.n_pre, b.tables, b.max_blocks,
                         c.block_size, od, w.ld_cat, gd, w.ld_proj, n_dec, L.hq, L.hk, L.dk, L.dv, L.dkp, L.dvp, L.scale,
-                        L.softcap, s);
+                        L.softcap, elems, L.out_scale, L.window, s);
     if (rc) return rc;
   }
   return BB_OK;
@@ -161,18 +188,19 @@ int latent_attention(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, co
   const int dq = L.dkp + L.rotp, width = L.kvrp + L.rotp;
   const int n_in = L.expand.w ? b.n_pre : 0;
   BB_TRY(bb_hy_latent_in(&c, &L, &w, &b, s));
-  BB_TRY(project(c, L.uq, at(c, w.proj, L.off_dq), w.ld_proj, w.q, w.ld_q, b.n, s));
+  if (L.uq.w) BB_TRY(project(c, L.uq, at(c, w.proj, L.off_dq), w.ld_proj, w.q, w.ld_q, b.n, s));
+  int ldq;
+  void* q = hy_latent_queries(c, L, w, &ldq);
   BB_TRY(bb_hy_latent_q(&c, &L, &w, &b, n_in, s));
   if (n_in > 0) {
     BB_TRY(bb_hy_latent_gather(&c, &L, &w, &b, s));
     BB_TRY(project(c, L.expand, w.ckv, w.ld_ckv, w.kvx, w.ld_kvx, b.n_exp, s));
-    BB_TRY(bb_flash_fwd_window(w.q, w.ld_q, w.kvx, at(c, w.kvx, (size_t)L.hq * dq), w.ld_kvx, b.n_exp, w.cat, w.ld_cat,
+    BB_TRY(bb_flash_fwd_window(q, ldq, w.kvx, at(c, w.kvx, (size_t)L.hq * dq), w.ld_kvx, b.n_exp, w.cat, w.ld_cat,
                                b.seq_row0, b.kv_row0, b.kv_pos0, b.seq_ctx, b.tile_seq, b.tile_qt, b.n_tiles, b.n_pre, L.hq,
-                               L.hq, dq, L.dvp, L.scale, L.window, s));
+                               L.hq, dq, L.dvp, L.scale, L.window, L.gate_kind == 1 ? at(c, w.proj, L.off_g) : nullptr, w.ld_proj, s));
   }
   const int rows = b.n - n_in;
-  BB_TRY(project_groups(c, L.w_abs, L.hq, L.kvrp, L.dkp, at(c, w.q, (size_t)n_in * w.ld_q), w.ld_q, dq, w.qa, w.ld_qa, width,
-                        rows, s));
+  BB_TRY(project_groups(c, L.w_abs, L.hq, L.kvrp, L.dkp, at(c, q, (size_t)n_in * ldq), ldq, dq, w.qa, w.ld_qa, width, rows, s));
   const int rc = bb_hy_latent_decode(&c, &L, &w, &b, b.n_pre - n_in, s);
   if (rc == BB_OK && n_in < b.n_pre) BB_TRY(bb_hy_latent_attn(&c, &L, &w, &b, n_in, b.n_pre, s));
   else if (rc == BB_ESIZE) BB_TRY(bb_hy_latent_attn(&c, &L, &w, &b, n_in, b.n, s));
@@ -193,6 +221,19 @@ int rglru(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBat
   return bb_hy_rglru(&c, &L, &w, &b, s);
 }
 
+int mlstm(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
+  int post = b.n_pre;                    // rows whose outputs are still to be normed and gated
+  BB_TRY(bb_hy_mlstm_scan(&c, &L, &w, &b, 0, b.ns_pre, s));
+  const int rc = bb_hy_mlstm_decode(&c, &L, &w, &b, s);
+  if (rc == BB_ESIZE) {
+    BB_TRY(bb_hy_mlstm_scan(&c, &L, &w, &b, b.ns_pre, b.ns - b.ns_pre, s));
+    post = b.n;
+  } else if (rc) {
+    return rc;
+  }
+  return bb_hy_head_post(&c, &L, &w, post, s);
+}
+
 int mixer(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
   switch (L.kind) {
     case 0: return attention(c, L, w, b, s);
@@ -200,6 +241,7 @@ int mixer(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBat
     case 2: return latent_attention(c, L, w, b, s);
     case 3: return general_delta(c, L, w, b, s);
     case 4: return rglru(c, L, w, b, s);
+    case 5: return mlstm(c, L, w, b, s);
     default: return BB_EARG;
   }
 }
@@ -210,7 +252,7 @@ constexpr int BESIDE_ROWS = 256;
 
 struct SideStream {
   cudaStream_t s = nullptr;
-  cudaEvent_t fork = nullptr, join = nullptr;
+  cudaEvent_t fork = nullptr, join = nullptr, ready = nullptr;
 };
 SideStream* side_stream() {
   static SideStream per_device[64];
@@ -221,6 +263,7 @@ SideStream* side_stream() {
   SideStream& d = per_device[dev];
   if (!d.s && (cudaEventCreateWithFlags(&d.fork, cudaEventDisableTiming) != cudaSuccess ||
                cudaEventCreateWithFlags(&d.join, cudaEventDisableTiming) != cudaSuccess ||
+               cudaEventCreateWithFlags(&d.ready, cudaEventDisableTiming) != cudaSuccess ||
                cudaStreamCreateWithFlags(&d.s, cudaStreamNonBlocking) != cudaSuccess))
     return nullptr;
   return &d;
@@ -264,14 +307,74 @@ int forward_depth(const BbHyCfg& c, const BbHyWork& w, const BbHyBatch& b, float
   return bb_hy_mix_norm(&c, c.n_layers, &w, &b, nullptr, s);
 }
 
+// y = x W_g^T per 128-row tile of the experts' rows
+int project_tiles(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const void* weights, int n, int k, const void* x, int ldx,
+                  void* y, int ldy, int tiles, void* s) {
+  if (c.dtype)
+    return bb_sgemm_tiles(static_cast<const float*>(x), static_cast<const float*>(weights), static_cast<float*>(y), tiles * 128, n, k,
+                          ldx, ldy, w.ex_tile, s);
+  // tile width: enough tiles to fill the machine
+  const int sms = sm_count();
+  const int bn = n >= 256 && tiles * ((n + 255) / 256) >= sms ? 256 : (n >= 128 && tiles * ((n + 127) / 128) >= sms / 2 ? 128 : 64);
+  return bb_gemm_bf16_grouped(x, weights, y, tiles * 128, n, k, ldx, k, ldy, 0, 0, 1, w.ex_tile, n, L.n_experts * n, nullptr, 0, 0, bn,
+                              s);
+}
+
+// Router logits in w.f32 -> the experts' outputs in w.ex_out, weights and rows of every token's choices
+int experts(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
+  const int tiles = bb_hy_moe_tiles(&L, b.n);
+  BB_TRY(bb_hy_route(&c, &L, &w, b.n, s));
+  BB_TRY(bb_hy_expert_rows(&c, &L, &w, b.n, s));
+  BB_TRY(project_tiles(c, L, w, L.w_egu, 2 * L.effp, c.dp, w.ex_in, c.dp, w.ex_gu, w.ld_gu, tiles, s));
+  BB_TRY(bb_hy_expert_glu(&c, &L, &w, b.n, s));
+  return project_tiles(c, L, w, L.w_edown, c.dp, L.effp, w.ex_act, w.ld_act, w.ex_out, c.dp, tiles, s);
+}
+
+// Layers that hy_start begins.  In small steps the fp32 products and the experts run beside the mixer.
+int forward_start(const BbHyCfg& c, const BbHyWork& w, const BbHyBatch& b, float* trace, void* s) {
+  SideStream* side = b.n <= BESIDE_ROWS ? side_stream() : nullptr;
+  const cudaStream_t main = (cudaStream_t)s;
+  const size_t level = (size_t)b.n * c.dp;
+  if (trace && b.n_want < b.n) return BB_EARG;       // the last layer's trace goes through the wanted rows' buffer
+  for (int li = 0; li < c.n_layers; ++li) {
+    const BbHyLayer& L = c.layers[li];
+    BB_TRY(bb_hy_start(&c, li, &w, &b, 0, trace && li ? trace + (li - 1) * level : nullptr, s));
+    const bool fork = side && L.n_experts > 0;
+    void* t = s;
+    if (fork) {
+      t = side->s;
+      BB_CUDA(cudaEventRecord(side->fork, main));
+      BB_CUDA(cudaStreamWaitEvent(side->s, side->fork, 0));
+    }
+    if (L.in32.w) BB_TRY(project_f32(c, L.in32, w.h, c.dp, w.f32, w.ld_f32, b.n, 1.f, 0, t));
+    const bool gates = L.kind == 5 || (L.beside && L.beside->kind == 5);
+    if (fork && gates) BB_CUDA(cudaEventRecord(side->ready, side->s));
+    if (L.n_experts > 0) BB_TRY(experts(c, L, w, b, t));
+    if (fork) BB_CUDA(cudaEventRecord(side->join, side->s));
+    BB_TRY(project(c, L.in, w.h, c.dp, w.proj, w.ld_proj, b.n, s));
+    if (fork && gates) BB_CUDA(cudaStreamWaitEvent(main, side->ready, 0));
+    BB_TRY(mixer(c, L, w, b, s));
+    if (L.beside) {
+      BbHyWork v = w;
+      v.cat = at(c, w.cat, L.beside->off_cat);
+      BB_TRY(mixer(c, *L.beside, v, b, s));
+    }
+    if (L.kind != 0 && L.ff > 0) BB_TRY(bb_hy_glu(&c, &L, &w, b.n, s));
+    BB_TRY(project_f32(c, L.out, w.cat, w.ld_cat, w.x, c.dp, b.n, c.residual_mult, 1, s));
+    if (fork) BB_CUDA(cudaStreamWaitEvent(main, side->join, 0));
+  }
+  if (trace) BB_TRY(bb_hy_start(&c, c.n_layers, &w, &b, 1, trace + (c.n_layers - 1) * level, s));
+  return bb_hy_start(&c, c.n_layers, &w, &b, 0, nullptr, s);
+}
+
 }  // namespace
 
 // One step.  Logits land in w->logits [n_want, vocabp]; `trace` (may be null): fp32 [n_layers][n][dp]
 // copies of the residual stream after every layer.
 BB_API int bb_hybrid_forward(const BbHyCfg* c, const BbHyWork* w, const BbHyBatch* b, float* trace, void* stream) {
   if (!c || !w || !b || b->n <= 0 || b->n > w->rows || b->n_want > w->want_rows) return BB_EARG;
-  if (c->depth_avg) {
-    BB_TRY(forward_depth(*c, *w, *b, trace, stream));
+  if (c->depth_avg || !c->embed_norm) {
+    BB_TRY(c->depth_avg ? forward_depth(*c, *w, *b, trace, stream) : forward_start(*c, *w, *b, trace, stream));
     if (b->n_want <= 0) return BB_OK;
     const BbHyLin head{c->head, c->vocabp, c->dp};
     return project_f32(*c, head, w->hn, c->dp, w->logits, c->vocabp, b->n_want, 1.f, 0, stream);

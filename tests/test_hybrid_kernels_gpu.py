@@ -93,12 +93,12 @@ def test_prefill_attention(shape, loud, softcap):
             tiles = [(s, t) for s in range(4) for t in range(-(-lens[s] // 128))]
             call("flash_fwd_paged_x", dq, dq.stride(0), kc, vc, out, out.stride(0), tables, mb, BS, kc.shape[0],
                  i32(np.concatenate([[0], np.cumsum(lens)]).tolist()), i32(ctx), i32([t[0] for t in tiles]),
-                 i32([t[1] for t in tiles]), len(tiles), n, hq, hk, dk, dv, scale, softcap, dg, ldg, stream_ptr())
+                 i32([t[1] for t in tiles]), len(tiles), n, hq, hk, dk, dv, scale, softcap, dg, ldg, 0, 1.0, 0, stream_ptr())
         else:
             pos = np.concatenate([np.arange(s, s + l) for s, l in zip(starts, lens)])
             seq = np.repeat(np.arange(4), lens)
             call("attn_rows", 1, dq, dq.stride(0), kc, vc, i32(pos.tolist()), i32(seq.tolist()), tables, mb, BS, out,
-                 out.stride(0), dg, ldg, n, hq, hk, dk, dv, dk, dv, scale, softcap, stream_ptr())
+                 out.stride(0), dg, ldg, n, hq, hk, dk, dv, dk, dv, scale, softcap, 0, 1.0, 0, stream_ptr())
         check_error()
         got = out.cpu().float()
         assert bool((got[:, hq * dv:] == 7.0).all())
@@ -135,10 +135,10 @@ def test_decode_attention(shape, splits, softcap):
                 po = torch.empty(B * hq * splits * (64 if dv <= 64 else 128), device="cuda")
                 pm = torch.empty(B * hq * splits * 2, device="cuda")
                 call("paged_decode_x", dq, dq.stride(0), kc, vc, tables, mb, i32(ctx), out, out.stride(0), po, pm, B, hq,
-                     hk, dk, dv, BS, splits, scale, softcap, dg, 16, stream_ptr())
+                     hk, dk, dv, BS, splits, scale, softcap, dg, 16, 0, 1.0, 0, stream_ptr())
             else:
                 call("attn_rows", 1, dq, dq.stride(0), kc, vc, i32(starts), i32(list(range(B))), tables, mb, BS, out,
-                     out.stride(0), dg, 16, B, hq, hk, dk, dv, dk, dv, scale, softcap, stream_ptr())
+                     out.stride(0), dg, 16, B, hq, hk, dk, dv, dk, dv, scale, softcap, 0, 1.0, 0, stream_ptr())
             check_error()
             got = out.cpu()
             for s in range(B):

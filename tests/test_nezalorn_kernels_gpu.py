@@ -58,7 +58,7 @@ def test_windowed_prefill_attention(hq, dq, dv, window):
     tiles = [(s, t) for s in range(4) for t in range(-(-lens[s] // 128))]
     call("flash_fwd_window", qb, qb.stride(0), kb, kb[:, hq * dq:], ldkv, kb.shape[0], out, out.stride(0),
          i32(np.concatenate([[0], np.cumsum(lens)])), i32(kv0), i32(lo), i32(ctx), i32([t[0] for t in tiles]),
-         i32([t[1] for t in tiles]), len(tiles), n, hq, hq, dq, dv, scale, window, stream_ptr())
+         i32([t[1] for t in tiles]), len(tiles), n, hq, hq, dq, dv, scale, window, None, 0, stream_ptr())
     check_error()
     got, qf, kf = out.cpu().double(), qb.cpu().double(), kb.cpu().double()
     assert bool((got[:, hq * dv:] == 7.0).all())
