@@ -88,8 +88,9 @@ class _Scratch:
                 po, pm = max(po, n * l.kvrp), max(pm, n * 2)
         self.part_o, self.part_ml = z(po, dtype=f32), z(pm, dtype=f32)
         # segment states of the chunked recurrence (prompt portions): two machine-fulls of states
-        npmax = max([l.n * l.p for l in eng.mixers if l.kind == 1], default=0)
-        self.seg = z(2 * 2 * eng.sm_count * (npmax + 1) if portions and not eng.fp32 and 0 < npmax <= 128 * 128 else 1, dtype=f32)
+        npmax = max([l.mem if l.kind == 5 else l.n * l.p for l in eng.mixers if l.kind in (1, 5) and max(l.n, l.p) <= 128],
+                    default=0)
+        self.seg = z(2 * 2 * eng.sm_count * (npmax + 1) if portions and not eng.fp32 and npmax else 1, dtype=f32)
         self.hn, self.logits = z(max(want, 1), eng.dp), z(max(want, 1), eng.vocabp, dtype=f32)
         w = self.work = hn.Work()
         for n in ("x", "h", "proj", "cat", "xbc", "dt", "y", "v_first", "part_o", "part_ml", "seg", "hn", "logits", "h2", "q",

@@ -79,6 +79,7 @@ int bb_hy_mlstm_gates(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, i
 int bb_hy_mlstm_scan(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int seq0, int n_seq,
                      void* stream);
 int bb_hy_mlstm_decode(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_mlstm_chunk(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
 int bb_hy_head_post(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int rows, void* stream);
 int bb_gemm_bf16_grouped(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc, int b_mn,
                          int out_mode, int group_mode, const int* tile_group, int b_group_rows, int b_total_rows,
@@ -222,16 +223,18 @@ int rglru(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBat
 }
 
 int mlstm(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
-  int post = b.n_pre;                    // rows whose outputs are still to be normed and gated
-  BB_TRY(bb_hy_mlstm_scan(&c, &L, &w, &b, 0, b.ns_pre, s));
-  const int rc = bb_hy_mlstm_decode(&c, &L, &w, &b, s);
-  if (rc == BB_ESIZE) {
-    BB_TRY(bb_hy_mlstm_scan(&c, &L, &w, &b, b.ns_pre, b.ns - b.ns_pre, s));
-    post = b.n;
-  } else if (rc) {
-    return rc;
+  int first = 0, rows = b.n_pre;         // sequences left to the scan; rows whose outputs are still to be normed and gated
+  if (b.n_pre > 0 && !c.dtype && L.np <= 128 && L.pp <= 128) {
+    BB_TRY(bb_hy_mlstm_gates(&c, &L, &w, b.n_pre, s));
+    BB_TRY(bb_mlstm_chunk(&c, &L, &w, &b, s));
+    first = b.ns_pre;
+    rows = 0;
   }
-  return bb_hy_head_post(&c, &L, &w, post, s);
+  const int rc = bb_hy_mlstm_decode(&c, &L, &w, &b, s);
+  if (rc == BB_ESIZE) rows = b.n;
+  else if (rc) return rc;
+  BB_TRY(bb_hy_mlstm_scan(&c, &L, &w, &b, first, (rc == BB_ESIZE ? b.ns : b.ns_pre) - first, s));
+  return bb_hy_head_post(&c, &L, &w, rows, s);
 }
 
 int mixer(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
