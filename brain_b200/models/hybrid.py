@@ -39,21 +39,25 @@ class HybridDecoder(nn.Module):
         """Random values at which every mechanism works in its usual range: projections that keep the
         scale of their input, norm gains near their neutral value, step sizes between 1e-3 and 1e-1, decay
         rates between 1 and 16."""
-        g = torch.Generator().manual_seed(seed)
+        dev = next(self.parameters()).device
+        g = torch.Generator(dev).manual_seed(seed)
 
         def uniform(shape, lo, hi):
-            return torch.rand(shape, generator=g) * (hi - lo) + lo
+            return torch.rand(shape, generator=g, device=dev) * (hi - lo) + lo
+
+        def normal(shape):
+            return torch.randn(shape, generator=g, device=dev)
 
         for name, shape in self.cfg.tensors():
             p = self.tensor(name)
             leaf = name.split(".", 2)[-1] if name[0] == "l" and name[1].isdigit() else name
             leaf = leaf.removeprefix("left.").removeprefix("right.")
             if leaf in ("embed.norm", "final.norm") or name.endswith((".norm1", ".norm2")):
-                v = 1.0 - self.cfg.traits.norm_offset + 0.1 * torch.randn(shape, generator=g)
+                v = 1.0 - self.cfg.traits.norm_offset + 0.1 * normal(shape)
             elif leaf in ("q.norm", "k.norm", "norm", "dq.norm", "dkv.norm"):
-                v = 1.0 + 0.1 * torch.randn(shape, generator=g)
+                v = 1.0 + 0.1 * normal(shape)
             elif name.endswith(".dwa"):
-                v = 0.2 * torch.randn(shape, generator=g) / shape[0]     # mostly the layer's own result
+                v = 0.2 * normal(shape) / shape[0]     # mostly the layer's own result
                 v[-1] += 1.0
             elif leaf == "act":
                 v = uniform(shape, 0.2, 0.8)
@@ -81,11 +85,11 @@ class HybridDecoder(nn.Module):
             elif leaf == "conv.b":
                 v = uniform(shape, -0.1, 0.1)
             elif name == "embed":
-                v = torch.randn(shape, generator=g) / self.cfg.embed_scale
+                v = normal(shape) / self.cfg.embed_scale
             elif name == "pos":
-                v = 0.3 * torch.randn(shape, generator=g)
+                v = 0.3 * normal(shape)
             else:
-                v = torch.randn(shape, generator=g) / math.sqrt(shape[-1])
+                v = normal(shape) / math.sqrt(shape[-1])
             p.copy_(v.to(p.dtype))
         return self
 

@@ -303,15 +303,55 @@ def run(size: str = "m", steps: int = 10, kernels: bool = True, n_seq: int = 4, 
     return res
 
 
-def steps(portion: int, seqs: int, ctx: int, n: int = 3, size: str = "m") -> None:
-    """``n`` equal steps of a two-layer model (one layer of each kind): prompts of ``portion`` tokens, or one
-    token each (``portion`` 1), at position ``ctx``.  A small program to put under a profiler."""
+def compare(size: str, shape: dict, designs, steps: int = 10, with_kernels: bool = True, n_seq: int = 4, T: int = 2048,
+            B: int = 64, ctx: int = 2048) -> dict:
+    """Throughput and kernel tables of hybrid decoders of equal size; ``designs``: (name, configuration, kernel table)."""
     from ..models.hybrid import HybridDecoder
     from ..ops import _cuda
     from ..serve.engine import make_engine
     from ..serve.hybrid import Entry
-    s = dict(SIZES[size], pairs=1, vocab=1024)
-    model = HybridDecoder(hybrid_config(s)).init_weights(0).to("cuda", torch.bfloat16)
+    root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+    try:
+        peaks = json.load(open(os.path.join(root, "MEASURED_PEAKS.json")))
+    except OSError:
+        peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+    vocab = SIZES[size]["vocab"]
+    blocks = max(n_seq * -(-T // 16), B * -(-(ctx + 16) // 16))
+    res = {"size": size, "shape": shape, "prefill_tokens_per_s": {}, "decode_tokens_per_s": {}, "kernels": {}}
+    timer = KernelTimer() if with_kernels else None
+    rng = np.random.default_rng(1)
+    launches0 = _cuda.launch_count
+    for name, cfg, table in designs:
+        with torch.device("cuda"):
+            model = HybridDecoder(cfg).to(torch.bfloat16).init_weights(0)
+        eng = make_engine(model, block_size=16, num_blocks=blocks, max_seq_len=-(-(max(T, ctx) + 16) // 16) * 16,
+                          max_prefill=T, max_batch=B)
+        del model
+        pre, dec = throughput(eng, n_seq, T, B, ctx, steps, vocab)
+        res["prefill_tokens_per_s"][name], res["decode_tokens_per_s"][name] = round(pre), round(dec)
+        if with_kernels:
+            per = -(-T // 16)
+            ent = [Entry(rng.integers(0, vocab, T), 0, np.arange(i * per, (i + 1) * per), i, [T - 1]) for i in range(n_seq)]
+            rows = table(eng, ent, "prefill", timer, peaks)
+            per = -(-(ctx + 1) // 16)
+            ent = [Entry(rng.integers(0, vocab, 1), ctx, np.arange(i * per, (i + 1) * per), i, [0]) for i in range(B)]
+            res["kernels"][name] = rows + table(eng, ent, "decode", timer, peaks)
+        _cuda.check_error()
+        del eng
+        torch.cuda.empty_cache()
+    res["gpu_launches"] = _cuda.launch_count - launches0
+    return res
+
+
+def equal_steps(cfg, portion: int, seqs: int, ctx: int, n: int) -> None:
+    """``n`` steps of ``seqs`` prompts of ``portion`` tokens each at position ``ctx``, for a profiler."""
+    from ..models.hybrid import HybridDecoder
+    from ..ops import _cuda
+    from ..serve.engine import make_engine
+    from ..serve.hybrid import Entry
+    cfg.vocab = 1024
+    with torch.device("cuda"):
+        model = HybridDecoder(cfg).to(torch.bfloat16).init_weights(0)
     per = (portion + ctx) // 16 + 1
     eng = make_engine(model, max_batch=seqs, block_size=16, num_blocks=seqs * per, max_seq_len=portion + ctx + 16,
                       max_prefill=portion)
@@ -322,6 +362,12 @@ def steps(portion: int, seqs: int, ctx: int, n: int = 3, size: str = "m") -> Non
     torch.cuda.synchronize()
     _cuda.check_error()
     print("ok")
+
+
+def steps(portion: int, seqs: int, ctx: int, n: int = 3, size: str = "m") -> None:
+    """``n`` equal steps of a two-layer model (one layer of each kind): prompts of ``portion`` tokens, or one
+    token each (``portion`` 1), at position ``ctx``.  A small program to put under a profiler."""
+    equal_steps(hybrid_config(dict(SIZES[size], pairs=1)), portion, seqs, ctx, n)
 
 
 if __name__ == "__main__":

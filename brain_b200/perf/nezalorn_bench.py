@@ -5,11 +5,6 @@ Throughput and kernels as in ``hybrid_bench``; each kernel names the other decod
 from __future__ import annotations
 
 import ctypes as C
-import json
-import os
-
-import numpy as np
-import torch
 
 from . import hybrid_bench as hb
 
@@ -141,65 +136,17 @@ def kernels(eng, entries, phase, timer, peaks):
     return out
 
 
-def run(size: str = "m", steps: int = 10, with_kernels: bool = True, n_seq: int = 4, T: int = 2048, B: int = 64,
-        ctx: int = 2048) -> dict:
-    from ..models.hybrid import HybridDecoder
-    from ..ops import _cuda
-    from ..serve.engine import make_engine
-    from ..serve.hybrid import Entry
-    root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
-    try:
-        peaks = json.load(open(os.path.join(root, "MEASURED_PEAKS.json")))
-    except OSError:
-        peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
-    vocab = hb.SIZES[size]["vocab"]
-    blocks = max(n_seq * -(-T // 16), B * -(-(ctx + 16) // 16))
-    shape = dict(SIZES[size], width=hb.SIZES[size]["width"], ff=hb.SIZES[size]["ff"] * 3 // 2, layers=2 * hb.SIZES[size]["pairs"])
-    res = {"size": size, "shape": shape, "prefill_tokens_per_s": {}, "decode_tokens_per_s": {}, "kernels": {}}
-    timer = hb.KernelTimer() if with_kernels else None
-    rng = np.random.default_rng(1)
-    launches0 = _cuda.launch_count
-    for name, cfg, table in (("nezalorn", config(size), kernels), ("pakalix", hb.hybrid_config(hb.SIZES[size]), hb.hybrid_kernels)):
-        model = HybridDecoder(cfg).init_weights(0).to("cuda", torch.bfloat16)
-        eng = make_engine(model, block_size=16, num_blocks=blocks, max_seq_len=-(-(max(T, ctx) + 16) // 16) * 16,
-                          max_prefill=T, max_batch=B)
-        del model
-        pre, dec = hb.throughput(eng, n_seq, T, B, ctx, steps, vocab)
-        res["prefill_tokens_per_s"][name], res["decode_tokens_per_s"][name] = round(pre), round(dec)
-        if with_kernels:
-            per = -(-T // 16)
-            ent = [Entry(rng.integers(0, vocab, T), 0, np.arange(i * per, (i + 1) * per), i, [T - 1]) for i in range(n_seq)]
-            rows = table(eng, ent, "prefill", timer, peaks)
-            per = -(-(ctx + 1) // 16)
-            ent = [Entry(rng.integers(0, vocab, 1), ctx, np.arange(i * per, (i + 1) * per), i, [0]) for i in range(B)]
-            res["kernels"][name] = rows + table(eng, ent, "decode", timer, peaks)
-        _cuda.check_error()
-        del eng
-        torch.cuda.empty_cache()
-    res["gpu_launches"] = _cuda.launch_count - launches0
-    return res
+def run(size: str = "m", steps: int = 10, with_kernels: bool = True, **kw) -> dict:
+    base = hb.SIZES[size]
+    shape = dict(SIZES[size], width=base["width"], ff=base["ff"] * 3 // 2, layers=2 * base["pairs"])
+    return hb.compare(size, shape, (("nezalorn", config(size), kernels), ("pakalix", hb.hybrid_config(base), hb.hybrid_kernels)),
+                      steps, with_kernels, **kw)
 
 
 def steps(portion: int, seqs: int, ctx: int, n: int = 3, size: str = "m") -> None:
     """``n`` equal steps of a four-layer model: prompts of ``portion`` tokens, or one token each (``portion`` 1), at
     position ``ctx``.  A small program to put under a profiler."""
-    from ..models.hybrid import HybridDecoder
-    from ..ops import _cuda
-    from ..serve.engine import make_engine
-    from ..serve.hybrid import Entry
-    cfg = config(size, layers=4)
-    cfg.vocab = 1024
-    model = HybridDecoder(cfg).init_weights(0).to("cuda", torch.bfloat16)
-    per = (portion + ctx) // 16 + 1
-    eng = make_engine(model, max_batch=seqs, block_size=16, num_blocks=seqs * per, max_seq_len=portion + ctx + 16,
-                      max_prefill=portion)
-    rng = np.random.default_rng(0)
-    for _ in range(n):
-        eng.step_logits([Entry(rng.integers(0, 1024, portion), ctx, np.arange(i * per, (i + 1) * per), i, [portion - 1])
-                         for i in range(seqs)])
-    torch.cuda.synchronize()
-    _cuda.check_error()
-    print("ok")
+    hb.equal_steps(config(size, layers=4), portion, seqs, ctx, n)
 
 
 if __name__ == "__main__":
