@@ -86,7 +86,9 @@ def kernels(eng, entries, phase, timer, peaks):
     row("sum of experts, norm", us, "norm", n * d * (4 + 4 + 2 + 2 * alone.top) / 1e9)
     for tag, l in (("both", both), ("memory", alone), ("latent", lat)):
         gemm(f"{tag}: input projections", "input projections", at("h"), d, l.inp, at("proj"), ld["proj"])
-    gemm("router and gates (fp32)", "input projections", at("h"), d, alone.in32, P(sc.f32.data_ptr()), ld["f32"], mode=1)
+    few = n <= 128
+    if not few:
+        gemm("router and gates (fp32)", "input projections", at("h"), d, alone.in32, P(sc.f32.data_ptr()), ld["f32"], mode=1)
     for tag, l in (("both", both), ("memory", alone), ("latent", lat)):
         gemm(f"{tag}: output projections + residual", "output projections", at("cat"), ld["cat"], l.out, P(sc.x.data_ptr()), d,
              mode=2)
@@ -98,10 +100,12 @@ def kernels(eng, entries, phase, timer, peaks):
     reset()
 
     def route():
-        rc = lib.bb_hy_route(cfg, le, w, n, stream_ptr())
+        rc = (lib.bb_hy_route_row if few else lib.bb_hy_route)(cfg, le, w, n, stream_ptr())
         assert rc == 0
     both_us = timer(lambda: (reset(), route()))
-    row("experts: routing", max(both_us - timer(reset), 0.1), "attention post", n * (alone.n_experts * 4 + alone.top * 12) / 1e9)
+    extra = (alone.in32.n + n) * d * 2 if few else 0
+    row("router and gates (fp32), routing" if few else "experts: routing", max(both_us - timer(reset), 0.1),
+        "input projections" if few else "attention post", (n * (alone.n_experts * 4 + alone.top * 12) + extra) / 1e9)
     rows_ = sc.pair_row.clone()
     reset()
     route()

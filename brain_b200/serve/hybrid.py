@@ -77,7 +77,7 @@ class _Scratch:
         self.pair_expert, self.pair_row = (z(max(rows * top, 1), dtype=i32) for _ in range(2))
         self.pair_w = z(max(rows * top, 1), dtype=f32)
         self.ex_count = z(max((l.n_experts for l in routed), default=1), dtype=i32)
-        self.ex_tile = z(max(moe // 128, 1), dtype=i32)
+        self.ex_tile = z(max(moe // 64, 1), dtype=i32)
         po = pm = 1
         for l in eng.mixers:
             if l.kind == 0 and dec and not eng.fp32:

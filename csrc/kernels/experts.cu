@@ -1,6 +1,7 @@
 // Mixture of experts of a serving step, everything but its matrix products, for bf16 and fp32 storage:
 //   hy_route         one warp per token: softmax over the router's fp32 logits, the best groups by their best
 //                    expert, the best experts of those, their weights; a place among the rows of each
+//   hy_route_row     few rows: the same behind the fp32 products themselves, one block per row
 //   hy_expert_rows   rows of the normed input to their experts' places, every expert's rows on 128-row tiles of
 //                    their own; the tiles' experts
 //   hy_expert_glu    clamped gated product of the experts' two halves
@@ -13,7 +14,7 @@
 
 namespace bb {
 
-constexpr int EX_THREADS = 256, EX_TOKENS = 4;   // tokens of a warp
+constexpr int EX_THREADS = 256;
 
 // Largest value of the warp and the lowest index that has it, in every lane.
 __device__ __forceinline__ void warp_best(float& v, int& i) {
@@ -28,94 +29,171 @@ __device__ __forceinline__ void warp_best(float& v, int& i) {
   }
 }
 
-// V: experts of a lane (expert j * 32 + lane).
+// The choices of one token by one warp: lane c < top gets the c-th expert and its weight.  V: experts of a lane
+// (expert j * 32 + lane).
 template <int V>
-__global__ void __launch_bounds__(EX_THREADS)
-hy_route_kernel(const __grid_constant__ BbHyLayer L, const float* __restrict__ logits, int ld, int* __restrict__ pair_expert,
-                int* __restrict__ pair_row, float* __restrict__ pair_w, int* __restrict__ count, int n, int tokens) {
-  __shared__ int hist[V * 32];
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, E = L.n_experts, size = E / L.groups_all;
-  for (int e = threadIdx.x; e < E; e += EX_THREADS) hist[e] = 0;
-  __syncthreads();
-  const int t0 = (blockIdx.x * (EX_THREADS / 32) + warp) * tokens;
-  for (int t = t0; t < min(t0 + tokens, n); ++t) {
-    float s[V], mx = -INFINITY, sum = 0.f;
+__device__ __forceinline__ void choose(const BbHyLayer& L, const float* logits, int& my_e, float& my_w) {
+  const int lane = threadIdx.x & 31, E = L.n_experts, size = E / L.groups_all;
+  float s[V], mx = -INFINITY, sum = 0.f;
+#pragma unroll
+  for (int j = 0; j < V; ++j) {
+    s[j] = j * 32 + lane < E ? logits[j * 32 + lane] : -INFINITY;
+    mx = fmaxf(mx, s[j]);
+  }
+  mx = warp_max(mx);
+#pragma unroll
+  for (int j = 0; j < V; ++j) {
+    s[j] = j * 32 + lane < E ? expf(s[j] - mx) : 0.f;
+    sum += s[j];
+  }
+  const float inv = 1.f / warp_sum(sum);
+#pragma unroll
+  for (int j = 0; j < V; ++j) s[j] *= inv;
+  // groups: take the best expert left in any group not yet kept, keep its group
+  bool kept[V];
+#pragma unroll
+  for (int j = 0; j < V; ++j) kept[j] = L.groups_keep >= L.groups_all;
+  auto best_of = [&](bool in, int& bi) {
+    float best = -1.f;
+    bi = 0x7fffffff;
 #pragma unroll
     for (int j = 0; j < V; ++j) {
-      s[j] = j * 32 + lane < E ? logits[(size_t)t * ld + j * 32 + lane] : -INFINITY;
-      mx = fmaxf(mx, s[j]);
-    }
-    mx = warp_max(mx);
-#pragma unroll
-    for (int j = 0; j < V; ++j) {
-      s[j] = j * 32 + lane < E ? expf(s[j] - mx) : 0.f;
-      sum += s[j];
-    }
-    const float inv = 1.f / warp_sum(sum);
-#pragma unroll
-    for (int j = 0; j < V; ++j) s[j] *= inv;
-    // groups: take the best expert left in any group not yet kept, keep its group
-    unsigned kept[V];        // bit: the expert's group is kept (an expert's own bit only)
-#pragma unroll
-    for (int j = 0; j < V; ++j) kept[j] = L.groups_keep >= L.groups_all;
-    if (L.groups_keep < L.groups_all) {
-      for (int g = 0; g < L.groups_keep; ++g) {
-        float best = -1.f;
-        int bi = 0x7fffffff;
-#pragma unroll
-        for (int j = 0; j < V; ++j) {
-          const int e = j * 32 + lane;
-          if (e < E && !kept[j] && s[j] > best) {
-            best = s[j];
-            bi = e;
-          }
-        }
-        warp_best(best, bi);
-        const int first = bi / size * size;
-#pragma unroll
-        for (int j = 0; j < V; ++j) {
-          const int e = j * 32 + lane;
-          if (e >= first && e < first + size) kept[j] = 1;
-        }
+      const int e = j * 32 + lane;
+      if (e < E && kept[j] == in && s[j] > best) {
+        best = s[j];
+        bi = e;
       }
     }
-    float total = 0.f, my_w = 0.f;
-    int my_e = 0;
-    for (int c = 0; c < L.top; ++c) {
-      float best = -1.f;
-      int bi = 0x7fffffff;
+    warp_best(best, bi);
+    return best;
+  };
+  if (L.groups_keep < L.groups_all)
+    for (int g = 0; g < L.groups_keep; ++g) {
+      int bi;
+      best_of(false, bi);
+      const int first = bi / size * size;
 #pragma unroll
       for (int j = 0; j < V; ++j) {
         const int e = j * 32 + lane;
-        if (e < E && kept[j] && s[j] > best) {
-          best = s[j];
-          bi = e;
-        }
-      }
-      warp_best(best, bi);
-#pragma unroll
-      for (int j = 0; j < V; ++j)
-        if (j * 32 + lane == bi) kept[j] = 0;
-      total += best;
-      if (lane == c) {
-        my_w = best;
-        my_e = bi;
+        if (e >= first && e < first + size) kept[j] = true;
       }
     }
-    if (lane < L.top) {
-      const size_t p = (size_t)t * L.top + lane;
-      my_e = min(my_e, E - 1);                     // (logits that are not numbers pick no expert)
-      pair_expert[p] = my_e;
-      pair_row[p] = atomicAdd(&hist[my_e], 1);     // place among the block's rows of this expert
-      pair_w[p] = my_w / (total + L.route_tiny) * L.route_scale;
+  float total = 0.f;
+  my_w = 0.f;
+  my_e = 0;
+  for (int c = 0; c < L.top; ++c) {
+    int bi;
+    const float best = best_of(true, bi);
+#pragma unroll
+    for (int j = 0; j < V; ++j)
+      if (j * 32 + lane == bi) kept[j] = false;
+    total += best;
+    if (lane == c) {
+      my_w = best;
+      my_e = min(bi, E - 1);                       // (logits that are not numbers pick no expert)
+    }
+  }
+  my_w = my_w / (total + L.route_tiny) * L.route_scale;
+}
+
+template <int V>
+__global__ void __launch_bounds__(EX_THREADS)
+hy_route_kernel(const __grid_constant__ BbHyLayer L, const float* __restrict__ logits, int ld, int* __restrict__ pair_expert,
+                int* __restrict__ pair_row, float* __restrict__ pair_w, int* __restrict__ count, int n) {
+  __shared__ int hist[V * 32];
+  const int lane = threadIdx.x & 31, E = L.n_experts, t = blockIdx.x * (EX_THREADS / 32) + (threadIdx.x >> 5);
+  for (int e = threadIdx.x; e < E; e += EX_THREADS) hist[e] = 0;
+  __syncthreads();
+  const bool mine = t < n && lane < L.top;
+  const size_t p = (size_t)t * L.top + lane;
+  int e = 0, place = 0;
+  if (t < n) {
+    float w;
+    choose<V>(L, logits + (size_t)t * ld, e, w);
+    if (mine) {
+      pair_expert[p] = e;
+      pair_w[p] = w;
+      place = atomicAdd(&hist[e], 1);              // place among the block's rows of this expert
     }
   }
   __syncthreads();
-  for (int e = threadIdx.x; e < E; e += EX_THREADS)
-    if (hist[e] > 0) hist[e] = atomicAdd(&count[e], hist[e]);   // ... and the block's first place among all
+  for (int i = threadIdx.x; i < E; i += EX_THREADS)
+    if (hist[i] > 0) hist[i] = atomicAdd(&count[i], hist[i]);   // ... and the block's first place among all
   __syncthreads();
-  const size_t p1 = (size_t)min(t0 + tokens, n) * L.top;
-  for (size_t p = (size_t)t0 * L.top + lane; p < p1; p += 32) pair_row[p] += hist[pair_expert[p]];
+  if (mine) pair_row[p] = hist[e] + place;
+}
+
+// Few rows: one block per row computes the fp32 products of the normed input (router logits, gates) and routes.
+// V = 0: nothing to route.
+constexpr int RR_THREADS = 512;
+
+template <typename T, int V>
+__global__ void __launch_bounds__(RR_THREADS)
+hy_route_row_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ h, int dp, float* __restrict__ out, int ld,
+                    int* __restrict__ pair_expert, int* __restrict__ pair_row, float* __restrict__ pair_w, int* __restrict__ count) {
+  extern __shared__ __align__(16) float s_h[];     // the row, then the products
+  float* s_out = s_h + dp;
+  const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_out = L.in32.n;
+  struct alignas(sizeof(T) * 8) Raw {
+    T v[8];
+  };
+  const T* W = static_cast<const T*>(L.in32.w);
+  // outputs of a warp at a time (n_out is a multiple of 8), vectors of each asked for together
+  constexpr int O = 4, U = sizeof(T) == 2 ? 4 : 2, STEP = 256 * U;
+  Raw w[U][O];
+  auto fetch = [&](int o, int i0) {
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+#pragma unroll
+      for (int q = 0; q < O; ++q)
+        if (i0 + u * 256 < dp) w[u][q] = *reinterpret_cast<const Raw*>(W + (size_t)(o + q) * dp + i0 + u * 256);
+  };
+  const int o0 = warp * O;
+  if (o0 < n_out) fetch(o0, lane * 8);             // on their way while the row is
+  for (int i = threadIdx.x * 8; i < dp; i += RR_THREADS * 8) {
+    float f[8];
+    load8(h + (size_t)r * dp + i, f);
+    store8(s_h + i, f);
+  }
+  __syncthreads();
+  for (int o = o0; o < n_out; o += RR_THREADS / 32 * O) {
+    float a[O] = {};
+    for (int i0 = lane * 8; i0 < dp; i0 += STEP) {
+      if (o != o0 || i0 >= 256) fetch(o, i0);
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        if (i0 + u * 256 >= dp) break;
+        float x[8];
+        load8(s_h + i0 + u * 256, x);
+#pragma unroll
+        for (int q = 0; q < O; ++q)
+#pragma unroll
+          for (int j = 0; j < 8; ++j) a[q] = fmaf(to_f(w[u][q].v[j]), x[j], a[q]);
+      }
+    }
+#pragma unroll
+    for (int q = 0; q < O; ++q) {
+      a[q] = warp_sum(a[q]);
+      if (lane == q) {
+        s_out[o + q] = a[q];
+        out[(size_t)r * ld + o + q] = a[q];
+      }
+    }
+  }
+  if constexpr (V > 0) {
+    __syncthreads();
+    if (warp == 0) {
+      int e;
+      float w;
+      choose<V>(L, s_out, e, w);
+      if (lane < L.top) {
+        const size_t p = (size_t)r * L.top + lane;
+        pair_expert[p] = e;
+        pair_w[p] = w;
+        pair_row[p] = atomicAdd(&count[e], 1);
+      }
+    }
+  }
 }
 
 // Every expert's first row, from the counts: rows of expert e start on a 128-row tile.
@@ -138,12 +216,12 @@ __device__ __forceinline__ void expert_offsets(const int* count, int E, int* off
   __syncthreads();
 }
 
-// A warp per token; the last block writes the tiles' experts.
+// A warp per token; the last block writes every tile's expert and, cap entries further, how many rows it has.
 template <typename T>
 __global__ void __launch_bounds__(EX_THREADS)
 hy_expert_rows_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ h, int dp, const int* __restrict__ pair_expert,
                       int* __restrict__ pair_row, const int* __restrict__ count, T* __restrict__ out, int* __restrict__ tiles,
-                      int n_tiles, int n) {
+                      int n_tiles, int cap, int n) {
   extern __shared__ int off[];
   const int E = L.n_experts;
   expert_offsets(count, E, off);
@@ -159,6 +237,7 @@ hy_expert_rows_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__
         e = lo;
       }
       tiles[t] = e;
+      tiles[cap + t] = e < 0 ? 0 : min(count[e] - (t * 128 - off[e]), 128);
     }
     return;
   }
@@ -193,10 +272,9 @@ hy_expert_rows_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__
 template <typename T>
 __global__ void __launch_bounds__(EX_THREADS)
 hy_expert_glu_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ gu, int ldgu, T* __restrict__ act, int lda,
-                     const int* __restrict__ tiles, int tile_blocks) {
+                     const int* __restrict__ tile_rows, int tile_blocks) {
   const int tile = blockIdx.x / tile_blocks;
-  if (tiles[tile] < 0) return;
-  const int vecs = L.effp / 8, total = 128 * vecs, stride = tile_blocks * EX_THREADS;
+  const int vecs = L.effp / 8, total = tile_rows[tile] * vecs, stride = tile_blocks * EX_THREADS;
   for (int i = (blockIdx.x % tile_blocks) * EX_THREADS + threadIdx.x; i < total; i += stride) {
     const size_t r = (size_t)tile * 128 + i / vecs;
     const int c = i % vecs * 8;
@@ -226,10 +304,9 @@ BB_API int bb_hy_route(const BbHyCfg*, const BbHyLayer* L, const BbHyWork* w, in
   const int E = L->n_experts;
   if (E > 1024 || L->top > 32) return BB_ESIZE;
   cudaStream_t s = (cudaStream_t)stream;
-  const int warps = EX_THREADS / 32, tokens = n >= 148 * warps * EX_TOKENS ? EX_TOKENS : 1;
-  const int grid = (n + warps * tokens - 1) / (warps * tokens);
+  const int grid = (n + EX_THREADS / 32 - 1) / (EX_THREADS / 32);
 #define BB_ROUTE(V) \
-  hy_route_kernel<V><<<grid, EX_THREADS, 0, s>>>(*L, w->f32, w->ld_f32, w->pair_expert, w->pair_row, w->pair_w, w->ex_count, n, tokens)
+  hy_route_kernel<V><<<grid, EX_THREADS, 0, s>>>(*L, w->f32, w->ld_f32, w->pair_expert, w->pair_row, w->pair_w, w->ex_count, n)
   if (E <= 32) BB_ROUTE(1);
   else if (E <= 64) BB_ROUTE(2);
   else if (E <= 128) BB_ROUTE(4);
@@ -237,6 +314,33 @@ BB_API int bb_hy_route(const BbHyCfg*, const BbHyLayer* L, const BbHyWork* w, in
   else BB_ROUTE(32);
 #undef BB_ROUTE
   return (int)cudaGetLastError();
+}
+
+namespace bb {
+template <typename T>
+static int launch_route_row(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, int n, cudaStream_t s) {
+  const int E = L.n_experts;
+  const size_t smem = 4 * ((size_t)c.dp + L.in32.n);
+  if (smem > 48 * 1024 || E > 256 || L.top > 32) return BB_ESIZE;
+#define BB_ROUTE_ROW(V)                                                                                                     \
+  hy_route_row_kernel<T, V><<<n, RR_THREADS, smem, s>>>(L, static_cast<const T*>(w.h), c.dp, w.f32, w.ld_f32, w.pair_expert, \
+                                                        w.pair_row, w.pair_w, w.ex_count)
+  if (E == 0) BB_ROUTE_ROW(0);
+  else if (E <= 32) BB_ROUTE_ROW(1);
+  else if (E <= 64) BB_ROUTE_ROW(2);
+  else if (E <= 128) BB_ROUTE_ROW(4);
+  else BB_ROUTE_ROW(8);
+#undef BB_ROUTE_ROW
+  return (int)cudaGetLastError();
+}
+}  // namespace bb
+
+// The fp32 products of the normed input -> w->f32, and with experts the routing; for few rows.  BB_ESIZE for rows or
+// expert counts it does not cover.
+BB_API int bb_hy_route_row(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream) {
+  if (n <= 0) return BB_OK;
+  return c->dtype ? launch_route_row<float>(*c, *L, *w, n, (cudaStream_t)stream)
+                  : launch_route_row<__nv_bfloat16>(*c, *L, *w, n, (cudaStream_t)stream);
 }
 
 BB_API int bb_hy_expert_rows(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream) {
@@ -247,24 +351,25 @@ BB_API int bb_hy_expert_rows(const BbHyCfg* c, const BbHyLayer* L, const BbHyWor
   const size_t smem = 4 * (size_t)(L->n_experts + 1);
   if (c->dtype)
     hy_expert_rows_kernel<float><<<grid, EX_THREADS, smem, s>>>(*L, static_cast<const float*>(w->h), c->dp, w->pair_expert, w->pair_row,
-                                                                w->ex_count, static_cast<float*>(w->ex_in), w->ex_tile, tiles, n);
+                                                                w->ex_count, static_cast<float*>(w->ex_in), w->ex_tile, tiles, w->moe_rows / 128, n);
   else
     hy_expert_rows_kernel<__nv_bfloat16><<<grid, EX_THREADS, smem, s>>>(*L, static_cast<const __nv_bfloat16*>(w->h), c->dp,
                                                                         w->pair_expert, w->pair_row, w->ex_count,
-                                                                        static_cast<__nv_bfloat16*>(w->ex_in), w->ex_tile, tiles, n);
+                                                                        static_cast<__nv_bfloat16*>(w->ex_in), w->ex_tile, tiles, w->moe_rows / 128, n);
   return (int)cudaGetLastError();
 }
 
 BB_API int bb_hy_expert_glu(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream) {
   if (n <= 0) return BB_OK;
   cudaStream_t s = (cudaStream_t)stream;
+  const int* rows = w->ex_tile + w->moe_rows / 128;
   const int tiles = moe_tiles(*L, n), per = (128 * (L->effp / 8) + 4 * EX_THREADS - 1) / (4 * EX_THREADS);
   if (c->dtype)
     hy_expert_glu_kernel<float><<<tiles * per, EX_THREADS, 0, s>>>(*L, static_cast<const float*>(w->ex_gu), w->ld_gu,
-                                                                   static_cast<float*>(w->ex_act), w->ld_act, w->ex_tile, per);
+                                                                   static_cast<float*>(w->ex_act), w->ld_act, rows, per);
   else
     hy_expert_glu_kernel<__nv_bfloat16><<<tiles * per, EX_THREADS, 0, s>>>(*L, static_cast<const __nv_bfloat16*>(w->ex_gu), w->ld_gu,
-                                                                           static_cast<__nv_bfloat16*>(w->ex_act), w->ld_act,
-                                                                           w->ex_tile, per);
+                                                                           static_cast<__nv_bfloat16*>(w->ex_act), w->ld_act, rows,
+                                                                           per);
   return (int)cudaGetLastError();
 }

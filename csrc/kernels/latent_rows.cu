@@ -44,14 +44,17 @@ __device__ __forceinline__ void rotate_pairs8(float (&f)[8], const Angles4& a) {
   }
 }
 
-// A thread's vectors of the row (query latent, then page row) stay in registers up to KEEP of them.
-template <typename T>
+// A thread's vectors of the row (query latent, then page row) stay in registers up to KEEP of them.  TPR threads share
+// a row: the block, or a warp where rows are short.
+template <typename T, int TPR>
 __global__ void __launch_bounds__(LAT_THREADS, sizeof(T) == 2 ? 10 : 6)
 hy_latent_in_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, int ld, const int* __restrict__ pos_,
-                    const int* __restrict__ row_seq, const int* __restrict__ tables, int max_blocks, int bs, float eps) {
+                    const int* __restrict__ row_seq, const int* __restrict__ tables, int max_blocks, int bs, float eps, int rows) {
   constexpr int KEEP = 2;
   __shared__ float buf[2][32];
-  const int r = blockIdx.x, width = L.kvrp + L.rotp, n = L.qrp + (L.own_kv ? width : 0);
+  const int tid = threadIdx.x % TPR, r = blockIdx.x * (LAT_THREADS / TPR) + threadIdx.x / TPR;
+  if (r >= rows) return;
+  const int width = L.kvrp + L.rotp, n = L.qrp + (L.own_kv ? width : 0);
   T* q = proj + (size_t)r * ld + L.off_dq;
   const T* c = proj + (size_t)r * ld + L.off_ckv;
   const int pos = pos_[r];
@@ -65,18 +68,18 @@ hy_latent_in_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, i
   };
 #pragma unroll
   for (int t = 0; t < KEEP; ++t) {
-    const int i = (threadIdx.x + t * LAT_THREADS) * 8;
+    const int i = (tid + t * TPR) * 8;
     if (i < n) load8(i < L.qrp ? q + i : c + (i - L.qrp), v[t]);
   }
   // the first vector's gains are asked for before the sums are known
   auto gains = [&](int i) { return i < L.qrp ? L.dq_norm + i : L.dkv_norm + (i - L.qrp); };
-  if (threadIdx.x * 8 < min(n, L.qrp + L.kvrp)) load8(gains(threadIdx.x * 8), gain);
+  if (tid * 8 < min(n, L.qrp + L.kvrp)) load8(gains(tid * 8), gain);
 #pragma unroll
   for (int t = 0; t < KEEP; ++t) {
-    const int i = (threadIdx.x + t * LAT_THREADS) * 8;
+    const int i = (tid + t * TPR) * 8;
     if (i < n) sum(i, v[t]);
   }
-  for (int i = (threadIdx.x + KEEP * LAT_THREADS) * 8; i < n; i += LAT_THREADS * 8) {
+  for (int i = (tid + KEEP * TPR) * 8; i < n; i += TPR * 8) {
     float f[8];
     load8(i < L.qrp ? q + i : c + (i - L.qrp), f);
     sum(i, f);
@@ -84,16 +87,18 @@ hy_latent_in_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, i
   const int blk = L.own_kv ? tables[(size_t)row_seq[r] * max_blocks + pos / bs] : 0;
   sq = warp_sum(sq);
   sc = warp_sum(sc);
-  if ((threadIdx.x & 31) == 0) {
-    buf[0][threadIdx.x >> 5] = sq;
-    buf[1][threadIdx.x >> 5] = sc;
-  }
-  __syncthreads();
-  sq = sc = 0.f;
+  if constexpr (TPR > 32) {
+    if ((threadIdx.x & 31) == 0) {
+      buf[0][threadIdx.x >> 5] = sq;
+      buf[1][threadIdx.x >> 5] = sc;
+    }
+    __syncthreads();
+    sq = sc = 0.f;
 #pragma unroll
-  for (int i = 0; i < LAT_THREADS / 32; ++i) {
-    sq += buf[0][i];
-    sc += buf[1][i];
+    for (int i = 0; i < LAT_THREADS / 32; ++i) {
+      sq += buf[0][i];
+      sc += buf[1][i];
+    }
   }
   const float rq = 1.f / sqrtf(sq / (float)max(L.qr, 1) + eps), rc = 1.f / sqrtf(sc / (float)L.kvr + eps);
   T* page = static_cast<T*>(L.kc) + ((size_t)blk * bs + pos % bs) * width;
@@ -125,10 +130,10 @@ hy_latent_in_kernel(const __grid_constant__ BbHyLayer L, T* __restrict__ proj, i
   };
 #pragma unroll
   for (int t = 0; t < KEEP; ++t) {
-    const int i = (threadIdx.x + t * LAT_THREADS) * 8;
+    const int i = (tid + t * TPR) * 8;
     if (i < n) emit(i, v[t], t == 0);
   }
-  for (int i = (threadIdx.x + KEEP * LAT_THREADS) * 8; i < n; i += LAT_THREADS * 8) {
+  for (int i = (tid + KEEP * TPR) * 8; i < n; i += TPR * 8) {
     float f[8];
     load8(i < L.qrp ? q + i : c + (i - L.qrp), f);
     emit(i, f, false);
@@ -247,13 +252,19 @@ using namespace bb;
 
 BB_API int bb_hy_latent_in(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream) {
   cudaStream_t s = (cudaStream_t)stream;
-  if (c->dtype)
-    hy_latent_in_kernel<float><<<b->n, LAT_THREADS, 0, s>>>(*L, static_cast<float*>(w->proj), w->ld_proj, b->pos, b->row_seq,
-                                                            b->tables, b->max_blocks, c->block_size, c->eps);
-  else
-    hy_latent_in_kernel<__nv_bfloat16><<<b->n, LAT_THREADS, 0, s>>>(*L, static_cast<__nv_bfloat16*>(w->proj), w->ld_proj,
-                                                                    b->pos, b->row_seq, b->tables, b->max_blocks,
-                                                                    c->block_size, c->eps);
+  const bool small = L->qrp + (L->own_kv ? L->kvrp + L->rotp : 0) <= 2 * 32 * 8;
+  const int grid = small ? (b->n + LAT_THREADS / 32 - 1) / (LAT_THREADS / 32) : b->n;
+#define BB_LAT_IN(T, TPR)                                                                                                    \
+  hy_latent_in_kernel<T, TPR><<<grid, LAT_THREADS, 0, s>>>(*L, static_cast<T*>(w->proj), w->ld_proj, b->pos, b->row_seq,     \
+                                                           b->tables, b->max_blocks, c->block_size, c->eps, b->n)
+  if (c->dtype) {
+    if (small) BB_LAT_IN(float, 32);
+    else BB_LAT_IN(float, LAT_THREADS);
+  } else {
+    if (small) BB_LAT_IN(__nv_bfloat16, 32);
+    else BB_LAT_IN(__nv_bfloat16, LAT_THREADS);
+  }
+#undef BB_LAT_IN
   return (int)cudaGetLastError();
 }
 

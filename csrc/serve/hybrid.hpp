@@ -146,12 +146,12 @@ struct BbHyWork {
   int ld_q, ld_qa, ld_ol, ld_ckv, ld_kvx, ld_aux, exp_rows;
   // fp32 products of the normed input; mixture of experts: rows sorted by expert, every expert's on 128-row
   // tiles of their own (input, both halves, their product, output), and of every (token, choice) its expert, row
-  // and weight; rows of every expert; expert of every tile (-1: unused)
+  // and weight; rows of every expert; expert of every tile (-1: unused), then how many rows every tile has
   float* f32;                              // [rows, ld_f32]
   void *ex_in, *ex_gu, *ex_act, *ex_out;   // [moe_rows, dp | ld_gu | ld_act | dp]
   int *pair_expert, *pair_row;             // [rows top]
   float* pair_w;
-  int *ex_count, *ex_tile;                 // [experts], [moe_rows / 128]
+  int *ex_count, *ex_tile;                 // [experts], [2][moe_rows / 128]
   int ld_f32, ld_gu, ld_act, moe_rows;
 };
 

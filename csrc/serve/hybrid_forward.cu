@@ -73,6 +73,7 @@ int bb_hy_kv_post(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const
 int bb_hy_glu(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream);
 int bb_hy_moe_tiles(const BbHyLayer* L, int n);
 int bb_hy_route(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream);
+int bb_hy_route_row(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream);
 int bb_hy_expert_rows(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream);
 int bb_hy_expert_glu(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream);
 int bb_hy_mlstm_gates(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream);
@@ -323,10 +324,19 @@ int project_tiles(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const
                               s);
 }
 
-// Router logits in w.f32 -> the experts' outputs in w.ex_out, weights and rows of every token's choices
+// fp32 products of the normed input, and every token's experts
+constexpr int ROUTE_ROWS = 128;    // up to here one kernel, a block per row
+
+int route(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
+  const int rc = b.n <= ROUTE_ROWS ? bb_hy_route_row(&c, &L, &w, b.n, s) : BB_ESIZE;
+  if (rc != BB_ESIZE) return rc;
+  BB_TRY(project_f32(c, L.in32, w.h, c.dp, w.f32, w.ld_f32, b.n, 1.f, 0, s));
+  return L.n_experts > 0 ? bb_hy_route(&c, &L, &w, b.n, s) : BB_OK;
+}
+
+// Every token's experts -> their outputs in w.ex_out, and the rows there
 int experts(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
   const int tiles = bb_hy_moe_tiles(&L, b.n);
-  BB_TRY(bb_hy_route(&c, &L, &w, b.n, s));
   BB_TRY(bb_hy_expert_rows(&c, &L, &w, b.n, s));
   BB_TRY(project_tiles(c, L, w, L.w_egu, 2 * L.effp, c.dp, w.ex_in, c.dp, w.ex_gu, w.ld_gu, tiles, s));
   BB_TRY(bb_hy_expert_glu(&c, &L, &w, b.n, s));
@@ -349,7 +359,7 @@ int forward_start(const BbHyCfg& c, const BbHyWork& w, const BbHyBatch& b, float
       BB_CUDA(cudaEventRecord(side->fork, main));
       BB_CUDA(cudaStreamWaitEvent(side->s, side->fork, 0));
     }
-    if (L.in32.w) BB_TRY(project_f32(c, L.in32, w.h, c.dp, w.f32, w.ld_f32, b.n, 1.f, 0, t));
+    if (L.in32.w) BB_TRY(route(c, L, w, b, t));
     const bool gates = L.kind == 5 || (L.beside && L.beside->kind == 5);
     if (fork && gates) BB_CUDA(cudaEventRecord(side->ready, side->s));
     if (L.n_experts > 0) BB_TRY(experts(c, L, w, b, t));

@@ -290,7 +290,7 @@ def test_routing_and_rows(E, top, groups, keep, n):
         tiles = lib().bb_hy_moe_tiles(C.byref(L), n)
         t = dict(ex_in=torch.zeros(tiles * 128, dp, device="cuda", dtype=dtype), pair_expert=i32(np.zeros(n * top)),
                  pair_row=i32(np.zeros(n * top)), pair_w=torch.zeros(n * top, device="cuda"), ex_count=i32(np.zeros(E)),
-                 ex_tile=i32(np.full(tiles + 1, 99)))
+                 ex_tile=i32(np.full(2 * tiles + 1, 99)))
         for k, v in t.items():
             setattr(w, k, v.data_ptr())
         w.h, w.f32, w.ld_f32, w.moe_rows = h.data_ptr(), logits.data_ptr(), ldz, tiles * 128
@@ -306,13 +306,46 @@ def test_routing_and_rows(E, top, groups, keep, n):
             assert expert[i].tolist() == [e for e, _ in want]
             assert np.allclose(weight[i], [x for _, x in want], rtol=2e-5, atol=1e-9)
         tile = t["ex_tile"].cpu().numpy()
-        assert tile[tiles] == 99 and len(set(row.ravel().tolist())) == n * top and row.max() < tiles * 128
+        assert tile[2 * tiles] == 99 and len(set(row.ravel().tolist())) == n * top and row.max() < tiles * 128
         assert np.array_equal(tile[row // 128], expert)
         assert t["ex_count"].cpu().numpy().tolist() == np.bincount(expert.ravel(), minlength=E).tolist()
         assert torch.equal(t["ex_in"][torch.from_numpy(row.ravel()).long().cuda()], h.repeat_interleave(top, 0))
         # every expert's rows lie on as many tiles as they need
+        assert np.array_equal(tile[tiles:2 * tiles], np.bincount(row.ravel() // 128, minlength=tiles))
         for e in range(E):
             assert (tile[:tiles] == e).sum() == -(-int((expert == e).sum()) // 128)
+
+
+@pytest.mark.parametrize("E,top,groups,keep,more", [(12, 3, 4, 2, 6), (0, 0, 1, 1, 8), (64, 8, 8, 4, 0), (200, 5, 2, 1, 10)])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_products_and_routing_of_few_rows(E, top, groups, keep, more, dtype):
+    from brain_b200.ops._cuda import check_error, lib, stream_ptr
+    from brain_b200.serve import hybrid_native as hn
+    n, dp, g = 33, 136, torch.Generator().manual_seed(E)
+    outs = hn.pad8(E) + hn.pad8(more)
+    h, W = (torch.randn(*s, generator=g).to(dtype) for s in ((n, dp), (outs, dp)))
+    hd, wd, out = h.cuda(), W.cuda(), torch.full((n, outs + 3), 7.0, device="cuda")
+    L, w, cfg = hn.Layer(), hn.Work(), hn.Cfg()
+    cfg.dtype, cfg.dp = int(dtype == torch.float32), dp
+    L.in32 = hn.Lin(wd.data_ptr(), outs, dp)
+    L.n_experts, L.top, L.groups_all, L.groups_keep, L.route_scale, L.route_tiny = E, top, groups, keep, 0.6, 1e-20
+    pe, pr, pw, count = i32(np.zeros(n * top + 1)), i32(np.zeros(n * top + 1)), torch.zeros(n * top + 1, device="cuda"), i32(np.zeros(E + 1))
+    w.h, w.f32, w.ld_f32 = hd.data_ptr(), out.data_ptr(), outs + 3
+    w.pair_expert, w.pair_row, w.pair_w, w.ex_count = (x.data_ptr() for x in (pe, pr, pw, count))
+    fn = lib().bb_hy_route_row
+    fn.restype = C.c_int
+    assert fn(C.byref(cfg), C.byref(L), C.byref(w), n, stream_ptr()) == 0
+    check_error()
+    want = h.double() @ W.double().t()
+    assert (out[:, :outs].cpu().double() - want).abs().max() < 2e-5 and bool((out[:, outs:] == 7.0).all())
+    if E:
+        expert, row, weight = (x[:-1].cpu().numpy().reshape(n, top) for x in (pe, pr, pw))
+        z, spec = out.cpu().double().numpy(), {"experts": E, "top": top, "groups": {"count": groups, "keep": keep}, "scale": 0.6}
+        for i in range(n):
+            ref = oracle.route(z[i, :E], spec)
+            assert expert[i].tolist() == [e for e, _ in ref] and np.allclose(weight[i], [x for _, x in ref], rtol=2e-5)
+        for e in range(E):
+            assert sorted(row[expert == e].tolist()) == list(range(int(count[e])))
 
 
 @pytest.mark.parametrize("G,N,K", [(3, 72, 40), (2, 8, 130), (1, 130, 8)])
