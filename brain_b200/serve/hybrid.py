@@ -67,6 +67,8 @@ class _Scratch:
         self.q, self.qa, self.ol, self.aux = z(rows, m["q"]), z(ab, m["qa"]), z(ab, m["ol"]), z(rows, m["aux"])
         self.ckv, self.kvx = z(max(exp, 1), m["ckv"]), z(max(exp, 1), m["kvx"])
         self.f32 = z(rows, m["f32"], dtype=f32)
+        self.part32 = z(-(-eng.dp // 64) * min(rows, 128) * m["f32"] if m["f32"] > 8 or any(l.in32.n for l in eng.layers) else 1,
+                        dtype=f32)
         # mixture of experts: every expert that has rows takes at most one 128-row tile that is not full
         routed = [l for l in eng.layers if l.n_experts]
         top = max((l.top for l in routed), default=0)
@@ -94,10 +96,10 @@ class _Scratch:
         self.hn, self.logits = z(max(want, 1), eng.dp), z(max(want, 1), eng.vocabp, dtype=f32)
         w = self.work = hn.Work()
         for n in ("x", "h", "proj", "cat", "xbc", "dt", "y", "v_first", "part_o", "part_ml", "seg", "hn", "logits", "h2", "q",
-                  "qa", "ol", "aux", "ckv", "kvx", "f32", "ex_in", "ex_gu", "ex_act", "ex_out", "pair_expert", "pair_row",
+                  "qa", "ol", "aux", "ckv", "kvx", "f32", "part32", "ex_in", "ex_gu", "ex_act", "ex_out", "pair_expert", "pair_row",
                   "pair_w", "ex_count", "ex_tile"):
             setattr(w, n, _ptr(getattr(self, n)))
-        w.seg_floats = self.seg.numel()
+        w.seg_floats, w.part32_floats = self.seg.numel(), self.part32.numel()
         w.rows, w.want_rows, w.exp_rows, w.moe_rows = rows, max(want, 1), exp, moe
         for k in m:
             setattr(w, "ld_" + k, m[k])

@@ -67,7 +67,8 @@ class Work(C.Structure):
                                  "pool_blocks")] + \
                [(n, P) for n in ("h2", "q", "qa", "ol", "ckv", "kvx", "aux")] + \
                [(n, I) for n in ("ld_q", "ld_qa", "ld_ol", "ld_ckv", "ld_kvx", "ld_aux", "exp_rows")] + \
-               [(n, P) for n in ("f32", "ex_in", "ex_gu", "ex_act", "ex_out", "pair_expert", "pair_row", "pair_w", "ex_count",
+               [("f32", P), ("part32", P), ("part32_floats", C.c_long)] + \
+               [(n, P) for n in ("ex_in", "ex_gu", "ex_act", "ex_out", "pair_expert", "pair_row", "pair_w", "ex_count",
                                  "ex_tile")] + \
                [(n, I) for n in ("ld_f32", "ld_gu", "ld_act", "moe_rows")]
 

@@ -1,7 +1,8 @@
 // Mixture of experts of a serving step, everything but its matrix products, for bf16 and fp32 storage:
 //   hy_route         one warp per token: softmax over the router's fp32 logits, the best groups by their best
 //                    expert, the best experts of those, their weights; a place among the rows of each
-//   hy_route_row     few rows: the same behind the fp32 products themselves, one block per row
+//   hy_products, hy_route_row   few rows: the router's products by slices of channels, added up where a block per row
+//                    routes
 //   hy_expert_rows   rows of the normed input to their experts' places, every expert's rows on 128-row tiles of
 //                    their own; the tiles' experts
 //   hy_expert_glu    clamped gated product of the experts' two halves
@@ -123,66 +124,85 @@ hy_route_kernel(const __grid_constant__ BbHyLayer L, const float* __restrict__ l
   if (mine) pair_row[p] = hist[e] + place;
 }
 
-// Few rows: one block per row computes the fp32 products of the normed input (router logits, gates) and routes.
-// V = 0: nothing to route.
-constexpr int RR_THREADS = 512;
+// Few rows: the fp32 products of the normed input (router logits, gates) by slices of PR_K channels side by side, ...
+constexpr int PR_TILE = 64, PR_K = 64;
 
-template <typename T, int V>
-__global__ void __launch_bounds__(RR_THREADS)
-hy_route_row_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ h, int dp, float* __restrict__ out, int ld,
-                    int* __restrict__ pair_expert, int* __restrict__ pair_row, float* __restrict__ pair_w, int* __restrict__ count) {
-  extern __shared__ __align__(16) float s_h[];     // the row, then the products
-  float* s_out = s_h + dp;
-  const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_out = L.in32.n;
+template <typename T>
+__global__ void __launch_bounds__(EX_THREADS)
+hy_products_kernel(const T* __restrict__ h, const T* __restrict__ W, int dp, int n, int n_out, float* __restrict__ part) {
+  __shared__ float sa[PR_TILE][PR_K + 1], sb[PR_TILE][PR_K + 1];
+  const int k0 = blockIdx.x * PR_K, o0 = blockIdx.y * PR_TILE, r0 = blockIdx.z * PR_TILE;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   struct alignas(sizeof(T) * 8) Raw {
     T v[8];
   };
-  const T* W = static_cast<const T*>(L.in32.w);
-  // outputs of a warp at a time (n_out is a multiple of 8), vectors of each asked for together
-  constexpr int O = 4, U = sizeof(T) == 2 ? 4 : 2, STEP = 256 * U;
-  Raw w[U][O];
-  auto fetch = [&](int o, int i0) {
+  constexpr int IT = PR_TILE * PR_K / 8 / EX_THREADS;
+  Raw a[IT], b[IT];
 #pragma unroll
-    for (int u = 0; u < U; ++u)
+  for (int i = 0; i < IT; ++i) {
+    const int v = threadIdx.x + i * EX_THREADS, r = v / (PR_K / 8), k = k0 + v % (PR_K / 8) * 8;
+    if (r0 + r < n && k < dp) a[i] = *reinterpret_cast<const Raw*>(h + (size_t)(r0 + r) * dp + k);
+    if (o0 + r < n_out && k < dp) b[i] = *reinterpret_cast<const Raw*>(W + (size_t)(o0 + r) * dp + k);
+  }
 #pragma unroll
-      for (int q = 0; q < O; ++q)
-        if (i0 + u * 256 < dp) w[u][q] = *reinterpret_cast<const Raw*>(W + (size_t)(o + q) * dp + i0 + u * 256);
-  };
-  const int o0 = warp * O;
-  if (o0 < n_out) fetch(o0, lane * 8);             // on their way while the row is
-  for (int i = threadIdx.x * 8; i < dp; i += RR_THREADS * 8) {
-    float f[8];
-    load8(h + (size_t)r * dp + i, f);
-    store8(s_h + i, f);
+  for (int i = 0; i < IT; ++i) {
+    const int v = threadIdx.x + i * EX_THREADS, r = v / (PR_K / 8), c = v % (PR_K / 8) * 8;
+    const bool in = k0 + c < dp;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      sa[r][c + j] = in && r0 + r < n ? to_f(a[i].v[j]) : 0.f;
+      sb[r][c + j] = in && o0 + r < n_out ? to_f(b[i].v[j]) : 0.f;
+    }
   }
   __syncthreads();
-  for (int o = o0; o < n_out; o += RR_THREADS / 32 * O) {
-    float a[O] = {};
-    for (int i0 = lane * 8; i0 < dp; i0 += STEP) {
-      if (o != o0 || i0 >= 256) fetch(o, i0);
+  float acc[4][4] = {};
+#pragma unroll 8
+  for (int k = 0; k < PR_K; ++k) {
+    float x[4], w[4];
 #pragma unroll
-      for (int u = 0; u < U; ++u) {
-        if (i0 + u * 256 >= dp) break;
-        float x[8];
-        load8(s_h + i0 + u * 256, x);
-#pragma unroll
-        for (int q = 0; q < O; ++q)
-#pragma unroll
-          for (int j = 0; j < 8; ++j) a[q] = fmaf(to_f(w[u][q].v[j]), x[j], a[q]);
-      }
+    for (int i = 0; i < 4; ++i) {
+      x[i] = sa[ty + 16 * i][k];
+      w[i] = sb[tx + 16 * i][k];
     }
 #pragma unroll
-    for (int q = 0; q < O; ++q) {
-      a[q] = warp_sum(a[q]);
-      if (lane == q) {
-        s_out[o + q] = a[q];
-        out[(size_t)r * ld + o + q] = a[q];
-      }
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(x[i], w[j], acc[i][j]);
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int r = r0 + ty + 16 * i, o = o0 + tx + 16 * j;
+      if (r < n && o < n_out) part[((size_t)blockIdx.x * n + r) * n_out + o] = acc[i][j];
     }
+}
+
+// ... then one block per row adds the slices up, in order, and routes.  V = 0: nothing to route.
+template <int V>
+__global__ void __launch_bounds__(EX_THREADS)
+hy_route_row_kernel(const __grid_constant__ BbHyLayer L, const float* __restrict__ part, int slices, float* __restrict__ out, int ld,
+                    int* __restrict__ pair_expert, int* __restrict__ pair_row, float* __restrict__ pair_w, int* __restrict__ count) {
+  extern __shared__ float s_out[];                 // [n_out], then [threads / n_out][n_out]
+  const int r = blockIdx.x, n = gridDim.x, n_out = L.in32.n, lane = threadIdx.x & 31;
+  const int per = max(EX_THREADS / n_out, 1);      // threads of an output
+  for (int o = threadIdx.x % n_out, g = threadIdx.x / n_out; o < n_out && g < per; o += EX_THREADS) {
+    float a = 0.f;
+    const int s0 = slices * g / per, s1 = slices * (g + 1) / per;
+#pragma unroll 8
+    for (int s = s0; s < s1; ++s) a += part[((size_t)s * n + r) * n_out + o];
+    s_out[n_out * (1 + g) + o] = a;
+  }
+  __syncthreads();
+  for (int o = threadIdx.x; o < n_out; o += EX_THREADS) {
+    float a = 0.f;
+    for (int g = 0; g < per; ++g) a += s_out[n_out * (1 + g) + o];
+    s_out[o] = a;
+    out[(size_t)r * ld + o] = a;
   }
   if constexpr (V > 0) {
     __syncthreads();
-    if (warp == 0) {
+    if (threadIdx.x < 32) {
       int e;
       float w;
       choose<V>(L, s_out, e, w);
@@ -316,15 +336,24 @@ BB_API int bb_hy_route(const BbHyCfg*, const BbHyLayer* L, const BbHyWork* w, in
   return (int)cudaGetLastError();
 }
 
-namespace bb {
-template <typename T>
-static int launch_route_row(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, int n, cudaStream_t s) {
-  const int E = L.n_experts;
-  const size_t smem = 4 * ((size_t)c.dp + L.in32.n);
-  if (smem > 48 * 1024 || E > 256 || L.top > 32) return BB_ESIZE;
-#define BB_ROUTE_ROW(V)                                                                                                     \
-  hy_route_row_kernel<T, V><<<n, RR_THREADS, smem, s>>>(L, static_cast<const T*>(w.h), c.dp, w.f32, w.ld_f32, w.pair_expert, \
-                                                        w.pair_row, w.pair_w, w.ex_count)
+// The fp32 products of the normed input -> w->f32, and with experts the routing; for few rows.  BB_ESIZE for more rows
+// than w->part32 holds slices of, and for sizes it does not cover.
+BB_API int bb_hy_route_row(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream) {
+  if (n <= 0) return BB_OK;
+  const int E = L->n_experts, n_out = L->in32.n, slices = (c->dp + PR_K - 1) / PR_K;
+  const size_t smem = 4 * (size_t)n_out * (1 + (n_out >= EX_THREADS ? 1 : EX_THREADS / n_out));
+  if ((long)slices * n * n_out > w->part32_floats || smem > 48 * 1024 || E > 256 || L->top > 32) return BB_ESIZE;
+  cudaStream_t s = (cudaStream_t)stream;
+  const dim3 grid(slices, (n_out + PR_TILE - 1) / PR_TILE, (n + PR_TILE - 1) / PR_TILE);
+  if (c->dtype)
+    hy_products_kernel<float><<<grid, EX_THREADS, 0, s>>>(static_cast<const float*>(w->h), static_cast<const float*>(L->in32.w), c->dp, n,
+                                                          n_out, w->part32);
+  else
+    hy_products_kernel<__nv_bfloat16><<<grid, EX_THREADS, 0, s>>>(static_cast<const __nv_bfloat16*>(w->h),
+                                                                  static_cast<const __nv_bfloat16*>(L->in32.w), c->dp, n, n_out, w->part32);
+#define BB_ROUTE_ROW(V)                                                                                                        \
+  hy_route_row_kernel<V><<<n, EX_THREADS, smem, s>>>(*L, w->part32, slices, w->f32, w->ld_f32, w->pair_expert, w->pair_row, \
+                                                     w->pair_w, w->ex_count)
   if (E == 0) BB_ROUTE_ROW(0);
   else if (E <= 32) BB_ROUTE_ROW(1);
   else if (E <= 64) BB_ROUTE_ROW(2);
@@ -332,15 +361,6 @@ static int launch_route_row(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork
   else BB_ROUTE_ROW(8);
 #undef BB_ROUTE_ROW
   return (int)cudaGetLastError();
-}
-}  // namespace bb
-
-// The fp32 products of the normed input -> w->f32, and with experts the routing; for few rows.  BB_ESIZE for rows or
-// expert counts it does not cover.
-BB_API int bb_hy_route_row(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream) {
-  if (n <= 0) return BB_OK;
-  return c->dtype ? launch_route_row<float>(*c, *L, *w, n, (cudaStream_t)stream)
-                  : launch_route_row<__nv_bfloat16>(*c, *L, *w, n, (cudaStream_t)stream);
 }
 
 BB_API int bb_hy_expert_rows(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream) {

@@ -263,7 +263,10 @@ static int launch_decode_v(const BbHyLayer& L, const BbHyWork& w, const BbHyBatc
 template <typename T>
 static int launch_decode(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, float eps, cudaStream_t s) {
   if (L.p % 4) return launch_decode_v<T, 1, 128>(L, w, b, eps, s);
-  return (long)L.n * L.p <= 128 * 128 ? launch_decode_v<T, 4, 128>(L, w, b, eps, s) : launch_decode_v<T, 4, 256>(L, w, b, eps, s);
+  // large states, and few blocks: more threads share one
+  return (long)L.n * L.p <= 128 * 128 && (long)(b.ns - b.ns_pre) * L.heads > 4 * sm_count()
+             ? launch_decode_v<T, 4, 128>(L, w, b, eps, s)
+             : launch_decode_v<T, 4, 256>(L, w, b, eps, s);
 }
 
 }  // namespace bb

@@ -565,24 +565,36 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
       }
     }
     }
+    constexpr int VR = PP / 8;     // 16-byte pieces of a row
+    constexpr int OUT_IT = 128 * VR / SSD_THREADS;
+    bf16x8 gate[GATED ? OUT_IT : 1];
+    if constexpr (GATED) {         // output gates, asked for ahead of the barrier
+#pragma unroll
+      for (int it = 0; it < OUT_IT; ++it) {
+        const int i = threadIdx.x + it * SSD_THREADS, rr = i / VR, q = i % VR;
+        if (rr < valid && q * 8 < L.pp)
+          gate[it] = *reinterpret_cast<const bf16x8*>(proj + (size_t)(c0 + rr) * ldp + L.off_gg + h * L.pp + q * 8);
+      }
+    }
     ok = __syncthreads_and(ok);
-    if (ok) {
-      constexpr int VR = PP / 8;   // 16-byte pieces of a row
-#pragma unroll 2
+    if constexpr (GATED) {
+#pragma unroll
+      for (int it = 0; it < OUT_IT; ++it) {
+        const int i = threadIdx.x + it * SSD_THREADS, rr = i / VR, q = i % VR, col = h * L.pp + q * 8;
+        if (ok && rr < valid && q * 8 < L.pp) {
+          float f[8], g[8], w[8];
+          unpack8(*reinterpret_cast<const bf16x8*>(sC + (q >> 3) * SSD_SUB + rr * 128 + (((q & 7) ^ (rr & 7)) << 4)), f);
+          unpack8(gate[it], g);
+          load8(L.gnorm + col, w);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) f[j] *= w[j] * sigmoid_as<__nv_bfloat16>(g[j]);
+          store8(y + (size_t)(c0 + rr) * ldy + col, f);
+        }
+      }
+    } else if (ok) {
       for (int i = threadIdx.x; i < valid * VR; i += SSD_THREADS) {
         const int rr = i / VR, q = i % VR;
-        if constexpr (GATED) {
-          const int col = h * L.pp + q * 8;
-          if (q * 8 < L.pp) {
-            float f[8], g[8], w[8];
-            unpack8(*reinterpret_cast<const bf16x8*>(sC + (q >> 3) * SSD_SUB + rr * 128 + (((q & 7) ^ (rr & 7)) << 4)), f);
-            load8(proj + (size_t)(c0 + rr) * ldp + L.off_gg + col, g);
-            load8(L.gnorm + col, w);
-#pragma unroll
-            for (int j = 0; j < 8; ++j) f[j] *= w[j] * sigmoid_as<__nv_bfloat16>(g[j]);
-            store8(y + (size_t)(c0 + rr) * ldy + col, f);
-          }
-        } else if (q * 8 < L.p)
+        if (q * 8 < L.p)
           *reinterpret_cast<uint4*>(y + (size_t)(c0 + rr) * ldy + h * L.p + q * 8) =
               *reinterpret_cast<const uint4*>(sC + (q >> 3) * SSD_SUB + rr * 128 + (((q & 7) ^ (rr & 7)) << 4));
       }
@@ -652,11 +664,11 @@ static int launch_ssd(const CUtensorMap& tmBC, const CUtensorMap& tmX, const BbH
   const int smem = GATED && (PP > 64 || L.n > 64) ? MOST : SsdCfg<PP>::SMEM;
   const __nv_bfloat16* proj = static_cast<const __nv_bfloat16*>(w.proj);
   // segments: as many as fill the machine once, of four chunks or more (a 2048-token prompt of 64 heads
-  // alone: 75 us against 112 us in one piece; at two chunks the extra launch costs more than it saves),
+  // alone: 75 us against 112 us in one piece; at two chunks the extra launch costs more than it saves; GATED: of two),
   // and as the scratch allows
   const long pairs = (long)b.ns_pre * L.heads, np = GATED ? L.mem : (long)L.n * L.p;
   int segs = (int)((PP == 64 && smem < 116 * 1024 ? 2 : 1) * sm_count() / pairs);
-  const int most = (b.max_len + 127) / 128 / 4;
+  const int most = (b.max_len + 127) / 128 / (GATED ? 2 : 4);
   if (segs > most) segs = most;
   if (segs > 16) segs = 16;
   while (segs > 1 && pairs * ((segs + 1) * np + segs) > w.seg_floats) --segs;

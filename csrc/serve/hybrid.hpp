@@ -147,7 +147,8 @@ struct BbHyWork {
   // fp32 products of the normed input; mixture of experts: rows sorted by expert, every expert's on 128-row
   // tiles of their own (input, both halves, their product, output), and of every (token, choice) its expert, row
   // and weight; rows of every expert; expert of every tile (-1: unused), then how many rows every tile has
-  float* f32;                              // [rows, ld_f32]
+  float *f32, *part32;                     // [rows, ld_f32]; slices of the same for few rows
+  long part32_floats;
   void *ex_in, *ex_gu, *ex_act, *ex_out;   // [moe_rows, dp | ld_gu | ld_act | dp]
   int *pair_expert, *pair_row;             // [rows top]
   float* pair_w;

@@ -325,7 +325,7 @@ int project_tiles(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const
 }
 
 // fp32 products of the normed input, and every token's experts
-constexpr int ROUTE_ROWS = 128;    // up to here one kernel, a block per row
+constexpr int ROUTE_ROWS = 128;    // up to here by slices of channels
 
 int route(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
   const int rc = b.n <= ROUTE_ROWS ? bb_hy_route_row(&c, &L, &w, b.n, s) : BB_ESIZE;

@@ -321,7 +321,7 @@ def test_routing_and_rows(E, top, groups, keep, n):
 def test_products_and_routing_of_few_rows(E, top, groups, keep, more, dtype):
     from brain_b200.ops._cuda import check_error, lib, stream_ptr
     from brain_b200.serve import hybrid_native as hn
-    n, dp, g = 33, 136, torch.Generator().manual_seed(E)
+    n, dp, g = 70, 136, torch.Generator().manual_seed(E)
     outs = hn.pad8(E) + hn.pad8(more)
     h, W = (torch.randn(*s, generator=g).to(dtype) for s in ((n, dp), (outs, dp)))
     hd, wd, out = h.cuda(), W.cuda(), torch.full((n, outs + 3), 7.0, device="cuda")
@@ -330,7 +330,8 @@ def test_products_and_routing_of_few_rows(E, top, groups, keep, more, dtype):
     L.in32 = hn.Lin(wd.data_ptr(), outs, dp)
     L.n_experts, L.top, L.groups_all, L.groups_keep, L.route_scale, L.route_tiny = E, top, groups, keep, 0.6, 1e-20
     pe, pr, pw, count = i32(np.zeros(n * top + 1)), i32(np.zeros(n * top + 1)), torch.zeros(n * top + 1, device="cuda"), i32(np.zeros(E + 1))
-    w.h, w.f32, w.ld_f32 = hd.data_ptr(), out.data_ptr(), outs + 3
+    part = torch.full((-(-dp // 64) * n * outs,), float("nan"), device="cuda")
+    w.h, w.f32, w.ld_f32, w.part32, w.part32_floats = hd.data_ptr(), out.data_ptr(), outs + 3, part.data_ptr(), part.numel()
     w.pair_expert, w.pair_row, w.pair_w, w.ex_count = (x.data_ptr() for x in (pe, pr, pw, count))
     fn = lib().bb_hy_route_row
     fn.restype = C.c_int
