@@ -161,9 +161,18 @@ hy_mlstm_decode_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict_
   };
   const bool fresh = b.pos[r] == 0;
   fetch(nr, lane);
-  const LogGates g = log_gates(L, raw[r * ldr + L.off32_i + h], raw[r * ldr + L.off32_f + h], h);
-  const float m0 = fresh ? 0.f : norm[N], m = fmaxf(g.f + m0, g.i), add = expf(g.i - m);
-  const float keep = fresh ? 0.f : expf(g.f + m0 - m);
+  __shared__ float s_gate[3];
+  if (threadIdx.x == 0) {
+    const LogGates g = log_gates(L, raw[r * ldr + L.off32_i + h], raw[r * ldr + L.off32_f + h], h);
+    const float m0 = fresh ? 0.f : norm[N], m = fmaxf(g.f + m0, g.i);
+    s_gate[0] = m;
+    s_gate[1] = expf(g.i - m);
+    s_gate[2] = fresh ? 0.f : expf(g.f + m0 - m);
+    norm[N] = m;
+  }
+  for (int p = threadIdx.x; p < P; p += THREADS) sv[p] = to_f(row[L.off_vv + h * L.pp + p]);
+  __syncthreads();
+  const float m = s_gate[0], add = s_gate[1], keep = s_gate[2];
   float nq = 0.f;
   for (int d = threadIdx.x; d < N; d += THREADS) {
     const float q = to_f(row[L.off_q + h * L.np + d]) * L.q_scale, k = to_f(row[L.off_kk + h * L.np + d]);
@@ -174,9 +183,7 @@ hy_mlstm_decode_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict_
     norm[d] = x;
     nq = fmaf(x, q, nq);
   }
-  for (int p = threadIdx.x; p < P; p += THREADS) sv[p] = to_f(row[L.off_vv + h * L.pp + p]);
   nq = block_sum(nq, part[0]);       // (its barrier also orders shared memory)
-  if (threadIdx.x == 0) norm[N] = m;
   for (int p = lane; p < pv; p += lanes) {
     float av[V], acc[V];
 #pragma unroll

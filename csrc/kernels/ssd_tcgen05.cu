@@ -23,8 +23,8 @@
 // segments of the main launch then start from the state carried in, decayed and summed over the segments
 // before them (GATED: each brought to a common stabiliser).
 //
-// 256 threads: TMEM lane = token (or state row), two warpgroups share a row's columns.  Thread 0 issues
-// TMA and MMA.  The phases of a chunk are separated by block barriers; with head sizes up to 64 two CTAs
+// TMEM lane = token (or state row); W warpgroups share a row's columns: two, or four where one CTA has the SM to
+// itself and GATED has the most to do between the MMAs.  Thread 0 issues TMA and MMA.  The phases of a chunk are separated by block barriers; with head sizes up to 64 two CTAs
 // share an SM (113 KB of shared memory, 256 TMEM columns each) and fill each other's gaps.
 // TMEM: G, then W as packed bf16 (value in its first 64 columns, remainder in the others); Y; S.
 #include "../common/host.hpp"
@@ -34,7 +34,6 @@
 
 namespace bb {
 
-constexpr int SSD_THREADS = 256;
 constexpr int SSD_SUB = 128 * 128;   // one swizzled sub-tile: 128 rows of 64 bf16
 
 template <int PP>
@@ -46,7 +45,8 @@ struct SsdCfg {
   static constexpr int OFF_S = OFF_X + PSUB * SSD_SUB;          // 2 PSUB: S as two terms, then X' as two terms
   static constexpr int OFF_E = OFF_S + 2 * PSUB * SSD_SUB;      // 128 floats, 8 partial sums, barriers
   static constexpr int SMEM = OFF_E + 1024;
-  static constexpr int GATED_FLOATS = 128 * 7 + 8 * 128 + 64;   // see GatedSmem
+  static constexpr int W = 2, GATED_W = PP == 64 ? 2 : 4;       // warpgroups
+  static constexpr int GATED_FLOATS = 128 * (2 + 6 * GATED_W) + 64;   // see GatedSmem
   // TMEM columns.  The state product of a chunk leaves its two terms side by side: the first added to S,
   // the second in T right behind it (one 2 PP wide MMA per step instead of two, which cost the same each).
   // With PP = 64 T lies over the first half of W, whose products are issued before.
@@ -57,10 +57,12 @@ struct SsdCfg {
 
 // What the gated form keeps beside the tiles: with head sizes up to 64 in the half of the query tile that stays free
 // (two CTAs then still share an SM), else behind everything.
+template <int W>
 struct GatedSmem {
-  float *n, *w, *sum, *nq, *part, *pm, *co;   // [128] normaliser, [128] token weights, [2][128] sums of a row's two
-                                              // halves, [2][128] n.q likewise, [8][128], [8], [34]
-  __device__ explicit GatedSmem(float* p) : n(p), w(p + 128), sum(p + 256), nq(p + 512), part(p + 768), pm(p + 1792), co(p + 1800) {}
+  float *n, *w, *sum, *nq, *part, *pm, *co;   // [128] normaliser, [128] token weights, [W][128] sums of a row's parts,
+                                              // [W][128] n.q likewise, [4 W][128], [4], [34]
+  __device__ explicit GatedSmem(float* p)
+      : n(p), w(p + 128), sum(p + 256), nq(sum + W * 128), part(nq + W * 128), pm(part + 4 * W * 128), co(pm + 4) {}
 };
 
 __device__ __forceinline__ float2 split_pair(float a, float b) {
@@ -90,14 +92,15 @@ __device__ __forceinline__ void store_split(uint8_t* hi, uint8_t* lo, int row, i
   }
 }
 
-template <int PP, bool LOCAL, bool GATED>
-__global__ void __launch_bounds__(SSD_THREADS, PP == 64 ? 2 : 1)
+template <int PP, bool LOCAL, bool GATED, int W>
+__global__ void __launch_bounds__(W * 128, PP == 64 ? 2 : 1)
 ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant__ CUtensorMap tmX,
                  const __grid_constant__ BbHyLayer L, const float* __restrict__ dt, int lddt,
                  __nv_bfloat16* __restrict__ y, int ldy, const __grid_constant__ BbHyBatch b, int segs,
                  float* __restrict__ seg, int* err, const __nv_bfloat16* __restrict__ proj, int ldp, float eps) {
   using Cfg = SsdCfg<PP>;
-  constexpr int PSUB = Cfg::PSUB, HC = PP / 2;   // HC: Y / S / X columns of a thread
+  constexpr int SSD_THREADS = W * 128;
+  constexpr int PSUB = Cfg::PSUB, HC = PP / W, GC = 128 / W;   // Y / S / X columns and G columns of a thread
   extern __shared__ __align__(1024) uint8_t smem[];
   uint8_t* sC = smem + Cfg::OFF_C;
   uint8_t* sB = smem + Cfg::OFF_B;
@@ -105,7 +108,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
   uint8_t* sS = smem + Cfg::OFF_S;
   uint8_t* sSl = sS + PSUB * SSD_SUB;
   float* s_e = reinterpret_cast<float*>(smem + Cfg::OFF_E);   // [128]
-  float* s_part = s_e + 128;                                  // [8] warp sums of the coming chunk
+  float* s_part = s_e + 128;                                  // [4] (of 8) warp sums of the coming chunk
   uint64_t* bars = reinterpret_cast<uint64_t*>(s_part + 8);
   uint64_t *b_tma = bars, *b_gy = bars + 1, *b_y = bars + 2, *b_s = bars + 3;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 4);
@@ -120,7 +123,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
   const float a2 = GATED ? 0.f : L.a[h] * kLog2e, D = GATED ? 0.f : L.d_skip[h];
   const size_t np = (size_t)L.n * L.p, mem = GATED ? L.mem : np;   // floats of a state
   float* state = L.ssm_state + ((size_t)slot * L.heads + h) * mem;
-  GatedSmem gs(reinterpret_cast<float*>(PP == 64 && nsub == 1 ? sC + SSD_SUB : smem + Cfg::SMEM));
+  GatedSmem<W> gs(reinterpret_cast<float*>(PP == 64 && nsub == 1 ? sC + SSD_SUB : smem + Cfg::SMEM));
 
   // this CTA's chunks, and the scratch of its (sequence, head): segment states, the state carried in, decays
   const int z = blockIdx.z, per = (n_chunks + segs - 1) / segs, z_last = (n_chunks - 1) / per;
@@ -241,7 +244,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
       const float v = __shfl_up_sync(0xffffffffu, cum_next, o);
       if (lane >= o) cum_next += v;
     }
-    if (lane == 31) s_part[warp] = cum_next;
+    if (lane == 31 && half == 0) s_part[warp] = cum_next;
     if constexpr (GATED) {
       d_next -= cum_next;                          // e, less the sum over the warps before this one
       max_next = d_next;
@@ -250,7 +253,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
         const float v = __shfl_up_sync(0xffffffffu, max_next, o);
         if (lane >= o) max_next = fmaxf(max_next, v);
       }
-      if (lane == 31) gs.pm[warp] = max_next;
+      if (lane == 31 && half == 0) gs.pm[warp] = max_next;
     }
   };
   load_dt(ch0);
@@ -293,8 +296,8 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
           mine = base;
           top = top_all;
         }
-        top_all = fmaxf(top_all, gs.pm[half * 4 + w] - base);
-        base += s_part[half * 4 + w];
+        top_all = fmaxf(top_all, gs.pm[w] - base);
+        base += s_part[w];
       }
       const float e = d - mine;
       top = fmaxf(top, max_next - mine);
@@ -310,7 +313,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
       }
     } else {
       float cum = cum_next;
-      for (int w = 0; w < (warp & 3); ++w) cum += s_part[half * 4 + w];
+      for (int w = 0; w < (warp & 3); ++w) cum += s_part[w];
       w_row = cum;
       dec = exp2f(total);
       if (half == 0) s_e[row] = d > 0.f ? cum - log2f(d) : INFINITY;
@@ -371,8 +374,8 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
     }
     __syncwarp();
     if constexpr (GATED) {
-      // this row's query with the normaliser, half of the channels to a thread
-      const int vec0 = half * nsub * 4, vecs = nsub * 4;      // vectors of 8 channels
+      // this row's query with the normaliser, a part of the channels to a thread
+      const int vecs = nsub * 8 / W, vec0 = half * vecs;      // vectors of 8 channels
       float a = 0.f;
       for (int v = 0; v < vecs; ++v) {
         const int q = vec0 + v;
@@ -387,10 +390,10 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
     ok = mbar_wait(b_gy, ph);
     tc_fence_after();
     __syncwarp();
-    // scores of this thread's 64 columns into registers before any thread writes weights over them
-    uint32_t g0[32], g1[32];
-    tmem_ld32(tG + half * 64, g0);
-    tmem_ld32(tG + half * 64 + 32, g1);
+    // scores of this thread's columns into registers before any thread writes weights over them
+    uint32_t g0[32], g1[GC == 64 ? 32 : 1];
+    tmem_ld32(tG + half * GC, g0);
+    if constexpr (GC == 64) tmem_ld32(tG + half * GC + 32, g1);
     tmem_wait_ld();
     tc_fence_before();
     ok = __syncthreads_and(ok);
@@ -400,8 +403,8 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
     }
     tc_fence_after();
     {
-      const float* e = s_e + half * 64;
-      const int lim = row - half * 64;   // columns j <= lim are in the past
+      const float* e = s_e + half * GC;
+      const int lim = row - half * GC;   // columns j <= lim are in the past
       float row_sum = 0.f;
       auto weights = [&](const uint32_t (&g)[32], int j0) {
         uint32_t hi[16], lo[16];
@@ -419,11 +422,11 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
           hi[(j >> 1) + 1] = __float_as_uint(s23.x);
           lo[(j >> 1) + 1] = __float_as_uint(s23.y);
         }
-        tmem_st16(tG + half * 32 + (j0 >> 1), hi);
-        tmem_st16(tG + 64 + half * 32 + (j0 >> 1), lo);
+        tmem_st16(tG + half * (GC / 2) + (j0 >> 1), hi);
+        tmem_st16(tG + 64 + half * (GC / 2) + (j0 >> 1), lo);
       };
       weights(g0, 0);
-      weights(g1, 32);
+      if constexpr (GC == 64) weights(g1, 32);
       if (GATED) gs.sum[half * 128 + row] = row_sum;
     }
     }
@@ -486,10 +489,10 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
     __syncwarp();
     if constexpr (GATED) {
       // the normaliser's new part: 8 channels of a few tokens to a thread, summed over the CTA below
-      const int nv = nsub * 8, v = threadIdx.x % nv, t0 = threadIdx.x / nv * (nv / 2);
+      const int nv = nsub * 8, v = threadIdx.x % nv, per = nv / W, t0 = threadIdx.x / nv * per;
       float a[8] = {};
 #pragma unroll 4
-      for (int t = t0; t < t0 + nv / 2; ++t) {
+      for (int t = t0; t < t0 + per; ++t) {
         float f[8];
         unpack8(*reinterpret_cast<const bf16x8*>(sB + (v >> 3) * SSD_SUB + t * 128 + (((v & 7) ^ (t & 7)) << 4)), f);
         const float w = gs.w[t];
@@ -512,7 +515,10 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
     // outputs go through the C tile's place (its products are behind us), so that a row's columns leave
     // as one contiguous piece
     if constexpr (GATED) {
-      const float nq = L.q_scale * (gs.nq[row] + gs.nq[128 + row] + gs.sum[row] + gs.sum[128 + row]);
+      float nq = 0.f;
+#pragma unroll
+      for (int w = 0; w < W; ++w) nq += gs.nq[w * 128 + row] + gs.sum[w * 128 + row];
+      nq *= L.q_scale;
       const float f = L.q_scale / (fmaxf(fabsf(nq), exp2f(-m_row)) + 1e-6f);
       float o[HC], ss = 0.f;
 #pragma unroll
@@ -532,11 +538,14 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
       if (threadIdx.x < L.n) {
         float v = gs.n[threadIdx.x] * dec;
 #pragma unroll
-        for (int w = 0; w < 8; ++w) v += gs.part[w * 128 + threadIdx.x];
+        for (int w = 0; w < 4 * W; ++w) v += gs.part[w * 128 + threadIdx.x];
         gs.n[threadIdx.x] = v;
       }
       __syncthreads();
-      const float rstd = rsqrtf((gs.sum[row] + gs.sum[128 + row]) / (float)L.p + eps);
+      ss = 0.f;
+#pragma unroll
+      for (int w = 0; w < W; ++w) ss += gs.sum[w * 128 + row];
+      const float rstd = rsqrtf(ss / (float)L.p + eps);
 #pragma unroll
       for (int q = 0; q < HC / 8; ++q) {
         const int col = half * HC + q * 8;
@@ -604,7 +613,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
       if (threadIdx.x < L.n) {
         float v = gs.n[threadIdx.x] * dec;
 #pragma unroll
-        for (int w = 0; w < 8; ++w) v += gs.part[w * 128 + threadIdx.x];
+        for (int w = 0; w < 4 * W; ++w) v += gs.part[w * 128 + threadIdx.x];
         gs.n[threadIdx.x] = v;
       }
     }
@@ -656,10 +665,11 @@ template <int PP, bool GATED>
 static int launch_ssd(const CUtensorMap& tmBC, const CUtensorMap& tmX, const BbHyLayer& L, const BbHyWork& w,
                       const BbHyBatch& b, const float* dt, int lddt, __nv_bfloat16* y, int ldy, float eps, cudaStream_t s) {
   static PerDeviceOnce once, once_local;
+  constexpr int W = GATED ? SsdCfg<PP>::GATED_W : SsdCfg<PP>::W;
   constexpr int MOST = SsdCfg<PP>::SMEM + (GATED ? 4 * SsdCfg<PP>::GATED_FLOATS : 0);
-  cudaError_t e = ensure_dyn_smem(once, ssd_chunk_kernel<PP, false, GATED>, MOST);
+  cudaError_t e = ensure_dyn_smem(once, ssd_chunk_kernel<PP, false, GATED, W>, MOST);
   if (e != cudaSuccess) return (int)e;
-  e = ensure_dyn_smem(once_local, ssd_chunk_kernel<PP, true, GATED>, MOST);
+  e = ensure_dyn_smem(once_local, ssd_chunk_kernel<PP, true, GATED, W>, MOST);
   if (e != cudaSuccess) return (int)e;
   const int smem = GATED && (PP > 64 || L.n > 64) ? MOST : SsdCfg<PP>::SMEM;
   const __nv_bfloat16* proj = static_cast<const __nv_bfloat16*>(w.proj);
@@ -675,12 +685,12 @@ static int launch_ssd(const CUtensorMap& tmBC, const CUtensorMap& tmX, const BbH
   if (segs < 2) segs = 1;
   const dim3 grid(b.ns_pre, L.heads, segs);
   if (segs > 1) {
-    ssd_chunk_kernel<PP, true, GATED><<<grid, SSD_THREADS, smem, s>>>(tmBC, tmX, L, dt, lddt, y, ldy, b, segs, w.seg,
+    ssd_chunk_kernel<PP, true, GATED, W><<<grid, W * 128, smem, s>>>(tmBC, tmX, L, dt, lddt, y, ldy, b, segs, w.seg,
                                                                       device_error_word(), proj, w.ld_proj, eps);
     e = cudaGetLastError();
     if (e != cudaSuccess) return (int)e;
   }
-  ssd_chunk_kernel<PP, false, GATED><<<grid, SSD_THREADS, smem, s>>>(tmBC, tmX, L, dt, lddt, y, ldy, b, segs, w.seg,
+  ssd_chunk_kernel<PP, false, GATED, W><<<grid, W * 128, smem, s>>>(tmBC, tmX, L, dt, lddt, y, ldy, b, segs, w.seg,
                                                                      device_error_word(), proj, w.ld_proj, eps);
   return (int)cudaGetLastError();
 }
