@@ -5,14 +5,15 @@ slots for the recurrent layers, one native call per step.
   sequences run together (``csrc/serve/hybrid_forward.cu``).  Every entry point - the scheduler's prefill,
   mixed and decode calls and :meth:`HybridEngine.step_logits` - goes through it.
 * Pages: per attention layer keys and values ``[num_blocks + 1, kv_heads, block_size, head size]``, per latent
-  attention layer with latents of its own ``[num_blocks + 1, block_size, latent | rotated key part]``.  State
-  slots: per recurrent layer the fp32 state (``[heads, state, head size]``, ``[heads, key, value]``, a matrix
-  memory with its normaliser and running maximum, or one value per channel) and, where it has a convolution, a ring of the last taps - 1 raw inputs.  A sequence at position
-  0 starts from zeros, so pages and slots are reused as they are.
+  attention layer with latents of its own ``[num_blocks + 1, block_size, latent | rotated key part]``.
+  State slots: per recurrent layer the fp32 state (``[heads, state, head size]``, ``[heads, key, value]``, a
+  matrix memory with its normaliser and running maximum, or one value per channel) and, where it has a
+  convolution, a ring of the last taps - 1 raw inputs.  A sequence at position 0 starts from zeros, so pages
+  and slots are reused as they are.
 * Mixtures of experts: rows of a step sorted by expert onto 128-row tiles, one grouped product per matrix.
 * ``dtype='bf16'``: bf16 weights, activations, pages and convolution inputs; the residual stream, norms,
-  rotation, scores, softmax, routers, step sizes, gates of a recurrence, decays and the recurrent state are fp32.  ``dtype='fp32'``:
-  everything in fp32, no tensor-core rounding."""
+  rotation, scores, softmax, routers, step sizes, gates of a recurrence, decays and the recurrent state are
+  fp32.  ``dtype='fp32'``: everything in fp32, no tensor-core rounding."""
 from __future__ import annotations
 
 import ctypes as C

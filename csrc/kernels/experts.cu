@@ -181,8 +181,9 @@ hy_products_kernel(const T* __restrict__ h, const T* __restrict__ W, int dp, int
 // ... then one block per row adds the slices up, in order, and routes.  V = 0: nothing to route.
 template <int V>
 __global__ void __launch_bounds__(EX_THREADS)
-hy_route_row_kernel(const __grid_constant__ BbHyLayer L, const float* __restrict__ part, int slices, float* __restrict__ out, int ld,
-                    int* __restrict__ pair_expert, int* __restrict__ pair_row, float* __restrict__ pair_w, int* __restrict__ count) {
+hy_route_row_kernel(const __grid_constant__ BbHyLayer L, const float* __restrict__ part, int slices,
+                    float* __restrict__ out, int ld, int* __restrict__ pair_expert, int* __restrict__ pair_row,
+                    float* __restrict__ pair_w, int* __restrict__ count) {
   extern __shared__ float s_out[];                 // [n_out], then [threads / n_out][n_out]
   const int r = blockIdx.x, n = gridDim.x, n_out = L.in32.n, lane = threadIdx.x & 31;
   const int per = max(EX_THREADS / n_out, 1);      // threads of an output
@@ -345,12 +346,12 @@ BB_API int bb_hy_route_row(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork*
   if ((long)slices * n * n_out > w->part32_floats || smem > 48 * 1024 || E > 256 || L->top > 32) return BB_ESIZE;
   cudaStream_t s = (cudaStream_t)stream;
   const dim3 grid(slices, (n_out + PR_TILE - 1) / PR_TILE, (n + PR_TILE - 1) / PR_TILE);
-  if (c->dtype)
-    hy_products_kernel<float><<<grid, EX_THREADS, 0, s>>>(static_cast<const float*>(w->h), static_cast<const float*>(L->in32.w), c->dp, n,
-                                                          n_out, w->part32);
-  else
-    hy_products_kernel<__nv_bfloat16><<<grid, EX_THREADS, 0, s>>>(static_cast<const __nv_bfloat16*>(w->h),
-                                                                  static_cast<const __nv_bfloat16*>(L->in32.w), c->dp, n, n_out, w->part32);
+#define BB_PRODUCTS(T)                                                                                       \
+  hy_products_kernel<T><<<grid, EX_THREADS, 0, s>>>(static_cast<const T*>(w->h), static_cast<const T*>(L->in32.w), \
+                                                    c->dp, n, n_out, w->part32)
+  if (c->dtype) BB_PRODUCTS(float);
+  else BB_PRODUCTS(__nv_bfloat16);
+#undef BB_PRODUCTS
 #define BB_ROUTE_ROW(V)                                                                                                        \
   hy_route_row_kernel<V><<<n, EX_THREADS, smem, s>>>(*L, w->part32, slices, w->f32, w->ld_f32, w->pair_expert, w->pair_row, \
                                                      w->pair_w, w->ex_count)
@@ -369,13 +370,13 @@ BB_API int bb_hy_expert_rows(const BbHyCfg* c, const BbHyLayer* L, const BbHyWor
   const int tiles = moe_tiles(*L, n), grid = (n + EX_THREADS / 32 - 1) / (EX_THREADS / 32) + 1;
   if (tiles * 128 > w->moe_rows) return BB_EARG;
   const size_t smem = 4 * (size_t)(L->n_experts + 1);
-  if (c->dtype)
-    hy_expert_rows_kernel<float><<<grid, EX_THREADS, smem, s>>>(*L, static_cast<const float*>(w->h), c->dp, w->pair_expert, w->pair_row,
-                                                                w->ex_count, static_cast<float*>(w->ex_in), w->ex_tile, tiles, w->moe_rows / 128, n);
-  else
-    hy_expert_rows_kernel<__nv_bfloat16><<<grid, EX_THREADS, smem, s>>>(*L, static_cast<const __nv_bfloat16*>(w->h), c->dp,
-                                                                        w->pair_expert, w->pair_row, w->ex_count,
-                                                                        static_cast<__nv_bfloat16*>(w->ex_in), w->ex_tile, tiles, w->moe_rows / 128, n);
+#define BB_ROWS(T)                                                                                           \
+  hy_expert_rows_kernel<T><<<grid, EX_THREADS, smem, s>>>(*L, static_cast<const T*>(w->h), c->dp, w->pair_expert, \
+                                                          w->pair_row, w->ex_count, static_cast<T*>(w->ex_in), \
+                                                          w->ex_tile, tiles, w->moe_rows / 128, n)
+  if (c->dtype) BB_ROWS(float);
+  else BB_ROWS(__nv_bfloat16);
+#undef BB_ROWS
   return (int)cudaGetLastError();
 }
 
@@ -384,12 +385,11 @@ BB_API int bb_hy_expert_glu(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork
   cudaStream_t s = (cudaStream_t)stream;
   const int* rows = w->ex_tile + w->moe_rows / 128;
   const int tiles = moe_tiles(*L, n), per = (128 * (L->effp / 8) + 4 * EX_THREADS - 1) / (4 * EX_THREADS);
-  if (c->dtype)
-    hy_expert_glu_kernel<float><<<tiles * per, EX_THREADS, 0, s>>>(*L, static_cast<const float*>(w->ex_gu), w->ld_gu,
-                                                                   static_cast<float*>(w->ex_act), w->ld_act, rows, per);
-  else
-    hy_expert_glu_kernel<__nv_bfloat16><<<tiles * per, EX_THREADS, 0, s>>>(*L, static_cast<const __nv_bfloat16*>(w->ex_gu), w->ld_gu,
-                                                                           static_cast<__nv_bfloat16*>(w->ex_act), w->ld_act, rows,
-                                                                           per);
+#define BB_GLU(T)                                                                                            \
+  hy_expert_glu_kernel<T><<<tiles * per, EX_THREADS, 0, s>>>(*L, static_cast<const T*>(w->ex_gu), w->ld_gu,  \
+                                                             static_cast<T*>(w->ex_act), w->ld_act, rows, per)
+  if (c->dtype) BB_GLU(float);
+  else BB_GLU(__nv_bfloat16);
+#undef BB_GLU
   return (int)cudaGetLastError();
 }

@@ -24,8 +24,8 @@
 // before them (GATED: each brought to a common stabiliser).
 //
 // TMEM lane = token (or state row); W warpgroups share a row's columns: two, or four where one CTA has the SM to
-// itself and GATED has the most to do between the MMAs.  Thread 0 issues TMA and MMA.  The phases of a chunk are separated by block barriers; with head sizes up to 64 two CTAs
-// share an SM (113 KB of shared memory, 256 TMEM columns each) and fill each other's gaps.
+// itself and GATED has the most to do between the MMAs.  Thread 0 issues TMA and MMA.  The phases of a chunk
+// are separated by block barriers; with head sizes up to 64 two CTAs share an SM (113 KB of shared memory, 256 TMEM columns each) and fill each other's gaps.
 // TMEM: G, then W as packed bf16 (value in its first 64 columns, remainder in the others); Y; S.
 #include "../common/host.hpp"
 #include "../common/ptx.cuh"
@@ -150,8 +150,8 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
   __syncthreads();
   tc_fence_after();
   const uint32_t tm = *tmem_slot;
-  const uint32_t tG = tm + Cfg::COL_G + lane_sel, tY = tm + Cfg::COL_Y + lane_sel + half * HC, tS = tm + Cfg::COL_S + lane_sel + half * HC,
-                 tT = tm + Cfg::COL_T + lane_sel + half * HC;
+  const uint32_t tG = tm + Cfg::COL_G + lane_sel, tY = tm + Cfg::COL_Y + lane_sel + half * HC,
+                 tS = tm + Cfg::COL_S + lane_sel + half * HC, tT = tm + Cfg::COL_T + lane_sel + half * HC;
   // The state between memory and TMEM goes through the operand tiles' place as fp32 [128][PP], columns
   // exclusive-or'ed with the row: a warp moves whole rows of memory, a thread reads or writes its own row.
   float* s_st = reinterpret_cast<float*>(sS);

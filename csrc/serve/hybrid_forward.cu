@@ -324,9 +324,9 @@ int project_tiles(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const
                               s);
 }
 
-// fp32 products of the normed input, and every token's experts
-constexpr int ROUTE_ROWS = 128;    // up to here by slices of channels
+constexpr int ROUTE_ROWS = 128;    // rows up to which these products run as slices of channels
 
+// fp32 products of the normed input, and every token's experts
 int route(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
   const int rc = b.n <= ROUTE_ROWS ? bb_hy_route_row(&c, &L, &w, b.n, s) : BB_ESIZE;
   if (rc != BB_ESIZE) return rc;
