@@ -25,7 +25,8 @@
 //
 // TMEM lane = token (or state row); W warpgroups share a row's columns: two, or four where one CTA has the SM to
 // itself and GATED has the most to do between the MMAs.  Thread 0 issues TMA and MMA.  The phases of a chunk
-// are separated by block barriers; with head sizes up to 64 two CTAs share an SM (113 KB of shared memory, 256 TMEM columns each) and fill each other's gaps.
+// are separated by block barriers; with head sizes up to 64 two CTAs share an SM (113 KB of shared memory, 256
+// TMEM columns each) and fill each other's gaps.
 // TMEM: G, then W as packed bf16 (value in its first 64 columns, remainder in the others); Y; S.
 #include "../common/host.hpp"
 #include "../common/ptx.cuh"
