@@ -31,7 +31,8 @@ NVCC_FLAGS = [
 #: --use_fast_math (IEEE division and square root in the AdamW update, exact exp/log in the CE)
 #: (the hybrid decoder's norms, recurrence and fp32 path: what is computed in 32-bit keeps its 32 bits)
 EXACT_MATH = {"adamw.cu", "rs_adamw.cu", "ce.cu", "hybrid_rows.cu", "mamba2.cu", "attn_rows.cu", "sgemm.cu",
-              "depth_rows.cu", "latent_rows.cu", "delta.cu", "rglru.cu", "mlstm.cu", "experts.cu"}
+              "depth_rows.cu", "latent_rows.cu", "delta.cu", "rglru.cu", "mlstm.cu", "experts.cu",
+              "stream_rows.cu", "head_rows.cu", "linear_state.cu"}
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread", "-march=x86-64-v3"]
 
 
@@ -169,10 +170,13 @@ def build_bounds(force: bool = False, verbose: bool = False) -> Path:
 #: what serving a hybrid decoder needs of the kernel library, for programs that compile on first use
 HYBRID_TUS = ["common/host.cu", "kernels/attn_rows.cu", "kernels/delta.cu", "kernels/depth_rows.cu", "kernels/experts.cu",
               "kernels/flash_fwd.cu",
-              "kernels/gemm_2cta.cu", "kernels/gemm_groups.cu", "kernels/gemm_tcgen05.cu", "kernels/hybrid_rows.cu",
-              "kernels/latent_decode.cu", "kernels/latent_rows.cu", "kernels/mamba2.cu", "kernels/mlstm.cu", "kernels/paged_kv.cu",
+              "kernels/gemm_2cta.cu", "kernels/gemm_groups.cu", "kernels/gemm_tcgen05.cu", "kernels/head_rows.cu",
+              "kernels/hybrid_rows.cu",
+              "kernels/latent_decode.cu", "kernels/latent_rows.cu", "kernels/linear_state.cu",
+              "kernels/mamba2.cu", "kernels/mlstm.cu", "kernels/paged_kv.cu",
               "kernels/rglru.cu",
-              "kernels/router_quant_sample.cu", "kernels/sgemm.cu", "kernels/ssd_tcgen05.cu", "serve/hybrid_forward.cu"]
+              "kernels/router_quant_sample.cu", "kernels/sgemm.cu", "kernels/ssd_tcgen05.cu",
+              "kernels/stream_rows.cu", "serve/hybrid_forward.cu"]
 HYBRID_LIB = LIBDIR / "libbrain_b200_hybrid.so"
 #: ... and of the host runtime (checkpoint reader, pages, slots, scheduler)
 HYBRID_HOST_SRCS = ["runtime/data.cpp", "runtime/safetensors.cpp", "runtime/serving.cpp"]

@@ -33,6 +33,8 @@ _ARCHS: List[Arch] = [
          "recurrence layers, depth averages", ("import", "infer", "serve", "trace")),
     Arch("zepesun", "hybrid", "Hybrid decoder: latent attention, matrix memories and windowed attention beside them, "
          "mixture of experts", ("import", "infer", "serve", "trace")),
+    Arch("povipel", "hybrid", "Hybrid decoder: retention, windowed attention with pooled blocks beside gated linear attention, "
+         "residual streams, looped layers, mixture of experts", ("import", "infer", "serve", "trace")),
     Arch("splat", "splat", "3D Gaussian splat rasteriser (headless)", ("render", "train"), built=True),
 ]
 

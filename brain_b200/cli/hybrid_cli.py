@@ -1,4 +1,4 @@
-"""``brain pakalix|nezalorn|zepesun <import|infer|serve|trace>``: hybrid decoders (attention and recurrent layers) on the
+"""``brain pakalix|nezalorn|zepesun|povipel <import|infer|serve|trace>``: hybrid decoders (attention and recurrent layers) on the
 serving engine.  ``--model`` takes a directory with ``config.json`` and ``model.safetensors`` or a brain
 checkpoint; prompts are text with ``--tokenizer`` or token ids with ``--tokens 1,2,3``."""
 from __future__ import annotations

@@ -37,7 +37,7 @@ model commands
   toymoe   train [--steps N --batch-size B --block-size T --lr X --out F]
            infer --weights F [--prompt 1,2,3,4 --max-new N --temperature X --top-k K]
            eval  --weights F [--samples N]
-  pakalix, nezalorn, zepesun
+  pakalix, nezalorn, zepesun, povipel
            import DIR [--out F | --id VENDOR/REPO]
            infer|serve --model DIR|F (--tokenizer T --prompt "..." | --tokens 1,2,3)... [--max-new N
                  --max-batch B --temp X --top-k K --top-p P --seed S --dtype bf16|fp32]

@@ -355,29 +355,41 @@ class AttentionSpec:
     rot: Optional[RotarySpec] = None
     v_mix: bool = False          # values mixed with those of the first layer that has this set
     window: Optional[int] = None     # keys a query sees, itself included (None: every earlier one)
-    qk_norm: bool = True         # root-mean-square norm over the whole query and the whole key projection
+    qk_norm: object = True       # root-mean-square norm of queries and keys: True over the whole projections, "head" over
+                                 # every head with one gain for all of them, False none
     bias: bool = False           # on the query, key, value and output projections
-    gate: str = "head"           # sigmoid gate on the output: one value per head, or one per element
+    gate: Optional[str] = "head"     # sigmoid gate on the output: one value per head, or one per element
+    pool: Optional[int] = None   # behind the window: one mean key and value per block of this many tokens
+    sink: bool = False           # a learned number per head in the softmax's denominator
+    turn_values: bool = False    # values rotated like keys (over all of a head), outputs rotated back
     kind = "attention"
     recurrent = False
 
     @staticmethod
-    def from_json(m: dict, **constants) -> "AttentionSpec":
+    def from_json(m: dict, interleaved: bool = False, **constants) -> "AttentionSpec":
         rot, mask = m.get("rot"), m.get("mask") or {}
         return AttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
                              scale=float(m["scale"]), softcap=float(m["softcap"]) if m.get("softcap") else None,
-                             rot=RotarySpec.from_json(rot) if rot else None, v_mix=bool(m.get("v_mix", False)),
-                             window=int(mask["size"]) if mask.get("size") else None, **constants)
+                             rot=RotarySpec.from_json(rot, interleaved=interleaved) if rot else None,
+                             v_mix=bool(m.get("v_mix", False)), window=int(mask["size"]) if mask.get("size") else None,
+                             pool=int(mask["pool"]) if mask.get("pool") else None, **constants)
 
     def to_json(self) -> dict:
-        m = {k: v for k, v in asdict(self).items() if v is not None and k not in ("window", "qk_norm", "bias", "gate")}
+        m = {k: v for k, v in asdict(self).items()
+             if v is not None and k not in ("window", "qk_norm", "bias", "gate", "pool", "sink", "turn_values")}
         if self.rot is not None:
             m["rot"] = {"dims": self.rot.dims, "base": self.rot.base}
         if self.window is not None:
             m["mask"] = {"size": self.window}
-        if not self.qk_norm:
+            if self.pool is not None:
+                m["mask"]["pool"] = self.pool
+        if self.qk_norm is not True:
             del m["v_mix"]
         return m
+
+    @property
+    def value_rot(self) -> Optional[RotarySpec]:
+        return RotarySpec(self.vdim, self.rot.base, interleaved=self.rot.interleaved) if self.turn_values and self.rot else None
 
     def check(self):
         if self.heads % self.kv_heads:
@@ -388,6 +400,14 @@ class AttentionSpec:
             raise ValueError("attention: the window holds at least the token itself")
         if not self.qk_norm and (self.rot is not None or self.v_mix):
             raise ValueError("attention: rotation and value mixing come with normed queries and keys")
+        if self.pool is not None and (self.pool < 1 or self.window is None):
+            raise ValueError("attention: pooled blocks hold a token or more and lie behind a window")
+        if self.turn_values and (self.rot is None or self.vdim % 2):
+            raise ValueError(f"attention: cannot rotate values of {self.vdim} dimensions")
+        if self.qk_norm == "head" and (self.softcap is not None or self.v_mix or self.bias):
+            raise ValueError("attention: soft caps, value mixing and biases do not come with norms per head")
+        if self.qk_norm != "head" and (self.pool is not None or self.sink or self.turn_values or self.gate is None):
+            raise ValueError("attention: pooled blocks, sinks and rotated values come with norms per head")
 
     def tensors(self, width: int):
         out = []
@@ -395,15 +415,24 @@ class AttentionSpec:
             out.append((n, (rows, width)))
             if self.bias:
                 out.append((n + ".b", (rows,)))
-        if self.qk_norm:
+        if self.qk_norm == "head":
+            out += [("q.norm", (self.dim,)), ("k.norm", (self.dim,))]
+        elif self.qk_norm:
             out += [("q.norm", (self.heads * self.dim,)), ("k.norm", (self.kv_heads * self.dim,))]
         if self.v_mix:
             out.append(("vmix", ()))
-        out += [("g", (self.heads * (self.vdim if self.gate == "element" else 1), width)), ("o", (width, self.heads * self.vdim))]
+        if self.sink:
+            out.append(("sink", (self.heads,)))
+        if self.gate is not None:
+            out.append(("g", (self.heads * (self.vdim if self.gate == "element" else 1), width)))
+        out.append(("o", (width, self.heads * self.vdim)))
         return out + [("o.b", (width,))] if self.bias else out
 
     def flops(self, T: int) -> float:
-        return 2.0 * self.heads * (self.dim + self.vdim) * min(T, self.window or T)
+        keys = min(T, self.window or T)
+        if self.pool is not None:
+            keys += (T - keys) // self.pool
+        return 2.0 * self.heads * (self.dim + self.vdim) * keys
 
 
 @dataclass
@@ -625,21 +654,113 @@ class MlstmSpec:
 
 
 @dataclass
+class GatedLinearSpec:
+    """Linear attention whose state (key x value channels per head) decays by a rate of its own for every key channel
+    and token, sigmoid(z)^(1 / tau) with z from a low-rank projection of ``decay_rank`` (0: as the checkpoint has it)."""
+    heads: int
+    dim: int                     # query / key head size
+    vdim: int
+    tau: float
+    decay_rank: int = 0
+    kind = "gated_linear"
+    recurrent = True
+
+    @staticmethod
+    def from_json(m: dict) -> "GatedLinearSpec":
+        return GatedLinearSpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), tau=float(m["tau"]),
+                               decay_rank=int(m.get("decay_rank") or 0))
+
+    def to_json(self) -> dict:
+        return {k: v for k, v in asdict(self).items() if v}
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    def fill(self, shape):
+        self.decay_rank = self.decay_rank or shape("a1")[0]
+
+    def check(self):
+        if not self.tau > 0:
+            raise ValueError("gated linear attention: the decay's root is positive")
+        if self.dim > 512:
+            raise ValueError("gated linear attention: heads of up to 512 key channels")
+
+    def tensors(self, width: int):
+        k, v = self.heads * self.dim, self.heads * self.vdim
+        return [("q", (k, width)), ("k", (k, width)), ("v", (v, width)), ("g", (v, width)), ("o", (width, v)),
+                ("norm", (self.vdim,)), ("a1", (self.decay_rank, width)), ("a2", (k, self.decay_rank)), ("a2.b", (k,))]
+
+    def flops(self, T: int) -> float:
+        return 6.0 * self.heads * self.dim * self.vdim
+
+
+@dataclass
+class RetentionSpec:
+    """Linear attention whose state decays by a constant per head; queries and keys are rotated."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: List[float]
+    rot: Optional[RotarySpec] = None
+    kind = "retention"
+    recurrent = True
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @staticmethod
+    def from_json(m: dict, interleaved: bool = False) -> "RetentionSpec":
+        rot = m.get("rot")
+        return RetentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), decay=[float(x) for x in m["decay"]],
+                             rot=RotarySpec.from_json(rot, interleaved=interleaved) if rot else None)
+
+    def to_json(self) -> dict:
+        m = {"heads": self.heads, "dim": self.dim, "vdim": self.vdim, "decay": list(self.decay)}
+        return m if self.rot is None else dict(m, rot={"dims": self.rot.dims, "base": self.rot.base})
+
+    def check(self):
+        if len(self.decay) != self.heads or not all(0.0 < x <= 1.0 for x in self.decay):
+            raise ValueError(f"retention: a decay in (0, 1] for each of {self.heads} heads")
+        if self.rot is not None and (self.rot.dims % 2 or self.rot.dims > self.dim):
+            raise ValueError(f"retention: cannot rotate {self.rot.dims} of {self.dim} dimensions")
+        if self.dim > 512:
+            raise ValueError("retention: heads of up to 512 key channels")
+
+    def tensors(self, width: int):
+        k, v = self.heads * self.dim, self.heads * self.vdim
+        return [("q", (k, width)), ("k", (k, width)), ("v", (v, width)), ("g", (v, width)), ("o", (width, v))]
+
+    def flops(self, T: int) -> float:
+        return 6.0 * self.heads * self.dim * self.vdim
+
+
+@dataclass
 class ParallelSpec:
-    """Two mixers reading the same input; their results are added with a factor each."""
+    """Two mixers reading the same input; their results are added with a factor each, either as they are or
+    (``normed``) each over its root mean square and times a gain."""
     left: object
     right: object
     left_scale: float
     right_scale: float
+    normed: bool = False
     kind = "parallel"
 
     @staticmethod
-    def from_json(m: dict, left, right) -> "ParallelSpec":
-        return ParallelSpec(left(m["left"]), right(m["right"]), float(m["left_scale"]), float(m["right_scale"]))
+    def from_json(m: dict, left, right, normed: bool = False) -> "ParallelSpec":
+        factor = (lambda n: 0.5) if normed else (lambda n: float(m[n]))
+        return ParallelSpec(left(m["left"]), right(m["right"]), factor("left_scale"), factor("right_scale"), normed)
 
     def to_json(self) -> dict:
-        return {"left": self.left.to_json(), "left_scale": self.left_scale, "right": self.right.to_json(),
-                "right_scale": self.right_scale}
+        m = {"left": self.left.to_json(), "right": self.right.to_json()}
+        return m if self.normed else dict(m, left_scale=self.left_scale, right_scale=self.right_scale)
+
+    def fill(self, shape):
+        for side in ("left", "right"):
+            m = getattr(self, side)
+            if hasattr(m, "fill"):
+                m.fill(lambda n, side=side: shape(side + "." + n))
 
     @property
     def recurrent(self) -> bool:
@@ -650,7 +771,8 @@ class ParallelSpec:
         self.right.check()
 
     def tensors(self, width: int):
-        return [(side + "." + n, s) for side in ("left", "right") for n, s in getattr(self, side).tensors(width)]
+        out = [(side + "." + n, s) for side in ("left", "right") for n, s in getattr(self, side).tensors(width)]
+        return out + [("left.out", (width,)), ("right.out", (width,))] if self.normed else out
 
     def flops(self, T: int) -> float:
         return self.left.flops(T) + self.right.flops(T)
@@ -713,33 +835,69 @@ class GeluGluSpec:
 
 
 @dataclass
+class GeluSpec:
+    """gelu (in its tanh form) between the up and down projections."""
+    ff: int
+    kind = "gelu"
+
+    @staticmethod
+    def from_json(f: dict) -> "GeluSpec":
+        return GeluSpec(int(f["ff"]))
+
+    def to_json(self) -> dict:
+        return {"kind": "dense", "ff": self.ff}
+
+    def tensors(self, width: int):
+        return [("up", (self.ff, width)), ("down", (width, self.ff))]
+
+
+@dataclass
+class SiluGluSpec:
+    """silu(gate) up between the gate / up and down projections: the clamped unit without its bounds."""
+    ff: int
+    kind = "silu_glu"
+    limit, alpha, shift = math.inf, 1.0, 0.0
+
+    @staticmethod
+    def from_json(f: dict) -> "SiluGluSpec":
+        return SiluGluSpec(int(f["ff"]))
+
+    def tensors(self, width: int):
+        return [("gate", (self.ff, width)), ("up", (self.ff, width)), ("down", (width, self.ff))]
+
+
+@dataclass
 class RoutedSpec:
-    """Mixture of clamped gated experts.  A router's softmax scores pick ``top`` experts of every token, within
-    the ``keep`` groups (of ``groups`` equal ones) whose best expert scores highest; their weights are their
-    scores over the scores' sum, times ``scale``.  An optional shared expert runs for every token."""
-    expert: ClampedGluSpec
+    """Mixture of gated experts.  A router's scores (their softmax, or the sigmoid of each) pick ``top`` experts of
+    every token, within the ``keep`` groups (of ``groups`` equal ones) whose best expert scores highest.  An expert's
+    weight is its score (softmax: over the chosen scores' sum), times ``scale``; it multiplies the expert's output, or
+    with ``weigh_input`` its input.  An optional shared expert runs for every token."""
+    expert: object
     experts: int
     top: int
     groups: int = 1
     keep: int = 1
     scale: float = 1.0
-    shared: Optional[ClampedGluSpec] = None
+    shared: Optional[object] = None
+    scores: str = "softmax"
+    weigh_input: bool = False
     kind = "routed"
     #: added to the sum that the chosen scores are divided by
     tiny = 1e-20
 
     @staticmethod
-    def from_json(f: dict) -> "RoutedSpec":
+    def from_json(f: dict, expert: type = ClampedGluSpec, **constants) -> "RoutedSpec":
         r, sh = f["router"], f.get("shared")
         g = r.get("groups") or {}
-        return RoutedSpec(ClampedGluSpec.from_json(f["expert"]), int(r["experts"]), int(r["top"]), int(g.get("count", 1)),
-                          int(g.get("keep", 1)), float(r.get("scale", 1.0)), ClampedGluSpec.from_json(sh) if sh else None)
+        return RoutedSpec(expert.from_json(f["expert"]), int(r["experts"]), int(r["top"]), int(g.get("count", 1)),
+                          int(g.get("keep", 1)), float(r.get("scale", 1.0)), expert.from_json(sh) if sh else None, **constants)
 
     def to_json(self) -> dict:
-        size = lambda e: {"ff": e.ff, "limit": e.limit}
-        out = {"kind": "moe", "expert": size(self.expert),
-               "router": {"experts": self.experts, "groups": {"count": self.groups, "keep": self.keep}, "scale": self.scale,
-                          "top": self.top}}
+        size = lambda e: {"ff": e.ff, "limit": e.limit} if e.kind == "clamped_glu" else {"ff": e.ff}
+        router = {"experts": self.experts, "top": self.top}
+        if self.scores == "softmax":
+            router.update(groups={"count": self.groups, "keep": self.keep}, scale=self.scale)
+        out = {"kind": "moe", "expert": size(self.expert), "router": router}
         return out if self.shared is None else dict(out, shared=size(self.shared))
 
     def check(self):
@@ -785,7 +943,7 @@ class HybridDesign:
     """What the layers of a design have in common."""
     mixers: tuple                # mixers its layers may name
     mlp: type                    # its dense feed-forward
-    routed: Optional[type] = None    # its mixture of experts
+    routed: Optional[object] = None  # its mixture of experts
     norm_offset: float = 0.0     # norms multiply by this plus the stored gain
     embed_norm: bool = False     # a norm behind the embedding
     positions: bool = False      # a factor on the embedding, and a learned vector per position added to it
@@ -793,6 +951,16 @@ class HybridDesign:
     depth_average: bool = False  # what a layer passes on is a weighted sum of all results so far
     tied: bool = False           # the embedding table is the output projection
     residual_mult: bool = False  # a factor on what a layer adds
+    streams: bool = False        # several copies of the residual stream: every sublayer (the mixer, then the feed-forward,
+                                 # each with a norm of its own) reads a weighted sum of them and is spread over their mixture
+    layer_norm: bool = False     # norms subtract the mean and have a bias
+    token_shift: bool = False    # a mixer's input is moved towards that of the token before, channel by channel
+    loop: bool = False           # a run of layers may be passed several times, with caches and states for each pass
+    logit_softcap: bool = False
+
+    @property
+    def embed_factor(self) -> bool:
+        return self.positions or self.streams
 
 
 _MATRIX_MEMORY = mixer_form(MlstmSpec)
@@ -805,7 +973,15 @@ HYBRID_FAMILY = {
                              mixer_form(ParallelSpec, left=mixer_form(AttentionSpec, qk_norm=False, bias=True, gate="element"),
                                         right=_MATRIX_MEMORY)),
                             GeluGluSpec, RoutedSpec, positions=True),
+    "Povipel": HybridDesign((mixer_form(RetentionSpec),
+                             mixer_form(ParallelSpec, normed=True, right=mixer_form(GatedLinearSpec),
+                                        left=mixer_form(AttentionSpec, interleaved=True, qk_norm="head", gate=None, sink=True,
+                                                        turn_values=True))),
+                            GeluSpec, mixer_form(RoutedSpec, expert=SiluGluSpec, scores="sigmoid", weigh_input=True),
+                            streams=True, layer_norm=True, token_shift=True, loop=True, logit_softcap=True),
 }
+#: copies of the residual stream that the kernels hold at once
+MAX_STREAMS = 16
 
 
 @dataclass
@@ -820,10 +996,22 @@ class HybridConfig:
     #: reserve pages for
     max_position_embeddings: int = 131072
     embed_scale: float = 1.0
+    streams: int = 1
+    #: (first, one past the last, times): layers that run several times in a row
+    loop: Optional[tuple] = None
+    logit_softcap: Optional[float] = None
 
     def __post_init__(self):
         if not self.layers:
             raise ValueError("a hybrid decoder needs at least one layer")
+        if not 1 <= self.streams <= MAX_STREAMS:
+            raise ValueError(f"{self.streams} residual streams: 1 to {MAX_STREAMS}")
+        if self.loop is not None:
+            a, b, times = self.loop
+            if not 0 <= a <= b <= len(self.layers) or times < 1:
+                raise ValueError(f"loop: layers {a} to {b} of {len(self.layers)}, {times} times")
+        if self.logit_softcap is not None and not self.logit_softcap > 0:
+            raise ValueError("the logits' bound is positive")
         vals = set()
         for i, l in enumerate(self.layers):
             m = l.mixer
@@ -850,6 +1038,15 @@ class HybridConfig:
         return len(self.layers)
 
     @property
+    def runs(self) -> List[int]:
+        """Which layer runs, pass by pass."""
+        n = self.n_layers
+        if self.loop is None:
+            return list(range(n))
+        a, b, times = self.loop
+        return list(range(a)) + list(range(a, b)) * times + list(range(b, n))
+
+    @property
     def d_model(self) -> int:
         return self.width
 
@@ -859,7 +1056,7 @@ class HybridConfig:
 
     @property
     def recurrent(self) -> bool:
-        return any(l.mixer.recurrent for l in self.layers)
+        return self.traits.token_shift or any(l.mixer.recurrent for l in self.layers)
 
     # ---- JSON: the design's own config file
     def to_json(self) -> dict:
@@ -869,15 +1066,24 @@ class HybridConfig:
                "norm": {"eps": self.eps}}
         if self.traits.residual_mult:
             out["residual_mult"] = self.residual_mult
+        if self.traits.embed_factor:
+            out["embedding"] = {"scale": self.embed_scale}
         if self.traits.positions:
-            out.update(embedding={"scale": self.embed_scale}, max_positions=self.max_position_embeddings)
+            out["max_positions"] = self.max_position_embeddings
+        if self.traits.streams:
+            out["streams"] = self.streams
+        if self.loop is not None:
+            out["loop"] = dict(zip(("start", "stop", "times"), self.loop))
+        if self.logit_softcap is not None:
+            out["logit_softcap"] = self.logit_softcap
         return out
 
     @staticmethod
     def from_json(c: dict) -> "HybridConfig":
         design = HYBRID_FAMILY[c["architecture"]]
         mixers = {m.kind: m for m in design.mixers}
-        mlps = {"dense": design.mlp, "moe": design.routed}
+        read = lambda f: f.from_json if isinstance(f, type) else f
+        mlps = {"dense": read(design.mlp), "moe": design.routed and read(design.routed)}
         layers = []
         for i, e in enumerate(c["layers"]):
             if e["type"] not in mixers:
@@ -886,11 +1092,18 @@ class HybridConfig:
             if f is not None and mlps.get(f.get("kind", "dense")) is None:
                 raise ValueError(f"layer {i}: unknown feed-forward {f['kind']!r}")
             layers.append(HybridLayer(mixers[e["type"]](e["mixer"]),
-                                      None if f is None else mlps[f.get("kind", "dense")].from_json(f)))
+                                      None if f is None else mlps[f.get("kind", "dense")](f)))
         more = {}
+        if design.embed_factor:
+            more["embed_scale"] = float((c.get("embedding") or {}).get("scale", 1.0))
         if design.positions:
-            more = dict(max_position_embeddings=int(c["max_positions"]),
-                        embed_scale=float((c.get("embedding") or {}).get("scale", 1.0)))
+            more["max_position_embeddings"] = int(c["max_positions"])
+        if design.streams:
+            more["streams"] = int(c.get("streams") or 1)
+        if design.loop and c.get("loop"):
+            more["loop"] = tuple(int(c["loop"][k]) for k in ("start", "stop", "times"))
+        if design.logit_softcap and c.get("logit_softcap"):
+            more["logit_softcap"] = float(c["logit_softcap"])
         return HybridConfig(vocab=int(c["vocab"]), width=int(c["width"]), layers=layers, eps=float(c["norm"]["eps"]),
                             residual_mult=float(c.get("residual_mult", 1.0)), design=c["architecture"], **more)
 
@@ -903,21 +1116,28 @@ class HybridConfig:
     def tensors(self):
         """(name, shape) of every tensor of a checkpoint, in order."""
         d, t = self.width, self.traits
+        norm = lambda n: [(n, (d,)), (n + ".b", (d,))] if t.layer_norm else [(n, (d,))]
         out = [("embed", (self.vocab, d))]
         if t.embed_norm:
             out.append(("embed.norm", (d,)))
         if t.positions:
             out.append(("pos", (self.max_position_embeddings, d)))
         for i, l in enumerate(self.layers):
-            out.append((f"l{i}.norm1", (d,)))
-            if t.two_norms and l.mlp is not None:
-                out.append((f"l{i}.norm2", (d,)))
+            out += norm(f"l{i}.norm1")
+            if (t.two_norms or t.streams) and l.mlp is not None:
+                out += norm(f"l{i}.norm2")
             out += [(f"l{i}.mix.{n}", s) for n, s in l.mixer.tensors(d)]
             if l.mlp is not None:
                 out += [(f"l{i}.mlp.{n}", s) for n, s in l.mlp.tensors(d)]
             if t.depth_average:
                 out.append((f"l{i}.dwa", (i + 2,)))
-        out.append(("final.norm", (d,)))
+            if t.streams:
+                n = self.streams
+                for q in (1,) if l.mlp is None else (1, 2):
+                    out += [(f"l{i}.hc{q}.in", (n,)), (f"l{i}.hc{q}.out", (n,)), (f"l{i}.hc{q}.mix", (n, n))]
+            if t.token_shift:
+                out.append((f"l{i}.shift", (d,)))
+        out += norm("final.norm")
         return out if t.tied else out + [("head", (self.vocab, d))]
 
     def param_list(self):

@@ -5,6 +5,8 @@ Nezalorn mixers: windowed latent attention, a generalised delta rule, or a real-
 what a layer passes on is a weighted sum of all results so far.
 Zepesun mixers: latent attention, a matrix memory with exponential gates, or windowed attention and a matrix
 memory side by side; feed-forwards dense or a mixture of experts; learned positions.
+Povipel mixers: retention, or windowed attention with pooled blocks behind the window beside gated linear attention;
+several residual streams, token shifts, layers that run several times.
 
 This is the weight container of the family (names, shapes, initial values, loading); its forward lives in
 the serving engine (``serve.hybrid.HybridEngine`` over ``csrc/serve/hybrid_forward.cu``)."""
@@ -52,7 +54,24 @@ class HybridDecoder(nn.Module):
             p = self.tensor(name)
             leaf = name.split(".", 2)[-1] if name[0] == "l" and name[1].isdigit() else name
             leaf = leaf.removeprefix("left.").removeprefix("right.")
-            if leaf in ("embed.norm", "final.norm") or name.endswith((".norm1", ".norm2")):
+            streams = self.cfg.streams
+            if name.endswith(("hc1.in", "hc2.in")):
+                v = (1.0 + 0.3 * normal(shape)) / streams
+            elif name.endswith(("hc1.out", "hc2.out")):
+                v = uniform(shape, 0.3, 1.2)
+            elif name.endswith(("hc1.mix", "hc2.mix")):
+                v = torch.eye(streams, device=dev) * 0.8 + 0.2 * normal(shape) / streams
+            elif name.endswith(".shift"):
+                v = uniform(shape, 0.0, 0.8)
+            elif name.endswith((".norm1.b", ".norm2.b")) or name == "final.norm.b":
+                v = 0.1 * normal(shape)
+            elif leaf == "sink":
+                v = uniform(shape, 0.0, 3.0)
+            elif leaf == "a2.b":
+                v = uniform(shape, -1.0, 5.0)                            # decays between fast and slow
+            elif leaf == "out":
+                v = 1.0 + 0.1 * normal(shape)
+            elif leaf in ("embed.norm", "final.norm") or name.endswith((".norm1", ".norm2")):
                 v = 1.0 - self.cfg.traits.norm_offset + 0.1 * normal(shape)
             elif leaf in ("q.norm", "k.norm", "norm", "dq.norm", "dkv.norm"):
                 v = 1.0 + 0.1 * normal(shape)
@@ -116,12 +135,14 @@ class HybridDecoder(nn.Module):
 
     def flops_per_token(self, T: int, train: bool = False) -> float:
         """Matrix-product FLOPs of one token with T tokens of context, attention and recurrence included."""
-        total = 0.0
+        total, runs = 0.0, self.cfg.runs
         for n, s in self.cfg.tensors():
-            if len(s) > 1 and n != "pos" and (n != "embed" or self.cfg.traits.tied) and not n.endswith((".conv", "a.b", "i.b")):
+            if len(s) > 1 and n != "pos" and ".hc" not in n and (n != "embed" or self.cfg.traits.tied) and not n.endswith((".conv", "a.b", "i.b")):
                 share = 1.0
                 if ".mlp.e" in n:            # of a token's own experts
                     f = self.cfg.layers[int(n[1:n.index(".")])].mlp
                     share = f.top / f.experts
+                if n[0] == "l" and n[1].isdigit():
+                    share *= runs.count(int(n[1:n.index(".")]))
                 total += 2.0 * share * math.prod(s)
-        return total + sum(l.mixer.flops(T) for l in self.cfg.layers)
+        return total + sum(self.cfg.layers[i].mixer.flops(T) for i in self.cfg.runs)

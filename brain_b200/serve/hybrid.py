@@ -1,15 +1,19 @@
-"""Serving engine of the hybrid decoders (Pakalix, Nezalorn, Zepesun): pages for the attention layers, recurrent-state
+"""Serving engine of the hybrid decoders (Pakalix, Nezalorn, Zepesun, Povipel): pages for the attention layers, recurrent-state
 slots for the recurrent layers, one native call per step.
 
 * A step is ONE packed batch: prompt portions of any length and single decoded tokens of several
   sequences run together (``csrc/serve/hybrid_forward.cu``).  Every entry point - the scheduler's prefill,
   mixed and decode calls and :meth:`HybridEngine.step_logits` - goes through it.
 * Pages: per attention layer keys and values ``[num_blocks + 1, kv_heads, block_size, head size]``, per latent
-  attention layer with latents of its own ``[num_blocks + 1, block_size, latent | rotated key part]``.
+  attention layer with latents of its own ``[num_blocks + 1, block_size, latent | rotated key part]``; where blocks of
+  tokens are pooled behind a window, their means ``[num_blocks + 1, kv_heads, ceil(block_size / pool), head size]``,
+  each in the page of the block's last token, so that the tokens' page table names them.
   State slots: per recurrent layer the fp32 state (``[heads, state, head size]``, ``[heads, key, value]``, a
   matrix memory with its normaliser and running maximum, or one value per channel) and, where it has a
-  convolution, a ring of the last taps - 1 raw inputs.  A sequence at position 0 starts from zeros, so pages
-  and slots are reused as they are.
+  convolution, a ring of the last taps - 1 raw inputs; with a token shift the last input of every layer.  A sequence
+  at position 0 starts from zeros, so pages and slots are reused as they are.
+* Layers that run several times share their weights; every pass is a layer of its own here, with its own pages and
+  slots.
 * Mixtures of experts: rows of a step sorted by expert onto 128-row tiles, one grouped product per matrix.
 * ``dtype='bf16'``: bf16 weights, activations, pages and convolution inputs; the residual stream, norms,
   rotation, scores, softmax, routers, step sizes, gates of a recurrence, decays and the recurrent state are
@@ -58,8 +62,10 @@ class _Scratch:
         z = lambda *s, dtype=dt: torch.zeros(*s, device=dev, dtype=dtype)
         f32 = torch.float32
         traits = eng.cfg.traits
-        self.x = z(eng.cfg.n_layers + 1 if traits.depth_average else 1, rows, eng.dp, dtype=f32)
-        self.h, self.h2 = z(rows, eng.dp), z(rows if traits.two_norms else 1, eng.dp)
+        self.x = z(eng.cfg.n_layers + 1 if traits.depth_average else eng.cfg.streams, rows, eng.dp, dtype=f32)
+        self.h, self.h2 = z(rows, eng.dp), z(rows if traits.two_norms or traits.token_shift and portions else 1, eng.dp)
+        self.ya, self.yb = (z(rows if traits.streams else 1, eng.dp) for _ in range(2))
+        self.pk = z(max(exp, 1) if portions else 1, m["pk"])
         self.proj, self.cat = z(rows, m["proj"]), z(rows, m["cat"])
         self.xbc, self.dt, self.y = z(rows, m["xbc"]), z(rows, m["dt"], dtype=f32), z(rows, m["y"])
         self.v_first = z(rows, m["v"])
@@ -91,17 +97,17 @@ class _Scratch:
                 po, pm = max(po, n * l.kvrp), max(pm, n * 2)
         self.part_o, self.part_ml = z(po, dtype=f32), z(pm, dtype=f32)
         # segment states of the chunked recurrence (prompt portions): two machine-fulls of states
-        npmax = max([l.mem if l.kind == 5 else l.n * l.p for l in eng.mixers if l.kind in (1, 5) and max(l.n, l.p) <= 128],
+        npmax = max([l.mem if l.kind == 5 else l.n * l.p for l in eng.mixers if l.kind in (1, 5, 7) and max(l.n, l.p) <= 128],
                     default=0)
         self.seg = z(2 * 2 * eng.sm_count * (npmax + 1) if portions and not eng.fp32 and npmax else 1, dtype=f32)
         self.hn, self.logits = z(max(want, 1), eng.dp), z(max(want, 1), eng.vocabp, dtype=f32)
         w = self.work = hn.Work()
         for n in ("x", "h", "proj", "cat", "xbc", "dt", "y", "v_first", "part_o", "part_ml", "seg", "hn", "logits", "h2", "q",
                   "qa", "ol", "aux", "ckv", "kvx", "f32", "part32", "ex_in", "ex_gu", "ex_act", "ex_out", "pair_expert", "pair_row",
-                  "pair_w", "ex_count", "ex_tile"):
+                  "pair_w", "ex_count", "ex_tile", "ya", "yb", "pk"):
             setattr(w, n, _ptr(getattr(self, n)))
         w.seg_floats, w.part32_floats = self.seg.numel(), self.part32.numel()
-        w.rows, w.want_rows, w.exp_rows, w.moe_rows = rows, max(want, 1), exp, moe
+        w.rows, w.want_rows, w.exp_rows, w.moe_rows, w.pk_rows = rows, max(want, 1), exp, moe, self.pk.shape[0]
         for k in m:
             setattr(w, "ld_" + k, m[k])
         w.splits, w.pool_blocks = _MAX_SPLITS, eng.num_blocks + 1
@@ -184,20 +190,47 @@ class HybridEngine(PagedEngineBase):
     def _pages(self, *shape) -> int:
         t = torch.zeros(self.num_blocks + 1, *shape, device=self.device, dtype=self.dtype)
         self.kv_bytes += t.numel() * t.element_size()
+        self._caches[t.data_ptr()] = lambda: self._pages(*shape)
         return self._hold(t)
 
     def _slots(self, *shape, dtype=torch.float32) -> int:
         t = torch.zeros(self.state_slots + 1, *shape, device=self.device, dtype=dtype)
         self.state_bytes += t.numel() * t.element_size()
+        self._caches[t.data_ptr()] = lambda: self._slots(*shape, dtype=dtype)
         return self._hold(t)
 
-    def _rotary(self, L, rot) -> None:
+    def _pass(self, dst, src) -> None:
+        """``dst``: another pass of layer ``src``, the same weights with pages and slots of its own."""
+        C.memmove(C.byref(dst), C.byref(src), C.sizeof(src))
+        for name in hn.CACHES:
+            p = getattr(src, name)
+            if p:
+                setattr(dst, name, self._caches[p]())
+        if src.beside:
+            side = hn.Layer()
+            self._pass(side, hn.Layer.from_address(src.beside))
+            self.mixers.append(side)
+            dst.beside = C.addressof(side)
+
+    def _angles(self, rot):
         key = (rot.dims, rot.base, str(rot.scaling))
         if key not in self._rope:
             f, mag = rot.frequencies()
             ang = torch.arange(self.max_blocks * self.block_size, dtype=torch.float64)[:, None] * torch.tensor(f, dtype=torch.float64)
             self._rope[key] = tuple((mag * t).float().to(self.device) for t in (ang.cos(), ang.sin()))
-        L.cos_t, L.sin_t, L.rot = *map(_ptr, self._rope[key]), rot.dims
+        return map(_ptr, self._rope[key])
+
+    def _rotary(self, L, rot) -> None:
+        L.cos_t, L.sin_t, L.rot = *self._angles(rot), rot.dims
+
+    def _paired_rows(self, w: torch.Tensor, heads: int, rot) -> torch.Tensor:
+        """Rows of a projection in the order in which a rotated pair's are neighbours."""
+        if rot is None or rot.interleaved:
+            return w
+        per = w.view(heads, -1, w.shape[1])
+        half = rot.dims // 2
+        order = [i // 2 + (i % 2) * half for i in range(rot.dims)] + list(range(rot.dims, per.shape[1]))
+        return per[:, order].reshape(w.shape)
 
     # Every packer adds what reads the normed input to ``stack`` (to ``stack32`` where the product stays fp32) and
     # returns the mixer's output projection with its padded input width.  ``scale``: a factor on the mixer's result.
@@ -208,9 +241,14 @@ class HybridEngine(PagedEngineBase):
         L.off_k = stack.add(self._rows(p + "k", m.kv_heads, m.dim))
         L.off_v = stack.add(self._rows(p + "v", m.kv_heads, m.vdim))
         elems = m.gate == "element"
-        L.off_g = stack.add(self._rows(p + "g", m.heads, m.vdim) if elems else self._mat(p + "g"))
-        L.gate_kind, L.out_scale, L.window = 2 if elems else 1, scale, m.window or 0
-        if m.qk_norm:
+        if m.gate is not None:
+            L.off_g = stack.add(self._rows(p + "g", m.heads, m.vdim) if elems else self._mat(p + "g"))
+        L.gate_kind, L.out_scale, L.window = (2 if elems else 1) if m.gate is not None else 0, scale, m.window or 0
+        if m.qk_norm == "head":
+            L.head_norm, L.q_norm, L.k_norm = 1, *(self._vec(self._tensor(p + n + ".norm"), dkp) for n in "qk")
+            if m.rot is not None and not m.rot.interleaved:
+                raise ValueError("attention with norms per head rotates neighbouring pairs")
+        elif m.qk_norm:
             L.q_norm, L.k_norm = self._head_vec(p + "q.norm", m.heads, m.dim), self._head_vec(p + "k.norm", m.kv_heads, m.dim)
         if m.bias:
             L.q_b, L.k_b, L.v_b = (self._head_vec(p + n + ".b", h, d) for n, h, d in
@@ -223,6 +261,15 @@ class HybridEngine(PagedEngineBase):
         L.v_role = 0 if not m.v_mix else (1 if i == first else 2)
         L.vmix = float(self._tensor(p + "vmix").float()) if m.v_mix else 0.0
         L.kc, L.vc = (self._pages(m.kv_heads, self.block_size, d) for d in (dkp, dvp))
+        if m.pool is not None:
+            L.pool, L.pool_rows = m.pool, -(-self.block_size // m.pool)
+            L.pkc, L.pvc = (self._pages(m.kv_heads, L.pool_rows, d) for d in (dkp, dvp))
+            self.least_pool = min(self.least_pool or m.pool, m.pool)
+            self._widest(pk=m.kv_heads * (dkp + dvp))
+        if m.sink:
+            L.sink = self._vec(self._tensor(p + "sink"), m.heads)
+        if m.value_rot is not None:
+            L.vcos_t, L.vsin_t = self._angles(m.value_rot)
         self._widest(v=m.kv_heads * dvp)
         return self._cols(p + "o", m.heads, m.vdim), m.heads * dvp
 
@@ -343,19 +390,56 @@ class HybridEngine(PagedEngineBase):
         self._widest(y=L.innerp)
         return self._cols(p + "o", H, m.vdim), L.innerp
 
+    def _pack_linear(self, L, m, p: str, stack, rot=None):
+        """What the forms of linear attention have in common: head sizes, projections, state."""
+        H, np_, pp = m.heads, pad8(m.dim), pad8(m.vdim)
+        L.heads, L.n, L.np, L.p, L.pp, L.inner, L.innerp, L.groups = H, m.dim, np_, m.vdim, pp, m.inner, H * pp, H
+        L.q_scale = m.dim ** -0.5
+        L.off_kk, L.off_q = (stack.add(hn.padded_rows(self._paired_rows(self._mat(p + n), H, rot), H, m.dim, np_)) for n in "kq")
+        L.off_vv, L.off_gg = (stack.add(self._rows(p + n, H, m.vdim)) for n in "vg")
+        L.ssm_state = self._slots(H, m.dim, m.vdim)
+        self._widest(y=L.innerp)
+        return self._cols(p + "o", H, m.vdim), L.innerp
+
+    def _pack_gated_linear(self, i: int, L, m, p: str, stack, scale: float = 1.0):
+        out = self._pack_linear(L, m, p, stack)
+        H, np_ = m.heads, pad8(m.dim)
+        L.kind, L.decay_root = 6, 1.0 / m.tau
+        L.wr, L.wrp, L.off_w1 = m.decay_rank, pad8(m.decay_rank), stack.add(self._mat(p + "a1"))
+        L.w2 = self._lin(hn.columns([(self._rows(p + "a2", H, m.dim), L.wrp)], H * np_))
+        L.w0 = self._head_vec(p + "a2.b", H, m.dim)
+        L.gnorm = self._hold(hn.head_vec(scale * self._tensor(p + "norm").float().repeat(H), H, m.vdim, L.pp, self.device))
+        self._widest(f32=H * np_)
+        return out
+
+    def _pack_retention(self, i: int, L, m, p: str, stack):
+        out = self._pack_linear(L, m, p, stack, m.rot)
+        decay = torch.tensor(m.decay, dtype=torch.float64)
+        L.kind, L.keep_less, L.a = 7, self._vec((decay - 1.0).float(), m.heads), self._vec(decay.log().float(), m.heads)
+        if m.rot is not None and m.rot.dims:
+            self._rotary(L, m.rot)
+        return out
+
     def _pack_parallel(self, i: int, L, m, p: str, stack):
-        left = self._pack_attention(i, L, m.left, p + "left.", stack, m.left_scale)
+        ls, rs = (1.0, 1.0) if m.normed else (m.left_scale, m.right_scale)
+        left = self._pack_attention(i, L, m.left, p + "left.", stack, ls)
         R = hn.Layer()
-        right = self._pack_mlstm(i, R, m.right, p + "right.", stack, m.right_scale)
+        right = getattr(self, "_pack_" + m.right.kind)(i, R, m.right, p + "right.", stack, rs)
         R.off_cat = left[1]
         self.mixers.append(R)                  # (kept alive there)
         L.beside = C.addressof(R)
+        if m.normed:                           # each has an output projection of its own, and a gain
+            R.out = self._lin(hn.columns([right], self.dp))
+            for side, name, s in ((L, "left.out", m.left_scale), (R, "right.out", m.right_scale)):
+                side.out_gain = self._vec(s * self._tensor(p + name).float(), self.dp)
+            self._widest(cat=left[1] + right[1])
+            return [left]
         return [left, right]
 
     def _pack_routed(self, L, f, p: str) -> None:
         effp, dp, E = pad8(f.expert.ff), self.dp, f.experts
         L.n_experts, L.top, L.groups_all, L.groups_keep, L.eff, L.effp = E, f.top, f.groups, f.keep, f.expert.ff, effp
-        L.route_scale, L.route_tiny = f.scale, f.tiny
+        L.route_scale, L.route_tiny, L.score_kind, L.weigh_input = f.scale, f.tiny, int(f.scores == "sigmoid"), int(f.weigh_input)
         L.e_limit, L.e_alpha, L.e_shift = f.expert.limit, f.expert.alpha, f.expert.shift
         gu = torch.zeros(E, 2, effp, dp, device=self.device, dtype=self.dtype)
         down = torch.zeros(E, dp, effp, device=self.device, dtype=self.dtype)
@@ -370,19 +454,29 @@ class HybridEngine(PagedEngineBase):
         cfg, dev, dp = self.cfg, self.device, self.dp
         traits = cfg.traits
         T = self._tensor = model.tensor
-        n = cfg.n_layers
+        runs = cfg.runs
+        n = len(runs)
         self.layers = (hn.Layer * n)()
         self.layer_list = [self.layers[i] for i in range(n)]
+        self._caches = {}                      # of a device pointer: how to make another like it
+        self.least_pool = None                 # smallest blocks that a layer pools
         self.mixers = list(self.layer_list)    # and the second mixers of layers that have two
-        self.ld = dict.fromkeys(("proj", "cat", "xbc", "dt", "y", "v", "q", "qa", "ol", "ckv", "kvx", "aux", "f32", "gu", "act"), 8)
+        self.ld = dict.fromkeys(("proj", "cat", "xbc", "dt", "y", "v", "q", "qa", "ol", "ckv", "kvx", "aux", "f32", "gu", "act", "pk"), 8)
         self.kv_bytes = self.state_bytes = self._matrix_bytes = 0
         # prompt portions of latent attention: whether they also take the absorbed form, and how many keys the
         # widest window of a layer holds (None: all)
         self.absorb_portions, self.exp_window = False, 1
         gain = lambda name: self._vec(traits.norm_offset + T(name).float(), dp)
-        for i, spec in enumerate(cfg.layers):
-            L, p = self.layers[i], f"l{i}."
-            L.norm = gain(p + "norm1")
+        bias = lambda name: self._vec(T(name + ".b"), dp) if traits.layer_norm else None
+        for run, i in enumerate(runs):
+            first = runs.index(i)
+            if first < run:
+                self._pass(self.layers[run], self.layers[first])
+                continue
+            L, p, spec = self.layers[run], f"l{i}.", cfg.layers[i]
+            L.norm, L.norm_b = gain(p + "norm1"), bias(p + "norm1")
+            if traits.token_shift:
+                L.shift, L.shift_state = self._vec(T(p + "shift"), dp), self._slots(dp, dtype=self.dtype)
             stack, self.stack32, self.out_bias = hn.RowStack(), hn.RowStack(), []
             f, fp = spec.mlp, p + "mlp."
             if f is not None and f.kind == "routed":
@@ -392,7 +486,17 @@ class HybridEngine(PagedEngineBase):
             sections = getattr(self, "_pack_" + spec.mixer.kind)(i, L, spec.mixer, p + "mix.", stack)
             sections = sections if isinstance(sections, list) else [sections]
             width = stack.n
-            if f is not None:
+            if traits.streams:                 # a feed-forward behind the mixer, each spread over the streams
+                for q in range(2 if spec.mlp is not None else 1):
+                    L.hc[q] = self._hold(torch.cat([T(f"{p}hc{q + 1}.{k}").float().reshape(-1) for k in ("in", "out", "mix")]).to(dev))
+                if spec.mlp is not None:
+                    L.norm2, L.norm2_b = gain(p + "norm2"), bias(p + "norm2")
+                if f is not None:
+                    ffp = pad8(f.ff)
+                    L.up = self._lin(hn.columns([(self._mat(fp + "up"), dp)], ffp))
+                    L.down = self._lin(hn.columns([(self._mat(fp + "down"), ffp)], dp))
+                    self._widest(proj=ffp, cat=ffp)
+            elif f is not None:
                 ffp = pad8(f.ff)
                 L.ff, L.off_act = f.ff, sum(w for _, w in sections)
                 if f.kind == "polynorm":
@@ -422,7 +526,7 @@ class HybridEngine(PagedEngineBase):
         c = self.ccfg = hn.Cfg()
         c.dtype, c.width, c.dp, c.vocab, c.vocabp = int(self.fp32), cfg.width, dp, cfg.vocab, self.vocabp
         c.n_layers, c.block_size, c.eps, c.residual_mult = n, self.block_size, cfg.eps, cfg.residual_mult
-        c.depth_avg = int(traits.depth_average)
+        c.depth_avg, c.streams, c.logit_cap = int(traits.depth_average), cfg.streams if traits.streams else 0, cfg.logit_softcap or 0.0
         pad_cols = lambda name: self._hold_matrix(hn.columns([(self._mat(name), dp)], self.vocabp))
         c.embed = pad_cols("embed")
         if traits.positions:
@@ -432,9 +536,9 @@ class HybridEngine(PagedEngineBase):
         c.embed_scale = cfg.embed_scale
         c.head = c.embed if traits.tied else pad_cols("head")
         c.embed_norm = gain("embed.norm") if traits.embed_norm else None
-        c.final_norm = gain("final.norm")
+        c.final_norm, c.final_norm_b = gain("final.norm"), bias("final.norm")
         c.layers = C.cast(self.layers, C.c_void_p)
-        del self._tensor, self.stack32, self.out_bias
+        del self._tensor, self.stack32, self.out_bias, self._caches
 
     # ------------------------------------------------------------------ accounting
     def kv_pool_bytes(self) -> int:
@@ -509,7 +613,8 @@ class HybridEngine(PagedEngineBase):
         exp_src, kv_row0, kv_pos0 = self._expansion(starts[:ns_pre], ctx[:ns_pre], tables)
         parts = [tok, pos, row_seq, row0, starts, ctx, slot, tables.reshape(-1),
                  np.array([t[0] for t in tiles], dtype=np.int32), np.array([t[1] for t in tiles], dtype=np.int32),
-                 np.array(want, dtype=np.int32), exp_src, kv_row0, kv_pos0]
+                 np.array(want, dtype=np.int32), exp_src, kv_row0, kv_pos0,
+                 np.concatenate([[0], np.cumsum(ctx[:ns_pre])]).astype(np.int32)]
         offs = np.concatenate([[0], np.cumsum([-(-p.size // 4) * 4 for p in parts])]).astype(np.int64)
         blob = np.zeros(int(offs[-1]), dtype=np.int32)
         for o, p in zip(offs[:-1].tolist(), parts):
@@ -518,13 +623,15 @@ class HybridEngine(PagedEngineBase):
         base = d_blob.data_ptr()
         b = hn.Batch()
         for name, o in zip(("tok", "pos", "row_seq", "seq_row0", "seq_pos0", "seq_ctx", "seq_slot", "tables", "tile_seq",
-                            "tile_qt", "want", "exp_src", "kv_row0", "kv_pos0"), offs[:-1].tolist()):
+                            "tile_qt", "want", "exp_src", "kv_row0", "kv_pos0", "ctx_row0"), offs[:-1].tolist()):
             setattr(b, name, base + 4 * o)
         b.max_blocks, b.n, b.n_pre, b.ns, b.ns_pre = self.max_blocks, n, n_pre, ns, ns_pre
         b.n_tiles, b.n_want, b.max_len, b.n_exp = len(tiles), len(want), max(lens[:ns_pre], default=0), exp_src.size
+        b.max_ctx = int(ctx[:ns_pre].max(initial=0))
+        pooled = int(ctx[:ns_pre].sum()) // self.least_pool if self.least_pool else 0
         up = lambda v, q: -(-v // q) * q
         sc = self._scratch_for("step", up(n, 256), up(len(want), 16), up(ns - ns_pre, 16) if ns > ns_pre else 0,
-                               up(exp_src.size, 256))
+                               up(max(exp_src.size, pooled), 256))
         return sc, b, d_blob
 
     def _expansion(self, starts, ctx, tables):
@@ -551,10 +658,10 @@ class HybridEngine(PagedEngineBase):
 
     @torch.no_grad()
     def residual_trace(self, tokens: Sequence[int]) -> torch.Tensor:
-        """The fp32 residual stream [layers, tokens, width] after every layer of one fresh sequence (pages
-        0.. and the dummy slot are used: for offline inspection of an idle engine)."""
+        """The fp32 residual stream [layer runs, tokens, width] (the sum where there are several) after every layer run
+        of one fresh sequence (pages 0.. and the dummy slot are used: for offline inspection of an idle engine)."""
         n = len(tokens)
-        out = torch.zeros(self.cfg.n_layers, n, self.dp, device=self.device)
+        out = torch.zeros(len(self.layers), n, self.dp, device=self.device)
         bt = np.arange(self.max_blocks, dtype=np.int32)
         self._step([Entry(np.asarray(tokens, dtype=np.int32), 0, bt, self.dummy_slot, list(range(n)))], out)
         torch.cuda.synchronize()

@@ -45,19 +45,28 @@ class Layer(C.Structure):
                 ("np", I), ("mem", I), ("gate_cap", F), ("q_scale", F), ("f_b", P),
                 ("n_experts", I), ("top", I), ("groups_all", I), ("groups_keep", I), ("eff", I), ("effp", I),
                 ("route_scale", F), ("route_tiny", F), ("e_limit", F), ("e_alpha", F), ("e_shift", F),
-                ("w_egu", P), ("w_edown", P)]
+                ("w_egu", P), ("w_edown", P), ("score_kind", I), ("weigh_input", I),
+                ("norm_b", P), ("norm2_b", P), ("shift", P), ("shift_state", P), ("hc", P * 2), ("down", Lin), ("out_gain", P),
+                ("head_norm", I), ("pool", I), ("pool_rows", I), ("pkc", P), ("pvc", P), ("sink", P), ("vcos_t", P), ("vsin_t", P),
+                ("decay_root", F), ("keep_less", P)]
+
+
+#: pages and slots of a layer
+CACHES = ("kc", "vc", "pkc", "pvc", "conv_state", "ssm_state", "shift_state")
 
 
 class Cfg(C.Structure):
     _fields_ = [("dtype", I), ("width", I), ("dp", I), ("vocab", I), ("vocabp", I), ("n_layers", I),
                 ("block_size", I), ("eps", F), ("residual_mult", F), ("embed", P), ("embed_norm", P),
-                ("final_norm", P), ("head", P), ("layers", P), ("pos", P), ("max_pos", I), ("embed_scale", F), ("depth_avg", I)]
+                ("final_norm", P), ("head", P), ("layers", P), ("pos", P), ("max_pos", I), ("embed_scale", F), ("depth_avg", I),
+                ("streams", I), ("final_norm_b", P), ("logit_cap", F)]
 
 
 class Batch(C.Structure):
     _fields_ = [(n, P) for n in ("tok", "pos", "row_seq", "seq_row0", "seq_pos0", "seq_ctx", "seq_slot", "tables",
                                  "tile_seq", "tile_qt", "want", "exp_src", "kv_row0", "kv_pos0")] + \
-               [(n, I) for n in ("n_exp", "max_blocks", "n", "n_pre", "ns", "ns_pre", "n_tiles", "n_want", "max_len")]
+               [(n, I) for n in ("n_exp", "max_blocks", "n", "n_pre", "ns", "ns_pre", "n_tiles", "n_want", "max_len")] + \
+               [("ctx_row0", P), ("max_ctx", I)]
 
 
 class Work(C.Structure):
@@ -70,7 +79,8 @@ class Work(C.Structure):
                [("f32", P), ("part32", P), ("part32_floats", C.c_long)] + \
                [(n, P) for n in ("ex_in", "ex_gu", "ex_act", "ex_out", "pair_expert", "pair_row", "pair_w", "ex_count",
                                  "ex_tile")] + \
-               [(n, I) for n in ("ld_f32", "ld_gu", "ld_act", "moe_rows")]
+               [(n, I) for n in ("ld_f32", "ld_gu", "ld_act", "moe_rows")] + \
+               [("ya", P), ("yb", P), ("pk", P), ("ld_pk", I), ("pk_rows", I)]
 
 
 def padded_rows(w: torch.Tensor, heads: int, size: int, sizep: int) -> torch.Tensor:

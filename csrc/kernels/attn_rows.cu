@@ -1,7 +1,9 @@
 // Attention of single query rows against the paged K/V pool, one warp per (row, query head): any head
-// sizes up to 512, bf16 or fp32 pages, soft-capped scores, windows, output gates (per head or per element).  It is the fp32 path and
-// the path of head sizes the tensor-core prefill and the split-KV decode kernels do not cover.
+// sizes up to 512, bf16 or fp32 pages, soft-capped scores, windows, means of blocks behind them, sinks, output gates (per
+// head or per element), outputs turned back.  It is the fp32 path and the path of head sizes the tensor-core prefill and
+// the split-KV decode kernels do not cover.
 #include "../common/host.hpp"
+#include "../common/pooled.hpp"
 #include "../common/ptx.cuh"
 #include "../common/rows.cuh"
 
@@ -14,7 +16,7 @@ attn_rows_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ kc, con
                  const int* __restrict__ pos, const int* __restrict__ row_seq, const int* __restrict__ tables,
                  int max_blocks, int bs, T* __restrict__ out, int ldo, const T* __restrict__ gate, int ldg, int rows,
                  int hq, int hk, int dk, int dv, int dkp, int dvp, float scale, float softcap, int gate_elems, float out_scale,
-                 int window) {
+                 int window, const BbPooled x) {
   const int w = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (w >= rows * hq) return;
   const int r = w / hq, h = w % hq, g = h / (hq / hk);
@@ -28,13 +30,23 @@ attn_rows_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ kc, con
   const int last = pos[r];
   const int* bt = tables + (size_t)row_seq[r] * max_blocks;
   float m = -INFINITY, l = 0.f;
-  for (int j = window > 0 ? max(last - window + 1, 0) : 0; j <= last; ++j) {
-    const size_t row = ((size_t)bt[j / bs] * hk + g) * bs + j % bs;
+  const int first = window > 0 ? max(last - window + 1, 0) : 0, means = x.pool > 0 ? first / x.pool : 0;
+  for (int j = first - means; j <= last; ++j) {
+    const T *kp = kc, *vp = vc;
+    size_t row;
+    if (j < first) {
+      const int e = (j - (first - means) + 1) * x.pool - 1;      // last token of the block
+      row = ((size_t)bt[e / bs] * hk + g) * x.pool_rows + e % bs / x.pool;
+      kp = static_cast<const T*>(x.pkc);
+      vp = static_cast<const T*>(x.pvc);
+    } else {
+      row = ((size_t)bt[j / bs] * hk + g) * bs + j % bs;
+    }
     float s = 0.f;
 #pragma unroll
     for (int i = 0; i < AR_VEC; ++i) {
       const int d = lane + 32 * i;
-      if (d < dk) s = fmaf(qf[i], to_f(kc[row * dkp + d]), s);
+      if (d < dk) s = fmaf(qf[i], to_f(kp[row * dkp + d]), s);
     }
     s = warp_sum(s);
     if (softcap > 0.f) s = softcap * tanhf(s / softcap);
@@ -45,7 +57,23 @@ attn_rows_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ kc, con
 #pragma unroll
     for (int i = 0; i < AR_VEC; ++i) {
       const int d = lane + 32 * i;
-      if (d < dv) o[i] = fmaf(p, to_f(vc[row * dvp + d]), o[i] * al);
+      if (d < dv) o[i] = fmaf(p, to_f(vp[row * dvp + d]), o[i] * al);
+    }
+  }
+  if (x.sink) {             // (against the maximum of both, so that neither exponential overflows)
+    const float sk = x.sink[h], mn = fmaxf(m, sk), al = expf(m - mn);
+    l = l * al + expf(sk - mn);
+#pragma unroll
+    for (int i = 0; i < AR_VEC; ++i) o[i] *= al;
+  }
+  if (x.vcos) {
+    const int half = x.vturn >> 1;
+#pragma unroll
+    for (int i = 0; i < AR_VEC; ++i) {
+      const int d = lane + 32 * i;
+      const size_t t = (size_t)last * half + min(d >> 1, half - 1);
+      const float other = __shfl_xor_sync(0xffffffffu, o[i], 1), co = x.vcos[t], si = x.vsin[t];
+      o[i] = fmaf(o[i], co, d & 1 ? -other * si : other * si);
     }
   }
   float f = out_scale / l;
@@ -64,21 +92,25 @@ attn_rows_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ kc, con
 
 // dtype 0 bf16, 1 fp32.  Row r attends keys [0, pos[r]] of sequence row_seq[r]; head h of q at column
 // h dkp, of out at column h dvp; gate (may be null): raw gate values, head h at column h, or with gate_elems one for
-// every output column.  window: the latest keys of a row, itself included (0: all).
-BB_API int bb_attn_rows(int dtype, const void* q, int ldq, const void* kc, const void* vc, const int* pos,
+// every output column.  window: the latest keys of a row, itself included (0: all); xt (may be null): what lies behind it,
+// sinks and rotated values.
+BB_API int bb_attn_rows_p(int dtype, const void* q, int ldq, const void* kc, const void* vc, const int* pos,
                         const int* row_seq, const int* tables, int max_blocks, int bs, void* out, int ldo,
                         const void* gate, int ldg, int rows, int hq, int hk, int dk, int dv, int dkp, int dvp,
-                        float scale, float softcap, int gate_elems, float out_scale, int window, void* stream) {
+                          float scale, float softcap, int gate_elems, float out_scale, int window, const BbPooled* xt,
+                          void* stream) {
   using namespace bb;
   if (rows <= 0) return BB_OK;
   const int d = dk > dvp ? dk : dvp;
   if (d > 512 || hq % hk) return BB_ESIZE;
+  const BbPooled x = xt ? *xt : BbPooled{};
+  if (x.pool > 0 && (window <= 0 || x.pool_rows * x.pool < bs)) return BB_EARG;
   const int grid = (int)(((long)rows * hq * 32 + 127) / 128);
   cudaStream_t s = (cudaStream_t)stream;
 #define BB_LAUNCH_AR(T, V)                                                                                          \
   attn_rows_kernel<T, V><<<grid, 128, 0, s>>>((const T*)q, ldq, (const T*)kc, (const T*)vc, pos, row_seq, tables,   \
                                               max_blocks, bs, (T*)out, ldo, (const T*)gate, ldg, rows, hq, hk, dk,  \
-                                              dv, dkp, dvp, scale, softcap, gate_elems, out_scale, window)
+                                              dv, dkp, dvp, scale, softcap, gate_elems, out_scale, window, x)
 #define BB_LAUNCH_AR_T(T)                  \
   do {                                     \
     if (d <= 64) BB_LAUNCH_AR(T, 2);       \
@@ -91,4 +123,12 @@ BB_API int bb_attn_rows(int dtype, const void* q, int ldq, const void* kc, const
 #undef BB_LAUNCH_AR_T
 #undef BB_LAUNCH_AR
   return (int)cudaGetLastError();
+}
+
+BB_API int bb_attn_rows(int dtype, const void* q, int ldq, const void* kc, const void* vc, const int* pos,
+                        const int* row_seq, const int* tables, int max_blocks, int bs, void* out, int ldo,
+                        const void* gate, int ldg, int rows, int hq, int hk, int dk, int dv, int dkp, int dvp,
+                        float scale, float softcap, int gate_elems, float out_scale, int window, void* stream) {
+  return bb_attn_rows_p(dtype, q, ldq, kc, vc, pos, row_seq, tables, max_blocks, bs, out, ldo, gate, ldg, rows, hq, hk, dk, dv,
+                        dkp, dvp, scale, softcap, gate_elems, out_scale, window, nullptr, stream);
 }

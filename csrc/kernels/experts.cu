@@ -31,7 +31,7 @@ __device__ __forceinline__ void warp_best(float& v, int& i) {
 }
 
 // The choices of one token by one warp: lane c < top gets the c-th expert and its weight.  V: experts of a lane
-// (expert j * 32 + lane).
+// (expert j * 32 + lane).  Scores are a softmax, the weights over the chosen ones' sum, or the sigmoid of every logit as it is.
 template <int V>
 __device__ __forceinline__ void choose(const BbHyLayer& L, const float* logits, int& my_e, float& my_w) {
   const int lane = threadIdx.x & 31, E = L.n_experts, size = E / L.groups_all;
@@ -41,15 +41,20 @@ __device__ __forceinline__ void choose(const BbHyLayer& L, const float* logits, 
     s[j] = j * 32 + lane < E ? logits[j * 32 + lane] : -INFINITY;
     mx = fmaxf(mx, s[j]);
   }
-  mx = warp_max(mx);
+  if (L.score_kind == 0) {
+    mx = warp_max(mx);
 #pragma unroll
-  for (int j = 0; j < V; ++j) {
-    s[j] = j * 32 + lane < E ? expf(s[j] - mx) : 0.f;
-    sum += s[j];
+    for (int j = 0; j < V; ++j) {
+      s[j] = j * 32 + lane < E ? expf(s[j] - mx) : 0.f;
+      sum += s[j];
+    }
+    const float inv = 1.f / warp_sum(sum);
+#pragma unroll
+    for (int j = 0; j < V; ++j) s[j] *= inv;
+  } else {
+#pragma unroll
+    for (int j = 0; j < V; ++j) s[j] = sigmoid_f(s[j]);
   }
-  const float inv = 1.f / warp_sum(sum);
-#pragma unroll
-  for (int j = 0; j < V; ++j) s[j] *= inv;
   // groups: take the best expert left in any group not yet kept, keep its group
   bool kept[V];
 #pragma unroll
@@ -94,7 +99,7 @@ __device__ __forceinline__ void choose(const BbHyLayer& L, const float* logits, 
       my_e = min(bi, E - 1);                       // (logits that are not numbers pick no expert)
     }
   }
-  my_w = my_w / (total + L.route_tiny) * L.route_scale;
+  my_w = (L.score_kind == 0 ? my_w / (total + L.route_tiny) : my_w) * L.route_scale;
 }
 
 template <int V>
@@ -237,12 +242,12 @@ __device__ __forceinline__ void expert_offsets(const int* count, int E, int* off
   __syncthreads();
 }
 
-// A warp per token; the last block writes every tile's expert and, cap entries further, how many rows it has.
+// A warp per token (its row times the expert's weight, where that multiplies the input); the last block writes every tile's expert and, cap entries further, how many rows it has.
 template <typename T>
 __global__ void __launch_bounds__(EX_THREADS)
 hy_expert_rows_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ h, int dp, const int* __restrict__ pair_expert,
-                      int* __restrict__ pair_row, const int* __restrict__ count, T* __restrict__ out, int* __restrict__ tiles,
-                      int n_tiles, int cap, int n) {
+                      int* __restrict__ pair_row, const float* __restrict__ pair_w, const int* __restrict__ count,
+                      T* __restrict__ out, int* __restrict__ tiles, int n_tiles, int cap, int n) {
   extern __shared__ int off[];
   const int E = L.n_experts;
   expert_offsets(count, E, off);
@@ -265,8 +270,10 @@ hy_expert_rows_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__
   const int lane = threadIdx.x & 31, t = blockIdx.x * (EX_THREADS / 32) + (threadIdx.x >> 5);
   if (t >= n) return;
   int row = 0;
+  float weight = 1.f;
   if (lane < L.top) {
     const size_t p = (size_t)t * L.top + lane;
+    if (L.weigh_input) weight = pair_w[p];
     row = min(off[pair_expert[p]] + pair_row[p], n_tiles * 128 - 1);
     pair_row[p] = row;
   }
@@ -283,9 +290,17 @@ hy_expert_rows_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__
       if (i0 + u * 32 + lane < dp / VN) x[u] = src[i0 + u * 32 + lane];
     for (int c = 0; c < L.top; ++c) {
       Vec* dst = reinterpret_cast<Vec*>(out + (size_t)__shfl_sync(0xffffffffu, row, c) * dp);
+      const float w = __shfl_sync(0xffffffffu, weight, c);
 #pragma unroll
-      for (int u = 0; u < U; ++u)
-        if (i0 + u * 32 + lane < dp / VN) dst[i0 + u * 32 + lane] = x[u];
+      for (int u = 0; u < U; ++u) {
+        if (i0 + u * 32 + lane >= dp / VN) continue;
+        Vec y = x[u];
+        if (L.weigh_input) {
+#pragma unroll
+          for (int j = 0; j < VN; ++j) y.v[j] = from_f<T>(to_f(y.v[j]) * w);
+        }
+        dst[i0 + u * 32 + lane] = y;
+      }
     }
   }
 }
@@ -372,7 +387,7 @@ BB_API int bb_hy_expert_rows(const BbHyCfg* c, const BbHyLayer* L, const BbHyWor
   const size_t smem = 4 * (size_t)(L->n_experts + 1);
 #define BB_ROWS(T)                                                                                           \
   hy_expert_rows_kernel<T><<<grid, EX_THREADS, smem, s>>>(*L, static_cast<const T*>(w->h), c->dp, w->pair_expert, \
-                                                          w->pair_row, w->ex_count, static_cast<T*>(w->ex_in), \
+                                                          w->pair_row, w->pair_w, w->ex_count, static_cast<T*>(w->ex_in), \
                                                           w->ex_tile, tiles, w->moe_rows / 128, n)
   if (c->dtype) BB_ROWS(float);
   else BB_ROWS(__nv_bfloat16);

@@ -18,6 +18,7 @@
 #include <cstdlib>
 
 #include "../common/host.hpp"
+#include "../common/pooled.hpp"
 #include "../common/ptx.cuh"
 #include "../common/tanh.cuh"
 
@@ -54,6 +55,12 @@ struct FaFwdArgs {
   // kv_pos0[seq]; WIN = 2: in pages
   const int *kv_row0, *kv_pos0;
   int window;
+  // WIN = 3: windows over pages, and behind the window the means of blocks of `pool` tokens (0: none), rows of a matrix
+  // of their own, those of a sequence from pool_row0[seq] / pool on; a number per head in the softmax's denominator;
+  // tables [position][vturn / 2] that turn every pair of output columns back by its row's angle (null: none)
+  int pool, vturn;
+  const int* pool_row0;
+  const float *sink, *vcos, *vsin;
 };
 
 // s <- s (c0 + s^2 (c1 + s^2 (...))) for two scores with packed fp32 arithmetic.
@@ -392,12 +399,13 @@ static constexpr float kFwdTruncLog2 = 0.0041778f;   // log2(1.0029), see the pa
 // the pool's blocks (one TMA copy per block and 64-column half) instead of one copy per tile.
 // EXT: see FaFwdArgs; head sizes below the tile's are zero-filled by the copies (K, V) or multiplied by
 // zeros (Q), P is rounded to nearest when it is packed.
-// WIN (with PAGED and EXT): windows, over rows of one matrix (1) or over pages (2); blocks that lie before every
-// query's window are not visited.
+// WIN (with PAGED and EXT): windows, over rows of one matrix (1) or over pages (2, 3); blocks that lie before every
+// query's window are not visited.  3: tiles of pooled rows (tmKp, tmVp) first, then those of the window.
 template <int HD, bool PAGED, int HDV = HD, bool EXT = false, int WIN = 0>
 __global__ void __launch_bounds__(192, 2)
 fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-               const __grid_constant__ CUtensorMap tmV, const FaFwdArgs args) {
+               const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmKp,
+               const __grid_constant__ CUtensorMap tmVp, const FaFwdArgs args) {
   using Cfg = FaFwdCfg<HD, HDV>;
   constexpr int NSUB = Cfg::NSUB, NSUBV = Cfg::NSUBV;
   extern __shared__ uint8_t smem_raw[];
@@ -436,6 +444,13 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
   const int window = WIN && args.window > 0 ? args.window : 0x3fffffff;
   const int j_first = WIN ? max(q0 + off - window + 1, 0) / 128 : 0;
   if (WIN) n_blocks -= j_first;
+  // tiles of pooled rows: as many as the tile's last query sees a row of
+  int n_pool = 0;
+  if constexpr (WIN == 3) {
+    const int behind = min(q0 + 128, T) + off - window;       // tokens behind that query's window
+    n_pool = args.pool > 0 && behind > 0 ? (behind / args.pool + 127) / 128 : 0;
+    n_blocks += n_pool;
+  }
   const int n_units = 2 * n_blocks;
   const int kv_base = WIN == 1 ? args.kv_row0[seq] + j_first * 128 : 0;
 
@@ -482,10 +497,14 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
 #pragma unroll
           for (int c = 0; c < NSUB; ++c)
             tma_load_3d(sK + c * Cfg::SUB_BYTES, &tmK, k_full, c * 64, kv_base + j * 128, kvh);
+        } else if (WIN == 3 && j < n_pool) {
+#pragma unroll
+          for (int c = 0; c < NSUB; ++c)
+            tma_load_3d(sK + c * Cfg::SUB_BYTES, &tmKp, k_full, c * 64, args.pool_row0[seq] / args.pool + j * 128, kvh);
         } else if (PAGED) {
           // pool layout [blocks][kv heads][block_rows][HD]: block i of this tile lands at row i*block_rows
           const int br = args.block_rows, per_tile = 128 / br;
-          const int jt = j_first + j;
+          const int jt = j_first + j - n_pool;
           const int* tab = args.block_tables + (size_t)seq * args.max_blocks + jt * per_tile;
           for (int i = 0; i < per_tile; ++i) {
             const bool live = (jt * 128 + i * br) < S && (jt * per_tile + i) < args.max_blocks;
@@ -508,9 +527,13 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
 #pragma unroll
           for (int c = 0; c < NSUBV; ++c)
             tma_load_3d(sV + c * Cfg::SUB_BYTES, &tmV, v_full, c * 64, kv_base + j * 128, kvh);
+        } else if (WIN == 3 && j < n_pool) {
+#pragma unroll
+          for (int c = 0; c < NSUBV; ++c)
+            tma_load_3d(sV + c * Cfg::SUB_BYTES, &tmVp, v_full, c * 64, args.pool_row0[seq] / args.pool + j * 128, kvh);
         } else if (PAGED) {
           const int br = args.block_rows, per_tile = 128 / br;
-          const int jt = j_first + j;
+          const int jt = j_first + j - n_pool;
           const int* tab = args.block_tables + (size_t)seq * args.max_blocks + jt * per_tile;
           for (int i = 0; i < per_tile; ++i) {
             const bool live = (jt * 128 + i * br) < S && (jt * per_tile + i) < args.max_blocks;
@@ -621,10 +644,16 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
         }
       }
       const float sc = capped ? 1.f : args.scale_log2;
-      const int kv0 = (WIN ? j_first * 128 : 0) + u * 64;
-      const int lim = kv_limit_row - kv0;  // columns <= lim are visible
-      const int low = WIN ? q_idx + off - window + 1 - kv0 : 0;   // ... and, with a window, columns >= low
-      const bool need_mask = (kv0 + 63 > kv_limit_row) || (WIN && low > 0);
+      int kv0 = (WIN ? (j_first - n_pool) * 128 : 0) + u * 64;
+      int lim = kv_limit_row - kv0;  // columns <= lim are visible
+      int low = WIN ? q_idx + off - window + 1 - kv0 : 0;   // ... and, with a window, columns >= low
+      if constexpr (WIN == 3) {
+        if (u < 2 * n_pool) {        // pooled rows: the blocks that end behind this query's window
+          lim = max(q_idx + off - window + 1, 0) / args.pool - 1 - u * 64;
+          low = 0;
+        }
+      }
+      const bool need_mask = lim < 63 || (WIN && low > 0);
       float mx = -INFINITY;
       if (!need_mask) {
         // four independent running maxima: one chain of 32 dependent FMNMX would leave the two warps
@@ -710,6 +739,9 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
       if (lane == 0) set_error(args.err, ERR_WAIT_SOFTMAX);
     } else {
       tc_fence_after();
+      if constexpr (WIN == 3) {
+        if (args.sink) l += exp2f(args.sink[h] * 1.4426950408889634f - m_ref);
+      }
       float inv = l > 0.f ? 1.f / l : 0.f;
       const __nv_bfloat16* grow = nullptr;     // this row's gates of every element
       if constexpr (EXT) {
@@ -741,6 +773,20 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
                 for (int j = 0; j < 8; ++j) {
                   const float gv = __uint_as_float(j & 1 ? gw[j >> 1] & 0xffff0000u : gw[j >> 1] << 16);
                   r[q * 8 + j] = __float_as_uint(__uint_as_float(r[q * 8 + j]) / (1.f + exp2f(-1.4426950408889634f * gv)));
+                }
+              }
+            }
+            if constexpr (WIN == 3) {
+              if (args.vcos) {       // columns past the true head size are zero, whatever they are turned by
+                const int half = args.vturn >> 1, p0 = (c * 32 + q * 8) >> 1;
+                const size_t t0 = (size_t)(q_idx + off) * half;
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                  const size_t t = t0 + min(p0 + j, half - 1);
+                  const float co = args.vcos[t], si = args.vsin[t];
+                  const float a = __uint_as_float(r[q * 8 + 2 * j]), b = __uint_as_float(r[q * 8 + 2 * j + 1]);
+                  r[q * 8 + 2 * j] = __float_as_uint(fmaf(a, co, b * si));
+                  r[q * 8 + 2 * j + 1] = __float_as_uint(fmaf(b, co, -a * si));
                 }
               }
             }
@@ -802,7 +848,7 @@ static int launch_fa_fwd(const void* q, int ldq, const void* k, int ldk, const v
     return (e && e[0] == '1') ? 1 : 2;
   }();
   if (form == 2 && a.timeline == nullptr)
-    fa_fwd2_kernel<HD, false><<<grid, 192, Cfg::SMEM, stream>>>(tmQ, tmK, tmV, a);
+    fa_fwd2_kernel<HD, false><<<grid, 192, Cfg::SMEM, stream>>>(tmQ, tmK, tmV, tmK, tmV, a);
   else
     fa_fwd_kernel<HD><<<grid, 192, Cfg::SMEM, stream>>>(tmQ, tmK, tmV, a);
   return (int)cudaGetLastError();
@@ -861,25 +907,26 @@ BB_API int bb_flash_fwd_paged(const void* q, int ldq, const void* k_pool, const 
     static PerDeviceOnce once;
     cudaError_t e = ensure_dyn_smem(once, fa_fwd2_kernel<128, true>, FaFwdCfg<128>::SMEM);
     if (e != cudaSuccess) return (int)e;
-    fa_fwd2_kernel<128, true><<<grid, 192, FaFwdCfg<128>::SMEM, s>>>(tmQ, tmK, tmV, a);
+    fa_fwd2_kernel<128, true><<<grid, 192, FaFwdCfg<128>::SMEM, s>>>(tmQ, tmK, tmV, tmK, tmV, a);
   } else {
     static PerDeviceOnce once;
     cudaError_t e = ensure_dyn_smem(once, fa_fwd2_kernel<64, true>, FaFwdCfg<64>::SMEM);
     if (e != cudaSuccess) return (int)e;
-    fa_fwd2_kernel<64, true><<<grid, 192, FaFwdCfg<64>::SMEM, s>>>(tmQ, tmK, tmV, a);
+    fa_fwd2_kernel<64, true><<<grid, 192, FaFwdCfg<64>::SMEM, s>>>(tmQ, tmK, tmV, tmK, tmV, a);
   }
   return (int)cudaGetLastError();
 }
 
 namespace bb {
 template <int HD, int HDV, int WIN = 0>
-static int launch_paged_x(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const FaFwdArgs& a,
-                          int n_tiles, cudaStream_t s) {
-  if (WIN == 0 && a.window > 0) return launch_paged_x<HD, HDV, 2>(tmQ, tmK, tmV, a, n_tiles, s);
+static int launch_paged_x(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const CUtensorMap& tmKp,
+                          const CUtensorMap& tmVp, const FaFwdArgs& a, int n_tiles, cudaStream_t s) {
+  if (WIN == 0 && (a.pool > 0 || a.sink || a.vcos)) return launch_paged_x<HD, HDV, 3>(tmQ, tmK, tmV, tmKp, tmVp, a, n_tiles, s);
+  if (WIN == 0 && a.window > 0) return launch_paged_x<HD, HDV, 2>(tmQ, tmK, tmV, tmKp, tmVp, a, n_tiles, s);
   static PerDeviceOnce once;
   const cudaError_t e = ensure_dyn_smem(once, fa_fwd2_kernel<HD, true, HDV, true, WIN>, FaFwdCfg<HD, HDV>::SMEM);
   if (e != cudaSuccess) return (int)e;
-  fa_fwd2_kernel<HD, true, HDV, true, WIN><<<dim3(n_tiles, a.hq, 1), 192, FaFwdCfg<HD, HDV>::SMEM, s>>>(tmQ, tmK, tmV, a);
+  fa_fwd2_kernel<HD, true, HDV, true, WIN><<<dim3(n_tiles, a.hq, 1), 192, FaFwdCfg<HD, HDV>::SMEM, s>>>(tmQ, tmK, tmV, tmKp, tmVp, a);
   return (int)cudaGetLastError();
 }
 }  // namespace bb
@@ -888,16 +935,19 @@ static int launch_paged_x(const CUtensorMap& tmQ, const CUtensorMap& tmK, const 
 // of 8, up to 128; zero padding counts as columns), scores softcap tanh(scale q.k / softcap) when softcap
 // > 0, an optional output gate (sigmoid of gate[row, head], or with gate_elems of gate[row, output column]), a
 // factor on the output, and a window of the latest keys (0: all).  Pools: bf16 [pool_blocks][hk][block_rows][dq | dv].
-BB_API int bb_flash_fwd_paged_x(const void* q, int ldq, const void* k_pool, const void* v_pool, void* out, int ldo,
+// x (may be null): what lies behind the window, sinks and rotated values.
+BB_API int bb_flash_fwd_paged_p(const void* q, int ldq, const void* k_pool, const void* v_pool, void* out, int ldo,
                                 const int* block_tables, int max_blocks, int block_rows, int pool_blocks,
                                 const int* seq_row0, const int* seq_ctx, const int* tile_seq, const int* tile_qt,
                                 int n_tiles, int total_rows, int hq, int hk, int dq, int dv, float scale, float softcap,
-                                const void* gate, int ldg, int gate_elems, float out_scale, int window, void* stream) {
+                                const void* gate, int ldg, int gate_elems, float out_scale, int window, const BbPooled* x,
+                                void* stream) {
   using namespace bb;
   if (n_tiles <= 0) return BB_OK;
   if (hq % hk || total_rows <= 0 || max_blocks <= 0 || pool_blocks <= 0) return BB_EARG;
   if (block_rows != 16 && block_rows != 32 && block_rows != 64 && block_rows != 128) return BB_ESIZE;
   if (dq % 8 || dv % 8 || dq > 128 || dv > 128 || ldq % 8 || ldo % 8) return BB_ESIZE;
+  if (x && (x->pool < 0 || (x->pool > 0 && (window <= 0 || x->ld_pk % 8 || !x->pool_row0)))) return BB_EARG;
   FaFwdArgs a{};
   a.O = static_cast<__nv_bfloat16*>(out);
   a.ldo = ldo;
@@ -906,6 +956,14 @@ BB_API int bb_flash_fwd_paged_x(const void* q, int ldq, const void* k_pool, cons
   a.scale_log2 = scale * 1.4426950408889634f;
   a.causal = 1;
   a.err = device_error_word();
+  if (x) {
+    a.pool = x->pool;
+    a.pool_row0 = x->pool_row0;
+    a.sink = x->sink;
+    a.vcos = x->vcos;
+    a.vsin = x->vsin;
+    a.vturn = x->vturn;
+  }
   a.block_tables = block_tables;
   a.seq_row0 = seq_row0;
   a.seq_ctx = seq_ctx;
@@ -937,11 +995,30 @@ BB_API int bb_flash_fwd_paged_x(const void* q, int ldq, const void* k_pool, cons
   if (rc) return rc;
   rc = make_tmap_2d(&tmV, bf, 2, v_pool, (uint64_t)dv, pool_rows, (uint64_t)dv * 2, 64, block_rows);
   if (rc) return rc;
+  CUtensorMap tmKp = tmK, tmVp = tmV;
+  if (a.pool > 0) {
+    const uint64_t ld = (uint64_t)x->ld_pk * 2;
+    rc = make_tmap_3d(&tmKp, bf, 2, x->pk, dq, x->pk_rows, hk, ld, (uint64_t)dq * 2, 64, 128);
+    if (rc) return rc;
+    rc = make_tmap_3d(&tmVp, bf, 2, static_cast<const __nv_bfloat16*>(x->pk) + hk * dq, dv, x->pk_rows, hk, ld, (uint64_t)dv * 2,
+                      64, 128);
+    if (rc) return rc;
+  }
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dq <= 64) return dv <= 64 ? launch_paged_x<64, 64>(tmQ, tmK, tmV, a, n_tiles, s)
-                                : launch_paged_x<64, 128>(tmQ, tmK, tmV, a, n_tiles, s);
-  return dv <= 64 ? launch_paged_x<128, 64>(tmQ, tmK, tmV, a, n_tiles, s)
-                  : launch_paged_x<128, 128>(tmQ, tmK, tmV, a, n_tiles, s);
+  if (dq <= 64) return dv <= 64 ? launch_paged_x<64, 64>(tmQ, tmK, tmV, tmKp, tmVp, a, n_tiles, s)
+                                : launch_paged_x<64, 128>(tmQ, tmK, tmV, tmKp, tmVp, a, n_tiles, s);
+  return dv <= 64 ? launch_paged_x<128, 64>(tmQ, tmK, tmV, tmKp, tmVp, a, n_tiles, s)
+                  : launch_paged_x<128, 128>(tmQ, tmK, tmV, tmKp, tmVp, a, n_tiles, s);
+}
+
+BB_API int bb_flash_fwd_paged_x(const void* q, int ldq, const void* k_pool, const void* v_pool, void* out, int ldo,
+                                const int* block_tables, int max_blocks, int block_rows, int pool_blocks,
+                                const int* seq_row0, const int* seq_ctx, const int* tile_seq, const int* tile_qt,
+                                int n_tiles, int total_rows, int hq, int hk, int dq, int dv, float scale, float softcap,
+                                const void* gate, int ldg, int gate_elems, float out_scale, int window, void* stream) {
+  return bb_flash_fwd_paged_p(q, ldq, k_pool, v_pool, out, ldo, block_tables, max_blocks, block_rows, pool_blocks, seq_row0,
+                              seq_ctx, tile_seq, tile_qt, n_tiles, total_rows, hq, hk, dq, dv, scale, softcap, gate, ldg,
+                              gate_elems, out_scale, window, nullptr, stream);
 }
 
 namespace bb {
@@ -951,7 +1028,7 @@ static int launch_window(const CUtensorMap& tmQ, const CUtensorMap& tmK, const C
   static PerDeviceOnce once;
   const cudaError_t e = ensure_dyn_smem(once, fa_fwd2_kernel<HD, true, HDV, true, 1>, FaFwdCfg<HD, HDV>::SMEM);
   if (e != cudaSuccess) return (int)e;
-  fa_fwd2_kernel<HD, true, HDV, true, 1><<<dim3(n_tiles, a.hq, 1), 192, FaFwdCfg<HD, HDV>::SMEM, s>>>(tmQ, tmK, tmV, a);
+  fa_fwd2_kernel<HD, true, HDV, true, 1><<<dim3(n_tiles, a.hq, 1), 192, FaFwdCfg<HD, HDV>::SMEM, s>>>(tmQ, tmK, tmV, tmK, tmV, a);
   return (int)cudaGetLastError();
 }
 }  // namespace bb

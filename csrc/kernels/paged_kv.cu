@@ -14,6 +14,7 @@
 // Reference contracts: crates/kernels/wgsl/{paged_kv_append_batched,paged_decode_scores_batched,
 // decode_softmax_batched,paged_decode_apply_batched}.wgsl, crates/qwen3/src/serve.rs:1262-1288.
 #include "../common/host.hpp"
+#include "../common/pooled.hpp"
 #include "../common/ptx.cuh"
 #include "../common/tanh.cuh"
 #include "../common/vec.cuh"
@@ -178,11 +179,14 @@ __device__ __forceinline__ void cp_async_wait() {
 
 //
 // EXT: key and value heads of their own sizes (dk / dv columns in memory, multiples of 8, at most HD /
-// HDV), soft-capped scores (x.cap_log2 tanh(x.cap_in q.k) in the log2 domain), and a window of the latest keys.
+// HDV), soft-capped scores (x.cap_log2 tanh(x.cap_in q.k) in the log2 domain), and a window of the latest keys with,
+// behind it, the means of blocks of x.pool tokens: keys of their own, counted before those of the window.
 struct PdExt {
   int dk, dv;
   float cap_in, cap_log2;   // cap_log2 = 0: no cap
   int window;               // 0: every key
+  int pool, pool_rows;      // pool = 0: none (see BbPooled)
+  const void *pkc, *pvc;
 };
 template <int HD, int G, bool I8, int HDV = HD, bool EXT = false>
 __global__ void __launch_bounds__(128, 3)
@@ -222,7 +226,9 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
   const int grp = lane >> 3, sub = lane & 7;
   const int rowk = EXT ? x.dk * ES : ROWB, rowv = EXT ? x.dv * ES : ROWBV;   // bytes of a stored row
   const int S = seqlens[b];
-  const int k_low = EXT && x.window > 0 ? max(S - x.window, 0) : 0;    // first key in the window
+  const int k_first = EXT && x.window > 0 ? max(S - x.window, 0) : 0;  // first token in the window
+  const int n_mean = EXT && x.pool > 0 ? k_first / x.pool : 0;         // blocks behind it: keys k_first - n_mean ..
+  const int k_low = k_first - n_mean;
   const int per_split = ((S - k_low + splits - 1) / splits + 31) / 32 * 32;
   const int k_begin = k_low + sp * per_split;
   const int k_end = min(S, k_begin + per_split);
@@ -238,10 +244,18 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, int ldq,
       const int kl = c / CPM, part = c % CPM;
       const int key = k0 + kl;
       if (key < k_end) {
-        const int blk = bt[key / bs], off = key % bs;
-        const size_t r = ((size_t)blk * hk + kvh) * bs + off;
-        if (!EXT || part * 16 < rowk) cp_async16(s_k + st * STAGE + kl * ROWB + part * 16, kc + r * rowk + part * 16);
-        if (!EXT || part * 16 < rowv) cp_async16(s_v + st * STAGEV + kl * ROWBV + part * 16, vc + r * rowv + part * 16);
+        const unsigned char *kp = kc, *vp = vc;
+        size_t r;
+        if (EXT && key < k_first) {
+          const int e = (key - k_low + 1) * x.pool - 1;          // last token of the block
+          r = ((size_t)bt[e / bs] * hk + kvh) * x.pool_rows + e % bs / x.pool;
+          kp = static_cast<const unsigned char*>(x.pkc);
+          vp = static_cast<const unsigned char*>(x.pvc);
+        } else {
+          r = ((size_t)bt[key / bs] * hk + kvh) * bs + key % bs;
+        }
+        if (!EXT || part * 16 < rowk) cp_async16(s_k + st * STAGE + kl * ROWB + part * 16, kp + r * rowk + part * 16);
+        if (!EXT || part * 16 < rowv) cp_async16(s_v + st * STAGEV + kl * ROWBV + part * 16, vp + r * rowv + part * 16);
       }
     }
     if constexpr (I8) {
@@ -506,9 +520,13 @@ __global__ void paged_decode_merge_kernel(const float* __restrict__ part_o,
                                           const float* __restrict__ part_ml,
                                           __nv_bfloat16* __restrict__ out, int ldo, int hq, int hd,
                                           int splits, int hd_out, const __nv_bfloat16* __restrict__ gate,
-                                          int ldg, int gate_elems, float out_scale) {
+                                          int ldg, int gate_elems, float out_scale,
+                                          const float* __restrict__ sink, const float* __restrict__ vcos,
+                                          const float* __restrict__ vsin, int vturn, const int* __restrict__ seqlens) {
   // hd: columns of a partial row; hd_out: columns of a head in the output; gate (may be null): raw
-  // output gate (one per head, or with gate_elems one per output column), the output is multiplied by its sigmoid
+  // output gate (one per head, or with gate_elems one per output column), the output is multiplied by its sigmoid;
+  // sink (may be null): a number per head in the denominator; vcos, vsin (may be null): tables [position][vturn / 2]
+  // that turn every pair of columns back by the angles of the sequence's last position
   const int b = blockIdx.x, h = blockIdx.y;
   const size_t base = ((size_t)b * hq + h) * splits;
   float mm = -INFINITY;
@@ -518,14 +536,24 @@ __global__ void paged_decode_merge_kernel(const float* __restrict__ part_o,
     const float ms = part_ml[(base + s) * 2];
     ll += (ms == -INFINITY) ? 0.f : part_ml[(base + s) * 2 + 1] * exp2f(ms - mm);
   }
+  if (sink) ll += exp2f(sink[h] * 1.4426950408889634f - mm);
   float inv = ll > 0.f ? out_scale / ll : 0.f;
   if (gate && !gate_elems) inv *= 1.f / (1.f + exp2f(-1.4426950408889634f * __bfloat162float(gate[(size_t)b * ldg + h])));
-  for (int c = threadIdx.x; c < hd_out; c += blockDim.x) {
+  for (int c0 = 0; c0 < hd_out; c0 += blockDim.x) {
+    const int c = c0 + threadIdx.x;
+    const bool live = c < hd_out;
     float acc = 0.f;
-    for (int s = 0; s < splits; ++s) {
+    for (int s = 0; live && s < splits; ++s) {
       const float ms = part_ml[(base + s) * 2];
       if (ms != -INFINITY) acc += part_o[(base + s) * hd + c] * exp2f(ms - mm);
     }
+    if (vcos) {
+      const int half = vturn >> 1;
+      const size_t t = (size_t)(seqlens[b] - 1) * half + min(c >> 1, half - 1);
+      const float other = __shfl_xor_sync(0xffffffffu, acc, 1), co = vcos[t], si = vsin[t];
+      acc = fmaf(acc, co, c & 1 ? -other * si : other * si);
+    }
+    if (!live) continue;
     if (gate_elems)
       acc *= 1.f / (1.f + exp2f(-1.4426950408889634f * __bfloat162float(gate[(size_t)b * ldg + h * hd_out + c])));
     out[(size_t)b * ldo + h * hd_out + c] = __float2bfloat16(acc * inv);
@@ -610,7 +638,8 @@ static int launch_paged_decode(bool i8, const void* q, int ldq, const void* kc, 
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
   paged_decode_merge_kernel<<<dim3(B, hq), 128, 0, s>>>(part_o, part_ml, (__nv_bfloat16*)out, ldo,
-                                                        hq, hd, splits, hd, nullptr, 0, 0, 1.f);
+                                                        hq, hd, splits, hd, nullptr, 0, 0, 1.f, nullptr, nullptr,
+                                                        nullptr, 0, nullptr);
   return (int)cudaGetLastError();
 }
 
@@ -626,19 +655,23 @@ BB_API int bb_paged_decode(const void* q, int ldq, const void* kc, const void* v
 
 // The same for key / value heads of their own sizes (dk / dv stored columns, multiples of 8, up to 128),
 // any number of query heads per kv head, scores softcap tanh(scale q.k / softcap) when softcap > 0, a window of the
-// latest keys (0: all), a factor on the output and an optional output gate (per head, or with gate_elems per element).  part_o: fp32 [B*hq*splits*(dv <= 64 ? 64 : 128)].
-BB_API int bb_paged_decode_x(const void* q, int ldq, const void* kc, const void* vc, const int* block_tables,
+// latest keys (0: all), a factor on the output and an optional output gate (per head, or with gate_elems per element).
+// xt (may be null): what lies behind the window, sinks and rotated values.
+// part_o: fp32 [B*hq*splits*(dv <= 64 ? 64 : 128)].
+BB_API int bb_paged_decode_p(const void* q, int ldq, const void* kc, const void* vc, const int* block_tables,
                              int max_blocks, const int* seqlens, void* out, int ldo, float* part_o, float* part_ml,
                              int B, int hq, int hk, int dk, int dv, int bs, int splits, float scale, float softcap,
-                             const void* gate, int ldg, int gate_elems, float out_scale, int window, void* stream) {
+                             const void* gate, int ldg, int gate_elems, float out_scale, int window, const BbPooled* xt,
+                             void* stream) {
   if (B <= 0) return BB_OK;
-  if (hq % hk || splits < 1) return BB_EARG;
+  const BbPooled e = xt ? *xt : BbPooled{};
+  if (hq % hk || splits < 1 || (e.pool > 0 && (window <= 0 || e.pool_rows * e.pool < bs))) return BB_EARG;
   if (dk % 8 || dv % 8 || dk > 128 || dv > 128 || ldq % 8) return BB_ESIZE;
   const int ratio = hq / hk;
   const int G = ratio % 4 == 0 ? 4 : (ratio % 3 == 0 ? 3 : (ratio % 2 == 0 ? 2 : 1));
   const int gsplit = ratio / G;
   dim3 grid(B, hk * gsplit, splits);
-  PdExt x{dk, dv, 0.f, 0.f, window};
+  PdExt x{dk, dv, 0.f, 0.f, window, e.pool, e.pool_rows, e.pkc, e.pvc};
   float sl2 = scale * 1.4426950408889634f;
   if (softcap > 0.f) {
     sl2 = scale / softcap;     // the query is pre-scaled so that q.k is the argument of tanh
@@ -664,12 +697,20 @@ BB_API int bb_paged_decode_x(const void* q, int ldq, const void* kc, const void*
   }
 #undef BB_LAUNCH_PXG
 #undef BB_LAUNCH_PX
-  cudaError_t e = cudaGetLastError();
-  if (e != cudaSuccess) return (int)e;
+  cudaError_t err = cudaGetLastError();
+  if (err != cudaSuccess) return (int)err;
   paged_decode_merge_kernel<<<dim3(B, hq), 128, 0, s>>>(part_o, part_ml, (__nv_bfloat16*)out, ldo, hq,
                                                         dv <= 64 ? 64 : 128, splits, dv, (const __nv_bfloat16*)gate, ldg,
-                                                        gate ? gate_elems : 0, out_scale);
+                                                        gate ? gate_elems : 0, out_scale, e.sink, e.vcos, e.vsin, e.vturn, seqlens);
   return (int)cudaGetLastError();
+}
+
+BB_API int bb_paged_decode_x(const void* q, int ldq, const void* kc, const void* vc, const int* block_tables,
+                             int max_blocks, const int* seqlens, void* out, int ldo, float* part_o, float* part_ml,
+                             int B, int hq, int hk, int dk, int dv, int bs, int splits, float scale, float softcap,
+                             const void* gate, int ldg, int gate_elems, float out_scale, int window, void* stream) {
+  return bb_paged_decode_p(q, ldq, kc, vc, block_tables, max_blocks, seqlens, out, ldo, part_o, part_ml, B, hq, hk, dk, dv, bs,
+                           splits, scale, softcap, gate, ldg, gate_elems, out_scale, window, nullptr, stream);
 }
 
 // int8 pools kc/vc with per-row scales ks/vs: fp32 [num_blocks, hk, bs].

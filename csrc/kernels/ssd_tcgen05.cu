@@ -18,6 +18,9 @@
 // The normaliser n follows S (in shared memory, on the CUDA cores): n.q_i is exp(m - M_i) (n.q_i) plus the sum of
 // row i of W.  A row leaves divided by max(|n.q|, exp(-m_i)), over its root mean square, times gain and gate.
 //
+// Without step sizes (dt null) they are 1 and the outputs take the factor q_scale: retention, whose decays are constants
+// of the heads.
+//
 // With few (sequence, head) pairs a portion is cut into segments of whole chunks that run side by side:
 // a first launch (LOCAL) computes what each segment adds to the state on its own, and its decay; the
 // segments of the main launch then start from the state carried in, decayed and summed over the segments
@@ -121,7 +124,9 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
   const int r0 = b.seq_row0[seq], len = b.seq_row0[seq + 1] - r0, slot = b.seq_slot[seq];
   const int n_chunks = (len + 127) / 128;
   const int nsub = (L.n + 63) / 64, nk = (L.n + 15) / 16;
-  const float a2 = GATED ? 0.f : L.a[h] * kLog2e, D = GATED ? 0.f : L.d_skip[h];
+  const float a2 = GATED ? 0.f : L.a[h] * kLog2e, D = GATED || !L.d_skip ? 0.f : L.d_skip[h];
+  const float y_scale = GATED || dt ? 1.f : L.q_scale;
+  const int pw = GATED || !L.pp ? L.p : L.pp;                   // columns of a head in the output
   const size_t np = (size_t)L.n * L.p, mem = GATED ? L.mem : np;   // floats of a state
   float* state = L.ssm_state + ((size_t)slot * L.heads + h) * mem;
   GatedSmem<W> gs(reinterpret_cast<float*>(PP == 64 && nsub == 1 ? sC + SSD_SUB : smem + Cfg::SMEM));
@@ -235,7 +240,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
       d_next = i < len ? dt[(size_t)(r0 + i) * lddt + L.off32_i + h] * kLog2e : -INFINITY;
       cum_next = i < len ? dt[(size_t)(r0 + i) * lddt + L.off32_f + h] * kLog2e : 0.f;
     } else {
-      d_next = i < len ? dt[(size_t)(r0 + i) * lddt + h] : 0.f;
+      d_next = i < len ? (dt ? dt[(size_t)(r0 + i) * lddt + h] : 1.f) : 0.f;
     }
   };
   auto scan_dt = [&]() {
@@ -569,7 +574,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
         unpack8(*reinterpret_cast<const bf16x8*>(sX + (col >> 6) * SSD_SUB + row * 128 +
                                                  ((((col & 63) >> 3) ^ (row & 7)) << 4)), f);
 #pragma unroll
-        for (int j = 0; j < 8; ++j) f[j] = fmaf(D, f[j], __uint_as_float(r[q * 8 + j]));
+        for (int j = 0; j < 8; ++j) f[j] = fmaf(D, f[j], __uint_as_float(r[q * 8 + j]) * y_scale);
         store8(reinterpret_cast<__nv_bfloat16*>(sC + (col >> 6) * SSD_SUB + row * 128 +
                                                 ((((col & 63) >> 3) ^ (row & 7)) << 4)), f);
       }
@@ -604,8 +609,8 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
     } else if (ok) {
       for (int i = threadIdx.x; i < valid * VR; i += SSD_THREADS) {
         const int rr = i / VR, q = i % VR;
-        if (q * 8 < L.p)
-          *reinterpret_cast<uint4*>(y + (size_t)(c0 + rr) * ldy + h * L.p + q * 8) =
+        if (q * 8 < pw)
+          *reinterpret_cast<uint4*>(y + (size_t)(c0 + rr) * ldy + h * pw + q * 8) =
               *reinterpret_cast<const uint4*>(sC + (q >> 3) * SSD_SUB + rr * 128 + (((q & 7) ^ (rr & 7)) << 4));
       }
     }
@@ -736,4 +741,23 @@ BB_API int bb_mlstm_chunk(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* 
   __nv_bfloat16* cat = static_cast<__nv_bfloat16*>(w->cat);
   return L->p <= 64 ? launch_ssd<64, true>(tmBC, tmX, *L, *w, *b, w->f32, w->ld_f32, cat, w->ld_cat, c->eps, s)
                     : launch_ssd<128, true>(tmBC, tmX, *L, *w, *b, w->f32, w->ld_f32, cat, w->ld_cat, c->eps, s);
+}
+
+// The same for retention: queries and keys (rotated) and values in w->proj -> outputs in w->y.  BB_ESIZE for heads above 128.
+BB_API int bb_retention_chunk(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream) {
+  using namespace bb;
+  if (b->ns_pre <= 0) return BB_OK;
+  if (c->dtype || L->np > 128 || L->pp > 128) return BB_ESIZE;
+  const __nv_bfloat16* proj = static_cast<const __nv_bfloat16*>(w->proj);
+  const uint64_t ld = (uint64_t)w->ld_proj * 2;
+  CUtensorMap tmBC, tmX;
+  const CUtensorMapDataType bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+  int rc = make_tmap_3d(&tmBC, bf, 2, proj + L->off_kk, L->np, b->n_pre, 2 * L->heads, ld, (uint64_t)L->np * 2, 64, 128);
+  if (rc) return rc;
+  rc = make_tmap_3d(&tmX, bf, 2, proj + L->off_vv, L->pp, b->n_pre, L->heads, ld, (uint64_t)L->pp * 2, 64, 128);
+  if (rc) return rc;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  __nv_bfloat16* y = static_cast<__nv_bfloat16*>(w->y);
+  return L->p <= 64 ? launch_ssd<64, false>(tmBC, tmX, *L, *w, *b, nullptr, 0, y, w->ld_y, 0.f, s)
+                    : launch_ssd<128, false>(tmBC, tmX, *L, *w, *b, nullptr, 0, y, w->ld_y, 0.f, s);
 }

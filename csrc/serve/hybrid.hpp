@@ -16,7 +16,7 @@ struct BbHyLin {
 
 struct BbHyLayer {
   int kind;            // 0 attention, 1 mamba2, 2 latent attention, 3 generalised delta rule, 4 gated linear recurrence,
-                       // 5 matrix memory (mLSTM)
+                       // 5 matrix memory (mLSTM), 6 gated linear attention, 7 retention
   const float* norm;   // [dp] gain of the layer's norm (one already added where it is stored around 0)
   BbHyLin in;          // every projection that reads the normed input, stacked along the rows
   BbHyLin out;         // mixer output projection | feed-forward down projection, side by side
@@ -92,6 +92,27 @@ struct BbHyLayer {
   int n_experts, top, groups_all, groups_keep, eff, effp;
   float route_scale, route_tiny, e_limit, e_alpha, e_shift;
   const void *w_egu, *w_edown;
+  // scores of a router: 0 softmax, over the sum of the chosen ones; 1 the sigmoid of each.  weigh_input: a row's weight
+  // multiplies what its expert reads (the outputs are then summed as they are)
+  int score_kind, weigh_input;
+  // residual streams: biases of the norms [dp], token shift [dp] (null: none) and the last input before it
+  // [slots][dp], connections of the mixer and the feed-forward: [in s | out s | mix s s, from and to]
+  const float *norm_b, *norm2_b, *shift;
+  void* shift_state;
+  const float *hc[2];
+  BbHyLin down;                            // of a feed-forward that follows its mixer (its `up` above)
+  const float* out_gain;                   // [dp] mixers side by side, each result normed (null: as it is)
+  // attention: norms per head (q_norm [dkp], k_norm [dkp] for every head), neighbouring pairs rotated; the means of
+  // blocks of `pool` tokens in pages of pool_rows rows, each in the page of its last token; a number per head [hq] in
+  // the softmax's denominator; tables [max_pos][dv / 2] that turn values, and outputs back (null: none)
+  int head_norm, pool, pool_rows;
+  void *pkc, *pvc;                         // [blocks][hk][pool_rows][dkp | dvp]
+  const float *sink, *vcos_t, *vsin_t;
+  // linear attention (heads of n key channels, padded np, and p value channels, padded pp; columns and state as a
+  // matrix memory's, the state without normaliser): decays sigmoid(z)^decay_root with z = w2 (columns off_w1) + w0, or
+  // constants: keep_less [heads] = decay - 1, a = its logarithm; gate silu(columns off_gg), gnorm [heads pp] or null
+  float decay_root;
+  const float* keep_less;
 };
 
 struct BbHyCfg {
@@ -105,6 +126,9 @@ struct BbHyCfg {
   int max_pos;
   float embed_scale;
   int depth_avg;                           // layers pass on weighted sums of all results (see BbHyWork::x)
+  int streams;                             // copies of the residual stream (0: one, without connections)
+  const float* final_norm_b;               // [dp] (null: none)
+  float logit_cap;                         // logits become cap tanh(logits / cap) (0: as they are)
 };
 
 // One packed batch: rows of prompt portions first (n_pre rows of ns_pre sequences), then one row for
@@ -121,11 +145,13 @@ struct BbHyBatch {
   const int *exp_src, *kv_row0, *kv_pos0;
   int n_exp;
   int max_blocks, n, n_pre, ns, ns_pre, n_tiles, n_want, max_len;   // max_len: longest portion
+  const int* ctx_row0;                     // [ns_pre] sum of the contexts of the portions before
+  int max_ctx;                             // longest context of a portion
 };
 
 struct BbHyWork {
   float* x;          // [rows, dp] residual stream; with depth averages [n_layers + 1][rows, dp]: the
-                     // embedding, then every layer's result
+                     // embedding, then every layer's result; with several streams [rows][streams][dp]
   void* h;           // [rows, dp]
   void* proj;        // [rows, ld_proj]
   void* cat;         // [rows, ld_cat]
@@ -154,6 +180,10 @@ struct BbHyWork {
   float* pair_w;
   int *ex_count, *ex_tile;                 // [experts], [2][moe_rows / 128]
   int ld_f32, ld_gu, ld_act, moe_rows;
+  // residual streams: results of a sublayer [rows, dp] (two of mixers side by side); pooled keys and values that prompt
+  // portions see, [pk_rows, ld_pk], of sequence s from ctx_row0[s] / pool on
+  void *ya, *yb, *pk;
+  int ld_pk, pk_rows;
 };
 
 // Rows and pitch of a latent attention layer's queries: through their own latent, or straight from the input.

@@ -11,12 +11,15 @@
 // Designs with depth averages keep every layer's result: a layer starts from the weighted sum of all of them
 // (written where its own result will be, so the output GEMM adds in place), and its feed-forward has a norm
 // and a GEMM of its own.
+// Designs with several residual streams run mixer and feed-forward one after the other; between any two of these one
+// kernel (hy_streams) spreads the result over the streams and makes the next input.
 // bf16: the tensor-core GEMM, paged flash prefill, split-KV decode attention and chunked state-space
 // kernels; fp32: the CUDA-core forms of the same steps.
 #include <cstdint>
 #include <mutex>
 
 #include "../common/host.hpp"
+#include "../common/pooled.hpp"
 #include "hybrid.hpp"
 
 using namespace bb;
@@ -55,19 +58,31 @@ int bb_flash_fwd_window(const void* q, int ldq, const void* k, const void* v, in
                         const int* seq_row0, const int* kv_row0, const int* kv_pos0, const int* seq_ctx, const int* tile_seq,
                         const int* tile_qt, int n_tiles, int total_rows, int hq, int hk, int dq, int dv, float scale,
                         int window, const void* gate, int ldg, void* stream);
-int bb_attn_rows(int dtype, const void* q, int ldq, const void* kc, const void* vc, const int* pos, const int* row_seq,
-                 const int* tables, int max_blocks, int bs, void* out, int ldo, const void* gate, int ldg, int rows, int hq,
-                 int hk, int dk, int dv, int dkp, int dvp, float scale, float softcap, int gate_elems, float out_scale,
-                 int window, void* stream);
-int bb_flash_fwd_paged_x(const void* q, int ldq, const void* k_pool, const void* v_pool, void* out, int ldo,
+int bb_attn_rows_p(int dtype, const void* q, int ldq, const void* kc, const void* vc, const int* pos, const int* row_seq,
+                   const int* tables, int max_blocks, int bs, void* out, int ldo, const void* gate, int ldg, int rows, int hq,
+                   int hk, int dk, int dv, int dkp, int dvp, float scale, float softcap, int gate_elems, float out_scale,
+                   int window, const BbPooled* x, void* stream);
+int bb_flash_fwd_paged_p(const void* q, int ldq, const void* k_pool, const void* v_pool, void* out, int ldo,
                          const int* block_tables, int max_blocks, int block_rows, int pool_blocks, const int* seq_row0,
                          const int* seq_ctx, const int* tile_seq, const int* tile_qt, int n_tiles, int total_rows, int hq,
                          int hk, int dq, int dv, float scale, float softcap, const void* gate, int ldg, int gate_elems,
-                         float out_scale, int window, void* stream);
-int bb_paged_decode_x(const void* q, int ldq, const void* kc, const void* vc, const int* block_tables, int max_blocks,
+                         float out_scale, int window, const BbPooled* x, void* stream);
+int bb_paged_decode_p(const void* q, int ldq, const void* kc, const void* vc, const int* block_tables, int max_blocks,
                       const int* seqlens, void* out, int ldo, float* part_o, float* part_ml, int B, int hq, int hk, int dk,
                       int dv, int bs, int splits, float scale, float softcap, const void* gate, int ldg, int gate_elems,
-                      float out_scale, int window, void* stream);
+                      float out_scale, int window, const BbPooled* x, void* stream);
+int bb_hy_heads(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_turn(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_pool(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int gather, void* stream);
+int bb_hy_streams(const BbHyCfg* c, const BbHyLayer* before, int fq, const BbHyLayer* next, int tq, const BbHyWork* w,
+                  const BbHyBatch* b, int all, float* trace, void* stream);
+int bb_hy_shift(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_gelu(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream);
+int bb_hy_cap(const BbHyCfg* c, const BbHyWork* w, int n, void* stream);
+int bb_hy_linear_scan(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_linear_decode(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_linear_post(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int rows, void* stream);
+int bb_retention_chunk(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
 int bb_hy_start(const BbHyCfg* c, int li, const BbHyWork* w, const BbHyBatch* b, int all, float* trace, void* stream);
 int bb_hy_kv_post(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
 int bb_hy_glu(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream);
@@ -130,22 +145,25 @@ const void* at(const BbHyCfg& c, const void* p, size_t elems) {
 void* at(const BbHyCfg& c, void* p, size_t elems) { return static_cast<char*>(p) + elems * (c.dtype ? 4 : 2); }
 
 int attention(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
-  if (L.q_norm) BB_TRY(bb_hy_attn_post(&c, &L, &w, &b, s));
+  if (L.head_norm) BB_TRY(bb_hy_heads(&c, &L, &w, &b, s));
+  else if (L.q_norm) BB_TRY(bb_hy_attn_post(&c, &L, &w, &b, s));
   else BB_TRY(bb_hy_kv_post(&c, &L, &w, &b, s));
   const void* q = at(c, w.proj, L.off_q);
   const void* gate = L.gate_kind ? at(c, w.proj, L.off_g) : nullptr;
   const int elems = L.gate_kind == 2;
   const int n_dec = b.n - b.n_pre;
+  const BbPooled x{L.pool, L.pool_rows, L.pkc, L.pvc, w.pk, w.ld_pk, w.pk_rows, b.ctx_row0, L.sink, L.vcos_t, L.vsin_t, L.dv};
   if (b.n_pre > 0) {
+    BB_TRY(bb_hy_pool(&c, &L, &w, &b, !c.dtype && L.dkp <= 128 && L.dvp <= 128, s));
     int rc = BB_ESIZE;
     if (!c.dtype)
-      rc = bb_flash_fwd_paged_x(q, w.ld_proj, L.kc, L.vc, w.cat, w.ld_cat, b.tables, b.max_blocks, c.block_size,
+      rc = bb_flash_fwd_paged_p(q, w.ld_proj, L.kc, L.vc, w.cat, w.ld_cat, b.tables, b.max_blocks, c.block_size,
                                 w.pool_blocks, b.seq_row0, b.seq_ctx, b.tile_seq, b.tile_qt, b.n_tiles, b.n_pre, L.hq, L.hk,
-                                L.dkp, L.dvp, L.scale, L.softcap, gate, w.ld_proj, elems, L.out_scale, L.window, s);
+                                L.dkp, L.dvp, L.scale, L.softcap, gate, w.ld_proj, elems, L.out_scale, L.window, &x, s);
     if (rc == BB_ESIZE)
-      rc = bb_attn_rows(c.dtype, q, w.ld_proj, L.kc, L.vc, b.pos, b.row_seq, b.tables, b.max_blocks, c.block_size, w.cat,
+      rc = bb_attn_rows_p(c.dtype, q, w.ld_proj, L.kc, L.vc, b.pos, b.row_seq, b.tables, b.max_blocks, c.block_size, w.cat,
                         w.ld_cat, gate, w.ld_proj, b.n_pre, L.hq, L.hk, L.dk, L.dv, L.dkp, L.dvp, L.scale, L.softcap, elems,
-                        L.out_scale, L.window, s);
+                          L.out_scale, L.window, &x, s);
     if (rc) return rc;
   }
   if (n_dec > 0) {
@@ -157,16 +175,17 @@ int attention(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbH
       // K/V splits: enough blocks to fill the machine, at most what the partial buffers were sized for
       const int base = n_dec * L.hk;
       int splits = (4 * sm_count() + base - 1) / base;
-      if (L.window > 0 && splits > (L.window + 31) / 32) splits = (L.window + 31) / 32;
+      const int keys = L.window + (L.pool > 0 ? b.max_blocks * c.block_size / L.pool : 0);
+      if (L.window > 0 && splits > (keys + 31) / 32) splits = (keys + 31) / 32;
       splits = splits < 1 ? 1 : (splits > w.splits ? w.splits : splits);
-      rc = bb_paged_decode_x(qd, w.ld_proj, L.kc, L.vc, b.tables + (size_t)b.ns_pre * b.max_blocks, b.max_blocks,
+      rc = bb_paged_decode_p(qd, w.ld_proj, L.kc, L.vc, b.tables + (size_t)b.ns_pre * b.max_blocks, b.max_blocks,
                              b.seq_ctx + b.ns_pre, od, w.ld_cat, w.part_o, w.part_ml, n_dec, L.hq, L.hk, L.dkp, L.dvp,
-                             c.block_size, splits, L.scale, L.softcap, gd, w.ld_proj, elems, L.out_scale, L.window, s);
+                             c.block_size, splits, L.scale, L.softcap, gd, w.ld_proj, elems, L.out_scale, L.window, &x, s);
     }
     if (rc == BB_ESIZE)
-      rc = bb_attn_rows(c.dtype, qd, w.ld_proj, L.kc, L.vc, b.pos + b.n_pre, b.row_seq + b.n_pre, b.tables, b.max_blocks,
+      rc = bb_attn_rows_p(c.dtype, qd, w.ld_proj, L.kc, L.vc, b.pos + b.n_pre, b.row_seq + b.n_pre, b.tables, b.max_blocks,
                         c.block_size, od, w.ld_cat, gd, w.ld_proj, n_dec, L.hq, L.hk, L.dk, L.dv, L.dkp, L.dvp, L.scale,
-                        L.softcap, elems, L.out_scale, L.window, s);
+                          L.softcap, elems, L.out_scale, L.window, &x, s);
     if (rc) return rc;
   }
   return BB_OK;
@@ -238,6 +257,25 @@ int mlstm(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBat
   return bb_hy_head_post(&c, &L, &w, rows, s);
 }
 
+int gated_linear(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
+  if (b.n_pre > 0) {
+    BB_TRY(project_f32(c, L.w2, at(c, w.proj, L.off_w1), w.ld_proj, w.f32, w.ld_f32, b.n_pre, 1.f, 0, s));
+    BB_TRY(bb_hy_linear_scan(&c, &L, &w, &b, s));
+  }
+  return bb_hy_linear_decode(&c, &L, &w, &b, s);
+}
+
+int retention(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
+  if (b.n_pre > 0) {
+    BB_TRY(bb_hy_turn(&c, &L, &w, &b, s));
+    const int rc = bb_retention_chunk(&c, &L, &w, &b, s);
+    if (rc == BB_ESIZE) BB_TRY(bb_hy_linear_scan(&c, &L, &w, &b, s));   // fp32, or sizes the tiles do not cover
+    else if (rc) return rc;
+    else BB_TRY(bb_hy_linear_post(&c, &L, &w, b.n_pre, s));
+  }
+  return bb_hy_linear_decode(&c, &L, &w, &b, s);
+}
+
 int mixer(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
   switch (L.kind) {
     case 0: return attention(c, L, w, b, s);
@@ -246,6 +284,8 @@ int mixer(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBat
     case 3: return general_delta(c, L, w, b, s);
     case 4: return rglru(c, L, w, b, s);
     case 5: return mlstm(c, L, w, b, s);
+    case 6: return gated_linear(c, L, w, b, s);
+    case 7: return retention(c, L, w, b, s);
     default: return BB_EARG;
   }
 }
@@ -380,17 +420,66 @@ int forward_start(const BbHyCfg& c, const BbHyWork& w, const BbHyBatch& b, float
   return bb_hy_start(&c, c.n_layers, &w, &b, 0, nullptr, s);
 }
 
+// Layers with several residual streams: mixer, then feed-forward, hy_streams before each and behind the last.  In small
+// steps mixers side by side run on two streams of the device.
+int forward_streams(const BbHyCfg& c, const BbHyWork& w, const BbHyBatch& b, float* trace, void* s) {
+  SideStream* side = b.n <= BESIDE_ROWS ? side_stream() : nullptr;
+  const cudaStream_t main = (cudaStream_t)s;
+  const size_t level = (size_t)b.n * c.dp;
+  const BbHyLayer* before = nullptr;
+  int fq = 0;
+  for (int li = 0; li < c.n_layers; ++li) {
+    const BbHyLayer& L = c.layers[li];
+    BB_TRY(bb_hy_streams(&c, before, fq, &L, 0, &w, &b, 0, trace && li ? trace + (li - 1) * level : nullptr, s));
+    BB_TRY(bb_hy_shift(&c, &L, &w, &b, s));
+    BB_TRY(project(c, L.in, w.h, c.dp, w.proj, w.ld_proj, b.n, s));
+    if (L.beside) {
+      BbHyWork v = w;
+      v.cat = at(c, w.cat, L.beside->off_cat);
+      const cudaStream_t t = side ? side->s : main;
+      if (side) {
+        BB_CUDA(cudaEventRecord(side->fork, main));
+        BB_CUDA(cudaStreamWaitEvent(side->s, side->fork, 0));
+      }
+      BB_TRY(mixer(c, *L.beside, v, b, t));
+      BB_TRY(project(c, L.beside->out, v.cat, w.ld_cat, w.yb, c.dp, b.n, t));
+      if (side) BB_CUDA(cudaEventRecord(side->join, side->s));
+    }
+    BB_TRY(mixer(c, L, w, b, s));
+    BB_TRY(project(c, L.out, w.cat, w.ld_cat, w.ya, c.dp, b.n, s));
+    if (L.beside && side) BB_CUDA(cudaStreamWaitEvent(main, side->join, 0));
+    before = &L;
+    fq = 0;
+    if (L.n_experts > 0 || L.down.w) {
+      BB_TRY(bb_hy_streams(&c, before, fq, &L, 1, &w, &b, 0, nullptr, s));
+      fq = 1;
+      if (L.n_experts > 0) {
+        BB_TRY(route(c, L, w, b, s));
+        BB_TRY(experts(c, L, w, b, s));
+      } else {
+        BB_TRY(project(c, L.up, w.h, c.dp, w.proj, w.ld_proj, b.n, s));
+        BB_TRY(bb_hy_gelu(&c, &L, &w, b.n, s));
+        BB_TRY(project(c, L.down, w.cat, w.ld_cat, w.ya, c.dp, b.n, s));
+      }
+    }
+  }
+  if (trace) BB_TRY(bb_hy_streams(&c, before, fq, nullptr, 0, &w, &b, 1, trace + (c.n_layers - 1) * level, s));
+  return bb_hy_streams(&c, before, fq, nullptr, 0, &w, &b, 0, nullptr, s);
+}
+
 }  // namespace
 
 // One step.  Logits land in w->logits [n_want, vocabp]; `trace` (may be null): fp32 [n_layers][n][dp]
 // copies of the residual stream after every layer.
 BB_API int bb_hybrid_forward(const BbHyCfg* c, const BbHyWork* w, const BbHyBatch* b, float* trace, void* stream) {
   if (!c || !w || !b || b->n <= 0 || b->n > w->rows || b->n_want > w->want_rows) return BB_EARG;
-  if (c->depth_avg || !c->embed_norm) {
-    BB_TRY(c->depth_avg ? forward_depth(*c, *w, *b, trace, stream) : forward_start(*c, *w, *b, trace, stream));
+  if (c->streams > 0 || c->depth_avg || !c->embed_norm) {
+    BB_TRY(c->streams > 0 ? forward_streams(*c, *w, *b, trace, stream)
+                          : (c->depth_avg ? forward_depth : forward_start)(*c, *w, *b, trace, stream));
     if (b->n_want <= 0) return BB_OK;
     const BbHyLin head{c->head, c->vocabp, c->dp};
-    return project_f32(*c, head, w->hn, c->dp, w->logits, c->vocabp, b->n_want, 1.f, 0, stream);
+    BB_TRY(project_f32(*c, head, w->hn, c->dp, w->logits, c->vocabp, b->n_want, 1.f, 0, stream));
+    return bb_hy_cap(c, w, b->n_want, stream);
   }
   BB_TRY(bb_hy_embed_norm(c, b->tok, w->x, b->n, stream));
   for (int li = 0; li < c->n_layers; ++li) {
