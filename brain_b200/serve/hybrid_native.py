@@ -83,6 +83,12 @@ class Work(C.Structure):
                [("ya", P), ("yb", P), ("pk", P), ("ld_pk", I), ("pk_rows", I)]
 
 
+class Pooled(C.Structure):
+    """``csrc/common/pooled.hpp``: what attention over a window has beside it."""
+    _fields_ = [("pool", I), ("pool_rows", I), ("pkc", P), ("pvc", P), ("pk", P), ("ld_pk", I), ("pk_rows", I), ("pool_row0", P),
+                ("sink", P), ("vcos", P), ("vsin", P), ("vturn", I)]
+
+
 def padded_rows(w: torch.Tensor, heads: int, size: int, sizep: int) -> torch.Tensor:
     """[heads * size, k] -> [heads * sizep, k], zero rows after every head."""
     if size == sizep:
@@ -151,8 +157,8 @@ def columns(sections: List[Tuple[torch.Tensor, int]], np_: int) -> torch.Tensor:
 
 def check_layout(lib) -> None:
     """The mirrors above have the library's structure sizes (a stale build raises here, not on the GPU)."""
-    out = (C.c_int * 4)()
+    out = (C.c_int * 5)()
     lib.bb_hybrid_sizes(out)
-    mine = [C.sizeof(s) for s in (Layer, Cfg, Batch, Work)]
+    mine = [C.sizeof(s) for s in (Layer, Cfg, Batch, Work, Pooled)]
     if list(out) != mine:
         raise RuntimeError(f"hybrid structures: library {list(out)}, binding {mine}; rebuild the native library")

@@ -5,7 +5,7 @@
 // constants of the heads, or sigmoid(z)^root of a token's z; what is carried is decay - 1 (expm1 of the logarithm), so that
 // a decay next to one keeps its rate.
 //   hy_linear_scan    prompt portions: the state of a (sequence, head, value columns) in registers, four or more key
-//                     channels times eight value columns to a thread; tokens come in tiles of 16 through shared memory
+//                     channels times eight value columns to a thread; tokens come in tiles through shared memory
 //   hy_linear_decode  one token per sequence: z, rotation, state, norm and gate in one kernel; the state is read and
 //                     written once
 //   hy_linear_post    norm and gate, where a head's columns were spread over blocks
@@ -26,7 +26,8 @@ __device__ __forceinline__ void copy16_async(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
 
-constexpr int LS_TOK = 16;       // tokens of a tile
+// tokens of a tile, by the channels that its lanes cover
+__host__ __device__ constexpr int scan_tokens(int wide) { return wide > 256 ? 8 : 16; }
 
 // What a tile keeps in shared memory, in floats: raw inputs (two tiles), decays, keys and queries [tok][channels], values
 // and outputs [tok][columns].
@@ -36,7 +37,8 @@ struct ScanTile {
   bool z;
   __host__ __device__ int raw_row() const { return (2 * np + 2 * pr) * (int)sizeof(T) + (z ? 4 * np : 0); }   // bytes of a token
   __host__ __device__ size_t bytes(int wide) const {
-    return (size_t)2 * LS_TOK * raw_row() + 4ull * LS_TOK * (3 * wide + 2 * pc);
+    const int tok = scan_tokens(wide);
+    return (size_t)2 * tok * raw_row() + 4ull * tok * (3 * wide + 2 * pc);
   }
 };
 
@@ -48,6 +50,7 @@ hy_linear_scan_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__
                       int ldz, T* __restrict__ out, int ldo, const __grid_constant__ BbHyBatch b, int seq0, int pc, float eps) {
   extern __shared__ __align__(16) unsigned char ls_smem[];
   constexpr int NW = NG * A;                          // channels that the lanes cover
+  constexpr int LS_TOK = scan_tokens(NW);
   const int seq = seq0 + blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * pc;
   const int tid = threadIdx.x, nt_all = blockDim.x, lane = tid & 31, ng = lane % NG;
   const int col = ((tid >> 5) * (32 / NG) + lane / NG) * 8;        // first of the thread's columns in the block

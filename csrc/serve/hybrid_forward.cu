@@ -506,5 +506,6 @@ BB_API int bb_hybrid_sizes(int* out) {
   out[1] = sizeof(BbHyCfg);
   out[2] = sizeof(BbHyBatch);
   out[3] = sizeof(BbHyWork);
+  out[4] = sizeof(BbPooled);
   return BB_OK;
 }

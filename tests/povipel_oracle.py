@@ -48,15 +48,14 @@ def rotate(x, pos, dims, base, interleaved, back=False):
 # ------------------------------------------------------------------------------------ mixers
 def seen(i, size, pool):
     """(tokens, pooled blocks) that position i attends to."""
-    toks = range(max(0, i - size + 1), i + 1)
-    return list(toks), [b for b in range(i // pool + 1) if b * pool + pool - 1 <= i - size]
+    toks = list(range(max(0, i - size + 1) if size else 0, i + 1))
+    return toks, [b for b in range(i // pool + 1) if b * pool + pool - 1 <= i - size] if pool else []
 
 
 def pooled_window(q, k, v, scale, size, pool, sink):
     """One head: q, k [T, D], v [T, E]; a window of tokens, means of the blocks behind it, a sink in the denominator."""
-    T, n = q.shape[0], q.shape[0] // pool
-    kp = k[:n * pool].reshape(n, pool, -1).mean(axis=1)
-    vp = v[:n * pool].reshape(n, pool, -1).mean(axis=1)
+    T, n = q.shape[0], q.shape[0] // pool if pool else 0
+    kp, vp = (x[:n * (pool or 1)].reshape(n, pool or 1, x.shape[1]).mean(axis=1) for x in (k, v))
     out = np.zeros((T, v.shape[1]))
     for i in range(T):
         toks, blocks = seen(i, size, pool)
@@ -69,7 +68,7 @@ def pooled_window(q, k, v, scale, size, pool, sink):
 
 def attention(h, W, p, m, eps):
     T, H, G, D, E = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    pos, rot = np.arange(T), m["rot"]
+    pos, rot, mask = np.arange(T), m["rot"], m.get("mask") or {}
     proj = lambda n, heads, size: (h @ W[p + n].T).reshape(T, heads, size)
     q = rotate(rms(proj("q", H, D), eps) * W[p + "q.norm"], pos, rot["dims"], rot["base"], True)
     k = rotate(rms(proj("k", G, D), eps) * W[p + "k.norm"], pos, rot["dims"], rot["base"], True)
@@ -77,7 +76,7 @@ def attention(h, W, p, m, eps):
     out = np.zeros((T, H, E))
     for i in range(H):
         g = i // (H // G)
-        out[:, i] = pooled_window(q[:, i], k[:, g], v[:, g], m["scale"], m["mask"]["size"], m["mask"]["pool"], W[p + "sink"][i])
+        out[:, i] = pooled_window(q[:, i], k[:, g], v[:, g], m["scale"], mask.get("size"), mask.get("pool"), W[p + "sink"][i])
     return rotate(out, pos, E, rot["base"], True, back=True).reshape(T, H * E) @ W[p + "o"].T
 
 
@@ -181,5 +180,5 @@ def forward(cfg, W, tokens, layers_out=None):
         if layers_out is not None:
             layers_out.append(X.sum(axis=0))
     z = layer_norm(X.sum(axis=0), W["final.norm"], W["final.norm.b"], eps) @ W["head"].T
-    cap = cfg["logit_softcap"]
-    return cap * np.tanh(z / cap)
+    cap = cfg.get("logit_softcap")
+    return cap * np.tanh(z / cap) if cap else z
