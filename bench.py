@@ -36,9 +36,9 @@ def parse():
     ap.add_argument("--micro-batch", type=int, default=4)
     ap.add_argument("--layers", type=int, default=0, help="debug only: override depth (invalidates the number)")
     ap.add_argument("--no-e2e", action="store_true")
-    ap.add_argument("--workload", default="train", choices=["train", "hybrid", "nezalorn", "zepesun"],
+    ap.add_argument("--workload", default="train", choices=["train", "hybrid", "nezalorn", "zepesun", "povipel"],
                     help="train: the headline benchmark; hybrid: prefill and decode of the hybrid decoder beside "
-                         "the dense one; nezalorn, zepesun: of that design beside the other hybrid decoders (one GPU)")
+                         "the dense one; nezalorn, zepesun, povipel: of that design beside the other hybrid decoders (one GPU)")
     ap.add_argument("--hybrid-size", default="m", choices=["s", "m", "l"])
     ap.add_argument("--no-kernels", action="store_true", help="serving workloads: throughput only")
     return ap.parse_args()
@@ -98,7 +98,7 @@ def hybrid_workload(args):
     torch.cuda.set_device(0)
     sampler = ClockSampler(0)
     sampler.start()
-    if args.workload in ("nezalorn", "zepesun"):
+    if args.workload in ("nezalorn", "zepesun", "povipel"):
         import importlib
         bench = importlib.import_module(f"brain_b200.perf.{args.workload}_bench")
         r = bench.run(args.hybrid_size, steps=max(args.steps, 3), with_kernels=not args.no_kernels)
