@@ -32,7 +32,7 @@ NVCC_FLAGS = [
 #: (the hybrid decoder's norms, recurrence and fp32 path: what is computed in 32-bit keeps its 32 bits)
 EXACT_MATH = {"adamw.cu", "rs_adamw.cu", "ce.cu", "hybrid_rows.cu", "mamba2.cu", "attn_rows.cu", "sgemm.cu",
               "depth_rows.cu", "latent_rows.cu", "delta.cu", "rglru.cu", "mlstm.cu", "experts.cu",
-              "stream_rows.cu", "head_rows.cu", "linear_state.cu"}
+              "stream_rows.cu", "head_rows.cu", "linear_state.cu", "gla_tcgen05.cu"}
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread", "-march=x86-64-v3"]
 
 
@@ -170,7 +170,7 @@ def build_bounds(force: bool = False, verbose: bool = False) -> Path:
 #: what serving a hybrid decoder needs of the kernel library, for programs that compile on first use
 HYBRID_TUS = ["common/host.cu", "kernels/attn_rows.cu", "kernels/delta.cu", "kernels/depth_rows.cu", "kernels/experts.cu",
               "kernels/flash_fwd.cu",
-              "kernels/gemm_2cta.cu", "kernels/gemm_groups.cu", "kernels/gemm_tcgen05.cu", "kernels/head_rows.cu",
+              "kernels/gemm_2cta.cu", "kernels/gemm_groups.cu", "kernels/gemm_tcgen05.cu", "kernels/gla_tcgen05.cu", "kernels/head_rows.cu",
               "kernels/hybrid_rows.cu",
               "kernels/latent_decode.cu", "kernels/latent_rows.cu", "kernels/linear_state.cu",
               "kernels/mamba2.cu", "kernels/mlstm.cu", "kernels/paged_kv.cu",

@@ -163,14 +163,17 @@ def kernels(eng, entries, phase, timer, peaks):
             row(f"{tag}: state step, norm, gate", t("bb_hy_linear_decode", cfg, lm, w, bb), "recurrence", (io + state) / 1e9)
         elif m is side:
             gemm("gated linear: decays (fp32)", "router", at("proj", m.off_w1), ld["proj"], m.w2, P(sc.f32.data_ptr()), ld["f32"], mode=1)
-            row("gated linear: scan, norm, gate", t("bb_hy_linear_scan", cfg, lm, w, bb), "recurrence",
+            row("gated linear: chunks, norm, gate", t("bb_gla_chunk", cfg, lm, w, bb), "recurrence",
+                (io + n * m.heads * m.np * 4 + state) / 1e9)
+            row("gated linear: pairs left to the scan", t("bb_hy_linear_scan", cfg, lm, w, bb, 1), "recurrence", 0.0)
+            row("gated linear: scan, norm, gate (fallback)", t("bb_hy_linear_scan", cfg, lm, w, bb, 0), "recurrence",
                 (io + n * m.heads * m.np * 4 + state) / 1e9)
         else:
             row("retention: rotation", t("bb_hy_turn", cfg, lm, w, bb), "attention post", n * m.heads * m.np * 8 / 1e9)
             row("retention: chunks", t("bb_retention_chunk", cfg, lm, w, bb), "recurrence",
                 (n * m.heads * (2 * m.np + 2 * m.pp) * 2 + state) / 1e9)
             row("retention: norm, gate", t("bb_hy_linear_post", cfg, lm, w, n), "post (glu)", n * m.heads * m.pp * 6 / 1e9)
-            row("retention: scan, norm, gate (fallback)", t("bb_hy_linear_scan", cfg, lm, w, bb), "recurrence", (io + state) / 1e9)
+            row("retention: scan, norm, gate (fallback)", t("bb_hy_linear_scan", cfg, lm, w, bb, 0), "recurrence", (io + state) / 1e9)
     row("logits: bound", t("bb_hy_cap", cfg, w, b.n_want), "post (glu)", b.n_want * eng.vocabp * 8 / 1e9)
     del blob
     return out

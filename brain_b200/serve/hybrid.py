@@ -74,8 +74,7 @@ class _Scratch:
         self.q, self.qa, self.ol, self.aux = z(rows, m["q"]), z(ab, m["qa"]), z(ab, m["ol"]), z(rows, m["aux"])
         self.ckv, self.kvx = z(max(exp, 1), m["ckv"]), z(max(exp, 1), m["kvx"])
         self.f32 = z(rows, m["f32"], dtype=f32)
-        self.part32 = z(-(-eng.dp // 64) * min(rows, 128) * m["f32"] if m["f32"] > 8 or any(l.in32.n for l in eng.layers) else 1,
-                        dtype=f32)
+        self.part32 = z(max(-(-eng.dp // 64) * min(rows, 128) * max(l.in32.n for l in eng.layers), 1), dtype=f32)
         # mixture of experts: every expert that has rows takes at most one 128-row tile that is not full
         routed = [l for l in eng.layers if l.n_experts]
         top = max((l.top for l in routed), default=0)
@@ -100,12 +99,19 @@ class _Scratch:
         npmax = max([l.mem if l.kind == 5 else l.n * l.p for l in eng.mixers if l.kind in (1, 5, 7) and max(l.n, l.p) <= 128],
                     default=0)
         self.seg = z(2 * 2 * eng.sm_count * (npmax + 1) if portions and not eng.fp32 and npmax else 1, dtype=f32)
+        # chunks of gated linear attention, one sequence's last ones not full
+        gla = [l for l in eng.mixers if l.kind == 6 and l.np <= 64 and l.pp <= 128] if portions and not eng.fp32 else []
+        slots = rows // 128 + 32
+        self.chunks = z(max((slots * l.heads * l.n * l.p for l in gla), default=1), dtype=f32)
+        self.chunk_flags = z(max((slots * l.heads for l in gla), default=1), dtype=i32)
         self.hn, self.logits = z(max(want, 1), eng.dp), z(max(want, 1), eng.vocabp, dtype=f32)
         w = self.work = hn.Work()
         for n in ("x", "h", "proj", "cat", "xbc", "dt", "y", "v_first", "part_o", "part_ml", "seg", "hn", "logits", "h2", "q",
                   "qa", "ol", "aux", "ckv", "kvx", "f32", "part32", "ex_in", "ex_gu", "ex_act", "ex_out", "pair_expert", "pair_row",
-                  "pair_w", "ex_count", "ex_tile", "ya", "yb", "pk"):
+                  "pair_w", "ex_count", "ex_tile", "ya", "yb", "pk", "chunks",
+                  "chunk_flags"):
             setattr(w, n, _ptr(getattr(self, n)))
+        w.chunk_floats, w.chunk_marks = self.chunks.numel(), self.chunk_flags.numel()
         w.seg_floats, w.part32_floats = self.seg.numel(), self.part32.numel()
         w.rows, w.want_rows, w.exp_rows, w.moe_rows, w.pk_rows = rows, max(want, 1), exp, moe, self.pk.shape[0]
         for k in m:
@@ -409,7 +415,7 @@ class HybridEngine(PagedEngineBase):
         L.w2 = self._lin(hn.columns([(self._rows(p + "a2", H, m.dim), L.wrp)], H * np_))
         L.w0 = self._head_vec(p + "a2.b", H, m.dim)
         L.gnorm = self._hold(hn.head_vec(scale * self._tensor(p + "norm").float().repeat(H), H, m.vdim, L.pp, self.device))
-        self._widest(f32=H * np_)
+        self._widest(f32=2 * H * np_)          # z, and in chunks the sums of the decays' logarithms
         return out
 
     def _pack_retention(self, i: int, L, m, p: str, stack):

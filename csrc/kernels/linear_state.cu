@@ -4,7 +4,7 @@
 // and the head's output is o over its root mean square, times a gain (or none) and the silu of a gate.  The decays are
 // constants of the heads, or sigmoid(z)^root of a token's z; what is carried is decay - 1 (expm1 of the logarithm), so that
 // a decay next to one keeps its rate.
-//   hy_linear_scan    prompt portions: the state of a (sequence, head, value columns) in registers, four or more key
+//   hy_linear_scan    prompt portions that the chunked kernels (gla_tcgen05, ssd_tcgen05) do not cover: the state of a (sequence, head, value columns) in registers, four or more key
 //                     channels times eight value columns to a thread; tokens come in tiles through shared memory
 //   hy_linear_decode  one token per sequence: z, rotation, state, norm and gate in one kernel; the state is read and
 //                     written once
@@ -43,15 +43,23 @@ struct ScanTile {
 };
 
 // NG lanes share a column's channels, A channels each; 32 / NG groups of 8 columns to a warp.  FUSE: the block has all of a
-// head's columns and finishes its rows (-> cat), else outputs go to y.
+// head's columns and finishes its rows (-> cat), else outputs go to y.  marks (may be null): of every (chunk of 128 tokens,
+// head); pairs without any are left alone.
 template <typename T, int NG, int A, bool FUSE>
 __global__ void __launch_bounds__(256)
 hy_linear_scan_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__ proj, int ld, const float* __restrict__ z,
-                      int ldz, T* __restrict__ out, int ldo, const __grid_constant__ BbHyBatch b, int seq0, int pc, float eps) {
+                      int ldz, T* __restrict__ out, int ldo, const __grid_constant__ BbHyBatch b, int pc,
+                      const int* __restrict__ marks, float eps) {
   extern __shared__ __align__(16) unsigned char ls_smem[];
   constexpr int NW = NG * A;                          // channels that the lanes cover
   constexpr int LS_TOK = scan_tokens(NW);
-  const int seq = seq0 + blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * pc;
+  const int seq = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * pc;
+  if (marks) {
+    const int n = (b.seq_row0[seq + 1] - b.seq_row0[seq] + 127) / 128, s0 = b.seq_row0[seq] / 128 + seq;
+    bool any = false;
+    for (int c = 0; c < n; ++c) any |= marks[(s0 + c) * L.heads + h] != 0;
+    if (!any) return;
+  }
   const int tid = threadIdx.x, nt_all = blockDim.x, lane = tid & 31, ng = lane % NG;
   const int col = ((tid >> 5) * (32 / NG) + lane / NG) * 8;        // first of the thread's columns in the block
   const int N = L.n, P = L.p;
@@ -346,19 +354,18 @@ hy_linear_post_kernel(const __grid_constant__ BbHyLayer L, const T* __restrict__
 }
 
 template <typename T>
-static int launch_post(const BbHyLayer& L, const BbHyWork& w, size_t r0, int rows, float eps, cudaStream_t s) {
+static int launch_post(const BbHyLayer& L, const BbHyWork& w, int rows, float eps, cudaStream_t s) {
   if (rows <= 0) return BB_OK;
   int lanes = 1;
   while (lanes < L.pp / 8 && lanes < 32) lanes <<= 1;
-  hy_linear_post_kernel<T><<<rows, LP_THREADS, 0, s>>>(L, static_cast<const T*>(w.proj) + r0 * w.ld_proj, w.ld_proj,
-                                                       static_cast<const T*>(w.y) + r0 * w.ld_y, w.ld_y,
-                                                       static_cast<T*>(w.cat) + r0 * w.ld_cat, w.ld_cat, lanes, eps);
+  hy_linear_post_kernel<T><<<rows, LP_THREADS, 0, s>>>(L, static_cast<const T*>(w.proj), w.ld_proj, static_cast<const T*>(w.y), w.ld_y,
+                                                       static_cast<T*>(w.cat), w.ld_cat, lanes, eps);
   return (int)cudaGetLastError();
 }
 
 template <typename T, int NG, int A>
-static int launch_scan_n(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, const float* z, int seq0, int n_seq,
-                         int first_row, int rows, float eps, cudaStream_t s) {
+static int launch_scan_n(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, const float* z, const int* marks,
+                         float eps, cudaStream_t s) {
   static PerDeviceOnce once, once_fused;
   constexpr int LIMIT = 200 * 1024;
   cudaError_t e = ensure_dyn_smem(once, hy_linear_scan_kernel<T, NG, A, false>, LIMIT);
@@ -367,12 +374,13 @@ static int launch_scan_n(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch&
   if (e != cudaSuccess) return (int)e;
   // columns of a block: up to eight warps, as few parts of a head as keep the machine's warps busy
   constexpr int WARP_COLS = 32 / NG * 8;
-  const long pairs = (long)n_seq * L.heads;
+  const long pairs = (long)b.ns_pre * L.heads;
   const int sms = sm_count();
   int pc = 0;
   long best = 0;
   for (int warps = 8; warps >= 1; warps >>= 1) {
     const int c = warps * WARP_COLS, parts = (L.p + c - 1) / c, used = parts > 1 ? warps : (L.p + WARP_COLS - 1) / WARP_COLS;
+    if (marks && parts > 1) continue;                          // (the other pairs' rows are finished)
     if (ScanTile<T>{L.np, parts > 1 ? c : used * WARP_COLS, c, z != nullptr}.bytes(NG * A) > LIMIT) continue;
     long cost = (pairs * parts + sms - 1) / sms * used;       // warps that follow one another on an SM
     cost = (cost < 4 ? 4 : cost) * 16 + (parts > 1 ? 4 : 0);  // (a split head takes another launch)
@@ -385,26 +393,26 @@ static int launch_scan_n(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch&
   const int parts = (L.p + pc - 1) / pc, threads = pc / WARP_COLS * 32;
   const size_t smem = ScanTile<T>{L.np, pc, pc, z != nullptr}.bytes(NG * A);
   const T* proj = static_cast<const T*>(w.proj);
-  const dim3 grid(n_seq, L.heads, parts);
+  const dim3 grid(b.ns_pre, L.heads, parts);
   if (parts == 1) {
     hy_linear_scan_kernel<T, NG, A, true><<<grid, threads, smem, s>>>(L, proj, w.ld_proj, z, w.ld_f32, static_cast<T*>(w.cat),
-                                                                      w.ld_cat, b, seq0, pc, eps);
+                                                                      w.ld_cat, b, pc, marks, eps);
     return (int)cudaGetLastError();
   }
   hy_linear_scan_kernel<T, NG, A, false><<<grid, threads, smem, s>>>(L, proj, w.ld_proj, z, w.ld_f32, static_cast<T*>(w.y),
-                                                                     w.ld_y, b, seq0, pc, eps);
+                                                                     w.ld_y, b, pc, marks, eps);
   e = cudaGetLastError();
-  return e != cudaSuccess ? (int)e : launch_post<T>(L, w, first_row, rows, eps, s);
+  return e != cudaSuccess ? (int)e : launch_post<T>(L, w, b.n_pre, eps, s);
 }
 template <typename T>
-static int launch_scan(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, const float* z, int seq0, int n_seq,
-                       int first_row, int rows, float eps, cudaStream_t s) {
-  if (n_seq <= 0) return BB_OK;
-  if (L.n <= 32) return launch_scan_n<T, 8, 4>(L, w, b, z, seq0, n_seq, first_row, rows, eps, s);
-  if (L.n <= 64) return launch_scan_n<T, 16, 4>(L, w, b, z, seq0, n_seq, first_row, rows, eps, s);
-  if (L.n <= 128) return launch_scan_n<T, 32, 4>(L, w, b, z, seq0, n_seq, first_row, rows, eps, s);
-  if (L.n <= 256) return launch_scan_n<T, 32, 8>(L, w, b, z, seq0, n_seq, first_row, rows, eps, s);
-  return L.n <= 512 ? launch_scan_n<T, 32, 16>(L, w, b, z, seq0, n_seq, first_row, rows, eps, s) : BB_ESIZE;
+static int launch_scan(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, const float* z, const int* marks, float eps,
+                       cudaStream_t s) {
+  if (b.ns_pre <= 0) return BB_OK;
+  if (L.n <= 32) return launch_scan_n<T, 8, 4>(L, w, b, z, marks, eps, s);
+  if (L.n <= 64) return launch_scan_n<T, 16, 4>(L, w, b, z, marks, eps, s);
+  if (L.n <= 128) return launch_scan_n<T, 32, 4>(L, w, b, z, marks, eps, s);
+  if (L.n <= 256) return launch_scan_n<T, 32, 8>(L, w, b, z, marks, eps, s);
+  return L.n <= 512 ? launch_scan_n<T, 32, 16>(L, w, b, z, marks, eps, s) : BB_ESIZE;
 }
 
 static int lanes_of(int p) {
@@ -440,12 +448,13 @@ static int launch_decode(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch&
 using namespace bb;
 
 // The prompt portions token by token: recurrence, norm and gate -> w->cat.  Queries and keys are rotated; z of a token in
-// w->f32 where decays are not constant.
-BB_API int bb_hy_linear_scan(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream) {
+// w->f32 where decays are not constant.  `marked`: only the pairs that bb_gla_chunk has marked.
+BB_API int bb_hy_linear_scan(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int marked, void* stream) {
   const float* z = L->w2.w ? w->f32 : nullptr;
+  const int* marks = marked ? w->chunk_flags : nullptr;
   cudaStream_t s = (cudaStream_t)stream;
-  return c->dtype ? launch_scan<float>(*L, *w, *b, z, 0, b->ns_pre, 0, b->n_pre, c->eps, s)
-                  : launch_scan<__nv_bfloat16>(*L, *w, *b, z, 0, b->ns_pre, 0, b->n_pre, c->eps, s);
+  return c->dtype ? launch_scan<float>(*L, *w, *b, z, marks, c->eps, s)
+                  : launch_scan<__nv_bfloat16>(*L, *w, *b, z, marks, c->eps, s);
 }
 
 // The single tokens -> w->cat; BB_ESIZE for heads the shared memory does not hold.
@@ -457,6 +466,6 @@ BB_API int bb_hy_linear_decode(const BbHyCfg* c, const BbHyLayer* L, const BbHyW
 
 // Norm and gate of the first `rows` rows of w->y -> w->cat.
 BB_API int bb_hy_linear_post(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int rows, void* stream) {
-  return c->dtype ? launch_post<float>(*L, *w, 0, rows, c->eps, (cudaStream_t)stream)
-                  : launch_post<__nv_bfloat16>(*L, *w, 0, rows, c->eps, (cudaStream_t)stream);
+  return c->dtype ? launch_post<float>(*L, *w, rows, c->eps, (cudaStream_t)stream)
+                  : launch_post<__nv_bfloat16>(*L, *w, rows, c->eps, (cudaStream_t)stream);
 }

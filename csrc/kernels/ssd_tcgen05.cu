@@ -34,6 +34,7 @@
 #include "../common/host.hpp"
 #include "../common/ptx.cuh"
 #include "../common/rows.cuh"
+#include "../common/split.cuh"
 #include "../serve/hybrid.hpp"
 
 namespace bb {
@@ -68,33 +69,6 @@ struct GatedSmem {
   __device__ explicit GatedSmem(float* p)
       : n(p), w(p + 128), sum(p + 256), nq(sum + W * 128), part(nq + W * 128), pm(part + 4 * W * 128), co(pm + 4) {}
 };
-
-__device__ __forceinline__ float2 split_pair(float a, float b) {
-  // packed bf16 pair of the values, packed pair of what rounding left over
-  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-  const float2 f = __bfloat1622float2(h);
-  const __nv_bfloat162 l = __floats2bfloat162_rn(a - f.x, b - f.y);
-  return make_float2(__uint_as_float(*reinterpret_cast<const uint32_t*>(&h)),
-                     __uint_as_float(*reinterpret_cast<const uint32_t*>(&l)));
-}
-
-// 32 fp32 values of row `row`, columns col0.. (a multiple of 8), as two bf16 terms into two swizzled tiles.
-__device__ __forceinline__ void store_split(uint8_t* hi, uint8_t* lo, int row, int col0, const float (&v)[32]) {
-#pragma unroll
-  for (int q = 0; q < 4; ++q) {
-    uint32_t h[4], l[4];
-#pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      const float2 t = split_pair(v[q * 8 + 2 * k], v[q * 8 + 2 * k + 1]);
-      h[k] = __float_as_uint(t.x);
-      l[k] = __float_as_uint(t.y);
-    }
-    const int col = col0 + q * 8;
-    const int o = (col >> 6) * SSD_SUB + row * 128 + ((((col & 63) >> 3) ^ (row & 7)) << 4);
-    *reinterpret_cast<uint4*>(hi + o) = make_uint4(h[0], h[1], h[2], h[3]);
-    *reinterpret_cast<uint4*>(lo + o) = make_uint4(l[0], l[1], l[2], l[3]);
-  }
-}
 
 template <int PP, bool LOCAL, bool GATED, int W>
 __global__ void __launch_bounds__(W * 128, PP == 64 ? 2 : 1)
@@ -349,7 +323,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
           r[j] = __float_as_uint(v[j] * dec);
         }
         tmem_st32(tS + c, r);
-        if (!LOCAL) store_split(sS, sSl, row, half * HC + c, v);
+        if (!LOCAL) store_split(sS, sSl, row, half * HC + c, v, SSD_SUB);
       }
       tmem_wait_st();
     }
@@ -462,7 +436,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tmBC, const __grid_constant
 #pragma unroll
           for (int j = 0; j < 8; ++j) v[q * 8 + j] = f[j] * w_in;
         }
-        store_split(sS, sSl, row, col0, v);   // the state operand is behind its products
+        store_split(sS, sSl, row, col0, v, SSD_SUB);   // the state operand is behind its products
       }
     }
     tmem_wait_st();

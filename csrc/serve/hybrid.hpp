@@ -184,6 +184,10 @@ struct BbHyWork {
   // portions see, [pk_rows, ld_pk], of sequence s from ctx_row0[s] / pool on
   void *ya, *yb, *pk;
   int ld_pk, pk_rows;
+  // chunks of gated linear attention: [n_pre / 128 + ns_pre][heads][n][p] and marks [..][heads]
+  float* chunks;
+  int* chunk_flags;
+  long chunk_floats, chunk_marks;
 };
 
 // Rows and pitch of a latent attention layer's queries: through their own latent, or straight from the input.

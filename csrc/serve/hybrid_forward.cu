@@ -79,7 +79,8 @@ int bb_hy_streams(const BbHyCfg* c, const BbHyLayer* before, int fq, const BbHyL
 int bb_hy_shift(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
 int bb_hy_gelu(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream);
 int bb_hy_cap(const BbHyCfg* c, const BbHyWork* w, int n, void* stream);
-int bb_hy_linear_scan(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_gla_chunk(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
+int bb_hy_linear_scan(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, int marked, void* stream);
 int bb_hy_linear_decode(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
 int bb_hy_linear_post(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int rows, void* stream);
 int bb_retention_chunk(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, const BbHyBatch* b, void* stream);
@@ -260,7 +261,9 @@ int mlstm(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBat
 int gated_linear(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, void* s) {
   if (b.n_pre > 0) {
     BB_TRY(project_f32(c, L.w2, at(c, w.proj, L.off_w1), w.ld_proj, w.f32, w.ld_f32, b.n_pre, 1.f, 0, s));
-    BB_TRY(bb_hy_linear_scan(&c, &L, &w, &b, s));
+    const int rc = bb_gla_chunk(&c, &L, &w, &b, s);
+    if (rc && rc != BB_ESIZE) return rc;
+    BB_TRY(bb_hy_linear_scan(&c, &L, &w, &b, rc == BB_OK, s));    // what is left: marked pairs, or fp32 and other sizes
   }
   return bb_hy_linear_decode(&c, &L, &w, &b, s);
 }
@@ -269,7 +272,7 @@ int retention(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, const BbH
   if (b.n_pre > 0) {
     BB_TRY(bb_hy_turn(&c, &L, &w, &b, s));
     const int rc = bb_retention_chunk(&c, &L, &w, &b, s);
-    if (rc == BB_ESIZE) BB_TRY(bb_hy_linear_scan(&c, &L, &w, &b, s));   // fp32, or sizes the tiles do not cover
+    if (rc == BB_ESIZE) BB_TRY(bb_hy_linear_scan(&c, &L, &w, &b, 0, s));   // fp32, or sizes the tiles do not cover
     else if (rc) return rc;
     else BB_TRY(bb_hy_linear_post(&c, &L, &w, b.n_pre, s));
   }

@@ -179,7 +179,9 @@ class Layer:
         b.ns, b.ns_pre, b.n, b.n_pre, b.max_len = ns, ns - dec, n, n - dec, max(lens)
         ctx = [a + s for a, s in zip(lens, starts)]
         b.max_ctx = max(ctx[:ns - dec], default=0)
-        return self.put(b, seq_row0=i32(np.concatenate([[0], np.cumsum(lens)])), seq_pos0=i32(starts), seq_ctx=i32(ctx),
+        tiles = [(s, t) for s in range(ns - dec) for t in range(-(-lens[s] // 128))][::-1]
+        b.n_tiles = len(tiles)
+        return self.put(b, tile_seq=i32([t[0] for t in tiles]), tile_qt=i32([t[1] for t in tiles]), seq_row0=i32(np.concatenate([[0], np.cumsum(lens)])), seq_pos0=i32(starts), seq_ctx=i32(ctx),
                         seq_slot=i32(slots or range(ns)), pos=i32(np.concatenate([np.arange(s, s + l) for s, l in zip(starts, lens)])),
                         row_seq=i32(np.repeat(np.arange(ns), lens)), ctx_row0=i32(np.concatenate([[0], np.cumsum(ctx)])))
 
@@ -294,14 +296,18 @@ class Memory(Layer):
             w2 = w2.to(dtype)
             L.decay_root, L.wr, L.wrp = root, R, R
             z = torch.tensor(rounded[:, o[4]:]) @ w2.double().reshape(-1, R).T
-            self.z = z.float().cuda().contiguous()
+            self.z = torch.cat([z.float(), torch.full((n, H * np_), 7.0)], 1).cuda().contiguous()
             w.ld_f32 = self.z.shape[1]
+            slots = self.b.n_pre // 128 + self.b.ns_pre
+            self.flags = i32(np.full(slots * H, 9))
+            self.put(w, chunks=torch.full((slots * H * N * P,), float("nan"), device="cuda"), chunk_flags=self.flags)
+            w.chunk_floats, w.chunk_marks = slots * H * N * P, slots * H
             dev = w2.cuda().contiguous()
             self.put(w, f32=self.z).put(L, w0=w0.float().reshape(-1).cuda())
             self.hold.append(dev)
             L.w2 = Lin(dev.data_ptr(), H * np_, R)
-            zz = (self.z.cpu().double() + w0.reshape(-1).float().double()).reshape(n, H, np_)[:, :, :N].numpy()
-            self.alpha = np.exp(-np.logaddexp(0.0, -zz) * np.float32(root))
+            self.w0, self.root = w0.float(), root
+            self.decays()
         else:
             d = np.asarray(decay, dtype=np.float64)
             self.put(L, keep_less=torch.tensor(d - 1.0).float().cuda(), a=torch.tensor(np.log(d)).float().cuda())
@@ -310,6 +316,13 @@ class Memory(Layer):
             ang = torch.arange(2048).double()[:, None] * torch.tensor([self.base ** (-2.0 * i / rot) for i in range(rot // 2)], dtype=torch.float64)
             L.rot = rot
             self.put(L, cos_t=ang.cos().float().cuda(), sin_t=ang.sin().float().cuda())
+
+    def decays(self):
+        z = (self.z[:, :self.H * self.np].cpu() + self.w0.reshape(-1)).double().reshape(self.n, self.H, self.np)[:, :, :self.N].numpy()
+        self.alpha = np.exp(-np.logaddexp(0.0, -z) * np.float32(self.root))
+
+    def b_rows(self, s):
+        return sum(self.lens[:s]), sum(self.lens[:s + 1])
 
     def check(self, rows, tol, state_tol, first=0):
         """Finished rows and states of the sequences from ``first`` on, against double precision."""
@@ -343,15 +356,49 @@ SLOTS = [3, 1, 0, 5, 8, 2, 4]
 @pytest.mark.parametrize("H,N,P", SIZES)
 def test_scan_with_a_tokens_own_decays(H, N, P, dtype):
     m = Memory(H, N, P, LENS, STARTS, dtype, slots=SLOTS)
-    assert m.call("bb_hy_linear_scan", m.L, m.w, m.b) == 0
+    assert m.call("bb_hy_linear_scan", m.L, m.w, m.b, 0) == 0
     m.check(m.cat, 0.02 if dtype == torch.bfloat16 else 1e-4, 1e-5)
 
 
 @pytest.mark.parametrize("bias", [-40.0, 12.0, 90.0])
 def test_scan_with_decays_near_zero_and_one(bias):
     m = Memory(2, 40, 24, [900, 3], [0, 700], torch.float32, bias=bias, root=1.0)
-    assert m.call("bb_hy_linear_scan", m.L, m.w, m.b) == 0
+    assert m.call("bb_hy_linear_scan", m.L, m.w, m.b, 0) == 0
     m.check(m.cat, 2e-4, 1e-5)
+
+
+@pytest.mark.parametrize("root,bias", [(0.1, 2.0), (0.9, 0.0), (1e-3, 5.0)])
+@pytest.mark.parametrize("H,N,P", [(3, 24, 40), (4, 64, 64), (2, 64, 128), (5, 13, 21), (2, 8, 8), (6, 40, 104), (1, 56, 72)])
+def test_chunks_with_a_tokens_own_decays(H, N, P, root, bias):
+    m = Memory(H, N, P, LENS, STARTS, torch.bfloat16, root=root, bias=bias, slots=SLOTS)
+    assert m.call("bb_gla_chunk", m.L, m.w, m.b) == 0
+    assert m.call("bb_hy_linear_scan", m.L, m.w, m.b, 1) == 0
+    m.check(m.cat, 0.02, 3e-5)
+
+
+def test_pairs_that_decay_too_fast_for_chunks_go_to_the_scan():
+    """One head's channel decays by e^-2 a token in one sequence, another's by e^-40: chunks leave both pairs alone, portions
+    too short for that much stay, and nobody else notices."""
+    m = Memory(3, 24, 40, LENS, STARTS, torch.bfloat16, root=1.0, bias=3.0, slots=SLOTS)
+    a, b = m.b_rows(1), m.b_rows(5)
+    for rows, h, ch, z in ((a, 0, 5, -2.0), (b, 2, 0, -40.0)):
+        m.z[rows[0]:rows[1], h * m.np + ch] = z - m.w0[h, ch]
+    m.decays()
+    assert m.call("bb_gla_chunk", m.L, m.w, m.b) == 0
+    flags, slot0 = m.flags.cpu().numpy().reshape(-1, 3), [sum(LENS[:s]) // 128 + s for s in range(len(LENS))]
+    marked = {(s, h) for s in range(len(LENS)) for h in range(3) if flags[slot0[s]:slot0[s] + -(-LENS[s] // 128), h].any()}
+    assert marked == {(1, 0), (5, 2)}
+    assert m.call("bb_hy_linear_scan", m.L, m.w, m.b, 1) == 0
+    m.check(m.cat, 0.02, 3e-5)
+
+
+def test_chunks_refuse_what_their_scratch_does_not_hold():
+    m = Memory(3, 24, 40, LENS, STARTS, torch.bfloat16)
+    m.w.chunk_floats -= 1
+    assert m.call("bb_gla_chunk", m.L, m.w, m.b) == -3
+    for N, P in ((72, 40), (24, 136)):
+        m = Memory(1, N, P, [3], [0], torch.bfloat16)
+        assert m.call("bb_gla_chunk", m.L, m.w, m.b) == -3
 
 
 @pytest.mark.parametrize("segments", [False, True])
@@ -376,7 +423,7 @@ def test_retention_in_chunks(H, N, P, rot, segments):
 def test_scan_with_constant_decays(H, N, P, rot, dtype):
     m = Memory(H, N, P, LENS, STARTS, dtype, decay=[1.0 - 1e-4 * 9.0 ** h for h in range(H)], rot=rot, slots=SLOTS, eps=0.2)
     assert m.call("bb_hy_turn", m.L, m.w, m.b) == 0
-    assert m.call("bb_hy_linear_scan", m.L, m.w, m.b) == 0
+    assert m.call("bb_hy_linear_scan", m.L, m.w, m.b, 0) == 0
     m.check(m.cat, 0.08 if dtype == torch.bfloat16 else 1e-4, 0.01 if dtype == torch.bfloat16 else 1e-5)
 
 
