@@ -165,7 +165,8 @@ def kernels(eng, entries, phase, timer, peaks):
             gemm("gated linear: decays (fp32)", "router", at("proj", m.off_w1), ld["proj"], m.w2, P(sc.f32.data_ptr()), ld["f32"], mode=1)
             row("gated linear: chunks, norm, gate", t("bb_gla_chunk", cfg, lm, w, bb), "recurrence",
                 (io + n * m.heads * m.np * 4 + state) / 1e9)
-            row("gated linear: pairs left to the scan", t("bb_hy_linear_scan", cfg, lm, w, bb, 1), "recurrence", 0.0)
+            row("gated linear: pairs left to the scan", t("bb_hy_linear_scan", cfg, lm, w, bb, 1), "recurrence",
+                n / 128 * m.heads * 4 / 1e9)
             row("gated linear: scan, norm, gate (fallback)", t("bb_hy_linear_scan", cfg, lm, w, bb, 0), "recurrence",
                 (io + n * m.heads * m.np * 4 + state) / 1e9)
         else:

@@ -780,10 +780,21 @@ fa_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ 
               if (args.vcos) {       // columns past the true head size are zero, whatever they are turned by
                 const int half = args.vturn >> 1, p0 = (c * 32 + q * 8) >> 1;
                 const size_t t0 = (size_t)(q_idx + off) * half;
+                float cs[4], sn[4];
+                if ((half & 3) == 0) {
+                  const float4 c4 = *reinterpret_cast<const float4*>(args.vcos + t0 + p0), s4 = *reinterpret_cast<const float4*>(args.vsin + t0 + p0);
+                  cs[0] = c4.x; cs[1] = c4.y; cs[2] = c4.z; cs[3] = c4.w;
+                  sn[0] = s4.x; sn[1] = s4.y; sn[2] = s4.z; sn[3] = s4.w;
+                } else {
+#pragma unroll
+                  for (int j = 0; j < 4; ++j) {
+                    cs[j] = args.vcos[t0 + min(p0 + j, half - 1)];
+                    sn[j] = args.vsin[t0 + min(p0 + j, half - 1)];
+                  }
+                }
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
-                  const size_t t = t0 + min(p0 + j, half - 1);
-                  const float co = args.vcos[t], si = args.vsin[t];
+                  const float co = cs[j], si = sn[j];
                   const float a = __uint_as_float(r[q * 8 + 2 * j]), b = __uint_as_float(r[q * 8 + 2 * j + 1]);
                   r[q * 8 + 2 * j] = __float_as_uint(fmaf(a, co, b * si));
                   r[q * 8 + 2 * j + 1] = __float_as_uint(fmaf(b, co, -a * si));

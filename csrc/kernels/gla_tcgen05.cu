@@ -31,19 +31,22 @@ __device__ __forceinline__ bool left_to_scan(const int* flags, const BbHyBatch& 
   return any;
 }
 
-// Two terms of one value into column c of a row of two swizzled tiles.
-__device__ __forceinline__ void put_split(uint8_t* hi, uint8_t* lo, int row, int c, float v) {
-  const __nv_bfloat16 a = __float2bfloat16(v);
+// Two terms of two values into columns c, c + 1 (c even) of a row of two swizzled tiles.
+__device__ __forceinline__ void put_split(uint8_t* hi, uint8_t* lo, int row, int c, float a, float b) {
+  const float2 t = split_pair(a, b);
   const int o = swizzled(row, c & ~7, GL_SUB) + (c & 7) * 2;
-  *reinterpret_cast<__nv_bfloat16*>(hi + o) = a;
-  *reinterpret_cast<__nv_bfloat16*>(lo + o) = __float2bfloat16(v - __bfloat162float(a));
+  *reinterpret_cast<float*>(hi + o) = t.x;
+  *reinterpret_cast<float*>(lo + o) = t.y;
+}
+__device__ __forceinline__ float2 load_pair(const __nv_bfloat16* p) {
+  return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
 }
 
 template <int PP>
 struct GlaParts {
   static constexpr int PSUB = PP / 64;
   static constexpr int OFF_K = 0, OFF_V = 2 * GL_SUB, OFF_E = OFF_V + PSUB * GL_SUB;   // keys, two terms; values; sums, barriers
-  static constexpr int SMEM = OFF_E + 4 * 64 * 4 + 64;
+  static constexpr int SMEM = OFF_E + 8 * 64 * 4 + 64;
 };
 
 template <int PP>
@@ -54,7 +57,7 @@ gla_parts_kernel(const __grid_constant__ CUtensorMap tmV, const __grid_constant_
   using Cfg = GlaParts<PP>;
   extern __shared__ __align__(1024) uint8_t smem[];
   uint8_t *sK = smem + Cfg::OFF_K, *sV = smem + Cfg::OFF_V;
-  float* s_sum = reinterpret_cast<float*>(smem + Cfg::OFF_E);      // [4][64]
+  float2* s_sum = reinterpret_cast<float2*>(smem + Cfg::OFF_E);    // [8][32]
   uint64_t *b_v = reinterpret_cast<uint64_t*>(s_sum + 256), *b_s = b_v + 1;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(b_v + 2);
   const int seq = b.tile_seq[blockIdx.x], c = b.tile_qt[blockIdx.x], h = blockIdx.y;
@@ -73,49 +76,57 @@ gla_parts_kernel(const __grid_constant__ CUtensorMap tmV, const __grid_constant_
     tmem_alloc(tmem_slot, PP);
     tmem_relinquish();
   }
-  // a channel's 32 tokens to a thread: logarithms of the decays and their running sum
-  const int ch = threadIdx.x & 63, seg = threadIdx.x >> 6;
-  float lg[32], sum = 0.f;
+  // two channels of 16 tokens to a thread: logarithms of the decays and their running sum
+  constexpr int TOK = 128 / (GL_THREADS / 32);
+  const int ch = lane * 2, t0 = warp * TOK;
+  const bool in = ch < L.np;                         // (channels past the true number have no keys and decay by nothing)
+  float2 lg[TOK], sum = make_float2(0.f, 0.f);
   {
-    const float* zr = z + (size_t)(r0 + seg * 32) * ldz + h * L.np + ch;
+    const float* zr = z + (size_t)(r0 + t0) * ldz + h * L.np + ch;
 #pragma unroll
-    for (int t = 0; t < 32; ++t) lg[t] = ch < L.n && seg * 32 + t < valid ? zr[(size_t)t * ldz] : 0.f;
-    const float bias = ch < L.n ? L.w0[h * L.np + ch] : 0.f;
+    for (int t = 0; t < TOK; ++t)
+      lg[t] = in && t0 + t < valid ? *reinterpret_cast<const float2*>(zr + (size_t)t * ldz) : make_float2(0.f, 0.f);
+    const float2 bias = in ? *reinterpret_cast<const float2*>(L.w0 + h * L.np + ch) : make_float2(0.f, 0.f);
+    auto log_decay = [&](float x) { return -L.decay_root * (fmaxf(-x, 0.f) + log1pf(expf(-fabsf(x)))); };
 #pragma unroll
-    for (int t = 0; t < 32; ++t) {
-      const float x = lg[t] + bias, d = -L.decay_root * (fmaxf(-x, 0.f) + log1pf(expf(-fabsf(x))));
-      sum += ch < L.n && seg * 32 + t < valid ? d : 0.f;
+    for (int t = 0; t < TOK; ++t) {
+      if (t0 + t < valid) {
+        if (ch < L.n) sum.x += log_decay(lg[t].x + bias.x);
+        if (ch + 1 < L.n) sum.y += log_decay(lg[t].y + bias.y);
+      }
       lg[t] = sum;
     }
   }
-  s_sum[seg * 64 + ch] = sum;
+  s_sum[warp * 32 + lane] = sum;
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  float base = 0.f, all = 0.f;
+  float2 base = make_float2(0.f, 0.f), all = base;
 #pragma unroll
-  for (int s = 0; s < 4; ++s) {
-    if (s == seg) base = all;
-    all += s_sum[s * 64 + ch];
+  for (int s = 0; s < GL_THREADS / 32; ++s) {
+    if (s == warp) base = all;
+    all.x += s_sum[s * 32 + lane].x;
+    all.y += s_sum[s * 32 + lane].y;
   }
   {
-    const __nv_bfloat16* kr = proj + (size_t)(r0 + seg * 32) * ld + L.off_kk + h * L.np + ch;
-    float* lr = logs + (size_t)(r0 + seg * 32) * ldz + h * L.np + ch;
+    const __nv_bfloat16* kr = proj + (size_t)(r0 + t0) * ld + L.off_kk + h * L.np + ch;
+    float* lr = logs + (size_t)(r0 + t0) * ldz + h * L.np + ch;
 #pragma unroll
-    for (int t = 0; t < 32; ++t) {
-      const int row = seg * 32 + t;
-      float k = 0.f;
-      if (ch < L.n && row < valid) {
-        const float l = base + lg[t];
-        lr[(size_t)t * ldz] = l;
-        k = __bfloat162float(kr[(size_t)t * ld]) * expf(all - l);
+    for (int t = 0; t < TOK; ++t) {
+      float2 k = make_float2(0.f, 0.f);
+      if (in && t0 + t < valid) {
+        const float2 l = make_float2(base.x + lg[t].x, base.y + lg[t].y);
+        *reinterpret_cast<float2*>(lr + (size_t)t * ldz) = l;
+        k = load_pair(kr + (size_t)t * ld);
+        k.x *= expf(all.x - l.x);
+        k.y *= expf(all.y - l.y);
       }
-      put_split(sK, sK + GL_SUB, row, ch, k);
+      put_split(sK, sK + GL_SUB, t0 + t, ch, k.x, k.y);
     }
   }
   fence_proxy_async_smem();
   bool ok = (smem_u32(smem) & 1023u) == 0 && mbar_wait(b_v, 0);
-  const int strong = __syncthreads_or(all < -GL_LIMIT);
+  const int strong = __syncthreads_or(fminf(all.x, all.y) < -GL_LIMIT);
   ok = __syncthreads_and(ok);
   if (threadIdx.x == 0) flags[slot] = strong;
   const uint32_t tm = *tmem_slot;
@@ -238,22 +249,27 @@ gla_outputs_kernel(const __grid_constant__ CUtensorMap tmV, const __grid_constan
   }
   const float* last = logs + (size_t)(r0 + valid - 1) * ldz + h * L.np;
   {
-    const int ch = threadIdx.x & 63, seg = threadIdx.x >> 6;
-    const bool in = ch < L.n;
-    const float mid = in ? 0.5f * last[ch] : 0.f;
-    const __nv_bfloat16* pr = proj + (size_t)(r0 + seg * 32) * ld + h * L.np + ch;
-    const float* lr = logs + (size_t)(r0 + seg * 32) * ldz + h * L.np + ch;
+    constexpr int TOK = 128 / (GL_THREADS / 32);
+    const int ch = lane * 2, t0 = warp * TOK;
+    const bool in = ch < L.np;
+    const float2 end = in ? *reinterpret_cast<const float2*>(last + ch) : make_float2(0.f, 0.f);
+    const __nv_bfloat16* pr = proj + (size_t)(r0 + t0) * ld + h * L.np + ch;
+    const float* lr = logs + (size_t)(r0 + t0) * ldz + h * L.np + ch;
 #pragma unroll 8
-    for (int t = 0; t < 32; ++t) {
-      const int i = seg * 32 + t;
-      float q = 0.f, k = 0.f;
-      if (in && i < valid) {
-        const float l = lr[(size_t)t * ldz] - mid;
-        q = __bfloat162float(pr[(size_t)t * ld + L.off_q]) * expf(l);
-        k = __bfloat162float(pr[(size_t)t * ld + L.off_kk]) * expf(-l);
+    for (int t = 0; t < TOK; ++t) {
+      float2 q = make_float2(0.f, 0.f), k = q;
+      if (in && t0 + t < valid) {
+        const float2 l = *reinterpret_cast<const float2*>(lr + (size_t)t * ldz);
+        const float x = l.x - 0.5f * end.x, y = l.y - 0.5f * end.y;
+        q = load_pair(pr + (size_t)t * ld + L.off_q);
+        k = load_pair(pr + (size_t)t * ld + L.off_kk);
+        q.x *= expf(x);
+        q.y *= expf(y);
+        k.x *= expf(-x);
+        k.y *= expf(-y);
       }
-      put_split(sQ, sQ + GL_SUB, i, ch, q);
-      put_split(sK, sK + GL_SUB, i, ch, k);
+      put_split(sQ, sQ + GL_SUB, t0 + t, ch, q.x, q.y);
+      put_split(sK, sK + GL_SUB, t0 + t, ch, k.x, k.y);
     }
   }
   {

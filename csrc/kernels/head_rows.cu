@@ -55,75 +55,142 @@ __device__ __forceinline__ T* pool_row(const BbHyLayer& L, bool key, PoolPlace a
   return base + (((size_t)at.blk * L.hk + head) * L.pool_rows + at.off) * (key ? L.dkp : L.dvp);
 }
 
-// (u, v) of neighbouring channels turned by the row's angles; c: channel of f[0].
-__device__ __forceinline__ void turn_pairs(float (&f)[8], const float* ct, const float* st, int c, int rot) {
+// Angles of the four pairs from channel c on (pairs past the rotated part stay where they are).
+__device__ __forceinline__ void load_angles(const float* ct, const float* st, int c, int rot, float (&co)[4], float (&si)[4]) {
+  const int i = c >> 1;
+  if (c + 8 <= rot && (rot & 7) == 0) {
+    const float4 a = *reinterpret_cast<const float4*>(ct + i), b = *reinterpret_cast<const float4*>(st + i);
+    co[0] = a.x; co[1] = a.y; co[2] = a.z; co[3] = a.w;
+    si[0] = b.x; si[1] = b.y; si[2] = b.z; si[3] = b.w;
+  } else {
 #pragma unroll
-  for (int j = 0; j < 4; ++j) {
-    const int i = (c >> 1) + j;
-    if (2 * i < rot) {
-      const float co = ct[i], si = st[i], u = f[2 * j], v = f[2 * j + 1];
-      f[2 * j] = fmaf(u, co, -v * si);
-      f[2 * j + 1] = fmaf(v, co, u * si);
+    for (int j = 0; j < 4; ++j) {
+      const bool in = 2 * (i + j) < rot;
+      co[j] = in ? ct[i + j] : 1.f;
+      si[j] = in ? st[i + j] : 0.f;
     }
   }
 }
+// (u, v) of neighbouring channels turned by them
+__device__ __forceinline__ void turn_pairs(float (&f)[8], const float (&co)[4], const float (&si)[4]) {
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const float u = f[2 * j], v = f[2 * j + 1];
+    f[2 * j] = fmaf(u, co[j], -v * si[j]);
+    f[2 * j + 1] = fmaf(v, co[j], u * si[j]);
+  }
+}
 
-// `lanes` threads (a power of two up to a warp) share a head.
+// A single token that ends a block: the block's means (the row's keys and values are written; every thread comes here).
+template <typename T>
+__device__ __forceinline__ void pool_single(const BbHyLayer& L, const int* bt, int bs, int pos) {
+  __syncthreads();
+  const PoolPlace at = pool_place(L, bt, pos, bs);
+  for (int v = threadIdx.x; v < L.hk * (L.dkp + L.dvp) / 8; v += blockDim.x) {
+    float m[8];
+    bool key;
+    int head, col;
+    pool_vector<T>(L, bt, bs, pos / L.pool, v, m, key, head, col);
+    store8(pool_row<T>(L, key, at, head) + col, m);
+  }
+}
+
+struct HeadArgs {
+  const int *pos, *row_seq, *tables;
+  int ld, max_blocks, bs, rows, n_pre, hq, hk, off_k, lanes;
+  float eps;
+};
+// A head of a row: queries, then keys, then values.
+template <typename T>
+struct HeadOf {
+  int part, h, size, rot, src;       // src: its first column in the projection
+  const float *gain, *ct, *st;
+  __device__ HeadOf(const BbHyLayer& L, const HeadArgs& a, int u) {
+    part = u < a.hq ? 0 : (u < a.hq + a.hk ? 1 : 2);
+    h = part == 0 ? u : (part == 1 ? u - a.hq : u - a.hq - a.hk);
+    size = part == 2 ? L.dvp : L.dkp;
+    src = (part == 0 ? L.off_q : (part == 1 ? a.off_k : L.off_v)) + h * size;
+    gain = part == 0 ? L.q_norm : (part == 1 ? L.k_norm : nullptr);
+    ct = part == 2 ? L.vcos_t : L.cos_t;
+    st = part == 2 ? L.vsin_t : L.sin_t;
+    rot = !ct ? 0 : (part == 2 ? L.dv : L.rot);
+  }
+  __device__ T* page(const BbHyLayer& L, const HeadArgs& a, int blk, int pos) const {
+    return static_cast<T*>(part == 1 ? L.kc : L.vc) + (((size_t)blk * L.hk + h) * a.bs + pos % a.bs) * size;
+  }
+};
+
+// Rows of prompt portions: `lanes` threads (a power of two up to a warp) share a head of one row and have a vector of it
+// each; rows and heads are one list, so that no warp waits for another.
+template <typename T>
+__global__ void __launch_bounds__(HR_THREADS, sizeof(T) == 2 ? 6 : 4)
+hy_heads_kernel(const __grid_constant__ BbHyLayer L, T* proj, const __grid_constant__ HeadArgs a, int heads) {
+  const int lane = threadIdx.x % a.lanes, unit = blockIdx.x * (HR_THREADS / a.lanes) + threadIdx.x / a.lanes, r = unit / heads;
+  const HeadOf<T> x(L, a, unit - r * heads);
+  const bool live = r < a.rows && lane * 8 < x.size;
+  T* src = proj + (size_t)r * a.ld + x.src + lane * 8;
+  float f[8] = {}, co[4], si[4], ss = 0.f;
+  T* dst = src;
+  if (live) {
+    load8(src, f);
+    const int pos = a.pos[r];
+    load_angles(x.ct + (size_t)pos * (x.rot >> 1), x.st + (size_t)pos * (x.rot >> 1), lane * 8, x.rot, co, si);
+    if (x.part > 0 && L.kc)
+      dst = x.page(L, a, a.tables[(size_t)a.row_seq[r] * a.max_blocks + pos / a.bs], pos) + lane * 8;
+  }
+  if (L.q_norm) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss = fmaf(f[j], f[j], ss);
+    for (int o = 1; o < a.lanes; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  }
+  if (!live) return;
+  if (x.gain) {
+    float g[8];
+    load8(x.gain + lane * 8, g);
+    const float rstd = 1.f / sqrtf(ss / (float)L.dk + a.eps);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) f[j] *= rstd * g[j];
+  }
+  turn_pairs(f, co, si);
+  store8(dst, f);
+}
+
+// The same with a row to a block: single tokens, and heads wider than a warp has vectors for.
 template <typename T>
 __global__ void __launch_bounds__(HR_THREADS)
-hy_heads_kernel(const __grid_constant__ BbHyLayer L, T* proj, int ld, const int* __restrict__ pos_,
-                const int* __restrict__ row_seq, const int* __restrict__ tables, int max_blocks, int bs, int n_pre, int hq,
-                int hk, int off_k, int lanes, float eps) {
-  const int r = blockIdx.x, lane = threadIdx.x % lanes, group = threadIdx.x / lanes, groups = blockDim.x / lanes;
-  T* row = proj + (size_t)r * ld;
-  const int pos = pos_[r];
+hy_head_rows_kernel(const __grid_constant__ BbHyLayer L, T* proj, const __grid_constant__ HeadArgs a, int r0) {
+  const int r = r0 + blockIdx.x, lane = threadIdx.x % a.lanes, group = threadIdx.x / a.lanes, groups = blockDim.x / a.lanes;
   const bool paged = L.kc != nullptr;
-  const int* bt = paged ? tables + (size_t)row_seq[r] * max_blocks : nullptr;
-  const int blk = paged ? bt[pos / bs] : 0, off = pos % bs;
-  const int heads = hq + hk + (paged ? hk : 0);
+  const int pos = a.pos[r], heads = a.hq + a.hk + (paged ? a.hk : 0);
+  const int* bt = paged ? a.tables + (size_t)a.row_seq[r] * a.max_blocks : nullptr;
   for (int h0 = 0; h0 < heads; h0 += groups) {
     const bool live = h0 + group < heads;
-    const int u = live ? h0 + group : 0, part = u < hq ? 0 : (u < hq + hk ? 1 : 2);
-    const int h = part == 0 ? u : (part == 1 ? u - hq : u - hq - hk);
-    const int size = part == 2 ? L.dvp : L.dkp, vecs = size / 8;
-    T* src = row + (part == 0 ? L.off_q : (part == 1 ? off_k : L.off_v)) + h * size;
-    T* dst = part == 0 || !paged
-                 ? src
-                 : static_cast<T*>(part == 1 ? L.kc : L.vc) + (((size_t)blk * L.hk + h) * bs + off) * size;
-    const float* gain = part == 0 ? L.q_norm : (part == 1 ? L.k_norm : nullptr);
-    const float *ct = part == 2 ? L.vcos_t : L.cos_t, *st = part == 2 ? L.vsin_t : L.sin_t;
-    const int rot = !ct ? 0 : (part == 2 ? L.dv : L.rot);
+    const HeadOf<T> x(L, a, live ? h0 + group : 0);
+    const int vecs = x.size / 8;
+    T* src = proj + (size_t)r * a.ld + x.src;
+    T* dst = x.part > 0 && paged ? x.page(L, a, bt[pos / a.bs], pos) : src;
     float f[8], ss = 0.f;
-    for (int v = lane; live && v < vecs; v += lanes) {
+    for (int v = lane; live && v < vecs; v += a.lanes) {
       load8(src + v * 8, f);
 #pragma unroll
       for (int j = 0; j < 8; ++j) ss = fmaf(f[j], f[j], ss);
     }
-    for (int o = 1; o < lanes; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    const float rstd = gain ? 1.f / sqrtf(ss / (float)L.dk + eps) : 1.f;
-    for (int v = lane; live && v < vecs; v += lanes) {
-      if (vecs > lanes) load8(src + v * 8, f);
-      if (gain) {
-        float g[8];
-        load8(gain + v * 8, g);
+    for (int o = 1; o < a.lanes; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float rstd = x.gain ? 1.f / sqrtf(ss / (float)L.dk + a.eps) : 1.f;
+    for (int v = lane; live && v < vecs; v += a.lanes) {
+      float g[8], co[4], si[4];
+      load8(src + v * 8, f);
+      if (x.gain) {
+        load8(x.gain + v * 8, g);
 #pragma unroll
         for (int j = 0; j < 8; ++j) f[j] *= rstd * g[j];
       }
-      if (rot) turn_pairs(f, ct + (size_t)pos * (rot >> 1), st + (size_t)pos * (rot >> 1), v * 8, rot);
+      load_angles(x.ct + (size_t)pos * (x.rot >> 1), x.st + (size_t)pos * (x.rot >> 1), v * 8, x.rot, co, si);
+      turn_pairs(f, co, si);
       store8(dst + v * 8, f);
     }
   }
-  if (r >= n_pre && L.pool && (pos + 1) % L.pool == 0) {
-    __syncthreads();
-    const PoolPlace at = pool_place(L, bt, pos, bs);
-    for (int v = threadIdx.x; v < L.hk * (L.dkp + L.dvp) / 8; v += blockDim.x) {
-      float m[8];
-      bool key;
-      int head, col;
-      pool_vector<T>(L, bt, bs, pos / L.pool, v, m, key, head, col);
-      store8(pool_row<T>(L, key, at, head) + col, m);
-    }
-  }
+  if (r >= a.n_pre && L.pool && (pos + 1) % L.pool == 0) pool_single<T>(L, bt, a.bs, pos);
 }
 
 // blockIdx.x: block of the sequence blockIdx.y.  seen (may be null): [rows][ld] keys | values of all heads, block b of
@@ -161,13 +228,18 @@ hy_pool_kernel(const __grid_constant__ BbHyLayer L, const int* __restrict__ tabl
 template <typename T>
 static int launch_heads(const BbHyLayer& L, const BbHyWork& w, const BbHyBatch& b, int bs, int rows, int hq, int hk, int off_k,
                         float eps, cudaStream_t s) {
-  const int widest = (L.kc && L.dvp > L.dkp ? L.dvp : L.dkp) / 8;
+  const int widest = (L.kc && L.dvp > L.dkp ? L.dvp : L.dkp) / 8, heads = hq + hk + (L.kc ? hk : 0);
   int lanes = 1;
   while (lanes < widest && lanes < 32) lanes <<= 1;
-  int threads = (hq + hk + (L.kc ? hk : 0)) * lanes;
-  threads = threads > HR_THREADS ? HR_THREADS : (threads + 31) & ~31;
-  hy_heads_kernel<T><<<rows, threads, 0, s>>>(L, static_cast<T*>(w.proj), w.ld_proj, b.pos, b.row_seq, b.tables, b.max_blocks,
-                                              bs, b.n_pre, hq, hk, off_k, lanes, eps);
+  const int listed = widest <= lanes ? b.n_pre : 0;      // rows that go as a list of heads
+  const HeadArgs a{b.pos, b.row_seq, b.tables, w.ld_proj, b.max_blocks, bs, listed, b.n_pre, hq, hk, off_k, lanes, eps};
+  T* proj = static_cast<T*>(w.proj);
+  if (listed > 0)
+    hy_heads_kernel<T><<<(int)(((long)listed * heads * lanes + HR_THREADS - 1) / HR_THREADS), HR_THREADS, 0, s>>>(L, proj, a, heads);
+  if (rows > listed) {
+    const int threads = heads * lanes < HR_THREADS ? (heads * lanes + 31) & ~31 : HR_THREADS;
+    hy_head_rows_kernel<T><<<rows - listed, threads, 0, s>>>(L, proj, a, listed);
+  }
   return (int)cudaGetLastError();
 }
 
