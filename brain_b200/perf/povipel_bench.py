@@ -67,7 +67,13 @@ def kernels(eng, entries, phase, timer, peaks):
 
     def gemm(name, like, a, lda, lin, y, ldy, rows=n, mode=0):
         us = t("bb_gemm_bf16", a, P(lin.w), y, P(None), rows, lin.n, lin.k, lda, lin.k, ldy, 0, 0, mode, C.c_float(1.0), 0, 0)
-        row(name, us, like, (rows * lin.k * 2 + lin.n * lin.k * 2 + rows * lin.n * (2, 4)[mode]) / 1e9, 2e-12 * rows * lin.n * lin.k)
+        row(name, us, like, (rows * lin.k * 2 + lin.n * lin.k * 2 + rows * lin.n * (2, 4, 8, 2)[mode]) / 1e9, 2e-12 * rows * lin.n * lin.k)
+
+    def result(name, a, lda, lin, which):           # a sublayer's result; small steps add it up in fp32
+        if n <= 256:
+            gemm(name, "output projections", a, lda, lin, P(getattr(sc, which + "32").data_ptr()), d, mode=2)
+        else:
+            gemm(name, "output projections", a, lda, lin, at(which), d)
 
     L = eng.layer_list
     first, both, ret = L[0], L[2 if len(L) > 2 else 0], L[1]
@@ -86,12 +92,11 @@ def kernels(eng, entries, phase, timer, peaks):
         row("token shift", t("bb_hy_shift", cfg, lb, w, bb), "post (glu)", n * d * 4 / 1e9)
     gemm("both: input projections", "input projections", at("h"), d, both.inp, at("proj"), ld["proj"])
     gemm("retention: input projections", "input projections", at("h"), d, ret.inp, at("proj"), ld["proj"])
-    gemm("attention: output projection", "output projections", at("cat"), ld["cat"], both.out, at("ya"), d)
-    gemm("gated linear: output projection", "output projections", at("cat", side.off_cat), ld["cat"], side.out, at("yb"), d)
-    gemm("retention: output projection", "output projections", at("cat"), ld["cat"], ret.out, at("ya"), d)
-    gemm("dense: up", "input projections", at("h"), d, first.up, at("proj"), ld["proj"])
-    row("dense: gelu", t("bb_hy_gelu", cfg, C.byref(first), w, n), "post (glu)", n * first.up.n * 4 / 1e9)
-    gemm("dense: down", "output projections", at("cat"), ld["cat"], first.down, at("ya"), d)
+    result("attention: output projection", at("cat"), ld["cat"], both.out, "ya")
+    result("gated linear: output projection", at("cat", side.off_cat), ld["cat"], side.out, "yb")
+    result("retention: output projection", at("cat"), ld["cat"], ret.out, "ya")
+    gemm("dense: up, gelu", "input projections", at("h"), d, first.up, at("cat"), ld["cat"], mode=3)
+    result("dense: down", at("cat"), ld["cat"], first.down, "ya")
     eng._run(sc, b)
     # experts
     if not few:

@@ -65,6 +65,7 @@ class _Scratch:
         self.x = z(eng.cfg.n_layers + 1 if traits.depth_average else eng.cfg.streams, rows, eng.dp, dtype=f32)
         self.h, self.h2 = z(rows, eng.dp), z(rows if traits.two_norms or traits.token_shift and portions else 1, eng.dp)
         self.ya, self.yb = (z(rows if traits.streams else 1, eng.dp) for _ in range(2))
+        self.ya32, self.yb32 = (z(min(rows, 256) if traits.streams else 1, eng.dp, dtype=f32) for _ in range(2))
         self.pk = z(max(exp, 1) if portions else 1, m["pk"])
         self.proj, self.cat = z(rows, m["proj"]), z(rows, m["cat"])
         self.xbc, self.dt, self.y = z(rows, m["xbc"]), z(rows, m["dt"], dtype=f32), z(rows, m["y"])
@@ -108,7 +109,7 @@ class _Scratch:
         w = self.work = hn.Work()
         for n in ("x", "h", "proj", "cat", "xbc", "dt", "y", "v_first", "part_o", "part_ml", "seg", "hn", "logits", "h2", "q",
                   "qa", "ol", "aux", "ckv", "kvx", "f32", "part32", "ex_in", "ex_gu", "ex_act", "ex_out", "pair_expert", "pair_row",
-                  "pair_w", "ex_count", "ex_tile", "ya", "yb", "pk", "chunks",
+                  "pair_w", "ex_count", "ex_tile", "ya", "yb", "ya32", "yb32", "pk", "chunks",
                   "chunk_flags"):
             setattr(w, n, _ptr(getattr(self, n)))
         w.chunk_floats, w.chunk_marks = self.chunks.numel(), self.chunk_flags.numel()

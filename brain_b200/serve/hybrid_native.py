@@ -80,7 +80,7 @@ class Work(C.Structure):
                [(n, P) for n in ("ex_in", "ex_gu", "ex_act", "ex_out", "pair_expert", "pair_row", "pair_w", "ex_count",
                                  "ex_tile")] + \
                [(n, I) for n in ("ld_f32", "ld_gu", "ld_act", "moe_rows")] + \
-               [("ya", P), ("yb", P), ("pk", P), ("ld_pk", I), ("pk_rows", I),
+               [("ya", P), ("yb", P), ("pk", P), ("ya32", P), ("yb32", P), ("ld_pk", I), ("pk_rows", I),
                 ("chunks", P), ("chunk_flags", P), ("chunk_floats", C.c_long), ("chunk_marks", C.c_long)]
 
 

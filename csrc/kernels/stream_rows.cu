@@ -4,7 +4,7 @@
 //                and the next one's input is the layer norm of sum_s in[s] x_s.  One pass over the streams.  Single tokens
 //                are also shifted towards the token before them, which their slot holds
 //   hy_shift     the same shift for the rows of prompt portions; the slot gets the portion's last input
-//   hy_gelu      gelu of a feed-forward's up projection
+//   hy_gelu      gelu of a feed-forward's up projection (fp32)
 //   hy_cap       logits <- cap tanh(logits / cap)
 #include "../common/host.hpp"
 #include "../common/rows.cuh"
@@ -22,6 +22,8 @@ struct StreamArgs {
   float emb_scale;
   int vocab;
   const void *ya, *yb;             // results; yb not null: both normed, times their gains
+  int y32;                         // results are fp32
+  float *zero_a, *zero_b;          // rows that the next results are added into (null: none)
   const float *gain_a, *gain_b;
   const void* ex_out;              // a token's experts (top = 0: none)
   const int* pair_row;
@@ -63,14 +65,17 @@ hy_streams_kernel(const __grid_constant__ StreamArgs a, T* __restrict__ h) {
       s_in[i] = i < a.s ? (a.to ? a.to[i] : 1.f) : 0.f;
     }
   }
-  const T *ya = static_cast<const T*>(a.ya) + (size_t)r * a.dp, *yb = static_cast<const T*>(a.yb) + (size_t)r * a.dp;
+  auto result = [&](const void* y, int i, float (&f)[8]) {
+    if (sizeof(T) == 2 && a.y32) load8(static_cast<const float*>(y) + (size_t)r * a.dp + i, f);
+    else load8(static_cast<const T*>(y) + (size_t)r * a.dp + i, f);
+  };
   float fa = 0.f, fb = 0.f;
   if (a.yb) {
     float ssa = 0.f, ssb = 0.f;
     for (int i = threadIdx.x * 8; i < a.dp; i += step) {
       float f[8], g[8];
-      load8(ya + i, f);
-      load8(yb + i, g);
+      result(a.ya, i, f);
+      result(a.yb, i, g);
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         ssa = fmaf(f[j], f[j], ssa);
@@ -117,8 +122,8 @@ hy_streams_kernel(const __grid_constant__ StreamArgs a, T* __restrict__ h) {
       }
       if (a.yb) {
         float f[8], g[8], ga[8], gb[8];
-        load8(ya + i, f);
-        load8(yb + i, g);
+        result(a.ya, i, f);
+        result(a.yb, i, g);
         load8(a.gain_a + i, ga);
         load8(a.gain_b + i, gb);
 #pragma unroll
@@ -133,7 +138,7 @@ hy_streams_kernel(const __grid_constant__ StreamArgs a, T* __restrict__ h) {
           for (int j = 0; j < 8; ++j) y[j] = fmaf(w, g[j], y[j]);
         }
       } else {
-        load8(ya + i, y);
+        result(a.ya, i, y);
       }
 #pragma unroll
       for (int t = 0; t < S; ++t) {
@@ -159,6 +164,9 @@ hy_streams_kernel(const __grid_constant__ StreamArgs a, T* __restrict__ h) {
 #pragma unroll
     for (int j = 0; j < 8; ++j) sum += u[j];
     store8(u_row + i, u);
+    const float none[8] = {};
+    if (a.zero_a) store8(a.zero_a + (size_t)r * a.dp + i, none);
+    if (a.zero_b) store8(a.zero_b + (size_t)r * a.dp + i, none);
   }
   const float mean = block_sum(sum, buf[2]) / (float)a.d;
   float ss = 0.f;
@@ -300,13 +308,18 @@ BB_API int bb_hy_streams(const BbHyCfg* c, const BbHyLayer* before, int fq, cons
       a.pair_w = before->weigh_input ? nullptr : w->pair_w;
       a.top = before->top;
     } else {
-      a.ya = w->ya;
+      a.y32 = hy_sums_y(*c, b->n);
+      a.ya = a.y32 ? w->ya32 : w->ya;
       if (fq == 0 && before->beside) {
-        a.yb = w->yb;
+        a.yb = a.y32 ? w->yb32 : w->yb;
         a.gain_a = before->out_gain;
         a.gain_b = before->beside->out_gain;
       }
     }
+  }
+  if (next && hy_sums_y(*c, b->n) && (tq == 0 || next->n_experts == 0)) {
+    a.zero_a = w->ya32;
+    a.zero_b = tq == 0 && next->beside ? w->yb32 : nullptr;
   }
   a.to = next ? next->hc[tq] : nullptr;
   a.w = next ? (tq ? next->norm2 : next->norm) : c->final_norm;
@@ -347,16 +360,15 @@ BB_API int bb_hy_shift(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, 
   return (int)cudaGetLastError();
 }
 
-// gelu of the layer's up projection (in the first columns of w->proj) -> the first columns of w->cat.
+// gelu of the layer's up projection (in the first columns of w->proj) -> the first columns of w->cat; the bf16 step has it in
+// the projection's epilogue.
 BB_API int bb_hy_gelu(const BbHyCfg* c, const BbHyLayer* L, const BbHyWork* w, int n, void* stream) {
   if (n <= 0) return BB_OK;
   cudaStream_t s = (cudaStream_t)stream;
   const dim3 grid(n, (L->up.n / 8 + ST_THREADS - 1) / ST_THREADS);
-#define BB_GELU(T) \
-  hy_gelu_kernel<T><<<grid, ST_THREADS, 0, s>>>(static_cast<const T*>(w->proj), w->ld_proj, static_cast<T*>(w->cat), w->ld_cat, L->up.n)
-  if (c->dtype) BB_GELU(float);
-  else BB_GELU(__nv_bfloat16);
-#undef BB_GELU
+  if (!c->dtype) return BB_EARG;
+  hy_gelu_kernel<float><<<grid, ST_THREADS, 0, s>>>(static_cast<const float*>(w->proj), w->ld_proj, static_cast<float*>(w->cat),
+                                                    w->ld_cat, L->up.n);
   return (int)cudaGetLastError();
 }
 

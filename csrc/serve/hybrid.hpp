@@ -180,15 +180,20 @@ struct BbHyWork {
   float* pair_w;
   int *ex_count, *ex_tile;                 // [experts], [2][moe_rows / 128]
   int ld_f32, ld_gu, ld_act, moe_rows;
-  // residual streams: results of a sublayer [rows, dp] (two of mixers side by side); pooled keys and values that prompt
+  // residual streams: results of a sublayer [rows, dp] (two of mixers side by side), in small bf16 steps (hy_sums_y) added
+  // up in fp32 where hy_streams has left zeros; pooled keys and values that prompt
   // portions see, [pk_rows, ld_pk], of sequence s from ctx_row0[s] / pool on
   void *ya, *yb, *pk;
+  float *ya32, *yb32;
   int ld_pk, pk_rows;
   // chunks of gated linear attention: [n_pre / 128 + ns_pre][heads][n][p] and marks [..][heads]
   float* chunks;
   int* chunk_flags;
   long chunk_floats, chunk_marks;
 };
+
+// Steps of few rows whose projections into the streams are cut along their inner extent, to fill the machine.
+static inline bool hy_sums_y(const BbHyCfg& c, int rows) { return !c.dtype && rows <= 256; }
 
 // Rows and pitch of a latent attention layer's queries: through their own latent, or straight from the input.
 static inline void* hy_latent_queries(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, int* ld) {

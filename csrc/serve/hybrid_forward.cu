@@ -423,6 +423,19 @@ int forward_start(const BbHyCfg& c, const BbHyWork& w, const BbHyBatch& b, float
   return bb_hy_start(&c, c.n_layers, &w, &b, 0, nullptr, s);
 }
 
+// A sublayer's result: y = x W^T, or in small steps added into zeros.
+int project_y(const BbHyCfg& c, const BbHyLin& L, const void* x, int ldx, void* y, float* y32, int rows, void* s) {
+  return hy_sums_y(c, rows) ? project_f32(c, L, x, ldx, y32, c.dp, rows, 1.f, 1, s) : project(c, L, x, ldx, y, c.dp, rows, s);
+}
+
+// gelu(x W^T)
+int project_gelu(const BbHyCfg& c, const BbHyLayer& L, const BbHyWork& w, int rows, void* s) {
+  if (!c.dtype)
+    return bb_gemm_bf16(w.h, L.up.w, w.cat, nullptr, rows, L.up.n, L.up.k, c.dp, L.up.k, w.ld_cat, 0, 0, 3, 1.f, 0, 0, s);
+  BB_TRY(project(c, L.up, w.h, c.dp, w.proj, w.ld_proj, rows, s));
+  return bb_hy_gelu(&c, &L, &w, rows, s);
+}
+
 // Layers with several residual streams: mixer, then feed-forward, hy_streams before each and behind the last.  In small
 // steps mixers side by side run on two streams of the device.
 int forward_streams(const BbHyCfg& c, const BbHyWork& w, const BbHyBatch& b, float* trace, void* s) {
@@ -445,11 +458,11 @@ int forward_streams(const BbHyCfg& c, const BbHyWork& w, const BbHyBatch& b, flo
         BB_CUDA(cudaStreamWaitEvent(side->s, side->fork, 0));
       }
       BB_TRY(mixer(c, *L.beside, v, b, t));
-      BB_TRY(project(c, L.beside->out, v.cat, w.ld_cat, w.yb, c.dp, b.n, t));
+      BB_TRY(project_y(c, L.beside->out, v.cat, w.ld_cat, w.yb, w.yb32, b.n, t));
       if (side) BB_CUDA(cudaEventRecord(side->join, side->s));
     }
     BB_TRY(mixer(c, L, w, b, s));
-    BB_TRY(project(c, L.out, w.cat, w.ld_cat, w.ya, c.dp, b.n, s));
+    BB_TRY(project_y(c, L.out, w.cat, w.ld_cat, w.ya, w.ya32, b.n, s));
     if (L.beside && side) BB_CUDA(cudaStreamWaitEvent(main, side->join, 0));
     before = &L;
     fq = 0;
@@ -460,9 +473,8 @@ int forward_streams(const BbHyCfg& c, const BbHyWork& w, const BbHyBatch& b, flo
         BB_TRY(route(c, L, w, b, s));
         BB_TRY(experts(c, L, w, b, s));
       } else {
-        BB_TRY(project(c, L.up, w.h, c.dp, w.proj, w.ld_proj, b.n, s));
-        BB_TRY(bb_hy_gelu(&c, &L, &w, b.n, s));
-        BB_TRY(project(c, L.down, w.cat, w.ld_cat, w.ya, c.dp, b.n, s));
+        BB_TRY(project_gelu(c, L, w, b.n, s));
+        BB_TRY(project_y(c, L.down, w.cat, w.ld_cat, w.ya, w.ya32, b.n, s));
       }
     }
   }
