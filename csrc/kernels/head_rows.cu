@@ -36,7 +36,7 @@ __device__ __forceinline__ void pool_vector(const BbHyLayer& L, const int* bt, i
 #pragma unroll
   for (int j = 0; j < 8; ++j) m[j] = 0.f;
   const int p0 = blk * L.pool;
-#pragma unroll 4
+#pragma unroll 8
   for (int t = 0; t < L.pool; ++t) {
     const int p = p0 + t;
     float f[8];
