@@ -1,5 +1,6 @@
 // Rows of heads between a projection and its mixer, fp32 arithmetic, bf16 or fp32 storage:
-//   hy_heads   per head: root-mean-square norm with one gain for all heads, rotation of neighbouring pairs; queries in
+//   hy_heads, hy_head_rows (portions as a list of heads; a row to a block)
+//              per head: root-mean-square norm with one gain for all heads, rotation of neighbouring pairs; queries in
 //              place, keys and (rotated) values into the sequence's page, or keys in place too where there are no pages.
 //              A single token that ends a block of the pooled cache also writes the block's means
 //   hy_pool    means of the blocks that end in prompt portions, and the means that their queries see as rows of one
